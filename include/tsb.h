@@ -382,6 +382,8 @@ TSB_API int32_t tsb_model_share(tsb_model* dst, int32_t dst_layer, const tsb_mod
  * right shapes and formats without a host copy; values are valid blocks with small scales). */
 TSB_API int32_t tsb_model_fill_synthetic(tsb_model* m, int32_t qtype, int32_t lm_head_qtype, uint64_t seed);
 TSB_API int64_t tsb_model_weight_bytes(const tsb_model* m);
+/* 1: the model's logit rows are f32 (every logits_out_host of its sessions then receives f32 values), 0: f16. */
+TSB_API int32_t tsb_model_logits_f32(const tsb_model* m);
 /* Routed feed-forward (the llama family's MoE layers: crates/runtime/src/families/llama/moe.rs:36-221, router
  * families/llama/router.rs:12-66).  tsb_model_set_moe, called before any tensor is uploaded, makes every layer's
  * feed-forward routed: n_experts experts of width moe_ffn, top_k per token (the config's dense `ffn` is then
@@ -396,6 +398,74 @@ TSB_API int32_t tsb_model_set_experts(tsb_model* m, int32_t layer, int32_t qtype
  * effective scale: logits[t, e] = sum over 64-column groups of fma(s, q.x, .) and fma(b, sum x, .), f32. */
 TSB_API int32_t tsb_router_logits(tsb_ctx* ctx, tsb_stream s, const void* q_u8, const void* scale_bf16, const void* bias_bf16,
                                   const void* x_f16, int32_t tokens, int32_t n_experts, int32_t d_model, float* logits_out);
+
+/* ------------------------------------------------------------ plain-weight decoders
+ * Decoders whose matrices are plain bfloat16 (or f32) and whose layers are put together from the mechanisms below; the
+ * reference has no counterpart.  One layer, in parallel form with one norm:
+ *     h = x * gain / sqrt(mean(x^2) + eps)                       one gain for all coordinates
+ *     x = x + mixer(shift(h)) + feed_forward(h)
+ *   shift (token_shift): h_t + (h_{t-1} - h_t) * mu, element by element; h_{-1} = 0
+ *   mixer: causal attention whose values are its keys, n_q_heads query heads over n_kv_heads key heads;
+ *     score = (q . k) * score_scale;  score_cap > 0: score = score_cap * tanh(score / score_cap);
+ *     log_bias: score -= r1[head] * ln(1 + r2[head] * distance);  window > 0: the last `window` positions only;
+ *     head_gate: each head's output times sigmoid of one number per head, projected from the mixer's input
+ *   feed_forward (ffn > 0): W_down(act(W_gate h) * (W_up h))
+ * then logits = W_head norm(x), through logit_cap * tanh(logits / logit_cap) when logit_cap > 0.
+ * Residual stream, norms, shift, scores, softmax and gates are f32 in both modes.  compute = TSB_BF16: matrices,
+ * activations and the key cache in bfloat16 with f32 accumulation; TSB_F32: everything in f32.
+ * The caches of such a model hold keys only, and per stream the last rows' h of every layer (a cursor can be moved back
+ * by max_rows rows, or to 0).  Verify passes are chains; tree rounds are refused with TSB_ERR_UNSUPPORTED. */
+enum { TSB_BF16 = 0, TSB_F32 = 1 };
+enum { TSB_ACT_GELU_TANH = 0, TSB_ACT_SILU = 1 };
+typedef struct tsb_plain_config {
+    int32_t n_layers, d_model, vocab, max_context, compute;
+    float norm_eps, logit_cap;
+} tsb_plain_config;
+typedef struct tsb_plain_layer {
+    int32_t n_q_heads, n_kv_heads, head_dim, window;
+    float score_scale, score_cap;
+    int32_t log_bias, head_gate, token_shift; /* 0 / 1 */
+    int32_t ffn, act;
+} tsb_plain_layer;
+enum {
+    TSB_P_EMBED = 0, TSB_P_HEAD, TSB_P_FINAL_NORM,                     /* layer ignored; [vocab, d], [vocab, d], [1] */
+    TSB_P_NORM, TSB_P_SHIFT,                                           /* [1], [d] */
+    TSB_P_Q, TSB_P_K, TSB_P_HEAD_GATE, TSB_P_R1, TSB_P_R2, TSB_P_O,    /* [H D, d], [G D, d], [H, d], [H], [H], [d, H D] */
+    TSB_P_FF_GATE, TSB_P_FF_UP, TSB_P_FF_DOWN                          /* [ffn, d], [ffn, d], [d, ffn] */
+};
+TSB_API int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const tsb_plain_layer* layers, tsb_model** out);
+/* Upload one tensor, rows x cols row-major (vectors: rows = 1); host_type says what the host data is (TSB_BF16 / TSB_F32). */
+TSB_API int32_t tsb_model_set_plain(tsb_model* m, int32_t layer, int32_t which, int32_t host_type, const void* host, int64_t rows, int64_t cols);
+/* Seeded random weights made on the device (benchmark set-up). */
+TSB_API int32_t tsb_model_fill_plain(tsb_model* m, uint64_t seed);
+
+/* The same mechanisms as operators.  `type` is TSB_BF16 or TSB_F32 and names the type of weights, activations and keys. */
+/* y[t, n] = sum_k W[n, k] x[t, k] in f32, through cap * tanh(y / cap) when cap > 0; add = 1: added to y instead.
+ * W: rows a multiple of 128, cols a multiple of 64 (pad with zeros); x: [x_rows, cols] with x_rows >= 32 allocated rows. */
+TSB_API int32_t tsb_plain_gemm(tsb_ctx* ctx, tsb_stream s, int32_t type, const void* w, int64_t rows, int64_t cols, const void* x, int32_t x_rows,
+                               int32_t tokens, float* y, int64_t y_stride, int32_t n_valid, float cap, int32_t add, void* workspace);
+/* The gate / up half of a feed-forward: W holds gate and up rows interleaved in groups of eight (eight gate rows, eight up
+ * rows, ...); a[t, p] = act(gate_p) * up_p in `type`, row stride a_stride. */
+TSB_API int32_t tsb_plain_gemm_pairs(tsb_ctx* ctx, tsb_stream s, int32_t type, const void* w, int64_t rows, int64_t cols, const void* x, int32_t x_rows,
+                                     int32_t tokens, void* a, int64_t a_stride, int32_t n_pairs, int32_t act, void* workspace);
+TSB_API size_t tsb_plain_gemm_workspace_bytes(const tsb_ctx* ctx); /* zeroed once by the caller */
+/* Norm and shift of the rows of a pass (f32 x [rows, d]): h_out and mix_out [rows, out_stride] in `type`; gain [1] and mu [d]
+ * f32 (mu NULL: no shift).  state: f32 [n_streams][ring][d], ring a power of two; every portion is at most ring - 1 rows. */
+TSB_API int32_t tsb_norm_shift_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, const float* x, int32_t d, const float* gain, float eps, const float* mu,
+                                    const tsb_row_desc* rows_dev, int32_t rows, float* state, int32_t n_streams, int32_t ring, void* mix_out,
+                                    void* h_out, int64_t out_stride);
+/* A key-only cache: tsb_kv_* take it (tsb_kv_write_rows / read_rows with host_v NULL).  head_dim is the stored size: a
+ * multiple of 4 (TSB_F32), or one of 32, 64, 96, 128, 192, 256 (TSB_BF16; pad smaller heads with zero columns). */
+TSB_API int32_t tsb_kv_create_keys(tsb_ctx* ctx, int32_t type, int32_t layers, int32_t kv_heads, int32_t head_dim, int32_t page_tokens,
+                                   int32_t num_pages, int32_t max_seqs, int32_t max_pages_per_seq, tsb_kv** out);
+/* Attention of rows over such a cache, keys of the rows themselves included (positions base + slot; a stream's rows are
+ * consecutive, slots 0, 1, ...).  group_rows lists the rows of every stream of the batch in order (host).  q and out are
+ * [rows, stride] in `type`; gate [rows, n_q_heads] f32 pre-activations or NULL; r1, r2 [n_q_heads] f32 or NULL. */
+TSB_API int32_t tsb_window_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, int32_t layer, const void* q, int64_t q_stride, void* out,
+                                     int64_t out_stride, const tsb_row_desc* rows_dev, const int32_t* group_rows, int32_t n_groups,
+                                     int32_t n_q_heads, float scale, float cap, const float* r1, const float* r2, const float* gate,
+                                     int32_t window, int32_t max_len, void* scratch);
+TSB_API size_t tsb_window_attention_scratch_bytes(const tsb_ctx* ctx); /* zeroed once by the caller */
 
 /* ------------------------------------------------------------------ resident weight file
  * The leading index region of the reference's resident weight file: 24-byte header, 72-byte entries, string
@@ -459,6 +529,11 @@ TSB_API int32_t tsb_session_set_comm(tsb_session* s, tsb_comm* c);
  * (crates/runtime/src/real_forward_traits.rs:6-60). */
 TSB_API int32_t tsb_session_create(tsb_ctx* ctx, const tsb_model* target, const tsb_model* draft, int32_t n_streams,
                                    int32_t max_rows, int32_t page_tokens, tsb_session** out);
+/* The same with the target's page pool sized by hand: the streams share pages for pool_tokens positions (0: every
+ * stream can reach the context window), and one step (tsb_session_step) may carry up to step_rows rows (0: n_streams *
+ * max_rows; only models whose passes may be ragged take more). */
+TSB_API int32_t tsb_session_create_pool(tsb_ctx* ctx, const tsb_model* target, const tsb_model* draft, int32_t n_streams, int32_t max_rows,
+                                        int32_t page_tokens, int64_t pool_tokens, int32_t step_rows, tsb_session** out);
 TSB_API void tsb_session_destroy(tsb_session* s);
 TSB_API tsb_kv* tsb_session_kv(tsb_session* s, int32_t which_model /* 0 target, 1 draft */);
 /* Number of kernel launches / CUDA-graph launches issued so far by this session's ctx is tsb_launch_count. */
@@ -588,6 +663,36 @@ TSB_API int32_t tsb_spec_run(tsb_session* s, int32_t stream, const int32_t* prom
  * one must reproduce token for token at temperature 0. */
 TSB_API int32_t tsb_sequential_run(tsb_session* s, int32_t stream, const int32_t* prompt, int32_t n_prompt,
                                    const tsb_run_config* cfg, int32_t* out_tokens, int32_t* out_emitted, tsb_run_result* res);
+
+/* ---- mixed steps and continuous batching
+ * One step over unequal portions of several streams: entry i feeds its next n_tokens tokens (prompt portion or decoded
+ * token) at the stream's cursor; `tokens` holds them entry after entry.  want holds, entry after entry, n_want ascending
+ * places inside the entry's tokens whose logits are asked for; they arrive in logits_out_host in that order, rows of
+ * vocab values (f32 or f16: tsb_model_logits_f32).  A stream appears at most once.  Pages are reserved before anything
+ * runs: a step that does not fit is refused with TSB_ERR_OOM and changes no cursor.  Plain-weight models run the entries as
+ * one batch (passes of up to step_rows rows); block-quantised models run them stream by stream. */
+typedef struct tsb_step_entry {
+    int32_t stream, n_tokens, n_want;
+} tsb_step_entry;
+TSB_API int32_t tsb_session_step(tsb_session* s, const tsb_step_entry* entries, int32_t n_entries, const int32_t* tokens, const int32_t* want,
+                                 void* logits_out_host);
+/* Serve a list of requests by continuous batching: requests are admitted in order while a stream and the pages for
+ * prompt + budget are free, every step carries one token of each decoding stream and, in the rows left, portions of at
+ * most prefill_chunk tokens of the prompts; the rows that end a prompt or decode are sampled on the device together, and
+ * a finished request's stream and pages go to the next one.  cfg: shaping (request i draws with seed shaping.seed + i),
+ * uniform_mode and stop tokens; its budgets are ignored.  out_tokens [n_requests, out_stride] receives the generated
+ * tokens (the stopping one included), out_counts their number, out_reasons 0 (budget) or 1 (stop token). */
+typedef struct tsb_serve_request {
+    int32_t n_prompt, max_new_tokens;
+} tsb_serve_request;
+typedef struct tsb_serve_stats {
+    int64_t steps, rows, prompt_rows, decode_rows;
+    int32_t most_live, _pad;
+    double seconds;
+} tsb_serve_stats;
+TSB_API int32_t tsb_serve_run(tsb_session* s, const tsb_serve_request* requests, int32_t n_requests, const int32_t* prompts, const tsb_run_config* cfg,
+                              int32_t prefill_chunk, int32_t* out_tokens, int32_t out_stride, int32_t* out_counts, int32_t* out_reasons,
+                              tsb_serve_stats* stats);
 
 /* One speculative round for every stream of the session in lockstep (the benchmark's step and the
  * serving inner loop): k draft steps + the row-only step, one batched verify of k+1 rows per stream, the

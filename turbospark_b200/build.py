@@ -26,8 +26,20 @@ FLAGS = [
 ] + os.environ.get("TSB_NVCC_EXTRA", "").split()
 
 
-def _sources():
-    return sorted(f for f in os.listdir(CSRC) if f.endswith(".cu"))
+# Units of one model family only; a library of one family leaves the other's out (build(family=...)).
+FAMILY_UNITS = {
+    "blocks": {"attention.cu", "attention_tc.cu", "comm.cu", "gemm_quant.cu", "gemm_wide.cu", "model_blocks.cu", "moe.cu", "resident.cu", "rowops.cu"},
+    "plain": {"attention_window.cu", "gemm_plain.cu", "model_plain.cu", "rowops_plain.cu"},
+}
+
+
+def _sources(family=None):
+    other = set().union(*(u for f, u in FAMILY_UNITS.items() if f != family)) if family else set()
+    return sorted(f for f in os.listdir(CSRC) if f.endswith(".cu") and f not in other)
+
+
+def _stale(out, deps):
+    return not os.path.exists(out) or os.path.getmtime(out) < max(os.path.getmtime(d) for d in deps)
 
 
 def _headers_mtime():
@@ -45,11 +57,14 @@ def _compile(src, verbose):
     return src, r.stderr
 
 
-def build(force=False, verbose=False):
+def build(force=False, verbose=False, family=None):
+    """Compile what is stale and link.  family: only that model family's units and the common ones, into a library of its
+    own; None: everything, into libtsb.so.  Returns the library's path."""
     os.makedirs(OUT, exist_ok=True)
+    lib = LIB if family is None else LIB[:-3] + "_%s.so" % family
     hm = _headers_mtime()
     todo, objs = [], []
-    for src in _sources():
+    for src in _sources(family):
         obj = os.path.join(OUT, src[:-3] + ".o")
         objs.append(obj)
         stale = (force or not os.path.exists(obj)
@@ -61,16 +76,25 @@ def build(force=False, verbose=False):
         with concurrent.futures.ThreadPoolExecutor(max_workers=min(8, len(todo))) as ex:
             for src, log in ex.map(lambda s: _compile(s, verbose), todo):
                 logs.append((src, log))
-    if todo or not os.path.exists(LIB):
-        cmd = [NVCC, "-shared", "-o", LIB] + objs + ["-gencode", "arch=compute_100a,code=sm_100a", "-lcudart"]
+    if todo or _stale(lib, objs):
+        part = "%s.%d" % (lib, os.getpid())
+        cmd = [NVCC, "-shared", "-o", part] + objs + ["-gencode", "arch=compute_100a,code=sm_100a", "-lcudart"]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError("link failed:\n%s\n%s" % (r.stdout, r.stderr))
+        os.replace(part, lib)
     if verbose:
         for src, log in logs:
             print("==", src)
             print(log)
-    return LIB
+    return lib
+
+
+def ensure(family):
+    """A library that serves models of this family: the full one when it is newer than every source, else the family's own,
+    compiled as far as needed."""
+    deps = [os.path.join(CSRC, f) for f in os.listdir(CSRC)] + [os.path.join(INCLUDE, "tsb.h")]
+    return LIB if not _stale(LIB, deps) else build(family=family)
 
 
 if __name__ == "__main__":

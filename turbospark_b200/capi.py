@@ -8,6 +8,14 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 Q4_K, Q6_K, MXFP4, Q5_K, Q8_0 = 0, 1, 2, 3, 4
 
 _lib = None
+_path = None
+
+
+def use_library(path):
+    """Load this build of the library instead of the in-tree one (before the first call of lib())."""
+    global _path
+    assert _lib is None or path == _path, "the library is already loaded"
+    _path = path
 
 
 class TsbError(RuntimeError):
@@ -18,7 +26,7 @@ class TsbError(RuntimeError):
 
 def lib_path():
     # TSB_LIB points at another build of the same library (kernel experiments); the default is the in-tree one
-    return os.environ.get("TSB_LIB") or os.path.join(_HERE, "libtsb.so")
+    return _path or os.environ.get("TSB_LIB") or os.path.join(_HERE, "libtsb.so")
 
 
 class RowDesc(C.Structure):
@@ -70,7 +78,8 @@ def lib():
         L.tsb_launch_count.argtypes = [C.c_void_p]
         L.tsb_uniform_u64.restype = C.c_uint64
         L.tsb_uniform_u64.argtypes = [C.c_int32, C.c_uint64, C.c_uint64]
-        for name in ("tsb_attn_scratch_bytes", "tsb_accept_scratch_bytes", "tsb_accept_history_scratch_bytes", "tsb_gemm_workspace_bytes"):
+        for name in ("tsb_attn_scratch_bytes", "tsb_accept_scratch_bytes", "tsb_accept_history_scratch_bytes", "tsb_gemm_workspace_bytes", "tsb_plain_gemm_workspace_bytes",
+                     "tsb_window_attention_scratch_bytes"):
             if hasattr(L, name):
                 getattr(L, name).restype = C.c_size_t
         if hasattr(L, "tsb_kv_cursor"):
@@ -274,6 +283,37 @@ class Ctx:
                                      C.c_int32(n_experts), C.c_int32(d_model), C.c_int32(ffn), _vp(x), _vp(residual), _vp(ids),
                                      _vp(weights), C.c_int32(tokens), C.c_int32(k), _vp(y)))
 
+    # ---- plain-weight operators (type: 0 bfloat16, 1 f32)
+    def zeroed(self, nbytes):
+        return self.to_device(np.zeros(nbytes, dtype=np.uint8))
+
+    def plain_gemm_workspace(self):
+        return self.zeroed(int(lib().tsb_plain_gemm_workspace_bytes(self.h)))
+
+    def window_attention_scratch(self):
+        return self.zeroed(int(lib().tsb_window_attention_scratch_bytes(self.h)))
+
+    def plain_gemm(self, type_, w, rows, cols, x, x_rows, tokens, y, y_stride, n_valid, workspace, cap=0.0, add=False, stream=None):
+        self.check(lib().tsb_plain_gemm(self.h, stream, C.c_int32(type_), _vp(w), C.c_int64(rows), C.c_int64(cols), _vp(x), C.c_int32(x_rows),
+                                        C.c_int32(tokens), _vp(y), C.c_int64(y_stride), C.c_int32(n_valid), C.c_float(cap), C.c_int32(int(add)),
+                                        _vp(workspace)))
+
+    def plain_gemm_pairs(self, type_, w, rows, cols, x, x_rows, tokens, a, a_stride, n_pairs, act, workspace, stream=None):
+        self.check(lib().tsb_plain_gemm_pairs(self.h, stream, C.c_int32(type_), _vp(w), C.c_int64(rows), C.c_int64(cols), _vp(x), C.c_int32(x_rows),
+                                              C.c_int32(tokens), _vp(a), C.c_int64(a_stride), C.c_int32(n_pairs), C.c_int32(act), _vp(workspace)))
+
+    def norm_shift_rows(self, type_, x, d, gain, eps, mu, rows_dev, rows, state, n_streams, ring, mix_out, h_out, out_stride, stream=None):
+        self.check(lib().tsb_norm_shift_rows(self.h, stream, C.c_int32(type_), _vp(x), C.c_int32(d), _vp(gain), C.c_float(eps), _vp(mu), _vp(rows_dev),
+                                             C.c_int32(rows), _vp(state), C.c_int32(n_streams), C.c_int32(ring), _vp(mix_out), _vp(h_out),
+                                             C.c_int64(out_stride)))
+
+    def window_attention(self, kv, layer, q, q_stride, out, out_stride, rows_dev, group_rows, n_q_heads, scale, cap, r1, r2, gate, window, max_len,
+                         scratch, stream=None):
+        gr = (C.c_int32 * len(group_rows))(*group_rows)
+        self.check(lib().tsb_window_attention(self.h, stream, kv.h, C.c_int32(layer), _vp(q), C.c_int64(q_stride), _vp(out), C.c_int64(out_stride),
+                                              _vp(rows_dev), gr, C.c_int32(len(group_rows)), C.c_int32(n_q_heads), C.c_float(scale), C.c_float(cap),
+                                              _vp(r1), _vp(r2), _vp(gate), C.c_int32(window), C.c_int32(max_len), _vp(scratch)))
+
     def residual_add(self, x, y, n, stream=None):
         self.check(lib().tsb_residual_add(self.h, stream, _vp(x), _vp(y), C.c_int64(n)))
 
@@ -337,3 +377,25 @@ class KvCache:
         if getattr(self, "h", None):
             lib().tsb_kv_destroy(self.h)
             self.h = None
+
+
+class KeyCache(KvCache):
+    """A key-only cache: rows of kv_heads * head_dim bfloat16 bit patterns (type 0) or f32 values (type 1)."""
+
+    def __init__(self, ctx, type_, layers, kv_heads, head_dim, page_tokens, num_pages, max_seqs, max_pages_per_seq):
+        self.ctx, self.type = ctx, type_
+        self.layers, self.kv_heads, self.head_dim = layers, kv_heads, head_dim
+        h = C.c_void_p()
+        ctx.check(lib().tsb_kv_create_keys(ctx.h, C.c_int32(type_), C.c_int32(layers), C.c_int32(kv_heads), C.c_int32(head_dim), C.c_int32(page_tokens),
+                                           C.c_int32(num_pages), C.c_int32(max_seqs), C.c_int32(max_pages_per_seq), C.byref(h)))
+        self.h = h
+
+    def write_rows(self, seq, layer, pos0, k, stream=None):
+        k = np.ascontiguousarray(k, dtype=np.float32 if self.type else np.uint16)
+        self.ctx.check(lib().tsb_kv_write_rows(self.h, stream, C.c_int32(seq), C.c_int32(layer), C.c_int64(pos0),
+                                               C.c_int32(k.size // (self.kv_heads * self.head_dim)), _vp(k), None))
+
+    def read_rows(self, seq, layer, pos0, n, stream=None):
+        k = np.empty((n, self.kv_heads * self.head_dim), dtype=np.float32 if self.type else np.uint16)
+        self.ctx.check(lib().tsb_kv_read_rows(self.h, stream, C.c_int32(seq), C.c_int32(layer), C.c_int64(pos0), C.c_int32(n), _vp(k), None))
+        return k

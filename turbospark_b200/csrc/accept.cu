@@ -823,21 +823,22 @@ struct PenaltyArgs {
     float repetition;         // clamped to the normal f32 range
     double presence, frequency;
 };
+template <typename LT>
 __global__ void __launch_bounds__(1024)
-    penalize_rows_kernel(const __half* __restrict__ target, const __half* __restrict__ draft, int k, int vocab, int rows_per_stream,
+    penalize_rows_kernel(const LT* __restrict__ target, const LT* __restrict__ draft, int k, int vocab, int rows_per_stream,
                          int64_t single_stride, PenaltyArgs pa, float* __restrict__ out_target, float* __restrict__ out_draft,
                          uint32_t* __restrict__ marks) {
     pdl_wait();
     const int b = blockIdx.x / rows_per_stream, r = blockIdx.x % rows_per_stream;
     const bool is_target = single_stride != 0 || r <= k;
-    const __half* row = single_stride ? target + (size_t)b * single_stride
+    const LT* row = single_stride ? target + (size_t)b * single_stride
                         : is_target   ? target + ((size_t)b * (k + 1) + r) * vocab
                                       : draft + ((size_t)b * k + (r - k - 1)) * vocab;
     float* out = single_stride ? out_target + (size_t)b * vocab
                  : is_target   ? out_target + ((size_t)b * (k + 1) + r) * vocab
                                : out_draft + ((size_t)b * k + (r - k - 1)) * vocab;
     uint32_t* mark = marks + (size_t)blockIdx.x * vocab;
-    for (int v = threadIdx.x; v < vocab; v += blockDim.x) out[v] = __half2float(row[v]);
+    for (int v = threadIdx.x; v < vocab; v += blockDim.x) out[v] = Logit<LT>::val(row[v]);
     const int extra = (single_stride == 0 && is_target) ? r : 0;  // proposals already committed when this row is shaped
     const int nh = pa.hist_len[b];
     const int n_eff = nh + extra;
@@ -897,11 +898,14 @@ static cudaError_t launch_accept_t(tsb_ctx* ctx, cudaStream_t st, const LT* targ
                               (const RowStats*)stats, out_dev, next_tokens, next_stride);
 }
 
-cudaError_t launch_accept(tsb_ctx* ctx, cudaStream_t st, const __half* target, const __half* draft, const int32_t* proposals,
+cudaError_t launch_accept(tsb_ctx* ctx, cudaStream_t st, LogitRows target, LogitRows draft, const int32_t* proposals,
                           int prop_stride, const uint64_t* uniforms, int batch, int k, int vocab, AcceptShape shape,
                           tsb_accept_out* out_dev, int32_t* next_tokens, int next_stride, void* scratch) {
-    return launch_accept_t<__half>(ctx, st, target, draft, proposals, prop_stride, uniforms, batch, k, vocab, shape, out_dev, next_tokens,
-                                   next_stride, scratch);
+    if (target.f32)
+        return launch_accept_t<float>(ctx, st, (const float*)target.p, (const float*)draft.p, proposals, prop_stride, uniforms, batch, k, vocab, shape,
+                                      out_dev, next_tokens, next_stride, scratch);
+    return launch_accept_t<__half>(ctx, st, (const __half*)target.p, (const __half*)draft.p, proposals, prop_stride, uniforms, batch, k, vocab, shape,
+                                   out_dev, next_tokens, next_stride, scratch);
 }
 
 template <typename LT>
@@ -917,11 +921,14 @@ static cudaError_t launch_sample_t(tsb_ctx* ctx, cudaStream_t st, const LT* logi
                               margins_dev, ctx->dev_error);
 }
 
-cudaError_t launch_sample(tsb_ctx* ctx, cudaStream_t st, const __half* logits, int64_t logits_stride,
+cudaError_t launch_sample(tsb_ctx* ctx, cudaStream_t st, LogitRows logits, int64_t logits_stride,
                           const uint64_t* uniforms, int uni_stride, int batch, int vocab, AcceptShape shape,
                           int32_t* tokens_dev, int token_stride, double* margins_dev, void* scratch) {
     (void)scratch;
-    return launch_sample_t<__half>(ctx, st, logits, logits_stride, uniforms, uni_stride, batch, vocab, shape, tokens_dev, token_stride,
+    if (logits.f32)
+        return launch_sample_t<float>(ctx, st, (const float*)logits.p, logits_stride, uniforms, uni_stride, batch, vocab, shape, tokens_dev, token_stride,
+                                      margins_dev);
+    return launch_sample_t<__half>(ctx, st, (const __half*)logits.p, logits_stride, uniforms, uni_stride, batch, vocab, shape, tokens_dev, token_stride,
                                    margins_dev);
 }
 
@@ -945,7 +952,17 @@ static PenaltyArgs penalty_args(const tsb_shaping& sh, const int32_t* history, i
     return pa;
 }
 
-cudaError_t launch_accept_history(tsb_ctx* ctx, cudaStream_t st, const __half* target, const __half* draft, const int32_t* proposals,
+// the penalised f32 copy of every row of an acceptance (single_stride == 0) or of one row per stream
+static cudaError_t launch_penalize(tsb_ctx* ctx, cudaStream_t st, int grid, LogitRows target, LogitRows draft, int k, int vocab, int rows_per_stream,
+                                   int64_t single_stride, const PenaltyArgs& pa, float* out_target, float* out_draft, uint32_t* marks) {
+    if (target.f32)
+        return tsb_launch(ctx, penalize_rows_kernel<float>, dim3((unsigned)grid), dim3(1024), 0, st, false, (const float*)target.p,
+                          (const float*)draft.p, k, vocab, rows_per_stream, single_stride, pa, out_target, out_draft, marks);
+    return tsb_launch(ctx, penalize_rows_kernel<__half>, dim3((unsigned)grid), dim3(1024), 0, st, false, (const __half*)target.p,
+                      (const __half*)draft.p, k, vocab, rows_per_stream, single_stride, pa, out_target, out_draft, marks);
+}
+
+cudaError_t launch_accept_history(tsb_ctx* ctx, cudaStream_t st, LogitRows target, LogitRows draft, const int32_t* proposals,
                                   int prop_stride, const uint64_t* uniforms, int batch, int k, int vocab, const tsb_shaping& sh,
                                   const int32_t* history, int hist_stride, const int32_t* hist_len, const int32_t* generated,
                                   tsb_accept_out* out_dev, void* scratch, int32_t* next_tokens, int next_stride) {
@@ -956,14 +973,14 @@ cudaError_t launch_accept_history(tsb_ctx* ctx, cudaStream_t st, const __half* t
     uint32_t* marks = reinterpret_cast<uint32_t*>(base + penalty_rows_bytes(batch, rps, vocab));
     cudaError_t e = cudaMemsetAsync(marks, 0, penalty_rows_bytes(batch, rps, vocab), st);
     if (e != cudaSuccess) return e;
-    e = tsb_launch(ctx, penalize_rows_kernel, dim3((unsigned)(batch * rps)), dim3(1024), 0, st, false, target, draft, k, vocab, rps, (int64_t)0,
-                   penalty_args(sh, history, hist_stride, hist_len, generated, proposals, prop_stride), t32, d32, marks);
+    e = launch_penalize(ctx, st, batch * rps, target, draft, k, vocab, rps, (int64_t)0,
+                        penalty_args(sh, history, hist_stride, hist_len, generated, proposals, prop_stride), t32, d32, marks);
     if (e != cudaSuccess) return e;
     return launch_accept_t<float>(ctx, st, t32, d32, proposals, prop_stride, uniforms, batch, k, vocab, AcceptShape(sh), out_dev, next_tokens,
                                   next_stride, scratch);
 }
 
-cudaError_t launch_sample_history(tsb_ctx* ctx, cudaStream_t st, const __half* logits, const uint64_t* uniforms, int batch, int vocab,
+cudaError_t launch_sample_history(tsb_ctx* ctx, cudaStream_t st, LogitRows logits, const uint64_t* uniforms, int batch, int vocab,
                                   const tsb_shaping& sh, const int32_t* history, int hist_stride, const int32_t* hist_len,
                                   const int32_t* generated, int32_t* tokens_dev, double* margins_dev, void* scratch, int64_t logits_stride,
                                   int uni_stride, int token_stride) {
@@ -973,8 +990,8 @@ cudaError_t launch_sample_history(tsb_ctx* ctx, cudaStream_t st, const __half* l
     uint32_t* marks = reinterpret_cast<uint32_t*>(base + penalty_rows_bytes(batch, 1, vocab));
     cudaError_t e = cudaMemsetAsync(marks, 0, penalty_rows_bytes(batch, 1, vocab), st);
     if (e != cudaSuccess) return e;
-    e = tsb_launch(ctx, penalize_rows_kernel, dim3((unsigned)batch), dim3(1024), 0, st, false, logits, (const __half*)nullptr, 0, vocab, 1,
-                   logits_stride, penalty_args(sh, history, hist_stride, hist_len, generated, nullptr, 0), l32, (float*)nullptr, marks);
+    e = launch_penalize(ctx, st, batch, logits, LogitRows(), 0, vocab, 1,
+                        logits_stride, penalty_args(sh, history, hist_stride, hist_len, generated, nullptr, 0), l32, nullptr, marks);
     if (e != cudaSuccess) return e;
     return launch_sample_t<float>(ctx, st, l32, vocab, uniforms, uni_stride, batch, vocab, AcceptShape(sh), tokens_dev, token_stride, margins_dev);
 }
@@ -984,13 +1001,19 @@ cudaError_t launch_topk_rows(tsb_ctx* ctx, cudaStream_t st, const __half* logits
     return tsb_launch(ctx, topk_rows_kernel, dim3((unsigned)n_rows), dim3(1024), 0, st, true, logits, vocab, rows_dev, width, out_dev);
 }
 
-cudaError_t launch_argmax_rows(tsb_ctx* ctx, cudaStream_t st, const __half* logits, int n_rows, int vocab, void* scratch) {
+cudaError_t launch_argmax_rows(tsb_ctx* ctx, cudaStream_t st, LogitRows logits, int n_rows, int vocab, void* scratch) {
     // the statistics kernel at temperature 0: max, first argmax and finiteness of every row (rows are "target rows")
     RowStats* stats = reinterpret_cast<RowStats*>(scratch);
     const size_t smem = slice_smem(vocab);
+    if (logits.f32) {
+        if (cudaError_t e = configure_kernels<float>(ctx); e != cudaSuccess) return e;
+        return tsb_launch_cluster(ctx, accept_stats_kernel<float>, dim3((unsigned)(n_rows * CL)), dim3(ACC_THREADS), smem, st, true, (unsigned)CL,
+                                  (const float*)logits.p, (const float*)nullptr, n_rows - 1, vocab, 0.0, TruncShape{0u, 0.0, 0.0}, stats, n_rows,
+                                  (int64_t)0);
+    }
     if (cudaError_t e = configure_kernels<__half>(ctx); e != cudaSuccess) return e;
     return tsb_launch_cluster(ctx, accept_stats_kernel<__half>, dim3((unsigned)(n_rows * CL)), dim3(ACC_THREADS), smem, st, true,
-                              (unsigned)CL, logits, (const __half*)nullptr, n_rows - 1, vocab, 0.0, TruncShape{0u, 0.0, 0.0}, stats, n_rows,
+                              (unsigned)CL, (const __half*)logits.p, (const __half*)nullptr, n_rows - 1, vocab, 0.0, TruncShape{0u, 0.0, 0.0}, stats, n_rows,
                               (int64_t)0);
 }
 

@@ -916,6 +916,7 @@ int32_t tsb_attn_decode_rows(tsb_ctx* ctx, tsb_stream s, tsb_kv* kv, int32_t lay
                              int32_t n_q_heads, float scale, int32_t max_len, void* scratch, size_t scratch_bytes) {
     if (!ctx || !kv) return TSB_ERR_INVALID;
     TSB_REQUIRE(ctx, q_f16 && out_f16 && rows_dev && scratch, "null buffer");
+    TSB_REQUIRE(ctx, kv->view.pool, "a key-only cache has no value rows (tsb_window_attention takes it)");
     TSB_REQUIRE(ctx, rows > 0 && rows_per_seq > 0 && rows % rows_per_seq == 0, "rows must be a whole number of streams");
     TSB_REQUIRE(ctx, rows_per_seq <= 128, "at most 128 in-flight rows per stream (mask width), got %d", rows_per_seq);
     TSB_REQUIRE(ctx, layer >= 0 && layer < kv->view.layers, "layer %d outside 0..%d", layer, kv->view.layers);
@@ -973,6 +974,7 @@ int32_t tsb_attn_decode_rows_static(tsb_ctx* ctx, tsb_stream s, tsb_kv* kv, int3
                                     int64_t q_stride, void* out_f16, const tsb_row_desc* rows_dev, int32_t rows,
                                     int32_t rows_per_seq, int32_t n_q_heads, float scale, int32_t max_len) {
     if (!ctx || !kv) return TSB_ERR_INVALID;
+    TSB_REQUIRE(ctx, kv->view.pool, "a key-only cache has no value rows (tsb_window_attention takes it)");
     TSB_REQUIRE(ctx, rows > 0 && n_q_heads > 0, "rows and n_q_heads must be positive");
     const size_t need = attn_scratch_bytes(rows, n_q_heads, kv->view.head_dim);
     if (need > ATTN_STATIC_BYTES)

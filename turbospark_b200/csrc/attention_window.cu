@@ -1,0 +1,542 @@
+// Sliding-window attention over a key-only paged cache (attention_window.cuh).
+//
+// bfloat16: one kernel template <D, MT, SL> on mma.sync m16n8k16.  A CTA owns one (query tile, key head, run of key tiles):
+// MT m-tiles of 16 queries - the tile's rows x the heads that share the key head - and walks 64-token key tiles that
+// cp.async brings into a three-stage ring.  The one tile in shared memory serves both products: K rows as the B operand
+// of S = Q K^T (ldmatrix) and as the B operand of O += P K (ldmatrix.trans), so a key byte is read once.  SL warps share an
+// m-tile, each taking 64 / SL tokens of every tile, and meet at the end.
+//   few queries (decode, short portions): SL = 4, the context is cut into runs so that the device is full; the last CTA of
+//   a tile to finish - decided by a ticket, nobody waits - adds the runs in order
+//   many queries (prompts): MT = 8, SL = 1
+// Only the key tiles inside the window of some query of the tile are visited; key tiles start at multiples of 64 positions
+// whatever the cut of the prompt, so a row meets its keys in the same grouping in every schedule.
+//
+// Score arithmetic in f32, base 2: v = cap log2(e) tanh(s scale / cap) - r1 log2(1 + r2 d).
+//
+// f32: one warp per (row, query head), lanes over keys for the scores and over columns for the sum; the reference-precision
+// mode, plain fused multiply-adds and the library's exp, tanh and log.
+#include <algorithm>
+
+#include "attention_window.cuh"
+
+namespace {
+
+constexpr int TOK = 64;   // tokens per key tile
+constexpr int NST = 3;    // key tiles in flight
+constexpr int WATTN_TICKETS = 16384;
+constexpr int WATTN_MAX_SPLITS = 64;
+
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm4_t(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+        : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+        : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool valid) {
+    const int n = valid ? 16 : 0;
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
+}
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float lg2(float x) {
+    float y;
+    asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float rcp(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
+    return *reinterpret_cast<const uint32_t*>(&h);
+}
+__device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+
+template <int D>
+struct Geo {
+    static constexpr int PITCH = D <= 32 ? 64 : D <= 64 ? 128 : D <= 128 ? 256 : 512;  // bytes of a row in shared memory
+    static constexpr int CH = D / 8;                                                  // 16-byte chunks of a row
+    // byte offset of chunk c of row r: the chunks of a row are permuted so that eight rows' worth of one chunk spread over
+    // all banks
+    static __device__ __forceinline__ uint32_t off(int r, int c) {
+        return (uint32_t)(r * PITCH + ((D <= 32 ? (c ^ ((r >> 1) & 3)) : (c ^ (r & 7))) << 4));
+    }
+};
+
+template <int D, int MT, int SL>
+constexpr size_t wattn_smem() {
+    const size_t ring = (size_t)NST * TOK * Geo<D>::PITCH + (SL == 1 ? (size_t)MT * 16 * Geo<D>::PITCH : 0);
+    const size_t merge = SL > 1 ? (size_t)MT * SL * 16 * ((D + 4) * 4 + 8) : 0;
+    return ring > merge ? ring : merge;
+}
+
+template <int D, int MT, int SL>
+__global__ void __launch_bounds__(32 * MT * SL, MT * SL <= 4 ? 3 : 1)
+    window_attn_kernel(const __grid_constant__ WindowAttn a, const AttnTile* __restrict__ tiles, int tiles_per_group, int rows_per_seq, int rows_per_tile,
+                       float* __restrict__ part_o, float2* __restrict__ part_ml, uint32_t* __restrict__ tickets, uint32_t* __restrict__ err) {
+    using G = Geo<D>;
+    constexpr int KS = D / 16, NO = D / 8, QT = 16 * MT, NTHR = 32 * MT * SL;
+    constexpr int WTOK = TOK / SL, NT8 = WTOK / 8, KK = WTOK / 16;
+    constexpr bool QREG = SL > 1 ? D <= 128 : D <= 64;  // query fragments stay in registers
+    extern __shared__ __align__(128) uint8_t smem[];
+    __shared__ uint32_t s_ticket;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
+    const int mt = warp % MT, sl = warp / MT;
+    const int kvh = blockIdx.y, n_splits = gridDim.x;
+    const int grp = a.n_q_heads / a.keys.kv_heads;
+
+    int row_first, n_rows;
+    if (tiles) {
+        row_first = tiles[blockIdx.z].row_first, n_rows = tiles[blockIdx.z].n_rows;
+    } else {
+        const int in_group = ((int)blockIdx.z % tiles_per_group) * rows_per_tile;
+        row_first = ((int)blockIdx.z / tiles_per_group) * rows_per_seq + in_group;
+        n_rows = min(rows_per_tile, rows_per_seq - in_group);
+    }
+    const tsb_row_desc rd0 = a.rows[row_first];
+    const int seq = rd0.seq, pos0 = rd0.base + rd0.slot;
+    const int n_queries = n_rows * grp;
+    if (seq < 0 || seq >= a.keys.max_seqs || n_queries > QT) {
+        if (threadIdx.x == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+        pdl_wait();
+        return;
+    }
+    // visible positions of the tile's queries, in whole key tiles; this CTA's run of them
+    const int lo = a.window > 0 ? max(0, pos0 - a.window + 1) & ~(TOK - 1) : 0;
+    const int hi = pos0 + n_rows;
+    const int total = (hi - lo + TOK - 1) / TOK;
+    const int per = (total + n_splits - 1) / n_splits;
+    const int t_first = min(total, (int)blockIdx.x * per), n_tiles = min(total, t_first + per) - t_first;
+    const int begin = lo + t_first * TOK;
+
+    const uint32_t ring = smem_u32(smem);
+    auto issue = [&](int tile, int stage) {
+        constexpr int TPR = NTHR / TOK;  // threads per token row
+        const int r = threadIdx.x / TPR, part = threadIdx.x % TPR;
+        const int pos = begin + tile * TOK + r;
+        const __nv_bfloat16* src = pos < hi ? key_row<__nv_bfloat16>(a.keys, seq, pos) : nullptr;
+        const bool ok = src != nullptr;
+        src = ok ? src + (int64_t)kvh * D : reinterpret_cast<const __nv_bfloat16*>(a.keys.base);
+        const uint32_t dst = ring + stage * (TOK * G::PITCH);
+#pragma unroll
+        for (int c = part; c < G::CH; c += TPR) cp16(dst + G::off(r, c), ok ? src + c * 8 : src, ok);
+        cp_async_commit();
+    };
+    auto prologue = [&]() {
+#pragma unroll
+        for (int i = 0; i < NST; i++) {
+            if (i < n_tiles) issue(i, i);
+            else cp_async_commit();
+        }
+    };
+    // key tiles of earlier passes may start moving while the kernel that writes this pass's rows still runs
+    const bool early = begin + NST * TOK <= rd0.base;
+    if (early) prologue();
+    pdl_wait();
+    if (!early) prologue();
+
+    // the lane's two queries: rows gid and gid + 8 of its m-tile
+    const __nv_bfloat16* qp[2];
+    int pq[2];
+    float r1[2] = {0.f, 0.f}, r2[2] = {0.f, 0.f};
+#pragma unroll
+    for (int h = 0; h < 2; h++) {
+        const int qi = mt * 16 + gid + 8 * h;
+        const bool v = qi < n_queries;
+        const int row = v ? qi / grp : 0, head = kvh * grp + (v ? qi % grp : 0);
+        pq[h] = v ? pos0 + row : -1;  // an empty query slot sees nothing
+        qp[h] = reinterpret_cast<const __nv_bfloat16*>(a.q) + (int64_t)(row_first + row) * a.q_stride + head * D;
+        if (a.r1) r1[h] = a.r1[head], r2[h] = a.r2[head];
+    }
+    uint32_t qa[QREG ? KS : 1][4];
+    const uint32_t q_smem = ring + NST * TOK * G::PITCH;
+    if (QREG) {
+#pragma unroll
+        for (int ks = 0; ks < (QREG ? KS : 0); ks++) {
+            qa[ks][0] = *reinterpret_cast<const uint32_t*>(qp[0] + 16 * ks + 2 * tig);
+            qa[ks][1] = *reinterpret_cast<const uint32_t*>(qp[1] + 16 * ks + 2 * tig);
+            qa[ks][2] = *reinterpret_cast<const uint32_t*>(qp[0] + 16 * ks + 8 + 2 * tig);
+            qa[ks][3] = *reinterpret_cast<const uint32_t*>(qp[1] + 16 * ks + 8 + 2 * tig);
+        }
+    } else if (SL == 1) {
+        for (int i = threadIdx.x; i < QT * G::CH; i += NTHR) {
+            const int qi = i / G::CH, c = i % G::CH;
+            uint4 v = make_uint4(0, 0, 0, 0);
+            if (qi < n_queries)
+                v = *reinterpret_cast<const uint4*>(reinterpret_cast<const __nv_bfloat16*>(a.q) + (int64_t)(row_first + qi / grp) * a.q_stride +
+                                                    (kvh * grp + qi % grp) * D + c * 8);
+            *reinterpret_cast<uint4*>(smem + NST * TOK * G::PITCH + G::off(qi, c)) = v;
+        }
+    }
+
+    constexpr float LOG2E = 1.4426950408889634f;
+    const bool capped = a.cap > 0.f, biased = a.r1 != nullptr;
+    const float s_in = capped ? a.scale / a.cap * (2.f * LOG2E) : a.scale * LOG2E;  // capped: the exponent of e^(2 s / cap) in base 2
+    const float c_out = a.cap * LOG2E;
+
+    float o[NO][4];
+#pragma unroll
+    for (int n = 0; n < NO; n++)
+#pragma unroll
+        for (int i = 0; i < 4; i++) o[n][i] = 0.f;
+    float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+
+    for (int tile = 0; tile < n_tiles; tile++) {
+        const int stage = tile % NST;
+        cp_async_wait<NST - 1>();
+        __syncthreads();
+        const uint32_t kt = ring + stage * (TOK * G::PITCH);
+        const int tok0 = sl * WTOK;
+        const int p0 = begin + tile * TOK + tok0;
+        float s[NT8][4];
+#pragma unroll
+        for (int n = 0; n < NT8; n++)
+#pragma unroll
+            for (int i = 0; i < 4; i++) s[n][i] = 0.f;
+#pragma unroll
+        for (int kp = 0; kp < KS / 2; kp++) {
+            uint32_t a0[4], a1[4];
+            if (QREG) {
+#pragma unroll
+                for (int i = 0; i < 4; i++) a0[i] = qa[QREG ? 2 * kp : 0][i], a1[i] = qa[QREG ? 2 * kp + 1 : 0][i];
+            } else if (SL == 1) {
+                const int r = mt * 16 + (lane & 15), c = kp * 4 + (lane >> 4);
+                ldsm4(a0, q_smem + G::off(r, c));
+                ldsm4(a1, q_smem + G::off(r, c + 2));
+            } else {
+                a0[0] = *reinterpret_cast<const uint32_t*>(qp[0] + 32 * kp + 2 * tig), a0[1] = *reinterpret_cast<const uint32_t*>(qp[1] + 32 * kp + 2 * tig);
+                a0[2] = *reinterpret_cast<const uint32_t*>(qp[0] + 32 * kp + 8 + 2 * tig), a0[3] = *reinterpret_cast<const uint32_t*>(qp[1] + 32 * kp + 8 + 2 * tig);
+                a1[0] = *reinterpret_cast<const uint32_t*>(qp[0] + 32 * kp + 16 + 2 * tig), a1[1] = *reinterpret_cast<const uint32_t*>(qp[1] + 32 * kp + 16 + 2 * tig);
+                a1[2] = *reinterpret_cast<const uint32_t*>(qp[0] + 32 * kp + 24 + 2 * tig), a1[3] = *reinterpret_cast<const uint32_t*>(qp[1] + 32 * kp + 24 + 2 * tig);
+            }
+#pragma unroll
+            for (int n = 0; n < NT8; n++) {
+                uint32_t b[4];
+                ldsm4(b, kt + G::off(tok0 + n * 8 + (lane & 7), kp * 4 + (lane >> 3)));
+                mma_bf16(s[n], a0, b[0], b[1]);
+                mma_bf16(s[n], a1, b[2], b[3]);
+            }
+        }
+        // scores to base-2 logits; the mask only where the tile meets an edge
+        const bool edge = p0 + WTOK > pos0 || (a.window > 0 && p0 <= pos0 + n_rows - 1 - a.window) || n_queries < QT;
+        float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+        for (int n = 0; n < NT8; n++)
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                const int h = i >> 1;
+                const int dist = pq[h] - (p0 + n * 8 + 2 * tig + (i & 1));
+                float v = s[n][i] * s_in;
+                if (capped) v = fmaf(-2.f * c_out, rcp(ex2(v) + 1.f), c_out);  // tanh(y) = 1 - 2 / (e^(2y) + 1)
+                if (biased) v = fmaf(-r1[h], lg2(fmaf(r2[h], (float)dist, 1.f)), v);
+                if (edge && (dist < 0 || (a.window > 0 && dist >= a.window))) v = -INFINITY;
+                s[n][i] = v;
+                mx[h] = fmaxf(mx[h], v);
+            }
+        float alpha[2], m_use[2];
+#pragma unroll
+        for (int h = 0; h < 2; h++) {
+            mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
+            mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
+            const float m_new = fmaxf(m_run[h], mx[h]);
+            m_use[h] = m_new == -INFINITY ? 0.f : m_new;
+            alpha[h] = ex2(m_run[h] - m_use[h]);  // 0 while nothing was visible
+            m_run[h] = m_new;
+        }
+        float rs[2] = {0.f, 0.f};
+        uint32_t pa[KK][4];
+#pragma unroll
+        for (int n = 0; n < NT8; n++) {
+            const float e0 = ex2(s[n][0] - m_use[0]), e1 = ex2(s[n][1] - m_use[0]);
+            const float e2 = ex2(s[n][2] - m_use[1]), e3 = ex2(s[n][3] - m_use[1]);
+            rs[0] += e0 + e1, rs[1] += e2 + e3;
+            pa[n >> 1][(n & 1) * 2] = pack_bf16(e0, e1);
+            pa[n >> 1][(n & 1) * 2 + 1] = pack_bf16(e2, e3);
+        }
+#pragma unroll
+        for (int h = 0; h < 2; h++) l_run[h] = fmaf(l_run[h], alpha[h], rs[h]);  // per lane; the quad's lanes meet at the end
+        if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
+#pragma unroll
+            for (int n = 0; n < NO; n++) o[n][0] *= alpha[0], o[n][1] *= alpha[0], o[n][2] *= alpha[1], o[n][3] *= alpha[1];
+        }
+#pragma unroll
+        for (int kk = 0; kk < KK; kk++) {
+#pragma unroll
+            for (int np = 0; np < NO / 2; np++) {
+                uint32_t b[4];
+                ldsm4_t(b, kt + G::off(tok0 + kk * 16 + (lane & 15), np * 2 + (lane >> 4)));
+                mma_bf16(o[2 * np], pa[kk], b[0], b[1]);
+                mma_bf16(o[2 * np + 1], pa[kk], b[2], b[3]);
+            }
+        }
+        __syncthreads();  // a stage is rewritten only after every warp is done with it
+        if (tile + NST < n_tiles) issue(tile + NST, stage);
+        else cp_async_commit();
+    }
+    cp_async_wait<0>();
+    pdl_launch_dependents();
+#pragma unroll
+    for (int h = 0; h < 2; h++) {
+        l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 1);
+        l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 2);
+    }
+
+    const int64_t tile_id = (int64_t)blockIdx.z * a.keys.kv_heads + kvh;
+    const int64_t share = (tile_id * n_splits + blockIdx.x) * QT;
+    __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out);
+    auto out_at = [&](int qi) { return out + (int64_t)(row_first + qi / grp) * a.out_stride + (kvh * grp + qi % grp) * D; };
+    auto factor = [&](int qi, float l) {  // 1 / sum, times the head's gate
+        const float inv = l > 0.f ? 1.f / l : 0.f;
+        return a.gate ? inv * sigmoid(a.gate[(int64_t)(row_first + qi / grp) * a.n_q_heads + kvh * grp + qi % grp]) : inv;
+    };
+
+    if (SL == 1) {
+#pragma unroll
+        for (int h = 0; h < 2; h++) {
+            const int qi = mt * 16 + gid + 8 * h;
+            if (qi >= n_queries) continue;
+            if (n_splits == 1) {
+                const float f = factor(qi, l_run[h]);
+                __nv_bfloat16* p = out_at(qi);
+#pragma unroll
+                for (int n = 0; n < NO; n++) *reinterpret_cast<uint32_t*>(p + n * 8 + 2 * tig) = pack_bf16(o[n][2 * h] * f, o[n][2 * h + 1] * f);
+            } else {
+                float* p = part_o + (share + qi) * D;
+#pragma unroll
+                for (int n = 0; n < NO; n++) *reinterpret_cast<float2*>(p + n * 8 + 2 * tig) = make_float2(o[n][2 * h], o[n][2 * h + 1]);
+                if (tig == 0) part_ml[share + qi] = make_float2(m_run[h], l_run[h]);
+            }
+        }
+    } else {
+        // the slices of an m-tile meet in shared memory (the ring is free now)
+        constexpr int DP = D + 4;
+        float* wo = reinterpret_cast<float*>(smem);
+        float2* wml = reinterpret_cast<float2*>(smem + (size_t)MT * SL * 16 * DP * 4);
+        __syncthreads();
+        float* dst = wo + (size_t)warp * 16 * DP;
+#pragma unroll
+        for (int n = 0; n < NO; n++) {
+            *reinterpret_cast<float2*>(dst + gid * DP + n * 8 + 2 * tig) = make_float2(o[n][0], o[n][1]);
+            *reinterpret_cast<float2*>(dst + (gid + 8) * DP + n * 8 + 2 * tig) = make_float2(o[n][2], o[n][3]);
+        }
+        if (tig == 0) {
+            wml[warp * 16 + gid] = make_float2(m_run[0], l_run[0]);
+            wml[warp * 16 + gid + 8] = make_float2(m_run[1], l_run[1]);
+        }
+        __syncthreads();
+        for (int i = threadIdx.x; i < n_queries * (D / 4); i += NTHR) {
+            const int qi = i / (D / 4), c = (i % (D / 4)) * 4, m0 = qi >> 4, qq = qi & 15;
+            float m = -INFINITY, l = 0.f;
+#pragma unroll
+            for (int k = 0; k < SL; k++) m = fmaxf(m, wml[(k * MT + m0) * 16 + qq].x);
+            const float mu = m == -INFINITY ? 0.f : m;
+            float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+            for (int k = 0; k < SL; k++) {
+                const int w = k * MT + m0;
+                const float2 v = wml[w * 16 + qq];
+                const float f = ex2(v.x - mu);
+                l = fmaf(v.y, f, l);
+                const float4 x = *reinterpret_cast<const float4*>(wo + ((size_t)w * 16 + qq) * DP + c);
+                acc.x = fmaf(x.x, f, acc.x), acc.y = fmaf(x.y, f, acc.y), acc.z = fmaf(x.z, f, acc.z), acc.w = fmaf(x.w, f, acc.w);
+            }
+            if (n_splits == 1) {
+                const float f = factor(qi, l);
+                *reinterpret_cast<uint2*>(out_at(qi) + c) = make_uint2(pack_bf16(acc.x * f, acc.y * f), pack_bf16(acc.z * f, acc.w * f));
+            } else {
+                *reinterpret_cast<float4*>(part_o + (share + qi) * D + c) = acc;
+                if (c == 0) part_ml[share + qi] = make_float2(m, l);
+            }
+        }
+    }
+    if (n_splits == 1) return;
+
+    // the last run of the tile to finish adds all of them, in order
+    __threadfence();
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        s_ticket = atomicAdd(&tickets[tile_id], 1u);
+        if (s_ticket == (uint32_t)n_splits - 1) tickets[tile_id] = 0;
+    }
+    __syncthreads();
+    if (s_ticket != (uint32_t)n_splits - 1) return;
+    __threadfence();
+    const int64_t first = tile_id * n_splits * QT;
+    for (int i = threadIdx.x; i < n_queries * (D / 4); i += NTHR) {
+        const int qi = i / (D / 4), c = (i % (D / 4)) * 4;
+        float m = -INFINITY, l = 0.f;
+        for (int k = 0; k < n_splits; k++) m = fmaxf(m, __ldcg(&part_ml[first + k * QT + qi]).x);
+        const float mu = m == -INFINITY ? 0.f : m;
+        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+        for (int k = 0; k < n_splits; k++) {
+            const float2 v = __ldcg(&part_ml[first + k * QT + qi]);
+            const float4 x = __ldcg(reinterpret_cast<const float4*>(part_o + (first + k * QT + qi) * D + c));
+            const float f = ex2(v.x - mu);
+            l = fmaf(v.y, f, l);
+            acc.x = fmaf(x.x, f, acc.x), acc.y = fmaf(x.y, f, acc.y), acc.z = fmaf(x.z, f, acc.z), acc.w = fmaf(x.w, f, acc.w);
+        }
+        const float f = factor(qi, l);
+        *reinterpret_cast<uint2*>(out_at(qi) + c) = make_uint2(pack_bf16(acc.x * f, acc.y * f), pack_bf16(acc.z * f, acc.w * f));
+    }
+}
+
+// ------------------------------------------------------------------ f32
+constexpr int F32_WARPS = 4;
+constexpr int F32_MAX_DIM = 512;
+__global__ void __launch_bounds__(F32_WARPS * 32) window_attn_f32_kernel(const __grid_constant__ WindowAttn a, int rows, uint32_t* __restrict__ err) {
+    __shared__ float qs[F32_WARPS][F32_MAX_DIM];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int64_t item = (int64_t)blockIdx.x * F32_WARPS + warp;
+    pdl_wait();
+    pdl_launch_dependents();
+    if (item >= (int64_t)rows * a.n_q_heads) return;
+    const int row = (int)(item / a.n_q_heads), head = (int)(item % a.n_q_heads);
+    const int D = a.keys.head_dim, kvh = head / (a.n_q_heads / a.keys.kv_heads);
+    const tsb_row_desc rd = a.rows[row];
+    const int pos = rd.base + rd.slot;
+    const float* q = reinterpret_cast<const float*>(a.q) + (int64_t)row * a.q_stride + (int64_t)head * D;
+    for (int i = lane; i < D; i += 32) qs[warp][i] = q[i];
+    __syncwarp();
+    const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+    const float r1 = a.r1 ? a.r1[head] : 0.f, r2 = a.r1 ? a.r2[head] : 0.f;
+    float m = -INFINITY, l = 0.f, acc[F32_MAX_DIM / 32];
+#pragma unroll
+    for (int i = 0; i < F32_MAX_DIM / 32; i++) acc[i] = 0.f;
+    for (int j0 = lo & ~31; j0 <= pos; j0 += 32) {
+        const int j = j0 + lane;
+        const bool seen = j >= lo && j <= pos;
+        const float* k = seen ? key_row<float>(a.keys, rd.seq, j) : nullptr;
+        if (seen && !k) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+        float s = -INFINITY;
+        if (k) {
+            k += (int64_t)kvh * D;
+            float dot = 0.f;
+            for (int i = 0; i < D; i += 4) {
+                const float4 v = *reinterpret_cast<const float4*>(k + i);
+                dot = fmaf(v.x, qs[warp][i], dot), dot = fmaf(v.y, qs[warp][i + 1], dot);
+                dot = fmaf(v.z, qs[warp][i + 2], dot), dot = fmaf(v.w, qs[warp][i + 3], dot);
+            }
+            s = dot * a.scale;
+            if (a.cap > 0.f) s = a.cap * tanhf(s / a.cap);
+            if (a.r1) s -= r1 * logf(1.f + r2 * (float)(pos - j));
+        }
+        float mx = s;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        const float m_new = fmaxf(m, mx);
+        if (m_new == -INFINITY) continue;
+        const float alpha = expf(m - m_new), p = expf(s - m_new);
+        m = m_new;
+        float ps = p;
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) ps += __shfl_xor_sync(0xffffffffu, ps, o);
+        l = fmaf(l, alpha, ps);
+#pragma unroll
+        for (int i = 0; i < F32_MAX_DIM / 32; i++) acc[i] *= alpha;
+        for (int t = 0; t < 32; t++) {
+            const float pt = __shfl_sync(0xffffffffu, p, t);
+            if (pt == 0.f) continue;  // the same for every lane
+            const float* kt = key_row<float>(a.keys, rd.seq, j0 + t);
+            if (!kt) continue;
+            kt += (int64_t)kvh * D;
+#pragma unroll
+            for (int i = 0; i < F32_MAX_DIM / 32; i++)
+                if (i * 32 + lane < D) acc[i] = fmaf(pt, kt[i * 32 + lane], acc[i]);
+        }
+    }
+    const float f = (l > 0.f ? 1.f / l : 0.f) * (a.gate ? sigmoid(a.gate[(int64_t)row * a.n_q_heads + head]) : 1.f);
+    float* out = reinterpret_cast<float*>(a.out) + (int64_t)row * a.out_stride + (int64_t)head * D;
+#pragma unroll
+    for (int i = 0; i < F32_MAX_DIM / 32; i++)
+        if (i * 32 + lane < D) out[i * 32 + lane] = acc[i] * f;
+}
+
+struct Launch {
+    const AttnTile* tiles;
+    int n_tiles, tiles_per_group, rows_per_seq, rows_per_tile, max_len;
+};
+
+// cut tiles: at most 2 CTAs per SM in the few-query kernel (64 queries), one in the many-query kernel (128)
+size_t part_queries(const tsb_ctx* ctx) { return (size_t)2 * (ctx->sm_count > 0 ? ctx->sm_count : 148) * WATTN_SMALL_Q; }
+
+template <int D, int MT, int SL>
+cudaError_t launch_one(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const Launch& l, void* scratch) {
+    const int sms = ctx->sm_count > 0 ? ctx->sm_count : 148;
+    const int base = l.n_tiles * a.keys.kv_heads;
+    const int span = a.window > 0 ? std::min(l.max_len, a.window + l.rows_per_tile) : l.max_len;
+    const int key_tiles = (span + TOK - 1) / TOK + (a.window > 0 ? 1 : 0);
+    // as many runs as fill the device (a few CTAs per SM in the few-query kernel), none shorter than two key tiles
+    const int want = (SL > 1 ? 2 * sms : sms) / std::max(base, 1);
+    int splits = std::max(1, std::min({want, (key_tiles + 1) / 2, WATTN_MAX_SPLITS}));
+    if (splits > 1 && ((int64_t)base * splits * 16 * MT > (int64_t)part_queries(ctx) || base > WATTN_TICKETS)) splits = 1;
+    uint32_t* tickets = static_cast<uint32_t*>(scratch);
+    float2* ml = reinterpret_cast<float2*>(tickets + WATTN_TICKETS);
+    float* po = reinterpret_cast<float*>(ml + part_queries(ctx));
+    constexpr size_t smem = wattn_smem<D, MT, SL>();
+    static SmemOptIn configured;
+    if (cudaError_t e = tsb_opt_in_smem(ctx, window_attn_kernel<D, MT, SL>, smem, configured); e != cudaSuccess) return e;
+    return tsb_launch(ctx, window_attn_kernel<D, MT, SL>, dim3((unsigned)splits, (unsigned)a.keys.kv_heads, (unsigned)l.n_tiles), dim3(32 * MT * SL), smem,
+                      st, true, a, l.tiles, l.tiles_per_group, l.rows_per_seq, l.rows_per_tile, po, ml, tickets, ctx->dev_error);
+}
+
+template <int MT, int SL>
+cudaError_t launch_dim(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const Launch& l, void* scratch) {
+    switch (a.keys.head_dim) {
+        case 32: return launch_one<32, MT, SL>(ctx, st, a, l, scratch);
+        case 64: return launch_one<64, MT, SL>(ctx, st, a, l, scratch);
+        case 96: return launch_one<96, MT, SL>(ctx, st, a, l, scratch);
+        case 128: return launch_one<128, MT, SL>(ctx, st, a, l, scratch);
+        case 192: return launch_one<192, MT, SL>(ctx, st, a, l, scratch);
+        case 256: return launch_one<256, MT, SL>(ctx, st, a, l, scratch);
+        default: return cudaErrorInvalidValue;
+    }
+}
+
+cudaError_t launch_small(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const Launch& l, int queries, void* scratch) {
+    if (queries <= 16) return launch_dim<1, 4>(ctx, st, a, l, scratch);
+    return launch_dim<4, 2>(ctx, st, a, l, scratch);
+}
+
+}  // namespace
+
+size_t wattn_scratch_bytes(const tsb_ctx* ctx) {
+    return WATTN_TICKETS * sizeof(uint32_t) + part_queries(ctx) * (sizeof(float2) + 256 * sizeof(float));
+}
+
+int wattn_pad_dim(int head_dim, bool f32) {
+    if (head_dim <= 0) return 0;
+    if (f32) return head_dim <= F32_MAX_DIM ? (head_dim + 3) / 4 * 4 : 0;
+    for (int d : {32, 64, 96, 128, 192, 256})
+        if (head_dim <= d) return d;
+    return 0;
+}
+
+bool wattn_supported(int head_dim, int group, bool f32) { return wattn_pad_dim(head_dim, f32) > 0 && group >= 1 && (f32 || group <= WATTN_LARGE_Q); }
+
+cudaError_t launch_window_attn(tsb_ctx* ctx, cudaStream_t st, bool f32, const WindowAttn& a, const AttnBatch& b, void* scratch) {
+    if (f32)
+        return tsb_launch(ctx, window_attn_f32_kernel, dim3((unsigned)(((int64_t)b.rows * a.n_q_heads + F32_WARPS - 1) / F32_WARPS)), dim3(F32_WARPS * 32),
+                          0, st, true, a, b.rows, ctx->dev_error);
+    const int grp = a.n_q_heads / a.keys.kv_heads, rpt = wattn_rows_per_tile(grp);
+    if (b.rows_per_seq > 0) {
+        const int groups = b.rows / b.rows_per_seq, queries = b.rows_per_seq * grp;
+        if (queries <= WATTN_SMALL_Q) return launch_small(ctx, st, a, Launch{nullptr, groups, 1, b.rows_per_seq, b.rows_per_seq, b.max_len}, queries, scratch);
+        const int tpg = (b.rows_per_seq + rpt - 1) / rpt;
+        return launch_dim<8, 1>(ctx, st, a, Launch{nullptr, groups * tpg, tpg, b.rows_per_seq, rpt, b.max_len}, scratch);
+    }
+    cudaError_t e = cudaSuccess;
+    if (b.n_large > 0) e = launch_dim<8, 1>(ctx, st, a, Launch{b.large, b.n_large, 1, 0, rpt, b.max_len}, scratch);
+    if (e == cudaSuccess && b.n_small > 0) e = launch_small(ctx, st, a, Launch{b.small, b.n_small, 1, 0, WATTN_SMALL_Q / grp, b.max_len}, b.small_queries, scratch);
+    return e;
+}

@@ -1,0 +1,42 @@
+// Attention over a key-only paged cache (a layer's values are its keys), with a sliding window, a soft cap on the
+// scores, a per-head logarithmic distance bias and a per-head output gate - each of them optional.
+#pragma once
+#include <cuda_bf16.h>
+
+#include "kv.cuh"
+
+struct WindowAttn {
+    KeyView keys{};
+    const void* q = nullptr;  // [rows, n_q_heads * keys.head_dim], the compute type
+    int64_t q_stride = 0;
+    const float* gate = nullptr;  // [rows, n_q_heads]: a head's output is multiplied by sigmoid(gate); null: no gate
+    void* out = nullptr;      // [rows, n_q_heads * keys.head_dim], the compute type
+    int64_t out_stride = 0;
+    const tsb_row_desc* rows = nullptr;  // position base + slot; the rows of a stream are consecutive
+    int n_q_heads = 0;
+    float scale = 1.f;        // score = (q . k) * scale
+    float cap = 0.f;          // > 0: score <- cap * tanh(score / cap)
+    const float *r1 = nullptr, *r2 = nullptr;  // per head: score <- score - r1 * ln(1 + r2 * distance); null: no bias
+    int window = 0;           // a query sees itself and the window - 1 positions before it; 0: every earlier position
+};
+
+// A query tile: consecutive rows of one stream times the query heads of one key head.
+struct AttnTile {
+    int32_t row_first, n_rows;
+};
+constexpr int WATTN_SMALL_Q = 64;   // queries (rows x heads per key head) of a stream up to which the few-query kernel takes them
+constexpr int WATTN_LARGE_Q = 128;  // queries per tile of the many-query kernel
+inline int wattn_rows_per_tile(int group) { return WATTN_LARGE_Q / group > 0 ? WATTN_LARGE_Q / group : 1; }
+
+// Where the query tiles of a pass come from: a uniform pass (rows_per_seq rows of every stream) or device lists made for
+// the layer's group size by wattn_make_tiles.
+struct AttnBatch {
+    int rows = 0, rows_per_seq = 0;
+    const AttnTile *small = nullptr, *large = nullptr;  // device
+    int n_small = 0, n_large = 0, small_queries = 0;    // small_queries: most queries of a small tile
+    int max_len = 0;                                    // longest visible context (sizes the splits)
+};
+size_t wattn_scratch_bytes(const tsb_ctx* ctx);  // zeroed once by the owner; the kernels leave its tickets at zero
+bool wattn_supported(int head_dim, int group, bool f32);
+int wattn_pad_dim(int head_dim, bool f32);       // the head size the kernels work on (zero columns behind the real ones); 0: too large
+cudaError_t launch_window_attn(tsb_ctx* ctx, cudaStream_t st, bool f32, const WindowAttn& a, const AttnBatch& b, void* scratch);

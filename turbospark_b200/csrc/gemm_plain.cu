@@ -1,0 +1,592 @@
+// Matrix products with plain weights.  Three kernels:
+//
+//   plain_few_kernel   bfloat16, up to 32 token rows: bound by the weight stream.  A warp multiplies a tile of 16 (or
+//                      2 x 16) weight rows on mma.sync.m16n8k16 with the tokens as the N side; the warps of a CTA split
+//                      the columns and meet in shared memory.  The order of the columns inside a product is free as
+//                      long as both operands agree, so a lane's fragments are contiguous 16-byte pieces of natural
+//                      row-major rows: no repacking of weights or activations, no shared-memory staging.
+//   plain_tc_kernel    bfloat16, more rows: tcgen05 tensor cores.  128 weight rows (M) x up to 256 tokens (N) per tile;
+//                      a producer thread feeds 64-column slices of both operands through TMA into a ring of
+//                      128-byte-swizzled stages, one thread issues the MMAs into one of two tensor-memory accumulators,
+//                      four warps run the epilogue of the tile before.  Persistent CTAs; products with too few tiles to
+//                      fill the device are cut along K, the last run of a tile to finish adds the runs in order.
+//   plain_f32_kernel   f32 throughout (fused multiply-adds on the CUDA cores): the reference-precision mode.
+//
+// All three share the epilogues: residual add, logits with a soft cap, and the projection epilogue that stores queries,
+// writes keys straight into the paged cache, keeps the head gates in f32 and joins gate / up pairs.
+#include <cuda.h>
+
+#include <algorithm>
+#include <map>
+#include <mutex>
+
+#include "gemm_plain.cuh"
+#include "tc05.cuh"
+
+namespace {
+
+__device__ __forceinline__ void put(float* p, float v) { *p = v; }
+__device__ __forceinline__ void put(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+
+// act(z) in f32.  0.5 z (1 + tanh(u)) = z / (1 + exp(-2u)); the reduced-precision path takes the fast exponential and
+// division (relative error a few 2^-22), the f32 path the library's.
+template <typename T>
+__device__ __forceinline__ float activate(int act, float z) {
+    const float u = act == PLAIN_GELU_TANH ? 1.5957691216057308f * (z + 0.044715f * z * z * z) : z;  // 2 sqrt(2 / pi)
+    if (sizeof(T) == 4) {
+        if (act == PLAIN_GELU_TANH) return 0.5f * z * (1.f + tanhf(0.5f * u));
+        return z / (1.f + expf(-u));
+    }
+    return __fdividef(z, 1.f + __expf(-u));
+}
+
+template <typename T>
+__device__ __forceinline__ void epi_one(const PlainEpi& e, int t, int n, float v, uint32_t* err) {
+    if (e.kind == PLAIN_STORE) {
+        if (n < e.n_valid) e.y[(int64_t)t * e.y_stride + n] = e.cap > 0.f ? e.cap * tanhf(v / e.cap) : v;
+    } else if (e.kind == PLAIN_ADD) {
+        if (n < e.n_valid) e.y[(int64_t)t * e.y_stride + n] += v;
+    } else {
+        if (n < e.q_rows) {
+            put(static_cast<T*>(e.q) + (int64_t)t * e.q_stride + n, v);
+        } else if (n < e.q_rows + e.k_rows) {
+            const tsb_row_desc& rd = e.rows[t];
+            T* p = key_row<T>(e.keys, rd.seq, rd.base + rd.slot);
+            if (p) put(p + (n - e.q_rows), v);
+            else atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+        } else if (n < e.q_rows + e.k_rows + e.gate_rows) {
+            e.gate[(int64_t)t * e.gate_rows + (n - e.q_rows - e.k_rows)] = v;
+        }
+    }
+}
+template <typename T>
+__device__ __forceinline__ void epi_pair(const PlainEpi& e, int t, int pair, float g, float u) {
+    if (pair < e.n_pairs) put(static_cast<T*>(e.a) + (int64_t)t * e.a_stride + pair, activate<T>(e.act, g) * u);
+}
+
+// does any output come from the rows at and after row0 (up to the next segment)?
+__device__ __forceinline__ bool tile_used(const PlainEpi& e, int row0) {
+    if (row0 >= e.pair_row0) return (row0 - e.pair_row0) / 2 < e.n_pairs;
+    return row0 < (e.kind == PLAIN_MIXER ? e.q_rows + e.k_rows + e.gate_rows : e.n_valid);
+}
+
+// ------------------------------------------------------------------ few rows
+constexpr int FEW_WARPS = 8;
+constexpr int FEW_UNROLL = 4;  // 64-column units in flight per warp
+
+__device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+        : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+        : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ uint4 ldg_stream(const void* p) {
+    uint4 v;
+    asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+    return v;
+}
+
+// NT token tiles of eight, MT row tiles of sixteen.
+template <int NT, int MT>
+__global__ void __launch_bounds__(FEW_WARPS * 32, 2)
+    plain_few_kernel(const __nv_bfloat16* __restrict__ w, int cols, const __nv_bfloat16* x, const __nv_bfloat16* x2, int64_t x_stride, int tokens,
+                     const __grid_constant__ PlainEpi epi, uint32_t* __restrict__ err) {
+    constexpr int U = MT == 1 ? FEW_UNROLL : FEW_UNROLL / 2;
+    constexpr int TOK = NT * 8, ROWS = MT * 16;
+    __shared__ float red[FEW_WARPS][ROWS][TOK + 1];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
+    const int row0 = blockIdx.x * ROWS;
+    const int units = cols / 64;
+    const bool pairs = row0 >= epi.pair_row0;
+    if (!tile_used(epi, row0)) return;  // padding between the mixer's rows and the pairs
+    const __nv_bfloat16* wp = w + (int64_t)(row0 + g) * cols + 8 * t4;
+    // a unit of 64 columns is two k = 32 halves; per half the lane holds columns 8 t4 .. 8 t4 + 7 of its two rows
+    uint4 wa[U][MT][4];
+    auto load_w = [&](int i, int u) {
+#pragma unroll
+        for (int m = 0; m < MT; m++) {
+            const __nv_bfloat16* p = wp + (int64_t)m * 16 * cols + (int64_t)u * 64;
+            wa[i][m][0] = ldg_stream(p);
+            wa[i][m][1] = ldg_stream(p + (int64_t)8 * cols);
+            wa[i][m][2] = ldg_stream(p + 32);
+            wa[i][m][3] = ldg_stream(p + (int64_t)8 * cols + 32);
+        }
+    };
+#pragma unroll
+    for (int i = 0; i < U; i++)
+        if (warp + i * FEW_WARPS < units) load_w(i, warp + i * FEW_WARPS);  // weights do not depend on the preceding kernel
+    pdl_wait();
+    const __nv_bfloat16* xb = (pairs ? x2 : x) + (int64_t)g * x_stride + 8 * t4;
+    float acc[MT][NT][4];
+#pragma unroll
+    for (int m = 0; m < MT; m++)
+#pragma unroll
+        for (int n = 0; n < NT; n++)
+#pragma unroll
+            for (int i = 0; i < 4; i++) acc[m][n][i] = 0.f;
+    for (int u0 = warp; u0 < units; u0 += U * FEW_WARPS) {
+#pragma unroll
+        for (int i = 0; i < U; i++) {
+            const int u = u0 + i * FEW_WARPS;
+            if (u >= units) break;
+#pragma unroll
+            for (int n = 0; n < NT; n++) {
+                const __nv_bfloat16* xp = xb + (int64_t)n * 8 * x_stride + (int64_t)u * 64;
+                const uint4 b0 = *reinterpret_cast<const uint4*>(xp), b1 = *reinterpret_cast<const uint4*>(xp + 32);
+#pragma unroll
+                for (int m = 0; m < MT; m++) {
+                    const uint32_t a0[4] = {wa[i][m][0].x, wa[i][m][1].x, wa[i][m][0].y, wa[i][m][1].y};
+                    const uint32_t a1[4] = {wa[i][m][0].z, wa[i][m][1].z, wa[i][m][0].w, wa[i][m][1].w};
+                    const uint32_t a2[4] = {wa[i][m][2].x, wa[i][m][3].x, wa[i][m][2].y, wa[i][m][3].y};
+                    const uint32_t a3[4] = {wa[i][m][2].z, wa[i][m][3].z, wa[i][m][2].w, wa[i][m][3].w};
+                    mma_bf16(acc[m][n], a0, b0.x, b0.y);
+                    mma_bf16(acc[m][n], a1, b0.z, b0.w);
+                    mma_bf16(acc[m][n], a2, b1.x, b1.y);
+                    mma_bf16(acc[m][n], a3, b1.z, b1.w);
+                }
+            }
+            const int un = u + U * FEW_WARPS;
+            if (un < units) load_w(i, un);
+        }
+    }
+    pdl_launch_dependents();
+#pragma unroll
+    for (int m = 0; m < MT; m++)
+#pragma unroll
+        for (int n = 0; n < NT; n++) {
+            red[warp][m * 16 + g][n * 8 + 2 * t4] = acc[m][n][0];
+            red[warp][m * 16 + g][n * 8 + 2 * t4 + 1] = acc[m][n][1];
+            red[warp][m * 16 + g + 8][n * 8 + 2 * t4] = acc[m][n][2];
+            red[warp][m * 16 + g + 8][n * 8 + 2 * t4 + 1] = acc[m][n][3];
+        }
+    __syncthreads();
+    auto total = [&](int r, int t) {
+        float v = 0.f;
+#pragma unroll
+        for (int i = 0; i < FEW_WARPS; i++) v += red[i][r][t];
+        return v;
+    };
+    if (pairs) {
+        for (int i = threadIdx.x; i < ROWS / 2 * tokens; i += FEW_WARPS * 32) {
+            const int p = i % (ROWS / 2), t = i / (ROWS / 2);
+            const int r = (p >> 3) * 16 + (p & 7);
+            epi_pair<__nv_bfloat16>(epi, t, (row0 - epi.pair_row0) / 2 + p, total(r, t), total(r + 8, t));
+        }
+    } else {
+        for (int i = threadIdx.x; i < ROWS * tokens; i += FEW_WARPS * 32) {
+            const int r = i % ROWS, t = i / ROWS;
+            epi_one<__nv_bfloat16>(epi, t, row0 + r, total(r, t), err);
+        }
+    }
+}
+
+// ------------------------------------------------------------------ f32
+constexpr int F32_TILE = 64, F32_K = 16;
+// 256 threads, 64 rows x 64 tokens, 4 x 4 per thread.  A thread's four rows are {0, 8, 16, 24} + r within a 32-row half:
+// both halves of a gate / up pair are its own.
+__global__ void __launch_bounds__(256)
+    plain_f32_kernel(const float* __restrict__ w, int cols, const float* x, const float* x2, int64_t x_stride, int tokens,
+                     const __grid_constant__ PlainEpi epi, uint32_t* __restrict__ err) {
+    __shared__ float ws[F32_K][F32_TILE + 4], xs[F32_K][F32_TILE + 4];
+    const int row0 = blockIdx.x * F32_TILE, tok0 = blockIdx.y * F32_TILE;
+    const bool pairs = row0 >= epi.pair_row0;
+    const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
+    const int rbase = (ty >> 3) * 32 + (ty & 7);
+    pdl_wait();
+    const float* xb = pairs ? x2 : x;
+    float acc[4][4] = {};
+    const int lr = threadIdx.x >> 2, lc = (threadIdx.x & 3) * 4;
+    for (int k0 = 0; k0 < cols; k0 += F32_K) {
+        const float4 a = *reinterpret_cast<const float4*>(w + (int64_t)(row0 + lr) * cols + k0 + lc);
+        float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (tok0 + lr < tokens) b = *reinterpret_cast<const float4*>(xb + (int64_t)(tok0 + lr) * x_stride + k0 + lc);
+        ws[lc][lr] = a.x, ws[lc + 1][lr] = a.y, ws[lc + 2][lr] = a.z, ws[lc + 3][lr] = a.w;
+        xs[lc][lr] = b.x, xs[lc + 1][lr] = b.y, xs[lc + 2][lr] = b.z, xs[lc + 3][lr] = b.w;
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < F32_K; k++) {
+            float wv[4], xv[4];
+#pragma unroll
+            for (int i = 0; i < 4; i++) wv[i] = ws[k][rbase + 8 * i], xv[i] = xs[k][tx + 16 * i];
+#pragma unroll
+            for (int i = 0; i < 4; i++)
+#pragma unroll
+                for (int j = 0; j < 4; j++) acc[i][j] = fmaf(wv[i], xv[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+    pdl_launch_dependents();
+#pragma unroll
+    for (int j = 0; j < 4; j++) {
+        const int t = tok0 + tx + 16 * j;
+        if (t >= tokens) continue;
+        if (pairs) {
+#pragma unroll
+            for (int h = 0; h < 2; h++) {
+                const int r = row0 - epi.pair_row0 + (ty >> 3) * 32 + 16 * h;  // the pair group's first row
+                epi_pair<float>(epi, t, r / 2 + (ty & 7), acc[2 * h][j], acc[2 * h + 1][j]);
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < 4; i++) epi_one<float>(epi, t, row0 + rbase + 8 * i, acc[i][j], err);
+        }
+    }
+}
+
+// ------------------------------------------------------------------ tensor memory
+constexpr int TCG_M = 128;        // weight rows per tile
+constexpr int TCG_K = 64;         // columns per stage (128 bytes: one swizzle row)
+constexpr int TCG_NMAX = 256;     // tokens per tile
+constexpr int TCG_EPI_WARPS = 4;  // warp w owns tensor-memory lanes 32 w .. 32 w + 31
+constexpr int TCG_THREADS = (TCG_EPI_WARPS + 2) * 32;
+constexpr int TCG_HEADER = 1024;
+constexpr int TCG_MAX_STAGES = 8;
+constexpr int TCG_SMEM_CAP = 224 * 1024;
+constexpr int TCG_TICKETS = 4096;
+constexpr int TCG_MAX_SPLITS = 16;
+
+struct TcgBars {
+    uint64_t full[TCG_MAX_STAGES], empty[TCG_MAX_STAGES];
+    uint64_t acc_full[2], acc_empty[2];
+    uint32_t tmem_base, failed, ticket;
+};
+
+__device__ __forceinline__ void tcg_g2s_2d(uint32_t dst_smem, const CUtensorMap* map, int x, int y, uint64_t* bar) {
+    asm volatile("cp.async.bulk.tensor.2d.shared::cluster.global.tile.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3}], [%4];" ::"r"(dst_smem),
+                 "l"(reinterpret_cast<uint64_t>(map)), "r"(x), "r"(y), "r"(smem_u32(bar))
+                 : "memory");
+}
+
+// Work item i: token tile i % n_tok_tiles, then the K run, then the row tile - neighbouring CTAs share weight rows.
+__global__ void __launch_bounds__(TCG_THREADS, 1)
+    plain_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap xmap, const __grid_constant__ CUtensorMap x2map,
+                    int n_row_tiles, int n_tok_tiles, int units, int ksplit, int nt, int stages, int tokens,
+                    const __grid_constant__ PlainEpi epi, float* __restrict__ part, uint32_t* __restrict__ tickets, uint32_t* __restrict__ err) {
+    extern __shared__ __align__(1024) uint8_t smem[];
+    TcgBars* bars = reinterpret_cast<TcgBars*>(smem);
+    uint8_t* ring = smem + TCG_HEADER;
+    const int stage_bytes = (TCG_M + nt) * 128;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int n_items = n_row_tiles * n_tok_tiles * ksplit;
+    const int run_units = (units + ksplit - 1) / ksplit;
+    const uint32_t tmem_cols = nt <= 16 ? 32u : nt <= 32 ? 64u : nt <= 64 ? 128u : nt <= 128 ? 256u : 512u;
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < stages; i++) mbar_init(&bars->full[i], 1), mbar_init(&bars->empty[i], 1);
+        for (int i = 0; i < 2; i++) mbar_init(&bars->acc_full[i], 1), mbar_init(&bars->acc_empty[i], TCG_EPI_WARPS);
+        bars->failed = 0;
+        mbar_fence_init();
+    }
+    if (warp == TCG_EPI_WARPS + 1) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&bars->tmem_base)), "r"(tmem_cols) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = bars->tmem_base;
+    struct Item {
+        int tok, run, row, u0, n;
+    };
+    auto item_of = [&](int i) {
+        Item it;
+        it.tok = i % n_tok_tiles;
+        it.run = (i / n_tok_tiles) % ksplit;
+        it.row = i / n_tok_tiles / ksplit;
+        it.u0 = it.run * run_units;
+        it.n = min(units, it.u0 + run_units) - it.u0;
+        return it;
+    };
+
+    if (warp == TCG_EPI_WARPS) {
+        if (lane == 0) {
+            // ---- producer.  Weights do not depend on the preceding kernel, activations do: the first stages' weight
+            // slices start before the wait, their activation slices after it.
+            bool ok = true;
+            uint32_t it = 0;
+            int early = 0;  // stages whose weight slice was fetched ahead
+            const bool has_work = (int)blockIdx.x < n_items;
+            if (has_work) {
+                const Item w0 = item_of(blockIdx.x);
+                early = min(stages, w0.n);
+                for (int s = 0; s < early; s++) {
+                    mbar_expect_tx(&bars->full[s], (uint32_t)stage_bytes);
+                    tcg_g2s_2d(smem_u32(ring + s * stage_bytes), &wmap, (w0.u0 + s) * TCG_K, w0.row * TCG_M, &bars->full[s]);
+                }
+            }
+            pdl_wait();
+            for (int i = blockIdx.x; i < n_items && ok; i += gridDim.x) {
+                const Item w = item_of(i);
+                const CUtensorMap* xm = w.row * TCG_M >= epi.pair_row0 ? &x2map : &xmap;
+                for (int u = 0; u < w.n && ok; u++, it++) {
+                    const int s = it % stages;
+                    const uint32_t dst = smem_u32(ring + s * stage_bytes);
+                    if ((int)it >= early) {
+                        if ((int)it >= stages) ok = mbar_wait(&bars->empty[s], ((it / stages) - 1) & 1, err);
+                        if (!ok) break;
+                        mbar_expect_tx(&bars->full[s], (uint32_t)stage_bytes);
+                        tcg_g2s_2d(dst, &wmap, (w.u0 + u) * TCG_K, w.row * TCG_M, &bars->full[s]);
+                    }
+                    tcg_g2s_2d(dst + TCG_M * 128, xm, (w.u0 + u) * TCG_K, w.tok * nt, &bars->full[s]);
+                }
+            }
+            if (!ok) bars->failed = 1;
+            // no copy is in flight when the CTA leaves, also when another role has given up
+            for (uint32_t k = it > (uint32_t)stages ? it - stages : 0; k < it; k++) mbar_wait(&bars->full[k % stages], (k / stages) & 1, err);
+        }
+    } else if (warp == TCG_EPI_WARPS + 1) {
+        // ---- MMA issue: the warp walks the items together, lane 0 issues.  f32 accumulate, bfloat16 operands, both
+        // K-major and 128-byte swizzled (eight-row groups 1024 bytes apart; a K = 16 step moves the start by 32 bytes)
+        const uint32_t leader = lane == 0 ? 1u : 0u;
+        const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(nt >> 3) << 17) | ((uint32_t)(TCG_M >> 4) << 24);
+        constexpr uint64_t DESC = ((uint64_t)1u << 16) | ((uint64_t)(1024u >> 4) << 32) | (1ull << 46) | (2ull << 61);
+        bool ok = true;
+        uint32_t it = 0, tile = 0;
+        for (int i = blockIdx.x; i < n_items && ok; i += gridDim.x, tile++) {
+            const Item w = item_of(i);
+            const uint32_t buf = tile & 1;
+            if (tile >= 2) ok = __all_sync(0xffffffffu, mbar_wait(&bars->acc_empty[buf], ((tile >> 1) - 1) & 1, err));
+            if (!ok) break;
+            tc_fence_after();
+            const uint32_t d = tmem + buf * (uint32_t)nt;
+            for (int u = 0; u < w.n; u++, it++) {
+                const int s = it % stages;
+                ok = __all_sync(0xffffffffu, mbar_wait(&bars->full[s], (it / stages) & 1, err));
+                if (!ok) break;
+                tc_fence_after();
+                const uint32_t a_addr = smem_u32(ring + s * stage_bytes);
+                const uint64_t da = DESC | (uint64_t)((a_addr >> 4) & 0x3FFFu);
+                const uint64_t db = DESC | (uint64_t)(((a_addr + TCG_M * 128) >> 4) & 0x3FFFu);
+                if (u == 0) tc_mma_ss<false>(leader, d, da, db, idesc);
+                else tc_mma_ss<true>(leader, d, da, db, idesc);
+#pragma unroll
+                for (int ks = 1; ks < TCG_K / 16; ks++) tc_mma_ss<true>(leader, d, da + 2u * ks, db + 2u * ks, idesc);
+                tc_commit_if(leader, &bars->empty[s]);
+            }
+            if (ok) tc_commit_if(leader, &bars->acc_full[buf]);
+        }
+        if (!ok && lane == 0) bars->failed = 1;
+    } else {
+        // ---- epilogue: thread = weight row of the tile, columns = tokens
+        pdl_wait();  // the residual stream and the cache belong to earlier kernels too
+        bool ok = true;
+        uint32_t tile = 0;
+        const uint32_t lane_base = (uint32_t)(warp * 32) << 16;
+        for (int i = blockIdx.x; i < n_items; i += gridDim.x, tile++) {
+            const Item w = item_of(i);
+            const uint32_t buf = tile & 1;
+            if (ok) ok = mbar_wait(&bars->acc_full[buf], (tile >> 1) & 1, err);
+            tc_fence_after();
+            const uint32_t src = tmem + lane_base + buf * (uint32_t)nt;
+            const int n = w.row * TCG_M + warp * 32 + lane;
+            const int tok0 = w.tok * nt, n_tok = min(nt, tokens - tok0);
+            const bool pairs = w.row * TCG_M >= epi.pair_row0;
+            auto finish16 = [&](int c0, const float (&v)[16]) {  // sixteen tokens of this row
+                if (pairs) {
+                    const int pair = (w.row * TCG_M - epi.pair_row0 + warp * 32) / 2 + (lane >> 4) * 8 + (lane & 7);
+#pragma unroll
+                    for (int j = 0; j < 16; j++) {
+                        const float up = __shfl_down_sync(0xffffffffu, v[j], 8);
+                        if (!(lane & 8) && c0 + j < n_tok) epi_pair<__nv_bfloat16>(epi, tok0 + c0 + j, pair, v[j], up);
+                    }
+                } else if (epi.kind == PLAIN_ADD) {
+                    // the loads of sixteen tokens are in flight together
+                    float old[16];
+                    const bool in = n < epi.n_valid;
+                    float* y = epi.y + (int64_t)(tok0 + c0) * epi.y_stride + n;
+#pragma unroll
+                    for (int j = 0; j < 16; j++) old[j] = in && c0 + j < n_tok ? y[(int64_t)j * epi.y_stride] : 0.f;
+#pragma unroll
+                    for (int j = 0; j < 16; j++)
+                        if (in && c0 + j < n_tok) y[(int64_t)j * epi.y_stride] = old[j] + v[j];
+                } else {
+#pragma unroll
+                    for (int j = 0; j < 16; j++)
+                        if (c0 + j < n_tok) epi_one<__nv_bfloat16>(epi, tok0 + c0 + j, n, v[j], err);
+                }
+            };
+            if (ksplit == 1) {
+                for (int c0 = 0; c0 < n_tok; c0 += 16) {
+                    uint32_t r[16];
+                    tc_ld16(src + c0, r);
+                    tc_wait_ld();
+                    float v[16];
+#pragma unroll
+                    for (int j = 0; j < 16; j++) v[j] = __uint_as_float(r[j]);
+                    if (ok) finish16(c0, v);
+                }
+                tc_fence_before();
+                __syncwarp();
+                if (lane == 0) mbar_arrive(&bars->acc_empty[buf]);
+            } else {
+                // a run of a cut tile: leave the sums, take a ticket; whoever takes the last one adds the runs in order
+                const int tix = w.row * n_tok_tiles + w.tok;
+                float* mine = part + ((int64_t)tix * ksplit + w.run) * (TCG_M * nt);
+                for (int c0 = 0; c0 < n_tok; c0 += 16) {
+                    uint32_t r[16];
+                    tc_ld16(src + c0, r);
+                    tc_wait_ld();
+#pragma unroll
+                    for (int j = 0; j < 16; j++) mine[(int64_t)(c0 + j) * TCG_M + warp * 32 + lane] = ok ? __uint_as_float(r[j]) : 0.f;
+                }
+                tc_fence_before();
+                __syncwarp();
+                if (lane == 0) mbar_arrive(&bars->acc_empty[buf]);
+                __threadfence();
+                asm volatile("bar.sync 1, %0;" ::"n"(TCG_EPI_WARPS * 32) : "memory");
+                if (threadIdx.x == 0) {
+                    const uint32_t t = atomicAdd(&tickets[tix], 1u);
+                    if (t == (uint32_t)ksplit - 1) tickets[tix] = 0;
+                    bars->ticket = t;
+                }
+                asm volatile("bar.sync 1, %0;" ::"n"(TCG_EPI_WARPS * 32) : "memory");
+                if (bars->ticket == (uint32_t)ksplit - 1) {
+                    __threadfence();
+                    const float* all = part + (int64_t)tix * ksplit * (TCG_M * nt);
+                    for (int c0 = 0; c0 < n_tok; c0 += 16) {
+                        float v[16];
+#pragma unroll
+                        for (int j = 0; j < 16; j++) v[j] = 0.f;
+                        for (int k = 0; k < ksplit; k++) {
+                            float p[16];
+#pragma unroll
+                            for (int j = 0; j < 16; j++) p[j] = __ldcg(all + (int64_t)k * (TCG_M * nt) + (int64_t)(c0 + j) * TCG_M + warp * 32 + lane);
+#pragma unroll
+                            for (int j = 0; j < 16; j++) v[j] += p[j];
+                        }
+                        finish16(c0, v);
+                    }
+                }
+                asm volatile("bar.sync 1, %0;" ::"n"(TCG_EPI_WARPS * 32) : "memory");  // the ticket word is reused by the next tile
+            }
+        }
+        if (!ok && lane == 0) bars->failed = 1;
+    }
+    pdl_launch_dependents();
+    tc_fence_before();
+    __syncthreads();
+    if (warp == TCG_EPI_WARPS + 1) {
+        tc_fence_after();
+        asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(tmem_cols) : "memory");
+    }
+}
+
+// 2-D bfloat16 tensor map over [rows][cols], box 64 columns x box_rows rows, 128-byte swizzle.  Encoding goes through the
+// driver entry point (no link against libcuda); maps are kept per (address, shape).
+cudaError_t tcg_map(const void* p, int64_t rows, int64_t cols, int64_t stride, int box_rows, CUtensorMap* out) {
+    typedef CUresult (*EncodeFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
+                                 const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+    static std::mutex mu;
+    static EncodeFn encode = nullptr;
+    struct Key {
+        const void* p;
+        int64_t rows, cols, stride;
+        int box;
+        bool operator<(const Key& o) const {
+            return p != o.p ? p < o.p : rows != o.rows ? rows < o.rows : cols != o.cols ? cols < o.cols : stride != o.stride ? stride < o.stride : box < o.box;
+        }
+    };
+    static std::map<Key, CUtensorMap> cache;
+    std::lock_guard<std::mutex> lock(mu);
+    if (!encode) {
+        void* fn = nullptr;
+        cudaDriverEntryPointQueryResult qres;
+        cudaError_t e = cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &fn, cudaEnableDefault, &qres);
+        if (e != cudaSuccess) return e;
+        if (!fn || qres != cudaDriverEntryPointSuccess) return cudaErrorNotSupported;
+        encode = reinterpret_cast<EncodeFn>(fn);
+    }
+    const Key key{p, rows, cols, stride, box_rows};
+    auto it = cache.find(key);
+    if (it == cache.end()) {
+        if (cache.size() > 8192) cache.clear();
+        CUtensorMap m;
+        const cuuint64_t gdim[2] = {(cuuint64_t)cols, (cuuint64_t)rows};
+        const cuuint64_t gstride[1] = {(cuuint64_t)stride * 2};
+        const cuuint32_t box[2] = {(cuuint32_t)TCG_K, (cuuint32_t)box_rows};
+        const cuuint32_t estride[2] = {1, 1};
+        if (encode(&m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(p), gdim, gstride, box, estride, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                   CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
+            return cudaErrorInvalidValue;
+        it = cache.emplace(key, m).first;
+    }
+    *out = it->second;
+    return cudaSuccess;
+}
+
+// How a product is cut: the token tile (32 .. 256 columns) and the number of K runs whose estimated time is least.  Time
+// in units of a 64-column step of the tensor pipe: an instruction costs at least a quarter of the N = 256 one's... a step
+// is bound by the MMA (proportional to the columns, 128 at the least) or by its bytes; each item adds a fixed cost and a
+// cut tile writes and reads its sums.
+struct TcgPlan {
+    int nt, ksplit, stages;
+};
+TcgPlan tcg_plan(const tsb_ctx* ctx, int row_tiles, int units, int tokens) {
+    TcgPlan best{256, 1, 4};
+    float best_cost = 1e30f;
+    const int sms = ctx->sm_count > 0 ? ctx->sm_count : 148;
+    for (int nt : {32, 64, 128, 256}) {
+        const int tok_tiles = (tokens + nt - 1) / nt;
+        if (nt > 32 && nt / 2 >= tokens) continue;  // half of the tile would stand empty
+        for (int ks = 1; ks <= TCG_MAX_SPLITS && ks <= units; ks++) {
+            const int run = (units + ks - 1) / ks;
+            if ((units + run - 1) / run != ks) continue;  // no empty runs
+            if (ks > 1 && row_tiles * tok_tiles > TCG_TICKETS) continue;
+            if (ks > 1 && (int64_t)row_tiles * tok_tiles * ks > 2 * sms) break;
+            const float step = std::max(nt <= 128 ? 0.75f : 1.f, (128.f + nt) / 384.f * 1.1f);
+            const float item = run * step + 6.f + (ks > 1 ? nt / 16.f * (1.f + 0.5f * ks) : nt / 64.f);
+            const int waves = (row_tiles * tok_tiles * ks + sms - 1) / sms;
+            const float cost = waves * item;
+            if (cost < best_cost - 1e-3f) best_cost = cost, best.nt = nt, best.ksplit = ks;
+        }
+    }
+    best.stages = std::min(TCG_MAX_STAGES, (TCG_SMEM_CAP - TCG_HEADER) / ((TCG_M + best.nt) * 128));
+    return best;
+}
+
+template <int NT, int MT>
+cudaError_t launch_few(tsb_ctx* ctx, cudaStream_t st, const PlainMat& w, const __nv_bfloat16* x, const __nv_bfloat16* x2, int64_t x_stride, int tokens,
+                       const PlainEpi& epi) {
+    return tsb_launch(ctx, plain_few_kernel<NT, MT>, dim3((unsigned)(w.rows / (16 * MT))), dim3(FEW_WARPS * 32), 0, st, true,
+                      (const __nv_bfloat16*)w.data, (int)w.cols, x, x2, x_stride, tokens, epi, ctx->dev_error);
+}
+
+constexpr int FEW_MAX = 32;  // token rows up to which the weight-streaming kernel runs
+
+}  // namespace
+
+size_t plain_gemm_workspace_bytes(const tsb_ctx* ctx) {
+    const int sms = ctx->sm_count > 0 ? ctx->sm_count : 148;
+    return TCG_TICKETS * sizeof(uint32_t) + (size_t)(2 * sms) * TCG_M * TCG_NMAX * sizeof(float);
+}
+
+cudaError_t launch_plain_gemm(tsb_ctx* ctx, cudaStream_t st, bool f32, const PlainMat& w, const void* x, const void* x2, int64_t x_stride, int x_rows,
+                              int tokens, const PlainEpi& epi, void* workspace) {
+    if (tokens <= 0) return cudaSuccess;
+    if (f32) {
+        dim3 grid((unsigned)(w.rows / F32_TILE), (unsigned)((tokens + F32_TILE - 1) / F32_TILE));
+        return tsb_launch(ctx, plain_f32_kernel, grid, dim3(256), 0, st, true, (const float*)w.data, (int)w.cols, (const float*)x, (const float*)x2,
+                          x_stride, tokens, epi, ctx->dev_error);
+    }
+    const __nv_bfloat16 *xb = (const __nv_bfloat16*)x, *xb2 = (const __nv_bfloat16*)x2;
+    if (tokens <= FEW_MAX) {
+        const bool two = w.rows / 32 >= 4 * ctx->sm_count;  // two row tiles per CTA halve the activation reads when there are rows enough
+        if (tokens <= 8) return two ? launch_few<1, 2>(ctx, st, w, xb, xb2, x_stride, tokens, epi) : launch_few<1, 1>(ctx, st, w, xb, xb2, x_stride, tokens, epi);
+        if (tokens <= 16) return two ? launch_few<2, 2>(ctx, st, w, xb, xb2, x_stride, tokens, epi) : launch_few<2, 1>(ctx, st, w, xb, xb2, x_stride, tokens, epi);
+        return two ? launch_few<4, 2>(ctx, st, w, xb, xb2, x_stride, tokens, epi) : launch_few<4, 1>(ctx, st, w, xb, xb2, x_stride, tokens, epi);
+    }
+    const int row_tiles = (int)(w.rows / TCG_M), units = (int)(w.cols / TCG_K);
+    const TcgPlan p = tcg_plan(ctx, row_tiles, units, tokens);
+    CUtensorMap wm, xm, xm2;
+    cudaError_t e = tcg_map(w.data, w.rows, w.cols, w.cols, TCG_M, &wm);
+    if (e == cudaSuccess) e = tcg_map(x, x_rows, w.cols, x_stride, p.nt, &xm);
+    if (e == cudaSuccess) e = tcg_map(x2 ? x2 : x, x_rows, w.cols, x_stride, p.nt, &xm2);
+    if (e != cudaSuccess) return e;
+    static SmemOptIn configured;
+    if ((e = tsb_opt_in_smem(ctx, plain_tc_kernel, (size_t)TCG_SMEM_CAP, configured)) != cudaSuccess) return e;
+    const int tok_tiles = (tokens + p.nt - 1) / p.nt;
+    const int items = row_tiles * tok_tiles * p.ksplit;
+    uint32_t* tickets = static_cast<uint32_t*>(workspace);
+    float* part = reinterpret_cast<float*>(tickets + TCG_TICKETS);
+    const size_t smem = TCG_HEADER + (size_t)p.stages * (TCG_M + p.nt) * 128;
+    return tsb_launch(ctx, plain_tc_kernel, dim3((unsigned)std::min(items, ctx->sm_count)), dim3(TCG_THREADS), smem, st, true, wm, xm, xm2, row_tiles,
+                      tok_tiles, units, p.ksplit, p.nt, p.stages, tokens, epi, part, tickets, ctx->dev_error);
+}

@@ -4,6 +4,8 @@
 #include <cstring>
 #include <new>
 
+#include <cuda_bf16.h>
+
 #include "kv.cuh"
 
 namespace {
@@ -113,13 +115,121 @@ __global__ void kv_fill_random_kernel(KvView kv, int seq, int tokens, uint64_t s
     }
 }
 
+__global__ void keys_fill_random_kernel(KeyView kv, int seq, int tokens, uint32_t seed) {
+    const int row = kv.kv_heads * kv.head_dim;
+    const int64_t total = (int64_t)tokens * row;
+    for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
+        const int pos = (int)(i / row), e = (int)(i - (int64_t)pos * row);
+        uint32_t h = hash32((uint32_t)i * 0x9E3779B9u + seed) ^ hash32((uint32_t)(i >> 32) + seed);
+        float acc = 0.f;
+#pragma unroll
+        for (int k = 0; k < 4; k++) {
+            h = hash32(h + 0x9E3779B9u * (k + 1));
+            acc += (float)(h >> 8) * (1.0f / 16777216.0f);
+        }
+        const float v = (acc - 2.0f) * 1.7320508f;
+        if (kv.elem_bytes == 4) {
+            if (float* p = key_row<float>(kv, seq, pos)) p[e] = v;
+        } else {
+            if (__nv_bfloat16* p = key_row<__nv_bfloat16>(kv, seq, pos)) p[e] = __float2bfloat16_rn(v);
+        }
+    }
+}
+
 int32_t kv_check(tsb_kv* kv, int32_t seq) {
     if (!kv) return TSB_ERR_INVALID;
     if (seq < 0 || seq >= kv->view.max_seqs) return tsb_fail(kv->ctx, TSB_ERR_INVALID, "stream %d outside 0..%d", seq, kv->view.max_seqs);
     return TSB_OK;
 }
 
+// page tables, free list and cursors, shared by both kinds of cache
+int32_t kv_init_pages(tsb_ctx* ctx, tsb_kv* kv, int page_tokens, int num_pages, int max_seqs, int max_pages_per_seq) {
+    kv->ctx = ctx;
+    KvView& v = kv->view;
+    v.page_tokens = page_tokens;
+    v.page_shift = 0;
+    while ((1 << v.page_shift) < page_tokens) v.page_shift++;
+    v.num_pages = num_pages, v.max_seqs = max_seqs, v.max_pages_per_seq = max_pages_per_seq;
+    const size_t pt = (size_t)max_seqs * max_pages_per_seq;
+    kv->page_table_host.assign(pt, -1);
+    cudaError_t e = cudaMalloc((void**)&kv->page_table_dev, pt * sizeof(int32_t));
+    if (e == cudaSuccess) e = cudaMemset(kv->page_table_dev, 0xFF, pt * sizeof(int32_t));
+    if (e != cudaSuccess) {
+        cudaGetLastError();
+        return tsb_fail(ctx, TSB_ERR_CUDA, "page table: %s", cudaGetErrorString(e));
+    }
+    v.page_table = kv->page_table_dev;
+    kv->free_pages.resize(num_pages);
+    for (int i = 0; i < num_pages; i++) kv->free_pages[i] = num_pages - 1 - i;  // pop_back hands out page 0 first
+    kv->pages_of_seq.assign(max_seqs, 0);
+    kv->cursor.assign(max_seqs, 0);
+    kv->state_lo.assign(max_seqs, 0);
+    return TSB_OK;
+}
+
+int32_t pool_alloc(tsb_ctx* ctx, size_t bytes, void** out) {
+    cudaError_t e = cudaMalloc(out, bytes);
+    if (e != cudaSuccess) {
+        cudaGetLastError();
+        return tsb_fail(ctx, TSB_ERR_OOM, "K/V pool of %zu bytes: %s", bytes, cudaGetErrorString(e));
+    }
+    // rows nobody has written yet are read by kernels that fetch whole pages (and mask them): they must hold finite values
+    e = cudaMemset(*out, 0, bytes);
+    if (e != cudaSuccess) {
+        cudaFree(*out);
+        *out = nullptr;
+        return tsb_fail(ctx, TSB_ERR_CUDA, "clearing the K/V pool: %s", cudaGetErrorString(e));
+    }
+    return TSB_OK;
+}
+
 }  // namespace
+
+int32_t kv_create_keys(tsb_ctx* ctx, int n_layers, const int32_t* kv_heads, const int32_t* head_dims, int elem_bytes, int page_tokens, int num_pages,
+                       int max_seqs, int max_pages_per_seq, tsb_kv** out) {
+    *out = nullptr;
+    TSB_REQUIRE(ctx, n_layers > 0 && num_pages > 0 && max_seqs > 0 && max_pages_per_seq > 0, "bad sizes");
+    TSB_REQUIRE(ctx, elem_bytes == 2 || elem_bytes == 4, "keys are bfloat16 or f32");
+    TSB_REQUIRE(ctx, page_tokens >= 16 && (page_tokens & (page_tokens - 1)) == 0, "page_tokens must be a power of two >= 16");
+    DeviceGuard g(ctx);
+    tsb_kv* kv = new (std::nothrow) tsb_kv();
+    if (!kv) return TSB_ERR_OOM;
+    int32_t rc = kv_init_pages(ctx, kv, page_tokens, num_pages, max_seqs, max_pages_per_seq);
+    size_t bytes = 0;
+    for (int l = 0; l < n_layers && rc == TSB_OK; l++) {
+        if (kv_heads[l] <= 0 || head_dims[l] <= 0 || (head_dims[l] * elem_bytes) % 16)
+            rc = tsb_fail(ctx, TSB_ERR_INVALID, "layer %d: bad head count or head size", l);
+        bytes += (size_t)num_pages * page_tokens * kv_heads[l] * head_dims[l] * elem_bytes;
+    }
+    if (rc == TSB_OK) rc = pool_alloc(ctx, bytes, (void**)&kv->key_pool);
+    if (rc) {
+        tsb_kv_destroy(kv);
+        return rc;
+    }
+    kv->view.layers = n_layers;
+    size_t off = 0;
+    for (int l = 0; l < n_layers; l++) {
+        KeyView k;
+        k.base = kv->key_pool + off, k.page_table = kv->page_table_dev;
+        k.kv_heads = kv_heads[l], k.head_dim = head_dims[l], k.elem_bytes = elem_bytes;
+        k.page_shift = kv->view.page_shift, k.page_tokens = page_tokens, k.num_pages = num_pages;
+        k.max_seqs = max_seqs, k.max_pages_per_seq = max_pages_per_seq;
+        kv->key_layers.push_back(k);
+        off += (size_t)num_pages * page_tokens * kv_heads[l] * head_dims[l] * elem_bytes;
+    }
+    *out = kv;
+    return TSB_OK;
+}
+
+int32_t kv_fill_keys(tsb_kv* kv, cudaStream_t st, int32_t seq, int64_t tokens, uint64_t seed) {
+    int32_t rc = tsb_kv_reserve(kv, seq, tokens);
+    if (rc) return rc;
+    DeviceGuard g(kv->ctx);
+    for (size_t l = 0; l < kv->key_layers.size(); l++)
+        TSB_CUDA(kv->ctx, tsb_launch(kv->ctx, keys_fill_random_kernel, dim3((unsigned)(kv->ctx->sm_count * 4)), dim3(256), 0, st, false, kv->key_layers[l],
+                                     (int)seq, (int)tokens, (uint32_t)(seed * 1000003u + l)));
+    return TSB_OK;
+}
 
 cudaError_t launch_rope_store_kv(tsb_ctx* ctx, cudaStream_t st, tsb_kv* kv, int layer, __half* qkv,
                                  const tsb_row_desc* rows_dev, int rows, int n_q_heads, float theta) {
@@ -139,43 +249,16 @@ int32_t tsb_kv_create(tsb_ctx* ctx, int32_t layers, int32_t kv_heads, int32_t he
     DeviceGuard g(ctx);
     tsb_kv* kv = new (std::nothrow) tsb_kv();
     if (!kv) return TSB_ERR_OOM;
-    kv->ctx = ctx;
     KvView& v = kv->view;
     v.layers = layers, v.kv_heads = kv_heads, v.head_dim = head_dim;
-    v.page_tokens = page_tokens;
-    v.page_shift = 0;
-    while ((1 << v.page_shift) < page_tokens) v.page_shift++;
-    v.num_pages = num_pages, v.max_seqs = max_seqs, v.max_pages_per_seq = max_pages_per_seq;
     v.kv_stride = (int64_t)num_pages * page_tokens * kv_heads * head_dim;
     v.layer_stride = 2 * v.kv_stride;
-    const size_t pool_bytes = (size_t)layers * v.layer_stride * sizeof(__half);
-    cudaError_t e = cudaMalloc((void**)&v.pool, pool_bytes);
-    if (e != cudaSuccess) {
-        cudaGetLastError();
-        delete kv;
-        return tsb_fail(ctx, TSB_ERR_OOM, "K/V pool of %zu bytes: %s", pool_bytes, cudaGetErrorString(e));
+    int32_t rc = kv_init_pages(ctx, kv, page_tokens, num_pages, max_seqs, max_pages_per_seq);
+    if (rc == TSB_OK) rc = pool_alloc(ctx, (size_t)layers * v.layer_stride * sizeof(__half), (void**)&v.pool);
+    if (rc) {
+        tsb_kv_destroy(kv);
+        return rc;
     }
-    // rows nobody has written yet are read by kernels that fetch whole pages (and mask them): they must hold finite values
-    e = cudaMemset(v.pool, 0, pool_bytes);
-    if (e != cudaSuccess) {
-        cudaFree(v.pool);
-        delete kv;
-        return tsb_fail(ctx, TSB_ERR_CUDA, "clearing the K/V pool: %s", cudaGetErrorString(e));
-    }
-    const size_t pt = (size_t)max_seqs * max_pages_per_seq;
-    kv->page_table_host.assign(pt, -1);
-    e = cudaMalloc((void**)&kv->page_table_dev, pt * sizeof(int32_t));
-    if (e == cudaSuccess) e = cudaMemset(kv->page_table_dev, 0xFF, pt * sizeof(int32_t));
-    if (e != cudaSuccess) {
-        cudaFree(v.pool);
-        delete kv;
-        return tsb_fail(ctx, TSB_ERR_CUDA, "page table: %s", cudaGetErrorString(e));
-    }
-    v.page_table = kv->page_table_dev;
-    kv->free_pages.resize(num_pages);
-    for (int i = 0; i < num_pages; i++) kv->free_pages[i] = num_pages - 1 - i;  // pop_back hands out page 0 first
-    kv->pages_of_seq.assign(max_seqs, 0);
-    kv->cursor.assign(max_seqs, 0);
     *out = kv;
     return TSB_OK;
 }
@@ -185,6 +268,7 @@ void tsb_kv_destroy(tsb_kv* kv) {
     DeviceGuard g(kv->ctx);
     cudaDeviceSynchronize();
     cudaFree(kv->view.pool);
+    cudaFree(kv->key_pool);
     cudaFree(kv->page_table_dev);
     delete kv;
 }
@@ -227,6 +311,7 @@ int32_t tsb_kv_reset(tsb_kv* kv, int32_t seq) {
     }
     kv->pages_of_seq[seq] = 0;
     kv->cursor[seq] = 0;
+    kv->state_lo[seq] = 0;
     if (have)
         TSB_CUDA(ctx, cudaMemcpy(kv->page_table_dev + (size_t)seq * v.max_pages_per_seq, row, (size_t)have * sizeof(int32_t),
                                  cudaMemcpyHostToDevice));
@@ -244,6 +329,13 @@ int32_t tsb_kv_set_cursor(tsb_kv* kv, int32_t seq, int64_t position) {
     if (position < 0 || position > (int64_t)kv->pages_of_seq[seq] * kv->view.page_tokens)
         return tsb_fail(kv->ctx, TSB_ERR_STATE, "cursor %lld outside the reserved %lld positions", (long long)position,
                         (long long)kv->pages_of_seq[seq] * kv->view.page_tokens);
+    if (kv->state_ring > 0) {
+        if (position != 0 && position < kv->cursor[seq] && position - 1 < kv->state_lo[seq])
+            return tsb_fail(kv->ctx, TSB_ERR_STATE, "cursor %lld: the row state before it is gone (kept from position %lld)", (long long)position,
+                            (long long)kv->state_lo[seq]);
+        if (position == 0) kv->state_lo[seq] = 0;
+        kv->state_lo[seq] = std::max<int64_t>(kv->state_lo[seq], position - (kv->state_ring - 1));
+    }
     kv->cursor[seq] = position;
     return TSB_OK;
 }
@@ -253,8 +345,7 @@ int32_t tsb_kv_rewind_by(tsb_kv* kv, int32_t seq, int64_t count) {
     if (rc) return rc;
     if (count < 0 || count > kv->cursor[seq])
         return tsb_fail(kv->ctx, TSB_ERR_STATE, "cannot rewind %lld rows from cursor %lld", (long long)count, (long long)kv->cursor[seq]);
-    kv->cursor[seq] -= count;
-    return TSB_OK;
+    return tsb_kv_set_cursor(kv, seq, kv->cursor[seq] - count);
 }
 
 static int32_t kv_copy_rows(tsb_kv* kv, tsb_stream s, int32_t seq, int32_t layer, int64_t pos0, int32_t n, void* hk, void* hv,
@@ -263,24 +354,28 @@ static int32_t kv_copy_rows(tsb_kv* kv, tsb_stream s, int32_t seq, int32_t layer
     if (rc) return rc;
     tsb_ctx* ctx = kv->ctx;
     const KvView& v = kv->view;
-    TSB_REQUIRE(ctx, layer >= 0 && layer < v.layers && n >= 0 && pos0 >= 0 && hk && hv, "bad arguments");
+    const bool keys = !kv->key_layers.empty();
+    TSB_REQUIRE(ctx, layer >= 0 && layer < v.layers && n >= 0 && pos0 >= 0 && hk && (keys || hv), "bad arguments");
     if (pos0 + n > (int64_t)kv->pages_of_seq[seq] * v.page_tokens)
         return tsb_fail(ctx, TSB_ERR_STATE, "rows %lld..%lld are not reserved", (long long)pos0, (long long)(pos0 + n));
     DeviceGuard g(ctx);
-    const size_t row = (size_t)v.kv_heads * v.head_dim;
+    // bytes of a row, and where the layer's K and V halves start (a key-only cache has one half)
+    const KeyView* kl = keys ? &kv->key_layers[layer] : nullptr;
+    const size_t row = keys ? (size_t)kl->kv_heads * kl->head_dim * kl->elem_bytes : (size_t)v.kv_heads * v.head_dim * sizeof(__half);
     const int32_t* pt = &kv->page_table_host[(size_t)seq * v.max_pages_per_seq];
     int64_t p = pos0;
     while (p < pos0 + n) {  // one copy per page run
         const int64_t in_page = p & (v.page_tokens - 1);
         const int64_t run = std::min<int64_t>(v.page_tokens - in_page, pos0 + n - p);
         const int64_t slot = (int64_t)pt[p >> v.page_shift] * v.page_tokens + in_page;
-        for (int which = 0; which < 2; which++) {
-            __half* dev = v.pool + (int64_t)layer * v.layer_stride + (int64_t)which * v.kv_stride + slot * (int64_t)row;
-            char* host = (char*)(which ? hv : hk) + (size_t)(p - pos0) * row * sizeof(__half);
+        for (int which = 0; which < (keys ? 1 : 2); which++) {
+            char* half = keys ? (char*)kl->base : (char*)(v.pool + (int64_t)layer * v.layer_stride + (int64_t)which * v.kv_stride);
+            char* dev = half + slot * (int64_t)row;
+            char* host = (char*)(which ? hv : hk) + (size_t)(p - pos0) * row;
             if (to_device)
-                TSB_CUDA(ctx, cudaMemcpyAsync(dev, host, (size_t)run * row * sizeof(__half), cudaMemcpyHostToDevice, (cudaStream_t)s));
+                TSB_CUDA(ctx, cudaMemcpyAsync(dev, host, (size_t)run * row, cudaMemcpyHostToDevice, (cudaStream_t)s));
             else
-                TSB_CUDA(ctx, cudaMemcpyAsync(host, dev, (size_t)run * row * sizeof(__half), cudaMemcpyDeviceToHost, (cudaStream_t)s));
+                TSB_CUDA(ctx, cudaMemcpyAsync(host, dev, (size_t)run * row, cudaMemcpyDeviceToHost, (cudaStream_t)s));
         }
         p += run;
     }
@@ -299,6 +394,7 @@ int32_t tsb_kv_read_rows(tsb_kv* kv, tsb_stream s, int32_t seq, int32_t layer, i
 int32_t tsb_kv_fill_random(tsb_kv* kv, tsb_stream s, int32_t seq, int64_t tokens, uint64_t seed) {
     int32_t rc = kv_check(kv, seq);
     if (rc) return rc;
+    if (!kv->key_layers.empty()) return kv_fill_keys(kv, (cudaStream_t)s, seq, tokens, seed);
     rc = tsb_kv_reserve(kv, seq, tokens);
     if (rc) return rc;
     tsb_ctx* ctx = kv->ctx;
@@ -313,6 +409,7 @@ int32_t tsb_rope_store_kv(tsb_ctx* ctx, tsb_stream s, tsb_kv* kv, int32_t layer,
     if (!ctx || !kv) return TSB_ERR_INVALID;
     TSB_REQUIRE(ctx, qkv_f16 && rows_dev && rows > 0 && n_q_heads > 0, "bad arguments");
     TSB_REQUIRE(ctx, layer >= 0 && layer < kv->view.layers, "layer %d outside 0..%d", layer, kv->view.layers);
+    TSB_REQUIRE(ctx, kv->view.pool, "a key-only cache has no value rows");
     DeviceGuard g(ctx);
     TSB_CUDA(ctx, launch_rope_store_kv(ctx, (cudaStream_t)s, kv, layer, (__half*)qkv_f16, rows_dev, rows, n_q_heads, theta));
     return TSB_OK;
@@ -334,6 +431,7 @@ int32_t tsb_kv_commit_path(tsb_ctx* ctx, tsb_stream s, tsb_kv* kv, int32_t seq, 
     bool identity = true;
     for (int r = 0; r < keep; r++) identity &= host_path[r] == (uint32_t)r;
     if (identity) return TSB_OK;  // a chain: nothing to move
+    if (!kv->key_layers.empty()) return tsb_fail(ctx, TSB_ERR_UNSUPPORTED, "a key-only cache keeps chains, not tree paths");
     DeviceGuard g(ctx);
     cudaStream_t st = (cudaStream_t)s;
     uint32_t* dpath = nullptr;

@@ -16,9 +16,25 @@ struct KvView {
     int64_t layer_stride;  // elements between layers
 };
 
+// One layer of a key-only cache (layers whose values are their keys): rows of kv_heads * head_dim elements, f32 or
+// bfloat16, [page][token_in_page][kv_head][head_dim].  Layers may differ in both.
+struct KeyView {
+    uint8_t* base;
+    const int32_t* page_table;
+    int kv_heads, head_dim, elem_bytes;
+    int page_shift, page_tokens, num_pages, max_seqs, max_pages_per_seq;
+};
+
 struct tsb_kv {
     tsb_ctx* ctx = nullptr;
-    KvView view{};
+    KvView view{};                    // page geometry; pool and strides of a key + value cache
+    std::vector<KeyView> key_layers;  // not empty: a key-only cache (view.pool is then null)
+    uint8_t* key_pool = nullptr;
+    // A model whose rows also need their predecessors' state keeps the last state_ring - 1 rows' worth of it per stream
+    // (0: no such state).  state_lo is the oldest position whose state is still there: a cursor may go back to 0 or to
+    // state_lo + 1 and later.
+    int state_ring = 0;
+    std::vector<int64_t> state_lo;
     int32_t* page_table_dev = nullptr;
     std::vector<int32_t> page_table_host;
     std::vector<int32_t> free_pages;
@@ -26,7 +42,22 @@ struct tsb_kv {
     std::vector<int64_t> cursor;
 };
 
+// A key-only cache of n_layers layers with their own head counts and (padded) head sizes.
+int32_t kv_create_keys(tsb_ctx* ctx, int n_layers, const int32_t* kv_heads, const int32_t* head_dims, int elem_bytes, int page_tokens, int num_pages,
+                       int max_seqs, int max_pages_per_seq, tsb_kv** out);
+// Seeded pseudo-random rows [0, tokens) of a stream in every layer of a key-only cache (reserves the pages).
+int32_t kv_fill_keys(tsb_kv* kv, cudaStream_t st, int32_t seq, int64_t tokens, uint64_t seed);
+
 #ifdef __CUDACC__
+// Row of a key-only layer at position `pos` of stream `seq`; nullptr outside the reserved pages.
+template <typename T>
+__device__ __forceinline__ T* key_row(const KeyView& kv, int seq, int pos) {
+    const int lp = pos >> kv.page_shift;
+    if (pos < 0 || seq < 0 || seq >= kv.max_seqs || lp >= kv.max_pages_per_seq) return nullptr;
+    const int page = kv.page_table[(size_t)seq * kv.max_pages_per_seq + lp];
+    if (page < 0) return nullptr;
+    return reinterpret_cast<T*>(kv.base) + ((int64_t)page * kv.page_tokens + (pos & (kv.page_tokens - 1))) * ((int64_t)kv.kv_heads * kv.head_dim);
+}
 // Row of (layer, which = 0 K / 1 V) holding position `pos` of stream `seq`; nullptr when the
 // position is outside the reserved pages (the caller records TSB_DEV_BAD_INDEX and skips).
 __device__ __forceinline__ __half* kv_row(const KvView& kv, int layer, int which, int seq, int pos) {

@@ -3,6 +3,7 @@
 #include <cmath>
 #include <vector>
 
+#include "accept.cuh"
 #include "gemm_quant.cuh"
 #include "kv.cuh"
 
@@ -29,9 +30,15 @@ struct LayerW {
     bool moe_owned = false;
 };
 
+struct ModelFamily;
+struct PlainModel;
+struct PlainRt;
+
 struct tsb_model {
     tsb_ctx* ctx = nullptr;
+    const ModelFamily* family = nullptr;
     tsb_model_config cfg{};
+    PlainModel* plain = nullptr;  // plain-weight family (model_plain.cuh); the fields below belong to the block family
     std::vector<LayerW> layers;
     Mat embed, lm_head;
     uint16_t* out_norm = nullptr;
@@ -86,6 +93,7 @@ struct ModelRt {
     __half *moe_w = nullptr, *moe_zero = nullptr;
     float* moe_unit_ss = nullptr;  // [R] sums of squares that make the q|k|v epilogue's 1/rms exactly one (the operand is already normed)
     void* moe_ws = nullptr;
+    PlainRt* plain = nullptr;     // the plain-weight family's buffers
     float* tp_partial = nullptr;  // [R, d_model] f32: this rank's share of the o_proj sums, summed over the ranks in place
     std::vector<std::vector<int32_t>> fed;  // per stream: tokens absorbed, by position (target only)
     std::vector<PendingVerify> pending;     // per stream (target only)
@@ -98,8 +106,11 @@ struct tsb_session {
     cudaStream_t stream = nullptr;
     cudaEvent_t ev[4] = {nullptr, nullptr, nullptr, nullptr};
     ModelRt target, draft;
-    __half* logits_target = nullptr;  // [n_streams * max_rows, vocab]
-    __half* logits_draft = nullptr;   // [n_streams, k, vocab]
+    int pass_rows = 0;                // rows one pass of the target may carry (at least n_streams * max_rows)
+    bool logits_f32 = false;          // the family's logit rows: f32, or f16
+    LogitRows logits_target;          // [logit_rows, vocab]
+    LogitRows logits_draft;           // [n_streams, k, vocab]
+    int logit_rows = 0;
     int32_t* feed_dev = nullptr;      // [n_streams, k + 1]: confirmed token, then the proposals
     int32_t* tok1_dev = nullptr;
     int32_t* tree_dev = nullptr;      // tree drafting scratch: 128 row ids, then 8 picks per row
@@ -113,6 +124,8 @@ struct tsb_session {
     tsb_row_desc* stage_rows_dev = nullptr;
     int32_t* stage_tok_dev = nullptr;
     int stage_cap = 0, stage_used = 0;
+    int32_t *stage_int_host = nullptr, *stage_int_dev = nullptr;  // tile lists and wanted rows of ragged passes
+    int stage_int_cap = 0, stage_int_used = 0;
     tsb_accept_out* accept_out_host = nullptr;
     uint64_t* uniforms_host = nullptr;
     int32_t* feed_host = nullptr;
@@ -141,6 +154,65 @@ struct tsb_session {
 // comm.cu: in-place f32 sum over the ranks on `st` (a no-op for a null or single-rank comm).
 cudaError_t comm_all_reduce_f32(tsb_comm* c, cudaStream_t st, float* buf, size_t count);
 int comm_world(const tsb_comm* c);
+
+// ---- what a session needs of a model, whatever its tensors and its forward pass look like
+// One forward pass over `rows` rows.  Row descriptors and token ids are already on the device; cursors are not touched.
+struct Pass {
+    const int32_t* tokens = nullptr;  // token of row r: tokens[r * token_stride]
+    int token_stride = 1;
+    const tsb_row_desc* rows_dev = nullptr;
+    int rows = 0;
+    int rows_per_seq = 0;             // rows of every stream of the pass, stream after stream; 0: `groups` tells
+    int max_len = 0;                  // longest cursor + rows of the pass
+    LogitRows logits;                 // null: no head.  Output row i sits at logits + i * logits_stride
+    int64_t logits_stride = 0;
+    bool last_rows_only = false;      // uniform passes: logits of each stream's last row only, one output row per stream
+    int only = 0;                     // PASS_*
+    // ragged passes (families with `ragged`)
+    const struct RowGroup* groups = nullptr;  // host
+    int n_groups = 0;
+    const int32_t* want_dev = nullptr;        // rows whose logits are asked for
+    int n_want = 0;
+};
+// Which launches of a pass are enqueued: all of them, or - for the two timing entry points - only the layer matmuls /
+// everything but the layer matmuls.
+enum { PASS_ALL = 0, PASS_MATMULS = 1, PASS_REST = 2 };
+struct RowGroup {  // the rows of one stream in a ragged pass
+    int seq, first_row, n_rows;
+    int64_t base;
+};
+struct SessionShape {
+    int n_streams, max_rows, page_tokens;
+    int num_pages;      // pages of the target's pool
+    int pages_per_seq;
+    int pass_rows;
+};
+struct ModelFamily {
+    const char* name;
+    bool f32_logits;
+    bool trees;   // verify passes may carry a tree (ancestor masks, path compaction)
+    bool ragged;  // passes may carry unequal portions of several streams
+    int32_t (*complete)(const tsb_model*);
+    void (*free_tensors)(tsb_model*);
+    int64_t (*weight_bytes)(const tsb_model*);
+    int32_t (*share)(tsb_model* dst, int32_t dst_layer, const tsb_model* src, int32_t src_layer);
+    int32_t (*runtime_init)(tsb_session*, ModelRt&, const tsb_model*, const SessionShape&, bool is_draft);
+    void (*runtime_free)(ModelRt&);
+    int32_t (*fill_context)(tsb_session*, ModelRt&, int stream, int64_t tokens, uint64_t seed);
+    cudaError_t (*forward)(tsb_session*, ModelRt&, const Pass&);
+};
+// Upload n integers through the pinned staging ring of ragged passes.
+int32_t session_stage_ints(tsb_session* s, const int32_t* data, int n, const int32_t** dev);
+int32_t dev_alloc(tsb_ctx* ctx, std::vector<void*>& owned, size_t bytes, void** out);
+// Host side of a uniform pass: descriptors for n_active streams x rows_per_seq rows, uploaded through the pinned staging
+// ring.  slot_parent == nullptr: a chain.  Returns the device pointers.
+int32_t stage_rows(tsb_session* s, ModelRt& rt, const int32_t* streams, int n_active, int rows_per_seq,
+                   const int32_t* slot_parent, const int32_t* tokens_host /* may be null */,
+                   const tsb_row_desc** rows_dev, const int32_t** tokens_dev, int* max_len);
+// One ragged pass (model.cu): groups[i] takes its n_rows tokens in order; want_rows lists the rows whose logits land in the
+// session's logit rows 0 .. n_want - 1.  rows <= pass_rows and n_want <= logit_rows; the groups' pages are reserved here.
+// Cursors and the record of fed tokens advance.
+int32_t session_ragged_pass(tsb_session* s, const RowGroup* groups, int n_groups, const int32_t* tokens, int rows, const int32_t* want_rows, int n_want);
 
 // One speculative round for the listed streams with k proposals each (model.cu).
 int32_t session_round_streams(tsb_session* s, const int32_t* streams, int n_active, int k, const tsb_run_config* cfg,

@@ -33,6 +33,19 @@ class RunResult(C.Structure):
                 ("decode_seconds", C.c_double)]
 
 
+class StepEntry(C.Structure):
+    _fields_ = [("stream", C.c_int32), ("n_tokens", C.c_int32), ("n_want", C.c_int32)]
+
+
+class ServeRequest(C.Structure):
+    _fields_ = [("n_prompt", C.c_int32), ("max_new_tokens", C.c_int32)]
+
+
+class ServeStats(C.Structure):
+    _fields_ = [(n, C.c_int64) for n in ("steps", "rows", "prompt_rows", "decode_rows")] + \
+               [("most_live", C.c_int32), ("_pad", C.c_int32), ("seconds", C.c_double)]
+
+
 def run_config(shaping_cfg, max_new_tokens, block, uniform_mode=0, stop_tokens=(), adaptive=0, tree_nodes=0, tree_branching=(),
                reuse_prefix=False, tree_best_first=False, tree_cand=0, tree_levels=None):
     rc = RunConfig()
@@ -122,17 +135,50 @@ class Model:
 
 
 class Session:
-    def __init__(self, ctx, target, draft, n_streams, max_rows, page_tokens=64):
+    def __init__(self, ctx, target, draft, n_streams, max_rows, page_tokens=64, pool_tokens=0, step_rows=0):
+        """pool_tokens > 0: the streams share pages for that many positions; step_rows: rows one step may carry."""
         self.ctx, self.target, self.draft = ctx, target, draft
         self.n_streams, self.max_rows = n_streams, max_rows
         h = C.c_void_p()
-        ctx.check(lib().tsb_session_create(ctx.h, target.h, draft.h if draft else None, C.c_int32(n_streams),
-                                           C.c_int32(max_rows), C.c_int32(page_tokens), C.byref(h)))
+        ctx.check(lib().tsb_session_create_pool(ctx.h, target.h, draft.h if draft else None, C.c_int32(n_streams), C.c_int32(max_rows),
+                                                C.c_int32(page_tokens), C.c_int64(pool_tokens), C.c_int32(step_rows), C.byref(h)))
         self.h = h
         self.vocab = target.cfg.vocab
+        # f32 logit rows, or f16 bit patterns
+        self.logits_dtype = np.float32 if lib().tsb_model_logits_f32(target.h) else np.uint16
 
     def _logits(self, n):
-        return np.empty((n, self.vocab), dtype=np.uint16)
+        return np.empty((n, self.vocab), dtype=self.logits_dtype)
+
+    def step(self, entries):
+        """One mixed step: entries = [(stream, tokens, wanted places), ...] -> logits [sum of wanted, vocab]."""
+        arr = (StepEntry * len(entries))()
+        toks, want = [], []
+        for i, (stream, tokens, places) in enumerate(entries):
+            arr[i].stream, arr[i].n_tokens, arr[i].n_want = stream, len(tokens), len(places)
+            toks.extend(tokens)
+            want.extend(places)
+        toks = np.asarray(toks, dtype=np.int32)
+        want = np.asarray(want, dtype=np.int32)
+        out = self._logits(want.size)
+        self.ctx.check(lib().tsb_session_step(self.h, arr, C.c_int32(len(entries)), toks.ctypes.data_as(C.c_void_p),
+                                              want.ctypes.data_as(C.c_void_p), out.ctypes.data_as(C.c_void_p)))
+        return out
+
+    def serve(self, prompts, budgets, rc, prefill_chunk=1024):
+        """Continuous batching over the session's streams -> ([generated tokens per request], [reasons], stats)."""
+        reqs = (ServeRequest * len(prompts))()
+        for i, (p, b) in enumerate(zip(prompts, budgets)):
+            reqs[i].n_prompt, reqs[i].max_new_tokens = len(p), b
+        flat = np.concatenate([np.asarray(p, dtype=np.int32) for p in prompts])
+        stride = max(budgets)
+        toks = np.zeros((len(prompts), stride), dtype=np.int32)
+        counts, reasons = np.zeros(len(prompts), dtype=np.int32), np.zeros(len(prompts), dtype=np.int32)
+        stats = ServeStats()
+        self.ctx.check(lib().tsb_serve_run(self.h, reqs, C.c_int32(len(prompts)), flat.ctypes.data_as(C.c_void_p), C.byref(rc),
+                                           C.c_int32(prefill_chunk), toks.ctypes.data_as(C.c_void_p), C.c_int32(stride),
+                                           counts.ctypes.data_as(C.c_void_p), reasons.ctypes.data_as(C.c_void_p), C.byref(stats)))
+        return [toks[i, :counts[i]].copy() for i in range(len(prompts))], reasons, stats
 
     def reset(self, stream=0):
         self.ctx.check(lib().tsb_producer_reset(self.h, C.c_int32(stream)))

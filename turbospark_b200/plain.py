@@ -1,0 +1,55 @@
+"""Binding of the plain-weight decoders (tsb_model_create_plain): layers put together from mechanisms, bfloat16 or f32."""
+import ctypes as C
+
+import numpy as np
+
+from .capi import lib
+from .model import Model
+
+BF16, F32 = 0, 1
+GELU_TANH, SILU = 0, 1
+(P_EMBED, P_HEAD, P_FINAL_NORM, P_NORM, P_SHIFT, P_Q, P_K, P_HEAD_GATE, P_R1, P_R2, P_O, P_FF_GATE, P_FF_UP,
+ P_FF_DOWN) = range(14)
+
+
+class PlainConfig(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("n_layers", "d_model", "vocab", "max_context", "compute")] + \
+               [("norm_eps", C.c_float), ("logit_cap", C.c_float)]
+
+
+class PlainLayer(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("n_q_heads", "n_kv_heads", "head_dim", "window")] + \
+               [("score_scale", C.c_float), ("score_cap", C.c_float)] + \
+               [(n, C.c_int32) for n in ("log_bias", "head_gate", "token_shift", "ffn", "act")]
+
+
+def bf16_bits(x):
+    """float32 -> bfloat16 bit patterns, round to nearest even."""
+    u = np.ascontiguousarray(x, dtype=np.float32).view(np.uint32)
+    return ((u + 0x7FFF + ((u >> 16) & 1)) >> 16).astype(np.uint16)
+
+
+def bf16_to_f32(bits):
+    return (np.asarray(bits, dtype=np.uint16).astype(np.uint32) << 16).view(np.float32)
+
+
+class PlainModel(Model):
+    def __init__(self, ctx, cfg, layers):
+        self.ctx, self.cfg, self.layers = ctx, cfg, list(layers)
+        arr = (PlainLayer * len(self.layers))(*self.layers)
+        h = C.c_void_p()
+        ctx.check(lib().tsb_model_create_plain(ctx.h, C.byref(cfg), arr, C.byref(h)))
+        self.h = h
+
+    def set(self, which, array, layer=-1):
+        """Upload one tensor: uint16 arrays are bfloat16 bit patterns, anything else is taken as float32."""
+        a = np.asarray(array)
+        host = BF16 if a.dtype == np.uint16 else F32
+        a = np.ascontiguousarray(a, dtype=np.uint16 if host == BF16 else np.float32)
+        rows, cols = a.shape if a.ndim == 2 else (1, a.size)
+        self.ctx.check(lib().tsb_model_set_plain(self.h, C.c_int32(layer), C.c_int32(which), C.c_int32(host), a.ctypes.data_as(C.c_void_p),
+                                                 C.c_int64(rows), C.c_int64(cols)))
+
+    def fill(self, seed=0):
+        """Seeded random weights made on the device."""
+        self.ctx.check(lib().tsb_model_fill_plain(self.h, C.c_uint64(seed)))
