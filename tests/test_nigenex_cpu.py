@@ -177,3 +177,27 @@ def test_oracle_logits_do_not_see_the_future():
     toks2 = toks.copy()
     toks2[30:] = 3
     assert np.allclose(a[:30], no.forward(w, cfg, toks2)[:30]) and not np.allclose(a[30:], no.forward(w, cfg, toks2)[30:])
+
+
+def test_every_mechanism_shows_in_the_test_models_logits():
+    """Each mechanism changed moves the logits by a hundred times what the f32 comparisons on the GPU allow (2e-5)."""
+    cfg = nm.CONFIGS["odd"]
+    w = nm.random_weights(cfg, 0)
+    toks = np.random.default_rng(1).integers(0, cfg["vocab"], size=140)
+    want = no.forward(w, cfg, toks)
+
+    def moved(edit_layer=None, zero=None, **top):
+        c, v = dict(copy.deepcopy(cfg), **top), dict(w)
+        for l in c["layers"]:
+            if edit_layer:
+                edit_layer(l)
+        if zero:
+            v.update({k: np.zeros_like(x) for k, x in v.items() if k.endswith(zero)})
+        return nm.logit_error(no.forward(v, c, toks), want).max()
+
+    least = 100 * 2e-5
+    assert moved(lambda l: l["mixer"]["mask"].update(size=36)) > least and moved(lambda l: l["mixer"]["mask"].update(size=38)) > least
+    assert moved(lambda l: l["mixer"].update(softcap=1e6)) > least and moved(lambda l: l["mixer"].update(scale=l["mixer"]["scale"] * 1.05)) > least
+    assert moved(norm={"eps": 2e-2}) > least and moved(logit_softcap=5.0) > least
+    for zero in (".shift", ".r1", ".r2", "mix.g", "mlp.up"):
+        assert moved(zero=zero) > least, zero
