@@ -362,6 +362,21 @@ def run_ours(args, rank, world, local_rank):
         dist.destroy_process_group()
 
 
+def run_design(args):
+    from turbospark_b200 import plainbench
+    hbm, src = peaks()
+    p = os.path.join(ROOT, "MEASURED_PEAKS.json")
+    tf = float(json.load(open(p))["bf16_tflops"]) if os.path.exists(p) else 1590.0
+    sampler = ClockSampler(0)
+    sampler.start()
+    t0 = time.time()
+    results, launches = plainbench.run(0, hbm, tf, shapes=args.shapes.split(","), steps=min(args.steps, 12), parts=args.parts.split(","))
+    sampler.window(t0, time.time())
+    print(json.dumps({"metric": "prefill and decode throughput, kernel times against their rooflines", "design": args.design, "data": "synthetic",
+                      "dtype": "bf16", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": src}, "gpu_launches": launches,
+                      "clocks": sampler.stop(), "results": results}), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -371,7 +386,15 @@ def main():
     ap.add_argument("--streams", type=int, default=1, help="independent request streams per GPU")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-streams64", action="store_true", help="skip the 64-streams-in-total leg")
+    ap.add_argument("--design", default="", choices=["", "nigenex"],
+                    help="instead of the default workload: prefill, decode and kernel times of this design beside the block-quantised dense model of "
+                         "equal size (one GPU)")
+    ap.add_argument("--shapes", default="8b,2b", help="layer shapes of --design, with commas between them")
+    ap.add_argument("--parts", default="kernels,models", help="what --design measures")
     args = ap.parse_args()
+    if args.design:
+        run_design(args)
+        return
     args.warmup = max(args.warmup, 3) if args.impl == "ours" else args.warmup
     rank = int(os.environ.get("RANK", "0"))
     world = int(os.environ.get("WORLD_SIZE", "1"))

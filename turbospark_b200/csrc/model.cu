@@ -63,7 +63,9 @@ int32_t stage_rows(tsb_session* s, ModelRt& rt, const int32_t* streams, int n_ac
     const int rows = n_active * rows_per_seq;
     TSB_REQUIRE(ctx, rows <= s->n_streams * s->max_rows, "%d rows exceed the session's %d", rows, s->n_streams * s->max_rows);
     TSB_REQUIRE(ctx, rows_per_seq <= 128, "at most 128 in-flight rows per stream");
-    if (slot_parent && !rt.model->family->trees)
+    bool chain = true;
+    for (int j = 0; slot_parent && j < rows_per_seq; j++) chain &= slot_parent[j] == j - 1;
+    if (!chain && !rt.model->family->trees)
         return tsb_fail(ctx, TSB_ERR_UNSUPPORTED, "%s models verify chains only: a row's state is its predecessor's, not its parent's", rt.model->family->name);
     if (s->stage_used + rows > s->stage_cap) {
         if (s->replay || s->capturing) return tsb_fail(ctx, TSB_ERR_STATE, "staging ring overflow inside a captured round");
