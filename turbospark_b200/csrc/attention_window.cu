@@ -467,8 +467,8 @@ struct Launch {
     int n_tiles, tiles_per_group, rows_per_seq, rows_per_tile, max_len;
 };
 
-// cut tiles: at most 2 CTAs per SM in the few-query kernel (64 queries), one in the many-query kernel (128)
-size_t part_queries(const tsb_ctx* ctx) { return (size_t)2 * (ctx->sm_count > 0 ? ctx->sm_count : 148) * WATTN_SMALL_Q; }
+// queries that the shares of cut tiles may hold
+size_t part_queries(const tsb_ctx* ctx) { return (size_t)4 * (ctx->sm_count > 0 ? ctx->sm_count : 148) * WATTN_SMALL_Q; }
 
 template <int D, int MT, int SL>
 cudaError_t launch_one(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const Launch& l, void* scratch) {
@@ -476,10 +476,17 @@ cudaError_t launch_one(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const
     const int base = l.n_tiles * a.keys.kv_heads;
     const int span = a.window > 0 ? std::min(l.max_len, a.window + l.rows_per_tile) : l.max_len;
     const int key_tiles = (span + TOK - 1) / TOK + (a.window > 0 ? 1 : 0);
-    // as many runs as fill the device (a few CTAs per SM in the few-query kernel), none shorter than two key tiles
-    const int want = (SL > 1 ? 2 * sms : sms) / std::max(base, 1);
-    int splits = std::max(1, std::min({want, (key_tiles + 1) / 2, WATTN_MAX_SPLITS}));
-    if (splits > 1 && ((int64_t)base * splits * 16 * MT > (int64_t)part_queries(ctx) || base > WATTN_TICKETS)) splits = 1;
+    // the number of runs whose waves come out most even; a CTA costs its key tiles plus about three tiles' time of fixed
+    // work, and a cut tile the merge of its runs
+    const int per_sm = SL == 1 ? 1 : MT == 1 ? 3 : 2;
+    int splits = 1;
+    float best = 1e30f;
+    for (int s = 1; s <= WATTN_MAX_SPLITS && s <= (key_tiles + 1) / 2; s++) {
+        if (s > 1 && ((int64_t)base * s * 16 * MT > (int64_t)part_queries(ctx) || base > WATTN_TICKETS)) break;
+        const int waves = (base * s + per_sm * sms - 1) / (per_sm * sms);
+        const float cost = (float)waves * ((float)((key_tiles + s - 1) / s) + 3.f) + (s > 1 ? 3.f + 0.1f * (float)s : 0.f);
+        if (cost < best - 1e-3f) best = cost, splits = s;
+    }
     uint32_t* tickets = static_cast<uint32_t*>(scratch);
     float2* ml = reinterpret_cast<float2*>(tickets + WATTN_TICKETS);
     float* po = reinterpret_cast<float*>(ml + part_queries(ctx));

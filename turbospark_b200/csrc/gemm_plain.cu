@@ -1,6 +1,6 @@
 // Matrix products with plain weights.  Three kernels:
 //
-//   plain_few_kernel   bfloat16, up to 32 token rows: bound by the weight stream.  A warp multiplies a tile of 16 (or
+//   plain_few_kernel   bfloat16, up to 16 token rows: bound by the weight stream.  A warp multiplies a tile of 16 (or
 //                      2 x 16) weight rows on mma.sync.m16n8k16 with the tokens as the N side; the warps of a CTA split
 //                      the columns and meet in shared memory.  The order of the columns inside a product is free as
 //                      long as both operands agree, so a lane's fragments are contiguous 16-byte pieces of natural
@@ -17,6 +17,7 @@
 #include <cuda.h>
 
 #include <algorithm>
+#include <cstdlib>
 #include <map>
 #include <mutex>
 
@@ -538,6 +539,14 @@ TcgPlan tcg_plan(const tsb_ctx* ctx, int row_tiles, int units, int tokens) {
             if (cost < best_cost - 1e-3f) best_cost = cost, best.nt = nt, best.ksplit = ks;
         }
     }
+    if (const char* env = getenv("TSB_PLAIN_PLAN")) {  // "tokens per tile,runs": experiments
+        int nt = 0, ks = 0;
+        if (sscanf(env, "%d,%d", &nt, &ks) == 2 && (nt == 32 || nt == 64 || nt == 128 || nt == 256) && ks >= 1 && ks <= TCG_MAX_SPLITS && ks <= units) {
+            const int run = (units + ks - 1) / ks, tt = (tokens + nt - 1) / nt;
+            ks = (units + run - 1) / run;
+            if (ks == 1 || (int64_t)row_tiles * tt * ks <= 2 * sms) best.nt = nt, best.ksplit = ks;
+        }
+    }
     best.stages = std::min(TCG_MAX_STAGES, (TCG_SMEM_CAP - TCG_HEADER) / ((TCG_M + best.nt) * 128));
     return best;
 }
@@ -549,7 +558,7 @@ cudaError_t launch_few(tsb_ctx* ctx, cudaStream_t st, const PlainMat& w, const _
                       (const __nv_bfloat16*)w.data, (int)w.cols, x, x2, x_stride, tokens, epi, ctx->dev_error);
 }
 
-constexpr int FEW_MAX = 32;  // token rows up to which the weight-streaming kernel runs
+constexpr int FEW_MAX = 16;  // token rows up to which the weight-streaming kernel runs
 
 }  // namespace
 
@@ -570,8 +579,7 @@ cudaError_t launch_plain_gemm(tsb_ctx* ctx, cudaStream_t st, bool f32, const Pla
     if (tokens <= FEW_MAX) {
         const bool two = w.rows / 32 >= 4 * ctx->sm_count;  // two row tiles per CTA halve the activation reads when there are rows enough
         if (tokens <= 8) return two ? launch_few<1, 2>(ctx, st, w, xb, xb2, x_stride, tokens, epi) : launch_few<1, 1>(ctx, st, w, xb, xb2, x_stride, tokens, epi);
-        if (tokens <= 16) return two ? launch_few<2, 2>(ctx, st, w, xb, xb2, x_stride, tokens, epi) : launch_few<2, 1>(ctx, st, w, xb, xb2, x_stride, tokens, epi);
-        return two ? launch_few<4, 2>(ctx, st, w, xb, xb2, x_stride, tokens, epi) : launch_few<4, 1>(ctx, st, w, xb, xb2, x_stride, tokens, epi);
+        return two ? launch_few<2, 2>(ctx, st, w, xb, xb2, x_stride, tokens, epi) : launch_few<2, 1>(ctx, st, w, xb, xb2, x_stride, tokens, epi);
     }
     const int row_tiles = (int)(w.rows / TCG_M), units = (int)(w.cols / TCG_K);
     const TcgPlan p = tcg_plan(ctx, row_tiles, units, tokens);
