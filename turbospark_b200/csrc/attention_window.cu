@@ -5,9 +5,11 @@
 // cp.async brings into a three-stage ring.  The one tile in shared memory serves both products: K rows as the B operand
 // of S = Q K^T (ldmatrix) and as the B operand of O += P K (ldmatrix.trans), so a key byte is read once.  SL warps share an
 // m-tile, each taking 64 / SL tokens of every tile, and meet at the end.
-//   few queries (decode, short portions): SL = 4, the context is cut into runs so that the device is full; the last CTA of
-//   a tile to finish - decided by a ticket, nobody waits - adds the runs in order
-//   many queries (prompts): MT = 8, SL = 1
+//   few queries (short portions): SL = 4 or 2; many queries whose geometry the tcgen05 kernel (attention_window_tc.cu) does
+//   not take: MT = 8, SL = 1
+// Up to eight queries per key head (decoded tokens) go to window_attn8_kernel, which puts the keys on the M side.
+// A context that does not fill the device with CTAs is cut into runs of key tiles: with up to 16 queries the last CTA of a
+// tile to finish - decided by a ticket, nobody waits - adds the runs in order, with more a merge launch does.
 // Only the key tiles inside the window of some query of the tile are visited; key tiles start at multiples of 64 positions
 // whatever the cut of the prompt, so a row meets its keys in the same grouping in every schedule.
 //
@@ -17,14 +19,12 @@
 // mode, plain fused multiply-adds and the library's exp, tanh and log.
 #include <algorithm>
 
-#include "attention_window.cuh"
+#include "attention_window_dev.cuh"
 
 namespace {
 
 constexpr int TOK = 64;   // tokens per key tile
 constexpr int NST = 3;    // key tiles in flight
-constexpr int WATTN_TICKETS = 16384;
-constexpr int WATTN_MAX_SPLITS = 64;
 
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
@@ -41,27 +41,6 @@ __device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool valid) 
     const int n = valid ? 16 : 0;
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
 }
-__device__ __forceinline__ float ex2(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-__device__ __forceinline__ float lg2(float x) {
-    float y;
-    asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-__device__ __forceinline__ float rcp(float x) {
-    float y;
-    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
-    const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
-    return *reinterpret_cast<const uint32_t*>(&h);
-}
-__device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
-
 template <int D>
 struct Geo {
     static constexpr int PITCH = D <= 32 ? 64 : D <= 64 ? 128 : D <= 128 ? 256 : 512;  // bytes of a row in shared memory
@@ -72,6 +51,75 @@ struct Geo {
         return (uint32_t)(r * PITCH + ((D <= 32 ? (c ^ ((r >> 1) & 3)) : (c ^ (r & 7))) << 4));
     }
 };
+
+// The SL warps that shared a query tile's tokens have left (m, l) and O per query in shared memory, wo[slice][QT][D + 4] and
+// wml[slice][QT].  One run: the finished rows are written.  Several runs (TICKET): the run's share goes to memory and the
+// last run of the tile to finish adds all of them, in order; without TICKET a merge launch does.
+template <int D, int QT, int SL, int NTHR, bool TICKET>
+__device__ __forceinline__ void finish_slices(const WindowAttn& a, int row_first, int kvh, int grp, int n_queries, int n_splits, const float* wo,
+                                              const float2* wml, float* __restrict__ part_o, float2* __restrict__ part_ml, uint32_t* __restrict__ tickets) {
+    constexpr int DP = D + 4;
+    __shared__ uint32_t s_ticket;
+    const int64_t tile_id = (int64_t)blockIdx.z * a.keys.kv_heads + kvh;
+    const int64_t share = (tile_id * n_splits + blockIdx.x) * QT;
+    auto store = [&](int qi, int c, float4 v, float l) {  // 1 / sum, times the head's gate
+        const int row = row_first + qi / grp, head = kvh * grp + qi % grp;
+        float f = l > 0.f ? 1.f / l : 0.f;
+        if (a.gate) f *= sigmoid(a.gate[(int64_t)row * a.n_q_heads + head]);
+        *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(a.out) + (int64_t)row * a.out_stride + head * D + c) =
+            make_uint2(pack_bf16(v.x * f, v.y * f), pack_bf16(v.z * f, v.w * f));
+    };
+    for (int i = threadIdx.x; i < n_queries * (D / 4); i += NTHR) {
+        const int qi = i / (D / 4), c = (i % (D / 4)) * 4;
+        float m = -INFINITY, l = 0.f;
+#pragma unroll
+        for (int k = 0; k < SL; k++) m = fmaxf(m, wml[k * QT + qi].x);
+        const float mu = m == -INFINITY ? 0.f : m;
+        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int k = 0; k < SL; k++) {
+            const float2 v = wml[k * QT + qi];
+            const float f = ex2(v.x - mu);
+            l = fmaf(v.y, f, l);
+            const float4 x = *reinterpret_cast<const float4*>(wo + (size_t)(k * QT + qi) * DP + c);
+            acc.x = fmaf(x.x, f, acc.x), acc.y = fmaf(x.y, f, acc.y), acc.z = fmaf(x.z, f, acc.z), acc.w = fmaf(x.w, f, acc.w);
+        }
+        if (n_splits == 1) {
+            store(qi, c, acc, l);
+        } else {
+            *reinterpret_cast<float4*>(part_o + (share + qi) * D + c) = acc;
+            if (c == 0) part_ml[share + qi] = make_float2(m, l);
+        }
+    }
+    if (!TICKET || n_splits == 1) return;
+    __threadfence();
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        s_ticket = atomicAdd(&tickets[tile_id], 1u);
+        if (s_ticket == (uint32_t)n_splits - 1) tickets[tile_id] = 0;
+    }
+    __syncthreads();
+    if (s_ticket != (uint32_t)n_splits - 1) return;
+    __threadfence();
+    const int64_t first = tile_id * n_splits * QT;
+    for (int i = threadIdx.x; i < n_queries * (D / 4); i += NTHR) {
+        const int qi = i / (D / 4), c = (i % (D / 4)) * 4;
+        float m = -INFINITY, l = 0.f;
+#pragma unroll 8
+        for (int k = 0; k < n_splits; k++) m = fmaxf(m, __ldcg(&part_ml[first + k * QT + qi]).x);
+        const float mu = m == -INFINITY ? 0.f : m;
+        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 8
+        for (int k = 0; k < n_splits; k++) {
+            const float2 v = __ldcg(&part_ml[first + k * QT + qi]);
+            const float4 x = __ldcg(reinterpret_cast<const float4*>(part_o + (first + k * QT + qi) * D + c));
+            const float f = ex2(v.x - mu);
+            l = fmaf(v.y, f, l);
+            acc.x = fmaf(x.x, f, acc.x), acc.y = fmaf(x.y, f, acc.y), acc.z = fmaf(x.z, f, acc.z), acc.w = fmaf(x.w, f, acc.w);
+        }
+        store(qi, c, acc, l);
+    }
+}
 
 template <int D, int MT, int SL>
 constexpr size_t wattn_smem() {
@@ -89,7 +137,6 @@ __global__ void __launch_bounds__(32 * MT * SL, MT * SL <= 4 ? 3 : 1)
     constexpr int WTOK = TOK / SL, NT8 = WTOK / 8, KK = WTOK / 16;
     constexpr bool QREG = SL > 1 ? D <= 128 : D <= 64;  // query fragments stay in registers
     extern __shared__ __align__(128) uint8_t smem[];
-    __shared__ uint32_t s_ticket;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
     const int mt = warp % MT, sl = warp / MT;
     const int kvh = blockIdx.y, n_splits = gridDim.x;
@@ -334,60 +381,247 @@ __global__ void __launch_bounds__(32 * MT * SL, MT * SL <= 4 ? 3 : 1)
             wml[warp * 16 + gid + 8] = make_float2(m_run[1], l_run[1]);
         }
         __syncthreads();
-        for (int i = threadIdx.x; i < n_queries * (D / 4); i += NTHR) {
-            const int qi = i / (D / 4), c = (i % (D / 4)) * 4, m0 = qi >> 4, qq = qi & 15;
-            float m = -INFINITY, l = 0.f;
-#pragma unroll
-            for (int k = 0; k < SL; k++) m = fmaxf(m, wml[(k * MT + m0) * 16 + qq].x);
-            const float mu = m == -INFINITY ? 0.f : m;
-            float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-            for (int k = 0; k < SL; k++) {
-                const int w = k * MT + m0;
-                const float2 v = wml[w * 16 + qq];
-                const float f = ex2(v.x - mu);
-                l = fmaf(v.y, f, l);
-                const float4 x = *reinterpret_cast<const float4*>(wo + ((size_t)w * 16 + qq) * DP + c);
-                acc.x = fmaf(x.x, f, acc.x), acc.y = fmaf(x.y, f, acc.y), acc.z = fmaf(x.z, f, acc.z), acc.w = fmaf(x.w, f, acc.w);
-            }
-            if (n_splits == 1) {
-                const float f = factor(qi, l);
-                *reinterpret_cast<uint2*>(out_at(qi) + c) = make_uint2(pack_bf16(acc.x * f, acc.y * f), pack_bf16(acc.z * f, acc.w * f));
-            } else {
-                *reinterpret_cast<float4*>(part_o + (share + qi) * D + c) = acc;
-                if (c == 0) part_ml[share + qi] = make_float2(m, l);
-            }
-        }
+        finish_slices<D, QT, SL, NTHR, MT == 1>(a, row_first, kvh, grp, n_queries, n_splits, wo, wml, part_o, part_ml, tickets);
     }
-    if (n_splits == 1) return;
+}
 
-    // the last run of the tile to finish adds all of them, in order
-    __threadfence();
-    __syncthreads();
-    if (threadIdx.x == 0) {
-        s_ticket = atomicAdd(&tickets[tile_id], 1u);
-        if (s_ticket == (uint32_t)n_splits - 1) tickets[tile_id] = 0;
+// ------------------------------------------------------------------ up to eight queries per key head
+// A decoded token's heads (or a few rows of a small group) fill the N side of the mma, the keys its M side: S^T = K Q^T and
+// O^T = K^T P^T.  No multiply and no exponential goes to empty query slots, and a warp needs so few registers that four
+// CTAs share an SM.  Four warps, each a quarter of every key tile.
+template <int D>
+struct Few8 {
+    static constexpr int TILE = D <= 64 ? 128 : 64;   // tokens per key tile: 16 KB and more in flight per stage
+    static constexpr int WTOK = TILE / 4, NK = WTOK / 16;
+    static constexpr size_t RING = (size_t)NST * TILE * Geo<D>::PITCH;
+    static constexpr size_t MERGE = (size_t)4 * 8 * ((D + 4) * 4 + 8);
+    static constexpr size_t SMEM = RING > MERGE ? RING : MERGE;
+    static constexpr int PER_SM = D <= 128 ? 4 : 2;
+};
+
+template <int D>
+__global__ void __launch_bounds__(128, Few8<D>::PER_SM)
+    window_attn8_kernel(const __grid_constant__ WindowAttn a, const AttnTile* __restrict__ tiles, int rows_per_seq, float* __restrict__ part_o,
+                        float2* __restrict__ part_ml, uint32_t* __restrict__ tickets, uint32_t* __restrict__ err) {
+    using G = Geo<D>;
+    using F = Few8<D>;
+    constexpr int KS = D / 16, NM = D / 16, NK = F::NK;
+    extern __shared__ __align__(128) uint8_t smem[];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
+    const int kvh = blockIdx.y, n_splits = gridDim.x;
+    const int grp = a.n_q_heads / a.keys.kv_heads;
+    const int row_first = tiles ? tiles[blockIdx.z].row_first : (int)blockIdx.z * rows_per_seq;
+    const int n_rows = tiles ? tiles[blockIdx.z].n_rows : rows_per_seq;
+    const tsb_row_desc rd0 = a.rows[row_first];
+    const int seq = rd0.seq, pos0 = rd0.base + rd0.slot;
+    const int n_queries = n_rows * grp;
+    if (seq < 0 || seq >= a.keys.max_seqs || n_queries > 8) {
+        if (threadIdx.x == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+        pdl_wait();
+        return;
     }
-    __syncthreads();
-    if (s_ticket != (uint32_t)n_splits - 1) return;
-    __threadfence();
-    const int64_t first = tile_id * n_splits * QT;
-    for (int i = threadIdx.x; i < n_queries * (D / 4); i += NTHR) {
-        const int qi = i / (D / 4), c = (i % (D / 4)) * 4;
-        float m = -INFINITY, l = 0.f;
-        for (int k = 0; k < n_splits; k++) m = fmaxf(m, __ldcg(&part_ml[first + k * QT + qi]).x);
-        const float mu = m == -INFINITY ? 0.f : m;
-        float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll 4
-        for (int k = 0; k < n_splits; k++) {
-            const float2 v = __ldcg(&part_ml[first + k * QT + qi]);
-            const float4 x = __ldcg(reinterpret_cast<const float4*>(part_o + (first + k * QT + qi) * D + c));
-            const float f = ex2(v.x - mu);
-            l = fmaf(v.y, f, l);
-            acc.x = fmaf(x.x, f, acc.x), acc.y = fmaf(x.y, f, acc.y), acc.z = fmaf(x.z, f, acc.z), acc.w = fmaf(x.w, f, acc.w);
+    // key tiles start at multiples of 64 positions; this CTA's run of them
+    const int lo = a.window > 0 ? max(0, pos0 - a.window + 1) & ~63 : 0;
+    const int hi = pos0 + n_rows;
+    const int total = (hi - lo + F::TILE - 1) / F::TILE;
+    const int per = (total + n_splits - 1) / n_splits;
+    const int t_first = min(total, (int)blockIdx.x * per), n_tiles = min(total, t_first + per) - t_first;
+    const int begin = lo + t_first * F::TILE;
+
+    const uint32_t ring = smem_u32(smem);
+    auto issue = [&](int tile, int stage) {
+        constexpr int TPR = 128 / F::TILE;  // threads per token row
+        const int r = threadIdx.x / TPR, part = threadIdx.x % TPR;
+        const int pos = begin + tile * F::TILE + r;
+        const __nv_bfloat16* src = pos < hi ? key_row<__nv_bfloat16>(a.keys, seq, pos) : nullptr;
+        const bool ok = src != nullptr;
+        src = ok ? src + (int64_t)kvh * D : reinterpret_cast<const __nv_bfloat16*>(a.keys.base);
+        const uint32_t dst = ring + stage * (F::TILE * G::PITCH);
+#pragma unroll
+        for (int c = part; c < G::CH; c += TPR) cp16(dst + G::off(r, c), ok ? src + c * 8 : src, ok);
+        cp_async_commit();
+    };
+    auto prologue = [&]() {
+#pragma unroll
+        for (int i = 0; i < NST; i++) {
+            if (i < n_tiles) issue(i, i);
+            else cp_async_commit();
         }
-        const float f = factor(qi, l);
-        *reinterpret_cast<uint2*>(out_at(qi) + c) = make_uint2(pack_bf16(acc.x * f, acc.y * f), pack_bf16(acc.z * f, acc.w * f));
+    };
+    const bool early = begin + NST * F::TILE <= rd0.base;  // key tiles of earlier passes
+    if (early) prologue();
+    // score columns of this lane: queries 2 tig and 2 tig + 1
+    int pq[2];
+    float r1[2] = {0.f, 0.f}, r2[2] = {0.f, 0.f};
+#pragma unroll
+    for (int h = 0; h < 2; h++) {
+        const int qi = 2 * tig + h;
+        const bool v = qi < n_queries;
+        const int head = kvh * grp + (v ? qi % grp : 0);
+        pq[h] = v ? pos0 + qi / grp : -1;  // an empty slot sees nothing
+        if (a.r1) r1[h] = a.r1[head], r2[h] = a.r2[head];
+    }
+    pdl_wait();
+    if (!early) prologue();
+    // Q^T fragments: lane column n = query gid
+    uint32_t qb[KS][2];
+    {
+        const bool v = gid < n_queries;
+        const uint32_t* q = reinterpret_cast<const uint32_t*>(reinterpret_cast<const __nv_bfloat16*>(a.q) + (int64_t)(row_first + (v ? gid / grp : 0)) * a.q_stride +
+                                                              (kvh * grp + (v ? gid % grp : 0)) * D);
+#pragma unroll
+        for (int ks = 0; ks < KS; ks++) qb[ks][0] = q[8 * ks + tig], qb[ks][1] = q[8 * ks + 4 + tig];
+    }
+    constexpr float LOG2E = 1.4426950408889634f;
+    const bool capped = a.cap > 0.f, biased = a.r1 != nullptr;
+    const float s_in = capped ? a.scale / a.cap * (2.f * LOG2E) : a.scale * LOG2E;
+    const float c_out = a.cap * LOG2E;
+    float o[NM][4];
+#pragma unroll
+    for (int n = 0; n < NM; n++)
+#pragma unroll
+        for (int i = 0; i < 4; i++) o[n][i] = 0.f;
+    float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+    for (int tile = 0; tile < n_tiles; tile++) {
+        const int stage = tile % NST;
+        cp_async_wait<NST - 1>();
+        __syncthreads();
+        const uint32_t kt = ring + stage * (F::TILE * G::PITCH);
+        const int tok0 = warp * F::WTOK, p0 = begin + tile * F::TILE + tok0;
+        float s[NK][4];  // rows gid, gid + 8 of sixteen keys x the lane's two queries
+#pragma unroll
+        for (int n = 0; n < NK; n++) {
+#pragma unroll
+            for (int i = 0; i < 4; i++) s[n][i] = 0.f;
+#pragma unroll
+            for (int ks = 0; ks < KS; ks++) {
+                uint32_t k[4];
+                ldsm4(k, kt + G::off(tok0 + n * 16 + (lane & 15), ks * 2 + (lane >> 4)));
+                mma_bf16(s[n], k, qb[ks][0], qb[ks][1]);
+            }
+        }
+        const bool edge = p0 + F::WTOK > pos0 || (a.window > 0 && p0 <= pos0 + n_rows - 1 - a.window) || n_queries < 8;
+        float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+        for (int n = 0; n < NK; n++)
+#pragma unroll
+            for (int i = 0; i < 4; i++) {
+                const int h = i & 1;
+                const int dist = pq[h] - (p0 + n * 16 + gid + (i >> 1) * 8);
+                float v = s[n][i] * s_in;
+                if (capped) v = fmaf(-2.f * c_out, rcp(ex2(v) + 1.f), c_out);
+                if (biased) v = fmaf(-r1[h], lg2(fmaf(r2[h], (float)dist, 1.f)), v);
+                if (edge && (dist < 0 || (a.window > 0 && dist >= a.window))) v = -INFINITY;
+                s[n][i] = v;
+                mx[h] = fmaxf(mx[h], v);
+            }
+        float alpha[2], m_use[2];
+#pragma unroll
+        for (int h = 0; h < 2; h++) {
+#pragma unroll
+            for (int o2 = 4; o2 < 32; o2 <<= 1) mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], o2));
+            const float m_new = fmaxf(m_run[h], mx[h]);
+            m_use[h] = m_new == -INFINITY ? 0.f : m_new;
+            alpha[h] = ex2(m_run[h] - m_use[h]);
+            m_run[h] = m_new;
+            l_run[h] *= alpha[h];
+        }
+        if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
+#pragma unroll
+            for (int n = 0; n < NM; n++) o[n][0] *= alpha[0], o[n][1] *= alpha[1], o[n][2] *= alpha[0], o[n][3] *= alpha[1];
+        }
+#pragma unroll
+        for (int n = 0; n < NK; n++) {
+            const float e0 = ex2(s[n][0] - m_use[0]), e1 = ex2(s[n][1] - m_use[1]), e2 = ex2(s[n][2] - m_use[0]), e3 = ex2(s[n][3] - m_use[1]);
+            l_run[0] += e0 + e2, l_run[1] += e1 + e3;
+            // (keys x queries) fragments to the B operand's (keys along the registers): an 8 x 8 transpose each
+            uint32_t b0 = pack_bf16(e0, e1), b1 = pack_bf16(e2, e3);
+            asm("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(b0) : "r"(b0));
+            asm("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(b1) : "r"(b1));
+#pragma unroll
+            for (int m = 0; m < NM; m++) {
+                // K^T: rows = columns of the head, from the key rows through the transposing load
+                uint32_t k[4];
+                ldsm4_t(k, kt + G::off(tok0 + n * 16 + ((lane >> 4) << 3) + (lane & 7), m * 2 + ((lane >> 3) & 1)));
+                mma_bf16(o[m], k, b0, b1);
+            }
+        }
+        __syncthreads();  // a stage is rewritten only after every warp is done with it
+        if (tile + NST < n_tiles) issue(tile + NST, stage);
+        else cp_async_commit();
+    }
+    cp_async_wait<0>();
+    pdl_launch_dependents();
+#pragma unroll
+    for (int h = 0; h < 2; h++)
+#pragma unroll
+        for (int o2 = 4; o2 < 32; o2 <<= 1) l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], o2);
+    constexpr int DP = D + 4;
+    float* wo = reinterpret_cast<float*>(smem);
+    float2* wml = reinterpret_cast<float2*>(smem + (size_t)4 * 8 * DP * 4);
+    __syncthreads();
+#pragma unroll
+    for (int m = 0; m < NM; m++)
+#pragma unroll
+        for (int i = 0; i < 4; i++) wo[(size_t)(warp * 8 + 2 * tig + (i & 1)) * DP + m * 16 + gid + (i >> 1) * 8] = o[m][i];
+    if (gid == 0) wml[warp * 8 + 2 * tig] = make_float2(m_run[0], l_run[0]), wml[warp * 8 + 2 * tig + 1] = make_float2(m_run[1], l_run[1]);
+    __syncthreads();
+    finish_slices<D, 8, 4, 128, true>(a, row_first, kvh, grp, n_queries, n_splits, wo, wml, part_o, part_ml, tickets);
+}
+
+// ------------------------------------------------------------------ merge of cut tiles
+// One CTA per row, a warp per query head in turn: the runs' weights sit in the lanes, the sums go over the runs in order.
+__global__ void __launch_bounds__(256)
+    window_attn_merge_kernel(const __grid_constant__ WindowAttn a, const AttnTile* __restrict__ tiles, int tiles_per_group, int rows_per_seq,
+                             int rows_per_tile, int n_splits, int slots, const float* __restrict__ part_o, const float2* __restrict__ part_ml) {
+    const int tile = blockIdx.x, r = blockIdx.y;
+    int row_first, n_rows;
+    if (tiles) {
+        row_first = tiles[tile].row_first, n_rows = tiles[tile].n_rows;
+    } else {
+        const int in_group = (tile % tiles_per_group) * rows_per_tile;
+        row_first = (tile / tiles_per_group) * rows_per_seq + in_group;
+        n_rows = min(rows_per_tile, rows_per_seq - in_group);
+    }
+    pdl_wait();
+    pdl_launch_dependents();
+    if (r >= n_rows) return;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int D = a.keys.head_dim, grp = a.n_q_heads / a.keys.kv_heads, R = WATTN_LARGE_Q / grp;
+    for (int head = warp; head < a.n_q_heads; head += 8) {
+        const int slot = (r / R) * WATTN_LARGE_Q + (r % R) * grp + head % grp;
+        const int64_t first = ((int64_t)tile * a.keys.kv_heads + head / grp) * n_splits * slots + slot;
+        float2 v[WATTN_MAX_SPLITS / 32];
+        float m = -INFINITY, l = 0.f;
+#pragma unroll
+        for (int i = 0; i < WATTN_MAX_SPLITS / 32; i++) {
+            const int k = i * 32 + lane;
+            v[i] = k < n_splits ? part_ml[first + (int64_t)k * slots] : make_float2(-INFINITY, 0.f);
+            m = fmaxf(m, v[i].x);
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+        const float mu = m == -INFINITY ? 0.f : m;
+#pragma unroll
+        for (int i = 0; i < WATTN_MAX_SPLITS / 32; i++) v[i].x = ex2(v[i].x - mu), l = fmaf(v[i].y, v[i].x, l);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) l += __shfl_xor_sync(0xffffffffu, l, o);
+        float f = l > 0.f ? 1.f / l : 0.f;
+        if (a.gate) f *= sigmoid(a.gate[(int64_t)(row_first + r) * a.n_q_heads + head]);
+        __nv_bfloat16* out = reinterpret_cast<__nv_bfloat16*>(a.out) + (int64_t)(row_first + r) * a.out_stride + (int64_t)head * D;
+        for (int c0 = 0; c0 < D; c0 += 128) {
+            const int c = c0 + lane * 4;
+            float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+            for (int k = 0; k < n_splits; k++) {
+                const float w = __shfl_sync(0xffffffffu, k < 32 ? v[0].x : v[1].x, k & 31);
+                if (c < D) {
+                    const float4 x = *reinterpret_cast<const float4*>(part_o + (first + (int64_t)k * slots) * D + c);
+                    acc.x = fmaf(x.x, w, acc.x), acc.y = fmaf(x.y, w, acc.y), acc.z = fmaf(x.z, w, acc.z), acc.w = fmaf(x.w, w, acc.w);
+                }
+            }
+            if (c < D) *reinterpret_cast<uint2*>(out + c) = make_uint2(pack_bf16(acc.x * f, acc.y * f), pack_bf16(acc.z * f, acc.w * f));
+        }
     }
 }
 
@@ -462,43 +696,30 @@ __global__ void __launch_bounds__(F32_WARPS * 32) window_attn_f32_kernel(const _
         if (i * 32 + lane < D) out[i * 32 + lane] = acc[i] * f;
 }
 
-struct Launch {
-    const AttnTile* tiles;
-    int n_tiles, tiles_per_group, rows_per_seq, rows_per_tile, max_len;
-};
-
-// queries that the shares of cut tiles may hold
-size_t part_queries(const tsb_ctx* ctx) { return (size_t)4 * (ctx->sm_count > 0 ? ctx->sm_count : 148) * WATTN_SMALL_Q; }
-
 template <int D, int MT, int SL>
-cudaError_t launch_one(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const Launch& l, void* scratch) {
-    const int sms = ctx->sm_count > 0 ? ctx->sm_count : 148;
-    const int base = l.n_tiles * a.keys.kv_heads;
-    const int span = a.window > 0 ? std::min(l.max_len, a.window + l.rows_per_tile) : l.max_len;
-    const int key_tiles = (span + TOK - 1) / TOK + (a.window > 0 ? 1 : 0);
-    // the number of runs whose waves come out most even; a CTA costs its key tiles plus about three tiles' time of fixed
-    // work, and a cut tile the merge of its runs
-    const int per_sm = SL == 1 ? 1 : MT == 1 ? 3 : 2;
-    int splits = 1;
-    float best = 1e30f;
-    for (int s = 1; s <= WATTN_MAX_SPLITS && s <= (key_tiles + 1) / 2; s++) {
-        if (s > 1 && ((int64_t)base * s * 16 * MT > (int64_t)part_queries(ctx) || base > WATTN_TICKETS)) break;
-        const int waves = (base * s + per_sm * sms - 1) / (per_sm * sms);
-        const float cost = (float)waves * ((float)((key_tiles + s - 1) / s) + 3.f) + (s > 1 ? 3.f + 0.1f * (float)s : 0.f);
-        if (cost < best - 1e-3f) best = cost, splits = s;
-    }
-    uint32_t* tickets = static_cast<uint32_t*>(scratch);
-    float2* ml = reinterpret_cast<float2*>(tickets + WATTN_TICKETS);
-    float* po = reinterpret_cast<float*>(ml + part_queries(ctx));
+cudaError_t launch_one(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch) {
+    const int splits = wattn_splits(ctx, a, l, TOK, 16 * MT, SL == 1 ? 1 : MT == 1 ? 3 : 2);
+    const WattnScratch sc = wattn_scratch(ctx, scratch);
     constexpr size_t smem = wattn_smem<D, MT, SL>();
     static SmemOptIn configured;
     if (cudaError_t e = tsb_opt_in_smem(ctx, window_attn_kernel<D, MT, SL>, smem, configured); e != cudaSuccess) return e;
-    return tsb_launch(ctx, window_attn_kernel<D, MT, SL>, dim3((unsigned)splits, (unsigned)a.keys.kv_heads, (unsigned)l.n_tiles), dim3(32 * MT * SL), smem,
-                      st, true, a, l.tiles, l.tiles_per_group, l.rows_per_seq, l.rows_per_tile, po, ml, tickets, ctx->dev_error);
+    cudaError_t e = tsb_launch(ctx, window_attn_kernel<D, MT, SL>, dim3((unsigned)splits, (unsigned)a.keys.kv_heads, (unsigned)l.n_tiles), dim3(32 * MT * SL),
+                               smem, st, true, a, l.tiles, l.tiles_per_group, l.rows_per_seq, l.rows_per_tile, sc.o, sc.ml, sc.tickets, ctx->dev_error);
+    return e == cudaSuccess && splits > 1 && MT > 1 ? launch_window_attn_merge(ctx, st, a, l, splits, 16 * MT, sc) : e;
+}
+
+template <int D>
+cudaError_t launch_eight(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch) {
+    const int splits = wattn_splits(ctx, a, l, Few8<D>::TILE, 8, Few8<D>::PER_SM);
+    const WattnScratch sc = wattn_scratch(ctx, scratch);
+    static SmemOptIn configured;
+    if (cudaError_t e = tsb_opt_in_smem(ctx, window_attn8_kernel<D>, Few8<D>::SMEM, configured); e != cudaSuccess) return e;
+    return tsb_launch(ctx, window_attn8_kernel<D>, dim3((unsigned)splits, (unsigned)a.keys.kv_heads, (unsigned)l.n_tiles), dim3(128), Few8<D>::SMEM, st, true, a,
+                      l.tiles, l.rows_per_seq, sc.o, sc.ml, sc.tickets, ctx->dev_error);
 }
 
 template <int MT, int SL>
-cudaError_t launch_dim(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const Launch& l, void* scratch) {
+cudaError_t launch_dim(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch) {
     switch (a.keys.head_dim) {
         case 32: return launch_one<32, MT, SL>(ctx, st, a, l, scratch);
         case 64: return launch_one<64, MT, SL>(ctx, st, a, l, scratch);
@@ -510,15 +731,36 @@ cudaError_t launch_dim(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const
     }
 }
 
-cudaError_t launch_small(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const Launch& l, int queries, void* scratch) {
+cudaError_t launch_small(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, int queries, void* scratch) {
+    if (queries <= 8) {
+        switch (a.keys.head_dim) {
+            case 32: return launch_eight<32>(ctx, st, a, l, scratch);
+            case 64: return launch_eight<64>(ctx, st, a, l, scratch);
+            case 96: return launch_eight<96>(ctx, st, a, l, scratch);
+            case 128: return launch_eight<128>(ctx, st, a, l, scratch);
+            case 192: return launch_eight<192>(ctx, st, a, l, scratch);
+            case 256: return launch_eight<256>(ctx, st, a, l, scratch);
+            default: return cudaErrorInvalidValue;
+        }
+    }
     if (queries <= 16) return launch_dim<1, 4>(ctx, st, a, l, scratch);
     return launch_dim<4, 2>(ctx, st, a, l, scratch);
 }
 
 }  // namespace
 
+cudaError_t launch_window_attn_merge(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, int splits, int slots, const WattnScratch& sc) {
+    return tsb_launch(ctx, window_attn_merge_kernel, dim3((unsigned)l.n_tiles, (unsigned)l.rows_per_tile), dim3(256), 0, st, true, a, l.tiles,
+                      l.tiles_per_group, l.rows_per_seq, l.rows_per_tile, splits, slots, (const float*)sc.o, (const float2*)sc.ml);
+}
+
 size_t wattn_scratch_bytes(const tsb_ctx* ctx) {
-    return WATTN_TICKETS * sizeof(uint32_t) + part_queries(ctx) * (sizeof(float2) + 256 * sizeof(float));
+    return WATTN_TICKETS * sizeof(uint32_t) + wattn_part_queries(ctx) * (sizeof(float2) + 256 * sizeof(float));
+}
+
+int wattn_rows_per_tile(int head_dim, int group) {
+    const int per = WATTN_LARGE_Q / group > 0 ? WATTN_LARGE_Q / group : 1;
+    return wattn_tc_supported(head_dim, group) ? 2 * per : per;
 }
 
 int wattn_pad_dim(int head_dim, bool f32) {
@@ -535,15 +777,18 @@ cudaError_t launch_window_attn(tsb_ctx* ctx, cudaStream_t st, bool f32, const Wi
     if (f32)
         return tsb_launch(ctx, window_attn_f32_kernel, dim3((unsigned)(((int64_t)b.rows * a.n_q_heads + F32_WARPS - 1) / F32_WARPS)), dim3(F32_WARPS * 32),
                           0, st, true, a, b.rows, ctx->dev_error);
-    const int grp = a.n_q_heads / a.keys.kv_heads, rpt = wattn_rows_per_tile(grp);
+    const int grp = a.n_q_heads / a.keys.kv_heads, rpt = wattn_rows_per_tile(a.keys.head_dim, grp);
+    auto large = [&](const WattnLaunch& l) {
+        return wattn_tc_supported(a.keys.head_dim, grp) ? launch_window_attn_tc(ctx, st, a, l, scratch) : launch_dim<8, 1>(ctx, st, a, l, scratch);
+    };
     if (b.rows_per_seq > 0) {
         const int groups = b.rows / b.rows_per_seq, queries = b.rows_per_seq * grp;
-        if (queries <= WATTN_SMALL_Q) return launch_small(ctx, st, a, Launch{nullptr, groups, 1, b.rows_per_seq, b.rows_per_seq, b.max_len}, queries, scratch);
+        if (queries <= WATTN_SMALL_Q) return launch_small(ctx, st, a, WattnLaunch{nullptr, groups, 1, b.rows_per_seq, b.rows_per_seq, b.max_len}, queries, scratch);
         const int tpg = (b.rows_per_seq + rpt - 1) / rpt;
-        return launch_dim<8, 1>(ctx, st, a, Launch{nullptr, groups * tpg, tpg, b.rows_per_seq, rpt, b.max_len}, scratch);
+        return large(WattnLaunch{nullptr, groups * tpg, tpg, b.rows_per_seq, rpt, b.max_len});
     }
     cudaError_t e = cudaSuccess;
-    if (b.n_large > 0) e = launch_dim<8, 1>(ctx, st, a, Launch{b.large, b.n_large, 1, 0, rpt, b.max_len}, scratch);
-    if (e == cudaSuccess && b.n_small > 0) e = launch_small(ctx, st, a, Launch{b.small, b.n_small, 1, 0, WATTN_SMALL_Q / grp, b.max_len}, b.small_queries, scratch);
+    if (b.n_large > 0) e = large(WattnLaunch{b.large, b.n_large, 1, 0, rpt, b.max_len});
+    if (e == cudaSuccess && b.n_small > 0) e = launch_small(ctx, st, a, WattnLaunch{b.small, b.n_small, 1, 0, WATTN_SMALL_Q / grp, b.max_len}, b.small_queries, scratch);
     return e;
 }

@@ -25,8 +25,8 @@ struct AttnTile {
     int32_t row_first, n_rows;
 };
 constexpr int WATTN_SMALL_Q = 64;   // queries (rows x heads per key head) of a stream up to which the few-query kernel takes them
-constexpr int WATTN_LARGE_Q = 128;  // queries per tile of the many-query kernel
-inline int wattn_rows_per_tile(int group) { return WATTN_LARGE_Q / group > 0 ? WATTN_LARGE_Q / group : 1; }
+constexpr int WATTN_LARGE_Q = 128;  // queries per tile of the many-query kernels (a tcgen05 CTA takes two such tiles)
+int wattn_rows_per_tile(int head_dim, int group);  // rows of a tile in the many-query kernel that takes this geometry
 
 // Where the query tiles of a pass come from: a uniform pass (rows_per_seq rows of every stream) or device lists made for
 // the layer's group size by wattn_make_tiles.

@@ -1,0 +1,75 @@
+// Shared by the sliding-window attention kernels: score arithmetic helpers and the launch description.
+#pragma once
+#include "attention_window.cuh"
+
+namespace {
+
+__device__ __forceinline__ float ex2(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float lg2(float x) {
+    float y;
+    asm("lg2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ float rcp(float x) {
+    float y;
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+__device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
+    const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
+    return *reinterpret_cast<const uint32_t*>(&h);
+}
+__device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+
+constexpr int WATTN_TICKETS = 16384;
+constexpr int WATTN_MAX_SPLITS = 64;
+
+}  // namespace
+
+struct WattnLaunch {
+    const AttnTile* tiles;  // null: a uniform pass
+    int n_tiles, tiles_per_group, rows_per_seq, rows_per_tile, max_len;
+};
+// Scratch of cut tiles: tickets, then (m, l) of every query slot, then the slots' sums.
+struct WattnScratch {
+    uint32_t* tickets;
+    float2* ml;
+    float* o;
+};
+inline size_t wattn_part_queries(const tsb_ctx* ctx) { return (size_t)4 * (ctx->sm_count > 0 ? ctx->sm_count : 148) * WATTN_SMALL_Q; }
+inline WattnScratch wattn_scratch(const tsb_ctx* ctx, void* p) {
+    WattnScratch s;
+    s.tickets = static_cast<uint32_t*>(p);
+    s.ml = reinterpret_cast<float2*>(s.tickets + WATTN_TICKETS);
+    s.o = reinterpret_cast<float*>(s.ml + wattn_part_queries(ctx));
+    return s;
+}
+// How many runs the key tiles of a launch are cut into: the number whose waves come out most even.  base: CTAs of an uncut
+// launch; a CTA costs its key tiles plus about three tiles' time of fixed work, a cut tile also the merge of its runs.
+inline int wattn_splits(const tsb_ctx* ctx, const WindowAttn& a, const WattnLaunch& l, int tile_tokens, int queries_per_cta, int ctas_per_sm) {
+    const int sms = ctx->sm_count > 0 ? ctx->sm_count : 148;
+    const int base = l.n_tiles * a.keys.kv_heads;
+    const int span = a.window > 0 && a.window + l.rows_per_tile < l.max_len ? a.window + l.rows_per_tile : l.max_len;
+    const int key_tiles = (span + tile_tokens - 1) / tile_tokens + (a.window > 0 ? 1 : 0);
+    int splits = 1;
+    float best = 1e30f;
+    for (int s = 1; s <= WATTN_MAX_SPLITS && s <= (key_tiles + 1) / 2; s++) {
+        if (s > 1 && ((int64_t)base * s * queries_per_cta > (int64_t)wattn_part_queries(ctx) || base > WATTN_TICKETS)) break;
+        const int waves = (base * s + ctas_per_sm * sms - 1) / (ctas_per_sm * sms);
+        const float cost = (float)waves * ((float)((key_tiles + s - 1) / s) + 3.f) + (s > 1 ? 3.f + 0.1f * (float)s : 0.f);
+        if (cost < best - 1e-3f) best = cost, splits = s;
+    }
+    return splits;
+}
+
+// Adds the runs of cut tiles, in order, and writes the finished rows.  A tile has `slots` query slots per run: row r of the
+// tile and head h sit in slot (r / R) * 128 + (r % R) * group + h with R = 128 / group.
+cudaError_t launch_window_attn_merge(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, int splits, int slots, const WattnScratch& sc);
+
+// The tcgen05 kernel for many queries (attention_window_tc.cu): head sizes 64 and 128, up to eight heads per key head.
+bool wattn_tc_supported(int head_dim, int group);
+cudaError_t launch_window_attn_tc(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch);

@@ -188,7 +188,7 @@ int32_t plain_fill_context(tsb_session* s, ModelRt& rt, int stream, int64_t toke
 
 // The query tiles of a ragged pass for one group size: few-query tiles hold a whole stream's rows.
 struct TileLists {
-    int group = 0;
+    int group = 0, rows_per_tile = 0;
     AttnBatch batch;
 };
 
@@ -211,13 +211,13 @@ cudaError_t plain_forward(tsb_session* s, ModelRt& rt, const Pass& p) {
         for (int i = 0; i < p.n_groups; i++) longest = std::max(longest, p.groups[i].n_rows);
         for (const PlainLayer& l : m->layers) {
             const int grp = l.cfg.n_q_heads / l.cfg.n_kv_heads;
+            const int rpt = wattn_rows_per_tile(l.head_pad, grp);
             bool have = m->f32;  // the f32 kernel takes rows one by one
-            for (const TileLists& t : lists) have |= t.group == grp;
+            for (const TileLists& t : lists) have |= t.group == grp && t.rows_per_tile == rpt;
             if (have) continue;
             std::vector<AttnTile> small, large;
             TileLists t;
-            t.group = grp;
-            const int rpt = wattn_rows_per_tile(grp);
+            t.group = grp, t.rows_per_tile = rpt;
             for (int i = 0; i < p.n_groups; i++) {
                 const RowGroup& g = p.groups[i];
                 if (g.n_rows * grp <= WATTN_SMALL_Q) {
@@ -261,7 +261,7 @@ cudaError_t plain_forward(tsb_session* s, ModelRt& rt, const Pass& p) {
         if (c.log_bias) a.r1 = l.r1, a.r2 = l.r2;
         AttnBatch batch;
         for (const TileLists& t : lists)
-            if (t.group == c.n_q_heads / c.n_kv_heads) batch = t.batch;
+            if (t.group == c.n_q_heads / c.n_kv_heads && t.rows_per_tile == wattn_rows_per_tile(l.head_pad, t.group)) batch = t.batch;
         batch.rows = p.rows, batch.rows_per_seq = p.rows_per_seq, batch.max_len = max_len;
         FW(launch_window_attn(ctx, st, m->f32, a, batch, b->attn_ws));
         PlainEpi out;
@@ -552,7 +552,7 @@ int32_t tsb_window_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, int32_t l
         TSB_CUDA(ctx, launch_window_attn(ctx, st, kv.elem_bytes == 4, a, b, scratch));
         return TSB_OK;
     }
-    const int grp = n_q_heads / kv.kv_heads, rpt = wattn_rows_per_tile(grp);
+    const int grp = n_q_heads / kv.kv_heads, rpt = wattn_rows_per_tile(kv.head_dim, grp);
     std::vector<AttnTile> small, large;
     for (int i = 0, r = 0; i < n_groups; r += group_rows[i], i++) {
         if (group_rows[i] * grp <= WATTN_SMALL_Q) {
