@@ -460,7 +460,7 @@ TSB_API int32_t tsb_kv_create_keys(tsb_ctx* ctx, int32_t type, int32_t layers, i
                                    int32_t num_pages, int32_t max_seqs, int32_t max_pages_per_seq, tsb_kv** out);
 /* Attention of rows over such a cache, keys of the rows themselves included (positions base + slot; a stream's rows are
  * consecutive, slots 0, 1, ...).  group_rows lists the rows of every stream of the batch in order (host).  q and out are
- * [rows, stride] in `type`; gate [rows, n_q_heads] f32 pre-activations or NULL; r1, r2 [n_q_heads] f32 or NULL. */
+ * [rows, stride] in `type`, rows on 32-byte boundaries (strides a multiple of 16); gate [rows, n_q_heads] f32 pre-activations or NULL; r1, r2 [n_q_heads] f32 or NULL. */
 TSB_API int32_t tsb_window_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, int32_t layer, const void* q, int64_t q_stride, void* out,
                                      int64_t out_stride, const tsb_row_desc* rows_dev, const int32_t* group_rows, int32_t n_groups,
                                      int32_t n_q_heads, float scale, float cap, const float* r1, const float* r2, const float* gate,

@@ -164,10 +164,13 @@ def attend(rig, type_, cache, groups, q, heads, scale, cap, r1, r2, gate, window
     n, _, dim = q.shape
     _, qu = quantise(q, type_)
     up = lambda a: None if a is None else ctx.to_device(np.asarray(a, dtype=np.float32))
-    out = ctx.zeroed(n * heads * dim * 4)
-    ctx.window_attention(cache.kv, 1, ctx.to_device(qu.reshape(n, -1)), heads * dim, out, heads * dim, ctx.to_device(descs(tsb, groups)),
+    stride = (heads * dim + 15) // 16 * 16
+    padded = np.zeros((n, stride), dtype=qu.dtype)
+    padded[:, :heads * dim] = qu.reshape(n, -1)
+    out = ctx.zeroed(n * stride * 4)
+    ctx.window_attention(cache.kv, 1, ctx.to_device(padded), stride, out, stride, ctx.to_device(descs(tsb, groups)),
                          [g[2] for g in groups], heads, scale, cap, up(r1), up(r2), up(gate), window, max(b + m for _, b, m in groups), rig["attn"])
-    return fetch(out, type_, (n, heads, dim))
+    return fetch(out, type_, (n, stride))[:, :heads * dim].reshape(n, heads, dim)
 
 
 def expect(cache, groups, q, scale, cap, r1, r2, gate, window, type_):
@@ -203,6 +206,22 @@ def test_attention_over_unequal_portions(rig, type_, heads, kv_heads, dim, windo
         got = attend(rig, type_, cache, groups, q, heads, scale, cap, r1, r2, gate, window)
         want = expect(cache, groups, q, scale, cap, r1.astype(np.float32), r2.astype(np.float32), gate.astype(np.float32), window, type_)
         assert np.abs(got - want).max() < tol, (sizes, np.abs(got - want).max())
+    cache.kv.close()
+
+
+@pytest.mark.parametrize("scale,cap", [(0.01, 50.0), (0.2, 50.0), (2.0, 50.0), (0.5, 1.0), (30.0, 20.0), (-0.4, 6.0)])
+@pytest.mark.parametrize("dim", [64, 128])
+@pytest.mark.parametrize("rows", [1, 10, 100])
+def test_scores_far_inside_and_far_beyond_the_cap(rig, rows, dim, scale, cap):
+    """The many-query kernel has a series for small scores and the exponential form for the rest: both, and tiles that mix."""
+    rng = np.random.default_rng(rows)
+    cache = Cache(rig, BF16, 2, dim, [300], rng)
+    q = rng.standard_normal((rows, 8, dim)) / np.sqrt(dim / 64)
+    q[:, 3] *= 0.01
+    r = np.full(8, 0.2, dtype=np.float32)
+    groups = [(0, 300 - rows, rows)]
+    got = attend(rig, BF16, cache, groups, q, 8, scale, cap, r, r, None, 200)
+    assert np.abs(got - expect(cache, groups, q, scale, cap, r, r, None, 200, BF16)).max() < 2.5e-2
     cache.kv.close()
 
 
@@ -285,4 +304,6 @@ def test_operators_refuse_what_they_do_not_cover(rig):
         ctx.attn_decode_rows(keys, 0, b, 64, b, b, 1, 1, 4, 1.0, 1, b)
     with pytest.raises(tsb.TsbError):
         ctx.window_attention(keys, 0, b, 64, b, 64, b, [1], 200, 1.0, 0.0, None, None, None, 0, 1, rig["attn"])
+    with pytest.raises(tsb.TsbError, match="32-byte"):
+        ctx.window_attention(keys, 0, b, 72, b, 64, b, [1], 1, 1.0, 0.0, None, None, None, 0, 1, rig["attn"])
     kv.close(), keys.close()

@@ -570,7 +570,7 @@ __global__ void __launch_bounds__(128, Few8<D>::PER_SM)
 }
 
 // ------------------------------------------------------------------ merge of cut tiles
-// One CTA per row, a warp per query head in turn: the runs' weights sit in the lanes, the sums go over the runs in order.
+// One CTA per row and eight query heads, a warp per head: the runs' weights sit in the lanes, the sums go over the runs in order.
 __global__ void __launch_bounds__(256)
     window_attn_merge_kernel(const __grid_constant__ WindowAttn a, const AttnTile* __restrict__ tiles, int tiles_per_group, int rows_per_seq,
                              int rows_per_tile, int n_splits, int slots, const float* __restrict__ part_o, const float2* __restrict__ part_ml) {
@@ -588,7 +588,8 @@ __global__ void __launch_bounds__(256)
     if (r >= n_rows) return;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int D = a.keys.head_dim, grp = a.n_q_heads / a.keys.kv_heads, R = WATTN_LARGE_Q / grp;
-    for (int head = warp; head < a.n_q_heads; head += 8) {
+    const int head = blockIdx.z * 8 + warp;
+    if (head < a.n_q_heads) {
         const int slot = (r / R) * WATTN_LARGE_Q + (r % R) * grp + head % grp;
         const int64_t first = ((int64_t)tile * a.keys.kv_heads + head / grp) * n_splits * slots + slot;
         float2 v[WATTN_MAX_SPLITS / 32];
@@ -750,7 +751,7 @@ cudaError_t launch_small(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, con
 }  // namespace
 
 cudaError_t launch_window_attn_merge(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, int splits, int slots, const WattnScratch& sc) {
-    return tsb_launch(ctx, window_attn_merge_kernel, dim3((unsigned)l.n_tiles, (unsigned)l.rows_per_tile), dim3(256), 0, st, true, a, l.tiles,
+    return tsb_launch(ctx, window_attn_merge_kernel, dim3((unsigned)l.n_tiles, (unsigned)l.rows_per_tile, (unsigned)((a.n_q_heads + 7) / 8)), dim3(256), 0, st, true, a, l.tiles,
                       l.tiles_per_group, l.rows_per_seq, l.rows_per_tile, splits, slots, (const float*)sc.o, (const float2*)sc.ml);
 }
 

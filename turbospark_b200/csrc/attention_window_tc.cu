@@ -54,6 +54,41 @@ __device__ __forceinline__ void wt_g2s_2d(uint32_t dst_smem, const CUtensorMap* 
 // byte offset of 16-byte chunk c of row r in a 128-byte-swizzled tile of 128 rows: 64-column blocks of 128 rows x 128 bytes
 __device__ __forceinline__ uint32_t wt_off(int r, int c) { return (uint32_t)((c >> 3) * (128 * 128) + r * 128 + (((c & 7) ^ (r & 7)) << 4)); }
 
+// Two f32 lanes per instruction.
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+    float2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;"
+        : "=l"(reinterpret_cast<unsigned long long&>(d))
+        : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)),
+          "l"(reinterpret_cast<const unsigned long long&>(c)));
+    return d;
+}
+__device__ __forceinline__ float2 add2(float2 a, float2 b) {
+    float2 d;
+    asm("add.rn.f32x2 %0, %1, %2;"
+        : "=l"(reinterpret_cast<unsigned long long&>(d))
+        : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)));
+    return d;
+}
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+    float2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;"
+        : "=l"(reinterpret_cast<unsigned long long&>(d))
+        : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)));
+    return d;
+}
+__device__ __forceinline__ float2 both(float x) { return make_float2(x, x); }
+__device__ __forceinline__ void st_32bytes(void* p, const uint32_t (&r)[8]) {  // one full sector per thread
+    asm volatile("st.global.v8.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8};" ::"l"(p), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]),
+                 "r"(r[7])
+                 : "memory");
+}
+
+// Within |y| <= TANH_SMALL, tanh(y) is its Taylor series y - y^3/3 + 2 y^5/15 - 17 y^7/315 + 62 y^9/2835; the first term left
+// out is 1382 y^11 / 155925, below 6e-8 of y there.  Scores well inside the cap - the usual case - then need no
+// special-function instruction but the softmax's own.
+constexpr float TANH_SMALL = 0.3f;
+
 template <int D>
 __global__ void __launch_bounds__(WT_THREADS, 1)
     window_attn_tc_kernel(const __grid_constant__ CUtensorMap kmap, int box_rows, const __grid_constant__ WindowAttn a, const AttnTile* __restrict__ tiles,
@@ -216,6 +251,10 @@ __global__ void __launch_bounds__(WT_THREADS, 1)
             constexpr float LOG2E = 1.4426950408889634f;
             const float s_in = capped ? a.scale / a.cap * (2.f * LOG2E) : a.scale * LOG2E;
             const float c_out = a.cap * LOG2E;
+            // the series in the raw score x, y = x scale / cap: x (k0 + k1 x^2 + ...), times cap log2(e)
+            const float y_in = capped ? a.scale / a.cap : 0.f, y2 = y_in * y_in, small = capped ? TANH_SMALL / fabsf(y_in) : 0.f;
+            const float k0 = c_out * y_in, k1 = k0 * y2 * (-1.f / 3.f), k2 = k0 * y2 * y2 * (2.f / 15.f), k3 = k0 * y2 * y2 * y2 * (-17.f / 315.f),
+                        k4 = k0 * y2 * y2 * y2 * y2 * (62.f / 2835.f);
             // bias tables: entry k of a head holds the bias at distance wg_first - p0 + rows_wg - 1 - k; row_l's key j is entry
             // rows_wg - 1 - row_l + j.  The pitch keeps the 32 queries of a warp on different banks.
             const int need = rows_wg + WT_TN - 1;
@@ -228,32 +267,51 @@ __global__ void __launch_bounds__(WT_THREADS, 1)
                 const int p0 = begin + t * WT_TN;
                 const float* bias = tab[t & 1] + tab_at;
                 if (biased) {
-                    for (int i = ql; i < grp * need; i += WT_QM) {
-                        const int h = i / need, k = i - h * need;
-                        const int dist = max(wg_first - p0 + rows_wg - 1 - k, 0);
-                        tab[t & 1][h * pitch + k] = a.r1[kvh * grp + h] * lg2(fmaf(a.r2[kvh * grp + h], (float)dist, 1.f));
+                    for (int h = 0; h < grp; h++) {
+                        const float r1 = a.r1[kvh * grp + h], r2 = a.r2[kvh * grp + h];
+                        for (int k = ql; k < need; k += WT_QM)
+                            tab[t & 1][h * pitch + k] = -r1 * lg2(fmaf(r2, (float)max(wg_first - p0 + rows_wg - 1 - k, 0), 1.f));
                     }
                     asm volatile("bar.sync %0, 128;" ::"r"(1 + x) : "memory");
                 }
                 if (ok) ok = mbar_wait(&bars->s_full[x], t & 1, err);
                 tc_fence_after();
                 float s[WT_TN];
+                {
+                    uint32_t r[WT_TN / 16][16];
 #pragma unroll
-                for (int c = 0; c < WT_TN; c += 32) {
-                    uint32_t r0[16], r1[16];
-                    tc_ld16(col_s + c, r0);
-                    tc_ld16(col_s + c + 16, r1);
+                    for (int c = 0; c < WT_TN / 16; c++) tc_ld16(col_s + 16 * c, r[c]);
                     tc_wait_ld();
 #pragma unroll
-                    for (int i = 0; i < 16; i++) s[c + i] = __uint_as_float(r0[i]) * s_in, s[c + 16 + i] = __uint_as_float(r1[i]) * s_in;
+                    for (int j = 0; j < WT_TN; j++) s[j] = __uint_as_float(r[j >> 4][j & 15]);
                 }
+                bool series = true;
                 if (capped) {
+                    float big = 0.f;
 #pragma unroll
-                    for (int j = 0; j < WT_TN; j++) s[j] = fmaf(-2.f * c_out, rcp(ex2(s[j]) + 1.f), c_out);
+                    for (int j = 0; j < WT_TN; j++) big = fmaxf(big, fabsf(s[j]));
+                    series = !__any_sync(0xffffffffu, big > small);
                 }
-                if (biased) {
+                if (capped && series) {
 #pragma unroll
-                    for (int j = 0; j < WT_TN; j++) s[j] -= bias[j];
+                    for (int j = 0; j < WT_TN; j += 2) {
+                        const float2 x = make_float2(s[j], s[j + 1]), z = mul2(x, x);
+                        const float2 w = fma2(z, fma2(z, fma2(z, fma2(z, both(k4), both(k3)), both(k2)), both(k1)), both(k0));
+                        const float2 v = fma2(x, w, biased ? make_float2(bias[j], bias[j + 1]) : both(0.f));
+                        s[j] = v.x, s[j + 1] = v.y;
+                    }
+                } else {
+                    if (capped) {
+#pragma unroll
+                        for (int j = 0; j < WT_TN; j++) s[j] = fmaf(-2.f * c_out, rcp(ex2(s[j] * s_in) + 1.f), c_out);
+                    } else {
+#pragma unroll
+                        for (int j = 0; j < WT_TN; j++) s[j] *= s_in;
+                    }
+                    if (biased) {
+#pragma unroll
+                        for (int j = 0; j < WT_TN; j++) s[j] += bias[j];
+                    }
                 }
                 if (p0 + WT_TN - 1 > wg_first || (a.window > 0 && wg_last - p0 >= a.window)) {  // the tile meets an edge of some row
                     const int j_max = pq - p0, j_min = a.window > 0 ? j_max - a.window + 1 : -0x7fffffff;
@@ -285,19 +343,20 @@ __global__ void __launch_bounds__(WT_THREADS, 1)
                     }
                 }
                 const float m_use = m_new == -INFINITY ? 0.f : m_new;
-                float rs[4] = {0.f, 0.f, 0.f, 0.f};
+                float2 rs[2] = {both(0.f), both(0.f)};
 #pragma unroll
                 for (int c = 0; c < WT_TN; c += 64) {
                     uint32_t pk[32];
 #pragma unroll
-                    for (int j = 0; j < 64; j += 4) {
-                        const float e0 = ex2(s[c + j] - m_use), e1 = ex2(s[c + j + 1] - m_use), e2 = ex2(s[c + j + 2] - m_use), e3 = ex2(s[c + j + 3] - m_use);
-                        rs[0] += e0, rs[1] += e1, rs[2] += e2, rs[3] += e3;
-                        pk[j >> 1] = pack_bf16(e0, e1), pk[(j >> 1) + 1] = pack_bf16(e2, e3);
+                    for (int j = 0; j < 64; j += 2) {
+                        float2 e = add2(make_float2(s[c + j], s[c + j + 1]), both(-m_use));
+                        e.x = ex2(e.x), e.y = ex2(e.y);
+                        rs[(j >> 1) & 1] = add2(rs[(j >> 1) & 1], e);
+                        pk[j >> 1] = pack_bf16(e.x, e.y);
                     }
                     tc_st32(col_s + (c >> 1), pk);
                 }
-                l_run = fmaf(l_run, alpha, (rs[0] + rs[1]) + (rs[2] + rs[3]));
+                l_run = fmaf(l_run, alpha, (rs[0].x + rs[0].y) + (rs[1].x + rs[1].y));
                 m_ref = m_new;
                 tc_wait_st();
                 tc_fence_before();
@@ -328,12 +387,15 @@ __global__ void __launch_bounds__(WT_THREADS, 1)
                     uint32_t w[8];
 #pragma unroll
                     for (int i = 0; i < 8; i++) w[i] = pack_bf16(v[2 * i] * f, v[2 * i + 1] * f);
-                    uint4* p = reinterpret_cast<uint4*>(reinterpret_cast<__nv_bfloat16*>(a.out) + (int64_t)row * a.out_stride + head * D + c);
-                    p[0] = make_uint4(w[0], w[1], w[2], w[3]), p[1] = make_uint4(w[4], w[5], w[6], w[7]);
+                    st_32bytes(reinterpret_cast<__nv_bfloat16*>(a.out) + (int64_t)row * a.out_stride + head * D + c, w);
                 } else {
-                    float4* p = reinterpret_cast<float4*>(part_o + share * D + c);
+                    uint32_t w[8];
 #pragma unroll
-                    for (int i = 0; i < 4; i++) p[i] = make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]);
+                    for (int h = 0; h < 2; h++) {
+#pragma unroll
+                        for (int i = 0; i < 8; i++) w[i] = __float_as_uint(v[8 * h + i]);
+                        st_32bytes(part_o + share * D + c + 8 * h, w);
+                    }
                 }
             }
             if (valid && n_splits > 1) part_ml[share] = make_float2(m_ref, l_run);

@@ -471,6 +471,7 @@ static int32_t check_gemm(tsb_ctx* ctx, int32_t type, const void* w, int64_t row
     TSB_REQUIRE(ctx, rows > 0 && rows % PLAIN_ROW_PAD == 0 && cols > 0 && cols % PLAIN_COL_PAD == 0, "rows must be a multiple of %d and cols of %d",
                 PLAIN_ROW_PAD, PLAIN_COL_PAD);
     TSB_REQUIRE(ctx, tokens > 0 && x_rows >= 32 && x_rows >= tokens, "x needs at least max(32, tokens) allocated rows");
+    TSB_REQUIRE(ctx, (uintptr_t)w % 16 == 0 && (uintptr_t)x % 16 == 0, "w and x must be 16-byte aligned");
     return TSB_OK;
 }
 
@@ -508,6 +509,8 @@ int32_t tsb_norm_shift_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, const floa
                             int64_t out_stride) {
     if (!ctx) return TSB_ERR_INVALID;
     TSB_REQUIRE(ctx, x && gain && rows_dev && mix_out && d > 0 && rows > 0 && out_stride >= d && (type == TSB_BF16 || type == TSB_F32), "bad arguments");
+    TSB_REQUIRE(ctx, (uintptr_t)x % 16 == 0 && (uintptr_t)mu % 16 == 0 && (uintptr_t)state % 16 == 0 && (uintptr_t)mix_out % 16 == 0 && (uintptr_t)h_out % 16 == 0,
+                "buffers must be 16-byte aligned");
     TSB_REQUIRE(ctx, !mu || (state && n_streams > 0 && ring >= 2 && (ring & (ring - 1)) == 0), "a shift needs its state, ring a power of two");
     DeviceGuard g(ctx);
     ShiftState st;
@@ -534,6 +537,9 @@ int32_t tsb_window_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, int32_t l
     const KeyView& kv = keys->key_layers[layer];
     TSB_REQUIRE(ctx, n_q_heads > 0 && n_q_heads % kv.kv_heads == 0 && wattn_supported(kv.head_dim, n_q_heads / kv.kv_heads, kv.elem_bytes == 4),
                 "query heads must be a multiple of the key heads, at most %d per key head", WATTN_LARGE_Q);
+    TSB_REQUIRE(ctx, (uintptr_t)q % 32 == 0 && (uintptr_t)out % 32 == 0 && q_stride % 16 == 0 && out_stride % 16 == 0 &&
+                         q_stride >= (int64_t)n_q_heads * kv.head_dim && out_stride >= (int64_t)n_q_heads * kv.head_dim,
+                "q and out rows hold every head and start on 32-byte boundaries (strides a multiple of 16)");
     cudaStream_t st = (cudaStream_t)s;
     DeviceGuard g(ctx);
     WindowAttn a;

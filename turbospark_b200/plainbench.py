@@ -54,11 +54,11 @@ class Peaks:
 
 
 # ------------------------------------------------------------------ kernels
-def random_bf16(ctx, n, seed):
+def random_bf16(ctx, n, seed, amp=0.05):
     import torch
     torch.manual_seed(seed)
     b = ctx.alloc(n * 2)
-    t = torch.empty(min(n, 1 << 22), device="cuda", dtype=torch.bfloat16).uniform_(-0.05, 0.05).view(torch.int16).cpu().numpy()
+    t = torch.empty(min(n, 1 << 22), device="cuda", dtype=torch.bfloat16).uniform_(-amp, amp).view(torch.int16).cpu().numpy()
     for at in range(0, n, t.size):
         m = min(t.size, n - at)
         ctx.check(capi.lib().tsb_memcpy_h2d(ctx.h, None, C.c_void_p(b.ptr + at * 2), t.ctypes.data_as(C.c_void_p), C.c_size_t(m * 2)))
@@ -111,7 +111,7 @@ def window_attention(ctx, peaks, name, hd, nq, nkv, context, rows, streams, wind
     for s in range(streams):
         kv.fill_random(s, context + rows, 7 + s)
     n = streams * rows
-    q, out = random_bf16(ctx, n * nq * hd, 3), ctx.alloc(n * nq * hd * 2)
+    q, out = random_bf16(ctx, n * nq * hd, 3, amp=3.5), ctx.alloc(n * nq * hd * 2)  # scores of standard deviation about 2
     gate = ctx.zeroed(n * nq * 4)
     r1, r2 = ctx.to_device(np.full(nq, 0.7, dtype=np.float32)), ctx.to_device(np.full(nq, 0.2, dtype=np.float32))
     rd = ctx.to_device(capi.row_descs([(s, context, j, context + j, 0) for s in range(streams) for j in range(rows)]))
