@@ -8,7 +8,7 @@
 //   plain_tc_kernel    bfloat16, more rows: tcgen05 tensor cores.  128 weight rows (M) x up to 256 tokens (N) per tile;
 //                      a producer thread feeds 64-column slices of both operands through TMA into a ring of
 //                      128-byte-swizzled stages, one thread issues the MMAs into one of two tensor-memory accumulators,
-//                      four warps run the epilogue of the tile before.  Persistent CTAs; products with too few tiles to
+//                      eight warps run the epilogue of the tile before.  Persistent CTAs; products with too few tiles to
 //                      fill the device are cut along K, the last run of a tile to finish adds the runs in order.
 //   plain_f32_kernel   f32 throughout (fused multiply-adds on the CUDA cores): the reference-precision mode.
 //
@@ -238,7 +238,7 @@ __global__ void __launch_bounds__(256)
 constexpr int TCG_M = 128;        // weight rows per tile
 constexpr int TCG_K = 64;         // columns per stage (128 bytes: one swizzle row)
 constexpr int TCG_NMAX = 256;     // tokens per tile
-constexpr int TCG_EPI_WARPS = 4;  // warp w owns tensor-memory lanes 32 w .. 32 w + 31
+constexpr int TCG_EPI_WARPS = 8;  // warp w owns tensor-memory lanes 32 (w % 4) .. + 31 and every other run of sixteen tokens
 constexpr int TCG_THREADS = (TCG_EPI_WARPS + 2) * 32;
 constexpr int TCG_HEADER = 1024;
 constexpr int TCG_MAX_STAGES = 8;
@@ -367,23 +367,24 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
         }
         if (!ok && lane == 0) bars->failed = 1;
     } else {
-        // ---- epilogue: thread = weight row of the tile, columns = tokens
+        // ---- epilogue: two threads per weight row of the tile, columns = tokens
         pdl_wait();  // the residual stream and the cache belong to earlier kernels too
         bool ok = true;
         uint32_t tile = 0;
-        const uint32_t lane_base = (uint32_t)(warp * 32) << 16;
+        const int quad = warp & 3, first16 = (warp >> 2) * 16;
+        const uint32_t lane_base = (uint32_t)(quad * 32) << 16;
         for (int i = blockIdx.x; i < n_items; i += gridDim.x, tile++) {
             const Item w = item_of(i);
             const uint32_t buf = tile & 1;
             if (ok) ok = mbar_wait(&bars->acc_full[buf], (tile >> 1) & 1, err);
             tc_fence_after();
             const uint32_t src = tmem + lane_base + buf * (uint32_t)nt;
-            const int n = w.row * TCG_M + warp * 32 + lane;
+            const int n = w.row * TCG_M + quad * 32 + lane;
             const int tok0 = w.tok * nt, n_tok = min(nt, tokens - tok0);
             const bool pairs = w.row * TCG_M >= epi.pair_row0;
             auto finish16 = [&](int c0, const float (&v)[16]) {  // sixteen tokens of this row
                 if (pairs) {
-                    const int pair = (w.row * TCG_M - epi.pair_row0 + warp * 32) / 2 + (lane >> 4) * 8 + (lane & 7);
+                    const int pair = (w.row * TCG_M - epi.pair_row0 + quad * 32) / 2 + (lane >> 4) * 8 + (lane & 7);
 #pragma unroll
                     for (int j = 0; j < 16; j++) {
                         const float up = __shfl_down_sync(0xffffffffu, v[j], 8);
@@ -406,7 +407,7 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
                 }
             };
             if (ksplit == 1) {
-                for (int c0 = 0; c0 < n_tok; c0 += 16) {
+                for (int c0 = first16; c0 < n_tok; c0 += 32) {
                     uint32_t r[16];
                     tc_ld16(src + c0, r);
                     tc_wait_ld();
@@ -422,12 +423,12 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
                 // a run of a cut tile: leave the sums, take a ticket; whoever takes the last one adds the runs in order
                 const int tix = w.row * n_tok_tiles + w.tok;
                 float* mine = part + ((int64_t)tix * ksplit + w.run) * (TCG_M * nt);
-                for (int c0 = 0; c0 < n_tok; c0 += 16) {
+                for (int c0 = first16; c0 < n_tok; c0 += 32) {
                     uint32_t r[16];
                     tc_ld16(src + c0, r);
                     tc_wait_ld();
 #pragma unroll
-                    for (int j = 0; j < 16; j++) mine[(int64_t)(c0 + j) * TCG_M + warp * 32 + lane] = ok ? __uint_as_float(r[j]) : 0.f;
+                    for (int j = 0; j < 16; j++) mine[(int64_t)(c0 + j) * TCG_M + quad * 32 + lane] = ok ? __uint_as_float(r[j]) : 0.f;
                 }
                 tc_fence_before();
                 __syncwarp();
@@ -443,14 +444,14 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
                 if (bars->ticket == (uint32_t)ksplit - 1) {
                     __threadfence();
                     const float* all = part + (int64_t)tix * ksplit * (TCG_M * nt);
-                    for (int c0 = 0; c0 < n_tok; c0 += 16) {
+                    for (int c0 = first16; c0 < n_tok; c0 += 32) {
                         float v[16];
 #pragma unroll
                         for (int j = 0; j < 16; j++) v[j] = 0.f;
                         for (int k = 0; k < ksplit; k++) {
                             float p[16];
 #pragma unroll
-                            for (int j = 0; j < 16; j++) p[j] = __ldcg(all + (int64_t)k * (TCG_M * nt) + (int64_t)(c0 + j) * TCG_M + warp * 32 + lane);
+                            for (int j = 0; j < 16; j++) p[j] = __ldcg(all + (int64_t)k * (TCG_M * nt) + (int64_t)(c0 + j) * TCG_M + quad * 32 + lane);
 #pragma unroll
                             for (int j = 0; j < 16; j++) v[j] += p[j];
                         }
