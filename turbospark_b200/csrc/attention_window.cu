@@ -5,15 +5,16 @@
 // cp.async brings into a three-stage ring.  The one tile in shared memory serves both products: K rows as the B operand
 // of S = Q K^T (ldmatrix) and as the B operand of O += P K (ldmatrix.trans), so a key byte is read once.  SL warps share an
 // m-tile, each taking 64 / SL tokens of every tile, and meet at the end.
-//   few queries (short portions): SL = 4 or 2; many queries whose geometry the tcgen05 kernel (attention_window_tc.cu) does
+//   few queries (short portions): MT = 1, 2, 4 and SL = 4, 4, 2; many queries whose geometry the tcgen05 kernel (attention_window_tc.cu) does
 //   not take: MT = 8, SL = 1
 // Up to eight queries per key head (decoded tokens) go to window_attn8_kernel, which puts the keys on the M side.
-// A context that does not fill the device with CTAs is cut into runs of key tiles: with up to 16 queries the last CTA of a
+// A context that does not fill the device with CTAs is cut into runs of key tiles: with up to eight queries the last CTA of a
 // tile to finish - decided by a ticket, nobody waits - adds the runs in order, with more a merge launch does.
 // Only the key tiles inside the window of some query of the tile are visited; key tiles start at multiples of 64 positions
 // whatever the cut of the prompt, so a row meets its keys in the same grouping in every schedule.
 //
-// Score arithmetic in f32, base 2: v = cap log2(e) tanh(s scale / cap) - r1 log2(1 + r2 d).
+// Score arithmetic in f32, base 2: v = cap log2(e) tanh(s scale / cap) - r1 log2(1 + r2 d); tanh by its series where every
+// score of the warp's tile is well inside the cap.
 //
 // f32: one warp per (row, query head), lanes over keys for the scores and over columns for the sum; the reference-precision
 // mode, plain fused multiply-adds and the library's exp, tanh and log.
@@ -51,6 +52,52 @@ struct Geo {
         return (uint32_t)(r * PITCH + ((D <= 32 ? (c ^ ((r >> 1) & 3)) : (c ^ (r & 7))) << 4));
     }
 };
+
+// Raw scores of an mma accumulator tile -> base-2 logits with cap, bias and mask, and the lane's running maximum per query.
+// KEYS_M: rows of the tile are keys (16 per n) and columns queries; else rows are queries and columns keys (8 per n).
+// db[h]: distance of the lane's first key from its query h.
+template <int N, bool KEYS_M>
+__device__ __forceinline__ void base2_logits(float (&s)[N][4], const WindowAttn& a, const ScoreConst& sc, const float (&db)[2], const float (&r1)[2],
+                                             const float (&r2)[2], bool edge, float (&mx)[2]) {
+    if (a.cap > 0.f) {
+        float big = 0.f;
+#pragma unroll
+        for (int n = 0; n < N; n++)
+#pragma unroll
+            for (int i = 0; i < 4; i++) big = fmaxf(big, fabsf(s[n][i]));
+        if (__any_sync(0xffffffffu, big > sc.small)) {
+#pragma unroll
+            for (int n = 0; n < N; n++)
+#pragma unroll
+                for (int i = 0; i < 4; i++) s[n][i] = fmaf(-2.f * sc.c_out, rcp(ex2(s[n][i] * sc.s_in) + 1.f), sc.c_out);  // tanh(y) = 1 - 2 / (e^(2y) + 1)
+        } else {
+#pragma unroll
+            for (int n = 0; n < N; n++)
+#pragma unroll
+                for (int i = 0; i < 4; i += 2) {
+                    const float2 x = make_float2(s[n][i], s[n][i + 1]), z = mul2(x, x);
+                    const float2 v = mul2(x, fma2(z, fma2(z, fma2(z, fma2(z, both(sc.k4), both(sc.k3)), both(sc.k2)), both(sc.k1)), both(sc.k0)));
+                    s[n][i] = v.x, s[n][i + 1] = v.y;
+                }
+        }
+    } else {
+#pragma unroll
+        for (int n = 0; n < N; n++)
+#pragma unroll
+            for (int i = 0; i < 4; i++) s[n][i] *= sc.s_in;
+    }
+    const float window = a.window > 0 ? (float)a.window : 3e38f;
+#pragma unroll
+    for (int n = 0; n < N; n++)
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const int h = KEYS_M ? i & 1 : i >> 1;
+            const float dist = db[h] - (float)(KEYS_M ? n * 16 + (i >> 1) * 8 : n * 8 + (i & 1));
+            if (a.r1) s[n][i] = fmaf(-r1[h], lg2(fmaf(r2[h], dist, 1.f)), s[n][i]);
+            if (edge && (dist < 0.f || dist >= window)) s[n][i] = -INFINITY;
+            mx[h] = fmaxf(mx[h], s[n][i]);
+        }
+}
 
 // The SL warps that shared a query tile's tokens have left (m, l) and O per query in shared memory, wo[slice][QT][D + 4] and
 // wml[slice][QT].  One run: the finished rows are written.  Several runs (TICKET): the run's share goes to memory and the
@@ -201,7 +248,7 @@ __global__ void __launch_bounds__(32 * MT * SL, MT * SL <= 4 ? 3 : 1)
         const int qi = mt * 16 + gid + 8 * h;
         const bool v = qi < n_queries;
         const int row = v ? qi / grp : 0, head = kvh * grp + (v ? qi % grp : 0);
-        pq[h] = v ? pos0 + row : -1;  // an empty query slot sees nothing
+        pq[h] = pos0 + row;  // an empty slot repeats the first query and is not stored
         qp[h] = reinterpret_cast<const __nv_bfloat16*>(a.q) + (int64_t)(row_first + row) * a.q_stride + head * D;
         if (a.r1) r1[h] = a.r1[head], r2[h] = a.r2[head];
     }
@@ -226,10 +273,7 @@ __global__ void __launch_bounds__(32 * MT * SL, MT * SL <= 4 ? 3 : 1)
         }
     }
 
-    constexpr float LOG2E = 1.4426950408889634f;
-    const bool capped = a.cap > 0.f, biased = a.r1 != nullptr;
-    const float s_in = capped ? a.scale / a.cap * (2.f * LOG2E) : a.scale * LOG2E;  // capped: the exponent of e^(2 s / cap) in base 2
-    const float c_out = a.cap * LOG2E;
+    const ScoreConst sc(a);
 
     float o[NO][4];
 #pragma unroll
@@ -274,22 +318,11 @@ __global__ void __launch_bounds__(32 * MT * SL, MT * SL <= 4 ? 3 : 1)
                 mma_bf16(s[n], a1, b[2], b[3]);
             }
         }
-        // scores to base-2 logits; the mask only where the tile meets an edge
-        const bool edge = p0 + WTOK > pos0 || (a.window > 0 && p0 <= pos0 + n_rows - 1 - a.window) || n_queries < QT;
+        // the mask only where the tile meets an edge
+        const bool edge = p0 + WTOK > pos0 || (a.window > 0 && p0 <= pos0 + n_rows - 1 - a.window);
         float mx[2] = {-INFINITY, -INFINITY};
-#pragma unroll
-        for (int n = 0; n < NT8; n++)
-#pragma unroll
-            for (int i = 0; i < 4; i++) {
-                const int h = i >> 1;
-                const int dist = pq[h] - (p0 + n * 8 + 2 * tig + (i & 1));
-                float v = s[n][i] * s_in;
-                if (capped) v = fmaf(-2.f * c_out, rcp(ex2(v) + 1.f), c_out);  // tanh(y) = 1 - 2 / (e^(2y) + 1)
-                if (biased) v = fmaf(-r1[h], lg2(fmaf(r2[h], (float)dist, 1.f)), v);
-                if (edge && (dist < 0 || (a.window > 0 && dist >= a.window))) v = -INFINITY;
-                s[n][i] = v;
-                mx[h] = fmaxf(mx[h], v);
-            }
+        const float db[2] = {(float)(pq[0] - p0 - 2 * tig), (float)(pq[1] - p0 - 2 * tig)};
+        base2_logits<NT8, false>(s, a, sc, db, r1, r2, edge, mx);
         float alpha[2], m_use[2];
 #pragma unroll
         for (int h = 0; h < 2; h++) {
@@ -381,7 +414,7 @@ __global__ void __launch_bounds__(32 * MT * SL, MT * SL <= 4 ? 3 : 1)
             wml[warp * 16 + gid + 8] = make_float2(m_run[1], l_run[1]);
         }
         __syncthreads();
-        finish_slices<D, QT, SL, NTHR, MT == 1>(a, row_first, kvh, grp, n_queries, n_splits, wo, wml, part_o, part_ml, tickets);
+        finish_slices<D, QT, SL, NTHR, false>(a, row_first, kvh, grp, n_queries, n_splits, wo, wml, part_o, part_ml, tickets);
     }
 }
 
@@ -458,7 +491,7 @@ __global__ void __launch_bounds__(128, Few8<D>::PER_SM)
         const int qi = 2 * tig + h;
         const bool v = qi < n_queries;
         const int head = kvh * grp + (v ? qi % grp : 0);
-        pq[h] = v ? pos0 + qi / grp : -1;  // an empty slot sees nothing
+        pq[h] = pos0 + (v ? qi / grp : 0);  // an empty slot repeats the first query and is not stored
         if (a.r1) r1[h] = a.r1[head], r2[h] = a.r2[head];
     }
     pdl_wait();
@@ -472,10 +505,7 @@ __global__ void __launch_bounds__(128, Few8<D>::PER_SM)
 #pragma unroll
         for (int ks = 0; ks < KS; ks++) qb[ks][0] = q[8 * ks + tig], qb[ks][1] = q[8 * ks + 4 + tig];
     }
-    constexpr float LOG2E = 1.4426950408889634f;
-    const bool capped = a.cap > 0.f, biased = a.r1 != nullptr;
-    const float s_in = capped ? a.scale / a.cap * (2.f * LOG2E) : a.scale * LOG2E;
-    const float c_out = a.cap * LOG2E;
+    const ScoreConst sc(a);
     float o[NM][4];
 #pragma unroll
     for (int n = 0; n < NM; n++)
@@ -500,21 +530,10 @@ __global__ void __launch_bounds__(128, Few8<D>::PER_SM)
                 mma_bf16(s[n], k, qb[ks][0], qb[ks][1]);
             }
         }
-        const bool edge = p0 + F::WTOK > pos0 || (a.window > 0 && p0 <= pos0 + n_rows - 1 - a.window) || n_queries < 8;
+        const bool edge = p0 + F::WTOK > pos0 || (a.window > 0 && p0 <= pos0 + n_rows - 1 - a.window);
         float mx[2] = {-INFINITY, -INFINITY};
-#pragma unroll
-        for (int n = 0; n < NK; n++)
-#pragma unroll
-            for (int i = 0; i < 4; i++) {
-                const int h = i & 1;
-                const int dist = pq[h] - (p0 + n * 16 + gid + (i >> 1) * 8);
-                float v = s[n][i] * s_in;
-                if (capped) v = fmaf(-2.f * c_out, rcp(ex2(v) + 1.f), c_out);
-                if (biased) v = fmaf(-r1[h], lg2(fmaf(r2[h], (float)dist, 1.f)), v);
-                if (edge && (dist < 0 || (a.window > 0 && dist >= a.window))) v = -INFINITY;
-                s[n][i] = v;
-                mx[h] = fmaxf(mx[h], v);
-            }
+        const float db[2] = {(float)(pq[0] - p0 - gid), (float)(pq[1] - p0 - gid)};
+        base2_logits<NK, true>(s, a, sc, db, r1, r2, edge, mx);
         float alpha[2], m_use[2];
 #pragma unroll
         for (int h = 0; h < 2; h++) {
@@ -706,7 +725,7 @@ cudaError_t launch_one(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const
     if (cudaError_t e = tsb_opt_in_smem(ctx, window_attn_kernel<D, MT, SL>, smem, configured); e != cudaSuccess) return e;
     cudaError_t e = tsb_launch(ctx, window_attn_kernel<D, MT, SL>, dim3((unsigned)splits, (unsigned)a.keys.kv_heads, (unsigned)l.n_tiles), dim3(32 * MT * SL),
                                smem, st, true, a, l.tiles, l.tiles_per_group, l.rows_per_seq, l.rows_per_tile, sc.o, sc.ml, sc.tickets, ctx->dev_error);
-    return e == cudaSuccess && splits > 1 && MT > 1 ? launch_window_attn_merge(ctx, st, a, l, splits, 16 * MT, sc) : e;
+    return e == cudaSuccess && splits > 1 ? launch_window_attn_merge(ctx, st, a, l, splits, 16 * MT, sc) : e;
 }
 
 template <int D>
@@ -745,6 +764,7 @@ cudaError_t launch_small(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, con
         }
     }
     if (queries <= 16) return launch_dim<1, 4>(ctx, st, a, l, scratch);
+    if (queries <= 32) return launch_dim<2, 4>(ctx, st, a, l, scratch);
     return launch_dim<4, 2>(ctx, st, a, l, scratch);
 }
 

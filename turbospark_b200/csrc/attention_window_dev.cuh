@@ -25,6 +25,51 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 }
 __device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
 
+// Two f32 lanes per instruction.
+__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
+    float2 d;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;"
+        : "=l"(reinterpret_cast<unsigned long long&>(d))
+        : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)),
+          "l"(reinterpret_cast<const unsigned long long&>(c)));
+    return d;
+}
+__device__ __forceinline__ float2 add2(float2 a, float2 b) {
+    float2 d;
+    asm("add.rn.f32x2 %0, %1, %2;"
+        : "=l"(reinterpret_cast<unsigned long long&>(d))
+        : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)));
+    return d;
+}
+__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
+    float2 d;
+    asm("mul.rn.f32x2 %0, %1, %2;"
+        : "=l"(reinterpret_cast<unsigned long long&>(d))
+        : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)));
+    return d;
+}
+__device__ __forceinline__ float2 both(float x) { return make_float2(x, x); }
+
+// Within |y| <= TANH_SMALL, tanh(y) is its Taylor series y - y^3/3 + 2 y^5/15 - 17 y^7/315 + 62 y^9/2835; the first term left
+// out is 1382 y^11 / 155925, below 6e-8 of y there.  Scores well inside the cap - the usual case - then need no
+// special-function instruction but the softmax's own.
+constexpr float TANH_SMALL = 0.3f;
+// Constants of the way from a raw score x = q . k to a base-2 logit: c_out tanh(x scale / cap), or x s_in without a cap.
+struct ScoreConst {
+    float s_in, c_out, small, k0, k1, k2, k3, k4;
+    __device__ __forceinline__ explicit ScoreConst(const WindowAttn& a) {
+        constexpr float LOG2E = 1.4426950408889634f;
+        const bool capped = a.cap > 0.f;
+        s_in = capped ? a.scale / a.cap * (2.f * LOG2E) : a.scale * LOG2E;  // capped: the exponent of e^(2 y) in base 2
+        c_out = a.cap * LOG2E;
+        // the series in x: x (k0 + k1 x^2 + ...)
+        const float y = capped ? a.scale / a.cap : 0.f, y2 = y * y;
+        small = capped ? TANH_SMALL / fabsf(y) : 0.f;
+        k0 = c_out * y, k1 = k0 * y2 * (-1.f / 3.f), k2 = k0 * y2 * y2 * (2.f / 15.f), k3 = k0 * y2 * y2 * y2 * (-17.f / 315.f);
+        k4 = k0 * y2 * y2 * y2 * y2 * (62.f / 2835.f);
+    }
+};
+
 constexpr int WATTN_TICKETS = 16384;
 constexpr int WATTN_MAX_SPLITS = 64;
 

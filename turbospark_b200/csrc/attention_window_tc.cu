@@ -54,40 +54,11 @@ __device__ __forceinline__ void wt_g2s_2d(uint32_t dst_smem, const CUtensorMap* 
 // byte offset of 16-byte chunk c of row r in a 128-byte-swizzled tile of 128 rows: 64-column blocks of 128 rows x 128 bytes
 __device__ __forceinline__ uint32_t wt_off(int r, int c) { return (uint32_t)((c >> 3) * (128 * 128) + r * 128 + (((c & 7) ^ (r & 7)) << 4)); }
 
-// Two f32 lanes per instruction.
-__device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
-    float2 d;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;"
-        : "=l"(reinterpret_cast<unsigned long long&>(d))
-        : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)),
-          "l"(reinterpret_cast<const unsigned long long&>(c)));
-    return d;
-}
-__device__ __forceinline__ float2 add2(float2 a, float2 b) {
-    float2 d;
-    asm("add.rn.f32x2 %0, %1, %2;"
-        : "=l"(reinterpret_cast<unsigned long long&>(d))
-        : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)));
-    return d;
-}
-__device__ __forceinline__ float2 mul2(float2 a, float2 b) {
-    float2 d;
-    asm("mul.rn.f32x2 %0, %1, %2;"
-        : "=l"(reinterpret_cast<unsigned long long&>(d))
-        : "l"(reinterpret_cast<const unsigned long long&>(a)), "l"(reinterpret_cast<const unsigned long long&>(b)));
-    return d;
-}
-__device__ __forceinline__ float2 both(float x) { return make_float2(x, x); }
 __device__ __forceinline__ void st_32bytes(void* p, const uint32_t (&r)[8]) {  // one full sector per thread
     asm volatile("st.global.v8.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8};" ::"l"(p), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]),
                  "r"(r[7])
                  : "memory");
 }
-
-// Within |y| <= TANH_SMALL, tanh(y) is its Taylor series y - y^3/3 + 2 y^5/15 - 17 y^7/315 + 62 y^9/2835; the first term left
-// out is 1382 y^11 / 155925, below 6e-8 of y there.  Scores well inside the cap - the usual case - then need no
-// special-function instruction but the softmax's own.
-constexpr float TANH_SMALL = 0.3f;
 
 template <int D>
 __global__ void __launch_bounds__(WT_THREADS, 1)
@@ -248,13 +219,7 @@ __global__ void __launch_bounds__(WT_THREADS, 1)
             const uint32_t lane_base = (uint32_t)((warp & 3) * 32) << 16;
             const uint32_t col_s = tmem + lane_base + WT_COL_S + (uint32_t)x * WT_TN, col_o = tmem + lane_base + WT_COL_O + (uint32_t)x * D;
             const bool capped = a.cap > 0.f, biased = a.r1 != nullptr;
-            constexpr float LOG2E = 1.4426950408889634f;
-            const float s_in = capped ? a.scale / a.cap * (2.f * LOG2E) : a.scale * LOG2E;
-            const float c_out = a.cap * LOG2E;
-            // the series in the raw score x, y = x scale / cap: x (k0 + k1 x^2 + ...), times cap log2(e)
-            const float y_in = capped ? a.scale / a.cap : 0.f, y2 = y_in * y_in, small = capped ? TANH_SMALL / fabsf(y_in) : 0.f;
-            const float k0 = c_out * y_in, k1 = k0 * y2 * (-1.f / 3.f), k2 = k0 * y2 * y2 * (2.f / 15.f), k3 = k0 * y2 * y2 * y2 * (-17.f / 315.f),
-                        k4 = k0 * y2 * y2 * y2 * y2 * (62.f / 2835.f);
+            const ScoreConst sc(a);
             // bias tables: entry k of a head holds the bias at distance wg_first - p0 + rows_wg - 1 - k; row_l's key j is entry
             // rows_wg - 1 - row_l + j.  The pitch keeps the 32 queries of a warp on different banks.
             const int need = rows_wg + WT_TN - 1;
@@ -290,23 +255,23 @@ __global__ void __launch_bounds__(WT_THREADS, 1)
                     float big = 0.f;
 #pragma unroll
                     for (int j = 0; j < WT_TN; j++) big = fmaxf(big, fabsf(s[j]));
-                    series = !__any_sync(0xffffffffu, big > small);
+                    series = !__any_sync(0xffffffffu, big > sc.small);
                 }
                 if (capped && series) {
 #pragma unroll
                     for (int j = 0; j < WT_TN; j += 2) {
                         const float2 x = make_float2(s[j], s[j + 1]), z = mul2(x, x);
-                        const float2 w = fma2(z, fma2(z, fma2(z, fma2(z, both(k4), both(k3)), both(k2)), both(k1)), both(k0));
+                        const float2 w = fma2(z, fma2(z, fma2(z, fma2(z, both(sc.k4), both(sc.k3)), both(sc.k2)), both(sc.k1)), both(sc.k0));
                         const float2 v = fma2(x, w, biased ? make_float2(bias[j], bias[j + 1]) : both(0.f));
                         s[j] = v.x, s[j + 1] = v.y;
                     }
                 } else {
                     if (capped) {
 #pragma unroll
-                        for (int j = 0; j < WT_TN; j++) s[j] = fmaf(-2.f * c_out, rcp(ex2(s[j] * s_in) + 1.f), c_out);
+                        for (int j = 0; j < WT_TN; j++) s[j] = fmaf(-2.f * sc.c_out, rcp(ex2(s[j] * sc.s_in) + 1.f), sc.c_out);
                     } else {
 #pragma unroll
-                        for (int j = 0; j < WT_TN; j++) s[j] *= s_in;
+                        for (int j = 0; j < WT_TN; j++) s[j] *= sc.s_in;
                     }
                     if (biased) {
 #pragma unroll
