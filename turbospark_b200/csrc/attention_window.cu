@@ -5,9 +5,10 @@
 // cp.async brings into a three-stage ring.  The one tile in shared memory serves both products: K rows as the B operand
 // of S = Q K^T (ldmatrix) and as the B operand of O += P K (ldmatrix.trans), so a key byte is read once.  SL warps share an
 // m-tile, each taking 64 / SL tokens of every tile, and meet at the end.
-//   few queries (short portions): MT = 1, 2, 4 and SL = 4, 4, 2; many queries whose geometry the tcgen05 kernel (attention_window_tc.cu) does
+//   few queries (short portions): MT = 1 or 4, SL = 4 or 2; many queries whose geometry the tcgen05 kernel (attention_window_tc.cu) does
 //   not take: MT = 8, SL = 1
-// Up to eight queries per key head (decoded tokens) go to window_attn8_kernel, which puts the keys on the M side.
+// Up to eight queries per key head (decoded tokens), and 17 to 32 (verify passes) with heads of up to 128 columns, go to
+// window_attn_few_kernel: keys on the M side.
 // A context that does not fill the device with CTAs is cut into runs of key tiles: with up to eight queries the last CTA of a
 // tile to finish - decided by a ticket, nobody waits - adds the runs in order, with more a merge launch does.
 // Only the key tiles inside the window of some query of the tile are visited; key tiles start at multiples of 64 positions
@@ -418,27 +419,28 @@ __global__ void __launch_bounds__(32 * MT * SL, MT * SL <= 4 ? 3 : 1)
     }
 }
 
-// ------------------------------------------------------------------ up to eight queries per key head
-// A decoded token's heads (or a few rows of a small group) fill the N side of the mma, the keys its M side: S^T = K Q^T and
-// O^T = K^T P^T.  No multiply and no exponential goes to empty query slots, and a warp needs so few registers that four
-// CTAs share an SM.  Four warps, each a quarter of every key tile.
-template <int D>
-struct Few8 {
+// ------------------------------------------------------------------ up to 32 queries per key head
+// The queries of a decoded token or a verify pass fill the N side of the mma in tiles of eight, the keys its M side:
+// S^T = K Q^T and O^T = K^T P^T.  Hardly a multiply or an exponential goes to empty query slots, a key fragment serves every
+// query tile, and one query tile needs so few registers that four CTAs share an SM.  Four warps, each a quarter of every
+// key tile.
+template <int D, int NQ>
+struct FewQ {
     static constexpr int TILE = D <= 64 ? 128 : 64;   // tokens per key tile: 16 KB and more in flight per stage
     static constexpr int WTOK = TILE / 4, NK = WTOK / 16;
     static constexpr size_t RING = (size_t)NST * TILE * Geo<D>::PITCH;
-    static constexpr size_t MERGE = (size_t)4 * 8 * ((D + 4) * 4 + 8);
+    static constexpr size_t MERGE = (size_t)4 * 8 * NQ * ((D + 4) * 4 + 8);
     static constexpr size_t SMEM = RING > MERGE ? RING : MERGE;
-    static constexpr int PER_SM = D <= 128 ? 4 : 2;
+    static constexpr int PER_SM = D > 128 ? 2 : NQ == 1 ? 4 : NQ == 2 ? 3 : 2;
 };
 
-template <int D>
-__global__ void __launch_bounds__(128, Few8<D>::PER_SM)
-    window_attn8_kernel(const __grid_constant__ WindowAttn a, const AttnTile* __restrict__ tiles, int rows_per_seq, float* __restrict__ part_o,
+template <int D, int NQ>
+__global__ void __launch_bounds__(128, FewQ<D, NQ>::PER_SM)
+    window_attn_few_kernel(const __grid_constant__ WindowAttn a, const AttnTile* __restrict__ tiles, int rows_per_seq, float* __restrict__ part_o,
                         float2* __restrict__ part_ml, uint32_t* __restrict__ tickets, uint32_t* __restrict__ err) {
     using G = Geo<D>;
-    using F = Few8<D>;
-    constexpr int KS = D / 16, NM = D / 16, NK = F::NK;
+    using F = FewQ<D, NQ>;
+    constexpr int KS = D / 16, NM = D / 16, NK = F::NK, QT = 8 * NQ;
     extern __shared__ __align__(128) uint8_t smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
     const int kvh = blockIdx.y, n_splits = gridDim.x;
@@ -448,7 +450,7 @@ __global__ void __launch_bounds__(128, Few8<D>::PER_SM)
     const tsb_row_desc rd0 = a.rows[row_first];
     const int seq = rd0.seq, pos0 = rd0.base + rd0.slot;
     const int n_queries = n_rows * grp;
-    if (seq < 0 || seq >= a.keys.max_seqs || n_queries > 8) {
+    if (seq < 0 || seq >= a.keys.max_seqs || n_queries > QT) {
         if (threadIdx.x == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
         pdl_wait();
         return;
@@ -483,109 +485,131 @@ __global__ void __launch_bounds__(128, Few8<D>::PER_SM)
     };
     const bool early = begin + NST * F::TILE <= rd0.base;  // key tiles of earlier passes
     if (early) prologue();
-    // score columns of this lane: queries 2 tig and 2 tig + 1
-    int pq[2];
-    float r1[2] = {0.f, 0.f}, r2[2] = {0.f, 0.f};
+    // score columns of this lane: queries 2 tig and 2 tig + 1 of every query tile
+    int pq[NQ][2];
+    float r1[NQ][2], r2[NQ][2];
 #pragma unroll
-    for (int h = 0; h < 2; h++) {
-        const int qi = 2 * tig + h;
-        const bool v = qi < n_queries;
-        const int head = kvh * grp + (v ? qi % grp : 0);
-        pq[h] = pos0 + (v ? qi / grp : 0);  // an empty slot repeats the first query and is not stored
-        if (a.r1) r1[h] = a.r1[head], r2[h] = a.r2[head];
-    }
+    for (int q = 0; q < NQ; q++)
+#pragma unroll
+        for (int h = 0; h < 2; h++) {
+            const int qi = q * 8 + 2 * tig + h;
+            const bool v = qi < n_queries;
+            const int head = kvh * grp + (v ? qi % grp : 0);
+            pq[q][h] = pos0 + (v ? qi / grp : 0);  // an empty slot repeats the first query and is not stored
+            r1[q][h] = a.r1 ? a.r1[head] : 0.f, r2[q][h] = a.r1 ? a.r2[head] : 0.f;
+        }
     pdl_wait();
     if (!early) prologue();
-    // Q^T fragments: lane column n = query gid
-    uint32_t qb[KS][2];
-    {
-        const bool v = gid < n_queries;
-        const uint32_t* q = reinterpret_cast<const uint32_t*>(reinterpret_cast<const __nv_bfloat16*>(a.q) + (int64_t)(row_first + (v ? gid / grp : 0)) * a.q_stride +
-                                                              (kvh * grp + (v ? gid % grp : 0)) * D);
+    // Q^T fragments: lane column n = query gid of the tile
+    uint32_t qb[NQ][KS][2];
 #pragma unroll
-        for (int ks = 0; ks < KS; ks++) qb[ks][0] = q[8 * ks + tig], qb[ks][1] = q[8 * ks + 4 + tig];
+    for (int q = 0; q < NQ; q++) {
+        const int qi = q * 8 + gid;
+        const bool v = qi < n_queries;
+        const uint32_t* p = reinterpret_cast<const uint32_t*>(reinterpret_cast<const __nv_bfloat16*>(a.q) + (int64_t)(row_first + (v ? qi / grp : 0)) * a.q_stride +
+                                                              (kvh * grp + (v ? qi % grp : 0)) * D);
+#pragma unroll
+        for (int ks = 0; ks < KS; ks++) qb[q][ks][0] = p[8 * ks + tig], qb[q][ks][1] = p[8 * ks + 4 + tig];
     }
     const ScoreConst sc(a);
-    float o[NM][4];
+    float o[NQ][NM][4];
+    float m_run[NQ][2], l_run[NQ][2];
 #pragma unroll
-    for (int n = 0; n < NM; n++)
+    for (int q = 0; q < NQ; q++) {
 #pragma unroll
-        for (int i = 0; i < 4; i++) o[n][i] = 0.f;
-    float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+        for (int n = 0; n < NM; n++)
+#pragma unroll
+            for (int i = 0; i < 4; i++) o[q][n][i] = 0.f;
+        m_run[q][0] = m_run[q][1] = -INFINITY, l_run[q][0] = l_run[q][1] = 0.f;
+    }
     for (int tile = 0; tile < n_tiles; tile++) {
         const int stage = tile % NST;
         cp_async_wait<NST - 1>();
         __syncthreads();
         const uint32_t kt = ring + stage * (F::TILE * G::PITCH);
         const int tok0 = warp * F::WTOK, p0 = begin + tile * F::TILE + tok0;
-        float s[NK][4];  // rows gid, gid + 8 of sixteen keys x the lane's two queries
+        float s[NQ][NK][4];  // rows gid, gid + 8 of sixteen keys x the lane's two queries
 #pragma unroll
         for (int n = 0; n < NK; n++) {
 #pragma unroll
-            for (int i = 0; i < 4; i++) s[n][i] = 0.f;
+            for (int q = 0; q < NQ; q++)
+#pragma unroll
+                for (int i = 0; i < 4; i++) s[q][n][i] = 0.f;
 #pragma unroll
             for (int ks = 0; ks < KS; ks++) {
                 uint32_t k[4];
                 ldsm4(k, kt + G::off(tok0 + n * 16 + (lane & 15), ks * 2 + (lane >> 4)));
-                mma_bf16(s[n], k, qb[ks][0], qb[ks][1]);
+#pragma unroll
+                for (int q = 0; q < NQ; q++) mma_bf16(s[q][n], k, qb[q][ks][0], qb[q][ks][1]);
             }
         }
         const bool edge = p0 + F::WTOK > pos0 || (a.window > 0 && p0 <= pos0 + n_rows - 1 - a.window);
-        float mx[2] = {-INFINITY, -INFINITY};
-        const float db[2] = {(float)(pq[0] - p0 - gid), (float)(pq[1] - p0 - gid)};
-        base2_logits<NK, true>(s, a, sc, db, r1, r2, edge, mx);
-        float alpha[2], m_use[2];
+        uint32_t pb[NQ][NK][2];
 #pragma unroll
-        for (int h = 0; h < 2; h++) {
+        for (int q = 0; q < NQ; q++) {
+            float mx[2] = {-INFINITY, -INFINITY};
+            const float db[2] = {(float)(pq[q][0] - p0 - gid), (float)(pq[q][1] - p0 - gid)};
+            base2_logits<NK, true>(s[q], a, sc, db, r1[q], r2[q], edge, mx);
+            float alpha[2], m_use[2];
 #pragma unroll
-            for (int o2 = 4; o2 < 32; o2 <<= 1) mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], o2));
-            const float m_new = fmaxf(m_run[h], mx[h]);
-            m_use[h] = m_new == -INFINITY ? 0.f : m_new;
-            alpha[h] = ex2(m_run[h] - m_use[h]);
-            m_run[h] = m_new;
-            l_run[h] *= alpha[h];
+            for (int h = 0; h < 2; h++) {
+#pragma unroll
+                for (int o2 = 4; o2 < 32; o2 <<= 1) mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], o2));
+                const float m_new = fmaxf(m_run[q][h], mx[h]);
+                m_use[h] = m_new == -INFINITY ? 0.f : m_new;
+                alpha[h] = ex2(m_run[q][h] - m_use[h]);
+                m_run[q][h] = m_new;
+                l_run[q][h] *= alpha[h];
+            }
+            if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
+#pragma unroll
+                for (int n = 0; n < NM; n++) o[q][n][0] *= alpha[0], o[q][n][1] *= alpha[1], o[q][n][2] *= alpha[0], o[q][n][3] *= alpha[1];
+            }
+#pragma unroll
+            for (int n = 0; n < NK; n++) {
+                const float e0 = ex2(s[q][n][0] - m_use[0]), e1 = ex2(s[q][n][1] - m_use[1]), e2 = ex2(s[q][n][2] - m_use[0]), e3 = ex2(s[q][n][3] - m_use[1]);
+                l_run[q][0] += e0 + e2, l_run[q][1] += e1 + e3;
+                // (keys x queries) fragments to the B operand's (keys along the registers): an 8 x 8 transpose each
+                uint32_t b0 = pack_bf16(e0, e1), b1 = pack_bf16(e2, e3);
+                asm("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(pb[q][n][0]) : "r"(b0));
+                asm("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(pb[q][n][1]) : "r"(b1));
+            }
         }
-        if (__any_sync(0xffffffffu, alpha[0] != 1.f || alpha[1] != 1.f)) {
 #pragma unroll
-            for (int n = 0; n < NM; n++) o[n][0] *= alpha[0], o[n][1] *= alpha[1], o[n][2] *= alpha[0], o[n][3] *= alpha[1];
-        }
-#pragma unroll
-        for (int n = 0; n < NK; n++) {
-            const float e0 = ex2(s[n][0] - m_use[0]), e1 = ex2(s[n][1] - m_use[1]), e2 = ex2(s[n][2] - m_use[0]), e3 = ex2(s[n][3] - m_use[1]);
-            l_run[0] += e0 + e2, l_run[1] += e1 + e3;
-            // (keys x queries) fragments to the B operand's (keys along the registers): an 8 x 8 transpose each
-            uint32_t b0 = pack_bf16(e0, e1), b1 = pack_bf16(e2, e3);
-            asm("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(b0) : "r"(b0));
-            asm("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(b1) : "r"(b1));
+        for (int n = 0; n < NK; n++)
 #pragma unroll
             for (int m = 0; m < NM; m++) {
                 // K^T: rows = columns of the head, from the key rows through the transposing load
                 uint32_t k[4];
                 ldsm4_t(k, kt + G::off(tok0 + n * 16 + ((lane >> 4) << 3) + (lane & 7), m * 2 + ((lane >> 3) & 1)));
-                mma_bf16(o[m], k, b0, b1);
+#pragma unroll
+                for (int q = 0; q < NQ; q++) mma_bf16(o[q][m], k, pb[q][n][0], pb[q][n][1]);
             }
-        }
         __syncthreads();  // a stage is rewritten only after every warp is done with it
         if (tile + NST < n_tiles) issue(tile + NST, stage);
         else cp_async_commit();
     }
     cp_async_wait<0>();
     pdl_launch_dependents();
-#pragma unroll
-    for (int h = 0; h < 2; h++)
-#pragma unroll
-        for (int o2 = 4; o2 < 32; o2 <<= 1) l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], o2);
     constexpr int DP = D + 4;
     float* wo = reinterpret_cast<float*>(smem);
-    float2* wml = reinterpret_cast<float2*>(smem + (size_t)4 * 8 * DP * 4);
+    float2* wml = reinterpret_cast<float2*>(smem + (size_t)4 * QT * DP * 4);
     __syncthreads();
 #pragma unroll
-    for (int m = 0; m < NM; m++)
+    for (int q = 0; q < NQ; q++) {
 #pragma unroll
-        for (int i = 0; i < 4; i++) wo[(size_t)(warp * 8 + 2 * tig + (i & 1)) * DP + m * 16 + gid + (i >> 1) * 8] = o[m][i];
-    if (gid == 0) wml[warp * 8 + 2 * tig] = make_float2(m_run[0], l_run[0]), wml[warp * 8 + 2 * tig + 1] = make_float2(m_run[1], l_run[1]);
+        for (int h = 0; h < 2; h++)
+#pragma unroll
+            for (int o2 = 4; o2 < 32; o2 <<= 1) l_run[q][h] += __shfl_xor_sync(0xffffffffu, l_run[q][h], o2);
+        const int slot = warp * QT + q * 8 + 2 * tig;
+#pragma unroll
+        for (int m = 0; m < NM; m++)
+#pragma unroll
+            for (int i = 0; i < 4; i++) wo[(size_t)(slot + (i & 1)) * DP + m * 16 + gid + (i >> 1) * 8] = o[q][m][i];
+        if (gid == 0) wml[slot] = make_float2(m_run[q][0], l_run[q][0]), wml[slot + 1] = make_float2(m_run[q][1], l_run[q][1]);
+    }
     __syncthreads();
-    finish_slices<D, 8, 4, 128, true>(a, row_first, kvh, grp, n_queries, n_splits, wo, wml, part_o, part_ml, tickets);
+    finish_slices<D, QT, 4, 128, NQ == 1>(a, row_first, kvh, grp, n_queries, n_splits, wo, wml, part_o, part_ml, tickets);
 }
 
 // ------------------------------------------------------------------ merge of cut tiles
@@ -728,18 +752,31 @@ cudaError_t launch_one(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const
     return e == cudaSuccess && splits > 1 ? launch_window_attn_merge(ctx, st, a, l, splits, 16 * MT, sc) : e;
 }
 
-template <int D>
-cudaError_t launch_eight(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch) {
-    const int splits = wattn_splits(ctx, a, l, Few8<D>::TILE, 8, Few8<D>::PER_SM);
+template <int D, int NQ>
+cudaError_t launch_few(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch) {
+    using F = FewQ<D, NQ>;
+    const int splits = wattn_splits(ctx, a, l, F::TILE, 8 * NQ, F::PER_SM);
     const WattnScratch sc = wattn_scratch(ctx, scratch);
     static SmemOptIn configured;
-    if (cudaError_t e = tsb_opt_in_smem(ctx, window_attn8_kernel<D>, Few8<D>::SMEM, configured); e != cudaSuccess) return e;
-    return tsb_launch(ctx, window_attn8_kernel<D>, dim3((unsigned)splits, (unsigned)a.keys.kv_heads, (unsigned)l.n_tiles), dim3(128), Few8<D>::SMEM, st, true, a,
-                      l.tiles, l.rows_per_seq, sc.o, sc.ml, sc.tickets, ctx->dev_error);
+    if (cudaError_t e = tsb_opt_in_smem(ctx, window_attn_few_kernel<D, NQ>, F::SMEM, configured); e != cudaSuccess) return e;
+    cudaError_t e = tsb_launch(ctx, window_attn_few_kernel<D, NQ>, dim3((unsigned)splits, (unsigned)a.keys.kv_heads, (unsigned)l.n_tiles), dim3(128), F::SMEM,
+                               st, true, a, l.tiles, l.rows_per_seq, sc.o, sc.ml, sc.tickets, ctx->dev_error);
+    return e == cudaSuccess && splits > 1 && NQ > 1 ? launch_window_attn_merge(ctx, st, a, l, splits, 8 * NQ, sc) : e;
+}
+// query tiles by the number of queries; head sizes above 128 have registers for one
+template <int D>
+cudaError_t launch_few_dim(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, int queries, void* scratch) {
+    if (queries <= 8) return launch_few<D, 1>(ctx, st, a, l, scratch);
+    if (queries <= 16) return launch_one<D, 1, 4>(ctx, st, a, l, scratch);  // sixteen query rows of one mma tile: faster than two tiles of eight
+    if constexpr (D <= 128) {
+        if (queries <= 24) return launch_few<D, 3>(ctx, st, a, l, scratch);
+        if (queries <= 32) return launch_few<D, 4>(ctx, st, a, l, scratch);
+    }
+    return launch_one<D, 4, 2>(ctx, st, a, l, scratch);
 }
 
 template <int MT, int SL>
-cudaError_t launch_dim(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch) {
+cudaError_t launch_large(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch) {
     switch (a.keys.head_dim) {
         case 32: return launch_one<32, MT, SL>(ctx, st, a, l, scratch);
         case 64: return launch_one<64, MT, SL>(ctx, st, a, l, scratch);
@@ -752,20 +789,15 @@ cudaError_t launch_dim(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const
 }
 
 cudaError_t launch_small(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, int queries, void* scratch) {
-    if (queries <= 8) {
-        switch (a.keys.head_dim) {
-            case 32: return launch_eight<32>(ctx, st, a, l, scratch);
-            case 64: return launch_eight<64>(ctx, st, a, l, scratch);
-            case 96: return launch_eight<96>(ctx, st, a, l, scratch);
-            case 128: return launch_eight<128>(ctx, st, a, l, scratch);
-            case 192: return launch_eight<192>(ctx, st, a, l, scratch);
-            case 256: return launch_eight<256>(ctx, st, a, l, scratch);
-            default: return cudaErrorInvalidValue;
-        }
+    switch (a.keys.head_dim) {
+        case 32: return launch_few_dim<32>(ctx, st, a, l, queries, scratch);
+        case 64: return launch_few_dim<64>(ctx, st, a, l, queries, scratch);
+        case 96: return launch_few_dim<96>(ctx, st, a, l, queries, scratch);
+        case 128: return launch_few_dim<128>(ctx, st, a, l, queries, scratch);
+        case 192: return launch_few_dim<192>(ctx, st, a, l, queries, scratch);
+        case 256: return launch_few_dim<256>(ctx, st, a, l, queries, scratch);
+        default: return cudaErrorInvalidValue;
     }
-    if (queries <= 16) return launch_dim<1, 4>(ctx, st, a, l, scratch);
-    if (queries <= 32) return launch_dim<2, 4>(ctx, st, a, l, scratch);
-    return launch_dim<4, 2>(ctx, st, a, l, scratch);
 }
 
 }  // namespace
@@ -800,7 +832,7 @@ cudaError_t launch_window_attn(tsb_ctx* ctx, cudaStream_t st, bool f32, const Wi
                           0, st, true, a, b.rows, ctx->dev_error);
     const int grp = a.n_q_heads / a.keys.kv_heads, rpt = wattn_rows_per_tile(a.keys.head_dim, grp);
     auto large = [&](const WattnLaunch& l) {
-        return wattn_tc_supported(a.keys.head_dim, grp) ? launch_window_attn_tc(ctx, st, a, l, scratch) : launch_dim<8, 1>(ctx, st, a, l, scratch);
+        return wattn_tc_supported(a.keys.head_dim, grp) ? launch_window_attn_tc(ctx, st, a, l, scratch) : launch_large<8, 1>(ctx, st, a, l, scratch);
     };
     if (b.rows_per_seq > 0) {
         const int groups = b.rows / b.rows_per_seq, queries = b.rows_per_seq * grp;
