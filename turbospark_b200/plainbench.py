@@ -172,7 +172,7 @@ def kernels(ctx, peaks, shape, iters):
     mm = [e for l in lines for e in l]
     att = []
     ctx_len = 8192 if window >= 4096 else 4096
-    for streams, rows in ((1, 1), (8, 1), (64, 1), (1, 128), (1, 2048)):
+    for streams, rows in ((1, 1), (8, 1), (64, 1), (1, 6), (64, 6), (1, 128), (1, 2048)):
         it = iters if rows < 2048 else max(4, iters // 4)
         att.append(window_attention(ctx, peaks, "window attention", hd, nq, nkv, ctx_len, rows, streams, window, it))
         if rows <= 128:  # over as many keys as the window holds
