@@ -515,10 +515,9 @@ cudaError_t tcg_map(const void* p, int64_t rows, int64_t cols, int64_t stride, i
     return cudaSuccess;
 }
 
-// How a product is cut: the token tile (32 .. 256 columns) and the number of K runs whose estimated time is least.  Time
-// in units of a 64-column step of the tensor pipe: an instruction costs at least a quarter of the N = 256 one's... a step
-// is bound by the MMA (proportional to the columns, 128 at the least) or by its bytes; each item adds a fixed cost and a
-// cut tile writes and reads its sums.
+// How a product is cut: the token tile (32 .. 256 columns) and the number of K runs whose estimated time is least.  Times are
+// in steps of 64 columns at 256 tokens.  A step costs its products (an instruction narrower than 128 tokens takes as long as
+// one of 128) or its bytes, whichever is more; an item adds fixed work and its epilogue, a cut tile writes and reads its sums.
 struct TcgPlan {
     int nt, ksplit, stages;
 };
