@@ -401,38 +401,61 @@ TSB_API int32_t tsb_router_logits(tsb_ctx* ctx, tsb_stream s, const void* q_u8, 
 
 /* ------------------------------------------------------------ plain-weight decoders
  * Decoders whose matrices are plain bfloat16 (or f32) and whose layers are put together from the mechanisms below; the
- * reference has no counterpart.  One layer, in parallel form with one norm:
- *     h = x * gain / sqrt(mean(x^2) + eps)                       one gain for all coordinates
- *     x = x + mixer(shift(h)) + feed_forward(h)
+ * reference has no counterpart.  x starts as embed_scale (0: one) times the token's embedding.  A layer has one of two forms:
+ *   parallel, one norm:   h = x * gain / sqrt(mean(x^2) + eps)                       one gain for all coordinates
+ *                         x = x + mixer(shift(h)) + feed_forward(h)
+ *   post_norm:            x = norm1(residual_scale * x + mixer(x)),  x = norm2(residual_scale * x + feed_forward(x))
+ *                         norm(y) = y * (1 + w) / sqrt(mean(y^2) + eps)              w per coordinate
  *   shift (token_shift): h_t + (h_{t-1} - h_t) * mu, element by element; h_{-1} = 0
- *   mixer: causal attention whose values are its keys, n_q_heads query heads over n_kv_heads key heads;
+ *   mixer: causal attention, n_q_heads query heads over n_kv_heads key heads (see below for latent layers).
+ *     value_dim = 0: the values are the keys; else values of value_dim columns with a projection of their own.
+ *     qk_norm: queries and keys normed per head over head_dim, with a weight per column for each;
+ *     q_temp_every > 0 (with qk_norm): q times 1 + q_temp_coef * ln(floor((p + 1) / q_temp_every) + 1) at position p;
  *     score = (q . k) * score_scale;  score_cap > 0: score = score_cap * tanh(score / score_cap);
  *     log_bias: score -= r1[head] * ln(1 + r2[head] * distance);  window > 0: the last `window` positions only;
- *     head_gate: each head's output times sigmoid of one number per head, projected from the mixer's input
- *   feed_forward (ffn > 0): W_down(act(W_gate h) * (W_up h))
+ *     sink: exp(sink[head]) joins the softmax's denominator;
+ *     head_gate: each head's output times sigmoid of one number per head, projected from the mixer's input;
+ *     value_gate: every output column times sigmoid of a number of its own, projected from the mixer's input
+ *   latent mixer (kv_rank > 0): the cache holds per position c, kv_rank numbers projected and normed (plain weight), and one
+ *     rotated key part of rot_dim columns for all heads.  Head: key = [W_uk c (head_dim), rotated part], value = W_uv c
+ *     (value_dim), query = [head_dim plain, rot_dim rotated] columns.  Coordinates i and i + rot_dim / 2 are rotated by position * f_i,
+ *     f_i = rot_base^(-2 i / rot_dim); rot_factor > 0 scales the frequencies between f_i and f_i / rot_factor by how often they
+ *     turn within rot_original positions (rot_fast .. rot_slow turns), and cos and sin by 0.1 ln(rot_factor) + 1.
+ *     kv_source = j + 1: the layer has no latent of its own and reads the one of layer j (0: its own).
+ *   feed_forward (ffn > 0): W_down(act(W_gate h) * (W_up h)); a post_norm layer without one has no norm2
  * then logits = W_head norm(x), through logit_cap * tanh(logits / logit_cap) when logit_cap > 0.
- * Residual stream, norms, shift, scores, softmax and gates are f32 in both modes.  compute = TSB_BF16: matrices,
- * activations and the key cache in bfloat16 with f32 accumulation; TSB_F32: everything in f32.
- * The caches of such a model hold keys only, and per stream the last rows' h of every layer (a cursor can be moved back
- * by max_rows rows, or to 0).  Verify passes are chains; tree rounds are refused with TSB_ERR_UNSUPPORTED. */
+ * Residual stream, norms, shift, rotation, scores, softmax and gates are f32 in both modes.  compute = TSB_BF16: matrices,
+ * activations and the cache in bfloat16 with f32 accumulation; TSB_F32: everything in f32.
+ * Models with a token shift keep per stream the last rows' h of every layer (a cursor can be moved back by max_rows rows, or to
+ * 0).  Verify passes are chains; tree rounds are refused with TSB_ERR_UNSUPPORTED. */
 enum { TSB_BF16 = 0, TSB_F32 = 1 };
 enum { TSB_ACT_GELU_TANH = 0, TSB_ACT_SILU = 1 };
 typedef struct tsb_plain_config {
     int32_t n_layers, d_model, vocab, max_context, compute;
     float norm_eps, logit_cap;
+    int32_t post_norm;
+    float residual_scale, embed_scale;
 } tsb_plain_config;
 typedef struct tsb_plain_layer {
     int32_t n_q_heads, n_kv_heads, head_dim, window;
     float score_scale, score_cap;
     int32_t log_bias, head_gate, token_shift; /* 0 / 1 */
     int32_t ffn, act;
+    int32_t value_dim, qk_norm, q_temp_every;
+    float q_temp_coef;
+    int32_t sink, value_gate; /* 0 / 1 */
+    int32_t kv_rank, rot_dim, kv_source;
+    double rot_base, rot_factor, rot_original, rot_fast, rot_slow;
 } tsb_plain_layer;
 enum {
-    TSB_P_EMBED = 0, TSB_P_HEAD, TSB_P_FINAL_NORM,                     /* layer ignored; [vocab, d], [vocab, d], [1] */
-    TSB_P_NORM, TSB_P_SHIFT,                                           /* [1], [d] */
+    TSB_P_EMBED = 0, TSB_P_HEAD, TSB_P_FINAL_NORM,                     /* layer ignored; [vocab, d], [vocab, d], [1] (post_norm: [d]) */
+    TSB_P_NORM, TSB_P_SHIFT,                                           /* [1] (post_norm: norm1, [d]), [d] */
     TSB_P_Q, TSB_P_K, TSB_P_HEAD_GATE, TSB_P_R1, TSB_P_R2, TSB_P_O,    /* [H D, d], [G D, d], [H, d], [H], [H], [d, H D] */
-    TSB_P_FF_GATE, TSB_P_FF_UP, TSB_P_FF_DOWN                          /* [ffn, d], [ffn, d], [d, ffn] */
-};
+    TSB_P_FF_GATE, TSB_P_FF_UP, TSB_P_FF_DOWN,                         /* [ffn, d], [ffn, d], [d, ffn] */
+    TSB_P_NORM2, TSB_P_V, TSB_P_Q_NORM, TSB_P_K_NORM,                  /* [d], [G E, d], [D], [D] with E = value_dim */
+    TSB_P_SINK, TSB_P_VALUE_GATE,                                      /* [H], [H E, d] */
+    TSB_P_DKV, TSB_P_DKV_NORM, TSB_P_UK, TSB_P_UV                      /* [kv_rank + rot_dim, d], [kv_rank], [H D, kv_rank], [H E, kv_rank] */
+};                                                                     /* with values: W_o [d, H E]; latent layers: W_q [H (D + rot_dim), d] */
 TSB_API int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const tsb_plain_layer* layers, tsb_model** out);
 /* Upload one tensor, rows x cols row-major (vectors: rows = 1); host_type says what the host data is (TSB_BF16 / TSB_F32). */
 TSB_API int32_t tsb_model_set_plain(tsb_model* m, int32_t layer, int32_t which, int32_t host_type, const void* host, int64_t rows, int64_t cols);

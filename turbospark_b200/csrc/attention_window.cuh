@@ -1,5 +1,6 @@
-// Attention over a key-only paged cache (a layer's values are its keys), with a sliding window, a soft cap on the
-// scores, a per-head logarithmic distance bias and a per-head output gate - each of them optional.
+// Attention over a plain paged cache - a layer's values are its keys, or stand behind them - with a sliding window, a soft cap
+// on the scores, a per-head logarithmic distance bias, a per-head sink, and output gates per head or per value column - each of
+// them optional.
 #pragma once
 #include <cuda_bf16.h>
 
@@ -18,6 +19,11 @@ struct WindowAttn {
     float cap = 0.f;          // > 0: score <- cap * tanh(score / cap)
     const float *r1 = nullptr, *r2 = nullptr;  // per head: score <- score - r1 * ln(1 + r2 * distance); null: no bias
     int window = 0;           // a query sees itself and the window - 1 positions before it; 0: every earlier position
+    const float* sink = nullptr;  // per head: exp(sink) joins the softmax's denominator
+    // [rows, n_q_heads * value columns], the compute type: a head's output is multiplied by the sigmoid, column by column
+    const void* value_gate = nullptr;
+    int64_t value_gate_stride = 0;
+    int value_dim = 0;        // value columns (the heads of out and value_gate are as wide); 0: as many as a key has
 };
 
 // A query tile: consecutive rows of one stream times the query heads of one key head.
@@ -26,7 +32,7 @@ struct AttnTile {
 };
 constexpr int WATTN_SMALL_Q = 64;   // queries (rows x heads per key head) of a stream up to which the few-query kernel takes them
 constexpr int WATTN_LARGE_Q = 128;  // queries per tile of the many-query kernels (a tcgen05 CTA takes two such tiles)
-int wattn_rows_per_tile(int head_dim, int group);  // rows of a tile in the many-query kernel that takes this geometry
+int wattn_rows_per_tile(int head_dim, int group, bool biased);  // rows of a tile in the many-query kernel that takes this geometry
 
 // Where the query tiles of a pass come from: a uniform pass (rows_per_seq rows of every stream) or device lists made for
 // the layer's group size by wattn_make_tiles.
@@ -39,4 +45,9 @@ struct AttnBatch {
 size_t wattn_scratch_bytes(const tsb_ctx* ctx);  // zeroed once by the owner; the kernels leave its tickets at zero
 bool wattn_supported(int head_dim, int group, bool f32);
 int wattn_pad_dim(int head_dim, bool f32);       // the head size the kernels work on (zero columns behind the real ones); 0: too large
+// The many-query kernel for keys and values of different widths: every query head has a key head of its own, `large` tiles of
+// wattn_wide_rows rows.  0: no such kernel.
+constexpr int WATTN_WIDE_ROWS = 2 * WATTN_LARGE_Q;
+bool wattn_wide_supported(int key_dim, int value_dim);
+cudaError_t launch_window_attn_wide(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const AttnBatch& b, void* scratch);
 cudaError_t launch_window_attn(tsb_ctx* ctx, cudaStream_t st, bool f32, const WindowAttn& a, const AttnBatch& b, void* scratch);

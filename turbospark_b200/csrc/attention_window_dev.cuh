@@ -25,6 +25,25 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
 }
 __device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
 
+// What a head's sum of weighted values is multiplied by (bfloat16 kernels: m and l in base 2): one over the sum of the weights -
+// the sink's among them - times the head's gate.
+__device__ __forceinline__ float head_factor(const WindowAttn& a, int row, int head, float m, float l) {
+    if (a.sink) l += ex2(a.sink[head] * 1.4426950408889634f - (m == -INFINITY ? 0.f : m));
+    float f = l > 0.f ? 1.f / l : 0.f;
+    if (a.gate) f *= sigmoid(a.gate[(int64_t)row * a.n_q_heads + head]);
+    return f;
+}
+// the gate of value column c, and of four from c (a multiple of four) on
+__device__ __forceinline__ const __nv_bfloat16* value_gate_at(const WindowAttn& a, int row, int head, int c) {
+    return static_cast<const __nv_bfloat16*>(a.value_gate) + (int64_t)row * a.value_gate_stride + (int64_t)head * (a.value_dim > 0 ? a.value_dim : a.keys.head_dim) + c;
+}
+__device__ __forceinline__ float value_gate(const WindowAttn& a, int row, int head, int c) { return sigmoid(__bfloat162float(*value_gate_at(a, row, head, c))); }
+__device__ __forceinline__ void value_gates(const WindowAttn& a, int row, int head, int c, float4& v) {
+    const uint2 w = *reinterpret_cast<const uint2*>(value_gate_at(a, row, head, c));
+    v.x *= sigmoid(__uint_as_float(w.x << 16)), v.y *= sigmoid(__uint_as_float(w.x & 0xFFFF0000u));
+    v.z *= sigmoid(__uint_as_float(w.y << 16)), v.w *= sigmoid(__uint_as_float(w.y & 0xFFFF0000u));
+}
+
 // Two f32 lanes per instruction.
 __device__ __forceinline__ float2 fma2(float2 a, float2 b, float2 c) {
     float2 d;
@@ -95,26 +114,34 @@ inline WattnScratch wattn_scratch(const tsb_ctx* ctx, void* p) {
 }
 // How many runs the key tiles of a launch are cut into: the number whose waves come out most even.  base: CTAs of an uncut
 // launch; a CTA costs its key tiles plus about three tiles' time of fixed work, a cut tile also the merge of its runs.
-inline int wattn_splits(const tsb_ctx* ctx, const WindowAttn& a, const WattnLaunch& l, int tile_tokens, int queries_per_cta, int ctas_per_sm) {
+inline int wattn_splits(const tsb_ctx* ctx, int window, const WattnLaunch& l, int tile_tokens, int queries_per_cta, int ctas_per_sm, int base,
+                        size_t part_queries) {
     const int sms = ctx->sm_count > 0 ? ctx->sm_count : 148;
-    const int base = l.n_tiles * a.keys.kv_heads;
-    const int span = a.window > 0 && a.window + l.rows_per_tile < l.max_len ? a.window + l.rows_per_tile : l.max_len;
-    const int key_tiles = (span + tile_tokens - 1) / tile_tokens + (a.window > 0 ? 1 : 0);
+    const int span = window > 0 && window + l.rows_per_tile < l.max_len ? window + l.rows_per_tile : l.max_len;
+    const int key_tiles = (span + tile_tokens - 1) / tile_tokens + (window > 0 ? 1 : 0);
     int splits = 1;
     float best = 1e30f;
     for (int s = 1; s <= WATTN_MAX_SPLITS && s <= (key_tiles + 1) / 2; s++) {
-        if (s > 1 && ((int64_t)base * s * queries_per_cta > (int64_t)wattn_part_queries(ctx) || base > WATTN_TICKETS)) break;
+        if (s > 1 && ((int64_t)base * s * queries_per_cta > (int64_t)part_queries || base > WATTN_TICKETS)) break;
         const int waves = (base * s + ctas_per_sm * sms - 1) / (ctas_per_sm * sms);
         const float cost = (float)waves * ((float)((key_tiles + s - 1) / s) + 3.f) + (s > 1 ? 3.f + 0.1f * (float)s : 0.f);
         if (cost < best - 1e-3f) best = cost, splits = s;
     }
     return splits;
 }
+inline int wattn_splits(const tsb_ctx* ctx, const WindowAttn& a, const WattnLaunch& l, int tile_tokens, int queries_per_cta, int ctas_per_sm) {
+    return wattn_splits(ctx, a.window, l, tile_tokens, queries_per_cta, ctas_per_sm, l.n_tiles * a.keys.kv_heads, wattn_part_queries(ctx));
+}
 
 // Adds the runs of cut tiles, in order, and writes the finished rows.  A tile has `slots` query slots per run: row r of the
 // tile and head h sit in slot (r / R) * 128 + (r % R) * group + h with R = 128 / group.
 cudaError_t launch_window_attn_merge(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, int splits, int slots, const WattnScratch& sc);
 
-// The tcgen05 kernel for many queries (attention_window_tc.cu): head sizes 64 and 128, up to eight heads per key head.
-bool wattn_tc_supported(int head_dim, int group);
+// The tcgen05 kernels for many queries (attention_window_tc.cuh): head sizes 64 and 128, with a distance bias up to eight heads
+// per key head.
+bool wattn_tc_supported(int head_dim, int group, bool biased);
 cudaError_t launch_window_attn_tc(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch);
+// The kernels for caches with values of their own (attention_kv.cu, attention_kv_tc.cu).
+cudaError_t launch_kv_attn_small(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, int queries, void* scratch);
+cudaError_t launch_kv_attn_large(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch);
+cudaError_t launch_kv_attn_tc(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch);

@@ -12,8 +12,8 @@
 //                      fill the device are cut along K, the last run of a tile to finish adds the runs in order.
 //   plain_f32_kernel   f32 throughout (fused multiply-adds on the CUDA cores): the reference-precision mode.
 //
-// All three share the epilogues: residual add, logits with a soft cap, and the projection epilogue that stores queries,
-// writes keys straight into the paged cache, keeps the head gates in f32 and joins gate / up pairs.
+// All three share the epilogues: residual add, logits with a soft cap, and the projection epilogue that sends the rows of a
+// packed matrix to buffers and straight into the paged cache, joins gate / up pairs and rotates the pairs of rotary parts.
 #include <cuda.h>
 
 #include <algorithm>
@@ -41,34 +41,98 @@ __device__ __forceinline__ float activate(int act, float z) {
     return __fdividef(z, 1.f + __expf(-u));
 }
 
+__device__ __forceinline__ float get(const float* p) { return *p; }
+__device__ __forceinline__ float get(const __nv_bfloat16* p) { return __bfloat162float(*p); }
+
+// Where row n of the matrix goes (PLAIN_MIXER).
+struct SegAt {
+    int kind = -1, col = 0, gate_col = 0;  // -1: nowhere
+    void* p = nullptr;
+    int64_t stride = 0;
+    const void* gate = nullptr;
+    int64_t gate_stride = 0;
+};
+__device__ __forceinline__ SegAt seg_at(const PlainEpi& e, int n) {
+    SegAt at;
+    int first = 0;
+#pragma unroll
+    for (int k = 0; k < PLAIN_SEGS; k++) {
+        if (k >= e.n_seg) break;
+        const PlainSeg& s = e.seg[k];
+        if (n < s.end) {
+            const int g = (n - first) / s.per, i = (n - first) - g * s.per;
+            if (i < s.valid) {
+                at.kind = s.kind, at.col = g * s.step + i, at.p = s.p, at.stride = s.stride;
+                at.gate = s.gate, at.gate_stride = s.gate_stride, at.gate_col = g * s.gate_step + i;
+            }
+            break;
+        }
+        first = s.end;
+    }
+    return at;
+}
+template <typename T>
+__device__ __forceinline__ void seg_put(const PlainEpi& e, const SegAt& at, int t, float v, uint32_t* err) {
+    if (at.kind == PLAIN_SEG_TYPED) {
+        if (at.gate) {
+            const float z = get(static_cast<const T*>(at.gate) + (int64_t)t * at.gate_stride + at.gate_col);
+            v *= 1.f / (1.f + expf(-z));
+        }
+        put(static_cast<T*>(at.p) + (int64_t)t * at.stride + at.col, v);
+    } else if (at.kind == PLAIN_SEG_F32) {
+        static_cast<float*>(at.p)[(int64_t)t * at.stride + at.col] = v;
+    } else if (at.kind == PLAIN_SEG_CACHE) {
+        const tsb_row_desc& rd = e.rows[t];
+        T* p = key_row<T>(e.keys, rd.seq, rd.base + rd.slot);
+        if (p) put(p + at.stride + at.col, v);
+        else atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+    }
+}
+
 template <typename T>
 __device__ __forceinline__ void epi_one(const PlainEpi& e, int t, int n, float v, uint32_t* err) {
     if (e.kind == PLAIN_STORE) {
         if (n < e.n_valid) e.y[(int64_t)t * e.y_stride + n] = e.cap > 0.f ? e.cap * tanhf(v / e.cap) : v;
     } else if (e.kind == PLAIN_ADD) {
-        if (n < e.n_valid) e.y[(int64_t)t * e.y_stride + n] += v;
-    } else {
-        if (n < e.q_rows) {
-            put(static_cast<T*>(e.q) + (int64_t)t * e.q_stride + n, v);
-        } else if (n < e.q_rows + e.k_rows) {
-            const tsb_row_desc& rd = e.rows[t];
-            T* p = key_row<T>(e.keys, rd.seq, rd.base + rd.slot);
-            if (p) put(p + (n - e.q_rows), v);
-            else atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
-        } else if (n < e.q_rows + e.k_rows + e.gate_rows) {
-            e.gate[(int64_t)t * e.gate_rows + (n - e.q_rows - e.k_rows)] = v;
+        if (n < e.n_valid) {
+            float* y = e.y + (int64_t)t * e.y_stride + n;
+            *y = fmaf(e.alpha, *y, v);
         }
+    } else {
+        seg_put<T>(e, seg_at(e, n), t, v, err);
     }
 }
 template <typename T>
-__device__ __forceinline__ void epi_pair(const PlainEpi& e, int t, int pair, float g, float u) {
-    if (pair < e.n_pairs) put(static_cast<T*>(e.a) + (int64_t)t * e.a_stride + pair, activate<T>(e.act, g) * u);
+__device__ __forceinline__ void epi_pair(const PlainEpi& e, int t, int pair, float g, float u, uint32_t* err) {
+    if (pair >= e.n_pairs) return;
+    const PlainRotate& r = e.rot;
+    if (r.half == 0) {
+        put(static_cast<T*>(e.a) + (int64_t)t * e.a_stride + pair, activate<T>(e.act, g) * u);
+        return;
+    }
+    const int head = pair / r.half, i = pair - head * r.half;
+    const float2 cs = r.table[(int64_t)t * r.half + i];
+    const float lo = fmaf(g, cs.x, -u * cs.y), hi = fmaf(u, cs.x, g * cs.y);
+    if (head < r.n_heads) {
+#pragma unroll
+        for (int k = 0; k < 2; k++) {
+            if (!r.q[k]) continue;
+            T* p = static_cast<T*>(r.q[k]) + (int64_t)t * r.q_stride[k] + head * r.q_step[k] + r.q_off[k] + i;
+            put(p, lo), put(p + r.half, hi);
+        }
+    } else {
+        const tsb_row_desc& rd = e.rows[t];
+        T* p = key_row<T>(e.keys, rd.seq, rd.base + rd.slot);
+        if (p) put(p + r.key_off + i, lo), put(p + r.key_off + r.half + i, hi);
+        else atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+    }
 }
 
-// does any output come from the rows at and after row0 (up to the next segment)?
-__device__ __forceinline__ bool tile_used(const PlainEpi& e, int row0) {
+// does any output come from the rows at and after row0 (up to the next segment, or to the end of the group)?
+__device__ __forceinline__ bool tile_used(const PlainEpi& e, int row0, int group_rows) {
     if (row0 >= e.pair_row0) return (row0 - e.pair_row0) / 2 < e.n_pairs;
-    return row0 < (e.kind == PLAIN_MIXER ? e.q_rows + e.k_rows + e.gate_rows : e.n_valid);
+    if (e.kind != PLAIN_MIXER) return row0 < e.n_valid;
+    return e.n_seg > 0 && row0 < e.seg[e.n_seg - 1].end && (group_rows == 0 || row0 % group_rows < e.seg[0].valid);
 }
 
 // ------------------------------------------------------------------ few rows
@@ -89,8 +153,8 @@ __device__ __forceinline__ uint4 ldg_stream(const void* p) {
 // NT token tiles of eight, MT row tiles of sixteen.
 template <int NT, int MT>
 __global__ void __launch_bounds__(FEW_WARPS * 32, 2)
-    plain_few_kernel(const __nv_bfloat16* __restrict__ w, int cols, const __nv_bfloat16* x, const __nv_bfloat16* x2, int64_t x_stride, int tokens,
-                     const __grid_constant__ PlainEpi epi, uint32_t* __restrict__ err) {
+    plain_few_kernel(const __nv_bfloat16* __restrict__ w, int cols, int group_rows, int group_cols, const __nv_bfloat16* x, const __nv_bfloat16* x2,
+                     int64_t x_stride, int tokens, const __grid_constant__ PlainEpi epi, uint32_t* __restrict__ err) {
     constexpr int U = MT == 1 ? FEW_UNROLL : FEW_UNROLL / 2;
     constexpr int TOK = NT * 8, ROWS = MT * 16;
     __shared__ float red[FEW_WARPS][ROWS][TOK + 1];
@@ -98,7 +162,7 @@ __global__ void __launch_bounds__(FEW_WARPS * 32, 2)
     const int row0 = blockIdx.x * ROWS;
     const int units = cols / 64;
     const bool pairs = row0 >= epi.pair_row0;
-    if (!tile_used(epi, row0)) return;  // padding between the mixer's rows and the pairs
+    if (!tile_used(epi, row0, group_rows)) return;  // padding between the mixer's rows and the pairs, or behind a group
     const __nv_bfloat16* wp = w + (int64_t)(row0 + g) * cols + 8 * t4;
     // a unit of 64 columns is two k = 32 halves; per half the lane holds columns 8 t4 .. 8 t4 + 7 of its two rows
     uint4 wa[U][MT][4];
@@ -116,7 +180,7 @@ __global__ void __launch_bounds__(FEW_WARPS * 32, 2)
     for (int i = 0; i < U; i++)
         if (warp + i * FEW_WARPS < units) load_w(i, warp + i * FEW_WARPS);  // weights do not depend on the preceding kernel
     pdl_wait();
-    const __nv_bfloat16* xb = (pairs ? x2 : x) + (int64_t)g * x_stride + 8 * t4;
+    const __nv_bfloat16* xb = (pairs ? x2 : x) + (int64_t)g * x_stride + 8 * t4 + (group_rows ? row0 / group_rows * group_cols : 0);
     float acc[MT][NT][4];
 #pragma unroll
     for (int m = 0; m < MT; m++)
@@ -171,7 +235,7 @@ __global__ void __launch_bounds__(FEW_WARPS * 32, 2)
         for (int i = threadIdx.x; i < ROWS / 2 * tokens; i += FEW_WARPS * 32) {
             const int p = i % (ROWS / 2), t = i / (ROWS / 2);
             const int r = (p >> 3) * 16 + (p & 7);
-            epi_pair<__nv_bfloat16>(epi, t, (row0 - epi.pair_row0) / 2 + p, total(r, t), total(r + 8, t));
+            epi_pair<__nv_bfloat16>(epi, t, (row0 - epi.pair_row0) / 2 + p, total(r, t), total(r + 8, t), err);
         }
     } else {
         for (int i = threadIdx.x; i < ROWS * tokens; i += FEW_WARPS * 32) {
@@ -186,7 +250,7 @@ constexpr int F32_TILE = 64, F32_K = 16;
 // 256 threads, 64 rows x 64 tokens, 4 x 4 per thread.  A thread's four rows are {0, 8, 16, 24} + r within a 32-row half:
 // both halves of a gate / up pair are its own.
 __global__ void __launch_bounds__(256)
-    plain_f32_kernel(const float* __restrict__ w, int cols, const float* x, const float* x2, int64_t x_stride, int tokens,
+    plain_f32_kernel(const float* __restrict__ w, int cols, int group_rows, int group_cols, const float* x, const float* x2, int64_t x_stride, int tokens,
                      const __grid_constant__ PlainEpi epi, uint32_t* __restrict__ err) {
     __shared__ float ws[F32_K][F32_TILE + 4], xs[F32_K][F32_TILE + 4];
     const int row0 = blockIdx.x * F32_TILE, tok0 = blockIdx.y * F32_TILE;
@@ -194,7 +258,7 @@ __global__ void __launch_bounds__(256)
     const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
     const int rbase = (ty >> 3) * 32 + (ty & 7);
     pdl_wait();
-    const float* xb = pairs ? x2 : x;
+    const float* xb = (pairs ? x2 : x) + (group_rows ? row0 / group_rows * group_cols : 0);
     float acc[4][4] = {};
     const int lr = threadIdx.x >> 2, lc = (threadIdx.x & 3) * 4;
     for (int k0 = 0; k0 < cols; k0 += F32_K) {
@@ -225,7 +289,7 @@ __global__ void __launch_bounds__(256)
 #pragma unroll
             for (int h = 0; h < 2; h++) {
                 const int r = row0 - epi.pair_row0 + (ty >> 3) * 32 + 16 * h;  // the pair group's first row
-                epi_pair<float>(epi, t, r / 2 + (ty & 7), acc[2 * h][j], acc[2 * h + 1][j]);
+                epi_pair<float>(epi, t, r / 2 + (ty & 7), acc[2 * h][j], acc[2 * h + 1][j], err);
             }
         } else {
 #pragma unroll
@@ -261,7 +325,7 @@ __device__ __forceinline__ void tcg_g2s_2d(uint32_t dst_smem, const CUtensorMap*
 // Work item i: token tile i % n_tok_tiles, then the K run, then the row tile - neighbouring CTAs share weight rows.
 __global__ void __launch_bounds__(TCG_THREADS, 1)
     plain_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap xmap, const __grid_constant__ CUtensorMap x2map,
-                    int n_row_tiles, int n_tok_tiles, int units, int ksplit, int nt, int stages, int tokens,
+                    int n_row_tiles, int n_tok_tiles, int units, int ksplit, int nt, int stages, int tokens, int group_rows, int group_cols,
                     const __grid_constant__ PlainEpi epi, float* __restrict__ part, uint32_t* __restrict__ tickets, uint32_t* __restrict__ err) {
     extern __shared__ __align__(1024) uint8_t smem[];
     TcgBars* bars = reinterpret_cast<TcgBars*>(smem);
@@ -318,6 +382,7 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
             for (int i = blockIdx.x; i < n_items && ok; i += gridDim.x) {
                 const Item w = item_of(i);
                 const CUtensorMap* xm = w.row * TCG_M >= epi.pair_row0 ? &x2map : &xmap;
+                const int x_col0 = group_rows ? w.row * TCG_M / group_rows * group_cols : 0;  // a multiple of the stage's 64 columns
                 for (int u = 0; u < w.n && ok; u++, it++) {
                     const int s = it % stages;
                     const uint32_t dst = smem_u32(ring + s * stage_bytes);
@@ -327,7 +392,7 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
                         mbar_expect_tx(&bars->full[s], (uint32_t)stage_bytes);
                         tcg_g2s_2d(dst, &wmap, (w.u0 + u) * TCG_K, w.row * TCG_M, &bars->full[s]);
                     }
-                    tcg_g2s_2d(dst + TCG_M * 128, xm, (w.u0 + u) * TCG_K, w.tok * nt, &bars->full[s]);
+                    tcg_g2s_2d(dst + TCG_M * 128, xm, x_col0 + (w.u0 + u) * TCG_K, w.tok * nt, &bars->full[s]);
                 }
             }
             if (!ok) bars->failed = 1;
@@ -382,13 +447,14 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
             const int n = w.row * TCG_M + quad * 32 + lane;
             const int tok0 = w.tok * nt, n_tok = min(nt, tokens - tok0);
             const bool pairs = w.row * TCG_M >= epi.pair_row0;
+            const SegAt at = epi.kind == PLAIN_MIXER && !pairs ? seg_at(epi, n) : SegAt();
             auto finish16 = [&](int c0, const float (&v)[16]) {  // sixteen tokens of this row
                 if (pairs) {
                     const int pair = (w.row * TCG_M - epi.pair_row0 + quad * 32) / 2 + (lane >> 4) * 8 + (lane & 7);
 #pragma unroll
                     for (int j = 0; j < 16; j++) {
                         const float up = __shfl_down_sync(0xffffffffu, v[j], 8);
-                        if (!(lane & 8) && c0 + j < n_tok) epi_pair<__nv_bfloat16>(epi, tok0 + c0 + j, pair, v[j], up);
+                        if (!(lane & 8) && c0 + j < n_tok) epi_pair<__nv_bfloat16>(epi, tok0 + c0 + j, pair, v[j], up, err);
                     }
                 } else if (epi.kind == PLAIN_ADD) {
                     // the loads of sixteen tokens are in flight together
@@ -399,7 +465,11 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
                     for (int j = 0; j < 16; j++) old[j] = in && c0 + j < n_tok ? y[(int64_t)j * epi.y_stride] : 0.f;
 #pragma unroll
                     for (int j = 0; j < 16; j++)
-                        if (in && c0 + j < n_tok) y[(int64_t)j * epi.y_stride] = old[j] + v[j];
+                        if (in && c0 + j < n_tok) y[(int64_t)j * epi.y_stride] = fmaf(epi.alpha, old[j], v[j]);
+                } else if (epi.kind == PLAIN_MIXER) {
+#pragma unroll
+                    for (int j = 0; j < 16; j++)
+                        if (c0 + j < n_tok) seg_put<__nv_bfloat16>(epi, at, tok0 + c0 + j, v[j], err);
                 } else {
 #pragma unroll
                     for (int j = 0; j < 16; j++)
@@ -559,7 +629,7 @@ cudaError_t launch_few(tsb_ctx* ctx, cudaStream_t st, const PlainMat& w, const _
     // last attention CTAs are packed on few SMs and run with their small L1 - 67 to 75 us instead of 27 at 4096 x 18432.
     const bool ahead = epi.kind != PLAIN_ADD;
     return tsb_launch(ctx, plain_few_kernel<NT, MT>, dim3((unsigned)(w.rows / (16 * MT))), dim3(FEW_WARPS * 32), 0, st, ahead,
-                      (const __nv_bfloat16*)w.data, (int)w.cols, x, x2, x_stride, tokens, epi, ctx->dev_error);
+                      (const __nv_bfloat16*)w.data, (int)w.cols, w.group_rows, w.group_cols, x, x2, x_stride, tokens, epi, ctx->dev_error);
 }
 
 constexpr int FEW_MAX = 16;  // token rows up to which the weight-streaming kernel runs
@@ -576,8 +646,8 @@ cudaError_t launch_plain_gemm(tsb_ctx* ctx, cudaStream_t st, bool f32, const Pla
     if (tokens <= 0) return cudaSuccess;
     if (f32) {
         dim3 grid((unsigned)(w.rows / F32_TILE), (unsigned)((tokens + F32_TILE - 1) / F32_TILE));
-        return tsb_launch(ctx, plain_f32_kernel, grid, dim3(256), 0, st, true, (const float*)w.data, (int)w.cols, (const float*)x, (const float*)x2,
-                          x_stride, tokens, epi, ctx->dev_error);
+        return tsb_launch(ctx, plain_f32_kernel, grid, dim3(256), 0, st, true, (const float*)w.data, (int)w.cols, w.group_rows, w.group_cols,
+                          (const float*)x, (const float*)x2, x_stride, tokens, epi, ctx->dev_error);
     }
     const __nv_bfloat16 *xb = (const __nv_bfloat16*)x, *xb2 = (const __nv_bfloat16*)x2;
     if (tokens <= FEW_MAX) {
@@ -589,8 +659,9 @@ cudaError_t launch_plain_gemm(tsb_ctx* ctx, cudaStream_t st, bool f32, const Pla
     const TcgPlan p = tcg_plan(ctx, row_tiles, units, tokens);
     CUtensorMap wm, xm, xm2;
     cudaError_t e = tcg_map(w.data, w.rows, w.cols, w.cols, TCG_M, &wm);
-    if (e == cudaSuccess) e = tcg_map(x, x_rows, w.cols, x_stride, p.nt, &xm);
-    if (e == cudaSuccess) e = tcg_map(x2 ? x2 : x, x_rows, w.cols, x_stride, p.nt, &xm2);
+    const int64_t x_cols = w.group_rows ? (w.rows / w.group_rows - 1) * w.group_cols + w.cols : w.cols;
+    if (e == cudaSuccess) e = tcg_map(x, x_rows, x_cols, x_stride, p.nt, &xm);
+    if (e == cudaSuccess) e = tcg_map(x2 ? x2 : x, x_rows, x_cols, x_stride, p.nt, &xm2);
     if (e != cudaSuccess) return e;
     static SmemOptIn configured;
     if ((e = tsb_opt_in_smem(ctx, plain_tc_kernel, (size_t)TCG_SMEM_CAP, configured)) != cudaSuccess) return e;
@@ -600,5 +671,5 @@ cudaError_t launch_plain_gemm(tsb_ctx* ctx, cudaStream_t st, bool f32, const Pla
     float* part = reinterpret_cast<float*>(tickets + TCG_TICKETS);
     const size_t smem = TCG_HEADER + (size_t)p.stages * (TCG_M + p.nt) * 128;
     return tsb_launch(ctx, plain_tc_kernel, dim3((unsigned)std::min(items, ctx->sm_count)), dim3(TCG_THREADS), smem, st, true, wm, xm, xm2, row_tiles,
-                      tok_tiles, units, p.ksplit, p.nt, p.stages, tokens, epi, part, tickets, ctx->dev_error);
+                      tok_tiles, units, p.ksplit, p.nt, p.stages, tokens, w.group_rows, w.group_cols, epi, part, tickets, ctx->dev_error);
 }

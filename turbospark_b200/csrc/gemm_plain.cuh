@@ -16,9 +16,37 @@ inline int64_t plain_pad(int64_t n, int64_t to) { return (n + to - 1) / to * to;
 
 enum PlainEpiKind {
     PLAIN_STORE = 0,  // y[t, n] = acc, through cap * tanh(acc / cap) when cap > 0
-    PLAIN_ADD = 1,    // y[t, n] += acc  (the residual stream)
-    PLAIN_MIXER = 2,  // the projections of a layer, by row: queries, keys straight into the cache, head gates, then
-                      // gate / up pairs of the feed-forward as act(gate) * up
+    PLAIN_ADD = 1,    // y[t, n] = alpha * y[t, n] + acc  (the residual stream)
+    PLAIN_MIXER = 2,  // by row of the matrix: segments with destinations of their own, then pairs of rows (gate and up of a
+                      // feed-forward as act(gate) * up, or the two coordinates of a rotation)
+};
+// Where the rows of a segment go.
+enum PlainSegKind {
+    PLAIN_SEG_TYPED = 0,  // an activation buffer of the compute type
+    PLAIN_SEG_F32 = 1,    // an f32 buffer
+    PLAIN_SEG_CACHE = 2,  // the cache row of the token
+};
+// Rows [end of the segment before, end) in groups of `per`, of which the first `valid` are kept: row i of group g lands at
+// element g * step + i of the token's row, which starts at p + t * stride (or, in the cache, `stride` elements into its row).
+struct PlainSeg {
+    int end = 0, kind = PLAIN_SEG_TYPED;
+    int per = 0x7fffffff, valid = 0x7fffffff, step = 0;
+    void* p = nullptr;
+    int64_t stride = 0;
+    const void* gate = nullptr;  // PLAIN_SEG_TYPED: times sigmoid of element g * gate_step + i of row t of this buffer (compute type)
+    int64_t gate_stride = 0;
+    int gate_step = 0;
+};
+constexpr int PLAIN_SEGS = 6;
+// Pairs (u, v) as coordinates i and i + half of a rotated part: u c - v s and v c + u s with (c, s) of the token's position.
+// Pair p belongs to head p / half; heads below n_heads are queries, the one behind them the key.
+struct PlainRotate {
+    int half = 0, n_heads = 0;           // half 0: no rotation
+    const float2* table = nullptr;       // [t, half]
+    void* q[2] = {nullptr, nullptr};     // one or two query buffers: element (head * q_step + q_off) of row t
+    int64_t q_stride[2] = {0, 0};
+    int q_step[2] = {0, 0}, q_off[2] = {0, 0};
+    int key_off = 0;                     // the key's elements start here in the cache row
 };
 enum PlainAct { PLAIN_GELU_TANH = 0, PLAIN_SILU = 1 };
 
@@ -27,14 +55,13 @@ struct PlainEpi {
     int n_valid = 0;       // PLAIN_STORE / PLAIN_ADD: rows of the matrix that have an output column
     float* y = nullptr;
     int64_t y_stride = 0;
-    float cap = 0.f;
+    float cap = 0.f, alpha = 1.f;
     // PLAIN_MIXER
-    void* q = nullptr;     // [t, q_rows], the compute type
-    int64_t q_stride = 0;
-    int q_rows = 0, k_rows = 0, gate_rows = 0;
+    PlainSeg seg[PLAIN_SEGS];
+    int n_seg = 0;
     KeyView keys{};
     const tsb_row_desc* rows = nullptr;
-    float* gate = nullptr;  // [t, gate_rows]: the gates' pre-activations
+    PlainRotate rot;             // half > 0: the pairs are rotated coordinates
     int pair_row0 = 0x7fffffff;  // the matrix row where the interleaved pairs start (a multiple of PLAIN_ROW_PAD)
     int n_pairs = 0, act = PLAIN_GELU_TANH;
     void* a = nullptr;      // [t, n_pairs], the compute type
@@ -44,6 +71,9 @@ struct PlainEpi {
 struct PlainMat {
     void* data = nullptr;     // bfloat16 or f32
     int64_t rows = 0, cols = 0;  // padded
+    // A block-diagonal product: rows of group g (group_rows each, a multiple of PLAIN_ROW_PAD) multiply the columns of x from
+    // g * group_cols on.  0: every row multiplies the same columns.
+    int group_rows = 0, group_cols = 0;
 };
 
 // Split sums of products with few row tiles: tickets, then f32 tiles.

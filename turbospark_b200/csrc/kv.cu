@@ -116,7 +116,7 @@ __global__ void kv_fill_random_kernel(KvView kv, int seq, int tokens, uint64_t s
 }
 
 __global__ void keys_fill_random_kernel(KeyView kv, int seq, int tokens, uint32_t seed) {
-    const int row = kv.kv_heads * kv.head_dim;
+    const int row = kv.row;
     const int64_t total = (int64_t)tokens * row;
     for (int64_t i = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (int64_t)gridDim.x * blockDim.x) {
         const int pos = (int)(i / row), e = (int)(i - (int64_t)pos * row);
@@ -185,8 +185,8 @@ int32_t pool_alloc(tsb_ctx* ctx, size_t bytes, void** out) {
 
 }  // namespace
 
-int32_t kv_create_keys(tsb_ctx* ctx, int n_layers, const int32_t* kv_heads, const int32_t* head_dims, int elem_bytes, int page_tokens, int num_pages,
-                       int max_seqs, int max_pages_per_seq, tsb_kv** out) {
+int32_t kv_create_keys(tsb_ctx* ctx, int n_layers, const KeyLayerShape* shapes, int elem_bytes, int page_tokens, int num_pages, int max_seqs,
+                       int max_pages_per_seq, tsb_kv** out) {
     *out = nullptr;
     TSB_REQUIRE(ctx, n_layers > 0 && num_pages > 0 && max_seqs > 0 && max_pages_per_seq > 0, "bad sizes");
     TSB_REQUIRE(ctx, elem_bytes == 2 || elem_bytes == 4, "keys are bfloat16 or f32");
@@ -196,10 +196,14 @@ int32_t kv_create_keys(tsb_ctx* ctx, int n_layers, const int32_t* kv_heads, cons
     if (!kv) return TSB_ERR_OOM;
     int32_t rc = kv_init_pages(ctx, kv, page_tokens, num_pages, max_seqs, max_pages_per_seq);
     size_t bytes = 0;
+    auto row_of = [&](int l) { return shapes[l].kv_heads * shapes[l].head_dim * (shapes[l].values ? 2 : 1); };
     for (int l = 0; l < n_layers && rc == TSB_OK; l++) {
-        if (kv_heads[l] <= 0 || head_dims[l] <= 0 || (head_dims[l] * elem_bytes) % 16)
+        const KeyLayerShape& k = shapes[l];
+        if (k.kv_heads <= 0 || k.head_dim <= 0 || (k.head_dim * elem_bytes) % 16)
             rc = tsb_fail(ctx, TSB_ERR_INVALID, "layer %d: bad head count or head size", l);
-        bytes += (size_t)num_pages * page_tokens * kv_heads[l] * head_dims[l] * elem_bytes;
+        else if (k.source < 0 || k.source > l || shapes[k.source].source != k.source || row_of(k.source) != row_of(l))
+            rc = tsb_fail(ctx, TSB_ERR_INVALID, "layer %d cannot read the rows of layer %d", l, k.source);
+        if (k.source == l) bytes += (size_t)num_pages * page_tokens * row_of(l) * elem_bytes;
     }
     if (rc == TSB_OK) rc = pool_alloc(ctx, bytes, (void**)&kv->key_pool);
     if (rc) {
@@ -210,12 +214,14 @@ int32_t kv_create_keys(tsb_ctx* ctx, int n_layers, const int32_t* kv_heads, cons
     size_t off = 0;
     for (int l = 0; l < n_layers; l++) {
         KeyView k;
-        k.base = kv->key_pool + off, k.page_table = kv->page_table_dev;
-        k.kv_heads = kv_heads[l], k.head_dim = head_dims[l], k.elem_bytes = elem_bytes;
+        const bool own = shapes[l].source == l;
+        k.base = own ? kv->key_pool + off : kv->key_layers[shapes[l].source].base, k.page_table = kv->page_table_dev;
+        k.kv_heads = shapes[l].kv_heads, k.head_dim = shapes[l].head_dim, k.elem_bytes = elem_bytes;
+        k.row = row_of(l), k.value_off = shapes[l].values ? k.head_dim : 0, k.head_step = k.head_dim + k.value_off;
         k.page_shift = kv->view.page_shift, k.page_tokens = page_tokens, k.num_pages = num_pages;
         k.max_seqs = max_seqs, k.max_pages_per_seq = max_pages_per_seq;
         kv->key_layers.push_back(k);
-        off += (size_t)num_pages * page_tokens * kv_heads[l] * head_dims[l] * elem_bytes;
+        if (own) off += (size_t)num_pages * page_tokens * k.row * elem_bytes;
     }
     *out = kv;
     return TSB_OK;
@@ -359,9 +365,9 @@ static int32_t kv_copy_rows(tsb_kv* kv, tsb_stream s, int32_t seq, int32_t layer
     if (pos0 + n > (int64_t)kv->pages_of_seq[seq] * v.page_tokens)
         return tsb_fail(ctx, TSB_ERR_STATE, "rows %lld..%lld are not reserved", (long long)pos0, (long long)(pos0 + n));
     DeviceGuard g(ctx);
-    // bytes of a row, and where the layer's K and V halves start (a key-only cache has one half)
+    // bytes of a row, and where the layer's K and V halves start (a plain cache has one)
     const KeyView* kl = keys ? &kv->key_layers[layer] : nullptr;
-    const size_t row = keys ? (size_t)kl->kv_heads * kl->head_dim * kl->elem_bytes : (size_t)v.kv_heads * v.head_dim * sizeof(__half);
+    const size_t row = keys ? (size_t)kl->row * kl->elem_bytes : (size_t)v.kv_heads * v.head_dim * sizeof(__half);
     const int32_t* pt = &kv->page_table_host[(size_t)seq * v.max_pages_per_seq];
     int64_t p = pos0;
     while (p < pos0 + n) {  // one copy per page run
@@ -409,7 +415,7 @@ int32_t tsb_rope_store_kv(tsb_ctx* ctx, tsb_stream s, tsb_kv* kv, int32_t layer,
     if (!ctx || !kv) return TSB_ERR_INVALID;
     TSB_REQUIRE(ctx, qkv_f16 && rows_dev && rows > 0 && n_q_heads > 0, "bad arguments");
     TSB_REQUIRE(ctx, layer >= 0 && layer < kv->view.layers, "layer %d outside 0..%d", layer, kv->view.layers);
-    TSB_REQUIRE(ctx, kv->view.pool, "a key-only cache has no value rows");
+    TSB_REQUIRE(ctx, kv->view.pool, "a plain cache takes no rotated f16 rows");
     DeviceGuard g(ctx);
     TSB_CUDA(ctx, launch_rope_store_kv(ctx, (cudaStream_t)s, kv, layer, (__half*)qkv_f16, rows_dev, rows, n_q_heads, theta));
     return TSB_OK;
@@ -431,7 +437,7 @@ int32_t tsb_kv_commit_path(tsb_ctx* ctx, tsb_stream s, tsb_kv* kv, int32_t seq, 
     bool identity = true;
     for (int r = 0; r < keep; r++) identity &= host_path[r] == (uint32_t)r;
     if (identity) return TSB_OK;  // a chain: nothing to move
-    if (!kv->key_layers.empty()) return tsb_fail(ctx, TSB_ERR_UNSUPPORTED, "a key-only cache keeps chains, not tree paths");
+    if (!kv->key_layers.empty()) return tsb_fail(ctx, TSB_ERR_UNSUPPORTED, "a plain cache keeps chains, not tree paths");
     DeviceGuard g(ctx);
     cudaStream_t st = (cudaStream_t)s;
     uint32_t* dpath = nullptr;

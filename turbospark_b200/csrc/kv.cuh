@@ -16,19 +16,30 @@ struct KvView {
     int64_t layer_stride;  // elements between layers
 };
 
-// One layer of a key-only cache (layers whose values are their keys): rows of kv_heads * head_dim elements, f32 or
-// bfloat16, [page][token_in_page][kv_head][head_dim].  Layers may differ in both.
+// One layer of a plain cache: token rows of `row` elements, f32 or bfloat16, [page][token_in_page][row].  A row holds
+// kv_heads heads, head_step elements apart; a head's key is head_dim elements from its start, its value starts value_off
+// elements behind it:
+//   values that are their keys   head_step = head_dim, value_off = 0
+//   keys and values              head_step = 2 head_dim, value_off = head_dim
+//   latent rows                  one head: the latent, which is also the value, then the rotated key part
+// Layers may differ in all of it.
 struct KeyView {
     uint8_t* base;
     const int32_t* page_table;
     int kv_heads, head_dim, elem_bytes;
+    int row, head_step, value_off;
     int page_shift, page_tokens, num_pages, max_seqs, max_pages_per_seq;
+};
+struct KeyLayerShape {
+    int kv_heads, head_dim;
+    bool values;   // a value of head_dim elements behind every key
+    int source;    // the layer whose rows this one reads (itself: rows of its own)
 };
 
 struct tsb_kv {
     tsb_ctx* ctx = nullptr;
     KvView view{};                    // page geometry; pool and strides of a key + value cache
-    std::vector<KeyView> key_layers;  // not empty: a key-only cache (view.pool is then null)
+    std::vector<KeyView> key_layers;  // not empty: a plain cache (view.pool is then null)
     uint8_t* key_pool = nullptr;
     // A model whose rows also need their predecessors' state keeps the last state_ring - 1 rows' worth of it per stream
     // (0: no such state).  state_lo is the oldest position whose state is still there: a cursor may go back to 0 or to
@@ -42,21 +53,21 @@ struct tsb_kv {
     std::vector<int64_t> cursor;
 };
 
-// A key-only cache of n_layers layers with their own head counts and (padded) head sizes.
-int32_t kv_create_keys(tsb_ctx* ctx, int n_layers, const int32_t* kv_heads, const int32_t* head_dims, int elem_bytes, int page_tokens, int num_pages,
-                       int max_seqs, int max_pages_per_seq, tsb_kv** out);
-// Seeded pseudo-random rows [0, tokens) of a stream in every layer of a key-only cache (reserves the pages).
+// A plain cache of n_layers layers with their own head counts and (padded) head sizes.
+int32_t kv_create_keys(tsb_ctx* ctx, int n_layers, const KeyLayerShape* shapes, int elem_bytes, int page_tokens, int num_pages, int max_seqs,
+                       int max_pages_per_seq, tsb_kv** out);
+// Seeded pseudo-random rows [0, tokens) of a stream in every layer of a plain cache (reserves the pages).
 int32_t kv_fill_keys(tsb_kv* kv, cudaStream_t st, int32_t seq, int64_t tokens, uint64_t seed);
 
 #ifdef __CUDACC__
-// Row of a key-only layer at position `pos` of stream `seq`; nullptr outside the reserved pages.
+// Row of a plain layer at position `pos` of stream `seq`; nullptr outside the reserved pages.
 template <typename T>
 __device__ __forceinline__ T* key_row(const KeyView& kv, int seq, int pos) {
     const int lp = pos >> kv.page_shift;
     if (pos < 0 || seq < 0 || seq >= kv.max_seqs || lp >= kv.max_pages_per_seq) return nullptr;
     const int page = kv.page_table[(size_t)seq * kv.max_pages_per_seq + lp];
     if (page < 0) return nullptr;
-    return reinterpret_cast<T*>(kv.base) + ((int64_t)page * kv.page_tokens + (pos & (kv.page_tokens - 1))) * ((int64_t)kv.kv_heads * kv.head_dim);
+    return reinterpret_cast<T*>(kv.base) + ((int64_t)page * kv.page_tokens + (pos & (kv.page_tokens - 1))) * kv.row;
 }
 // Row of (layer, which = 0 K / 1 V) holding position `pos` of stream `seq`; nullptr when the
 // position is outside the reserved pages (the caller records TSB_DEV_BAD_INDEX and skips).

@@ -1,13 +1,21 @@
 // The plain-weight decoder family (tsb_model_create_plain): models, session buffers, forward pass.
 //
-// A layer is four launches, plus the embedding before the first and norm + head after the last:
+// A layer in parallel form is four launches, plus the embedding before the first and norm + head after the last:
 //   norm + token shift           f32 residual stream -> the mixer's input and the feed-forward's input
 //   input matmul                 one packed matrix over queries | keys | head gates | gate-up pairs; its epilogue stores the
 //                                queries, writes the keys into their cache slots, keeps the gates in f32 and leaves
 //                                act(gate) * up beside the attention output
-//   window attention             over the key-only cache, gate applied where a head's output is finished
+//   window attention             over the cache, gate applied where a head's output is finished
 //   output matmul                [W_o | W_down] over [heads | feed-forward]: the two sublayers of a parallel layer add up
 //                                inside one product, whose epilogue adds it to the stream
+// In post-norm form the sublayers follow each other, each ending in an output matmul that adds to the scaled stream and a norm
+// that rewrites the stream (f32) and its copy in the compute type.  Mixers of that form:
+//   keys and values              input matmul over queries | keys | values (values go straight to the cache); norm per head of queries
+//                                and keys, which writes the cache; attention
+//   latent                       input matmul over queries | latent | value gates | rotated pairs, whose epilogue rotates queries
+//                                and the shared key part in f32 and stores the latter in the cache; norm of the latent into the cache; then
+//                                short portions: absorb (queries to the latent's space), attention over latent rows, lift (sums of
+//                                latents to gated values); long portions: expansion of the stream's latents to keys and values, attention
 #include <algorithm>
 #include <cstring>
 #include <new>
@@ -72,24 +80,40 @@ int32_t plain_complete(const tsb_model* tm) {
     TSB_REQUIRE(ctx, (m->set & want) == want, "embedding, head or final norm missing");
     for (size_t i = 0; i < m->layers.size(); i++) {
         const PlainLayer& l = m->layers[i];
-        uint32_t w = 1u << TSB_P_NORM | 1u << TSB_P_Q | 1u << TSB_P_K | 1u << TSB_P_O;
+        uint32_t w = 1u << TSB_P_NORM | 1u << TSB_P_Q | 1u << TSB_P_O;
+        if (l.mixer == MIX_LATENT) {
+            w |= 1u << TSB_P_UK | 1u << TSB_P_UV;
+            if (l.source == (int)i) w |= 1u << TSB_P_DKV | 1u << TSB_P_DKV_NORM;
+        } else {
+            w |= 1u << TSB_P_K;
+        }
+        if (l.mixer == MIX_KV) w |= 1u << TSB_P_V;
+        if (l.cfg.qk_norm) w |= 1u << TSB_P_Q_NORM | 1u << TSB_P_K_NORM;
+        if (l.cfg.sink) w |= 1u << TSB_P_SINK;
+        if (l.cfg.value_gate) w |= 1u << TSB_P_VALUE_GATE;
         if (l.cfg.token_shift) w |= 1u << TSB_P_SHIFT;
         if (l.cfg.head_gate) w |= 1u << TSB_P_HEAD_GATE;
         if (l.cfg.log_bias) w |= 1u << TSB_P_R1 | 1u << TSB_P_R2;
         if (l.cfg.ffn > 0) w |= 1u << TSB_P_FF_GATE | 1u << TSB_P_FF_UP | 1u << TSB_P_FF_DOWN;
+        if (l.cfg.ffn > 0 && l.post_norm) w |= 1u << TSB_P_NORM2;
         TSB_REQUIRE(ctx, (l.set & w) == w, "layer %zu is missing a tensor (have %x, need %x)", i, l.set, w);
     }
     return TSB_OK;
+}
+
+void free_layer(tsb_ctx* ctx, PlainLayer& l) {
+    if (!l.owned) return;
+    for (void** p : l.buffers())
+        if (*p) tsb_free(ctx, *p);
 }
 
 void plain_free(tsb_model* tm) {
     PlainModel* m = tm->plain;
     if (!m) return;
     tsb_ctx* ctx = tm->ctx;
-    for (PlainLayer& l : m->layers)
-        if (l.owned)
-            for (void* p : {l.in.data, l.out.data, (void*)l.gain, (void*)l.mu, (void*)l.r1, (void*)l.r2})
-                if (p) tsb_free(ctx, p);
+    for (PlainLayer& l : m->layers) free_layer(ctx, l);
+    for (PlainRotation& r : m->rotations)
+        if (r.freq) tsb_free(ctx, r.freq);
     if (m->owned)
         for (void* p : {m->head.data, m->embed, (void*)m->final_gain})
             if (p) tsb_free(ctx, p);
@@ -97,14 +121,24 @@ void plain_free(tsb_model* tm) {
     tm->plain = nullptr;
 }
 
+// numbers of a layer's matrices that a pass over few rows reads
+int64_t layer_numbers(const PlainLayer& l, int64_t d) {
+    const tsb_plain_layer& c = l.cfg;
+    const int64_t H = c.n_q_heads, G = c.n_kv_heads, D = c.head_dim, E = l.mixer == MIX_KEYS ? D : c.value_dim;
+    int64_t n = d * (H * E + (c.head_gate ? H : 0) + (c.value_gate ? H * E : 0) + 3 * (int64_t)c.ffn);
+    if (l.mixer == MIX_LATENT) {
+        n += d * H * (D + c.rot_dim) + (int64_t)c.kv_rank * H * (D + E);
+        if (c.kv_source == 0) n += d * (c.kv_rank + c.rot_dim);
+    } else {
+        n += d * (H * D + G * D + (l.mixer == MIX_KV ? G * E : 0));
+    }
+    return n;
+}
 // bytes a pass reads of the matrices (the embedding is read by rows and not counted)
 int64_t plain_weight_bytes(const tsb_model* tm) {
     const PlainModel* m = tm->plain;
     int64_t n = (int64_t)m->cfg.vocab * m->cfg.d_model;
-    for (const PlainLayer& l : m->layers) {
-        const tsb_plain_layer& c = l.cfg;
-        n += (int64_t)m->cfg.d_model * ((int64_t)c.head_dim * (2 * c.n_q_heads + c.n_kv_heads) + (c.head_gate ? c.n_q_heads : 0) + 3 * (int64_t)c.ffn);
-    }
+    for (const PlainLayer& l : m->layers) n += layer_numbers(l, m->cfg.d_model);
     return n * m->elem;
 }
 
@@ -112,7 +146,8 @@ int32_t plain_share(tsb_model* dt, int32_t dst_layer, const tsb_model* st, int32
     tsb_ctx* ctx = dt->ctx;
     PlainModel* d = dt->plain;
     const PlainModel* s = st->plain;
-    TSB_REQUIRE(ctx, d->cfg.d_model == s->cfg.d_model && d->cfg.vocab == s->cfg.vocab && d->f32 == s->f32, "models differ in width, vocabulary or type");
+    TSB_REQUIRE(ctx, d->cfg.d_model == s->cfg.d_model && d->cfg.vocab == s->cfg.vocab && d->f32 == s->f32 && d->cfg.post_norm == s->cfg.post_norm,
+                "models differ in width, vocabulary, type or form");
     if (dst_layer < 0) {
         if (d->owned)
             for (void* p : {d->head.data, d->embed, (void*)d->final_gain})
@@ -123,10 +158,10 @@ int32_t plain_share(tsb_model* dt, int32_t dst_layer, const tsb_model* st, int32
     TSB_REQUIRE(ctx, dst_layer < d->cfg.n_layers && src_layer >= 0 && src_layer < s->cfg.n_layers, "layer out of range");
     PlainLayer& l = d->layers[dst_layer];
     TSB_REQUIRE(ctx, memcmp(&l.cfg, &s->layers[src_layer].cfg, sizeof l.cfg) == 0, "layer shapes differ");
-    if (l.owned)
-        for (void* p : {l.in.data, l.out.data, (void*)l.gain, (void*)l.mu, (void*)l.r1, (void*)l.r2})
-            if (p) tsb_free(ctx, p);
+    free_layer(ctx, l);
+    const int rotation = l.rotation, source = l.source;
     l = s->layers[src_layer];
+    l.rotation = rotation, l.source = source;
     l.owned = false;
     return TSB_OK;
 }
@@ -136,38 +171,72 @@ void plain_runtime_free(ModelRt& rt) {
     rt.plain = nullptr;
 }
 
+constexpr int EXPAND_MIN_ROWS = 64;                 // rows of a portion from which on its latents are expanded
+constexpr size_t EXPAND_MAX_BYTES = 2ull << 30;
+
 int32_t plain_runtime_init(tsb_session* s, ModelRt& rt, const tsb_model* tm, const SessionShape& shape, bool is_draft) {
     (void)is_draft;
     tsb_ctx* ctx = s->ctx;
     const PlainModel* m = tm->plain;
     rt.model = tm;
-    std::vector<int32_t> heads, dims;
-    for (const PlainLayer& l : m->layers) heads.push_back(l.cfg.n_kv_heads), dims.push_back(l.head_pad);
-    int32_t rc = kv_create_keys(ctx, m->cfg.n_layers, heads.data(), dims.data(), m->elem, shape.page_tokens, shape.num_pages, shape.n_streams,
-                                shape.pages_per_seq, &rt.kv);
+    std::vector<KeyLayerShape> shapes;
+    for (const PlainLayer& l : m->layers) {
+        if (l.mixer == MIX_LATENT) shapes.push_back({1, l.key_dim, false, l.source});
+        else shapes.push_back({l.cfg.n_kv_heads, l.head_pad, l.mixer == MIX_KV, (int)shapes.size()});
+    }
+    int32_t rc = kv_create_keys(ctx, m->cfg.n_layers, shapes.data(), m->elem, shape.page_tokens, shape.num_pages, shape.n_streams, shape.pages_per_seq, &rt.kv);
     if (rc) return rc;
     PlainRt* p = rt.plain = new (std::nothrow) PlainRt();
     if (!p) return TSB_ERR_OOM;
     // matmul operands are read in whole token tiles
     p->rows = (int)plain_pad(std::max(shape.pass_rows, 32), 32);
     p->in_stride = m->d_pad;
+    int64_t wide = 0, latent = 0;
     for (const PlainLayer& l : m->layers) {
-        p->q_stride = std::max<int64_t>(p->q_stride, l.q_rows);
+        const int64_t H = l.cfg.n_q_heads;
+        p->q_stride = std::max<int64_t>(p->q_stride, plain_pad(H * l.head_pad, 16));
         p->cat_stride = std::max<int64_t>(p->cat_stride, l.out.cols);
         p->gate_stride = std::max(p->gate_stride, l.cfg.n_q_heads);
+        if (l.post_norm) p->act_stride = std::max<int64_t>(p->act_stride, l.ffn_pad);
+        if (l.cfg.qk_norm) p->raw_stride = std::max<int64_t>(p->raw_stride, (H + l.cfg.n_kv_heads) * l.cfg.head_dim);
+        if (l.cfg.value_gate) p->value_gate_stride = std::max<int64_t>(p->value_gate_stride, plain_pad(H * l.value_pad, 16));
+        if (l.mixer != MIX_LATENT) continue;
+        p->raw_stride = std::max<int64_t>(p->raw_stride, l.cfg.kv_rank);
+        p->absorbed_stride = std::max<int64_t>(p->absorbed_stride, H * l.key_dim);
+        p->sums_stride = std::max<int64_t>(p->sums_stride, H * l.rank_pad);
+        if (l.expands) wide = std::max<int64_t>(wide, H * (l.head_pad + l.value_pad)), latent = std::max<int64_t>(latent, l.key_dim);
     }
     p->fin_rows = (int)plain_pad(std::max(std::max(shape.n_streams * shape.max_rows, std::min(shape.pass_rows, 256)), 32), 32);
     auto A = [&](size_t bytes, void** q) {
+        if (bytes == 0) return (int32_t)TSB_OK;
         int32_t r = dev_alloc(ctx, s->owned, bytes, q);
         if (r == TSB_OK && cudaMemset(*q, 0, bytes) != cudaSuccess) r = tsb_fail(ctx, TSB_ERR_CUDA, "clearing a work buffer failed");
         return r;
     };
     const size_t R = p->rows, e = m->elem;
-    if ((rc = A(R * m->cfg.d_model * 4, (void**)&p->x)) || (rc = A(R * p->in_stride * e, &p->mix)) || (rc = A(R * p->in_stride * e, &p->h)) ||
-        (rc = A(R * p->q_stride * e, &p->q)) || (rc = A(R * p->cat_stride * e, &p->cat)) || (rc = A(R * p->gate_stride * 4, (void**)&p->gate)) ||
-        (rc = A((size_t)p->fin_rows * p->in_stride * e, &p->fin)) || (rc = A(plain_gemm_workspace_bytes(ctx), &p->gemm_ws)) ||
-        (rc = A(wattn_scratch_bytes(ctx), &p->attn_ws)))
+    if ((rc = A(R * m->cfg.d_model * 4, (void**)&p->x)) || (rc = A(R * p->in_stride * e, &p->mix)) ||
+        (rc = A(m->cfg.post_norm ? 0 : R * p->in_stride * e, &p->h)) || (rc = A(R * p->q_stride * e, &p->q)) || (rc = A(R * p->cat_stride * e, &p->cat)) ||
+        (rc = A(R * p->gate_stride * 4, (void**)&p->gate)) || (rc = A((size_t)p->fin_rows * p->in_stride * e, &p->fin)) ||
+        (rc = A(plain_gemm_workspace_bytes(ctx), &p->gemm_ws)) || (rc = A(wattn_scratch_bytes(ctx), &p->attn_ws)) ||
+        (rc = A(R * p->act_stride * e, &p->act)) || (rc = A(R * p->raw_stride * 4, (void**)&p->raw)) || (rc = A(R * p->absorbed_stride * e, &p->absorbed)) ||
+        (rc = A(R * p->sums_stride * e, &p->sums)) || (rc = A(R * p->value_gate_stride * e, &p->value_gate)))
         return rc;
+    for (const PlainRotation& r : m->rotations) {
+        float2* t = nullptr;
+        if ((rc = A(R * (r.dims / 2) * sizeof(float2), (void**)&t))) return rc;
+        p->rotary.push_back(t);
+    }
+    if (wide > 0 && shape.pass_rows >= EXPAND_MIN_ROWS) {
+        ExpandRt& x = p->expand;
+        const int64_t tokens = (int64_t)shape.num_pages * shape.page_tokens;
+        const int64_t room = (int64_t)(EXPAND_MAX_BYTES / ((size_t)(wide + latent) * e));
+        x.pages = (int)std::min<int64_t>(tokens / EXPAND_PAGE + shape.n_streams, room / EXPAND_PAGE);
+        x.max_seqs = shape.n_streams;
+        x.pages_per_seq = (int)(((int64_t)shape.pages_per_seq * shape.page_tokens + EXPAND_PAGE - 1) / EXPAND_PAGE);
+        if ((rc = A((size_t)x.pages * EXPAND_PAGE * wide * e, &x.wide)) || (rc = A((size_t)x.pages * EXPAND_PAGE * latent * e, &x.latents)) ||
+            (rc = A((size_t)x.max_seqs * x.pages_per_seq * sizeof(int32_t), (void**)&x.table)))
+            return rc;
+    }
     if (m->any_shift) {
         ShiftState& st = p->shift;
         st.width = m->cfg.d_model, st.n_streams = shape.n_streams;
@@ -186,10 +255,336 @@ int32_t plain_fill_context(tsb_session* s, ModelRt& rt, int stream, int64_t toke
     return kv_fill_keys(rt.kv, s->stream, stream, tokens, seed);  // the shift state keeps what it holds
 }
 
-// The query tiles of a ragged pass for one group size: few-query tiles hold a whole stream's rows.
+// ------------------------------------------------------------------ packed rows of a layer's input matrix
+struct InRows {
+    int64_t q = 0, k = 0, v = 0, head_gate = 0, value_gate = 0;  // first rows; latent layers: k is the latent
+    int64_t segments = 0;                                        // end of the rows with destinations of their own
+    int64_t pairs = 0, n_pairs = 0;                              // interleaved pairs behind them (gate and up, or rotated coordinates)
+    int64_t rows = 0;
+};
+InRows in_rows(const PlainLayer& l) {
+    const tsb_plain_layer& c = l.cfg;
+    const int64_t H = c.n_q_heads, G = c.n_kv_heads, E = c.value_dim;
+    const bool own = c.kv_source == 0;
+    InRows r;
+    int64_t at = l.mixer == MIX_KEYS ? l.q_rows : H * c.head_dim;
+    r.k = at;
+    at += l.mixer == MIX_KEYS ? l.k_rows : l.mixer == MIX_KV ? G * c.head_dim : own ? c.kv_rank : 0;
+    r.v = at;
+    if (l.mixer == MIX_KV) at += G * E;
+    r.head_gate = at;
+    if (c.head_gate) at += H;
+    r.value_gate = at;
+    if (c.value_gate) at += H * E;
+    r.segments = at;
+    r.pairs = plain_pad(at, PLAIN_ROW_PAD);
+    if (l.mixer == MIX_LATENT) r.n_pairs = (H + (own ? 1 : 0)) * (c.rot_dim / 2);
+    else if (!l.post_norm) r.n_pairs = l.ffn_pad;
+    r.rows = r.pairs + plain_pad(2 * plain_pad(r.n_pairs, 8), PLAIN_ROW_PAD);
+    return r;
+}
+
+// ------------------------------------------------------------------ forward pass
+// The query tiles of a ragged pass for one geometry, and which streams of the pass they are made of.
+enum TileSet { TILES_ALL = 0, TILES_LATENT, TILES_LATENT_SHORT, TILES_WIDE };
 struct TileLists {
-    int group = 0, rows_per_tile = 0;
+    int set, group, rows_per_tile;
     AttnBatch batch;
+};
+// What a pass knows about its portions before the first launch.
+struct PassPlan {
+    std::vector<TileLists> lists;
+    int max_len = 0, longest = 0, longest_short = 0;
+    // portions whose latents are expanded, and the rows that hold all the others
+    std::vector<ExpandStream> expanded;
+    std::vector<bool> is_expanded;
+    const ExpandStream* expanded_dev = nullptr;
+    int expanded_pages = 0, expanded_len = 0, short_first = 0, short_rows = 0;
+
+    const AttnBatch* find(int set, int group, int rows_per_tile) const {
+        for (const TileLists& t : lists)
+            if (t.set == set && t.group == group && t.rows_per_tile == rows_per_tile) return &t.batch;
+        return nullptr;
+    }
+};
+
+int latent_most_rows(const PassPlan& plan, const Pass& p, const PlainLayer& l) {
+    return p.rows_per_seq > 0 ? p.rows_per_seq : l.expands ? plan.longest_short : plan.longest;
+}
+
+int32_t plan_pass(tsb_session* s, const PlainModel* m, const PlainRt* b, const Pass& p, PassPlan& plan) {
+    plan.max_len = (p.max_len + 511) / 512 * 512;  // the split plan changes only every 512 positions (graph reuse)
+    plan.longest = p.rows_per_seq;
+    plan.short_rows = p.rows;
+    if (p.rows_per_seq > 0) return TSB_OK;
+    plan.is_expanded.assign(p.n_groups, false);
+    int first_short = p.rows, end_short = 0;
+    for (int i = 0; i < p.n_groups; i++) {
+        const RowGroup& g = p.groups[i];
+        plan.longest = std::max(plan.longest, g.n_rows);
+        const int len = (int)g.base + g.n_rows, pages = (len + EXPAND_PAGE - 1) / EXPAND_PAGE;
+        if (g.n_rows >= EXPAND_MIN_ROWS && plan.expanded_pages + pages <= b->expand.pages) {
+            plan.is_expanded[i] = true;
+            plan.expanded.push_back({g.first_row, g.n_rows, plan.expanded_pages});
+            plan.expanded_pages += pages, plan.expanded_len = std::max(plan.expanded_len, len);
+        } else {
+            first_short = std::min(first_short, g.first_row), end_short = std::max(end_short, g.first_row + g.n_rows);
+            plan.longest_short = std::max(plan.longest_short, g.n_rows);
+        }
+    }
+    plan.short_first = first_short, plan.short_rows = std::max(0, end_short - first_short);
+    if (!plan.expanded.empty()) {
+        const int32_t* dev = nullptr;
+        if (int32_t rc = session_stage_ints(s, reinterpret_cast<const int32_t*>(plan.expanded.data()), (int)plan.expanded.size() * 3, &dev)) return rc;
+        plan.expanded_dev = reinterpret_cast<const ExpandStream*>(dev);
+    }
+    if (m->f32) return TSB_OK;  // the f32 kernel takes rows one by one
+    auto add = [&](int set, int group, int rpt, int small_queries) -> int32_t {
+        if (plan.find(set, group, rpt)) return TSB_OK;
+        std::vector<AttnTile> small, large;
+        TileLists t;
+        t.set = set, t.group = group, t.rows_per_tile = rpt;
+        for (int i = 0; i < p.n_groups; i++) {
+            const RowGroup& g = p.groups[i];
+            if ((set == TILES_LATENT_SHORT && plan.is_expanded[i]) || (set == TILES_WIDE && !plan.is_expanded[i])) continue;
+            if (g.n_rows * group <= small_queries) {
+                small.push_back({g.first_row, g.n_rows});
+                t.batch.small_queries = std::max(t.batch.small_queries, g.n_rows * group);
+            } else {
+                for (int r = 0; r < g.n_rows; r += rpt) large.push_back({g.first_row + r, std::min(rpt, g.n_rows - r)});
+            }
+        }
+        if (set == TILES_LATENT || set == TILES_LATENT_SHORT) small.swap(large);
+        t.batch.n_small = (int)small.size(), t.batch.n_large = (int)large.size();
+        small.insert(small.end(), large.begin(), large.end());
+        const int32_t* dev = nullptr;
+        if (int32_t rc = session_stage_ints(s, reinterpret_cast<const int32_t*>(small.data()), (int)small.size() * 2, &dev)) return rc;
+        t.batch.small = reinterpret_cast<const AttnTile*>(dev), t.batch.large = t.batch.small + t.batch.n_small;
+        t.batch.rows = p.rows, t.batch.max_len = plan.max_len;
+        plan.lists.push_back(t);
+        return TSB_OK;
+    };
+    for (const PlainLayer& l : m->layers) {
+        int32_t rc = TSB_OK;
+        if (l.mixer != MIX_LATENT) {
+            const int grp = l.cfg.n_q_heads / l.cfg.n_kv_heads;
+            rc = add(TILES_ALL, grp, wattn_rows_per_tile(l.head_pad, grp, l.cfg.log_bias != 0), WATTN_SMALL_Q);
+        } else {
+            const int most = latent_most_rows(plan, p, l);
+            if (most > 0) rc = add(l.expands ? TILES_LATENT_SHORT : TILES_LATENT, l.cfg.n_q_heads, latent_attn_tiling(l.cfg.n_q_heads, l.rank_pad, most).rows, 0);
+            if (rc == TSB_OK && l.expands && !plan.expanded.empty()) rc = add(TILES_WIDE, 1, WATTN_WIDE_ROWS, 0);
+        }
+        if (rc) return rc;
+    }
+    return TSB_OK;
+}
+
+struct Forward {
+    tsb_session* s;
+    ModelRt& rt;
+    const Pass& p;
+    tsb_ctx* ctx;
+    cudaStream_t st;
+    const PlainModel* m;
+    PlainRt* b;
+    const PassPlan& plan;
+
+    void* at(void* base, int64_t elements) const { return static_cast<uint8_t*>(base) + (size_t)elements * m->elem; }
+    cudaError_t matmul(const PlainMat& w, const void* x, const void* x2, int64_t stride, const PlainEpi& epi) const {
+        return launch_plain_gemm(ctx, st, m->f32, w, x, x2, stride, b->rows, p.rows, epi, b->gemm_ws);
+    }
+
+    // projections of a layer: x to the mixer's rows, x2 to the (gate, up) pairs of a parallel layer
+    cudaError_t project(int L, const void* x, const void* x2) const {
+        const PlainLayer& l = m->layers[L];
+        const tsb_plain_layer& c = l.cfg;
+        const InRows r = in_rows(l);
+        PlainEpi e;
+        e.kind = PLAIN_MIXER, e.keys = rt.kv->key_layers[L], e.rows = p.rows_dev;
+        auto seg = [&](int64_t end, int kind, void* to, int64_t stride, int64_t per = 0x7fffffff, int64_t step = 0) {
+            PlainSeg& g = e.seg[e.n_seg++];
+            g.end = (int)end, g.kind = kind, g.p = to, g.stride = stride, g.per = (int)per, g.step = (int)step;
+        };
+        if (l.mixer == MIX_KEYS) {
+            seg(r.k, PLAIN_SEG_TYPED, b->q, b->q_stride);
+            seg(r.v, PLAIN_SEG_CACHE, nullptr, 0);
+        } else if (l.mixer == MIX_KV) {
+            if (c.qk_norm) {
+                seg(r.v, PLAIN_SEG_F32, b->raw, b->raw_stride);
+            } else {
+                seg(r.k, PLAIN_SEG_TYPED, b->q, b->q_stride, c.head_dim, l.head_pad);
+                seg(r.v, PLAIN_SEG_CACHE, nullptr, 0, c.head_dim, e.keys.head_step);
+            }
+            seg(r.head_gate, PLAIN_SEG_CACHE, nullptr, e.keys.value_off, c.value_dim, e.keys.head_step);
+        } else {
+            seg(r.k, PLAIN_SEG_TYPED, b->q, b->q_stride, c.head_dim, l.head_pad);
+            if (r.v > r.k) seg(r.v, PLAIN_SEG_F32, b->raw, b->raw_stride);
+            if (c.rot_dim > 0) {
+                PlainRotate& t = e.rot;
+                t.half = c.rot_dim / 2, t.n_heads = c.n_q_heads, t.table = b->rotary[l.rotation], t.key_off = c.kv_rank;
+                t.q[0] = b->q, t.q_stride[0] = b->q_stride, t.q_step[0] = l.head_pad, t.q_off[0] = c.head_dim;
+                t.q[1] = b->absorbed, t.q_stride[1] = b->absorbed_stride, t.q_step[1] = l.key_dim, t.q_off[1] = c.kv_rank;
+            }
+        }
+        if (c.head_gate) seg(r.value_gate, PLAIN_SEG_F32, b->gate, c.n_q_heads);
+        if (c.value_gate) seg(r.segments, PLAIN_SEG_TYPED, b->value_gate, b->value_gate_stride, c.value_dim, l.value_pad);
+        if (r.n_pairs > 0) {
+            e.pair_row0 = (int)r.pairs, e.n_pairs = (int)r.n_pairs, e.act = c.act;
+            e.a = at(b->cat, l.o_cols), e.a_stride = l.out.cols;  // a rotation does not use them
+        }
+        return matmul(l.in, x, x2, b->in_stride, e);
+    }
+
+    cudaError_t head_norms(int L) const {
+        const PlainLayer& l = m->layers[L];
+        const tsb_plain_layer& c = l.cfg;
+        HeadNorms h;
+        h.raw = b->raw, h.raw_stride = b->raw_stride, h.eps = m->cfg.norm_eps, h.keys = rt.kv->key_layers[L], h.rows = p.rows_dev;
+        if (l.mixer == MIX_LATENT) {
+            h.n_k = 1, h.width = c.kv_rank, h.k_weight = l.c_norm;
+        } else {
+            h.n_q = c.n_q_heads, h.n_k = c.n_kv_heads, h.width = c.head_dim, h.q_weight = l.q_norm, h.k_weight = l.k_norm;
+            h.temp_coef = c.q_temp_coef, h.temp_every = c.q_temp_every;
+            h.q = b->q, h.q_stride = b->q_stride, h.q_step = h.q_width = l.head_pad;
+        }
+        return launch_head_norms(ctx, st, m->f32, h, p.rows);
+    }
+
+    WindowAttn attention_of(const PlainLayer& l) const {
+        const tsb_plain_layer& c = l.cfg;
+        WindowAttn a;
+        a.q = b->q, a.q_stride = b->q_stride, a.out = b->cat, a.out_stride = l.out.cols, a.rows = p.rows_dev;
+        a.n_q_heads = c.n_q_heads, a.scale = c.score_scale, a.cap = c.score_cap, a.window = c.window;
+        a.gate = c.head_gate ? b->gate : nullptr;
+        if (c.value_gate) a.value_gate = b->value_gate, a.value_gate_stride = b->value_gate_stride;
+        if (c.log_bias) a.r1 = l.r1, a.r2 = l.r2;
+        if (c.sink) a.sink = l.sink;
+        return a;
+    }
+
+    cudaError_t attend(int L) const {
+        const PlainLayer& l = m->layers[L];
+        const int grp = l.cfg.n_q_heads / l.cfg.n_kv_heads;
+        WindowAttn a = attention_of(l);
+        a.keys = rt.kv->key_layers[L];
+        AttnBatch batch;
+        if (const AttnBatch* t = plan.find(TILES_ALL, grp, wattn_rows_per_tile(l.head_pad, grp, l.cfg.log_bias != 0))) batch = *t;
+        batch.rows = p.rows, batch.rows_per_seq = p.rows_per_seq, batch.max_len = plan.max_len;
+        return launch_window_attn(ctx, st, m->f32, a, batch, b->attn_ws);
+    }
+
+    // Short portions: queries go to the latents' space, the heads' sums of latents come back from it.
+    cudaError_t attend_absorbed(int L, int first, int rows) const {
+        const PlainLayer& l = m->layers[L];
+        const tsb_plain_layer& c = l.cfg;
+        auto product = [&](const PlainMat& w, void* x, int64_t x_stride, void* y, int64_t y_stride, int valid, int step, bool gated) {
+            PlainEpi e;
+            e.kind = PLAIN_MIXER, e.n_seg = 1;
+            PlainSeg& g = e.seg[0];
+            g.end = (int)w.rows, g.per = w.group_rows, g.valid = valid, g.step = step, g.p = at(y, first * y_stride), g.stride = y_stride;
+            if (gated) g.gate = at(b->value_gate, first * b->value_gate_stride), g.gate_stride = b->value_gate_stride, g.gate_step = l.value_pad;
+            return launch_plain_gemm(ctx, st, m->f32, w, at(x, first * x_stride), nullptr, x_stride, b->rows - first, rows, e, b->gemm_ws);
+        };
+        cudaError_t e = product(l.absorb, b->q, b->q_stride, b->absorbed, b->absorbed_stride, c.kv_rank, l.key_dim, false);
+        if (e != cudaSuccess) return e;
+        if (m->f32) {
+            WindowAttn a = attention_of(l);
+            a.keys = rt.kv->key_layers[L], a.q = b->absorbed, a.q_stride = b->absorbed_stride, a.out = b->sums, a.out_stride = b->sums_stride;
+            a.value_dim = l.rank_pad, a.value_gate = nullptr;
+            AttnBatch batch;
+            batch.rows = p.rows, batch.max_len = plan.max_len;
+            e = launch_window_attn(ctx, st, true, a, batch, b->attn_ws);
+        } else {
+            LatentAttn a;
+            a.keys = rt.kv->key_layers[L], a.q = b->absorbed, a.q_stride = b->absorbed_stride, a.out = b->sums, a.out_stride = b->sums_stride;
+            a.rows = p.rows_dev, a.n_heads = c.n_q_heads, a.value_dim = l.rank_pad, a.scale = c.score_scale, a.sink = c.sink ? l.sink : nullptr;
+            const int most = latent_most_rows(plan, p, l);
+            AttnBatch batch;
+            if (const AttnBatch* t = plan.find(l.expands ? TILES_LATENT_SHORT : TILES_LATENT, c.n_q_heads, latent_attn_tiling(c.n_q_heads, l.rank_pad, most).rows))
+                batch = *t;
+            batch.rows = p.rows, batch.rows_per_seq = p.rows_per_seq, batch.max_len = plan.max_len;
+            e = launch_latent_attn(ctx, st, a, batch, most, b->attn_ws);
+        }
+        if (e != cudaSuccess) return e;
+        return product(l.lift, b->sums, b->sums_stride, b->cat, l.out.cols, c.value_dim, l.value_pad, c.value_gate != 0);
+    }
+
+    // Long portions: keys and values of every visible position, then attention with a key head per query head.
+    cudaError_t attend_expanded(int L) const {
+        const PlainLayer& l = m->layers[L];
+        const tsb_plain_layer& c = l.cfg;
+        const int H = c.n_q_heads;
+        LatentGather g;
+        g.cache = rt.kv->key_layers[L];
+        KeyView& w = g.wide;
+        w.base = static_cast<uint8_t*>(b->expand.wide), w.page_table = b->expand.table;
+        w.kv_heads = H, w.head_dim = l.head_pad, w.elem_bytes = m->elem;
+        w.value_off = l.head_pad, w.head_step = l.head_pad + l.value_pad, w.row = H * w.head_step;
+        w.page_tokens = EXPAND_PAGE, w.num_pages = b->expand.pages, w.max_seqs = b->expand.max_seqs, w.max_pages_per_seq = b->expand.pages_per_seq;
+        for (w.page_shift = 0; 1 << w.page_shift < EXPAND_PAGE;) w.page_shift++;
+        g.wide_table = b->expand.table, g.latents = b->expand.latents;
+        g.kv_rank = c.kv_rank, g.rot_dim = c.rot_dim, g.key_off = c.head_dim, g.rows = p.rows_dev, g.streams = plan.expanded_dev;
+        cudaError_t e = launch_latent_gather(ctx, st, g, (int)plan.expanded.size(), plan.expanded_len);
+        if (e != cudaSuccess) return e;
+        PlainEpi x;
+        x.kind = PLAIN_MIXER, x.n_seg = 2;
+        x.seg[0].end = H * c.head_dim, x.seg[0].per = c.head_dim, x.seg[1].end = H * (c.head_dim + c.value_dim), x.seg[1].per = c.value_dim;
+        for (PlainSeg& k : x.seg) k.p = w.base, k.stride = w.row, k.step = w.head_step;
+        x.seg[1].p = at(w.base, w.value_off);
+        e = launch_plain_gemm(ctx, st, false, l.expand, b->expand.latents, nullptr, l.key_dim, b->expand.pages * EXPAND_PAGE, plan.expanded_pages * EXPAND_PAGE, x,
+                              b->gemm_ws);
+        if (e != cudaSuccess) return e;
+        WindowAttn a = attention_of(l);
+        a.keys = w, a.value_dim = l.value_pad;
+        return launch_window_attn_wide(ctx, st, a, *plan.find(TILES_WIDE, 1, WATTN_WIDE_ROWS), b->attn_ws);
+    }
+
+    // from the projections to the heads' outputs, side by side in b->cat
+    cudaError_t mix(int L) const {
+        const PlainLayer& l = m->layers[L];
+        cudaError_t e = cudaSuccess;
+        if (l.cfg.qk_norm || (l.mixer == MIX_LATENT && l.source == L)) e = head_norms(L);
+        if (e != cudaSuccess) return e;
+        if (l.mixer != MIX_LATENT) return attend(L);
+        const bool expand = l.expands && !plan.expanded.empty();
+        const int first = expand ? plan.short_first : 0, rows = expand ? plan.short_rows : p.rows;
+        if (rows > 0) e = attend_absorbed(L, first, rows);  // rows of long portions in between are overwritten below
+        return e == cudaSuccess && expand ? attend_expanded(L) : e;
+    }
+
+    cudaError_t add_to_stream(const PlainMat& w, const void* x, int64_t stride) const {
+        PlainEpi e;
+        e.kind = PLAIN_ADD, e.y = b->x, e.y_stride = m->cfg.d_model, e.n_valid = m->cfg.d_model;
+        if (m->cfg.post_norm) e.alpha = m->cfg.residual_scale;
+        return matmul(w, x, nullptr, stride, e);
+    }
+
+    // [W_o | W_down] over [heads | feed-forward]: both sublayers read the normed input, and add up in one product
+    cudaError_t parallel_layer(int L, bool use_before) const {
+        const PlainLayer& l = m->layers[L];
+        const tsb_plain_layer& c = l.cfg;
+        cudaError_t e = launch_norm_shift(ctx, st, m->f32, b->x, m->cfg.d_model, l.gain, m->cfg.norm_eps, c.token_shift ? l.mu : nullptr, p.rows_dev, p.rows,
+                                          b->shift, L, use_before, b->mix, c.ffn > 0 ? b->h : nullptr, b->in_stride);
+        if (e == cudaSuccess) e = project(L, b->mix, b->h);
+        if (e == cudaSuccess) e = mix(L);
+        return e == cudaSuccess ? add_to_stream(l.out, b->cat, l.out.cols) : e;
+    }
+
+    // the stream itself is the sublayers' input (b->mix holds it in the compute type), and is normed after each sum
+    cudaError_t post_norm_layer(int L) const {
+        const PlainLayer& l = m->layers[L];
+        cudaError_t e = project(L, b->mix, b->mix);
+        if (e == cudaSuccess) e = mix(L);
+        if (e == cudaSuccess) e = add_to_stream(l.out, b->cat, l.out.cols);
+        auto norm = [&](const float* w) { return launch_post_norm(ctx, st, m->f32, b->x, m->cfg.d_model, w, m->cfg.norm_eps, p.rows, b->mix, b->in_stride); };
+        if (e == cudaSuccess) e = norm(l.gain);
+        if (e != cudaSuccess || l.cfg.ffn == 0) return e;
+        PlainEpi g;
+        g.kind = PLAIN_MIXER, g.pair_row0 = 0, g.n_pairs = l.ffn_pad, g.act = l.cfg.act, g.a = b->act, g.a_stride = l.ffn_pad;
+        e = matmul(l.ff_in, b->mix, b->mix, b->in_stride, g);
+        if (e == cudaSuccess) e = add_to_stream(l.ff_out, b->act, l.ffn_pad);
+        return e == cudaSuccess ? norm(l.norm2) : e;
+    }
 };
 
 cudaError_t plain_forward(tsb_session* s, ModelRt& rt, const Pass& p) {
@@ -198,82 +593,31 @@ cudaError_t plain_forward(tsb_session* s, ModelRt& rt, const Pass& p) {
     const PlainModel* m = rt.model->plain;
     PlainRt* b = rt.plain;
     const int d = m->cfg.d_model;
+    const bool post = m->cfg.post_norm != 0;
+    PassPlan plan;
+    if (plan_pass(s, m, b, p, plan) != TSB_OK) return cudaErrorMemoryAllocation;
+    const Forward f{s, rt, p, ctx, st, m, b, plan};
     cudaError_t e;
 #define FW(x)                           \
     do {                                \
         e = (x);                        \
         if (e != cudaSuccess) return e; \
     } while (0)
-    const int max_len = (p.max_len + 511) / 512 * 512;  // the split plan changes only every 512 positions (graph reuse)
-    std::vector<TileLists> lists;
-    int longest = p.rows_per_seq;
-    if (p.rows_per_seq == 0) {
-        for (int i = 0; i < p.n_groups; i++) longest = std::max(longest, p.groups[i].n_rows);
-        for (const PlainLayer& l : m->layers) {
-            const int grp = l.cfg.n_q_heads / l.cfg.n_kv_heads;
-            const int rpt = wattn_rows_per_tile(l.head_pad, grp);
-            bool have = m->f32;  // the f32 kernel takes rows one by one
-            for (const TileLists& t : lists) have |= t.group == grp && t.rows_per_tile == rpt;
-            if (have) continue;
-            std::vector<AttnTile> small, large;
-            TileLists t;
-            t.group = grp, t.rows_per_tile = rpt;
-            for (int i = 0; i < p.n_groups; i++) {
-                const RowGroup& g = p.groups[i];
-                if (g.n_rows * grp <= WATTN_SMALL_Q) {
-                    small.push_back({g.first_row, g.n_rows});
-                    t.batch.small_queries = std::max(t.batch.small_queries, g.n_rows * grp);
-                } else {
-                    for (int r = 0; r < g.n_rows; r += rpt) large.push_back({g.first_row + r, std::min(rpt, g.n_rows - r)});
-                }
-            }
-            t.batch.n_small = (int)small.size(), t.batch.n_large = (int)large.size();
-            small.insert(small.end(), large.begin(), large.end());
-            const int32_t* dev = nullptr;
-            if (session_stage_ints(s, reinterpret_cast<const int32_t*>(small.data()), (int)small.size() * 2, &dev) != TSB_OK) return cudaErrorMemoryAllocation;
-            t.batch.small = reinterpret_cast<const AttnTile*>(dev), t.batch.large = t.batch.small + t.batch.n_small;
-            lists.push_back(t);
-        }
-    }
-    const bool use_before = m->any_shift && longest >= b->shift.ring_rows;
-    FW(launch_plain_embed(ctx, st, m->f32, m->embed, m->cfg.vocab, d, p.tokens, p.token_stride, p.rows, b->x));
+    const bool use_before = m->any_shift && plan.longest >= b->shift.ring_rows;
+    FW(launch_plain_embed(ctx, st, m->f32, m->embed, m->cfg.vocab, d, p.tokens, p.token_stride, p.rows, m->cfg.embed_scale, b->x, post ? b->mix : nullptr,
+                          b->in_stride));
     if (use_before) FW(launch_shift_before(ctx, st, b->shift, m->cfg.n_layers, p.rows_dev, p.rows));
-    for (int L = 0; L < m->cfg.n_layers; L++) {
-        const PlainLayer& l = m->layers[L];
-        const tsb_plain_layer& c = l.cfg;
-        FW(launch_norm_shift(ctx, st, m->f32, b->x, d, l.gain, m->cfg.norm_eps, c.token_shift ? l.mu : nullptr, p.rows_dev, p.rows, b->shift, L, use_before,
-                             b->mix, c.ffn > 0 ? b->h : nullptr, b->in_stride));
-        const int64_t cat_stride = l.out.cols;
-        PlainEpi in;
-        in.kind = PLAIN_MIXER;
-        in.q = b->q, in.q_stride = l.q_rows, in.q_rows = l.q_rows, in.k_rows = l.k_rows;
-        in.keys = rt.kv->key_layers[L], in.rows = p.rows_dev;
-        in.gate = b->gate, in.gate_rows = c.head_gate ? c.n_q_heads : 0;
-        if (c.ffn > 0) {
-            in.pair_row0 = (int)(l.in.rows - 2 * l.ffn_pad), in.n_pairs = l.ffn_pad, in.act = c.act;
-            in.a = static_cast<uint8_t*>(b->cat) + (size_t)l.o_cols * m->elem, in.a_stride = cat_stride;
-        }
-        FW(launch_plain_gemm(ctx, st, m->f32, l.in, b->mix, b->h, b->in_stride, b->rows, p.rows, in, b->gemm_ws));
-        WindowAttn a;
-        a.keys = rt.kv->key_layers[L], a.q = b->q, a.q_stride = l.q_rows;
-        a.gate = c.head_gate ? b->gate : nullptr, a.out = b->cat, a.out_stride = cat_stride, a.rows = p.rows_dev;
-        a.n_q_heads = c.n_q_heads, a.scale = c.score_scale, a.cap = c.score_cap, a.window = c.window;
-        if (c.log_bias) a.r1 = l.r1, a.r2 = l.r2;
-        AttnBatch batch;
-        for (const TileLists& t : lists)
-            if (t.group == c.n_q_heads / c.n_kv_heads && t.rows_per_tile == wattn_rows_per_tile(l.head_pad, t.group)) batch = t.batch;
-        batch.rows = p.rows, batch.rows_per_seq = p.rows_per_seq, batch.max_len = max_len;
-        FW(launch_window_attn(ctx, st, m->f32, a, batch, b->attn_ws));
-        PlainEpi out;
-        out.kind = PLAIN_ADD, out.y = b->x, out.y_stride = d, out.n_valid = d;
-        FW(launch_plain_gemm(ctx, st, m->f32, l.out, b->cat, nullptr, cat_stride, b->rows, p.rows, out, b->gemm_ws));
+    for (size_t i = 0; i < m->rotations.size(); i++) {
+        const PlainRotation& r = m->rotations[i];
+        FW(launch_rotary_table(ctx, st, r.freq, r.dims / 2, r.magnitude, p.rows_dev, p.rows, b->rotary[i]));
     }
+    for (int L = 0; L < m->cfg.n_layers; L++) FW(post ? f.post_norm_layer(L) : f.parallel_layer(L, use_before));
     if (p.logits) {
         const bool last = p.last_rows_only && p.rows_per_seq > 1;
         const int n = p.rows_per_seq == 0 ? p.n_want : last ? p.rows / p.rows_per_seq : p.rows;
         if (n > 0) {
-            FW(launch_norm_rows(ctx, st, m->f32, b->x, d, m->final_gain, m->cfg.norm_eps, p.rows_per_seq == 0 ? p.want_dev : nullptr,
-                                last ? p.rows_per_seq - 1 : 0, last ? p.rows_per_seq : 1, n, b->fin, b->in_stride));
+            FW(launch_norm_rows(ctx, st, m->f32, b->x, d, m->final_gain, post ? m->final_gain : nullptr, m->cfg.norm_eps,
+                                p.rows_per_seq == 0 ? p.want_dev : nullptr, last ? p.rows_per_seq - 1 : 0, last ? p.rows_per_seq : 1, n, b->fin, b->in_stride));
             PlainEpi hd;
             hd.kind = PLAIN_STORE, hd.y = static_cast<float*>(p.logits.p), hd.y_stride = p.logits_stride, hd.n_valid = m->cfg.vocab, hd.cap = m->cfg.logit_cap;
             FW(launch_plain_gemm(ctx, st, m->f32, m->head, b->fin, nullptr, b->in_stride, b->fin_rows, n, hd, b->gemm_ws));
@@ -281,6 +625,36 @@ cudaError_t plain_forward(tsb_session* s, ModelRt& rt, const Pass& p) {
     }
 #undef FW
     return cudaSuccess;
+}
+
+// ------------------------------------------------------------------ rotations
+int rotation_of(PlainModel* m, const tsb_plain_layer& c) {
+    PlainRotation r;
+    r.dims = c.rot_dim, r.base = c.rot_base, r.factor = c.rot_factor, r.original = c.rot_original, r.fast = c.rot_fast, r.slow = c.rot_slow;
+    for (size_t i = 0; i < m->rotations.size(); i++) {
+        const PlainRotation& o = m->rotations[i];
+        if (o.dims == r.dims && o.base == r.base && o.factor == r.factor && o.original == r.original && o.fast == r.fast && o.slow == r.slow) return (int)i;
+    }
+    m->rotations.push_back(r);
+    return (int)m->rotations.size() - 1;
+}
+
+int32_t upload_rotation(tsb_ctx* ctx, PlainRotation& r) {
+    std::vector<float> freq(r.dims / 2);
+    const bool scaled = r.factor > 0;
+    // the pair that turns t times within the original context
+    auto pair_with_turns = [&](double t) { return r.dims * log(r.original / (2 * M_PI * t)) / (2 * log(r.base)); };
+    const double lo = scaled ? std::max(floor(pair_with_turns(r.fast)), 0.0) : 0;
+    const double hi = scaled ? std::min(ceil(pair_with_turns(r.slow)), (double)r.dims - 1) : 0;
+    for (int i = 0; i < r.dims / 2; i++) {
+        const double f = pow(r.base, -2.0 * i / r.dims);
+        const double ramp = scaled ? std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0) : 0;
+        freq[i] = (float)(scaled ? f / r.factor * ramp + f * (1 - ramp) : f);
+    }
+    r.magnitude = scaled ? (float)(0.1 * log(r.factor) + 1.0) : 1.f;
+    if (int32_t rc = tsb_alloc(ctx, freq.size() * 4, (void**)&r.freq)) return rc;
+    TSB_CUDA(ctx, cudaMemcpy(r.freq, freq.data(), freq.size() * 4, cudaMemcpyHostToDevice));
+    return TSB_OK;
 }
 
 const ModelFamily PLAIN_FAMILY = {
@@ -301,13 +675,34 @@ int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const 
     const bool f32 = cfg->compute == TSB_F32;
     for (int i = 0; i < cfg->n_layers; i++) {
         const tsb_plain_layer& l = layers[i];
-        TSB_REQUIRE(ctx, l.n_q_heads > 0 && l.n_kv_heads > 0 && l.head_dim > 0 && l.n_q_heads % l.n_kv_heads == 0,
+        const bool latent = l.kv_rank > 0;
+        TSB_REQUIRE(ctx, l.n_q_heads > 0 && l.head_dim > 0 && (latent || (l.n_kv_heads > 0 && l.n_q_heads % l.n_kv_heads == 0)),
                     "layer %d: query heads must be a positive multiple of the key heads", i);
-        TSB_REQUIRE(ctx, l.window >= 0 && l.ffn >= 0, "layer %d: window and ffn must not be negative", i);
+        TSB_REQUIRE(ctx, l.window >= 0 && l.ffn >= 0 && l.value_dim >= 0 && l.kv_rank >= 0 && l.rot_dim >= 0, "layer %d: sizes must not be negative", i);
         TSB_REQUIRE(ctx, l.act == TSB_ACT_GELU_TANH || l.act == TSB_ACT_SILU, "layer %d: unknown activation", i);
-        if (!wattn_supported(l.head_dim, l.n_q_heads / l.n_kv_heads, f32))
-            return tsb_fail(ctx, TSB_ERR_UNSUPPORTED, "layer %d: head size %d with %d query heads per key head is outside the attention kernels", i, l.head_dim,
-                            l.n_q_heads / l.n_kv_heads);
+        TSB_REQUIRE(ctx, l.q_temp_every >= 0 && (l.q_temp_every == 0 || l.qk_norm), "layer %d: a query temperature goes with normed queries", i);
+        TSB_REQUIRE(ctx, !l.qk_norm || (l.value_dim > 0 && !latent), "layer %d: normed queries and keys go with values of their own", i);
+        TSB_REQUIRE(ctx, !cfg->post_norm || !l.token_shift, "layer %d: a token shift goes with the parallel form", i);
+        if (latent) {
+            TSB_REQUIRE(ctx, cfg->post_norm && l.value_dim > 0 && l.rot_dim % 2 == 0 && (l.rot_dim == 0 || l.rot_base > 0),
+                        "layer %d: a latent layer has values, an even rotated part and the post-norm form", i);
+            TSB_REQUIRE(ctx, !l.window && l.score_cap <= 0.f && !l.log_bias && !l.head_gate, "layer %d: a latent layer has no window, cap, bias or head gates", i);
+            TSB_REQUIRE(ctx, l.kv_source >= 0 && l.kv_source <= i, "layer %d reads the latent of a layer before it", i);
+            if (l.kv_source > 0) {
+                const tsb_plain_layer& o = layers[l.kv_source - 1];
+                TSB_REQUIRE(ctx, o.kv_rank == l.kv_rank && o.rot_dim == l.rot_dim && o.kv_source == 0, "layer %d: layer %d has no latent of this shape", i,
+                            l.kv_source - 1);
+            }
+            int dk = 0, dv = 0;
+            if (!latent_attn_dims(l.kv_rank, l.rot_dim, &dk, &dv) || dk > 1024)
+                return tsb_fail(ctx, TSB_ERR_UNSUPPORTED, "layer %d: latents of %d + %d numbers are outside the attention kernels", i, l.kv_rank, l.rot_dim);
+        } else {
+            TSB_REQUIRE(ctx, l.kv_source == 0 && l.rot_dim == 0, "layer %d: only latent layers rotate or read another layer's rows", i);
+            const int head = std::max(l.head_dim, l.value_dim);
+            if (!wattn_supported(head, l.n_q_heads / l.n_kv_heads, f32))
+                return tsb_fail(ctx, TSB_ERR_UNSUPPORTED, "layer %d: head size %d with %d query heads per key head is outside the attention kernels", i, head,
+                                l.n_q_heads / l.n_kv_heads);
+        }
     }
     tsb_model* tm = new (std::nothrow) tsb_model();
     PlainModel* m = new (std::nothrow) PlainModel();
@@ -322,21 +717,47 @@ int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const 
     tm->cfg.n_q_heads = layers[0].n_q_heads, tm->cfg.n_kv_heads = layers[0].n_kv_heads, tm->cfg.head_dim = layers[0].head_dim, tm->cfg.ffn = layers[0].ffn;
     tm->cfg.rms_eps = cfg->norm_eps;
     m->cfg = *cfg, m->f32 = f32, m->elem = f32 ? 4 : 2;
+    if (m->cfg.embed_scale == 0.f) m->cfg.embed_scale = 1.f;
     m->d_pad = plain_pad(cfg->d_model, PLAIN_COL_PAD);
     m->head.rows = plain_pad(cfg->vocab, PLAIN_ROW_PAD), m->head.cols = m->d_pad;
     m->layers.resize(cfg->n_layers);
+    const int64_t out_rows = plain_pad(cfg->d_model, PLAIN_ROW_PAD);
     for (int i = 0; i < cfg->n_layers; i++) {
         PlainLayer& l = m->layers[i];
         l.cfg = layers[i];
-        m->any_shift |= l.cfg.token_shift != 0;
-        l.head_pad = wattn_pad_dim(l.cfg.head_dim, f32);
-        l.q_rows = l.cfg.n_q_heads * l.head_pad, l.k_rows = l.cfg.n_kv_heads * l.head_pad;
-        l.ffn_pad = (int)plain_pad(l.cfg.ffn, 64);
-        l.in.rows = plain_pad(l.q_rows + l.k_rows + (l.cfg.head_gate ? l.cfg.n_q_heads : 0), PLAIN_ROW_PAD) + 2 * l.ffn_pad;
-        l.in.cols = m->d_pad;
-        l.o_cols = (int)plain_pad(l.q_rows, PLAIN_COL_PAD);
-        l.out.rows = plain_pad(cfg->d_model, PLAIN_ROW_PAD), l.out.cols = l.o_cols + l.ffn_pad;
+        const tsb_plain_layer& c = l.cfg;
+        const int H = c.n_q_heads;
+        l.post_norm = cfg->post_norm != 0;
+        l.mixer = c.kv_rank > 0 ? MIX_LATENT : c.value_dim > 0 ? MIX_KV : MIX_KEYS;
+        l.source = c.kv_source > 0 ? c.kv_source - 1 : i;
+        m->any_shift |= c.token_shift != 0;
+        if (l.mixer == MIX_LATENT) {
+            l.head_pad = (int)plain_pad(c.head_dim + c.rot_dim, PLAIN_COL_PAD), l.value_pad = (int)plain_pad(c.value_dim, PLAIN_COL_PAD);
+            latent_attn_dims(c.kv_rank, c.rot_dim, &l.key_dim, &l.rank_pad);
+            l.expands = !f32 && wattn_wide_supported(l.head_pad, l.value_pad);
+            l.rotation = c.rot_dim > 0 ? rotation_of(m, c) : -1;
+            l.absorb.group_rows = (int)plain_pad(c.kv_rank, PLAIN_ROW_PAD), l.absorb.group_cols = l.head_pad;
+            l.absorb.rows = (int64_t)H * l.absorb.group_rows, l.absorb.cols = plain_pad(c.head_dim, PLAIN_COL_PAD);
+            l.lift.group_rows = (int)plain_pad(c.value_dim, PLAIN_ROW_PAD), l.lift.group_cols = l.rank_pad;
+            l.lift.rows = (int64_t)H * l.lift.group_rows, l.lift.cols = plain_pad(c.kv_rank, PLAIN_COL_PAD);
+            l.expand.rows = plain_pad((int64_t)H * (c.head_dim + c.value_dim), PLAIN_ROW_PAD), l.expand.cols = l.lift.cols;
+        } else {
+            l.head_pad = l.value_pad = wattn_pad_dim(std::max(c.head_dim, c.value_dim), f32);
+        }
+        l.q_rows = H * l.head_pad, l.k_rows = c.n_kv_heads * l.head_pad;
+        l.ffn_pad = (int)plain_pad(c.ffn, 64);
+        l.in.rows = in_rows(l).rows, l.in.cols = m->d_pad;
+        l.o_cols = (int)plain_pad((int64_t)H * l.value_pad, PLAIN_COL_PAD);
+        l.out.rows = out_rows, l.out.cols = l.o_cols + (l.post_norm ? 0 : l.ffn_pad);
+        l.ff_in.rows = 2 * (int64_t)l.ffn_pad, l.ff_in.cols = m->d_pad;
+        l.ff_out.rows = out_rows, l.ff_out.cols = l.ffn_pad;
     }
+    DeviceGuard g(ctx);
+    for (PlainRotation& r : m->rotations)
+        if (int32_t rc = upload_rotation(ctx, r)) {
+            tsb_model_destroy(tm);
+            return rc;
+        }
     *out = tm;
     return TSB_OK;
 }
@@ -348,23 +769,34 @@ int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t
     TSB_REQUIRE(ctx, host && (host_type == TSB_BF16 || host_type == TSB_F32), "null data or unknown host type");
     PlainModel* m = tm->plain;
     const int64_t d = m->cfg.d_model, V = m->cfg.vocab;
+    const bool post = m->cfg.post_norm != 0;
     PlainLayer* l = nullptr;
     if (which >= TSB_P_NORM) {
         TSB_REQUIRE(ctx, layer >= 0 && layer < m->cfg.n_layers, "layer %d outside the model", layer);
         l = &m->layers[layer];
     }
     const tsb_plain_layer c = l ? l->cfg : tsb_plain_layer{};
-    const int64_t H = c.n_q_heads, G = c.n_kv_heads, D = c.head_dim, F = c.ffn;
-    int64_t wr = 1, wc = 1;
+    const bool latent = l && l->mixer == MIX_LATENT, own_latent = latent && c.kv_source == 0;
+    const int64_t H = c.n_q_heads, G = c.n_kv_heads, D = c.head_dim, F = c.ffn, E = l && l->mixer != MIX_KEYS ? c.value_dim : D, R = c.kv_rank;
+    int64_t wr = 1, wc = 1;  // expected shape; -1: no such tensor
     switch (which) {
         case TSB_P_EMBED: case TSB_P_HEAD: wr = V, wc = d; break;
-        case TSB_P_FINAL_NORM: case TSB_P_NORM: break;
+        case TSB_P_FINAL_NORM: case TSB_P_NORM: wc = post ? d : 1; break;
+        case TSB_P_NORM2: wc = post && F > 0 ? d : -1; break;
         case TSB_P_SHIFT: wc = c.token_shift ? d : -1; break;
-        case TSB_P_Q: wr = H * D, wc = d; break;
-        case TSB_P_K: wr = G * D, wc = d; break;
+        case TSB_P_Q: wr = H * (D + c.rot_dim), wc = d; break;
+        case TSB_P_K: wr = latent ? -1 : G * D, wc = d; break;
+        case TSB_P_V: wr = l->mixer == MIX_KV ? G * E : -1, wc = d; break;
+        case TSB_P_Q_NORM: case TSB_P_K_NORM: wc = c.qk_norm ? D : -1; break;
+        case TSB_P_SINK: wc = c.sink ? H : -1; break;
         case TSB_P_HEAD_GATE: wr = c.head_gate ? H : -1, wc = d; break;
+        case TSB_P_VALUE_GATE: wr = c.value_gate ? H * E : -1, wc = d; break;
         case TSB_P_R1: case TSB_P_R2: wc = c.log_bias ? H : -1; break;
-        case TSB_P_O: wr = d, wc = H * D; break;
+        case TSB_P_DKV: wr = own_latent ? R + c.rot_dim : -1, wc = d; break;
+        case TSB_P_DKV_NORM: wc = own_latent ? R : -1; break;
+        case TSB_P_UK: wr = latent ? H * D : -1, wc = R; break;
+        case TSB_P_UV: wr = latent ? H * E : -1, wc = R; break;
+        case TSB_P_O: wr = d, wc = H * E; break;
         case TSB_P_FF_GATE: case TSB_P_FF_UP: wr = F > 0 ? F : -1, wc = d; break;
         case TSB_P_FF_DOWN: wr = d, wc = F > 0 ? F : -1; break;
         default: return tsb_fail(ctx, TSB_ERR_INVALID, "no such tensor (%d)", which);
@@ -376,11 +808,24 @@ int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t
     int32_t rc;
     std::vector<uint8_t> v;
     // small f32 vectors
-    float** vec = which == TSB_P_FINAL_NORM ? &m->final_gain : which == TSB_P_NORM ? &l->gain : which == TSB_P_SHIFT ? &l->mu
-                : which == TSB_P_R1 ? &l->r1 : which == TSB_P_R2 ? &l->r2 : nullptr;
+    float** vec = nullptr;
+    switch (which) {
+        case TSB_P_FINAL_NORM: vec = &m->final_gain; break;
+        case TSB_P_NORM: vec = &l->gain; break;
+        case TSB_P_NORM2: vec = &l->norm2; break;
+        case TSB_P_SHIFT: vec = &l->mu; break;
+        case TSB_P_R1: vec = &l->r1; break;
+        case TSB_P_R2: vec = &l->r2; break;
+        case TSB_P_Q_NORM: vec = &l->q_norm; break;
+        case TSB_P_K_NORM: vec = &l->k_norm; break;
+        case TSB_P_DKV_NORM: vec = &l->c_norm; break;
+        case TSB_P_SINK: vec = &l->sink; break;
+    }
     uint32_t& set = l ? l->set : m->set;
     if (vec) {
         convert(host, host_type, wc, true, v);
+        if (post && (which == TSB_P_FINAL_NORM || which == TSB_P_NORM || which == TSB_P_NORM2))  // stored as the distance from one
+            for (int64_t i = 0; i < wc; i++) reinterpret_cast<float*>(v.data())[i] += 1.f;
         if (!*vec && (rc = tsb_alloc(ctx, (size_t)wc * 4, (void**)vec))) return rc;
         TSB_CUDA(ctx, cudaMemcpy(*vec, v.data(), v.size(), cudaMemcpyHostToDevice));
         set |= 1u << which;
@@ -394,34 +839,87 @@ int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t
         set |= 1u << which;
         return TSB_OK;
     }
-    PlainMat& mat = which == TSB_P_HEAD ? m->head : which == TSB_P_O || which == TSB_P_FF_DOWN ? l->out : l->in;
-    if (!mat.data && (rc = zeroed(ctx, (size_t)mat.rows * mat.cols * es, &mat.data))) return rc;
-    uint8_t* base = static_cast<uint8_t*>(mat.data);
-    const size_t pitch = (size_t)mat.cols * es;
-    // block of n_rows x n_cols of the host tensor at (hr, hc) -> the packed matrix at (dr, dc)
-    auto put = [&](int64_t dr, int64_t dc, int64_t hr, int64_t hc, int64_t n_rows, int64_t n_cols) {
-        return cudaMemcpy2D(base + (size_t)dr * pitch + (size_t)dc * es, pitch, v.data() + ((size_t)hr * wc + hc) * es, (size_t)wc * es, (size_t)n_cols * es,
-                            (size_t)n_rows, cudaMemcpyHostToDevice);
+    // block of n_rows x n_cols of the host tensor (hw columns wide) at (hr, hc) -> the packed matrix at (dr, dc)
+    auto put_from = [&](PlainMat& mat, const uint8_t* data, int64_t hw, int64_t dr, int64_t dc, int64_t hr, int64_t hc, int64_t n_rows, int64_t n_cols) -> int32_t {
+        if (!mat.data)
+            if (int32_t r = zeroed(ctx, (size_t)mat.rows * mat.cols * es, &mat.data)) return r;
+        const size_t pitch = (size_t)mat.cols * es;
+        TSB_CUDA(ctx, cudaMemcpy2D(static_cast<uint8_t*>(mat.data) + (size_t)dr * pitch + (size_t)dc * es, pitch, data + ((size_t)hr * hw + hc) * es, (size_t)hw * es,
+                                   (size_t)n_cols * es, (size_t)n_rows, cudaMemcpyHostToDevice));
+        return TSB_OK;
+    };
+    auto put = [&](PlainMat& mat, int64_t dr, int64_t dc, int64_t hr, int64_t hc, int64_t n_rows, int64_t n_cols) {
+        return put_from(mat, v.data(), wc, dr, dc, hr, hc, n_rows, n_cols);
+    };
+#define PUT(...)                                  \
+    do {                                          \
+        if ((rc = put(__VA_ARGS__))) return rc;   \
+    } while (0)
+    // rows hr + i and hr + half + i of the host tensor are the coordinates of pair `first` + i
+    const InRows at = l ? in_rows(*l) : InRows();
+    auto put_pairs = [&](int64_t first, int64_t hr, int64_t half) -> int32_t {
+        for (int64_t i = 0; i < half;) {
+            const int64_t p = first + i, n = std::min<int64_t>(8 - p % 8, half - i), dr = at.pairs + p / 8 * 16 + p % 8;
+            int32_t r = put(l->in, dr, 0, hr + i, 0, n, d);
+            if (r == TSB_OK) r = put(l->in, dr + 8, 0, hr + half + i, 0, n, d);
+            if (r) return r;
+            i += n;
+        }
+        return TSB_OK;
     };
     switch (which) {
-        case TSB_P_HEAD: TSB_CUDA(ctx, put(0, 0, 0, 0, wr, wc)); break;
+        case TSB_P_HEAD: PUT(m->head, 0, 0, 0, 0, wr, wc); break;
         case TSB_P_Q:
-            for (int64_t h = 0; h < H; h++) TSB_CUDA(ctx, put(h * l->head_pad, 0, h * D, 0, D, d));
+            if (l->mixer == MIX_KV) {
+                PUT(l->in, at.q, 0, 0, 0, wr, d);
+            } else {
+                const int64_t step = latent ? D : l->head_pad, from = D + c.rot_dim;
+                for (int64_t h = 0; h < H; h++) {
+                    PUT(l->in, at.q + h * step, 0, h * from, 0, D, d);
+                    if ((rc = put_pairs(h * (c.rot_dim / 2), h * from + D, c.rot_dim / 2))) return rc;
+                }
+            }
             break;
         case TSB_P_K:
-            for (int64_t h = 0; h < G; h++) TSB_CUDA(ctx, put(l->q_rows + h * l->head_pad, 0, h * D, 0, D, d));
+            if (l->mixer == MIX_KV) PUT(l->in, at.k, 0, 0, 0, wr, d);
+            else for (int64_t h = 0; h < G; h++) PUT(l->in, at.k + h * l->head_pad, 0, h * D, 0, D, d);
             break;
-        case TSB_P_HEAD_GATE: TSB_CUDA(ctx, put(l->q_rows + l->k_rows, 0, 0, 0, H, d)); break;
-        case TSB_P_O:
-            for (int64_t h = 0; h < H; h++) TSB_CUDA(ctx, put(0, h * l->head_pad, 0, h * D, d, D));
+        case TSB_P_V: PUT(l->in, at.v, 0, 0, 0, wr, d); break;
+        case TSB_P_DKV:
+            PUT(l->in, at.k, 0, 0, 0, R, d);
+            if ((rc = put_pairs(H * (c.rot_dim / 2), R, c.rot_dim / 2))) return rc;
             break;
-        case TSB_P_FF_GATE: case TSB_P_FF_UP: {
-            const int64_t row0 = mat.rows - 2 * l->ffn_pad + (which == TSB_P_FF_UP ? 8 : 0);
-            for (int64_t i = 0; i < F; i += 8) TSB_CUDA(ctx, put(row0 + 2 * i, 0, i, 0, std::min<int64_t>(8, F - i), d));
+        case TSB_P_HEAD_GATE: PUT(l->in, at.head_gate, 0, 0, 0, H, d); break;
+        case TSB_P_VALUE_GATE: PUT(l->in, at.value_gate, 0, 0, 0, wr, d); break;
+        case TSB_P_UK: {
+            std::vector<uint8_t> t(v.size());  // head by head transposed: [H][R][D]
+            auto transpose = [&](const auto* from, auto* to) {
+                for (int64_t h = 0; h < H; h++)
+                    for (int64_t i = 0; i < D; i++)
+                        for (int64_t k = 0; k < R; k++) to[(h * R + k) * D + i] = from[(h * D + i) * R + k];
+            };
+            if (m->f32) transpose((const uint32_t*)v.data(), (uint32_t*)t.data());
+            else transpose((const uint16_t*)v.data(), (uint16_t*)t.data());
+            for (int64_t h = 0; h < H; h++)
+                if ((rc = put_from(l->absorb, t.data(), D, h * l->absorb.group_rows, 0, h * R, 0, R, D))) return rc;
+            if (l->expands) PUT(l->expand, 0, 0, 0, 0, H * D, R);
             break;
         }
-        case TSB_P_FF_DOWN: TSB_CUDA(ctx, put(0, l->o_cols, 0, 0, d, F)); break;
+        case TSB_P_UV:
+            for (int64_t h = 0; h < H; h++) PUT(l->lift, h * l->lift.group_rows, 0, h * E, 0, E, R);
+            if (l->expands) PUT(l->expand, H * D, 0, 0, 0, H * E, R);
+            break;
+        case TSB_P_O:
+            for (int64_t h = 0; h < H; h++) PUT(l->out, 0, h * l->value_pad, 0, h * E, d, E);
+            break;
+        case TSB_P_FF_GATE: case TSB_P_FF_UP: {
+            const int64_t row0 = (post ? 0 : at.pairs) + (which == TSB_P_FF_UP ? 8 : 0);
+            for (int64_t i = 0; i < F; i += 8) PUT(post ? l->ff_in : l->in, row0 + 2 * i, 0, i, 0, std::min<int64_t>(8, F - i), d);
+            break;
+        }
+        case TSB_P_FF_DOWN: PUT(post ? l->ff_out : l->out, 0, post ? 0 : l->o_cols, 0, 0, d, F); break;
     }
+#undef PUT
     set |= 1u << which;
     return TSB_OK;
 }
@@ -435,25 +933,34 @@ int32_t tsb_model_fill_plain(tsb_model* tm, uint64_t seed) {
     uint32_t sd = (uint32_t)seed * 2654435761u + (uint32_t)(seed >> 32) + 1u;
     int32_t rc = TSB_OK;
     auto fill = [&](void** p, bool f32, int64_t rows, int64_t cols, int64_t valid, float mid, float amp) {
-        if (rc) return;
+        if (rc || rows * cols == 0) return;
         if (!*p && (rc = tsb_alloc(ctx, (size_t)rows * cols * (f32 ? 4 : 2), p))) return;
         if (f32) fill_plain_kernel<float><<<1024, 256>>>((float*)*p, rows, cols, valid, mid, amp, sd);
         else fill_plain_kernel<__nv_bfloat16><<<1024, 256>>>((__nv_bfloat16*)*p, rows, cols, valid, mid, amp, sd);
         sd = sd * 1664525u + 1013904223u;
     };
-    const int64_t d = m->cfg.d_model;
-    const float a_in = sqrtf(3.f / (float)d);
+    auto matrix = [&](PlainMat& w, int64_t valid, float gain) { fill(&w.data, m->f32, w.rows, w.cols, valid, 0.f, gain * sqrtf(3.f / (float)valid)); };
+    auto vector = [&](float*& p, int64_t n, float mid, float amp) { fill((void**)&p, true, 1, n, n, mid, amp); };
+    const int64_t d = m->cfg.d_model, gains = m->cfg.post_norm ? d : 1;
     fill(&m->embed, m->f32, m->cfg.vocab, d, d, 0.f, 1.7f);
-    fill(&m->head.data, m->f32, m->head.rows, m->head.cols, d, 0.f, a_in);
-    fill((void**)&m->final_gain, true, 1, 1, 1, 1.f, 0.f);
+    matrix(m->head, d, 1.f);
+    vector(m->final_gain, gains, 1.f, 0.f);
     m->set = ~0u;
     for (PlainLayer& l : m->layers) {
-        fill(&l.in.data, m->f32, l.in.rows, l.in.cols, d, 0.f, a_in);
-        fill(&l.out.data, m->f32, l.out.rows, l.out.cols, l.out.cols, 0.f, 0.5f * sqrtf(3.f / (float)l.out.cols));
-        fill((void**)&l.gain, true, 1, 1, 1, 1.f, 0.f);
-        fill((void**)&l.mu, true, 1, d, d, 0.5f, 0.4f);
-        fill((void**)&l.r1, true, 1, l.cfg.n_q_heads, l.cfg.n_q_heads, 1.f, 0.5f);
-        fill((void**)&l.r2, true, 1, l.cfg.n_q_heads, l.cfg.n_q_heads, 0.3f, 0.2f);
+        const tsb_plain_layer& c = l.cfg;
+        matrix(l.in, d, 1.f);
+        matrix(l.out, l.out.cols, 0.5f);
+        vector(l.gain, gains, 1.f, 0.f);
+        if (c.token_shift) vector(l.mu, d, 0.5f, 0.4f);
+        if (c.log_bias) vector(l.r1, c.n_q_heads, 1.f, 0.5f), vector(l.r2, c.n_q_heads, 0.3f, 0.2f);
+        if (c.sink) vector(l.sink, c.n_q_heads, 0.f, 1.f);
+        if (c.qk_norm) vector(l.q_norm, c.head_dim, 1.f, 0.2f), vector(l.k_norm, c.head_dim, 1.f, 0.2f);
+        if (l.post_norm && c.ffn > 0) matrix(l.ff_in, d, 1.f), matrix(l.ff_out, c.ffn, 0.5f), vector(l.norm2, d, 1.f, 0.f);
+        if (l.mixer == MIX_LATENT) {
+            vector(l.c_norm, c.kv_rank, 1.f, 0.f);
+            matrix(l.absorb, c.head_dim, 1.f), matrix(l.lift, c.kv_rank, 1.f);
+            if (l.expands) matrix(l.expand, c.kv_rank, 1.f);
+        }
         l.set = ~0u;
     }
     if (rc) return rc;
@@ -524,8 +1031,9 @@ int32_t tsb_kv_create_keys(tsb_ctx* ctx, int32_t type, int32_t layers, int32_t k
     if (!ctx || !out) return TSB_ERR_INVALID;
     TSB_REQUIRE(ctx, (type == TSB_BF16 || type == TSB_F32) && layers > 0 && kv_heads > 0, "unknown type or bad sizes");
     TSB_REQUIRE(ctx, wattn_pad_dim(head_dim, type == TSB_F32) == head_dim, "head size %d is not one the attention kernels work on", head_dim);
-    std::vector<int32_t> h((size_t)layers, kv_heads), d((size_t)layers, head_dim);
-    return kv_create_keys(ctx, layers, h.data(), d.data(), type == TSB_F32 ? 4 : 2, page_tokens, num_pages, max_seqs, max_pages_per_seq, out);
+    std::vector<KeyLayerShape> shapes;
+    for (int l = 0; l < layers; l++) shapes.push_back({kv_heads, head_dim, false, l});
+    return kv_create_keys(ctx, layers, shapes.data(), type == TSB_F32 ? 4 : 2, page_tokens, num_pages, max_seqs, max_pages_per_seq, out);
 }
 
 int32_t tsb_window_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, int32_t layer, const void* q, int64_t q_stride, void* out, int64_t out_stride,
@@ -558,7 +1066,7 @@ int32_t tsb_window_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, int32_t l
         TSB_CUDA(ctx, launch_window_attn(ctx, st, kv.elem_bytes == 4, a, b, scratch));
         return TSB_OK;
     }
-    const int grp = n_q_heads / kv.kv_heads, rpt = wattn_rows_per_tile(kv.head_dim, grp);
+    const int grp = n_q_heads / kv.kv_heads, rpt = wattn_rows_per_tile(kv.head_dim, grp, r1 != nullptr);
     std::vector<AttnTile> small, large;
     for (int i = 0, r = 0; i < n_groups; r += group_rows[i], i++) {
         if (group_rows[i] * grp <= WATTN_SMALL_Q) {

@@ -14,13 +14,18 @@ __device__ __forceinline__ float get(const __nv_bfloat16* p) { return __bfloat16
 
 template <typename T>
 __global__ void __launch_bounds__(ROW_THREADS)
-    plain_embed_kernel(const T* __restrict__ table, int vocab, int d, const int32_t* tokens, int token_stride, float* x, uint32_t* __restrict__ err) {
+    plain_embed_kernel(const T* __restrict__ table, int vocab, int d, const int32_t* tokens, int token_stride, float scale, float* x, T* out,
+                       int64_t out_stride, uint32_t* __restrict__ err) {
     pdl_wait();
     pdl_launch_dependents();
     const int tok = tokens[(int64_t)blockIdx.x * token_stride];
     const bool ok = tok >= 0 && tok < vocab;
     if (!ok && threadIdx.x == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
-    for (int i = threadIdx.x; i < d; i += ROW_THREADS) x[(int64_t)blockIdx.x * d + i] = ok ? get(table + (int64_t)tok * d + i) : 0.f;
+    for (int i = threadIdx.x; i < d; i += ROW_THREADS) {
+        const float v = ok ? scale * get(table + (int64_t)tok * d + i) : 0.f;
+        x[(int64_t)blockIdx.x * d + i] = v;
+        if (out) put(out + (int64_t)blockIdx.x * out_stride + i, v);
+    }
 }
 
 // sums of squares of one or two rows over the CTA, in a fixed order
@@ -154,8 +159,8 @@ __global__ void __launch_bounds__(ROW_THREADS) shift_before_kernel(ShiftState st
 
 template <typename T>
 __global__ void __launch_bounds__(ROW_THREADS)
-    norm_rows_kernel(const float* x, int d, const float* __restrict__ gain, float eps, const int32_t* __restrict__ want, int want_first, int want_step,
-                     T* out, int64_t out_stride) {
+    norm_rows_kernel(const float* x, int d, const float* __restrict__ gain, const float* __restrict__ weight, float eps, const int32_t* __restrict__ want,
+                     int want_first, int want_step, T* out, int64_t out_stride) {
     pdl_wait();
     pdl_launch_dependents();
     const int r = want ? want[blockIdx.x] : (int)blockIdx.x * want_step + want_first;
@@ -163,19 +168,146 @@ __global__ void __launch_bounds__(ROW_THREADS)
     float2 ss = make_float2(0.f, 0.f);
     for (int i = threadIdx.x; i < d; i += ROW_THREADS) ss.x = fmaf(xr[i], xr[i], ss.x);
     ss = block_sum2(ss);
-    const float s = *gain / sqrtf(ss.x / (float)d + eps);
-    for (int i = threadIdx.x; i < d; i += ROW_THREADS) put(out + (int64_t)blockIdx.x * out_stride + i, xr[i] * s);
+    const float s = (weight ? 1.f : *gain) / sqrtf(ss.x / (float)d + eps);
+    for (int i = threadIdx.x; i < d; i += ROW_THREADS) put(out + (int64_t)blockIdx.x * out_stride + i, xr[i] * s * (weight ? weight[i] : 1.f));
+}
+
+// VEC as in the norm + shift kernel: a thread holds its columns of the row in registers.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(ROW_THREADS)
+    post_norm_kernel(float* x, int d, const float* __restrict__ weight, float eps, T* out, int64_t out_stride) {
+    float* xr = x + (int64_t)blockIdx.x * d;
+    T* o = out + (int64_t)blockIdx.x * out_stride;
+    float4 w[VEC ? ROW_VECS : 1];
+    if (VEC) {
+#pragma unroll
+        for (int k = 0; k < ROW_VECS; k++) {
+            const int i = (k * ROW_THREADS + threadIdx.x) * 4;
+            if (i < d) w[k] = *reinterpret_cast<const float4*>(weight + i);
+        }
+    }
+    pdl_wait();
+    pdl_launch_dependents();
+    float2 ss = make_float2(0.f, 0.f);
+    if (VEC) {
+        float4 v[ROW_VECS];
+#pragma unroll
+        for (int k = 0; k < ROW_VECS; k++) {
+            const int i = (k * ROW_THREADS + threadIdx.x) * 4;
+            v[k] = i < d ? *reinterpret_cast<const float4*>(xr + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int k = 0; k < ROW_VECS; k++) ss.x = sum4(v[k], ss.x);
+        const float s = 1.f / sqrtf(block_sum2(ss).x / (float)d + eps);
+#pragma unroll
+        for (int k = 0; k < ROW_VECS; k++) {
+            const int i = (k * ROW_THREADS + threadIdx.x) * 4;
+            if (i >= d) break;
+            const float4 h = make_float4(v[k].x * s * w[k].x, v[k].y * s * w[k].y, v[k].z * s * w[k].z, v[k].w * s * w[k].w);
+            put4(xr + i, h);
+            put4(o + i, h);
+        }
+        return;
+    }
+    for (int i = threadIdx.x; i < d; i += ROW_THREADS) ss.x = fmaf(xr[i], xr[i], ss.x);
+    const float s = 1.f / sqrtf(block_sum2(ss).x / (float)d + eps);
+    for (int i = threadIdx.x; i < d; i += ROW_THREADS) {
+        const float h = xr[i] * s * weight[i];
+        xr[i] = h;
+        put(o + i, h);
+    }
+}
+
+// a warp per (row, head)
+template <typename T>
+__global__ void __launch_bounds__(ROW_THREADS) head_norms_kernel(const __grid_constant__ HeadNorms h, int rows, uint32_t* __restrict__ err) {
+    const int lane = threadIdx.x & 31;
+    const int64_t item = (int64_t)blockIdx.x * (ROW_THREADS / 32) + (threadIdx.x >> 5);
+    const int per = h.n_q + h.n_k;
+    const bool in = item < (int64_t)rows * per;
+    const int r = in ? (int)(item / per) : 0, head = in ? (int)(item % per) : 0;
+    const tsb_row_desc rd = h.rows[r];
+    pdl_wait();
+    pdl_launch_dependents();
+    if (!in) return;
+    const bool query = head < h.n_q;
+    const float* src = h.raw + (int64_t)r * h.raw_stride + (int64_t)head * h.width;
+    const float* w = query ? h.q_weight : h.k_weight;
+    float ss = 0.f;
+    for (int i = lane; i < h.width; i += 32) ss = fmaf(src[i], src[i], ss);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    float s = 1.f / sqrtf(ss / (float)h.width + h.eps);
+    const int pos = rd.base + rd.slot;
+    T* dst;
+    int width = h.width;
+    if (query) {
+        if (h.temp_every > 0) s *= 1.f + h.temp_coef * logf((float)((pos + 1) / h.temp_every + 1));
+        dst = static_cast<T*>(h.q) + (int64_t)r * h.q_stride + (int64_t)head * h.q_step;
+        width = h.q_width;
+    } else {
+        dst = key_row<T>(h.keys, rd.seq, pos);
+        if (!dst) {
+            if (lane == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+            return;
+        }
+        dst += (int64_t)(head - h.n_q) * h.keys.head_step;
+    }
+    for (int i = lane; i < width; i += 32) put(dst + i, i < h.width ? src[i] * s * w[i] : 0.f);
+}
+
+__global__ void __launch_bounds__(ROW_THREADS)
+    rotary_table_kernel(const float* __restrict__ freq, int half, float magnitude, const tsb_row_desc* __restrict__ rows, int n, float2* table) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const int64_t k = (int64_t)blockIdx.x * ROW_THREADS + threadIdx.x;
+    if (k >= (int64_t)n * half) return;
+    const tsb_row_desc& rd = rows[k / half];
+    float s, c;
+    sincosf((float)(rd.base + rd.slot) * freq[k % half], &s, &c);
+    table[k] = make_float2(magnitude * c, magnitude * s);
+}
+
+// a CTA per position and stream
+__global__ void __launch_bounds__(ROW_THREADS) latent_gather_kernel(const __grid_constant__ LatentGather g, uint32_t* __restrict__ err) {
+    const ExpandStream es = g.streams[blockIdx.y];
+    const tsb_row_desc rd = g.rows[es.first_row];
+    const int pos = blockIdx.x, len = rd.base + es.n_rows;
+    pdl_wait();
+    pdl_launch_dependents();
+    if (pos >= len) return;
+    const int wide_lp = pos >> g.wide.page_shift, wide_page = es.first_page + wide_lp;
+    if (rd.seq < 0 || rd.seq >= g.wide.max_seqs || wide_lp >= g.wide.max_pages_per_seq || wide_page >= g.wide.num_pages) {
+        if (threadIdx.x == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+        return;
+    }
+    if (threadIdx.x == 0 && (pos & (g.wide.page_tokens - 1)) == 0) g.wide_table[(int64_t)rd.seq * g.wide.max_pages_per_seq + wide_lp] = wide_page;
+    const __nv_bfloat16* src = key_row<__nv_bfloat16>(g.cache, rd.seq, pos);
+    if (!src) {
+        if (threadIdx.x == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+        return;
+    }
+    const int64_t at = (int64_t)wide_page * g.wide.page_tokens + (pos & (g.wide.page_tokens - 1));
+    const uint4* s16 = reinterpret_cast<const uint4*>(src);
+    uint4* d16 = reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(g.latents) + at * g.cache.row);
+    for (int i = threadIdx.x; i < g.cache.row / 8; i += ROW_THREADS) d16[i] = s16[i];
+    __nv_bfloat16* wide = reinterpret_cast<__nv_bfloat16*>(g.wide.base) + at * g.wide.row;
+    const int tail = g.wide.head_dim - g.key_off;
+    for (int i = threadIdx.x; i < g.wide.kv_heads * tail; i += ROW_THREADS) {
+        const int head = i / tail, k = i - head * tail;
+        wide[(int64_t)head * g.wide.head_step + g.key_off + k] = k < g.rot_dim ? src[g.kv_rank + k] : __float2bfloat16_rn(0.f);
+    }
 }
 
 }  // namespace
 
 cudaError_t launch_plain_embed(tsb_ctx* ctx, cudaStream_t st, bool f32, const void* table, int vocab, int d, const int32_t* tokens, int token_stride,
-                               int rows, float* x) {
+                               int rows, float scale, float* x, void* out, int64_t out_stride) {
     if (f32)
         return tsb_launch(ctx, plain_embed_kernel<float>, dim3((unsigned)rows), dim3(ROW_THREADS), 0, st, true, (const float*)table, vocab, d, tokens,
-                          token_stride, x, ctx->dev_error);
+                          token_stride, scale, x, (float*)out, out_stride, ctx->dev_error);
     return tsb_launch(ctx, plain_embed_kernel<__nv_bfloat16>, dim3((unsigned)rows), dim3(ROW_THREADS), 0, st, true, (const __nv_bfloat16*)table, vocab, d,
-                      tokens, token_stride, x, ctx->dev_error);
+                      tokens, token_stride, scale, x, (__nv_bfloat16*)out, out_stride, ctx->dev_error);
 }
 
 cudaError_t launch_norm_shift(tsb_ctx* ctx, cudaStream_t st, bool f32, const float* x, int d, const float* gain, float eps, const float* mu,
@@ -194,11 +326,35 @@ cudaError_t launch_shift_before(tsb_ctx* ctx, cudaStream_t st, ShiftState state,
     return tsb_launch(ctx, shift_before_kernel, dim3((unsigned)rows, (unsigned)layers), dim3(ROW_THREADS), 0, st, true, state, rows_dev);
 }
 
-cudaError_t launch_norm_rows(tsb_ctx* ctx, cudaStream_t st, bool f32, const float* x, int d, const float* gain, float eps, const int32_t* want_dev,
-                             int want_first, int want_step, int n, void* out, int64_t out_stride) {
+cudaError_t launch_norm_rows(tsb_ctx* ctx, cudaStream_t st, bool f32, const float* x, int d, const float* gain, const float* weight, float eps,
+                             const int32_t* want_dev, int want_first, int want_step, int n, void* out, int64_t out_stride) {
     if (f32)
-        return tsb_launch(ctx, norm_rows_kernel<float>, dim3((unsigned)n), dim3(ROW_THREADS), 0, st, true, x, d, gain, eps, want_dev, want_first, want_step,
-                          (float*)out, out_stride);
-    return tsb_launch(ctx, norm_rows_kernel<__nv_bfloat16>, dim3((unsigned)n), dim3(ROW_THREADS), 0, st, true, x, d, gain, eps, want_dev, want_first,
-                      want_step, (__nv_bfloat16*)out, out_stride);
+        return tsb_launch(ctx, norm_rows_kernel<float>, dim3((unsigned)n), dim3(ROW_THREADS), 0, st, true, x, d, gain, weight, eps, want_dev, want_first,
+                          want_step, (float*)out, out_stride);
+    return tsb_launch(ctx, norm_rows_kernel<__nv_bfloat16>, dim3((unsigned)n), dim3(ROW_THREADS), 0, st, true, x, d, gain, weight, eps, want_dev,
+                      want_first, want_step, (__nv_bfloat16*)out, out_stride);
+}
+
+cudaError_t launch_post_norm(tsb_ctx* ctx, cudaStream_t st, bool f32, float* x, int d, const float* weight, float eps, int rows, void* out,
+                             int64_t out_stride) {
+    auto run = [&](auto kernel, auto* o) { return tsb_launch(ctx, kernel, dim3((unsigned)rows), dim3(ROW_THREADS), 0, st, true, x, d, weight, eps, o, out_stride); };
+    const bool vec = d % 4 == 0 && out_stride % 4 == 0 && d <= 4 * ROW_THREADS * ROW_VECS;
+    if (f32) return run(vec ? post_norm_kernel<float, true> : post_norm_kernel<float, false>, (float*)out);
+    return run(vec ? post_norm_kernel<__nv_bfloat16, true> : post_norm_kernel<__nv_bfloat16, false>, (__nv_bfloat16*)out);
+}
+
+cudaError_t launch_head_norms(tsb_ctx* ctx, cudaStream_t st, bool f32, const HeadNorms& h, int rows) {
+    constexpr int WARPS = ROW_THREADS / 32;
+    const dim3 grid((unsigned)(((int64_t)rows * (h.n_q + h.n_k) + WARPS - 1) / WARPS));
+    return tsb_launch(ctx, f32 ? head_norms_kernel<float> : head_norms_kernel<__nv_bfloat16>, grid, dim3(ROW_THREADS), 0, st, true, h, rows, ctx->dev_error);
+}
+
+cudaError_t launch_rotary_table(tsb_ctx* ctx, cudaStream_t st, const float* freq, int half, float magnitude, const tsb_row_desc* rows_dev, int rows,
+                                float2* table) {
+    return tsb_launch(ctx, rotary_table_kernel, dim3((unsigned)(((int64_t)rows * half + ROW_THREADS - 1) / ROW_THREADS)), dim3(ROW_THREADS), 0, st, true, freq,
+                      half, magnitude, rows_dev, rows, table);
+}
+
+cudaError_t launch_latent_gather(tsb_ctx* ctx, cudaStream_t st, const LatentGather& g, int n_streams, int max_len) {
+    return tsb_launch(ctx, latent_gather_kernel, dim3((unsigned)max_len, (unsigned)n_streams), dim3(ROW_THREADS), 0, st, true, g, ctx->dev_error);
 }

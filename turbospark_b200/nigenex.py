@@ -5,14 +5,9 @@ its keys, with capped scores, a logarithmic distance bias and one output gate pe
 capped logits.  Every size and constant comes from config.json.
 """
 from . import plain
+from .plain import need as _need
 
 ARCHITECTURE = "Nigenex"
-
-
-def _need(d, key, where):
-    if not isinstance(d, dict) or key not in d:
-        raise ValueError("config: %s has no '%s'" % (where, key))
-    return d[key]
 
 
 def parse_config(config, max_context, compute=plain.BF16):
@@ -61,11 +56,4 @@ def load_tensors(model, get):
 
 
 def build(ctx, config, get, max_context, compute):
-    cfg, layers = parse_config(config, max_context, compute)
-    model = plain.PlainModel(ctx, cfg, layers)
-    try:
-        load_tensors(model, get)
-    except Exception:
-        model.close()
-        raise
-    return model
+    return plain.build(ctx, *parse_config(config, max_context, compute), load_tensors, get)

@@ -9,18 +9,29 @@ from .model import Model
 BF16, F32 = 0, 1
 GELU_TANH, SILU = 0, 1
 (P_EMBED, P_HEAD, P_FINAL_NORM, P_NORM, P_SHIFT, P_Q, P_K, P_HEAD_GATE, P_R1, P_R2, P_O, P_FF_GATE, P_FF_UP,
- P_FF_DOWN) = range(14)
+ P_FF_DOWN, P_NORM2, P_V, P_Q_NORM, P_K_NORM, P_SINK, P_VALUE_GATE, P_DKV, P_DKV_NORM, P_UK, P_UV) = range(24)
 
 
 class PlainConfig(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("n_layers", "d_model", "vocab", "max_context", "compute")] + \
-               [("norm_eps", C.c_float), ("logit_cap", C.c_float)]
+               [("norm_eps", C.c_float), ("logit_cap", C.c_float), ("post_norm", C.c_int32), ("residual_scale", C.c_float),
+                ("embed_scale", C.c_float)]
 
 
 class PlainLayer(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("n_q_heads", "n_kv_heads", "head_dim", "window")] + \
                [("score_scale", C.c_float), ("score_cap", C.c_float)] + \
-               [(n, C.c_int32) for n in ("log_bias", "head_gate", "token_shift", "ffn", "act")]
+               [(n, C.c_int32) for n in ("log_bias", "head_gate", "token_shift", "ffn", "act", "value_dim", "qk_norm", "q_temp_every")] + \
+               [("q_temp_coef", C.c_float)] + \
+               [(n, C.c_int32) for n in ("sink", "value_gate", "kv_rank", "rot_dim", "kv_source")] + \
+               [(n, C.c_double) for n in ("rot_base", "rot_factor", "rot_original", "rot_fast", "rot_slow")]
+
+
+def need(d, key, where):
+    """The value of a key that a configuration must have."""
+    if not isinstance(d, dict) or key not in d:
+        raise ValueError("config: %s has no '%s'" % (where, key))
+    return d[key]
 
 
 def bf16_bits(x):
@@ -53,3 +64,14 @@ class PlainModel(Model):
     def fill(self, seed=0):
         """Seeded random weights made on the device."""
         self.ctx.check(lib().tsb_model_fill_plain(self.h, C.c_uint64(seed)))
+
+
+def build(ctx, cfg, layers, load_tensors, get):
+    """A model with its tensors: load_tensors(model, get) uploads what get(name) returns."""
+    model = PlainModel(ctx, cfg, layers)
+    try:
+        load_tensors(model, get)
+    except Exception:
+        model.close()
+        raise
+    return model
