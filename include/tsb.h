@@ -488,6 +488,42 @@ TSB_API int32_t tsb_window_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, i
                                      int64_t out_stride, const tsb_row_desc* rows_dev, const int32_t* group_rows, int32_t n_groups,
                                      int32_t n_q_heads, float scale, float cap, const float* r1, const float* r2, const float* gate,
                                      int32_t window, int32_t max_len, void* scratch);
+/* The same over any plain cache, with everything a layer may add to it. */
+TSB_API int32_t tsb_kv_create_plain(tsb_ctx* ctx, int32_t type, int32_t layers, int32_t kv_heads, int32_t key_dim, int32_t value_dim, int32_t page_tokens,
+                                    int32_t num_pages, int32_t max_seqs, int32_t max_pages_per_seq, tsb_kv** out); /* value_dim 0: the values are the keys;
+                                    else rows of [key, value] per head */
+typedef struct tsb_attention_extras {
+    float cap;                    /* > 0: soft cap */
+    int32_t window;               /* > 0: sliding window */
+    const float *r1, *r2;         /* distance bias, [n_q_heads] or NULL */
+    const float* head_gate;       /* [rows, n_q_heads] f32 pre-activations or NULL */
+    const float* sink;            /* [n_q_heads] or NULL */
+    const void* value_gate;       /* [rows, n_q_heads * value columns] pre-activations in `type`, or NULL */
+    int64_t value_gate_stride;
+} tsb_attention_extras;
+/* bfloat16 with keys and values of different widths: one query head per key head, keys of 64, 128 or 192, values of 64 or 128 columns. */
+TSB_API int32_t tsb_plain_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, int32_t layer, const void* q, int64_t q_stride, void* out,
+                                    int64_t out_stride, const tsb_row_desc* rows_dev, const int32_t* group_rows, int32_t n_groups,
+                                    int32_t n_q_heads, float scale, const tsb_attention_extras* extras, int32_t max_len, void* scratch);
+/* Attention over latent rows (a cache of one head whose first value_dim columns are the value): every query head reads the same
+ * row.  q [rows, n_heads, key columns], out [rows, n_heads, value_dim].  value_dim 64, 128, 192, 256, 384 or 512; key columns a
+ * multiple of 32, at least value_dim. */
+TSB_API int32_t tsb_latent_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* cache, int32_t layer, const void* q, int64_t q_stride, void* out,
+                                     int64_t out_stride, const tsb_row_desc* rows_dev, const int32_t* group_rows, int32_t n_groups, int32_t n_heads,
+                                     int32_t value_dim, float scale, const float* sink, int32_t max_len, void* scratch);
+/* A product per head: y[t, h * y_step + n] = sum_k W[h * head_rows + n, k] x[t, h * x_step + k] for n < n_valid, in `type`, times
+ * sigmoid(gate[t, h * gate_step + n]) when a gate is given.  head_rows a multiple of 128, cols and x_step multiples of 64. */
+TSB_API int32_t tsb_plain_gemm_heads(tsb_ctx* ctx, tsb_stream s, int32_t type, const void* w, int32_t heads, int32_t head_rows, int64_t cols, const void* x,
+                                     int64_t x_stride, int32_t x_step, int32_t x_rows, int32_t tokens, void* y, int64_t y_stride, int32_t y_step,
+                                     int32_t n_valid, const void* gate, int64_t gate_stride, int32_t gate_step, void* workspace);
+/* x[r, :] = x * weight / sqrt(mean(x^2) + eps) in place (f32), and to out in `type`. */
+TSB_API int32_t tsb_post_norm_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, float* x, int32_t d, const float* weight, float eps, int32_t rows, void* out,
+                                   int64_t out_stride);
+/* Per-head norms of projected queries and keys (f32 raw [rows, (n_q + n_k) * width]): queries to q [rows, n_q, key columns], times
+ * 1 + temp_coef ln(floor((p + 1) / temp_every) + 1) when temp_every > 0; keys to the cache at the rows' positions. */
+TSB_API int32_t tsb_head_norm_rows(tsb_ctx* ctx, tsb_stream s, tsb_kv* cache, int32_t layer, const float* raw, int64_t raw_stride, int32_t n_q, int32_t n_k,
+                                   int32_t width, const float* q_weight, const float* k_weight, float eps, float temp_coef, int32_t temp_every,
+                                   const tsb_row_desc* rows_dev, int32_t rows, void* q, int64_t q_stride);
 TSB_API size_t tsb_window_attention_scratch_bytes(const tsb_ctx* ctx); /* zeroed once by the caller */
 
 /* ------------------------------------------------------------------ resident weight file

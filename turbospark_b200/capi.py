@@ -314,6 +314,38 @@ class Ctx:
                                               _vp(rows_dev), gr, C.c_int32(len(group_rows)), C.c_int32(n_q_heads), C.c_float(scale), C.c_float(cap),
                                               _vp(r1), _vp(r2), _vp(gate), C.c_int32(window), C.c_int32(max_len), _vp(scratch)))
 
+    def plain_attention(self, kv, layer, q, q_stride, out, out_stride, rows_dev, group_rows, n_q_heads, scale, max_len, scratch, stream=None, cap=0.0,
+                        window=0, r1=None, r2=None, head_gate=None, sink=None, value_gate=None, value_gate_stride=0):
+        gr = (C.c_int32 * len(group_rows))(*group_rows)
+        x = AttentionExtras(cap, window, _vp(r1), _vp(r2), _vp(head_gate), _vp(sink), _vp(value_gate), value_gate_stride)
+        self.check(lib().tsb_plain_attention(self.h, stream, kv.h, C.c_int32(layer), _vp(q), C.c_int64(q_stride), _vp(out), C.c_int64(out_stride),
+                                             _vp(rows_dev), gr, C.c_int32(len(group_rows)), C.c_int32(n_q_heads), C.c_float(scale), C.byref(x),
+                                             C.c_int32(max_len), _vp(scratch)))
+
+    def latent_attention(self, kv, layer, q, q_stride, out, out_stride, rows_dev, group_rows, n_heads, value_dim, scale, sink, max_len, scratch,
+                         stream=None):
+        gr = (C.c_int32 * len(group_rows))(*group_rows)
+        self.check(lib().tsb_latent_attention(self.h, stream, kv.h, C.c_int32(layer), _vp(q), C.c_int64(q_stride), _vp(out), C.c_int64(out_stride),
+                                              _vp(rows_dev), gr, C.c_int32(len(group_rows)), C.c_int32(n_heads), C.c_int32(value_dim), C.c_float(scale),
+                                              _vp(sink), C.c_int32(max_len), _vp(scratch)))
+
+    def plain_gemm_heads(self, type_, w, heads, head_rows, cols, x, x_stride, x_step, x_rows, tokens, y, y_stride, y_step, n_valid, workspace, gate=None,
+                         gate_stride=0, gate_step=0, stream=None):
+        self.check(lib().tsb_plain_gemm_heads(self.h, stream, C.c_int32(type_), _vp(w), C.c_int32(heads), C.c_int32(head_rows), C.c_int64(cols), _vp(x),
+                                              C.c_int64(x_stride), C.c_int32(x_step), C.c_int32(x_rows), C.c_int32(tokens), _vp(y), C.c_int64(y_stride),
+                                              C.c_int32(y_step), C.c_int32(n_valid), _vp(gate), C.c_int64(gate_stride), C.c_int32(gate_step),
+                                              _vp(workspace)))
+
+    def post_norm_rows(self, type_, x, d, weight, eps, rows, out, out_stride, stream=None):
+        self.check(lib().tsb_post_norm_rows(self.h, stream, C.c_int32(type_), _vp(x), C.c_int32(d), _vp(weight), C.c_float(eps), C.c_int32(rows), _vp(out),
+                                            C.c_int64(out_stride)))
+
+    def head_norm_rows(self, kv, layer, raw, raw_stride, n_q, n_k, width, q_weight, k_weight, eps, rows_dev, rows, q, q_stride, temp_coef=0.0, temp_every=0,
+                       stream=None):
+        self.check(lib().tsb_head_norm_rows(self.h, stream, kv.h, C.c_int32(layer), _vp(raw), C.c_int64(raw_stride), C.c_int32(n_q), C.c_int32(n_k),
+                                            C.c_int32(width), _vp(q_weight), _vp(k_weight), C.c_float(eps), C.c_float(temp_coef), C.c_int32(temp_every),
+                                            _vp(rows_dev), C.c_int32(rows), _vp(q), C.c_int64(q_stride)))
+
     def residual_add(self, x, y, n, stream=None):
         self.check(lib().tsb_residual_add(self.h, stream, _vp(x), _vp(y), C.c_int64(n)))
 
@@ -379,15 +411,21 @@ class KvCache:
             self.h = None
 
 
-class KeyCache(KvCache):
-    """A key-only cache: rows of kv_heads * head_dim bfloat16 bit patterns (type 0) or f32 values (type 1)."""
+class AttentionExtras(C.Structure):
+    _fields_ = [("cap", C.c_float), ("window", C.c_int32)] + [(n, C.c_void_p) for n in ("r1", "r2", "head_gate", "sink", "value_gate")] + \
+               [("value_gate_stride", C.c_int64)]
 
-    def __init__(self, ctx, type_, layers, kv_heads, head_dim, page_tokens, num_pages, max_seqs, max_pages_per_seq):
+
+class PlainCache(KvCache):
+    """A plain cache: rows of kv_heads * [key, value] (value_dim 0: the values are the keys), bfloat16 bit patterns (type 0) or f32
+    values (type 1)."""
+
+    def __init__(self, ctx, type_, layers, kv_heads, key_dim, value_dim, page_tokens, num_pages, max_seqs, max_pages_per_seq):
         self.ctx, self.type = ctx, type_
-        self.layers, self.kv_heads, self.head_dim = layers, kv_heads, head_dim
+        self.layers, self.kv_heads, self.head_dim = layers, kv_heads, key_dim + value_dim
         h = C.c_void_p()
-        ctx.check(lib().tsb_kv_create_keys(ctx.h, C.c_int32(type_), C.c_int32(layers), C.c_int32(kv_heads), C.c_int32(head_dim), C.c_int32(page_tokens),
-                                           C.c_int32(num_pages), C.c_int32(max_seqs), C.c_int32(max_pages_per_seq), C.byref(h)))
+        ctx.check(lib().tsb_kv_create_plain(ctx.h, C.c_int32(type_), C.c_int32(layers), C.c_int32(kv_heads), C.c_int32(key_dim), C.c_int32(value_dim),
+                                            C.c_int32(page_tokens), C.c_int32(num_pages), C.c_int32(max_seqs), C.c_int32(max_pages_per_seq), C.byref(h)))
         self.h = h
 
     def write_rows(self, seq, layer, pos0, k, stream=None):
@@ -399,3 +437,15 @@ class KeyCache(KvCache):
         k = np.empty((n, self.kv_heads * self.head_dim), dtype=np.float32 if self.type else np.uint16)
         self.ctx.check(lib().tsb_kv_read_rows(self.h, stream, C.c_int32(seq), C.c_int32(layer), C.c_int64(pos0), C.c_int32(n), _vp(k), None))
         return k
+
+
+class KeyCache(PlainCache):
+    """A key-only cache: the head size must be one that the attention kernels work on."""
+
+    def __init__(self, ctx, type_, layers, kv_heads, head_dim, page_tokens, num_pages, max_seqs, max_pages_per_seq):
+        self.ctx, self.type = ctx, type_
+        self.layers, self.kv_heads, self.head_dim = layers, kv_heads, head_dim
+        h = C.c_void_p()
+        ctx.check(lib().tsb_kv_create_keys(ctx.h, C.c_int32(type_), C.c_int32(layers), C.c_int32(kv_heads), C.c_int32(head_dim), C.c_int32(page_tokens),
+                                           C.c_int32(num_pages), C.c_int32(max_seqs), C.c_int32(max_pages_per_seq), C.byref(h)))
+        self.h = h

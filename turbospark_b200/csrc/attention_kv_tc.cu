@@ -10,8 +10,12 @@ bool wattn_wide_supported(int key_dim, int value_dim) {
 }
 
 cudaError_t launch_window_attn_wide(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const AttnBatch& b, void* scratch) {
-    if (b.n_large == 0) return cudaSuccess;
-    const WattnLaunch l{b.large, b.n_large, 1, 0, WATTN_WIDE_ROWS, b.max_len};
+    WattnLaunch l{b.large, b.n_large, 1, 0, WATTN_WIDE_ROWS, b.max_len};
+    if (b.rows_per_seq > 0) {
+        const int tpg = (b.rows_per_seq + WATTN_WIDE_ROWS - 1) / WATTN_WIDE_ROWS;
+        l = WattnLaunch{nullptr, b.rows / b.rows_per_seq * tpg, tpg, b.rows_per_seq, WATTN_WIDE_ROWS, b.max_len};
+    }
+    if (l.n_tiles == 0) return cudaSuccess;
     const int dk = a.keys.head_dim, dv = a.value_dim;
     if (dk == 64 && dv == 64) return launch_tc<64, 64, 128, true>(ctx, st, a, l, scratch);
     if (dk == 64 && dv == 128) return launch_tc<64, 128, 128, true>(ctx, st, a, l, scratch);

@@ -45,8 +45,8 @@ struct AttnBatch {
 size_t wattn_scratch_bytes(const tsb_ctx* ctx);  // zeroed once by the owner; the kernels leave its tickets at zero
 bool wattn_supported(int head_dim, int group, bool f32);
 int wattn_pad_dim(int head_dim, bool f32);       // the head size the kernels work on (zero columns behind the real ones); 0: too large
-// The many-query kernel for keys and values of different widths: every query head has a key head of its own, `large` tiles of
-// wattn_wide_rows rows.  0: no such kernel.
+// The many-query kernel for keys and values of different widths: every query head has a key head of its own; the `large` tiles
+// of a list have at most WATTN_WIDE_ROWS rows.
 constexpr int WATTN_WIDE_ROWS = 2 * WATTN_LARGE_Q;
 bool wattn_wide_supported(int key_dim, int value_dim);
 cudaError_t launch_window_attn_wide(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const AttnBatch& b, void* scratch);

@@ -196,10 +196,10 @@ int32_t kv_create_keys(tsb_ctx* ctx, int n_layers, const KeyLayerShape* shapes, 
     if (!kv) return TSB_ERR_OOM;
     int32_t rc = kv_init_pages(ctx, kv, page_tokens, num_pages, max_seqs, max_pages_per_seq);
     size_t bytes = 0;
-    auto row_of = [&](int l) { return shapes[l].kv_heads * shapes[l].head_dim * (shapes[l].values ? 2 : 1); };
+    auto row_of = [&](int l) { return shapes[l].kv_heads * (shapes[l].head_dim + shapes[l].value_dim); };
     for (int l = 0; l < n_layers && rc == TSB_OK; l++) {
         const KeyLayerShape& k = shapes[l];
-        if (k.kv_heads <= 0 || k.head_dim <= 0 || (k.head_dim * elem_bytes) % 16)
+        if (k.kv_heads <= 0 || k.head_dim <= 0 || k.value_dim < 0 || (k.head_dim * elem_bytes) % 16 || (k.value_dim * elem_bytes) % 16)
             rc = tsb_fail(ctx, TSB_ERR_INVALID, "layer %d: bad head count or head size", l);
         else if (k.source < 0 || k.source > l || shapes[k.source].source != k.source || row_of(k.source) != row_of(l))
             rc = tsb_fail(ctx, TSB_ERR_INVALID, "layer %d cannot read the rows of layer %d", l, k.source);
@@ -217,7 +217,7 @@ int32_t kv_create_keys(tsb_ctx* ctx, int n_layers, const KeyLayerShape* shapes, 
         const bool own = shapes[l].source == l;
         k.base = own ? kv->key_pool + off : kv->key_layers[shapes[l].source].base, k.page_table = kv->page_table_dev;
         k.kv_heads = shapes[l].kv_heads, k.head_dim = shapes[l].head_dim, k.elem_bytes = elem_bytes;
-        k.row = row_of(l), k.value_off = shapes[l].values ? k.head_dim : 0, k.head_step = k.head_dim + k.value_off;
+        k.row = row_of(l), k.value_off = shapes[l].value_dim ? k.head_dim : 0, k.head_step = k.head_dim + shapes[l].value_dim;
         k.page_shift = kv->view.page_shift, k.page_tokens = page_tokens, k.num_pages = num_pages;
         k.max_seqs = max_seqs, k.max_pages_per_seq = max_pages_per_seq;
         kv->key_layers.push_back(k);

@@ -20,7 +20,7 @@ struct KvView {
 // kv_heads heads, head_step elements apart; a head's key is head_dim elements from its start, its value starts value_off
 // elements behind it:
 //   values that are their keys   head_step = head_dim, value_off = 0
-//   keys and values              head_step = 2 head_dim, value_off = head_dim
+//   keys and values              head_step = head_dim + the value's elements, value_off = head_dim
 //   latent rows                  one head: the latent, which is also the value, then the rotated key part
 // Layers may differ in all of it.
 struct KeyView {
@@ -32,7 +32,7 @@ struct KeyView {
 };
 struct KeyLayerShape {
     int kv_heads, head_dim;
-    bool values;   // a value of head_dim elements behind every key
+    int value_dim; // elements of the value behind every key (0: the values are the keys)
     int source;    // the layer whose rows this one reads (itself: rows of its own)
 };
 

@@ -18,6 +18,7 @@
 //                                latents to gated values); long portions: expansion of the stream's latents to keys and values, attention
 #include <algorithm>
 #include <cstring>
+#include <functional>
 #include <new>
 
 #include "model_plain.cuh"
@@ -181,8 +182,8 @@ int32_t plain_runtime_init(tsb_session* s, ModelRt& rt, const tsb_model* tm, con
     rt.model = tm;
     std::vector<KeyLayerShape> shapes;
     for (const PlainLayer& l : m->layers) {
-        if (l.mixer == MIX_LATENT) shapes.push_back({1, l.key_dim, false, l.source});
-        else shapes.push_back({l.cfg.n_kv_heads, l.head_pad, l.mixer == MIX_KV, (int)shapes.size()});
+        if (l.mixer == MIX_LATENT) shapes.push_back({1, l.key_dim, 0, l.source});
+        else shapes.push_back({l.cfg.n_kv_heads, l.head_pad, l.mixer == MIX_KV ? l.head_pad : 0, (int)shapes.size()});
     }
     int32_t rc = kv_create_keys(ctx, m->cfg.n_layers, shapes.data(), m->elem, shape.page_tokens, shape.num_pages, shape.n_streams, shape.pages_per_seq, &rt.kv);
     if (rc) return rc;
@@ -640,7 +641,7 @@ int rotation_of(PlainModel* m, const tsb_plain_layer& c) {
 }
 
 int32_t upload_rotation(tsb_ctx* ctx, PlainRotation& r) {
-    std::vector<float> freq(r.dims / 2);
+    std::vector<double> freq(r.dims / 2);
     const bool scaled = r.factor > 0;
     // the pair that turns t times within the original context
     auto pair_with_turns = [&](double t) { return r.dims * log(r.original / (2 * M_PI * t)) / (2 * log(r.base)); };
@@ -649,11 +650,11 @@ int32_t upload_rotation(tsb_ctx* ctx, PlainRotation& r) {
     for (int i = 0; i < r.dims / 2; i++) {
         const double f = pow(r.base, -2.0 * i / r.dims);
         const double ramp = scaled ? std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0) : 0;
-        freq[i] = (float)(scaled ? f / r.factor * ramp + f * (1 - ramp) : f);
+        freq[i] = scaled ? f / r.factor * ramp + f * (1 - ramp) : f;
     }
     r.magnitude = scaled ? (float)(0.1 * log(r.factor) + 1.0) : 1.f;
-    if (int32_t rc = tsb_alloc(ctx, freq.size() * 4, (void**)&r.freq)) return rc;
-    TSB_CUDA(ctx, cudaMemcpy(r.freq, freq.data(), freq.size() * 4, cudaMemcpyHostToDevice));
+    if (int32_t rc = tsb_alloc(ctx, freq.size() * sizeof(double), (void**)&r.freq)) return rc;
+    TSB_CUDA(ctx, cudaMemcpy(r.freq, freq.data(), freq.size() * sizeof(double), cudaMemcpyHostToDevice));
     return TSB_OK;
 }
 
@@ -1029,30 +1030,73 @@ int32_t tsb_norm_shift_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, const floa
 int32_t tsb_kv_create_keys(tsb_ctx* ctx, int32_t type, int32_t layers, int32_t kv_heads, int32_t head_dim, int32_t page_tokens, int32_t num_pages,
                            int32_t max_seqs, int32_t max_pages_per_seq, tsb_kv** out) {
     if (!ctx || !out) return TSB_ERR_INVALID;
-    TSB_REQUIRE(ctx, (type == TSB_BF16 || type == TSB_F32) && layers > 0 && kv_heads > 0, "unknown type or bad sizes");
     TSB_REQUIRE(ctx, wattn_pad_dim(head_dim, type == TSB_F32) == head_dim, "head size %d is not one the attention kernels work on", head_dim);
+    return tsb_kv_create_plain(ctx, type, layers, kv_heads, head_dim, 0, page_tokens, num_pages, max_seqs, max_pages_per_seq, out);
+}
+
+int32_t tsb_kv_create_plain(tsb_ctx* ctx, int32_t type, int32_t layers, int32_t kv_heads, int32_t key_dim, int32_t value_dim, int32_t page_tokens,
+                            int32_t num_pages, int32_t max_seqs, int32_t max_pages_per_seq, tsb_kv** out) {
+    if (!ctx || !out) return TSB_ERR_INVALID;
+    TSB_REQUIRE(ctx, (type == TSB_BF16 || type == TSB_F32) && layers > 0 && kv_heads > 0, "unknown type or bad sizes");
     std::vector<KeyLayerShape> shapes;
-    for (int l = 0; l < layers; l++) shapes.push_back({kv_heads, head_dim, false, l});
+    for (int l = 0; l < layers; l++) shapes.push_back({kv_heads, key_dim, value_dim, l});
     return kv_create_keys(ctx, layers, shapes.data(), type == TSB_F32 ? 4 : 2, page_tokens, num_pages, max_seqs, max_pages_per_seq, out);
+}
+
+// The tiles of a batch of unequal portions, uploaded behind the launches before it: launch(batch) with them, then freed.
+static int32_t with_tiles(tsb_ctx* ctx, cudaStream_t st, const std::vector<AttnTile>& small, const std::vector<AttnTile>& large, AttnBatch b,
+                          const std::function<cudaError_t(const AttnBatch&)>& launch) {
+    // a captured copy would read the list again at every replay, when it is gone
+    cudaStreamCaptureStatus capture = cudaStreamCaptureStatusNone;
+    TSB_CUDA(ctx, cudaStreamIsCapturing(st, &capture));
+    if (capture != cudaStreamCaptureStatusNone) return tsb_fail(ctx, TSB_ERR_UNSUPPORTED, "portions of unequal length cannot be captured in a graph");
+    std::vector<AttnTile> all = small;
+    all.insert(all.end(), large.begin(), large.end());
+    AttnTile* dev = nullptr;
+    TSB_CUDA(ctx, cudaMallocAsync((void**)&dev, all.size() * sizeof(AttnTile), st));
+    cudaError_t e = cudaMemcpyAsync(dev, all.data(), all.size() * sizeof(AttnTile), cudaMemcpyHostToDevice, st);
+    b.n_small = (int)small.size(), b.n_large = (int)large.size(), b.small = dev, b.large = dev + b.n_small;
+    if (e == cudaSuccess) e = launch(b);
+    cudaError_t e2 = cudaFreeAsync(dev, st);
+    TSB_CUDA(ctx, e);
+    TSB_CUDA(ctx, e2);
+    return TSB_OK;
 }
 
 int32_t tsb_window_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, int32_t layer, const void* q, int64_t q_stride, void* out, int64_t out_stride,
                              const tsb_row_desc* rows_dev, const int32_t* group_rows, int32_t n_groups, int32_t n_q_heads, float scale, float cap,
                              const float* r1, const float* r2, const float* gate, int32_t window, int32_t max_len, void* scratch) {
+    tsb_attention_extras x{};
+    x.cap = cap, x.r1 = r1, x.r2 = r2, x.head_gate = gate, x.window = window;
+    return tsb_plain_attention(ctx, s, keys, layer, q, q_stride, out, out_stride, rows_dev, group_rows, n_groups, n_q_heads, scale, &x, max_len, scratch);
+}
+
+int32_t tsb_plain_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, int32_t layer, const void* q, int64_t q_stride, void* out, int64_t out_stride,
+                            const tsb_row_desc* rows_dev, const int32_t* group_rows, int32_t n_groups, int32_t n_q_heads, float scale,
+                            const tsb_attention_extras* extras, int32_t max_len, void* scratch) {
     if (!ctx || !keys) return TSB_ERR_INVALID;
-    TSB_REQUIRE(ctx, !keys->key_layers.empty() && layer >= 0 && layer < (int)keys->key_layers.size(), "a key-only cache and one of its layers expected");
-    TSB_REQUIRE(ctx, q && out && rows_dev && group_rows && n_groups > 0 && scratch && (r1 == nullptr) == (r2 == nullptr) && window >= 0, "bad arguments");
+    const tsb_attention_extras x = extras ? *extras : tsb_attention_extras{};
+    TSB_REQUIRE(ctx, !keys->key_layers.empty() && layer >= 0 && layer < (int)keys->key_layers.size(), "a plain cache and one of its layers expected");
+    TSB_REQUIRE(ctx, q && out && rows_dev && group_rows && n_groups > 0 && scratch && (x.r1 == nullptr) == (x.r2 == nullptr) && x.window >= 0, "bad arguments");
     const KeyView& kv = keys->key_layers[layer];
-    TSB_REQUIRE(ctx, n_q_heads > 0 && n_q_heads % kv.kv_heads == 0 && wattn_supported(kv.head_dim, n_q_heads / kv.kv_heads, kv.elem_bytes == 4),
-                "query heads must be a multiple of the key heads, at most %d per key head", WATTN_LARGE_Q);
+    const bool f32 = kv.elem_bytes == 4;
+    const int vd = kv.value_off ? kv.head_step - kv.value_off : kv.head_dim;
+    const bool wide = vd != kv.head_dim;  // keys and values of different widths: the many-query kernel alone takes them
+    const int grp = n_q_heads / kv.kv_heads;
+    TSB_REQUIRE(ctx, n_q_heads > 0 && n_q_heads % kv.kv_heads == 0 && (f32 ? kv.head_dim <= 1024 && vd <= 512 : wide ? grp == 1 && wattn_wide_supported(kv.head_dim, vd) && !x.r1
+                     : wattn_supported(kv.head_dim, grp, false) && wattn_pad_dim(kv.head_dim, false) == kv.head_dim),
+                "query heads must be a multiple of the key heads, at most %d per key head, and the head size one the kernels take", WATTN_LARGE_Q);
     TSB_REQUIRE(ctx, (uintptr_t)q % 32 == 0 && (uintptr_t)out % 32 == 0 && q_stride % 16 == 0 && out_stride % 16 == 0 &&
-                         q_stride >= (int64_t)n_q_heads * kv.head_dim && out_stride >= (int64_t)n_q_heads * kv.head_dim,
+                         q_stride >= (int64_t)n_q_heads * kv.head_dim && out_stride >= (int64_t)n_q_heads * vd,
                 "q and out rows hold every head and start on 32-byte boundaries (strides a multiple of 16)");
+    TSB_REQUIRE(ctx, !x.value_gate || ((uintptr_t)x.value_gate % 32 == 0 && x.value_gate_stride % 16 == 0 && x.value_gate_stride >= (int64_t)n_q_heads * vd),
+                "rows of value gates hold every head and start on 32-byte boundaries");
     cudaStream_t st = (cudaStream_t)s;
     DeviceGuard g(ctx);
     WindowAttn a;
-    a.keys = kv, a.q = q, a.q_stride = q_stride, a.out = out, a.out_stride = out_stride, a.gate = gate, a.rows = rows_dev;
-    a.n_q_heads = n_q_heads, a.scale = scale, a.cap = cap, a.r1 = r1, a.r2 = r2, a.window = window;
+    a.keys = kv, a.q = q, a.q_stride = q_stride, a.out = out, a.out_stride = out_stride, a.gate = x.head_gate, a.rows = rows_dev;
+    a.n_q_heads = n_q_heads, a.scale = scale, a.cap = x.cap, a.r1 = x.r1, a.r2 = x.r2, a.window = x.window;
+    a.sink = x.sink, a.value_gate = x.value_gate, a.value_gate_stride = x.value_gate_stride, a.value_dim = vd;
     AttnBatch b;
     b.max_len = max_len;
     bool uniform = true;
@@ -1061,31 +1105,117 @@ int32_t tsb_window_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, int32_t l
         b.rows += group_rows[i];
         uniform &= group_rows[i] == group_rows[0];
     }
-    if (uniform) {
-        b.rows_per_seq = group_rows[0];
-        TSB_CUDA(ctx, launch_window_attn(ctx, st, kv.elem_bytes == 4, a, b, scratch));
+    if (f32 || uniform) {
+        if (uniform) b.rows_per_seq = group_rows[0];
+        TSB_CUDA(ctx, wide && !f32 ? launch_window_attn_wide(ctx, st, a, b, scratch) : launch_window_attn(ctx, st, f32, a, b, scratch));
         return TSB_OK;
     }
-    const int grp = n_q_heads / kv.kv_heads, rpt = wattn_rows_per_tile(kv.head_dim, grp, r1 != nullptr);
+    const int rpt = wide ? WATTN_WIDE_ROWS : wattn_rows_per_tile(kv.head_dim, grp, x.r1 != nullptr);
     std::vector<AttnTile> small, large;
     for (int i = 0, r = 0; i < n_groups; r += group_rows[i], i++) {
-        if (group_rows[i] * grp <= WATTN_SMALL_Q) {
+        if (!wide && group_rows[i] * grp <= WATTN_SMALL_Q) {
             small.push_back({r, group_rows[i]});
             b.small_queries = std::max(b.small_queries, group_rows[i] * grp);
         } else {
             for (int k = 0; k < group_rows[i]; k += rpt) large.push_back({r + k, std::min(rpt, group_rows[i] - k)});
         }
     }
-    b.n_small = (int)small.size(), b.n_large = (int)large.size();
-    small.insert(small.end(), large.begin(), large.end());
-    AttnTile* dev = nullptr;
-    TSB_CUDA(ctx, cudaMallocAsync((void**)&dev, small.size() * sizeof(AttnTile), st));
-    cudaError_t e = cudaMemcpyAsync(dev, small.data(), small.size() * sizeof(AttnTile), cudaMemcpyHostToDevice, st);
-    b.small = dev, b.large = dev + b.n_small;
-    if (e == cudaSuccess) e = launch_window_attn(ctx, st, kv.elem_bytes == 4, a, b, scratch);
-    cudaError_t e2 = cudaFreeAsync(dev, st);
-    TSB_CUDA(ctx, e);
-    TSB_CUDA(ctx, e2);
+    return with_tiles(ctx, st, small, large, b, [&](const AttnBatch& t) {
+        return wide ? launch_window_attn_wide(ctx, st, a, t, scratch) : launch_window_attn(ctx, st, false, a, t, scratch);
+    });
+}
+
+int32_t tsb_latent_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* cache, int32_t layer, const void* q, int64_t q_stride, void* out, int64_t out_stride,
+                             const tsb_row_desc* rows_dev, const int32_t* group_rows, int32_t n_groups, int32_t n_heads, int32_t value_dim, float scale,
+                             const float* sink, int32_t max_len, void* scratch) {
+    if (!ctx || !cache) return TSB_ERR_INVALID;
+    TSB_REQUIRE(ctx, !cache->key_layers.empty() && layer >= 0 && layer < (int)cache->key_layers.size(), "a plain cache and one of its layers expected");
+    const KeyView& kv = cache->key_layers[layer];
+    int key_pad = 0, value_pad = 0;
+    TSB_REQUIRE(ctx, q && out && rows_dev && group_rows && n_groups > 0 && scratch && n_heads > 0 && kv.kv_heads == 1 && kv.value_off == 0, "bad arguments");
+    TSB_REQUIRE(ctx, latent_attn_dims(value_dim, kv.head_dim - value_dim, &key_pad, &value_pad) && value_pad == value_dim && key_pad == kv.head_dim,
+                "a row of %d numbers, the first %d of them the value, is not one the kernels work on", kv.head_dim, value_dim);
+    TSB_REQUIRE(ctx, (uintptr_t)q % 32 == 0 && (uintptr_t)out % 32 == 0 && q_stride % 16 == 0 && out_stride % 16 == 0 &&
+                         q_stride >= (int64_t)n_heads * kv.head_dim && out_stride >= (int64_t)n_heads * value_dim,
+                "q and out rows hold every head and start on 32-byte boundaries (strides a multiple of 16)");
+    cudaStream_t st = (cudaStream_t)s;
+    DeviceGuard g(ctx);
+    AttnBatch b;
+    b.max_len = max_len;
+    int most = 0;
+    bool uniform = true;
+    for (int i = 0; i < n_groups; i++) {
+        TSB_REQUIRE(ctx, group_rows[i] > 0, "every stream of the batch has rows");
+        b.rows += group_rows[i], most = std::max(most, group_rows[i]);
+        uniform &= group_rows[i] == group_rows[0];
+    }
+    if (kv.elem_bytes == 4) {
+        WindowAttn a;
+        a.keys = kv, a.q = q, a.q_stride = q_stride, a.out = out, a.out_stride = out_stride, a.rows = rows_dev, a.n_q_heads = n_heads, a.scale = scale;
+        a.sink = sink, a.value_dim = value_dim;
+        TSB_CUDA(ctx, launch_window_attn(ctx, st, true, a, b, scratch));
+        return TSB_OK;
+    }
+    LatentAttn a;
+    a.keys = kv, a.q = q, a.q_stride = q_stride, a.out = out, a.out_stride = out_stride, a.rows = rows_dev, a.n_heads = n_heads, a.value_dim = value_dim;
+    a.scale = scale, a.sink = sink;
+    if (uniform) {
+        b.rows_per_seq = most;
+        TSB_CUDA(ctx, launch_latent_attn(ctx, st, a, b, most, scratch));
+        return TSB_OK;
+    }
+    const int rpt = latent_attn_tiling(n_heads, value_dim, most).rows;
+    std::vector<AttnTile> tiles;
+    for (int i = 0, r = 0; i < n_groups; r += group_rows[i], i++)
+        for (int k = 0; k < group_rows[i]; k += rpt) tiles.push_back({r + k, std::min(rpt, group_rows[i] - k)});
+    return with_tiles(ctx, st, tiles, {}, b, [&](const AttnBatch& t) { return launch_latent_attn(ctx, st, a, t, most, scratch); });
+}
+
+int32_t tsb_plain_gemm_heads(tsb_ctx* ctx, tsb_stream s, int32_t type, const void* w, int32_t heads, int32_t head_rows, int64_t cols, const void* x,
+                             int64_t x_stride, int32_t x_step, int32_t x_rows, int32_t tokens, void* y, int64_t y_stride, int32_t y_step, int32_t n_valid,
+                             const void* gate, int64_t gate_stride, int32_t gate_step, void* workspace) {
+    if (!ctx) return TSB_ERR_INVALID;
+    int32_t rc = check_gemm(ctx, type, w, (int64_t)heads * head_rows, cols, x, x_rows, tokens, workspace);
+    if (rc) return rc;
+    TSB_REQUIRE(ctx, heads > 0 && head_rows % PLAIN_ROW_PAD == 0 && x_step % PLAIN_COL_PAD == 0 && (heads - 1) * (int64_t)x_step + cols <= x_stride && x_stride % 8 == 0,
+                "a head's rows are a multiple of %d, its columns start at multiples of %d inside the row", PLAIN_ROW_PAD, PLAIN_COL_PAD);
+    TSB_REQUIRE(ctx, y && n_valid > 0 && n_valid <= head_rows && (heads - 1) * (int64_t)y_step + n_valid <= y_stride, "bad output");
+    DeviceGuard g(ctx);
+    PlainEpi e;
+    e.kind = PLAIN_MIXER, e.n_seg = 1;
+    PlainSeg& k = e.seg[0];
+    k.end = heads * head_rows, k.per = head_rows, k.valid = n_valid, k.step = y_step, k.p = y, k.stride = y_stride;
+    k.gate = gate, k.gate_stride = gate_stride, k.gate_step = gate_step;
+    PlainMat m{const_cast<void*>(w), (int64_t)heads * head_rows, cols};
+    m.group_rows = head_rows, m.group_cols = x_step;
+    TSB_CUDA(ctx, launch_plain_gemm(ctx, (cudaStream_t)s, type == TSB_F32, m, x, nullptr, x_stride, x_rows, tokens, e, workspace));
+    return TSB_OK;
+}
+
+int32_t tsb_post_norm_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, float* x, int32_t d, const float* weight, float eps, int32_t rows, void* out,
+                           int64_t out_stride) {
+    if (!ctx) return TSB_ERR_INVALID;
+    TSB_REQUIRE(ctx, x && weight && out && d > 0 && rows > 0 && out_stride >= d && (type == TSB_BF16 || type == TSB_F32), "bad arguments");
+    TSB_REQUIRE(ctx, (uintptr_t)x % 16 == 0 && (uintptr_t)weight % 16 == 0 && (uintptr_t)out % 16 == 0, "buffers must be 16-byte aligned");
+    DeviceGuard g(ctx);
+    TSB_CUDA(ctx, launch_post_norm(ctx, (cudaStream_t)s, type == TSB_F32, x, d, weight, eps, rows, out, out_stride));
+    return TSB_OK;
+}
+
+int32_t tsb_head_norm_rows(tsb_ctx* ctx, tsb_stream s, tsb_kv* cache, int32_t layer, const float* raw, int64_t raw_stride, int32_t n_q, int32_t n_k, int32_t width,
+                           const float* q_weight, const float* k_weight, float eps, float temp_coef, int32_t temp_every, const tsb_row_desc* rows_dev,
+                           int32_t rows, void* q, int64_t q_stride) {
+    if (!ctx || !cache) return TSB_ERR_INVALID;
+    TSB_REQUIRE(ctx, !cache->key_layers.empty() && layer >= 0 && layer < (int)cache->key_layers.size(), "a plain cache and one of its layers expected");
+    const KeyView& kv = cache->key_layers[layer];
+    TSB_REQUIRE(ctx, raw && rows_dev && rows > 0 && n_q >= 0 && n_k >= 0 && n_k <= kv.kv_heads && n_q + n_k > 0 && width > 0 && width <= kv.head_dim &&
+                         raw_stride >= (int64_t)(n_q + n_k) * width && (n_q == 0 || (q && q_weight && q_stride >= (int64_t)n_q * kv.head_dim)) &&
+                         (n_k == 0 || k_weight) && temp_every >= 0, "bad arguments");
+    DeviceGuard g(ctx);
+    HeadNorms h;
+    h.raw = raw, h.raw_stride = raw_stride, h.n_q = n_q, h.n_k = n_k, h.width = width, h.q_weight = q_weight, h.k_weight = k_weight, h.eps = eps;
+    h.temp_coef = temp_coef, h.temp_every = temp_every, h.q = q, h.q_stride = q_stride, h.q_step = h.q_width = kv.head_dim, h.keys = kv, h.rows = rows_dev;
+    TSB_CUDA(ctx, launch_head_norms(ctx, (cudaStream_t)s, kv.elem_bytes == 4, h, rows));
     return TSB_OK;
 }
 

@@ -38,11 +38,11 @@ struct PlainLayer {
     }
 };
 
-// Frequencies of one kind of rotary position, f32 on the device.
+// Frequencies of one kind of rotary position.
 struct PlainRotation {
     int dims = 0;
     double base = 0, factor = 0, original = 0, fast = 0, slow = 0;
-    float* freq = nullptr;     // [dims / 2]
+    double* freq = nullptr;    // device, [dims / 2]
     float magnitude = 1.f;
 };
 

@@ -257,14 +257,17 @@ __global__ void __launch_bounds__(ROW_THREADS) head_norms_kernel(const __grid_co
 }
 
 __global__ void __launch_bounds__(ROW_THREADS)
-    rotary_table_kernel(const float* __restrict__ freq, int half, float magnitude, const tsb_row_desc* __restrict__ rows, int n, float2* table) {
+    rotary_table_kernel(const double* __restrict__ freq, int half, float magnitude, const tsb_row_desc* __restrict__ rows, int n, float2* table) {
     pdl_wait();
     pdl_launch_dependents();
     const int64_t k = (int64_t)blockIdx.x * ROW_THREADS + threadIdx.x;
     if (k >= (int64_t)n * half) return;
     const tsb_row_desc& rd = rows[k / half];
+    constexpr double TURN = 6.283185307179586476925;
+    double a = (double)(rd.base + rd.slot) * freq[k % half];
+    a -= TURN * rint(a * (1.0 / TURN));
     float s, c;
-    sincosf((float)(rd.base + rd.slot) * freq[k % half], &s, &c);
+    sincosf((float)a, &s, &c);
     table[k] = make_float2(magnitude * c, magnitude * s);
 }
 
@@ -349,7 +352,7 @@ cudaError_t launch_head_norms(tsb_ctx* ctx, cudaStream_t st, bool f32, const Hea
     return tsb_launch(ctx, f32 ? head_norms_kernel<float> : head_norms_kernel<__nv_bfloat16>, grid, dim3(ROW_THREADS), 0, st, true, h, rows, ctx->dev_error);
 }
 
-cudaError_t launch_rotary_table(tsb_ctx* ctx, cudaStream_t st, const float* freq, int half, float magnitude, const tsb_row_desc* rows_dev, int rows,
+cudaError_t launch_rotary_table(tsb_ctx* ctx, cudaStream_t st, const double* freq, int half, float magnitude, const tsb_row_desc* rows_dev, int rows,
                                 float2* table) {
     return tsb_launch(ctx, rotary_table_kernel, dim3((unsigned)(((int64_t)rows * half + ROW_THREADS - 1) / ROW_THREADS)), dim3(ROW_THREADS), 0, st, true, freq,
                       half, magnitude, rows_dev, rows, table);

@@ -51,8 +51,8 @@ struct HeadNorms {
 };
 cudaError_t launch_head_norms(tsb_ctx* ctx, cudaStream_t st, bool f32, const HeadNorms& h, int rows);
 
-// table[r, i] = magnitude * (cos, sin)(position of row r * freq[i]), i below half
-cudaError_t launch_rotary_table(tsb_ctx* ctx, cudaStream_t st, const float* freq, int half, float magnitude, const tsb_row_desc* rows_dev, int rows,
+// table[r, i] = magnitude * (cos, sin)(position of row r * freq[i]), i below half; the product is reduced to one turn in double
+cudaError_t launch_rotary_table(tsb_ctx* ctx, cudaStream_t st, const double* freq, int half, float magnitude, const tsb_row_desc* rows_dev, int rows,
                                 float2* table);
 
 // Cached latent rows of whole streams, for their expansion to keys and values (bfloat16).  Stream i of the list (first row of
