@@ -1,12 +1,16 @@
 // Attention over latent rows (attention_latent.cuh), bfloat16, mma.sync m16n8k16.
 //
-// A CTA owns a query tile - 16 MT (row, head) pairs of one stream - and a run of 64-token key tiles, which cp.async brings into a
-// ring of row-padded stages.  One tile in shared memory serves both products.  Eight warps:
-//   scores   MT warps share a group of 8 MT keys, each with sixteen of the queries; all of them walk the whole key width
-//   softmax  row maxima of the key groups meet in shared memory; every warp keeps the running maximum of every query
-//   output   every warp owns DV / 8 value columns of all queries; the weights come from shared memory
-// so the accumulators of a 512-column value fit in registers and a key byte is read from memory once.  Key tiles start at
-// multiples of 64 positions.  A context that does not fill the device with CTAs is cut into runs; a merge launch adds them in order.
+// A CTA owns a query tile - 16 MT (row, head) pairs of one stream - and a run of 64-token key tiles, which one warp fetches row by
+// row with bulk copies into a ring of stages.  One tile in shared memory serves both products, and a key byte is read from memory
+// once.  Eight warps:
+//   scores   KS warps split the key columns, 8 / KS groups of them the keys; a warp's part of every query stays in registers, so this
+//            product reads each key fragment once and nothing else.  The parts meet in shared memory.
+//   softmax  256 / (16 MT) threads per query add the parts, mask, keep the running maximum and sum, leave the weights (bfloat16)
+//            and the factor of the earlier sums
+//   output   every warp owns DV / 8 value columns of all queries
+// so the accumulators of a 512-column value fit in registers.  Key tiles start at multiples of 64 positions.  A context that does
+// not fill the device with CTAs is cut into runs; a merge launch adds them in order.
+// Waits for copies are bounded; when one runs out the launch is marked failed, the CTA waits for what it has in flight and returns.
 #include <algorithm>
 
 #include "attention_latent.cuh"
@@ -16,7 +20,9 @@ namespace {
 
 constexpr int LT_TOK = 64, LT_WARPS = 8, LT_THREADS = LT_WARPS * 32;
 constexpr int LT_SMEM_CAP = 227 * 1024;
-constexpr int LT_P_PITCH = LT_TOK * 2 + 16;
+constexpr int LT_P_PITCH = LT_TOK * 2 + 16;    // bytes
+constexpr int LT_S_PITCH = LT_TOK + 8;         // floats
+constexpr int LT_HEADER = 128;                 // barriers
 
 __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
@@ -32,30 +38,36 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], 
         : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
         : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool valid) {
-    const int n = valid ? 16 : 0;
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
-}
 
-__host__ __device__ constexpr int lt_pitch(int key_dim) { return key_dim * 2 + 16; }  // key_dim a multiple of 32: eight rows of a chunk meet all banks
-template <int DV>
-constexpr int lt_stages() { return DV > 256 ? 2 : 3; }
-template <int DV, int MT>
-size_t lt_smem(int key_dim) {
-    return (size_t)(lt_stages<DV>() * LT_TOK + 16 * MT) * lt_pitch(key_dim) + 16 * MT * (LT_P_PITCH + LT_WARPS * 4);
-}
-constexpr int lt_per_sm(int dv, int mt) { return dv <= 128 ? 2 : dv <= 256 && mt <= 2 ? 2 : 1; }
+// DV value columns, key columns in KW blocks of 64, MT query tiles of sixteen.
+template <int DV, int KW, int MT>
+struct LtGeo {
+    static constexpr int KS = DV > 128 ? 4 : 2, GROUPS = LT_WARPS / KS, KEYS = LT_TOK / GROUPS;  // keys of a warp's scores
+    static constexpr int STEPS = KW * 4 / KS;                                                  // sixteen-column steps of a warp's part
+    static constexpr int PITCH = KW * 128 + 16;  // bytes of a key row: eight rows of a chunk meet all banks
+    static constexpr int STAGES = DV > 256 ? 2 : 3, STAGE = LT_TOK * PITCH, QT = 16 * MT;
+    static constexpr size_t SMEM = (size_t)LT_HEADER + STAGES * STAGE + (size_t)KS * QT * LT_S_PITCH * 4 + QT * (LT_P_PITCH + 8);
+    static constexpr int PER_SM = DV <= 128 ? 2 : 1;
+};
 
-template <int DV, int MT>
-__global__ void __launch_bounds__(LT_THREADS, lt_per_sm(DV, MT))
+template <int DV, int KW, int MT>
+__global__ void __launch_bounds__(LT_THREADS, LtGeo<DV, KW, MT>::PER_SM)
     latent_attn_kernel(const __grid_constant__ LatentAttn a, const AttnTile* __restrict__ tiles, int tiles_per_group, int rows_per_seq, int rows_per_tile,
                        int heads_per_tile, float* __restrict__ part_o, float2* __restrict__ part_ml, uint32_t* __restrict__ err) {
-    constexpr int QT = 16 * MT, NG = LT_WARPS / MT, NK = MT, NST = lt_stages<DV>();  // key groups; n-tiles of eight keys per warp
-    constexpr int ND = DV / 64;                                                      // n-tiles of eight value columns per warp
+    using G = LtGeo<DV, KW, MT>;
+    constexpr int QT = G::QT, NST = G::STAGES, KS = G::KS, NT = G::KEYS / 8;
+    constexpr int ND = DV / 64;                                       // n-tiles of eight value columns per warp
+    constexpr int TPQ = LT_THREADS / QT, PER = LT_TOK / TPQ;            // threads per query, scores per thread
     extern __shared__ __align__(128) uint8_t smem[];
+    uint64_t* full = reinterpret_cast<uint64_t*>(smem);
+    uint8_t* ring = smem + LT_HEADER;
+    float* parts = reinterpret_cast<float*>(ring + NST * G::STAGE);                   // [KS][QT][LT_S_PITCH]
+    uint8_t* p_tile = reinterpret_cast<uint8_t*>(parts + KS * QT * LT_S_PITCH);       // [QT], bfloat16
+    float* alphas = reinterpret_cast<float*>(p_tile + QT * LT_P_PITCH);               // [QT]; the sums at the end
+    float* maxima = alphas + QT;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
-    const int mt = warp % MT, kg = warp / MT;
-    const int n_splits = gridDim.x, DK = a.keys.head_dim, pitch = lt_pitch(DK);
+    const int kq = warp % KS, kg = warp / KS;
+    const int n_splits = gridDim.x, DK = a.keys.head_dim;
     int row_first, n_rows;
     if (tiles) {
         row_first = tiles[blockIdx.z].row_first, n_rows = tiles[blockIdx.z].n_rows;
@@ -68,7 +80,7 @@ __global__ void __launch_bounds__(LT_THREADS, lt_per_sm(DV, MT))
     const int seq = rd0.seq, pos0 = rd0.base + rd0.slot;
     const int head0 = blockIdx.y * heads_per_tile, heads = min(heads_per_tile, a.n_heads - head0);
     const int n_queries = n_rows * heads;
-    if (seq < 0 || seq >= a.keys.max_seqs || n_queries > QT) {
+    if (seq < 0 || seq >= a.keys.max_seqs || n_queries > QT || DK > KW * 64) {
         if (threadIdx.x == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
         pdl_wait();
         return;
@@ -77,150 +89,170 @@ __global__ void __launch_bounds__(LT_THREADS, lt_per_sm(DV, MT))
     const int total = (hi + LT_TOK - 1) / LT_TOK, per = (total + n_splits - 1) / n_splits;
     const int t_first = min(total, (int)blockIdx.x * per), n_tiles = min(total, t_first + per) - t_first;
     const int begin = t_first * LT_TOK;
+    const uint32_t ring_s = smem_u32(ring), p_smem = smem_u32(p_tile);
 
-    uint8_t* q_tile = smem + (size_t)NST * LT_TOK * pitch;
-    uint8_t* p_tile = q_tile + QT * pitch;
-    float* group_max = reinterpret_cast<float*>(p_tile + QT * LT_P_PITCH);  // [QT][NG]; the groups' sums at the end
-    const uint32_t ring = smem_u32(smem), q_smem = smem_u32(q_tile), p_smem = smem_u32(p_tile);
-
+    if (threadIdx.x == 0) {
+        for (int i = 0; i < NST; i++) mbar_init(&full[i], 1);
+        mbar_fence_init();
+    }
+    // columns behind the row's: finite, and the queries have zeros there
+    for (int i = threadIdx.x; i < NST * LT_TOK * (KW * 8 - DK / 8); i += LT_THREADS) {
+        const int r = i / (KW * 8 - DK / 8), c = DK / 8 + i % (KW * 8 - DK / 8);
+        *reinterpret_cast<uint4*>(ring + (size_t)r * G::PITCH + c * 16) = make_uint4(0, 0, 0, 0);
+    }
+    __syncthreads();
+    // warp 0: two rows a lane.  Positions past the end are masked later; their slots repeat the last row.
     auto issue = [&](int tile) {
-        if (tile < n_tiles) {
-            // four threads a token row
-            const int r = threadIdx.x >> 2, pos = begin + tile * LT_TOK + r;
-            const __nv_bfloat16* src = pos < hi ? key_row<__nv_bfloat16>(a.keys, seq, pos) : nullptr;
-            const bool ok = src != nullptr;
-            if (!ok) src = reinterpret_cast<const __nv_bfloat16*>(a.keys.base);
-            const uint32_t dst = ring + (tile % NST) * LT_TOK * pitch + r * pitch;
-            for (int c = threadIdx.x & 3; c < DK / 8; c += 4) cp16(dst + c * 16, ok ? src + c * 8 : src, ok);
+        if (tile >= n_tiles) return;
+        uint64_t* bar = &full[tile % NST];
+        if (lane == 0) mbar_expect_tx(bar, (uint32_t)(LT_TOK * DK * 2));
+        __syncwarp();
+#pragma unroll
+        for (int i = 0; i < 2; i++) {
+            const int r = lane + 32 * i, pos = min(begin + tile * LT_TOK + r, hi - 1);
+            const __nv_bfloat16* src = key_row<__nv_bfloat16>(a.keys, seq, pos);
+            if (!src) {  // not a reserved position: flagged; the copy keeps its byte count
+                atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+                src = reinterpret_cast<const __nv_bfloat16*>(a.keys.base);
+            }
+            bulk_g2s(ring + (size_t)((tile % NST) * LT_TOK + r) * G::PITCH, src, (uint32_t)(DK * 2), bar);
         }
-        cp_async_commit();
     };
     const bool early = begin + (NST - 1) * LT_TOK <= rd0.base;  // keys of earlier passes
-    if (early) {
+    if (early && warp == 0) {
 #pragma unroll
         for (int i = 0; i < NST - 1; i++) issue(i);
     }
     pdl_wait();
-    if (!early) {
+    if (!early && warp == 0) {
 #pragma unroll
         for (int i = 0; i < NST - 1; i++) issue(i);
     }
-    for (int i = threadIdx.x; i < QT * (DK / 8); i += LT_THREADS) {
-        const int qi = i / (DK / 8), c = i % (DK / 8);
-        uint4 v = make_uint4(0, 0, 0, 0);
-        if (qi < n_queries)
-            v = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(a.q) + (int64_t)(row_first + qi / heads) * a.q_stride +
-                                                (int64_t)(head0 + qi % heads) * DK + c * 8);
-        *reinterpret_cast<uint4*>(q_tile + qi * pitch + c * 16) = v;
-    }
-    // positions of the lane's two score rows; empty slots repeat the first query and are not stored
-    int pq[2];
-#pragma unroll
-    for (int h = 0; h < 2; h++) {
-        const int qi = mt * 16 + gid + 8 * h;
-        pq[h] = pos0 + (qi < n_queries ? qi / heads : 0);
-    }
-    const float scale2 = a.scale * 1.4426950408889634f;
-    float o[MT][ND][4];
-    float m_run[MT][2], l_run[2] = {0.f, 0.f};
+    // this warp's part of the queries
+    uint32_t qf[MT][G::STEPS][4];
 #pragma unroll
     for (int m = 0; m < MT; m++) {
-        m_run[m][0] = m_run[m][1] = -INFINITY;
+        const uint32_t* qp[2];
+#pragma unroll
+        for (int h = 0; h < 2; h++) {
+            const int qi = m * 16 + gid + 8 * h;
+            qp[h] = qi < n_queries ? reinterpret_cast<const uint32_t*>(static_cast<const __nv_bfloat16*>(a.q) + (int64_t)(row_first + qi / heads) * a.q_stride +
+                                                                      (int64_t)(head0 + qi % heads) * DK)
+                                   : nullptr;
+        }
+#pragma unroll
+        for (int k = 0; k < G::STEPS; k++) {
+            const int c = (kq * G::STEPS + k) * 16;
+#pragma unroll
+            for (int i = 0; i < 4; i++) qf[m][k][i] = qp[i & 1] && c < DK ? qp[i & 1][c / 2 + (i >> 1) * 4 + tig] : 0u;
+        }
+    }
+    // the thread's query of the softmax
+    const int sq = threadIdx.x / TPQ, sj = threadIdx.x % TPQ;
+    const int pq = pos0 + (sq < n_queries ? sq / heads : 0);  // an empty slot repeats the first query and is not stored
+    const float scale2 = a.scale * 1.4426950408889634f;
+    float m_run = -INFINITY, l_run = 0.f;
+    float o[MT][ND][4];
+#pragma unroll
+    for (int m = 0; m < MT; m++)
 #pragma unroll
         for (int n = 0; n < ND; n++)
 #pragma unroll
             for (int i = 0; i < 4; i++) o[m][n][i] = 0.f;
-    }
     const int col0 = warp * (DV / LT_WARPS);
+    bool ok = true;
 
     for (int tile = 0; tile < n_tiles; tile++) {
-        cp_async_wait<NST - 2>();
-        __syncthreads();  // the tile is here, and every warp is done with the stage and the weights of the one before
-        issue(tile + NST - 1);
-        const uint32_t kt = ring + (tile % NST) * LT_TOK * pitch;
-        const int key0 = kg * 8 * NK;
-        float s[NK][4], s2[NK][4];
+        // the tile is here, and every warp is done with the stage and the weights of the one before
+        ok = __syncthreads_and(mbar_wait(&full[tile % NST], (tile / NST) & 1, err));
+        if (!ok) break;
+        if (warp == 0) issue(tile + NST - 1);
+        const uint32_t kt = ring_s + (tile % NST) * G::STAGE;
+        float s[MT][NT][4];
 #pragma unroll
-        for (int n = 0; n < NK; n++)
+        for (int m = 0; m < MT; m++)
 #pragma unroll
-            for (int i = 0; i < 4; i++) s[n][i] = 0.f, s2[n][i] = 0.f;
-        const uint32_t qa = q_smem + (mt * 16 + (lane & 15)) * pitch + (lane >> 4) * 16;
-        const uint32_t ka = kt + (key0 + (lane & 7)) * pitch + (lane >> 3) * 16;
-#pragma unroll 2
-        for (int kp = 0; kp < DK / 32; kp++) {
-            uint32_t a0[4], a1[4];
-            ldsm4(a0, qa + kp * 64);
-            ldsm4(a1, qa + kp * 64 + 32);
+            for (int n = 0; n < NT; n++)
 #pragma unroll
-            for (int n = 0; n < NK; n++) {
+                for (int i = 0; i < 4; i++) s[m][n][i] = 0.f;
+        const uint32_t ka = kt + (kg * G::KEYS + (lane & 7) + ((lane >> 4) << 3)) * G::PITCH + kq * G::STEPS * 32 + ((lane >> 3) & 1) * 16;
+#pragma unroll
+        for (int k = 0; k < G::STEPS; k++) {
+#pragma unroll
+            for (int n = 0; n < NT; n += 2) {
                 uint32_t b[4];
-                ldsm4(b, ka + n * 8 * pitch + kp * 64);
-                mma_bf16(s[n], a0, b[0], b[1]);
-                mma_bf16(s2[n], a1, b[2], b[3]);
+                ldsm4(b, ka + n * 8 * G::PITCH + k * 32);
+#pragma unroll
+                for (int m = 0; m < MT; m++) {
+                    mma_bf16(s[m][n], qf[m][k], b[0], b[1]);
+                    mma_bf16(s[m][n + 1], qf[m][k], b[2], b[3]);
+                }
             }
         }
-        const int p0 = begin + tile * LT_TOK;
-        const bool edge = p0 + LT_TOK > pos0 + 1;
-        float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
-        for (int n = 0; n < NK; n++)
+        for (int m = 0; m < MT; m++)
 #pragma unroll
-            for (int i = 0; i < 4; i++) {
-                float v = (s[n][i] + s2[n][i]) * scale2;
-                if (edge && p0 + key0 + n * 8 + 2 * tig + (i & 1) > pq[i >> 1]) v = -INFINITY;
-                s[n][i] = v;
-                mx[i >> 1] = fmaxf(mx[i >> 1], v);
+            for (int n = 0; n < NT; n++) {
+                float* d = parts + (kq * QT + m * 16 + gid) * LT_S_PITCH + kg * G::KEYS + n * 8 + 2 * tig;
+                *reinterpret_cast<float2*>(d) = make_float2(s[m][n][0], s[m][n][1]);
+                *reinterpret_cast<float2*>(d + 8 * LT_S_PITCH) = make_float2(s[m][n][2], s[m][n][3]);
+            }
+        __syncthreads();
+        {
+            const int p0 = begin + tile * LT_TOK;
+            float v[PER];
+            float mx = -INFINITY;
+#pragma unroll
+            for (int c = 0; c < PER; c += 4) {
+                const int col = (c / 4 * TPQ + sj) * 4;
+                float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+                for (int k = 0; k < KS; k++) {
+                    const float4 y = *reinterpret_cast<const float4*>(parts + (k * QT + sq) * LT_S_PITCH + col);
+                    x.x += y.x, x.y += y.y, x.z += y.z, x.w += y.w;
+                }
+                const float xs[4] = {x.x, x.y, x.z, x.w};
+#pragma unroll
+                for (int i = 0; i < 4; i++) {
+                    v[c + i] = p0 + col + i <= pq ? xs[i] * scale2 : -INFINITY;
+                    mx = fmaxf(mx, v[c + i]);
+                }
             }
 #pragma unroll
-        for (int h = 0; h < 2; h++) {
-            mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 1));
-            mx[h] = fmaxf(mx[h], __shfl_xor_sync(0xffffffffu, mx[h], 2));
-            if (tig == 0) group_max[(mt * 16 + gid + 8 * h) * NG + kg] = mx[h];
+            for (int d = TPQ / 2; d > 0; d >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, d));
+            const float m_new = fmaxf(m_run, mx), use = m_new == -INFINITY ? 0.f : m_new;
+            const float alpha = ex2(m_run - use);  // 0 while nothing was visible
+            m_run = m_new;
+            float sum = 0.f;
+#pragma unroll
+            for (int c = 0; c < PER; c += 4) {
+                const int col = (c / 4 * TPQ + sj) * 4;
+#pragma unroll
+                for (int i = 0; i < 4; i++) v[c + i] = ex2(v[c + i] - use), sum += v[c + i];
+                *reinterpret_cast<uint2*>(p_tile + sq * LT_P_PITCH + col * 2) = make_uint2(pack_bf16(v[c], v[c + 1]), pack_bf16(v[c + 2], v[c + 3]));
+            }
+            l_run = fmaf(l_run, alpha, sum);
+            if (sj == 0) alphas[sq] = alpha;
         }
         __syncthreads();
-        float alpha[MT][2], m_mine[2] = {0.f, 0.f};
+        float al[MT][2];
         bool moved = false;
 #pragma unroll
         for (int m = 0; m < MT; m++)
 #pragma unroll
-            for (int h = 0; h < 2; h++) {
-                const float* g = group_max + (m * 16 + gid + 8 * h) * NG;
-                float v = m_run[m][h];
-#pragma unroll
-                for (int k = 0; k < NG; k += 2) {
-                    const float2 x = *reinterpret_cast<const float2*>(g + k);
-                    v = fmaxf(v, fmaxf(x.x, x.y));
-                }
-                const float use = v == -INFINITY ? 0.f : v;
-                alpha[m][h] = ex2(m_run[m][h] - use);
-                moved |= m_run[m][h] != v;
-                m_run[m][h] = v;
-                if (m == mt) {
-                    m_mine[h] = use;
-                    l_run[h] *= alpha[m][h];
-                }
-            }
-#pragma unroll
-        for (int n = 0; n < NK; n++) {
-            const float e0 = ex2(s[n][0] - m_mine[0]), e1 = ex2(s[n][1] - m_mine[0]), e2 = ex2(s[n][2] - m_mine[1]), e3 = ex2(s[n][3] - m_mine[1]);
-            l_run[0] += e0 + e1, l_run[1] += e2 + e3;
-            const int c = (key0 + n * 8 + 2 * tig) * 2;
-            *reinterpret_cast<uint32_t*>(p_tile + (mt * 16 + gid) * LT_P_PITCH + c) = pack_bf16(e0, e1);
-            *reinterpret_cast<uint32_t*>(p_tile + (mt * 16 + gid + 8) * LT_P_PITCH + c) = pack_bf16(e2, e3);
-        }
+            for (int h = 0; h < 2; h++) al[m][h] = alphas[m * 16 + gid + 8 * h], moved |= al[m][h] != 1.f;
         if (__any_sync(0xffffffffu, moved)) {
 #pragma unroll
             for (int m = 0; m < MT; m++)
 #pragma unroll
-                for (int n = 0; n < ND; n++) o[m][n][0] *= alpha[m][0], o[m][n][1] *= alpha[m][0], o[m][n][2] *= alpha[m][1], o[m][n][3] *= alpha[m][1];
+                for (int n = 0; n < ND; n++) o[m][n][0] *= al[m][0], o[m][n][1] *= al[m][0], o[m][n][2] *= al[m][1], o[m][n][3] *= al[m][1];
         }
-        __syncthreads();
 #pragma unroll
         for (int kk = 0; kk < LT_TOK / 16; kk++) {
             uint32_t pa[MT][4];
 #pragma unroll
             for (int m = 0; m < MT; m++) ldsm4(pa[m], p_smem + (m * 16 + (lane & 15)) * LT_P_PITCH + kk * 32 + (lane >> 4) * 16);
-            const uint32_t va = kt + (kk * 16 + (lane & 15)) * pitch + col0 * 2;
+            const uint32_t va = kt + (kk * 16 + (lane & 15)) * G::PITCH + col0 * 2;
 #pragma unroll
             for (int np = 0; np < ND / 2; np++) {
                 uint32_t b[4];
@@ -239,16 +271,14 @@ __global__ void __launch_bounds__(LT_THREADS, lt_per_sm(DV, MT))
             }
         }
     }
-    cp_async_wait<0>();
+    // no copy is in flight when the CTA leaves
+    if (!ok && warp == 0)
+        for (int i = 0; i < NST; i++) mbar_wait(&full[i], 0u, err), mbar_wait(&full[i], 1u, err);
     pdl_launch_dependents();
-    // the key groups' sums meet
     __syncthreads();
 #pragma unroll
-    for (int h = 0; h < 2; h++) {
-        l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 1);
-        l_run[h] += __shfl_xor_sync(0xffffffffu, l_run[h], 2);
-        if (tig == 0) group_max[(mt * 16 + gid + 8 * h) * NG + kg] = l_run[h];
-    }
+    for (int d = TPQ / 2; d > 0; d >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, d);
+    if (sj == 0) alphas[sq] = l_run, maxima[sq] = m_run;
     __syncthreads();
     const int64_t tile_id = (int64_t)blockIdx.z * gridDim.y + blockIdx.y;
     const int64_t share = (tile_id * n_splits + blockIdx.x) * QT;
@@ -258,13 +288,10 @@ __global__ void __launch_bounds__(LT_THREADS, lt_per_sm(DV, MT))
         for (int h = 0; h < 2; h++) {
             const int qi = m * 16 + gid + 8 * h;
             if (qi >= n_queries) continue;
-            float l = 0.f;
-#pragma unroll
-            for (int k = 0; k < NG; k++) l += group_max[qi * NG + k];
+            const float l = alphas[qi], mx = maxima[qi];
             const int head = head0 + qi % heads;
             if (n_splits == 1) {
-                if (a.sink) l += ex2(a.sink[head] * 1.4426950408889634f - m_run[m][h]);
-                const float f = 1.f / l;
+                const float f = 1.f / (a.sink ? l + ex2(a.sink[head] * 1.4426950408889634f - mx) : l);
                 __nv_bfloat16* p = static_cast<__nv_bfloat16*>(a.out) + (int64_t)(row_first + qi / heads) * a.out_stride + (int64_t)head * DV + col0;
 #pragma unroll
                 for (int n = 0; n < ND; n++) *reinterpret_cast<uint32_t*>(p + n * 8 + 2 * tig) = pack_bf16(o[m][n][2 * h] * f, o[m][n][2 * h + 1] * f);
@@ -272,7 +299,7 @@ __global__ void __launch_bounds__(LT_THREADS, lt_per_sm(DV, MT))
                 float* p = part_o + (share + qi) * DV + col0;
 #pragma unroll
                 for (int n = 0; n < ND; n++) *reinterpret_cast<float2*>(p + n * 8 + 2 * tig) = make_float2(o[m][n][2 * h], o[m][n][2 * h + 1]);
-                if (warp == 0 && tig == 0) part_ml[share + qi] = make_float2(m_run[m][h], l);
+                if (warp == 0 && tig == 0) part_ml[share + qi] = make_float2(mx, l);
             }
         }
 }
@@ -329,28 +356,28 @@ __global__ void __launch_bounds__(128)
     }
 }
 
-template <int DV, int MT>
+template <int DV, int KW, int MT>
 cudaError_t launch_one(tsb_ctx* ctx, cudaStream_t st, const LatentAttn& a, const WattnLaunch& l, int heads_per_tile, void* scratch) {
+    using G = LtGeo<DV, KW, MT>;
     const int head_tiles = (a.n_heads + heads_per_tile - 1) / heads_per_tile, base = l.n_tiles * head_tiles;
-    const size_t smem = lt_smem<DV, MT>(a.keys.head_dim);
-    const int per_sm = std::min(lt_per_sm(DV, MT), std::max(1, (int)(LT_SMEM_CAP / (smem + 1024))));
-    const int splits = wattn_splits(ctx, 0, l, LT_TOK, 16 * MT, per_sm, base, std::min(wattn_part_queries(ctx), wattn_part_queries(ctx) * 256 / DV));
+    const int splits = wattn_splits(ctx, 0, l, LT_TOK, G::QT, G::PER_SM, base, std::min(wattn_part_queries(ctx), wattn_part_queries(ctx) * 256 / DV));
     const WattnScratch sc = wattn_scratch(ctx, scratch);
     static SmemOptIn configured;
-    if (cudaError_t e = tsb_opt_in_smem(ctx, latent_attn_kernel<DV, MT>, LT_SMEM_CAP, configured); e != cudaSuccess) return e;
-    cudaError_t e = tsb_launch(ctx, latent_attn_kernel<DV, MT>, dim3((unsigned)splits, (unsigned)head_tiles, (unsigned)l.n_tiles), dim3(LT_THREADS), smem, st,
-                               true, a, l.tiles, l.tiles_per_group, l.rows_per_seq, l.rows_per_tile, heads_per_tile, sc.o, sc.ml, ctx->dev_error);
+    static_assert(G::SMEM <= (size_t)LT_SMEM_CAP, "");
+    if (cudaError_t e = tsb_opt_in_smem(ctx, latent_attn_kernel<DV, KW, MT>, G::SMEM, configured); e != cudaSuccess) return e;
+    cudaError_t e = tsb_launch(ctx, latent_attn_kernel<DV, KW, MT>, dim3((unsigned)splits, (unsigned)head_tiles, (unsigned)l.n_tiles), dim3(LT_THREADS),
+                               G::SMEM, st, true, a, l.tiles, l.tiles_per_group, l.rows_per_seq, l.rows_per_tile, heads_per_tile, sc.o, sc.ml, ctx->dev_error);
     if (e == cudaSuccess && splits > 1)
-        e = tsb_launch(ctx, latent_merge_kernel, dim3(16 * MT, (unsigned)head_tiles, (unsigned)l.n_tiles), dim3(128), 0, st, true, a, l.tiles,
-                       l.tiles_per_group, l.rows_per_seq, l.rows_per_tile, heads_per_tile, splits, 16 * MT, (const float*)sc.o, (const float2*)sc.ml);
+        e = tsb_launch(ctx, latent_merge_kernel, dim3(G::QT, (unsigned)head_tiles, (unsigned)l.n_tiles), dim3(128), 0, st, true, a, l.tiles, l.tiles_per_group,
+                       l.rows_per_seq, l.rows_per_tile, heads_per_tile, splits, G::QT, (const float*)sc.o, (const float2*)sc.ml);
     return e;
 }
 template <int DV>
 cudaError_t launch_dim(tsb_ctx* ctx, cudaStream_t st, const LatentAttn& a, const WattnLaunch& l, const LatentTiling& t, void* scratch) {
-    if (t.queries == 16) return launch_one<DV, 1>(ctx, st, a, l, t.heads, scratch);
-    if (t.queries == 32) return launch_one<DV, 2>(ctx, st, a, l, t.heads, scratch);
-    if constexpr (DV <= 256) return launch_one<DV, 4>(ctx, st, a, l, t.heads, scratch);
-    return cudaErrorInvalidValue;
+    constexpr int KW = DV / 64 + 1;
+    if (a.keys.head_dim <= KW * 64)
+        return t.queries == 16 ? launch_one<DV, KW, 1>(ctx, st, a, l, t.heads, scratch) : launch_one<DV, KW, 2>(ctx, st, a, l, t.heads, scratch);
+    return t.queries == 16 ? launch_one<DV, KW + 1, 1>(ctx, st, a, l, t.heads, scratch) : launch_one<DV, KW + 1, 2>(ctx, st, a, l, t.heads, scratch);
 }
 
 }  // namespace
@@ -359,28 +386,25 @@ bool latent_attn_dims(int kv_rank, int rot_dim, int* key_dim, int* value_dim) {
     for (int dv : {64, 128, 192, 256, 384, 512}) {
         if (kv_rank > dv) continue;
         const int dk = std::max((kv_rank + rot_dim + 31) / 32 * 32, dv);
-        // the largest query tile of this width has to fit beside the ring
-        const size_t smem = dv > 256 ? lt_smem<512, 2>(dk) : lt_smem<256, 4>(dk);
-        if (smem > (size_t)LT_SMEM_CAP) return false;
+        if (dk > dv + 128) return false;
         *key_dim = dk, *value_dim = dv;
         return true;
     }
     return false;
 }
 
-LatentTiling latent_attn_tiling(int n_heads, int value_dim, int most_rows) {
-    const int most = value_dim > 256 ? 32 : 64;
+LatentTiling latent_attn_tiling(const tsb_ctx* ctx, int n_heads, int most_rows, int n_rows, int max_len) {
     LatentTiling t;
-    t.queries = 16;
-    while (t.queries < most && t.queries < n_heads * most_rows) t.queries *= 2;
+    // sixteen queries a tile where 32 would leave SMs idle: the key tiles of few streams
+    const int64_t work = (int64_t)((n_rows * (int64_t)n_heads + 31) / 32) * ((max_len + LT_TOK - 1) / LT_TOK);
+    t.queries = n_heads * most_rows <= 16 || work < ctx->sm_count ? 16 : 32;
     const int head_tiles = (n_heads + t.queries - 1) / t.queries;
     t.heads = (n_heads + head_tiles - 1) / head_tiles;
     t.rows = std::max(1, std::min(most_rows, t.queries / t.heads));
     return t;
 }
 
-cudaError_t launch_latent_attn(tsb_ctx* ctx, cudaStream_t st, const LatentAttn& a, const AttnBatch& b, int most_rows, void* scratch) {
-    const LatentTiling t = latent_attn_tiling(a.n_heads, a.value_dim, most_rows);
+cudaError_t launch_latent_attn(tsb_ctx* ctx, cudaStream_t st, const LatentAttn& a, const AttnBatch& b, const LatentTiling& t, void* scratch) {
     WattnLaunch l{b.small, b.n_small, 1, 0, t.rows, b.max_len};
     if (b.rows_per_seq > 0) {
         const int tpg = (b.rows_per_seq + t.rows - 1) / t.rows;

@@ -22,6 +22,7 @@ bool latent_attn_dims(int kv_rank, int rot_dim, int* key_dim, int* value_dim);
 struct LatentTiling {
     int queries, heads, rows;  // queries of a tile, heads of it, rows of it
 };
-LatentTiling latent_attn_tiling(int n_heads, int value_dim, int most_rows);
-// `large` is not used: every tile of b.small has at most the tiling's rows (most_rows: the longest portion of the pass)
-cudaError_t launch_latent_attn(tsb_ctx* ctx, cudaStream_t st, const LatentAttn& a, const AttnBatch& b, int most_rows, void* scratch);
+// most_rows: the longest portion of the launch, n_rows: rows of all portions, max_len: the longest visible context
+LatentTiling latent_attn_tiling(const tsb_ctx* ctx, int n_heads, int most_rows, int n_rows, int max_len);
+// `large` is not used: every tile of b.small has at most the tiling's rows
+cudaError_t launch_latent_attn(tsb_ctx* ctx, cudaStream_t st, const LatentAttn& a, const AttnBatch& b, const LatentTiling& t, void* scratch);

@@ -150,20 +150,23 @@ __device__ __forceinline__ uint4 ldg_stream(const void* p) {
     return v;
 }
 
-// NT token tiles of eight, MT row tiles of sixteen.
-template <int NT, int MT>
+// NT token tiles of eight, MT row tiles of sixteen.  WK warps split the columns of a row tile; products with few columns have
+// several row tiles per CTA instead.  blockIdx.y: which 8 NT tokens.
+template <int NT, int MT, int WK>
 __global__ void __launch_bounds__(FEW_WARPS * 32, 2)
     plain_few_kernel(const __nv_bfloat16* __restrict__ w, int cols, int group_rows, int group_cols, const __nv_bfloat16* x, const __nv_bfloat16* x2,
                      int64_t x_stride, int tokens, const __grid_constant__ PlainEpi epi, uint32_t* __restrict__ err) {
     constexpr int U = MT == 1 ? FEW_UNROLL : FEW_UNROLL / 2;
-    constexpr int TOK = NT * 8, ROWS = MT * 16;
-    __shared__ float red[FEW_WARPS][ROWS][TOK + 1];
-    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
-    const int row0 = blockIdx.x * ROWS;
+    constexpr int TOK = NT * 8, WROWS = MT * 16, ROWS = WROWS * (FEW_WARPS / WK);
+    __shared__ float red[FEW_WARPS][WROWS][TOK + 1];
+    const int warp = (threadIdx.x >> 5) % WK, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
+    const int wrow = (threadIdx.x >> 5) / WK * WROWS, row0 = blockIdx.x * ROWS;
+    const int tok0 = blockIdx.y * TOK;
+    tokens = min(tokens - tok0, TOK);
     const int units = cols / 64;
     const bool pairs = row0 >= epi.pair_row0;
     if (!tile_used(epi, row0, group_rows)) return;  // padding between the mixer's rows and the pairs, or behind a group
-    const __nv_bfloat16* wp = w + (int64_t)(row0 + g) * cols + 8 * t4;
+    const __nv_bfloat16* wp = w + (int64_t)(row0 + wrow + g) * cols + 8 * t4;
     // a unit of 64 columns is two k = 32 halves; per half the lane holds columns 8 t4 .. 8 t4 + 7 of its two rows
     uint4 wa[U][MT][4];
     auto load_w = [&](int i, int u) {
@@ -178,9 +181,9 @@ __global__ void __launch_bounds__(FEW_WARPS * 32, 2)
     };
 #pragma unroll
     for (int i = 0; i < U; i++)
-        if (warp + i * FEW_WARPS < units) load_w(i, warp + i * FEW_WARPS);  // weights do not depend on the preceding kernel
+        if (warp + i * WK < units) load_w(i, warp + i * WK);  // weights do not depend on the preceding kernel
     pdl_wait();
-    const __nv_bfloat16* xb = (pairs ? x2 : x) + (int64_t)g * x_stride + 8 * t4 + (group_rows ? row0 / group_rows * group_cols : 0);
+    const __nv_bfloat16* xb = (pairs ? x2 : x) + (int64_t)(tok0 + g) * x_stride + 8 * t4 + (group_rows ? row0 / group_rows * group_cols : 0);
     float acc[MT][NT][4];
 #pragma unroll
     for (int m = 0; m < MT; m++)
@@ -188,10 +191,10 @@ __global__ void __launch_bounds__(FEW_WARPS * 32, 2)
         for (int n = 0; n < NT; n++)
 #pragma unroll
             for (int i = 0; i < 4; i++) acc[m][n][i] = 0.f;
-    for (int u0 = warp; u0 < units; u0 += U * FEW_WARPS) {
+    for (int u0 = warp; u0 < units; u0 += U * WK) {
 #pragma unroll
         for (int i = 0; i < U; i++) {
-            const int u = u0 + i * FEW_WARPS;
+            const int u = u0 + i * WK;
             if (u >= units) break;
 #pragma unroll
             for (int n = 0; n < NT; n++) {
@@ -210,7 +213,7 @@ __global__ void __launch_bounds__(FEW_WARPS * 32, 2)
                     mma_bf16(acc[m][n], a3, b1.z, b1.w);
                 }
             }
-            const int un = u + U * FEW_WARPS;
+            const int un = u + U * WK;
             if (un < units) load_w(i, un);
         }
     }
@@ -219,28 +222,29 @@ __global__ void __launch_bounds__(FEW_WARPS * 32, 2)
     for (int m = 0; m < MT; m++)
 #pragma unroll
         for (int n = 0; n < NT; n++) {
-            red[warp][m * 16 + g][n * 8 + 2 * t4] = acc[m][n][0];
-            red[warp][m * 16 + g][n * 8 + 2 * t4 + 1] = acc[m][n][1];
-            red[warp][m * 16 + g + 8][n * 8 + 2 * t4] = acc[m][n][2];
-            red[warp][m * 16 + g + 8][n * 8 + 2 * t4 + 1] = acc[m][n][3];
+            float(*mine)[TOK + 1] = red[threadIdx.x >> 5];
+            mine[m * 16 + g][n * 8 + 2 * t4] = acc[m][n][0];
+            mine[m * 16 + g][n * 8 + 2 * t4 + 1] = acc[m][n][1];
+            mine[m * 16 + g + 8][n * 8 + 2 * t4] = acc[m][n][2];
+            mine[m * 16 + g + 8][n * 8 + 2 * t4 + 1] = acc[m][n][3];
         }
     __syncthreads();
     auto total = [&](int r, int t) {
         float v = 0.f;
 #pragma unroll
-        for (int i = 0; i < FEW_WARPS; i++) v += red[i][r][t];
+        for (int i = 0; i < WK; i++) v += red[r / WROWS * WK + i][r % WROWS][t];
         return v;
     };
     if (pairs) {
         for (int i = threadIdx.x; i < ROWS / 2 * tokens; i += FEW_WARPS * 32) {
             const int p = i % (ROWS / 2), t = i / (ROWS / 2);
             const int r = (p >> 3) * 16 + (p & 7);
-            epi_pair<__nv_bfloat16>(epi, t, (row0 - epi.pair_row0) / 2 + p, total(r, t), total(r + 8, t), err);
+            epi_pair<__nv_bfloat16>(epi, tok0 + t, (row0 - epi.pair_row0) / 2 + p, total(r, t), total(r + 8, t), err);
         }
     } else {
         for (int i = threadIdx.x; i < ROWS * tokens; i += FEW_WARPS * 32) {
             const int r = i % ROWS, t = i / ROWS;
-            epi_one<__nv_bfloat16>(epi, t, row0 + r, total(r, t), err);
+            epi_one<__nv_bfloat16>(epi, tok0 + t, row0 + r, total(r, t), err);
         }
     }
 }
@@ -322,7 +326,129 @@ __device__ __forceinline__ void tcg_g2s_2d(uint32_t dst_smem, const CUtensorMap*
                  : "memory");
 }
 
+// Where the outputs of one thread of the tensor-memory epilogue go: row n of the matrix, or, in a tile of pairs, every other token of
+// the pair that the row belongs to.
+struct TcgOut {
+    SegAt at;             // rows with a destination of their own
+    bool pairs = false, cache = false, in = false;
+    int tok0, pair = 0, head = 0, col = 0;  // head, col: of a rotated pair
+    __device__ __forceinline__ TcgOut(const PlainEpi& e, int row0, int n, int lane, int tok0_) : tok0(tok0_) {
+        pairs = row0 >= e.pair_row0;
+        if (e.kind != PLAIN_MIXER) {
+            in = n < e.n_valid, at.col = n;
+        } else if (!pairs) {
+            at = seg_at(e, n);
+            in = at.kind >= 0, cache = at.kind == PLAIN_SEG_CACHE;
+        } else {
+            pair = ((n & ~31) - e.pair_row0) / 2 + (lane >> 4) * 8 + (lane & 7);
+            in = pair < e.n_pairs;
+            if (e.rot.half > 0) head = pair / e.rot.half, col = pair - head * e.rot.half, cache = in && head >= e.rot.n_heads;
+        }
+    }
+    static __device__ __forceinline__ float gate_of(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+
+    // sixteen tokens from tok0 + c0 on
+    template <int KIND>
+    __device__ __forceinline__ void store(const PlainEpi& e, float (&v)[16], int c0, int n_tok, int lane, bool to_cache, uint32_t* err) const {
+        const int t0 = tok0 + c0, left = in ? n_tok - c0 : 0;  // tokens this thread stores
+        if (KIND != PLAIN_MIXER) {
+            float* y = e.y + (int64_t)t0 * e.y_stride + (in ? at.col : 0);
+            const int64_t step = e.y_stride;
+            if (KIND == PLAIN_ADD) {
+                float old[16];
+#pragma unroll
+                for (int j = 0; j < 16; j++) old[j] = j < left ? y[j * step] : 0.f;
+#pragma unroll
+                for (int j = 0; j < 16; j++)
+                    if (j < left) y[j * step] = fmaf(e.alpha, old[j], v[j]);
+            } else {
+                if (e.cap > 0.f) {
+#pragma unroll 1
+                    for (int k = 0; k < 16; k++) {  // rotates the array through one element: one copy of the function
+                        const float x = e.cap * tanhf(v[0] / e.cap);
+#pragma unroll
+                        for (int j = 0; j < 15; j++) v[j] = v[j + 1];
+                        v[15] = x;
+                    }
+                }
+#pragma unroll
+                for (int j = 0; j < 16; j++)
+                    if (j < left) y[j * step] = v[j];
+            }
+        } else if (!pairs) {
+            if (at.kind == PLAIN_SEG_F32) {
+                float* y = static_cast<float*>(at.p) + (int64_t)t0 * at.stride + at.col;
+#pragma unroll
+                for (int j = 0; j < 16; j++)
+                    if (j < left) y[j * at.stride] = v[j];
+            } else if (at.kind == PLAIN_SEG_TYPED) {
+                if (at.gate) {
+                    const __nv_bfloat16* g = static_cast<const __nv_bfloat16*>(at.gate) + (int64_t)t0 * at.gate_stride + at.gate_col;
+                    float z[16];
+#pragma unroll
+                    for (int j = 0; j < 16; j++) z[j] = j < left ? __bfloat162float(g[j * at.gate_stride]) : 0.f;
+#pragma unroll
+                    for (int j = 0; j < 16; j++) v[j] *= gate_of(z[j]);
+                }
+                __nv_bfloat16* y = static_cast<__nv_bfloat16*>(at.p) + (int64_t)t0 * at.stride + at.col;
+#pragma unroll
+                for (int j = 0; j < 16; j++)
+                    if (j < left) put(y + j * at.stride, v[j]);
+            }
+            if (to_cache) {  // the lanes look up the sixteen tokens' rows, every lane stores to all of them
+                const __nv_bfloat16* row = cache_row(e, t0, n_tok - c0, lane, err);
+#pragma unroll
+                for (int j = 0; j < 16; j++) {
+                    __nv_bfloat16* p = reinterpret_cast<__nv_bfloat16*>(__shfl_sync(0xffffffffu, reinterpret_cast<unsigned long long>(row), j));
+                    if (cache && p) put(p + at.stride + at.col, v[j]);
+                }
+            }
+        } else {
+            // The two rows of a pair sit eight lanes apart: after one exchange the lower lane has both coordinates of the even token, the
+            // upper lane those of the odd one.
+            const bool upper = lane & 8;
+            const __nv_bfloat16* row = to_cache ? cache_row(e, t0, n_tok - c0, lane, err) : nullptr;
+            const PlainRotate& r = e.rot;
+#pragma unroll
+            for (int j = 0; j < 16; j += 2) {
+                const float other = __shfl_xor_sync(0xffffffffu, upper ? v[j] : v[j + 1], 8);
+                const float a = upper ? other : v[j], b = upper ? v[j + 1] : other;
+                const int k = j + (upper ? 1 : 0);
+                __nv_bfloat16* p = nullptr;
+                if (to_cache) p = reinterpret_cast<__nv_bfloat16*>(__shfl_sync(0xffffffffu, reinterpret_cast<unsigned long long>(row), k));
+                if (k >= left) continue;
+                if (r.half == 0) {
+                    put(static_cast<__nv_bfloat16*>(e.a) + (int64_t)(t0 + k) * e.a_stride + pair, activate<__nv_bfloat16>(e.act, a) * b);
+                    continue;
+                }
+                const float2 cs = r.table[(int64_t)(t0 + k) * r.half + col];
+                const float lo = fmaf(a, cs.x, -b * cs.y), hi = fmaf(b, cs.x, a * cs.y);
+                if (cache) {
+                    if (p) put(p + r.key_off + col, lo), put(p + r.key_off + r.half + col, hi);
+                } else {
+#pragma unroll
+                    for (int x = 0; x < 2; x++) {
+                        if (!r.q[x]) continue;
+                        __nv_bfloat16* q = static_cast<__nv_bfloat16*>(r.q[x]) + (int64_t)(t0 + k) * r.q_stride[x] + head * r.q_step[x] + r.q_off[x] + col;
+                        put(q, lo), put(q + r.half, hi);
+                    }
+                }
+            }
+        }
+    }
+
+private:
+    static __device__ __forceinline__ __nv_bfloat16* cache_row(const PlainEpi& e, int t0, int left, int lane, uint32_t* err) {
+        if ((lane & 15) >= left) return nullptr;
+        const tsb_row_desc& rd = e.rows[t0 + (lane & 15)];
+        __nv_bfloat16* p = key_row<__nv_bfloat16>(e.keys, rd.seq, rd.base + rd.slot);
+        if (!p) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+        return p;
+    }
+};
+
 // Work item i: token tile i % n_tok_tiles, then the K run, then the row tile - neighbouring CTAs share weight rows.
+template <int KIND>
 __global__ void __launch_bounds__(TCG_THREADS, 1)
     plain_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap xmap, const __grid_constant__ CUtensorMap x2map,
                     int n_row_tiles, int n_tok_tiles, int units, int ksplit, int nt, int stages, int tokens, int group_rows, int group_cols,
@@ -432,7 +558,8 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
         }
         if (!ok && lane == 0) bars->failed = 1;
     } else {
-        // ---- epilogue: two threads per weight row of the tile, columns = tokens
+        // ---- epilogue: two threads per weight row of the tile, columns = tokens.  One destination per tile and thread, one short
+        // loop per kind of destination: the code of a kind has to stay in the instruction cache.
         pdl_wait();  // the residual stream and the cache belong to earlier kernels too
         bool ok = true;
         uint32_t tile = 0;
@@ -446,59 +573,18 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
             const uint32_t src = tmem + lane_base + buf * (uint32_t)nt;
             const int n = w.row * TCG_M + quad * 32 + lane;
             const int tok0 = w.tok * nt, n_tok = min(nt, tokens - tok0);
-            const bool pairs = w.row * TCG_M >= epi.pair_row0;
-            const SegAt at = epi.kind == PLAIN_MIXER && !pairs ? seg_at(epi, n) : SegAt();
-            auto finish16 = [&](int c0, const float (&v)[16]) {  // sixteen tokens of this row
-                if (pairs) {
-                    const int pair = (w.row * TCG_M - epi.pair_row0 + quad * 32) / 2 + (lane >> 4) * 8 + (lane & 7);
-#pragma unroll
-                    for (int j = 0; j < 16; j++) {
-                        const float up = __shfl_down_sync(0xffffffffu, v[j], 8);
-                        if (!(lane & 8) && c0 + j < n_tok) epi_pair<__nv_bfloat16>(epi, tok0 + c0 + j, pair, v[j], up, err);
-                    }
-                } else if (epi.kind == PLAIN_ADD) {
-                    // the loads of sixteen tokens are in flight together
-                    float old[16];
-                    const bool in = n < epi.n_valid;
-                    float* y = epi.y + (int64_t)(tok0 + c0) * epi.y_stride + n;
-#pragma unroll
-                    for (int j = 0; j < 16; j++) old[j] = in && c0 + j < n_tok ? y[(int64_t)j * epi.y_stride] : 0.f;
-#pragma unroll
-                    for (int j = 0; j < 16; j++)
-                        if (in && c0 + j < n_tok) y[(int64_t)j * epi.y_stride] = fmaf(epi.alpha, old[j], v[j]);
-                } else if (epi.kind == PLAIN_MIXER) {
-#pragma unroll
-                    for (int j = 0; j < 16; j++)
-                        if (c0 + j < n_tok) seg_put<__nv_bfloat16>(epi, at, tok0 + c0 + j, v[j], err);
-                } else {
-#pragma unroll
-                    for (int j = 0; j < 16; j++)
-                        if (c0 + j < n_tok) epi_one<__nv_bfloat16>(epi, tok0 + c0 + j, n, v[j], err);
-                }
-            };
-            if (ksplit == 1) {
-                for (int c0 = first16; c0 < n_tok; c0 += 32) {
-                    uint32_t r[16];
-                    tc_ld16(src + c0, r);
-                    tc_wait_ld();
-                    float v[16];
-#pragma unroll
-                    for (int j = 0; j < 16; j++) v[j] = __uint_as_float(r[j]);
-                    if (ok) finish16(c0, v);
-                }
-                tc_fence_before();
-                __syncwarp();
-                if (lane == 0) mbar_arrive(&bars->acc_empty[buf]);
-            } else {
+            bool finish = ok;
+            const float* all = nullptr;
+            if (ksplit > 1) {
                 // a run of a cut tile: leave the sums, take a ticket; whoever takes the last one adds the runs in order
                 const int tix = w.row * n_tok_tiles + w.tok;
-                float* mine = part + ((int64_t)tix * ksplit + w.run) * (TCG_M * nt);
+                float* mine = part + ((int64_t)tix * ksplit + w.run) * (TCG_M * nt) + quad * 32 + lane;
                 for (int c0 = first16; c0 < n_tok; c0 += 32) {
                     uint32_t r[16];
                     tc_ld16(src + c0, r);
                     tc_wait_ld();
 #pragma unroll
-                    for (int j = 0; j < 16; j++) mine[(int64_t)(c0 + j) * TCG_M + quad * 32 + lane] = ok ? __uint_as_float(r[j]) : 0.f;
+                    for (int j = 0; j < 16; j++) mine[(c0 + j) * TCG_M] = ok ? __uint_as_float(r[j]) : 0.f;
                 }
                 tc_fence_before();
                 __syncwarp();
@@ -511,24 +597,38 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
                     bars->ticket = t;
                 }
                 asm volatile("bar.sync 1, %0;" ::"n"(TCG_EPI_WARPS * 32) : "memory");
-                if (bars->ticket == (uint32_t)ksplit - 1) {
-                    __threadfence();
-                    const float* all = part + (int64_t)tix * ksplit * (TCG_M * nt);
-                    for (int c0 = first16; c0 < n_tok; c0 += 32) {
-                        float v[16];
+                finish = bars->ticket == (uint32_t)ksplit - 1;
+                __threadfence();
+                all = part + (int64_t)tix * ksplit * (TCG_M * nt) + quad * 32 + lane;
+                asm volatile("bar.sync 1, %0;" ::"n"(TCG_EPI_WARPS * 32) : "memory");  // the ticket word is reused by the next tile
+            }
+            const TcgOut out(epi, w.row * TCG_M, n, lane, tok0);
+            const bool to_cache = KIND == PLAIN_MIXER && __any_sync(0xffffffffu, out.cache);
+            // one loop over the tile's tokens, sixteen at a time
+            if (finish)
+                for (int c0 = first16; c0 < n_tok; c0 += 32) {
+                    float v[16];
+                    __syncwarp();
+                    if (ksplit == 1) {
+                        uint32_t r[16];
+                        tc_ld16(src + c0, r);
+                        tc_wait_ld();
+#pragma unroll
+                        for (int j = 0; j < 16; j++) v[j] = __uint_as_float(r[j]);
+                    } else {
 #pragma unroll
                         for (int j = 0; j < 16; j++) v[j] = 0.f;
                         for (int k = 0; k < ksplit; k++) {
-                            float p[16];
 #pragma unroll
-                            for (int j = 0; j < 16; j++) p[j] = __ldcg(all + (int64_t)k * (TCG_M * nt) + (int64_t)(c0 + j) * TCG_M + quad * 32 + lane);
-#pragma unroll
-                            for (int j = 0; j < 16; j++) v[j] += p[j];
+                            for (int j = 0; j < 16; j++) v[j] += __ldcg(all + (int64_t)k * (TCG_M * nt) + (c0 + j) * TCG_M);
                         }
-                        finish16(c0, v);
                     }
+                    out.store<KIND>(epi, v, c0, n_tok, lane, to_cache, err);
                 }
-                asm volatile("bar.sync 1, %0;" ::"n"(TCG_EPI_WARPS * 32) : "memory");  // the ticket word is reused by the next tile
+            if (ksplit == 1) {
+                tc_fence_before();
+                __syncwarp();
+                if (lane == 0) mbar_arrive(&bars->acc_empty[buf]);
             }
         }
         if (!ok && lane == 0) bars->failed = 1;
@@ -622,17 +722,33 @@ TcgPlan tcg_plan(const tsb_ctx* ctx, int row_tiles, int units, int tokens) {
     return best;
 }
 
-template <int NT, int MT>
+template <int NT, int MT, int WK>
 cudaError_t launch_few(tsb_ctx* ctx, cudaStream_t st, const PlainMat& w, const __nv_bfloat16* x, const __nv_bfloat16* x2, int64_t x_stride, int tokens,
                        const PlainEpi& epi) {
     // Not launched ahead of the attention kernel's end (the output product follows it): CTAs that become resident beside the
     // last attention CTAs are packed on few SMs and run with their small L1 - 67 to 75 us instead of 27 at 4096 x 18432.
     const bool ahead = epi.kind != PLAIN_ADD;
-    return tsb_launch(ctx, plain_few_kernel<NT, MT>, dim3((unsigned)(w.rows / (16 * MT))), dim3(FEW_WARPS * 32), 0, st, ahead,
+    const dim3 grid((unsigned)(w.rows / (16 * MT * (FEW_WARPS / WK))), (unsigned)((tokens + 8 * NT - 1) / (8 * NT)));
+    return tsb_launch(ctx, plain_few_kernel<NT, MT, WK>, grid, dim3(FEW_WARPS * 32), 0, st, ahead,
                       (const __nv_bfloat16*)w.data, (int)w.cols, w.group_rows, w.group_cols, x, x2, x_stride, tokens, epi, ctx->dev_error);
 }
 
 constexpr int FEW_MAX = 16;  // token rows up to which the weight-streaming kernel runs
+// A product with few columns (one head's worth) is too short for the tensor-memory pipeline: the weight-streaming kernel takes it
+// sixteen tokens at a time, its weights coming from the L2 cache after the first.
+constexpr int FEW_SHORT_UNITS = 8, FEW_SHORT_MAX = 128;
+constexpr int64_t FEW_SHORT_BYTES = 16 << 20;
+template <int NT>
+cudaError_t launch_few_any(tsb_ctx* ctx, cudaStream_t st, const PlainMat& w, const __nv_bfloat16* x, const __nv_bfloat16* x2, int64_t x_stride, int tokens,
+                           const PlainEpi& epi) {
+    const int units = (int)(w.cols / TCG_K);
+    if (units == 1) return launch_few<NT, 1, 1>(ctx, st, w, x, x2, x_stride, tokens, epi);
+    if (units < 4) return launch_few<NT, 1, 2>(ctx, st, w, x, x2, x_stride, tokens, epi);
+    if (units < 8) return launch_few<NT, 1, 4>(ctx, st, w, x, x2, x_stride, tokens, epi);
+    // two row tiles per CTA halve the activation reads when there are rows enough
+    if (w.rows / 32 >= 4 * ctx->sm_count) return launch_few<NT, 2, 8>(ctx, st, w, x, x2, x_stride, tokens, epi);
+    return launch_few<NT, 1, 8>(ctx, st, w, x, x2, x_stride, tokens, epi);
+}
 
 }  // namespace
 
@@ -650,11 +766,8 @@ cudaError_t launch_plain_gemm(tsb_ctx* ctx, cudaStream_t st, bool f32, const Pla
                           (const float*)x, (const float*)x2, x_stride, tokens, epi, ctx->dev_error);
     }
     const __nv_bfloat16 *xb = (const __nv_bfloat16*)x, *xb2 = (const __nv_bfloat16*)x2;
-    if (tokens <= FEW_MAX) {
-        const bool two = w.rows / 32 >= 4 * ctx->sm_count;  // two row tiles per CTA halve the activation reads when there are rows enough
-        if (tokens <= 8) return two ? launch_few<1, 2>(ctx, st, w, xb, xb2, x_stride, tokens, epi) : launch_few<1, 1>(ctx, st, w, xb, xb2, x_stride, tokens, epi);
-        return two ? launch_few<2, 2>(ctx, st, w, xb, xb2, x_stride, tokens, epi) : launch_few<2, 1>(ctx, st, w, xb, xb2, x_stride, tokens, epi);
-    }
+    if (tokens <= FEW_MAX || (tokens <= FEW_SHORT_MAX && w.cols <= FEW_SHORT_UNITS * TCG_K && w.rows * w.cols * 2 <= FEW_SHORT_BYTES))
+        return tokens <= 8 ? launch_few_any<1>(ctx, st, w, xb, xb2, x_stride, tokens, epi) : launch_few_any<2>(ctx, st, w, xb, xb2, x_stride, tokens, epi);
     const int row_tiles = (int)(w.rows / TCG_M), units = (int)(w.cols / TCG_K);
     const TcgPlan p = tcg_plan(ctx, row_tiles, units, tokens);
     CUtensorMap wm, xm, xm2;
@@ -663,13 +776,18 @@ cudaError_t launch_plain_gemm(tsb_ctx* ctx, cudaStream_t st, bool f32, const Pla
     if (e == cudaSuccess) e = tcg_map(x, x_rows, x_cols, x_stride, p.nt, &xm);
     if (e == cudaSuccess) e = tcg_map(x2 ? x2 : x, x_rows, x_cols, x_stride, p.nt, &xm2);
     if (e != cudaSuccess) return e;
-    static SmemOptIn configured;
-    if ((e = tsb_opt_in_smem(ctx, plain_tc_kernel, (size_t)TCG_SMEM_CAP, configured)) != cudaSuccess) return e;
     const int tok_tiles = (tokens + p.nt - 1) / p.nt;
     const int items = row_tiles * tok_tiles * p.ksplit;
     uint32_t* tickets = static_cast<uint32_t*>(workspace);
     float* part = reinterpret_cast<float*>(tickets + TCG_TICKETS);
     const size_t smem = TCG_HEADER + (size_t)p.stages * (TCG_M + p.nt) * 128;
-    return tsb_launch(ctx, plain_tc_kernel, dim3((unsigned)std::min(items, ctx->sm_count)), dim3(TCG_THREADS), smem, st, true, wm, xm, xm2, row_tiles,
-                      tok_tiles, units, p.ksplit, p.nt, p.stages, tokens, w.group_rows, w.group_cols, epi, part, tickets, ctx->dev_error);
+    auto run = [&](auto kernel, SmemOptIn& configured) {
+        if (cudaError_t r = tsb_opt_in_smem(ctx, kernel, (size_t)TCG_SMEM_CAP, configured); r != cudaSuccess) return r;
+        return tsb_launch(ctx, kernel, dim3((unsigned)std::min(items, ctx->sm_count)), dim3(TCG_THREADS), smem, st, true, wm, xm, xm2, row_tiles, tok_tiles,
+                          units, p.ksplit, p.nt, p.stages, tokens, w.group_rows, w.group_cols, epi, part, tickets, ctx->dev_error);
+    };
+    static SmemOptIn configured[3];
+    if (epi.kind == PLAIN_STORE) return run(plain_tc_kernel<PLAIN_STORE>, configured[0]);
+    if (epi.kind == PLAIN_ADD) return run(plain_tc_kernel<PLAIN_ADD>, configured[1]);
+    return run(plain_tc_kernel<PLAIN_MIXER>, configured[2]);
 }

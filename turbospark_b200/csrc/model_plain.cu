@@ -199,10 +199,10 @@ int32_t plain_runtime_init(tsb_session* s, ModelRt& rt, const tsb_model* tm, con
         p->cat_stride = std::max<int64_t>(p->cat_stride, l.out.cols);
         p->gate_stride = std::max(p->gate_stride, l.cfg.n_q_heads);
         if (l.post_norm) p->act_stride = std::max<int64_t>(p->act_stride, l.ffn_pad);
-        if (l.cfg.qk_norm) p->raw_stride = std::max<int64_t>(p->raw_stride, (H + l.cfg.n_kv_heads) * l.cfg.head_dim);
+        if (l.cfg.qk_norm) p->raw_stride = std::max<int64_t>(p->raw_stride, plain_pad((H + l.cfg.n_kv_heads) * l.cfg.head_dim, 4));
         if (l.cfg.value_gate) p->value_gate_stride = std::max<int64_t>(p->value_gate_stride, plain_pad(H * l.value_pad, 16));
         if (l.mixer != MIX_LATENT) continue;
-        p->raw_stride = std::max<int64_t>(p->raw_stride, l.cfg.kv_rank);
+        p->raw_stride = std::max<int64_t>(p->raw_stride, plain_pad(l.cfg.kv_rank, 4));
         p->absorbed_stride = std::max<int64_t>(p->absorbed_stride, H * l.key_dim);
         p->sums_stride = std::max<int64_t>(p->sums_stride, H * l.rank_pad);
         if (l.expands) wide = std::max<int64_t>(wide, H * (l.head_pad + l.value_pad)), latent = std::max<int64_t>(latent, l.key_dim);
@@ -295,7 +295,7 @@ struct TileLists {
 // What a pass knows about its portions before the first launch.
 struct PassPlan {
     std::vector<TileLists> lists;
-    int max_len = 0, longest = 0, longest_short = 0;
+    int max_len = 0, longest = 0, longest_short = 0, rows_short = 0;
     // portions whose latents are expanded, and the rows that hold all the others
     std::vector<ExpandStream> expanded;
     std::vector<bool> is_expanded;
@@ -309,8 +309,9 @@ struct PassPlan {
     }
 };
 
-int latent_most_rows(const PassPlan& plan, const Pass& p, const PlainLayer& l) {
-    return p.rows_per_seq > 0 ? p.rows_per_seq : l.expands ? plan.longest_short : plan.longest;
+LatentTiling latent_tiling(const tsb_ctx* ctx, const PassPlan& plan, const Pass& p, const PlainLayer& l) {
+    const bool all = p.rows_per_seq > 0 || !l.expands;
+    return latent_attn_tiling(ctx, l.cfg.n_q_heads, all ? plan.longest : plan.longest_short, all ? p.rows : plan.rows_short, plan.max_len);
 }
 
 int32_t plan_pass(tsb_session* s, const PlainModel* m, const PlainRt* b, const Pass& p, PassPlan& plan) {
@@ -330,7 +331,7 @@ int32_t plan_pass(tsb_session* s, const PlainModel* m, const PlainRt* b, const P
             plan.expanded_pages += pages, plan.expanded_len = std::max(plan.expanded_len, len);
         } else {
             first_short = std::min(first_short, g.first_row), end_short = std::max(end_short, g.first_row + g.n_rows);
-            plan.longest_short = std::max(plan.longest_short, g.n_rows);
+            plan.longest_short = std::max(plan.longest_short, g.n_rows), plan.rows_short += g.n_rows;
         }
     }
     plan.short_first = first_short, plan.short_rows = std::max(0, end_short - first_short);
@@ -371,8 +372,8 @@ int32_t plan_pass(tsb_session* s, const PlainModel* m, const PlainRt* b, const P
             const int grp = l.cfg.n_q_heads / l.cfg.n_kv_heads;
             rc = add(TILES_ALL, grp, wattn_rows_per_tile(l.head_pad, grp, l.cfg.log_bias != 0), WATTN_SMALL_Q);
         } else {
-            const int most = latent_most_rows(plan, p, l);
-            if (most > 0) rc = add(l.expands ? TILES_LATENT_SHORT : TILES_LATENT, l.cfg.n_q_heads, latent_attn_tiling(l.cfg.n_q_heads, l.rank_pad, most).rows, 0);
+            if (!l.expands || plan.longest_short > 0)
+                rc = add(l.expands ? TILES_LATENT_SHORT : TILES_LATENT, l.cfg.n_q_heads, latent_tiling(s->ctx, plan, p, l).rows, 0);
             if (rc == TSB_OK && l.expands && !plan.expanded.empty()) rc = add(TILES_WIDE, 1, WATTN_WIDE_ROWS, 0);
         }
         if (rc) return rc;
@@ -499,12 +500,11 @@ struct Forward {
             LatentAttn a;
             a.keys = rt.kv->key_layers[L], a.q = b->absorbed, a.q_stride = b->absorbed_stride, a.out = b->sums, a.out_stride = b->sums_stride;
             a.rows = p.rows_dev, a.n_heads = c.n_q_heads, a.value_dim = l.rank_pad, a.scale = c.score_scale, a.sink = c.sink ? l.sink : nullptr;
-            const int most = latent_most_rows(plan, p, l);
+            const LatentTiling tiling = latent_tiling(ctx, plan, p, l);
             AttnBatch batch;
-            if (const AttnBatch* t = plan.find(l.expands ? TILES_LATENT_SHORT : TILES_LATENT, c.n_q_heads, latent_attn_tiling(c.n_q_heads, l.rank_pad, most).rows))
-                batch = *t;
+            if (const AttnBatch* t = plan.find(l.expands ? TILES_LATENT_SHORT : TILES_LATENT, c.n_q_heads, tiling.rows)) batch = *t;
             batch.rows = p.rows, batch.rows_per_seq = p.rows_per_seq, batch.max_len = plan.max_len;
-            e = launch_latent_attn(ctx, st, a, batch, most, b->attn_ws);
+            e = launch_latent_attn(ctx, st, a, batch, tiling, b->attn_ws);
         }
         if (e != cudaSuccess) return e;
         return product(l.lift, b->sums, b->sums_stride, b->cat, l.out.cols, c.value_dim, l.value_pad, c.value_gate != 0);
@@ -1159,16 +1159,17 @@ int32_t tsb_latent_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* cache, int32_t 
     LatentAttn a;
     a.keys = kv, a.q = q, a.q_stride = q_stride, a.out = out, a.out_stride = out_stride, a.rows = rows_dev, a.n_heads = n_heads, a.value_dim = value_dim;
     a.scale = scale, a.sink = sink;
+    const LatentTiling tiling = latent_attn_tiling(ctx, n_heads, most, b.rows, max_len);
     if (uniform) {
         b.rows_per_seq = most;
-        TSB_CUDA(ctx, launch_latent_attn(ctx, st, a, b, most, scratch));
+        TSB_CUDA(ctx, launch_latent_attn(ctx, st, a, b, tiling, scratch));
         return TSB_OK;
     }
-    const int rpt = latent_attn_tiling(n_heads, value_dim, most).rows;
+    const int rpt = tiling.rows;
     std::vector<AttnTile> tiles;
     for (int i = 0, r = 0; i < n_groups; r += group_rows[i], i++)
         for (int k = 0; k < group_rows[i]; k += rpt) tiles.push_back({r + k, std::min(rpt, group_rows[i] - k)});
-    return with_tiles(ctx, st, tiles, {}, b, [&](const AttnBatch& t) { return launch_latent_attn(ctx, st, a, t, most, scratch); });
+    return with_tiles(ctx, st, tiles, {}, b, [&](const AttnBatch& t) { return launch_latent_attn(ctx, st, a, t, tiling, scratch); });
 }
 
 int32_t tsb_plain_gemm_heads(tsb_ctx* ctx, tsb_stream s, int32_t type, const void* w, int32_t heads, int32_t head_rows, int64_t cols, const void* x,

@@ -218,11 +218,12 @@ __global__ void __launch_bounds__(ROW_THREADS)
     }
 }
 
-// a warp per (row, head)
-template <typename T>
+// LANES lanes per (row, head).  VEC > 0: the width is a multiple of four and at most 4 LANES VEC, and a lane holds its columns in
+// registers.
+template <typename T, int LANES, int VEC>
 __global__ void __launch_bounds__(ROW_THREADS) head_norms_kernel(const __grid_constant__ HeadNorms h, int rows, uint32_t* __restrict__ err) {
-    const int lane = threadIdx.x & 31;
-    const int64_t item = (int64_t)blockIdx.x * (ROW_THREADS / 32) + (threadIdx.x >> 5);
+    const int lane = threadIdx.x & (LANES - 1);
+    const int64_t item = (int64_t)blockIdx.x * (ROW_THREADS / LANES) + threadIdx.x / LANES;
     const int per = h.n_q + h.n_k;
     const bool in = item < (int64_t)rows * per;
     const int r = in ? (int)(item / per) : 0, head = in ? (int)(item % per) : 0;
@@ -234,9 +235,22 @@ __global__ void __launch_bounds__(ROW_THREADS) head_norms_kernel(const __grid_co
     const float* src = h.raw + (int64_t)r * h.raw_stride + (int64_t)head * h.width;
     const float* w = query ? h.q_weight : h.k_weight;
     float ss = 0.f;
-    for (int i = lane; i < h.width; i += 32) ss = fmaf(src[i], src[i], ss);
+    float4 v[VEC > 0 ? VEC : 1], g[VEC > 0 ? VEC : 1];
+    if (VEC > 0) {
 #pragma unroll
-    for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        for (int k = 0; k < VEC; k++) {
+            const int i = (k * LANES + lane) * 4;
+            v[k] = i < h.width ? *reinterpret_cast<const float4*>(src + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+            g[k] = i < h.width ? *reinterpret_cast<const float4*>(w + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+        for (int k = 0; k < VEC; k++) ss = sum4(v[k], ss);
+    } else {
+        for (int i = lane; i < h.width; i += LANES) ss = fmaf(src[i], src[i], ss);
+    }
+    const uint32_t mask = LANES == 32 ? 0xffffffffu : ((1u << (LANES & 31)) - 1) << (threadIdx.x & 31 & ~(LANES - 1));
+#pragma unroll
+    for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(mask, ss, o);
     float s = 1.f / sqrtf(ss / (float)h.width + h.eps);
     const int pos = rd.base + rd.slot;
     T* dst;
@@ -253,7 +267,16 @@ __global__ void __launch_bounds__(ROW_THREADS) head_norms_kernel(const __grid_co
         }
         dst += (int64_t)(head - h.n_q) * h.keys.head_step;
     }
-    for (int i = lane; i < width; i += 32) put(dst + i, i < h.width ? src[i] * s * w[i] : 0.f);
+    if (VEC > 0) {
+#pragma unroll
+        for (int k = 0; k < VEC; k++) {
+            const int i = (k * LANES + lane) * 4;
+            if (i < h.width) put4(dst + i, make_float4(v[k].x * s * g[k].x, v[k].y * s * g[k].y, v[k].z * s * g[k].z, v[k].w * s * g[k].w));
+        }
+        for (int i = h.width + lane; i < width; i += LANES) put(dst + i, 0.f);
+        return;
+    }
+    for (int i = lane; i < width; i += LANES) put(dst + i, i < h.width ? src[i] * s * w[i] : 0.f);
 }
 
 __global__ void __launch_bounds__(ROW_THREADS)
@@ -347,9 +370,20 @@ cudaError_t launch_post_norm(tsb_ctx* ctx, cudaStream_t st, bool f32, float* x, 
 }
 
 cudaError_t launch_head_norms(tsb_ctx* ctx, cudaStream_t st, bool f32, const HeadNorms& h, int rows) {
-    constexpr int WARPS = ROW_THREADS / 32;
-    const dim3 grid((unsigned)(((int64_t)rows * (h.n_q + h.n_k) + WARPS - 1) / WARPS));
-    return tsb_launch(ctx, f32 ? head_norms_kernel<float> : head_norms_kernel<__nv_bfloat16>, grid, dim3(ROW_THREADS), 0, st, true, h, rows, ctx->dev_error);
+    auto run = [&](auto kernel, int lanes) {
+        const int per_cta = ROW_THREADS / lanes;
+        const dim3 grid((unsigned)(((int64_t)rows * (h.n_q + h.n_k) + per_cta - 1) / per_cta));
+        return tsb_launch(ctx, kernel, grid, dim3(ROW_THREADS), 0, st, true, h, rows, ctx->dev_error);
+    };
+    const bool vec = h.width % 4 == 0 && h.width <= 512 && h.raw_stride % 4 == 0 && (uintptr_t)h.raw % 16 == 0 && h.q_step % 4 == 0 && h.q_stride % 4 == 0;
+    if (f32) {
+        if (vec && h.width <= 64) return run(head_norms_kernel<float, 8, 2>, 8);
+        if (vec && h.width <= 128) return run(head_norms_kernel<float, 16, 2>, 16);
+        return vec ? run(head_norms_kernel<float, 32, 4>, 32) : run(head_norms_kernel<float, 32, 0>, 32);
+    }
+    if (vec && h.width <= 64) return run(head_norms_kernel<__nv_bfloat16, 8, 2>, 8);
+    if (vec && h.width <= 128) return run(head_norms_kernel<__nv_bfloat16, 16, 2>, 16);
+    return vec ? run(head_norms_kernel<__nv_bfloat16, 32, 4>, 32) : run(head_norms_kernel<__nv_bfloat16, 32, 0>, 32);
 }
 
 cudaError_t launch_rotary_table(tsb_ctx* ctx, cudaStream_t st, const double* freq, int half, float magnitude, const tsb_row_desc* rows_dev, int rows,
