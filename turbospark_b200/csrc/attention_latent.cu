@@ -1,8 +1,8 @@
 // Attention over latent rows (attention_latent.cuh), bfloat16, mma.sync m16n8k16.
 //
-// A CTA owns a query tile - 16 MT (row, head) pairs of one stream - and a run of 64-token key tiles, which one warp fetches row by
-// row with bulk copies into a ring of stages.  One tile in shared memory serves both products, and a key byte is read from memory
-// once.  Eight warps:
+// A CTA owns a query tile - 16 MT (row, head) pairs of one stream - and a run of 64-token key tiles, fetched row by row with
+// bulk copies into a ring of stages.  One tile in shared memory serves both products, and a key byte is read from memory once.
+// Eight warps:
 //   scores   KS warps split the key columns, 8 / KS groups of them the keys; a warp's part of every query stays in registers, so this
 //            product reads each key fragment once and nothing else.  The parts meet in shared memory.
 //   softmax  256 / (16 MT) threads per query add the parts, mask, keep the running maximum and sum, leave the weights (bfloat16)
@@ -10,7 +10,8 @@
 //   output   every warp owns DV / 8 value columns of all queries
 // so the accumulators of a 512-column value fit in registers.  Key tiles start at multiples of 64 positions.  A context that does
 // not fill the device with CTAs is cut into runs; a merge launch adds them in order.
-// Waits for copies are bounded; when one runs out the launch is marked failed, the CTA waits for what it has in flight and returns.
+// Waits for copies are bounded; when one runs out the launch is marked failed and the warps go on meeting until the end, where the
+// CTA waits (again with a limit) for what it has in flight.
 #include <algorithm>
 
 #include "attention_latent.cuh"
@@ -92,7 +93,7 @@ __global__ void __launch_bounds__(LT_THREADS, LtGeo<DV, KW, MT>::PER_SM)
     const uint32_t ring_s = smem_u32(ring), p_smem = smem_u32(p_tile);
 
     if (threadIdx.x == 0) {
-        for (int i = 0; i < NST; i++) mbar_init(&full[i], 1);
+        for (int i = 0; i < NST; i++) mbar_init(&full[i], LT_WARPS);
         mbar_fence_init();
     }
     // columns behind the row's: finite, and the queries have zeros there
@@ -101,33 +102,28 @@ __global__ void __launch_bounds__(LT_THREADS, LtGeo<DV, KW, MT>::PER_SM)
         *reinterpret_cast<uint4*>(ring + (size_t)r * G::PITCH + c * 16) = make_uint4(0, 0, 0, 0);
     }
     __syncthreads();
-    // warp 0: two rows a lane.  Positions past the end are masked later; their slots repeat the last row.
-    auto issue = [&](int tile) {
+    // Every warp fetches eight rows of a tile, a lane each.  Positions past the end are masked later; their slots repeat the last row.
+    // The row's address is looked up a tile ahead.
+    auto row_of = [&](int tile) -> const __nv_bfloat16* {
+        if (lane >= 8 || tile >= n_tiles) return nullptr;
+        const __nv_bfloat16* src = key_row<__nv_bfloat16>(a.keys, seq, min(begin + tile * LT_TOK + warp * 8 + lane, hi - 1));
+        if (src) return src;
+        atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);  // not a reserved position: flagged; the copy keeps its byte count
+        return reinterpret_cast<const __nv_bfloat16*>(a.keys.base);
+    };
+    auto issue = [&](int tile, const __nv_bfloat16* src) {
         if (tile >= n_tiles) return;
         uint64_t* bar = &full[tile % NST];
-        if (lane == 0) mbar_expect_tx(bar, (uint32_t)(LT_TOK * DK * 2));
+        if (lane == 0) mbar_expect_tx(bar, (uint32_t)(8 * DK * 2));
         __syncwarp();
-#pragma unroll
-        for (int i = 0; i < 2; i++) {
-            const int r = lane + 32 * i, pos = min(begin + tile * LT_TOK + r, hi - 1);
-            const __nv_bfloat16* src = key_row<__nv_bfloat16>(a.keys, seq, pos);
-            if (!src) {  // not a reserved position: flagged; the copy keeps its byte count
-                atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
-                src = reinterpret_cast<const __nv_bfloat16*>(a.keys.base);
-            }
-            bulk_g2s(ring + (size_t)((tile % NST) * LT_TOK + r) * G::PITCH, src, (uint32_t)(DK * 2), bar);
-        }
+        if (lane < 8) bulk_g2s(ring + (size_t)((tile % NST) * LT_TOK + warp * 8 + lane) * G::PITCH, src, (uint32_t)(DK * 2), bar);
     };
     const bool early = begin + (NST - 1) * LT_TOK <= rd0.base;  // keys of earlier passes
-    if (early && warp == 0) {
+    if (!early) pdl_wait();
 #pragma unroll
-        for (int i = 0; i < NST - 1; i++) issue(i);
-    }
-    pdl_wait();
-    if (!early && warp == 0) {
-#pragma unroll
-        for (int i = 0; i < NST - 1; i++) issue(i);
-    }
+    for (int i = 0; i < NST - 1; i++) issue(i, row_of(i));
+    const __nv_bfloat16* next_row = row_of(NST - 1);
+    if (early) pdl_wait();
     // this warp's part of the queries
     uint32_t qf[MT][G::STEPS][4];
 #pragma unroll
@@ -164,9 +160,10 @@ __global__ void __launch_bounds__(LT_THREADS, LtGeo<DV, KW, MT>::PER_SM)
 
     for (int tile = 0; tile < n_tiles; tile++) {
         // the tile is here, and every warp is done with the stage and the weights of the one before
-        ok = __syncthreads_and(mbar_wait(&full[tile % NST], (tile / NST) & 1, err));
-        if (!ok) break;
-        if (warp == 0) issue(tile + NST - 1);
+        if (ok) ok = mbar_wait(&full[tile % NST], (tile / NST) & 1, err);  // a wait that ran out: the launch is marked, its result void
+        __syncthreads();
+        issue(tile + NST - 1, next_row);
+        next_row = row_of(tile + NST);
         const uint32_t kt = ring_s + (tile % NST) * G::STAGE;
         float s[MT][NT][4];
 #pragma unroll
@@ -270,10 +267,9 @@ __global__ void __launch_bounds__(LT_THREADS, LtGeo<DV, KW, MT>::PER_SM)
                 for (int m = 0; m < MT; m++) mma_bf16(o[m][ND - 1], pa[m], b0, b1);
             }
         }
-    }
-    // no copy is in flight when the CTA leaves
-    if (!ok && warp == 0)
-        for (int i = 0; i < NST; i++) mbar_wait(&full[i], 0u, err), mbar_wait(&full[i], 1u, err);
+        }
+    if (!ok)  // no copy is in flight when the CTA leaves
+        for (int i = max(0, n_tiles - NST); i < n_tiles; i++) mbar_wait(&full[i % NST], (i / NST) & 1, err);
     pdl_launch_dependents();
     __syncthreads();
 #pragma unroll

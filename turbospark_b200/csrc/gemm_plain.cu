@@ -737,7 +737,7 @@ constexpr int FEW_MAX = 16;  // token rows up to which the weight-streaming kern
 // A product with few columns (one head's worth) is too short for the tensor-memory pipeline: the weight-streaming kernel takes it
 // sixteen tokens at a time, its weights coming from the L2 cache after the first.
 constexpr int FEW_SHORT_UNITS = 8, FEW_SHORT_MAX = 128;
-constexpr int64_t FEW_SHORT_BYTES = 16 << 20;
+constexpr int64_t FEW_SHORT_BYTES = 8 << 20;  // of weights, read once per sixteen tokens
 template <int NT>
 cudaError_t launch_few_any(tsb_ctx* ctx, cudaStream_t st, const PlainMat& w, const __nv_bfloat16* x, const __nv_bfloat16* x2, int64_t x_stride, int tokens,
                            const PlainEpi& epi) {
@@ -766,7 +766,7 @@ cudaError_t launch_plain_gemm(tsb_ctx* ctx, cudaStream_t st, bool f32, const Pla
                           (const float*)x, (const float*)x2, x_stride, tokens, epi, ctx->dev_error);
     }
     const __nv_bfloat16 *xb = (const __nv_bfloat16*)x, *xb2 = (const __nv_bfloat16*)x2;
-    if (tokens <= FEW_MAX || (tokens <= FEW_SHORT_MAX && w.cols <= FEW_SHORT_UNITS * TCG_K && w.rows * w.cols * 2 <= FEW_SHORT_BYTES))
+    if (tokens <= FEW_MAX || (tokens <= FEW_SHORT_MAX && w.cols <= FEW_SHORT_UNITS * TCG_K && w.rows * w.cols * 2 * ((tokens + 15) / 16) <= FEW_SHORT_BYTES))
         return tokens <= 8 ? launch_few_any<1>(ctx, st, w, xb, xb2, x_stride, tokens, epi) : launch_few_any<2>(ctx, st, w, xb, xb2, x_stride, tokens, epi);
     const int row_tiles = (int)(w.rows / TCG_M), units = (int)(w.cols / TCG_K);
     const TcgPlan p = tcg_plan(ctx, row_tiles, units, tokens);
