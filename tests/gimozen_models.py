@@ -41,9 +41,11 @@ CONFIGS = {
     # a head of 192 columns in expanded form, a value of 128
     "wide_heads": config(160, 97, [latent(3, 100, 60, 72, 130, 64), attention(12, 1, 64, 64, 100), latent(2, 130, 60, 128, 130, 40, kv_from=0)], eps=1e-6),
     # heads that no expanded kernel takes, a latent above 256, key and value sizes above 128
-    "large": config(128, 64, [latent(2, 160, 48, 150, 300, 48), attention(4, 2, 130, 200, 32), attention(2, 1, 72, 96, 8)], alpha=1.0, embed=0.7),
+    "large": config(128, 64, [latent(2, 160, 48, 150, 300, 48), attention(4, 2, 130, 200, 32), attention(2, 1, 72, 96, 8)], embed=0.7),
     # many heads over one latent row: more than a query tile holds
     "many_heads": config(128, 75, [latent(40, 8, 6, 8, 30, 64), attention(24, 1, 16, 16, 64, temp=(1.0, 1))]),
+    # constants that are one
+    "ones": config(96, 60, [attention(2, 2, 16, 16, 32, scale=0.15, temp=(1.0, 1)), latent(2, 16, 4, 16, 24, None, scale=0.15)], alpha=1.0, embed=1.0),
     "single": config(64, 40, [latent(1, 16, 2, 16, 8, 16, scale=0.2), attention(1, 1, 16, 8, 1, scale=0.2)], embed=1.0),
 }
 
