@@ -401,11 +401,15 @@ TSB_API int32_t tsb_router_logits(tsb_ctx* ctx, tsb_stream s, const void* q_u8, 
 
 /* ------------------------------------------------------------ plain-weight decoders
  * Decoders whose matrices are plain bfloat16 (or f32) and whose layers are put together from the mechanisms below; the
- * reference has no counterpart.  x starts as embed_scale (0: one) times the token's embedding.  A layer has one of two forms:
+ * reference has no counterpart.  x starts as embed_scale (0: one) times the token's embedding, plus row p of a learned table at
+ * position p (positions > 0: that many rows).  A layer has one of three forms:
  *   parallel, one norm:   h = x * gain / sqrt(mean(x^2) + eps)                       one gain for all coordinates
  *                         x = x + mixer(shift(h)) + feed_forward(h)
  *   post_norm:            x = norm1(residual_scale * x + mixer(x)),  x = norm2(residual_scale * x + feed_forward(x))
  *                         norm(y) = y * (1 + w) / sqrt(mean(y^2) + eps)              w per coordinate
+ *   output_norm:          x = x + norm1(mixer(conv1(x))),  x = x + norm2(feed_forward(conv2(x)))
+ *                         norm(y) = y * w / sqrt(mean(y^2) + eps), the mean over each of norm_groups (0: one) equal parts of y
+ *                         conv(h)_t = h_t + sum_j w[:, j] * h_(t - conv_taps + 1 + j), zeros before the start (conv_taps 0: h itself)
  *   shift (token_shift): h_t + (h_{t-1} - h_t) * mu, element by element; h_{-1} = 0
  *   mixer: causal attention, n_q_heads query heads over n_kv_heads key heads (see below for latent layers).
  *     value_dim = 0: the values are the keys; else values of value_dim columns with a projection of their own.
@@ -415,19 +419,36 @@ TSB_API int32_t tsb_router_logits(tsb_ctx* ctx, tsb_stream s, const void* q_u8, 
  *     log_bias: score -= r1[head] * ln(1 + r2[head] * distance);  window > 0: the last `window` positions only;
  *     sink: exp(sink[head]) joins the softmax's denominator;
  *     head_gate: each head's output times sigmoid of one number per head, projected from the mixer's input;
- *     value_gate: every output column times sigmoid of a number of its own, projected from the mixer's input
+ *     value_gate: every output column times sigmoid of a number of its own, projected from the mixer's input;
+ *     in the output_norm form also: qkv_bias: q, k and v have biases; qk_norm = TSB_NORM_PROJECTION: queries, and keys, normed over all
+ *     heads at once, a weight per row of the projection; linear_bias: score -= 2^(-8 (h + 1) / n_q_heads) * distance for head h; chunk > 0:
+ *     a position sees the earlier ones of its own run of `chunk` positions, counted from position 0
+ *   recurrent mixer (recurrence > 0, output_norm form): heads with a state S [rec_dim, rec_vdim] in f32,
+ *     S_t = decay_t S_(t-1) + k_t v_t^T, o_t = S_t^T q_t, starting from zero
+ *     TSB_REC_FORGET: q = silu(W_q h), v = W_v h; per row of S: decay = f = l + (1 - l) sigmoid(W_f h + b_f), k = 1 - f; o normed per head
+ *       (a weight per column, shared by the heads)
+ *     TSB_REC_MLSTM: q = W_q h rec_dim^(-1/2), k = W_k h, v = W_v h; per head i = c tanh((W_i h + b_i) / c), f = ln sigmoid(c tanh((W_f h +
+ *       b_f) / c)) with c = rec_cap; m_t = max(f + m_(t-1), i), m_0 = 0; decay = exp(f + m_(t-1) - m_t), k scaled by exp(i - m_t); n is S
+ *       with v = 1; o / (max(|n . q|, exp(-m)) + 1e-6), normed per head, a weight per column of every head, times sigmoid(W_g h)
+ *     TSB_REC_SSD: W_in h = z | x | B | C | dt; x, B, C (rec_groups of rec_dim columns) through a causal convolution per channel with
+ *       bias and silu; dt = softplus(dt + b); decay = exp(-exp(A_log) dt), k = dt B, v = x, q = C; o + D x, times silu(z), normed in
+ *       rec_norm_groups parts with a weight per column
+ *     with n_q_heads > 0 as well the layer has both, side by side: attn_scale * attention + rec_scale * recurrence
  *   latent mixer (kv_rank > 0): the cache holds per position c, kv_rank numbers projected and normed (plain weight), and one
  *     rotated key part of rot_dim columns for all heads.  Head: key = [W_uk c (head_dim), rotated part], value = W_uv c
  *     (value_dim), query = [head_dim plain, rot_dim rotated] columns.  Coordinates i and i + rot_dim / 2 are rotated by position * f_i,
  *     f_i = rot_base^(-2 i / rot_dim); rot_factor > 0 scales the frequencies between f_i and f_i / rot_factor by how often they
  *     turn within rot_original positions (rot_fast .. rot_slow turns), and cos and sin by 0.1 ln(rot_factor) + 1.
  *     kv_source = j + 1: the layer has no latent of its own and reads the one of layer j (0: its own).
- *   feed_forward (ffn > 0): W_down(act(W_gate h) * (W_up h)); a post_norm layer without one has no norm2
+ *   feed_forward (ffn > 0): W_down(act(W_gate h) * (W_up h)); a post_norm or output_norm layer without one has no norm2
+ *     experts > 0 (output_norm form): `experts` of them; s = sigmoid(W_router h), choice = s + correction; of expert_groups equal groups the
+ *     expert_keep ones with the largest sum of their two largest choices stay, the expert_top largest choices in them are taken, and
+ *     the sum of their outputs is weighted with s
  * then logits = W_head norm(x), through logit_cap * tanh(logits / logit_cap) when logit_cap > 0.
  * Residual stream, norms, shift, rotation, scores, softmax and gates are f32 in both modes.  compute = TSB_BF16: matrices,
  * activations and the cache in bfloat16 with f32 accumulation; TSB_F32: everything in f32.
- * Models with a token shift keep per stream the last rows' h of every layer (a cursor can be moved back by max_rows rows, or to
- * 0).  Verify passes are chains; tree rounds are refused with TSB_ERR_UNSUPPORTED. */
+ * Models with a token shift, a convolution or a recurrence keep per stream what the next row needs of the last rows of every layer (a
+ * cursor can be moved back by max_rows rows after a pass of at most that many, or to 0).  Verify passes are chains; tree rounds are refused with TSB_ERR_UNSUPPORTED. */
 enum { TSB_BF16 = 0, TSB_F32 = 1 };
 enum { TSB_ACT_GELU_TANH = 0, TSB_ACT_SILU = 1 };
 typedef struct tsb_plain_config {
@@ -435,7 +456,10 @@ typedef struct tsb_plain_config {
     float norm_eps, logit_cap;
     int32_t post_norm;
     float residual_scale, embed_scale;
+    int32_t output_norm, norm_groups, conv_taps, positions;
 } tsb_plain_config;
+enum { TSB_NORM_HEAD = 1, TSB_NORM_PROJECTION = 2 };                                   /* qk_norm */
+enum { TSB_REC_NONE = 0, TSB_REC_FORGET = 1, TSB_REC_MLSTM = 2, TSB_REC_SSD = 3 };      /* recurrence */
 typedef struct tsb_plain_layer {
     int32_t n_q_heads, n_kv_heads, head_dim, window;
     float score_scale, score_cap;
@@ -446,6 +470,11 @@ typedef struct tsb_plain_layer {
     int32_t sink, value_gate; /* 0 / 1 */
     int32_t kv_rank, rot_dim, kv_source;
     double rot_base, rot_factor, rot_original, rot_fast, rot_slow;
+    int32_t qkv_bias, linear_bias, chunk;
+    float attn_scale, rec_scale; /* of a layer with both mixers */
+    int32_t recurrence, rec_heads, rec_dim, rec_vdim, rec_groups, rec_taps, rec_norm_groups;
+    float rec_cap;
+    int32_t experts, expert_top, expert_groups, expert_keep;
 } tsb_plain_layer;
 enum {
     TSB_P_EMBED = 0, TSB_P_HEAD, TSB_P_FINAL_NORM,                     /* layer ignored; [vocab, d], [vocab, d], [1] (post_norm: [d]) */
@@ -454,7 +483,16 @@ enum {
     TSB_P_FF_GATE, TSB_P_FF_UP, TSB_P_FF_DOWN,                         /* [ffn, d], [ffn, d], [d, ffn] */
     TSB_P_NORM2, TSB_P_V, TSB_P_Q_NORM, TSB_P_K_NORM,                  /* [d], [G E, d], [D], [D] with E = value_dim */
     TSB_P_SINK, TSB_P_VALUE_GATE,                                      /* [H], [H E, d] */
-    TSB_P_DKV, TSB_P_DKV_NORM, TSB_P_UK, TSB_P_UV                      /* [kv_rank + rot_dim, d], [kv_rank], [H D, kv_rank], [H E, kv_rank] */
+    TSB_P_DKV, TSB_P_DKV_NORM, TSB_P_UK, TSB_P_UV,                     /* [kv_rank + rot_dim, d], [kv_rank], [H D, kv_rank], [H E, kv_rank] */
+    TSB_P_POSITIONS,                                                   /* layer ignored; [positions, d] */
+    TSB_P_CONV1, TSB_P_CONV2,                                          /* [d, conv_taps] */
+    TSB_P_Q_BIAS, TSB_P_K_BIAS, TSB_P_V_BIAS,                          /* [H D], [G D], [G E]; projection norms: TSB_P_Q_NORM [H D], TSB_P_K_NORM [G D] */
+    TSB_P_ROUTER, TSB_P_CORRECTION,                                    /* [experts, d], [experts]; TSB_P_FF_*: the experts' matrices one after another */
+    TSB_P_REC_Q, TSB_P_REC_K, TSB_P_REC_V, TSB_P_REC_GATE,             /* [h D, d], [h D, d], [h E, d], [h E, d] with h, D, E = rec_heads, rec_dim, rec_vdim */
+    TSB_P_REC_F, TSB_P_REC_F_BIAS, TSB_P_REC_LOWER,                    /* FORGET: [h D, d], [h D], [h D]; MLSTM: [h, d], [h] */
+    TSB_P_REC_I, TSB_P_REC_I_BIAS, TSB_P_REC_NORM, TSB_P_REC_O,        /* [h, d], [h], [E] (FORGET) or [h E], [d, h E] */
+    TSB_P_REC_IN, TSB_P_REC_CONV, TSB_P_REC_CONV_BIAS,                 /* SSD: [2 h E + 2 rec_groups D + h, d], [h E + 2 rec_groups D, rec_taps], ... */
+    TSB_P_REC_DT_BIAS, TSB_P_REC_A_LOG, TSB_P_REC_D                    /* [h] each */
 };                                                                     /* with values: W_o [d, H E]; latent layers: W_q [H (D + rot_dim), d] */
 TSB_API int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const tsb_plain_layer* layers, tsb_model** out);
 /* Upload one tensor, rows x cols row-major (vectors: rows = 1); host_type says what the host data is (TSB_BF16 / TSB_F32). */
@@ -500,6 +538,9 @@ typedef struct tsb_attention_extras {
     const float* sink;            /* [n_q_heads] or NULL */
     const void* value_gate;       /* [rows, n_q_heads * value columns] pre-activations in `type`, or NULL */
     int64_t value_gate_stride;
+    const float* slopes;          /* [n_q_heads] or NULL: score -= slope * distance (not with r1, r2) */
+    int32_t chunk;                /* > 0: keys of the query's own run of `chunk` positions (not with a window) */
+    float out_scale;              /* of the outputs; 0: one */
 } tsb_attention_extras;
 /* bfloat16 with keys and values of different widths: one query head per key head, keys of 64, 128 or 192, values of 64 or 128 columns. */
 TSB_API int32_t tsb_plain_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, int32_t layer, const void* q, int64_t q_stride, void* out,

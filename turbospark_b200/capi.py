@@ -315,9 +315,10 @@ class Ctx:
                                               _vp(r1), _vp(r2), _vp(gate), C.c_int32(window), C.c_int32(max_len), _vp(scratch)))
 
     def plain_attention(self, kv, layer, q, q_stride, out, out_stride, rows_dev, group_rows, n_q_heads, scale, max_len, scratch, stream=None, cap=0.0,
-                        window=0, r1=None, r2=None, head_gate=None, sink=None, value_gate=None, value_gate_stride=0):
+                        window=0, r1=None, r2=None, head_gate=None, sink=None, value_gate=None, value_gate_stride=0, slopes=None, chunk=0, out_scale=0.0):
         gr = (C.c_int32 * len(group_rows))(*group_rows)
-        x = AttentionExtras(cap, window, _vp(r1), _vp(r2), _vp(head_gate), _vp(sink), _vp(value_gate), value_gate_stride)
+        x = AttentionExtras(cap, window, _vp(r1), _vp(r2), _vp(head_gate), _vp(sink), _vp(value_gate), value_gate_stride,
+                            _vp(slopes), chunk, out_scale)
         self.check(lib().tsb_plain_attention(self.h, stream, kv.h, C.c_int32(layer), _vp(q), C.c_int64(q_stride), _vp(out), C.c_int64(out_stride),
                                              _vp(rows_dev), gr, C.c_int32(len(group_rows)), C.c_int32(n_q_heads), C.c_float(scale), C.byref(x),
                                              C.c_int32(max_len), _vp(scratch)))
@@ -413,7 +414,7 @@ class KvCache:
 
 class AttentionExtras(C.Structure):
     _fields_ = [("cap", C.c_float), ("window", C.c_int32)] + [(n, C.c_void_p) for n in ("r1", "r2", "head_gate", "sink", "value_gate")] + \
-               [("value_gate_stride", C.c_int64)]
+               [("value_gate_stride", C.c_int64), ("slopes", C.c_void_p), ("chunk", C.c_int32), ("out_scale", C.c_float)]
 
 
 class PlainCache(KvCache):

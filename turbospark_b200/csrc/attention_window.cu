@@ -101,7 +101,8 @@ __global__ void __launch_bounds__(F32_WARPS * 32) window_attn_f32_kernel(const _
     const float* q = reinterpret_cast<const float*>(a.q) + (int64_t)row * a.q_stride + (int64_t)head * D;
     for (int i = lane; i < D; i += 32) qs[warp][i] = q[i];
     __syncwarp();
-    const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+    const int lo = first_visible(a, pos);
+    const float slope = a.slopes ? a.slopes[head] : 0.f;
     const float r1 = a.r1 ? a.r1[head] : 0.f, r2 = a.r1 ? a.r2[head] : 0.f;
     // a sink is a score without a key or a value: it opens the sum
     float m = a.sink ? a.sink[head] : -INFINITY, l = a.sink ? 1.f : 0.f, acc[F32_MAX_DIM / 32];
@@ -124,6 +125,7 @@ __global__ void __launch_bounds__(F32_WARPS * 32) window_attn_f32_kernel(const _
             s = dot * a.scale;
             if (a.cap > 0.f) s = a.cap * tanhf(s / a.cap);
             if (a.r1) s -= r1 * logf(1.f + r2 * (float)(pos - j));
+            if (a.slopes) s -= slope * (float)(pos - j);
         }
         float mx = s;
 #pragma unroll
@@ -149,7 +151,7 @@ __global__ void __launch_bounds__(F32_WARPS * 32) window_attn_f32_kernel(const _
                 if (i * 32 + lane < DV) acc[i] = fmaf(pt, kt[i * 32 + lane], acc[i]);
         }
     }
-    const float f = (l > 0.f ? 1.f / l : 0.f) * (a.gate ? sigmoid(a.gate[(int64_t)row * a.n_q_heads + head]) : 1.f);
+    const float f = (l > 0.f ? a.out_scale / l : 0.f) * (a.gate ? sigmoid(a.gate[(int64_t)row * a.n_q_heads + head]) : 1.f);
     float* out = reinterpret_cast<float*>(a.out) + (int64_t)row * a.out_stride + (int64_t)head * DV;
     const float* vg = a.value_gate ? reinterpret_cast<const float*>(a.value_gate) + (int64_t)row * a.value_gate_stride + (int64_t)head * DV : nullptr;
 #pragma unroll

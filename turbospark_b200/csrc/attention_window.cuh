@@ -1,6 +1,6 @@
-// Attention over a plain paged cache - a layer's values are its keys, or stand behind them - with a sliding window, a soft cap
-// on the scores, a per-head logarithmic distance bias, a per-head sink, and output gates per head or per value column - each of
-// them optional.
+// Attention over a plain paged cache - a layer's values are its keys, or stand behind them - with a sliding window
+// or a chunk mask, a soft cap on the scores, a per-head logarithmic or linear distance bias, a per-head sink, and output gates per head
+// or per value column - each of them optional.
 #pragma once
 #include <cuda_bf16.h>
 
@@ -18,11 +18,14 @@ struct WindowAttn {
     float scale = 1.f;        // score = (q . k) * scale
     float cap = 0.f;          // > 0: score <- cap * tanh(score / cap)
     const float *r1 = nullptr, *r2 = nullptr;  // per head: score <- score - r1 * ln(1 + r2 * distance); null: no bias
+    const float* slopes = nullptr;             // per head: score <- score - slope * distance; null: no such bias (not with r1)
+    int chunk = 0;            // > 0: a query sees the positions of its own chunk (counted from position 0) up to itself; not with a window
     int window = 0;           // a query sees itself and the window - 1 positions before it; 0: every earlier position
     const float* sink = nullptr;  // per head: exp(sink) joins the softmax's denominator
     // [rows, n_q_heads * value columns], the compute type: a head's output is multiplied by the sigmoid, column by column
     const void* value_gate = nullptr;
     int64_t value_gate_stride = 0;
+    float out_scale = 1.f;    // of the heads' outputs
     int value_dim = 0;        // value columns (the heads of out and value_gate are as wide); 0: as many as a key has
 };
 

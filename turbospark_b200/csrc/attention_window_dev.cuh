@@ -31,7 +31,15 @@ __device__ __forceinline__ float head_factor(const WindowAttn& a, int row, int h
     if (a.sink) l += ex2(a.sink[head] * 1.4426950408889634f - (m == -INFINITY ? 0.f : m));
     float f = l > 0.f ? 1.f / l : 0.f;
     if (a.gate) f *= sigmoid(a.gate[(int64_t)row * a.n_q_heads + head]);
-    return f;
+    return f * a.out_scale;
+}
+// the earliest position that a query at `pos` sees
+__device__ __forceinline__ int first_visible(const WindowAttn& a, int pos) {
+    return a.window > 0 ? max(0, pos - a.window + 1) : a.chunk > 0 ? pos - pos % a.chunk : 0;
+}
+// how many positions, itself included, a query at `pos` sees at most (a number no distance reaches: all of them)
+__device__ __forceinline__ float visible_span(const WindowAttn& a, int pos) {
+    return a.window > 0 ? (float)a.window : a.chunk > 0 ? (float)(pos % a.chunk + 1) : 3e38f;
 }
 // the gate of value column c, and of four from c (a multiple of four) on
 __device__ __forceinline__ const __nv_bfloat16* value_gate_at(const WindowAttn& a, int row, int head, int c) {
@@ -130,7 +138,7 @@ inline int wattn_splits(const tsb_ctx* ctx, int window, const WattnLaunch& l, in
     return splits;
 }
 inline int wattn_splits(const tsb_ctx* ctx, const WindowAttn& a, const WattnLaunch& l, int tile_tokens, int queries_per_cta, int ctas_per_sm) {
-    return wattn_splits(ctx, a.window, l, tile_tokens, queries_per_cta, ctas_per_sm, l.n_tiles * a.keys.kv_heads, wattn_part_queries(ctx));
+    return wattn_splits(ctx, a.window > 0 ? a.window : a.chunk, l, tile_tokens, queries_per_cta, ctas_per_sm, l.n_tiles * a.keys.kv_heads, wattn_part_queries(ctx));
 }
 
 // Adds the runs of cut tiles, in order, and writes the finished rows.  A tile has `slots` query slots per run: row r of the

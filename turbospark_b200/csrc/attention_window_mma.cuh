@@ -39,10 +39,11 @@ struct Geo {
 
 // Raw scores of an mma accumulator tile -> base-2 logits with cap, bias and mask, and the lane's running maximum per query.
 // KEYS_M: rows of the tile are keys (16 per n) and columns queries; else rows are queries and columns keys (8 per n).
-// db[h]: distance of the lane's first key from its query h.
+// db[h]: distance of the lane's first key from its query h; span[h]: the distance from which on the query sees nothing.  A linear bias has its
+// slope, times log2(e), in r1.
 template <int N, bool KEYS_M>
 __device__ __forceinline__ void base2_logits(float (&s)[N][4], const WindowAttn& a, const ScoreConst& sc, const float (&db)[2], const float (&r1)[2],
-                                             const float (&r2)[2], bool edge, float (&mx)[2]) {
+                                             const float (&r2)[2], const float (&span)[2], bool edge, float (&mx)[2]) {
     if (a.cap > 0.f) {
         float big = 0.f;
 #pragma unroll
@@ -70,7 +71,6 @@ __device__ __forceinline__ void base2_logits(float (&s)[N][4], const WindowAttn&
 #pragma unroll
             for (int i = 0; i < 4; i++) s[n][i] *= sc.s_in;
     }
-    const float window = a.window > 0 ? (float)a.window : 3e38f;
 #pragma unroll
     for (int n = 0; n < N; n++)
 #pragma unroll
@@ -78,7 +78,8 @@ __device__ __forceinline__ void base2_logits(float (&s)[N][4], const WindowAttn&
             const int h = KEYS_M ? i & 1 : i >> 1;
             const float dist = db[h] - (float)(KEYS_M ? n * 16 + (i >> 1) * 8 : n * 8 + (i & 1));
             if (a.r1) s[n][i] = fmaf(-r1[h], lg2(fmaf(r2[h], dist, 1.f)), s[n][i]);
-            if (edge && (dist < 0.f || dist >= window)) s[n][i] = -INFINITY;
+            if (a.slopes) s[n][i] = fmaf(-r1[h], dist, s[n][i]);
+            if (edge && (dist < 0.f || dist >= span[h])) s[n][i] = -INFINITY;
             mx[h] = fmaxf(mx[h], s[n][i]);
         }
 }
@@ -191,8 +192,8 @@ __global__ void __launch_bounds__(32 * MT * SL, MT * SL <= 4 ? 3 : 1)
         return;
     }
     // visible positions of the tile's queries, in whole key tiles; this CTA's run of them
-    const int lo = a.window > 0 ? max(0, pos0 - a.window + 1) & ~(TOK - 1) : 0;
-    const int hi = pos0 + n_rows;
+    const int lo = first_visible(a, pos0) & ~(TOK - 1);
+    const int hi = pos0 + n_rows, lo_last = first_visible(a, hi - 1);
     const int total = (hi - lo + TOK - 1) / TOK;
     const int per = (total + n_splits - 1) / n_splits;
     const int t_first = min(total, (int)blockIdx.x * per), n_tiles = min(total, t_first + per) - t_first;
@@ -231,7 +232,7 @@ __global__ void __launch_bounds__(32 * MT * SL, MT * SL <= 4 ? 3 : 1)
     // the lane's two queries: rows gid and gid + 8 of its m-tile
     const __nv_bfloat16* qp[2];
     int pq[2];
-    float r1[2] = {0.f, 0.f}, r2[2] = {0.f, 0.f};
+    float r1[2] = {0.f, 0.f}, r2[2] = {0.f, 0.f}, span[2];
 #pragma unroll
     for (int h = 0; h < 2; h++) {
         const int qi = mt * 16 + gid + 8 * h;
@@ -240,6 +241,8 @@ __global__ void __launch_bounds__(32 * MT * SL, MT * SL <= 4 ? 3 : 1)
         pq[h] = pos0 + row;  // an empty slot repeats the first query and is not stored
         qp[h] = reinterpret_cast<const __nv_bfloat16*>(a.q) + (int64_t)(row_first + row) * a.q_stride + head * D;
         if (a.r1) r1[h] = a.r1[head], r2[h] = a.r2[head];
+        if (a.slopes) r1[h] = a.slopes[head] * 1.4426950408889634f;
+        span[h] = visible_span(a, pq[h]);
     }
     uint32_t qa[QREG ? KS : 1][4];
     const uint32_t q_smem = ring + NST * STAGE;
@@ -308,10 +311,10 @@ __global__ void __launch_bounds__(32 * MT * SL, MT * SL <= 4 ? 3 : 1)
             }
         }
         // the mask only where the tile meets an edge
-        const bool edge = p0 + WTOK > pos0 || (a.window > 0 && p0 <= pos0 + n_rows - 1 - a.window);
+        const bool edge = p0 + WTOK > pos0 || p0 < lo_last;
         float mx[2] = {-INFINITY, -INFINITY};
         const float db[2] = {(float)(pq[0] - p0 - 2 * tig), (float)(pq[1] - p0 - 2 * tig)};
-        base2_logits<NT8, false>(s, a, sc, db, r1, r2, edge, mx);
+        base2_logits<NT8, false>(s, a, sc, db, r1, r2, span, edge, mx);
         float alpha[2], m_use[2];
 #pragma unroll
         for (int h = 0; h < 2; h++) {
@@ -446,8 +449,8 @@ __global__ void __launch_bounds__(128, FewQ<D, NQ, KV>::PER_SM)
         return;
     }
     // key tiles start at multiples of 64 positions; this CTA's run of them
-    const int lo = a.window > 0 ? max(0, pos0 - a.window + 1) & ~63 : 0;
-    const int hi = pos0 + n_rows;
+    const int lo = first_visible(a, pos0) & ~63;
+    const int hi = pos0 + n_rows, lo_last = first_visible(a, hi - 1);
     const int total = (hi - lo + F::TILE - 1) / F::TILE;
     const int per = (total + n_splits - 1) / n_splits;
     const int t_first = min(total, (int)blockIdx.x * per), n_tiles = min(total, t_first + per) - t_first;
@@ -481,7 +484,7 @@ __global__ void __launch_bounds__(128, FewQ<D, NQ, KV>::PER_SM)
     if (early) prologue();
     // score columns of this lane: queries 2 tig and 2 tig + 1 of every query tile
     int pq[NQ][2];
-    float r1[NQ][2], r2[NQ][2];
+    float r1[NQ][2], r2[NQ][2], span[NQ][2];
 #pragma unroll
     for (int q = 0; q < NQ; q++)
 #pragma unroll
@@ -490,7 +493,8 @@ __global__ void __launch_bounds__(128, FewQ<D, NQ, KV>::PER_SM)
             const bool v = qi < n_queries;
             const int head = kvh * grp + (v ? qi % grp : 0);
             pq[q][h] = pos0 + (v ? qi / grp : 0);  // an empty slot repeats the first query and is not stored
-            r1[q][h] = a.r1 ? a.r1[head] : 0.f, r2[q][h] = a.r1 ? a.r2[head] : 0.f;
+            r1[q][h] = a.slopes ? a.slopes[head] * 1.4426950408889634f : a.r1 ? a.r1[head] : 0.f, r2[q][h] = a.r1 ? a.r2[head] : 0.f;
+            span[q][h] = visible_span(a, pq[q][h]);
         }
     pdl_wait();
     if (!early) prologue();
@@ -537,13 +541,13 @@ __global__ void __launch_bounds__(128, FewQ<D, NQ, KV>::PER_SM)
                 for (int q = 0; q < NQ; q++) mma_bf16(s[q][n], k, qb[q][ks][0], qb[q][ks][1]);
             }
         }
-        const bool edge = p0 + F::WTOK > pos0 || (a.window > 0 && p0 <= pos0 + n_rows - 1 - a.window);
+        const bool edge = p0 + F::WTOK > pos0 || p0 < lo_last;
         uint32_t pb[NQ][NK][2];
 #pragma unroll
         for (int q = 0; q < NQ; q++) {
             float mx[2] = {-INFINITY, -INFINITY};
             const float db[2] = {(float)(pq[q][0] - p0 - gid), (float)(pq[q][1] - p0 - gid)};
-            base2_logits<NK, true>(s[q], a, sc, db, r1[q], r2[q], edge, mx);
+            base2_logits<NK, true>(s[q], a, sc, db, r1[q], r2[q], span[q], edge, mx);
             float alpha[2], m_use[2];
 #pragma unroll
             for (int h = 0; h < 2; h++) {

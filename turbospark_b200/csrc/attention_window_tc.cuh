@@ -106,7 +106,7 @@ __global__ void __launch_bounds__(WT_THREADS, 1)
     if (!seq_ok) n_rows = 0;
     const int n_wg = n_rows > rows_wg ? 2 : 1;
     // visible positions, in key tiles that start at a copy box; this CTA's run of them
-    const int lo = a.window > 0 ? max(0, pos0 - a.window + 1) & ~(box_rows - 1) : 0;
+    const int lo = first_visible(a, pos0) & ~(box_rows - 1);
     const int hi = pos0 + n_rows;
     const int total = seq_ok ? (hi - lo + WT_TN - 1) / WT_TN : 0;
     const int per = (total + n_splits - 1) / n_splits;
@@ -241,6 +241,8 @@ __global__ void __launch_bounds__(WT_THREADS, 1)
             const uint32_t col_s = tmem + lane_base + WT_COL_S + (uint32_t)x * 128, col_o = tmem + lane_base + WT_COL_O + (uint32_t)x * DV;
             const bool capped = a.cap > 0.f, biased = Geo::TABLES && a.r1 != nullptr;
             const ScoreConst sc(a);
+            const float slope = a.slopes ? a.slopes[kvh * grp + min(head_l, grp - 1)] * 1.4426950408889634f : 0.f;
+            const int lo_last = first_visible(a, wg_last), lo_mine = first_visible(a, pq);
             // bias tables: entry k of a head holds the bias at distance wg_first - p0 + rows_wg - 1 - k; row_l's key j is entry
             // rows_wg - 1 - row_l + j.  The pitch keeps the 32 queries of a warp on different banks.
             const int need = rows_wg + WT_TN - 1;
@@ -299,8 +301,13 @@ __global__ void __launch_bounds__(WT_THREADS, 1)
                         for (int j = 0; j < WT_TN; j++) s[j] += bias[j];
                     }
                 }
-                if (p0 + WT_TN - 1 > wg_first || (a.window > 0 && wg_last - p0 >= a.window)) {  // the tile meets an edge of some row
-                    const int j_max = pq - p0, j_min = a.window > 0 ? j_max - a.window + 1 : -0x7fffffff;
+                if (a.slopes) {
+                    const float at0 = -slope * (float)(pq - p0);
+#pragma unroll
+                    for (int j = 0; j < WT_TN; j++) s[j] += fmaf(slope, (float)j, at0);
+                }
+                if (p0 + WT_TN - 1 > wg_first || p0 < lo_last) {  // the tile meets an edge of some row
+                    const int j_max = pq - p0, j_min = lo_mine - p0;
 #pragma unroll
                     for (int j = 0; j < WT_TN; j++)
                         if (j > j_max || j < j_min) s[j] = -INFINITY;

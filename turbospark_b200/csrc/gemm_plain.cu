@@ -99,6 +99,7 @@ __device__ __forceinline__ void epi_one(const PlainEpi& e, int t, int n, float v
             *y = fmaf(e.alpha, *y, v);
         }
     } else {
+        if (e.bias) v += e.bias[n];
         seg_put<T>(e, seg_at(e, n), t, v, err);
     }
 }
@@ -151,18 +152,26 @@ __device__ __forceinline__ uint4 ldg_stream(const void* p) {
 }
 
 // NT token tiles of eight, MT row tiles of sixteen.  WK warps split the columns of a row tile; products with few columns have
-// several row tiles per CTA instead.  blockIdx.y: which 8 NT tokens.
-template <int NT, int MT, int WK>
+// several row tiles per CTA instead.  blockIdx.y: which 8 NT tokens; EXPERTS: which chunk of slots.
+template <int NT, int MT, int WK, bool EXPERTS>
 __global__ void __launch_bounds__(FEW_WARPS * 32, 2)
     plain_few_kernel(const __nv_bfloat16* __restrict__ w, int cols, int group_rows, int group_cols, const __nv_bfloat16* x, const __nv_bfloat16* x2,
-                     int64_t x_stride, int tokens, const __grid_constant__ PlainEpi epi, uint32_t* __restrict__ err) {
+                     int64_t x_stride, int tokens, const __grid_constant__ PlainEpi epi, const __grid_constant__ PlainExperts ex, uint32_t* __restrict__ err) {
     constexpr int U = MT == 1 ? FEW_UNROLL : FEW_UNROLL / 2;
     constexpr int TOK = NT * 8, WROWS = MT * 16, ROWS = WROWS * (FEW_WARPS / WK);
     __shared__ float red[FEW_WARPS][WROWS][TOK + 1];
     const int warp = (threadIdx.x >> 5) % WK, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
     const int wrow = (threadIdx.x >> 5) / WK * WROWS, row0 = blockIdx.x * ROWS;
-    const int tok0 = blockIdx.y * TOK;
-    tokens = min(tokens - tok0, TOK);
+    int tok0 = blockIdx.y * TOK;
+    if (EXPERTS) {  // which rows of which matrix is known only now
+        pdl_wait();
+        if ((int)blockIdx.y >= *ex.n_chunks) return;
+        const ExpertChunk c = ex.chunks[blockIdx.y];
+        w += (int64_t)c.expert * gridDim.x * ROWS * cols;
+        tok0 = c.first, tokens = min(c.n, TOK);
+    } else {
+        tokens = min(tokens - tok0, TOK);
+    }
     const int units = cols / 64;
     const bool pairs = row0 >= epi.pair_row0;
     if (!tile_used(epi, row0, group_rows)) return;  // padding between the mixer's rows and the pairs, or behind a group
@@ -182,8 +191,14 @@ __global__ void __launch_bounds__(FEW_WARPS * 32, 2)
 #pragma unroll
     for (int i = 0; i < U; i++)
         if (warp + i * WK < units) load_w(i, warp + i * WK);  // weights do not depend on the preceding kernel
-    pdl_wait();
-    const __nv_bfloat16* xb = (pairs ? x2 : x) + (int64_t)(tok0 + g) * x_stride + 8 * t4 + (group_rows ? row0 / group_rows * group_cols : 0);
+    if (!EXPERTS) pdl_wait();
+    const __nv_bfloat16* xb = (pairs ? x2 : x) + 8 * t4 + (group_rows ? row0 / group_rows * group_cols : 0);
+    int64_t x_at[NT];
+#pragma unroll
+    for (int n = 0; n < NT; n++) {
+        const int t = tok0 + n * 8 + g;
+        x_at[n] = (EXPERTS && ex.token_of ? (n * 8 + g < tokens ? ex.token_of[t] : 0) : t) * x_stride;
+    }
     float acc[MT][NT][4];
 #pragma unroll
     for (int m = 0; m < MT; m++)
@@ -198,7 +213,7 @@ __global__ void __launch_bounds__(FEW_WARPS * 32, 2)
             if (u >= units) break;
 #pragma unroll
             for (int n = 0; n < NT; n++) {
-                const __nv_bfloat16* xp = xb + (int64_t)n * 8 * x_stride + (int64_t)u * 64;
+                const __nv_bfloat16* xp = xb + x_at[n] + (int64_t)u * 64;
                 uint4 b0 = make_uint4(0, 0, 0, 0), b1 = b0;
                 if (n * 8 + g < tokens) b0 = *reinterpret_cast<const uint4*>(xp), b1 = *reinterpret_cast<const uint4*>(xp + 32);
 #pragma unroll
@@ -253,22 +268,31 @@ __global__ void __launch_bounds__(FEW_WARPS * 32, 2)
 constexpr int F32_TILE = 64, F32_K = 16;
 // 256 threads, 64 rows x 64 tokens, 4 x 4 per thread.  A thread's four rows are {0, 8, 16, 24} + r within a 32-row half:
 // both halves of a gate / up pair are its own.
+template <bool EXPERTS>
 __global__ void __launch_bounds__(256)
     plain_f32_kernel(const float* __restrict__ w, int cols, int group_rows, int group_cols, const float* x, const float* x2, int64_t x_stride, int tokens,
-                     const __grid_constant__ PlainEpi epi, uint32_t* __restrict__ err) {
+                     const __grid_constant__ PlainEpi epi, const __grid_constant__ PlainExperts ex, uint32_t* __restrict__ err) {
     __shared__ float ws[F32_K][F32_TILE + 4], xs[F32_K][F32_TILE + 4];
-    const int row0 = blockIdx.x * F32_TILE, tok0 = blockIdx.y * F32_TILE;
+    const int row0 = blockIdx.x * F32_TILE;
+    int tok0 = blockIdx.y * F32_TILE;
     const bool pairs = row0 >= epi.pair_row0;
     const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
     const int rbase = (ty >> 3) * 32 + (ty & 7);
     pdl_wait();
+    if (EXPERTS) {
+        if ((int)blockIdx.y >= *ex.n_chunks) return;
+        const ExpertChunk c = ex.chunks[blockIdx.y];
+        w += (int64_t)c.expert * gridDim.x * F32_TILE * cols;
+        tok0 = c.first, tokens = c.first + min(c.n, F32_TILE);
+    }
     const float* xb = (pairs ? x2 : x) + (group_rows ? row0 / group_rows * group_cols : 0);
     float acc[4][4] = {};
     const int lr = threadIdx.x >> 2, lc = (threadIdx.x & 3) * 4;
+    const int64_t x_at = (EXPERTS && ex.token_of ? (tok0 + lr < tokens ? ex.token_of[tok0 + lr] : 0) : tok0 + lr) * x_stride;
     for (int k0 = 0; k0 < cols; k0 += F32_K) {
         const float4 a = *reinterpret_cast<const float4*>(w + (int64_t)(row0 + lr) * cols + k0 + lc);
         float4 b = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (tok0 + lr < tokens) b = *reinterpret_cast<const float4*>(xb + (int64_t)(tok0 + lr) * x_stride + k0 + lc);
+        if (tok0 + lr < tokens) b = *reinterpret_cast<const float4*>(xb + x_at + k0 + lc);
         ws[lc][lr] = a.x, ws[lc + 1][lr] = a.y, ws[lc + 2][lr] = a.z, ws[lc + 3][lr] = a.w;
         xs[lc][lr] = b.x, xs[lc + 1][lr] = b.y, xs[lc + 2][lr] = b.z, xs[lc + 3][lr] = b.w;
         __syncthreads();
@@ -331,6 +355,7 @@ __device__ __forceinline__ void tcg_g2s_2d(uint32_t dst_smem, const CUtensorMap*
 struct TcgOut {
     SegAt at;             // rows with a destination of their own
     bool pairs = false, cache = false, in = false;
+    float bias = 0.f;
     int tok0, pair = 0, head = 0, col = 0;  // head, col: of a rotated pair
     __device__ __forceinline__ TcgOut(const PlainEpi& e, int row0, int n, int lane, int tok0_) : tok0(tok0_) {
         pairs = row0 >= e.pair_row0;
@@ -339,6 +364,7 @@ struct TcgOut {
         } else if (!pairs) {
             at = seg_at(e, n);
             in = at.kind >= 0, cache = at.kind == PLAIN_SEG_CACHE;
+            if (e.bias && in) bias = e.bias[n];
         } else {
             pair = ((n & ~31) - e.pair_row0) / 2 + (lane >> 4) * 8 + (lane & 7);
             in = pair < e.n_pairs;
@@ -376,6 +402,10 @@ struct TcgOut {
                     if (j < left) y[j * step] = v[j];
             }
         } else if (!pairs) {
+            if (e.bias) {
+#pragma unroll
+                for (int j = 0; j < 16; j++) v[j] += bias;
+            }
             if (at.kind == PLAIN_SEG_F32) {
                 float* y = static_cast<float*>(at.p) + (int64_t)t0 * at.stride + at.col;
 #pragma unroll
@@ -447,18 +477,22 @@ private:
     }
 };
 
-// Work item i: token tile i % n_tok_tiles, then the K run, then the row tile - neighbouring CTAs share weight rows.
-template <int KIND>
+// Work item i: token tile i % n_tok_tiles, then the K run, then the row tile - neighbouring CTAs share weight rows.  EXPERTS: expert by
+// expert, with as many token tiles as its slots need; the counts are on the device.
+constexpr int TCG_EXPERT_BYTES = 2 * (EXPERTS_MAX + 2) * sizeof(int);  // behind the ring: first slots, first token tiles
+template <int KIND, bool EXPERTS>
 __global__ void __launch_bounds__(TCG_THREADS, 1)
     plain_tc_kernel(const __grid_constant__ CUtensorMap wmap, const __grid_constant__ CUtensorMap xmap, const __grid_constant__ CUtensorMap x2map,
                     int n_row_tiles, int n_tok_tiles, int units, int ksplit, int nt, int stages, int tokens, int group_rows, int group_cols,
-                    const __grid_constant__ PlainEpi epi, float* __restrict__ part, uint32_t* __restrict__ tickets, uint32_t* __restrict__ err) {
+                    const __grid_constant__ PlainEpi epi, const __grid_constant__ PlainExperts ex, float* __restrict__ part, uint32_t* __restrict__ tickets,
+                    uint32_t* __restrict__ err) {
     extern __shared__ __align__(1024) uint8_t smem[];
     TcgBars* bars = reinterpret_cast<TcgBars*>(smem);
     uint8_t* ring = smem + TCG_HEADER;
     const int stage_bytes = (TCG_M + nt) * 128;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int n_items = n_row_tiles * n_tok_tiles * ksplit;
+    int n_items = n_row_tiles * n_tok_tiles * ksplit;
+    int *slot0 = reinterpret_cast<int*>(ring + stages * stage_bytes), *tile0 = slot0 + EXPERTS_MAX + 2;
     const int run_units = (units + ksplit - 1) / ksplit;
     const uint32_t tmem_cols = nt <= 16 ? 32u : nt <= 32 ? 64u : nt <= 64 ? 128u : nt <= 128 ? 256u : 512u;
     if (threadIdx.x == 0) {
@@ -471,20 +505,55 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
         asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&bars->tmem_base)), "r"(tmem_cols) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
+    if (EXPERTS) {
+        pdl_wait();  // the lists come from the kernels before
+        for (int e = threadIdx.x; e <= ex.n; e += TCG_THREADS) slot0[e] = ex.first[e];
+        __syncthreads();
+        if (warp == 0) {
+            int sum = 0;
+            for (int e0 = 0; e0 < ex.n; e0 += 32) {
+                const int e = e0 + lane, n = e < ex.n ? (slot0[e + 1] - slot0[e] + nt - 1) / nt : 0;
+                int s = n;
+#pragma unroll
+                for (int o = 1; o < 32; o <<= 1) {
+                    const int v = __shfl_up_sync(0xffffffffu, s, o);
+                    if (lane >= o) s += v;
+                }
+                if (e < ex.n) tile0[e] = sum + s - n;
+                sum += __shfl_sync(0xffffffffu, s, 31);
+            }
+            if (lane == 0) tile0[ex.n] = sum;
+        }
+    }
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
     const uint32_t tmem = bars->tmem_base;
+    if (EXPERTS) n_items = tile0[ex.n] * n_row_tiles;
     struct Item {
-        int tok, run, row, u0, n;
+        int tok, run, row, u0, n, tok0, n_tok, wrow;  // wrow: row of the matrix behind the weight map
     };
     auto item_of = [&](int i) {
         Item it;
+        if (EXPERTS) {
+            int lo = 0, hi = ex.n;  // the last expert that starts at or before item i, empty ones skipped by the search's upper end
+            while (hi - lo > 1) {
+                const int mid = (lo + hi) >> 1;
+                if (tile0[mid] * n_row_tiles <= i) lo = mid;
+                else hi = mid;
+            }
+            const int tiles = tile0[lo + 1] - tile0[lo], j = i - tile0[lo] * n_row_tiles;
+            it.tok = j % tiles, it.row = j / tiles, it.run = 0, it.u0 = 0, it.n = units;
+            it.tok0 = slot0[lo] + it.tok * nt, it.n_tok = min(nt, slot0[lo + 1] - it.tok0);
+            it.wrow = (lo * n_row_tiles + it.row) * TCG_M;
+            return it;
+        }
         it.tok = i % n_tok_tiles;
         it.run = (i / n_tok_tiles) % ksplit;
         it.row = i / n_tok_tiles / ksplit;
         it.u0 = it.run * run_units;
         it.n = min(units, it.u0 + run_units) - it.u0;
+        it.tok0 = it.tok * nt, it.n_tok = min(nt, tokens - it.tok0), it.wrow = it.row * TCG_M;
         return it;
     };
 
@@ -496,15 +565,15 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
             uint32_t it = 0;
             int early = 0;  // stages whose weight slice was fetched ahead
             const bool has_work = (int)blockIdx.x < n_items;
-            if (has_work) {
+            if (has_work && !EXPERTS) {
                 const Item w0 = item_of(blockIdx.x);
                 early = min(stages, w0.n);
                 for (int s = 0; s < early; s++) {
                     mbar_expect_tx(&bars->full[s], (uint32_t)stage_bytes);
-                    tcg_g2s_2d(smem_u32(ring + s * stage_bytes), &wmap, (w0.u0 + s) * TCG_K, w0.row * TCG_M, &bars->full[s]);
+                    tcg_g2s_2d(smem_u32(ring + s * stage_bytes), &wmap, (w0.u0 + s) * TCG_K, w0.wrow, &bars->full[s]);
                 }
             }
-            pdl_wait();
+            if (!EXPERTS) pdl_wait();
             for (int i = blockIdx.x; i < n_items && ok; i += gridDim.x) {
                 const Item w = item_of(i);
                 const CUtensorMap* xm = w.row * TCG_M >= epi.pair_row0 ? &x2map : &xmap;
@@ -516,9 +585,9 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
                         if ((int)it >= stages) ok = mbar_wait(&bars->empty[s], ((it / stages) - 1) & 1, err);
                         if (!ok) break;
                         mbar_expect_tx(&bars->full[s], (uint32_t)stage_bytes);
-                        tcg_g2s_2d(dst, &wmap, (w.u0 + u) * TCG_K, w.row * TCG_M, &bars->full[s]);
+                        tcg_g2s_2d(dst, &wmap, (w.u0 + u) * TCG_K, w.wrow, &bars->full[s]);
                     }
-                    tcg_g2s_2d(dst + TCG_M * 128, xm, x_col0 + (w.u0 + u) * TCG_K, w.tok * nt, &bars->full[s]);
+                    tcg_g2s_2d(dst + TCG_M * 128, xm, x_col0 + (w.u0 + u) * TCG_K, w.tok0, &bars->full[s]);
                 }
             }
             if (!ok) bars->failed = 1;
@@ -560,7 +629,7 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
     } else {
         // ---- epilogue: two threads per weight row of the tile, columns = tokens.  One destination per tile and thread, one short
         // loop per kind of destination: the code of a kind has to stay in the instruction cache.
-        pdl_wait();  // the residual stream and the cache belong to earlier kernels too
+        if (!EXPERTS) pdl_wait();  // the residual stream and the cache belong to earlier kernels too
         bool ok = true;
         uint32_t tile = 0;
         const int quad = warp & 3, first16 = (warp >> 2) * 16;
@@ -572,7 +641,7 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
             tc_fence_after();
             const uint32_t src = tmem + lane_base + buf * (uint32_t)nt;
             const int n = w.row * TCG_M + quad * 32 + lane;
-            const int tok0 = w.tok * nt, n_tok = min(nt, tokens - tok0);
+            const int tok0 = w.tok0, n_tok = w.n_tok;
             bool finish = ok;
             const float* all = nullptr;
             if (ksplit > 1) {
@@ -729,8 +798,22 @@ cudaError_t launch_few(tsb_ctx* ctx, cudaStream_t st, const PlainMat& w, const _
     // last attention CTAs are packed on few SMs and run with their small L1 - 67 to 75 us instead of 27 at 4096 x 18432.
     const bool ahead = epi.kind != PLAIN_ADD;
     const dim3 grid((unsigned)(w.rows / (16 * MT * (FEW_WARPS / WK))), (unsigned)((tokens + 8 * NT - 1) / (8 * NT)));
-    return tsb_launch(ctx, plain_few_kernel<NT, MT, WK>, grid, dim3(FEW_WARPS * 32), 0, st, ahead,
-                      (const __nv_bfloat16*)w.data, (int)w.cols, w.group_rows, w.group_cols, x, x2, x_stride, tokens, epi, ctx->dev_error);
+    return tsb_launch(ctx, plain_few_kernel<NT, MT, WK, false>, grid, dim3(FEW_WARPS * 32), 0, st, ahead,
+                      (const __nv_bfloat16*)w.data, (int)w.cols, w.group_rows, w.group_cols, x, x2, x_stride, tokens, epi, PlainExperts{}, ctx->dev_error);
+}
+template <int NT, int WK>
+cudaError_t launch_few_experts(tsb_ctx* ctx, cudaStream_t st, const PlainMat& w, const __nv_bfloat16* x, int64_t x_stride, const PlainExperts& ex, const PlainEpi& epi) {
+    const dim3 grid((unsigned)(w.rows / (16 * (FEW_WARPS / WK))), (unsigned)expert_chunks_max(ex.slots, ex.n, ex.chunk_slots));
+    return tsb_launch(ctx, plain_few_kernel<NT, 1, WK, true>, grid, dim3(FEW_WARPS * 32), 0, st, true, (const __nv_bfloat16*)w.data, (int)w.cols, 0, 0, x, x, x_stride,
+                      0, epi, ex, ctx->dev_error);
+}
+template <int NT>
+cudaError_t launch_few_experts_any(tsb_ctx* ctx, cudaStream_t st, const PlainMat& w, const __nv_bfloat16* x, int64_t x_stride, const PlainExperts& ex, const PlainEpi& epi) {
+    const int units = (int)(w.cols / TCG_K);
+    if (units == 1) return launch_few_experts<NT, 1>(ctx, st, w, x, x_stride, ex, epi);
+    if (units < 4) return launch_few_experts<NT, 2>(ctx, st, w, x, x_stride, ex, epi);
+    if (units < 8) return launch_few_experts<NT, 4>(ctx, st, w, x, x_stride, ex, epi);
+    return launch_few_experts<NT, 8>(ctx, st, w, x, x_stride, ex, epi);
 }
 
 constexpr int FEW_MAX = 16;  // token rows up to which the weight-streaming kernel runs
@@ -762,8 +845,8 @@ cudaError_t launch_plain_gemm(tsb_ctx* ctx, cudaStream_t st, bool f32, const Pla
     if (tokens <= 0) return cudaSuccess;
     if (f32) {
         dim3 grid((unsigned)(w.rows / F32_TILE), (unsigned)((tokens + F32_TILE - 1) / F32_TILE));
-        return tsb_launch(ctx, plain_f32_kernel, grid, dim3(256), 0, st, true, (const float*)w.data, (int)w.cols, w.group_rows, w.group_cols,
-                          (const float*)x, (const float*)x2, x_stride, tokens, epi, ctx->dev_error);
+        return tsb_launch(ctx, plain_f32_kernel<false>, grid, dim3(256), 0, st, true, (const float*)w.data, (int)w.cols, w.group_rows, w.group_cols,
+                          (const float*)x, (const float*)x2, x_stride, tokens, epi, PlainExperts{}, ctx->dev_error);
     }
     const __nv_bfloat16 *xb = (const __nv_bfloat16*)x, *xb2 = (const __nv_bfloat16*)x2;
     if (tokens <= FEW_MAX || (tokens <= FEW_SHORT_MAX && w.cols <= FEW_SHORT_UNITS * TCG_K && w.rows * w.cols * 2 * ((tokens + 15) / 16) <= FEW_SHORT_BYTES))
@@ -784,10 +867,39 @@ cudaError_t launch_plain_gemm(tsb_ctx* ctx, cudaStream_t st, bool f32, const Pla
     auto run = [&](auto kernel, SmemOptIn& configured) {
         if (cudaError_t r = tsb_opt_in_smem(ctx, kernel, (size_t)TCG_SMEM_CAP, configured); r != cudaSuccess) return r;
         return tsb_launch(ctx, kernel, dim3((unsigned)std::min(items, ctx->sm_count)), dim3(TCG_THREADS), smem, st, true, wm, xm, xm2, row_tiles, tok_tiles,
-                          units, p.ksplit, p.nt, p.stages, tokens, w.group_rows, w.group_cols, epi, part, tickets, ctx->dev_error);
+                          units, p.ksplit, p.nt, p.stages, tokens, w.group_rows, w.group_cols, epi, PlainExperts{}, part, tickets, ctx->dev_error);
     };
     static SmemOptIn configured[3];
-    if (epi.kind == PLAIN_STORE) return run(plain_tc_kernel<PLAIN_STORE>, configured[0]);
-    if (epi.kind == PLAIN_ADD) return run(plain_tc_kernel<PLAIN_ADD>, configured[1]);
-    return run(plain_tc_kernel<PLAIN_MIXER>, configured[2]);
+    if (epi.kind == PLAIN_STORE) return run(plain_tc_kernel<PLAIN_STORE, false>, configured[0]);
+    if (epi.kind == PLAIN_ADD) return run(plain_tc_kernel<PLAIN_ADD, false>, configured[1]);
+    return run(plain_tc_kernel<PLAIN_MIXER, false>, configured[2]);
+}
+
+cudaError_t launch_plain_gemm_experts(tsb_ctx* ctx, cudaStream_t st, bool f32, bool tensor, const PlainMat& w, const void* x, int64_t x_stride, int x_rows,
+                                      const PlainExperts& ex, const PlainEpi& epi) {
+    if (ex.slots <= 0) return cudaSuccess;
+    if (ex.n > EXPERTS_MAX || epi.kind != PLAIN_MIXER) return cudaErrorInvalidValue;
+    if (f32) {
+        const dim3 grid((unsigned)(w.rows / F32_TILE), (unsigned)expert_chunks_max(ex.slots, ex.n, ex.chunk_slots));
+        return tsb_launch(ctx, plain_f32_kernel<true>, grid, dim3(256), 0, st, true, (const float*)w.data, (int)w.cols, 0, 0, (const float*)x, (const float*)x, x_stride, 0,
+                          epi, ex, ctx->dev_error);
+    }
+    const __nv_bfloat16* xb = (const __nv_bfloat16*)x;
+    if (!tensor)
+        return ex.chunk_slots <= 8 ? launch_few_experts_any<1>(ctx, st, w, xb, x_stride, ex, epi) : launch_few_experts_any<2>(ctx, st, w, xb, x_stride, ex, epi);
+    if (ex.token_of) return cudaErrorInvalidValue;
+    const int row_tiles = (int)(w.rows / TCG_M), units = (int)(w.cols / TCG_K);
+    int nt = 32;  // a tile that holds an expert's slots when they are spread evenly, with some room
+    while (nt < TCG_NMAX && nt < ex.slots / ex.n * 5 / 4) nt *= 2;
+    const int stages = std::min(TCG_MAX_STAGES, (TCG_SMEM_CAP - TCG_HEADER - TCG_EXPERT_BYTES) / ((TCG_M + nt) * 128));
+    CUtensorMap wm, xm;
+    cudaError_t e = tcg_map(w.data, w.rows * ex.n, w.cols, w.cols, TCG_M, &wm);
+    if (e == cudaSuccess) e = tcg_map(x, x_rows, w.cols, x_stride, nt, &xm);
+    if (e != cudaSuccess) return e;
+    const size_t smem = TCG_HEADER + (size_t)stages * (TCG_M + nt) * 128 + TCG_EXPERT_BYTES;
+    static SmemOptIn configured;
+    if ((e = tsb_opt_in_smem(ctx, plain_tc_kernel<PLAIN_MIXER, true>, (size_t)TCG_SMEM_CAP, configured)) != cudaSuccess) return e;
+    const int64_t items = (int64_t)(ex.slots / nt + std::min(ex.n, ex.slots)) * row_tiles;
+    return tsb_launch(ctx, plain_tc_kernel<PLAIN_MIXER, true>, dim3((unsigned)std::min<int64_t>(items, ctx->sm_count)), dim3(TCG_THREADS), smem, st, true, wm, xm, xm,
+                      row_tiles, 1, units, 1, nt, stages, 0, 0, 0, epi, ex, (float*)nullptr, (uint32_t*)nullptr, ctx->dev_error);
 }

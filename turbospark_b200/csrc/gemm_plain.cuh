@@ -4,6 +4,7 @@
 #include <cuda_bf16.h>
 
 #include "common.cuh"
+#include "experts.cuh"
 #include "kv.cuh"
 
 // Weight matrices are packed for the kernels when they are uploaded: rows padded with zero rows to a multiple of
@@ -59,6 +60,7 @@ struct PlainEpi {
     // PLAIN_MIXER
     PlainSeg seg[PLAIN_SEGS];
     int n_seg = 0;
+    const float* bias = nullptr;  // per row of the matrix, added to the rows of segments; null: none
     KeyView keys{};
     const tsb_row_desc* rows = nullptr;
     PlainRotate rot;             // half > 0: the pairs are rotated coordinates
@@ -76,9 +78,25 @@ struct PlainMat {
     int group_rows = 0, group_cols = 0;
 };
 
+// A product per expert: the matrix holds n matrices of w.rows rows one after another, and the slots of an expert (experts.cuh) multiply its
+// own.  Output rows are slots.
+struct PlainExperts {
+    int n = 0, slots = 0;
+    const int32_t* first = nullptr;      // [n + 1]
+    const int32_t* token_of = nullptr;   // row of x of a slot; null: x has a row per slot
+    const ExpertChunk* chunks = nullptr;
+    const int32_t* n_chunks = nullptr;
+    int chunk_slots = 0;
+};
+
 // Split sums of products with few row tiles: tickets, then f32 tiles.
 size_t plain_gemm_workspace_bytes(const tsb_ctx* ctx);
 // Rows of the matrix below epi.pair_row0 multiply x, the others x2; both have x_rows allocated rows of x_stride elements
 // (x_rows * x_stride elements are readable, and finite rows past `tokens` are not needed).
 cudaError_t launch_plain_gemm(tsb_ctx* ctx, cudaStream_t st, bool f32, const PlainMat& w, const void* x, const void* x2, int64_t x_stride, int x_rows,
                               int tokens, const PlainEpi& epi, void* workspace);
+// Slots by expert; x_rows, x_stride as above, epi.kind PLAIN_MIXER.  tensor: on the tensor-memory kernel (bfloat16, x by slots); else chunks
+// of at most EXPERT_CHUNK_FEW (bfloat16) or EXPERT_CHUNK_F32 slots.
+constexpr int EXPERT_CHUNK_FEW = 16, EXPERT_CHUNK_F32 = 64;
+cudaError_t launch_plain_gemm_experts(tsb_ctx* ctx, cudaStream_t st, bool f32, bool tensor, const PlainMat& w, const void* x, int64_t x_stride, int x_rows,
+                                      const PlainExperts& ex, const PlainEpi& epi);

@@ -199,13 +199,13 @@ int32_t kv_create_keys(tsb_ctx* ctx, int n_layers, const KeyLayerShape* shapes, 
     auto row_of = [&](int l) { return shapes[l].kv_heads * (shapes[l].head_dim + shapes[l].value_dim); };
     for (int l = 0; l < n_layers && rc == TSB_OK; l++) {
         const KeyLayerShape& k = shapes[l];
-        if (k.kv_heads <= 0 || k.head_dim <= 0 || k.value_dim < 0 || (k.head_dim * elem_bytes) % 16 || (k.value_dim * elem_bytes) % 16)
+        if (k.kv_heads < 0 || (k.kv_heads > 0 && k.head_dim <= 0) || k.value_dim < 0 || (k.head_dim * elem_bytes) % 16 || (k.value_dim * elem_bytes) % 16)
             rc = tsb_fail(ctx, TSB_ERR_INVALID, "layer %d: bad head count or head size", l);
         else if (k.source < 0 || k.source > l || shapes[k.source].source != k.source || row_of(k.source) != row_of(l))
             rc = tsb_fail(ctx, TSB_ERR_INVALID, "layer %d cannot read the rows of layer %d", l, k.source);
         if (k.source == l) bytes += (size_t)num_pages * page_tokens * row_of(l) * elem_bytes;
     }
-    if (rc == TSB_OK) rc = pool_alloc(ctx, bytes, (void**)&kv->key_pool);
+    if (rc == TSB_OK) rc = pool_alloc(ctx, std::max<size_t>(bytes, 16), (void**)&kv->key_pool);
     if (rc) {
         tsb_kv_destroy(kv);
         return rc;
@@ -232,7 +232,7 @@ int32_t kv_fill_keys(tsb_kv* kv, cudaStream_t st, int32_t seq, int64_t tokens, u
     if (rc) return rc;
     DeviceGuard g(kv->ctx);
     for (size_t l = 0; l < kv->key_layers.size(); l++)
-        TSB_CUDA(kv->ctx, tsb_launch(kv->ctx, keys_fill_random_kernel, dim3((unsigned)(kv->ctx->sm_count * 4)), dim3(256), 0, st, false, kv->key_layers[l],
+        if (kv->key_layers[l].row > 0) TSB_CUDA(kv->ctx, tsb_launch(kv->ctx, keys_fill_random_kernel, dim3((unsigned)(kv->ctx->sm_count * 4)), dim3(256), 0, st, false, kv->key_layers[l],
                                      (int)seq, (int)tokens, (uint32_t)(seed * 1000003u + l)));
     return TSB_OK;
 }

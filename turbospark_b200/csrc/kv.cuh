@@ -31,7 +31,7 @@ struct KeyView {
     int page_shift, page_tokens, num_pages, max_seqs, max_pages_per_seq;
 };
 struct KeyLayerShape {
-    int kv_heads, head_dim;
+    int kv_heads, head_dim;  // no heads: the layer has no rows
     int value_dim; // elements of the value behind every key (0: the values are the keys)
     int source;    // the layer whose rows this one reads (itself: rows of its own)
 };

@@ -16,6 +16,10 @@
 //                                and the shared key part in f32 and stores the latter in the cache; norm of the latent into the cache; then
 //                                short portions: absorb (queries to the latent's space), attention over latent rows, lift (sums of
 //                                latents to gated values); long portions: expansion of the stream's latents to keys and values, attention
+// In output-norm form a sublayer reads the stream through a short convolution, and its output is normed and added by one kernel that also
+// makes the next sublayer's input (launch_sublayer_end); the stream goes back and forth between two buffers.  Mixers: attention over keys
+// and values, a recurrence (recurrence.cuh), or both side by side - one input matmul, one output matmul over [heads | recurrence].
+// Routed feed-forwards: router matmul, choice and lists, a grouped product each for gate-up pairs and down.
 #include <algorithm>
 #include <cstring>
 #include <functional>
@@ -77,27 +81,40 @@ void convert(const void* host, int host_type, int64_t n, bool f32, std::vector<u
 int32_t plain_complete(const tsb_model* tm) {
     tsb_ctx* ctx = tm->ctx;
     const PlainModel* m = tm->plain;
-    const uint32_t want = 1u << TSB_P_EMBED | 1u << TSB_P_HEAD | 1u << TSB_P_FINAL_NORM;
+    uint64_t want = 1ull << TSB_P_EMBED | 1ull << TSB_P_HEAD | 1ull << TSB_P_FINAL_NORM;
+    if (m->cfg.positions > 0) want |= 1ull << TSB_P_POSITIONS;
     TSB_REQUIRE(ctx, (m->set & want) == want, "embedding, head or final norm missing");
     for (size_t i = 0; i < m->layers.size(); i++) {
         const PlainLayer& l = m->layers[i];
-        uint32_t w = 1u << TSB_P_NORM | 1u << TSB_P_Q | 1u << TSB_P_O;
-        if (l.mixer == MIX_LATENT) {
-            w |= 1u << TSB_P_UK | 1u << TSB_P_UV;
-            if (l.source == (int)i) w |= 1u << TSB_P_DKV | 1u << TSB_P_DKV_NORM;
-        } else {
-            w |= 1u << TSB_P_K;
-        }
-        if (l.mixer == MIX_KV) w |= 1u << TSB_P_V;
-        if (l.cfg.qk_norm) w |= 1u << TSB_P_Q_NORM | 1u << TSB_P_K_NORM;
-        if (l.cfg.sink) w |= 1u << TSB_P_SINK;
-        if (l.cfg.value_gate) w |= 1u << TSB_P_VALUE_GATE;
-        if (l.cfg.token_shift) w |= 1u << TSB_P_SHIFT;
-        if (l.cfg.head_gate) w |= 1u << TSB_P_HEAD_GATE;
-        if (l.cfg.log_bias) w |= 1u << TSB_P_R1 | 1u << TSB_P_R2;
-        if (l.cfg.ffn > 0) w |= 1u << TSB_P_FF_GATE | 1u << TSB_P_FF_UP | 1u << TSB_P_FF_DOWN;
-        if (l.cfg.ffn > 0 && l.post_norm) w |= 1u << TSB_P_NORM2;
-        TSB_REQUIRE(ctx, (l.set & w) == w, "layer %zu is missing a tensor (have %x, need %x)", i, l.set, w);
+        uint64_t w = 1ull << TSB_P_NORM;
+        auto need = [&](bool on, std::initializer_list<int> ids) {
+            for (int id : ids)
+                if (on) w |= 1ull << id;
+        };
+        const int rec = l.cfg.recurrence;
+        need(l.mixer != MIX_NONE, {TSB_P_Q, TSB_P_O});
+        need(l.mixer == MIX_LATENT, {TSB_P_UK, TSB_P_UV});
+        need(l.mixer == MIX_LATENT && l.source == (int)i, {TSB_P_DKV, TSB_P_DKV_NORM});
+        need(l.mixer == MIX_KEYS || l.mixer == MIX_KV, {TSB_P_K});
+        need(l.mixer == MIX_KV, {TSB_P_V});
+        need(l.cfg.qk_norm, {TSB_P_Q_NORM, TSB_P_K_NORM});
+        need(l.cfg.qkv_bias, {TSB_P_Q_BIAS, TSB_P_K_BIAS, TSB_P_V_BIAS});
+        need(l.cfg.sink, {TSB_P_SINK});
+        need(l.cfg.value_gate, {TSB_P_VALUE_GATE});
+        need(l.cfg.token_shift, {TSB_P_SHIFT});
+        need(l.cfg.head_gate, {TSB_P_HEAD_GATE});
+        need(l.cfg.log_bias, {TSB_P_R1, TSB_P_R2});
+        need(rec, {TSB_P_REC_NORM, TSB_P_REC_O});
+        need(rec == TSB_REC_FORGET || rec == TSB_REC_MLSTM, {TSB_P_REC_Q, TSB_P_REC_V, TSB_P_REC_F, TSB_P_REC_F_BIAS});
+        need(rec == TSB_REC_FORGET, {TSB_P_REC_LOWER});
+        need(rec == TSB_REC_MLSTM, {TSB_P_REC_K, TSB_P_REC_GATE, TSB_P_REC_I, TSB_P_REC_I_BIAS});
+        need(rec == TSB_REC_SSD, {TSB_P_REC_IN, TSB_P_REC_CONV, TSB_P_REC_CONV_BIAS, TSB_P_REC_DT_BIAS, TSB_P_REC_A_LOG, TSB_P_REC_D});
+        need(m->cfg.conv_taps > 0, {TSB_P_CONV1});
+        need(m->cfg.conv_taps > 0 && l.cfg.ffn > 0, {TSB_P_CONV2});
+        need(l.cfg.ffn > 0, {TSB_P_FF_GATE, TSB_P_FF_UP, TSB_P_FF_DOWN});
+        need(l.cfg.ffn > 0 && l.post_norm, {TSB_P_NORM2});
+        need(l.cfg.experts > 0, {TSB_P_ROUTER, TSB_P_CORRECTION});
+        TSB_REQUIRE(ctx, (l.set & w) == w, "layer %zu is missing a tensor (have %llx, need %llx)", i, (unsigned long long)l.set, (unsigned long long)w);
     }
     return TSB_OK;
 }
@@ -116,21 +133,33 @@ void plain_free(tsb_model* tm) {
     for (PlainRotation& r : m->rotations)
         if (r.freq) tsb_free(ctx, r.freq);
     if (m->owned)
-        for (void* p : {m->head.data, m->embed, (void*)m->final_gain})
+        for (void* p : {m->head.data, m->embed, m->positions, (void*)m->final_gain})
             if (p) tsb_free(ctx, p);
     delete m;
     tm->plain = nullptr;
 }
 
-// numbers of a layer's matrices that a pass over few rows reads
+// rows of a recurrence in the input matrix: vectors in the compute type, gates in f32
+int64_t rec_typed_rows(const tsb_plain_layer& c) {
+    const int64_t h = c.rec_heads, D = c.rec_dim, E = c.rec_vdim;
+    return c.recurrence == TSB_REC_FORGET ? h * (D + E) : c.recurrence == TSB_REC_MLSTM ? 2 * h * (D + E) : c.recurrence == TSB_REC_SSD ? 2 * h * E + 2 * c.rec_groups * D : 0;
+}
+int64_t rec_gate_rows(const tsb_plain_layer& c) {
+    const int64_t h = c.rec_heads;
+    return c.recurrence == TSB_REC_FORGET ? h * c.rec_dim : c.recurrence == TSB_REC_MLSTM ? 2 * h : c.recurrence == TSB_REC_SSD ? h : 0;
+}
+int64_t rec_conv_channels(const tsb_plain_layer& c) { return c.recurrence == TSB_REC_SSD ? (int64_t)c.rec_heads * c.rec_vdim + 2 * (int64_t)c.rec_groups * c.rec_dim : 0; }
+// numbers of a layer's matrices that a pass over one row reads
 int64_t layer_numbers(const PlainLayer& l, int64_t d) {
     const tsb_plain_layer& c = l.cfg;
     const int64_t H = c.n_q_heads, G = c.n_kv_heads, D = c.head_dim, E = l.mixer == MIX_KEYS ? D : c.value_dim;
-    int64_t n = d * (H * E + (c.head_gate ? H : 0) + (c.value_gate ? H * E : 0) + 3 * (int64_t)c.ffn);
+    int64_t n = d * (H * E + (c.head_gate ? H : 0) + (c.value_gate ? H * E : 0));
+    n += c.experts > 0 ? d * (c.experts + 3 * (int64_t)c.ffn * c.expert_top) : d * 3 * (int64_t)c.ffn;
+    n += d * (rec_typed_rows(c) + rec_gate_rows(c) + (c.recurrence ? (int64_t)c.rec_heads * c.rec_vdim : 0));
     if (l.mixer == MIX_LATENT) {
         n += d * H * (D + c.rot_dim) + (int64_t)c.kv_rank * H * (D + E);
         if (c.kv_source == 0) n += d * (c.kv_rank + c.rot_dim);
-    } else {
+    } else if (l.mixer != MIX_NONE) {
         n += d * (H * D + G * D + (l.mixer == MIX_KV ? G * E : 0));
     }
     return n;
@@ -147,13 +176,14 @@ int32_t plain_share(tsb_model* dt, int32_t dst_layer, const tsb_model* st, int32
     tsb_ctx* ctx = dt->ctx;
     PlainModel* d = dt->plain;
     const PlainModel* s = st->plain;
-    TSB_REQUIRE(ctx, d->cfg.d_model == s->cfg.d_model && d->cfg.vocab == s->cfg.vocab && d->f32 == s->f32 && d->cfg.post_norm == s->cfg.post_norm,
+    TSB_REQUIRE(ctx, d->cfg.d_model == s->cfg.d_model && d->cfg.vocab == s->cfg.vocab && d->f32 == s->f32 && d->cfg.post_norm == s->cfg.post_norm &&
+                         d->cfg.output_norm == s->cfg.output_norm && d->cfg.conv_taps == s->cfg.conv_taps && d->cfg.positions == s->cfg.positions,
                 "models differ in width, vocabulary, type or form");
     if (dst_layer < 0) {
         if (d->owned)
-            for (void* p : {d->head.data, d->embed, (void*)d->final_gain})
+            for (void* p : {d->head.data, d->embed, d->positions, (void*)d->final_gain})
                 if (p) tsb_free(ctx, p);
-        d->head = s->head, d->embed = s->embed, d->final_gain = s->final_gain, d->set = s->set, d->owned = false;
+        d->head = s->head, d->embed = s->embed, d->positions = s->positions, d->final_gain = s->final_gain, d->set = s->set, d->owned = false;
         return TSB_OK;
     }
     TSB_REQUIRE(ctx, dst_layer < d->cfg.n_layers && src_layer >= 0 && src_layer < s->cfg.n_layers, "layer out of range");
@@ -172,6 +202,57 @@ void plain_runtime_free(ModelRt& rt) {
     rt.plain = nullptr;
 }
 
+// Rings of the convolutions and states of the recurrences.  A cursor may go back by max_rows rows after a pass of as many, so the states of
+// max_rows + 1 positions are kept, and the convolutions' inputs as far back as the oldest of them looks.
+int32_t states_init(tsb_session* s, const PlainModel* m, const SessionShape& shape, StreamStates& st) {
+    tsb_ctx* ctx = s->ctx;
+    auto zero = [&](size_t bytes, void** q) -> int32_t {
+        if (bytes == 0) return TSB_OK;
+        if (int32_t rc = dev_alloc(ctx, s->owned, bytes, q)) return rc;
+        TSB_CUDA(ctx, cudaMemset(*q, 0, bytes));
+        return TSB_OK;
+    };
+    bool any = m->cfg.conv_taps > 1;
+    st.keep = std::max(0, m->cfg.conv_taps - 1);
+    for (const PlainLayer& l : m->layers)
+        if (l.cfg.recurrence) any = true, st.keep = std::max(st.keep, l.cfg.rec_taps - 1);
+    if (!any) return TSB_OK;
+    for (st.ring = 2; st.ring < shape.max_rows + 1;) st.ring *= 2;
+    for (st.row_ring = 2; st.row_ring < st.ring + st.keep;) st.row_ring *= 2;
+    std::vector<RowRing> rings;
+    int32_t rc = TSB_OK;
+    auto ring = [&](std::vector<RowRing>& list, int64_t width, int taps) {
+        RowRing r;
+        r.width = (int)width, r.ring_rows = st.row_ring, r.keep = std::max(0, taps - 1), r.n_streams = shape.n_streams;
+        if (width > 0 && r.keep > 0 && rc == TSB_OK) {
+            const size_t row = (size_t)shape.n_streams * width * 4;
+            rc = zero(row * r.ring_rows, (void**)&r.ring);
+            if (rc == TSB_OK) rc = zero(row * r.keep, (void**)&r.before);
+            rings.push_back(r);
+        }
+        list.push_back(r);
+    };
+    for (const PlainLayer& l : m->layers) {
+        const tsb_plain_layer& c = l.cfg;
+        ring(st.conv1, m->cfg.d_model, m->cfg.conv_taps);
+        ring(st.conv2, c.ffn > 0 ? m->cfg.d_model : 0, m->cfg.conv_taps);
+        ring(st.rec, rec_conv_channels(c), c.rec_taps);
+        RecurrentState r;
+        r.ring = st.ring, r.n_streams = shape.n_streams;
+        const size_t heads = (size_t)shape.n_streams * st.ring * c.rec_heads;
+        if (c.recurrence && rc == TSB_OK) rc = zero(heads * c.rec_dim * recurrence_v_pitch(c.rec_vdim) * 4, (void**)&r.s);
+        if (c.recurrence == TSB_REC_MLSTM && rc == TSB_OK) rc = zero(heads * c.rec_dim * 4, (void**)&r.norm);
+        if (c.recurrence == TSB_REC_MLSTM && rc == TSB_OK) rc = zero(heads * 4, (void**)&r.top);
+        st.states.push_back(r);
+    }
+    if (rc) return rc;
+    st.n_rings = (int)rings.size();
+    if (st.n_rings == 0) return TSB_OK;
+    if ((rc = zero(rings.size() * sizeof(RowRing), (void**)&st.rings_dev))) return rc;
+    TSB_CUDA(ctx, cudaMemcpy(st.rings_dev, rings.data(), rings.size() * sizeof(RowRing), cudaMemcpyHostToDevice));
+    return TSB_OK;
+}
+
 constexpr int EXPAND_MIN_ROWS = 64;                 // rows of a portion from which on its latents are expanded
 constexpr size_t EXPAND_MAX_BYTES = 2ull << 30;
 
@@ -183,6 +264,7 @@ int32_t plain_runtime_init(tsb_session* s, ModelRt& rt, const tsb_model* tm, con
     std::vector<KeyLayerShape> shapes;
     for (const PlainLayer& l : m->layers) {
         if (l.mixer == MIX_LATENT) shapes.push_back({1, l.key_dim, 0, l.source});
+        else if (l.mixer == MIX_NONE) shapes.push_back({0, 0, 0, (int)shapes.size()});
         else shapes.push_back({l.cfg.n_kv_heads, l.head_pad, l.mixer == MIX_KV ? l.head_pad : 0, (int)shapes.size()});
     }
     int32_t rc = kv_create_keys(ctx, m->cfg.n_layers, shapes.data(), m->elem, shape.page_tokens, shape.num_pages, shape.n_streams, shape.pages_per_seq, &rt.kv);
@@ -192,13 +274,19 @@ int32_t plain_runtime_init(tsb_session* s, ModelRt& rt, const tsb_model* tm, con
     // matmul operands are read in whole token tiles
     p->rows = (int)plain_pad(std::max(shape.pass_rows, 32), 32);
     p->in_stride = m->d_pad;
-    int64_t wide = 0, latent = 0;
+    int64_t wide = 0, latent = 0, experts = 0, top = 0, expert_ffn = 0;
     for (const PlainLayer& l : m->layers) {
-        const int64_t H = l.cfg.n_q_heads;
+        const int64_t H = l.cfg.n_q_heads, inner = (int64_t)l.cfg.rec_heads * l.cfg.rec_vdim;
+        p->rec_stride = std::max<int64_t>(p->rec_stride, plain_pad(rec_typed_rows(l.cfg), 16));
+        p->rec_mixed_stride = std::max<int64_t>(p->rec_mixed_stride, plain_pad(rec_conv_channels(l.cfg), 16));
+        if (l.cfg.recurrence) p->rec_out_stride = std::max<int64_t>(p->rec_out_stride, plain_pad(inner, 4));
+        p->raw_rec = std::max<int64_t>(p->raw_rec, l.cfg.qk_norm ? plain_pad((H + l.cfg.n_kv_heads) * l.cfg.head_dim, 4) : 0);
+        if (l.cfg.experts > 0)
+            experts = std::max<int64_t>(experts, l.cfg.experts), top = std::max<int64_t>(top, l.cfg.expert_top), expert_ffn = std::max<int64_t>(expert_ffn, l.ffn_pad);
         p->q_stride = std::max<int64_t>(p->q_stride, plain_pad(H * l.head_pad, 16));
         p->cat_stride = std::max<int64_t>(p->cat_stride, l.out.cols);
         p->gate_stride = std::max(p->gate_stride, l.cfg.n_q_heads);
-        if (l.post_norm) p->act_stride = std::max<int64_t>(p->act_stride, l.ffn_pad);
+        if (l.post_norm && l.cfg.experts == 0) p->act_stride = std::max<int64_t>(p->act_stride, l.ffn_pad);
         if (l.cfg.qk_norm) p->raw_stride = std::max<int64_t>(p->raw_stride, plain_pad((H + l.cfg.n_kv_heads) * l.cfg.head_dim, 4));
         if (l.cfg.value_gate) p->value_gate_stride = std::max<int64_t>(p->value_gate_stride, plain_pad(H * l.value_pad, 16));
         if (l.mixer != MIX_LATENT) continue;
@@ -207,6 +295,8 @@ int32_t plain_runtime_init(tsb_session* s, ModelRt& rt, const tsb_model* tm, con
         p->sums_stride = std::max<int64_t>(p->sums_stride, H * l.rank_pad);
         if (l.expands) wide = std::max<int64_t>(wide, H * (l.head_pad + l.value_pad)), latent = std::max<int64_t>(latent, l.key_dim);
     }
+    for (const PlainLayer& l : m->layers)
+        if (l.cfg.recurrence) p->raw_stride = std::max<int64_t>(p->raw_stride, plain_pad(p->raw_rec + rec_gate_rows(l.cfg), 4));
     p->fin_rows = (int)plain_pad(std::max(std::max(shape.n_streams * shape.max_rows, std::min(shape.pass_rows, 256)), 32), 32);
     auto A = [&](size_t bytes, void** q) {
         if (bytes == 0) return (int32_t)TSB_OK;
@@ -216,12 +306,31 @@ int32_t plain_runtime_init(tsb_session* s, ModelRt& rt, const tsb_model* tm, con
     };
     const size_t R = p->rows, e = m->elem;
     if ((rc = A(R * m->cfg.d_model * 4, (void**)&p->x)) || (rc = A(R * p->in_stride * e, &p->mix)) ||
-        (rc = A(m->cfg.post_norm ? 0 : R * p->in_stride * e, &p->h)) || (rc = A(R * p->q_stride * e, &p->q)) || (rc = A(R * p->cat_stride * e, &p->cat)) ||
+        (rc = A(m->cfg.post_norm || m->cfg.output_norm ? 0 : R * p->in_stride * e, &p->h)) || (rc = A(R * p->q_stride * e, &p->q)) || (rc = A(R * p->cat_stride * e, &p->cat)) ||
         (rc = A(R * p->gate_stride * 4, (void**)&p->gate)) || (rc = A((size_t)p->fin_rows * p->in_stride * e, &p->fin)) ||
         (rc = A(plain_gemm_workspace_bytes(ctx), &p->gemm_ws)) || (rc = A(wattn_scratch_bytes(ctx), &p->attn_ws)) ||
         (rc = A(R * p->act_stride * e, &p->act)) || (rc = A(R * p->raw_stride * 4, (void**)&p->raw)) || (rc = A(R * p->absorbed_stride * e, &p->absorbed)) ||
         (rc = A(R * p->sums_stride * e, &p->sums)) || (rc = A(R * p->value_gate_stride * e, &p->value_gate)))
         return rc;
+    if (m->cfg.output_norm) {
+        const size_t slots = plain_pad(R * top, 32) + 256;  // token tiles of a product may reach behind the last slot
+        p->expert_rows = top > 0 ? (int)slots : 0;
+        if ((rc = A(R * m->cfg.d_model * 4, (void**)&p->x2)) || (rc = A(R * m->cfg.d_model * 4, (void**)&p->y)) || (rc = A(R * p->rec_stride * e, &p->rec)) ||
+            (rc = A(R * p->rec_mixed_stride * e, &p->rec_mixed)) || (rc = A(R * p->rec_out_stride * 4, (void**)&p->rec_out)))
+            return rc;
+        if (top > 0) {
+            ExpertLists& x = p->lists;
+            const size_t ints = R * top * sizeof(int32_t);
+            if ((rc = A(R * experts * 4, (void**)&p->router_logits)) || (rc = A(slots * p->in_stride * e, &p->expert_in)) ||
+                (rc = A(slots * expert_ffn * e, &p->expert_act)) || (rc = A(slots * m->cfg.d_model * e, &p->expert_out)) || (rc = A(ints, (void**)&x.ids)) ||
+                (rc = A(ints, (void**)&x.weight)) || (rc = A(ints, (void**)&x.slot_of)) || (rc = A(ints, (void**)&x.token_of)) ||
+                (rc = A((experts + 1) * sizeof(int32_t), (void**)&x.first)) || (rc = A((experts + R * top / 8 + 1) * sizeof(ExpertChunk), (void**)&x.chunks)) ||
+                (rc = A(sizeof(int32_t), (void**)&x.n_chunks)))
+                return rc;
+        }
+        if ((rc = states_init(s, m, shape, p->states))) return rc;
+        if (p->states.ring > 0) rt.kv->state_ring = p->states.ring + 1;
+    }
     for (const PlainRotation& r : m->rotations) {
         float2* t = nullptr;
         if ((rc = A(R * (r.dims / 2) * sizeof(float2), (void**)&t))) return rc;
@@ -259,6 +368,7 @@ int32_t plain_fill_context(tsb_session* s, ModelRt& rt, int stream, int64_t toke
 // ------------------------------------------------------------------ packed rows of a layer's input matrix
 struct InRows {
     int64_t q = 0, k = 0, v = 0, head_gate = 0, value_gate = 0;  // first rows; latent layers: k is the latent
+    int64_t rec = 0, rec_gate = 0;                               // of the recurrence's vectors and gates
     int64_t segments = 0;                                        // end of the rows with destinations of their own
     int64_t pairs = 0, n_pairs = 0;                              // interleaved pairs behind them (gate and up, or rotated coordinates)
     int64_t rows = 0;
@@ -268,15 +378,19 @@ InRows in_rows(const PlainLayer& l) {
     const int64_t H = c.n_q_heads, G = c.n_kv_heads, E = c.value_dim;
     const bool own = c.kv_source == 0;
     InRows r;
-    int64_t at = l.mixer == MIX_KEYS ? l.q_rows : H * c.head_dim;
+    int64_t at = l.mixer == MIX_NONE ? 0 : l.mixer == MIX_KEYS ? l.q_rows : H * c.head_dim;
     r.k = at;
-    at += l.mixer == MIX_KEYS ? l.k_rows : l.mixer == MIX_KV ? G * c.head_dim : own ? c.kv_rank : 0;
+    at += l.mixer == MIX_NONE ? 0 : l.mixer == MIX_KEYS ? l.k_rows : l.mixer == MIX_KV ? G * c.head_dim : own ? c.kv_rank : 0;
     r.v = at;
     if (l.mixer == MIX_KV) at += G * E;
     r.head_gate = at;
     if (c.head_gate) at += H;
     r.value_gate = at;
     if (c.value_gate) at += H * E;
+    r.rec = at;
+    at += rec_typed_rows(c);
+    r.rec_gate = at;
+    at += rec_gate_rows(c);
     r.segments = at;
     r.pairs = plain_pad(at, PLAIN_ROW_PAD);
     if (l.mixer == MIX_LATENT) r.n_pairs = (H + (own ? 1 : 0)) * (c.rot_dim / 2);
@@ -301,6 +415,9 @@ struct PassPlan {
     std::vector<bool> is_expanded;
     const ExpandStream* expanded_dev = nullptr;
     int expanded_pages = 0, expanded_len = 0, short_first = 0, short_rows = 0;
+    // output-norm form: runs of rows for the row operators; portions whose recurrences go row by row, and chunk by chunk
+    RowTiles runs, by_row, by_chunk;
+    bool use_before = false;
 
     const AttnBatch* find(int set, int group, int rows_per_tile) const {
         for (const TileLists& t : lists)
@@ -314,11 +431,52 @@ LatentTiling latent_tiling(const tsb_ctx* ctx, const PassPlan& plan, const Pass&
     return latent_attn_tiling(ctx, l.cfg.n_q_heads, all ? plan.longest : plan.longest_short, all ? p.rows : plan.rows_short, plan.max_len);
 }
 
-int32_t plan_pass(tsb_session* s, const PlainModel* m, const PlainRt* b, const Pass& p, PassPlan& plan) {
+constexpr int CHUNK_MIN_ROWS = 32;  // rows of a portion from which on its recurrences go chunk by chunk
+
+int32_t plan_states(tsb_session* s, const PlainModel* m, const ModelRt& rt, const Pass& p, PassPlan& plan) {
+    const StreamStates& states = rt.plain->states;
+    plan.use_before = states.n_rings > 0 && plan.longest + states.keep > states.row_ring;
+    const int per = sublayer_rows_per_tile(s->ctx, p.rows);
+    if (p.rows_per_seq > 0) {
+        plan.runs = RowTiles::uniform(p.rows, p.rows_per_seq, per);
+        plan.by_row = RowTiles::uniform(p.rows, p.rows_per_seq, p.rows_per_seq);
+        return TSB_OK;
+    }
+    bool chunks = !m->f32;
+    for (const PlainLayer& l : m->layers) {
+        Recurrence r;
+        r.kind = l.cfg.recurrence, r.dim = l.cfg.rec_dim, r.vdim = l.cfg.rec_vdim;
+        if (l.cfg.recurrence) chunks &= recurrence_chunks_supported(r);
+    }
+    std::vector<AttnTile> runs, by_row, by_chunk;
+    for (int i = 0; i < p.n_groups; i++) {
+        const RowGroup& g = p.groups[i];
+        for (int r = 0; r < g.n_rows; r += per) runs.push_back({g.first_row + r, std::min(per, g.n_rows - r)});
+        const bool long_portion = chunks && g.n_rows >= CHUNK_MIN_ROWS;
+        (long_portion ? by_chunk : by_row).push_back({g.first_row, g.n_rows});
+        if (long_portion) rt.kv->state_lo[g.seq] = g.base + g.n_rows - 1;  // the states in between are not kept
+    }
+    auto stage = [&](const std::vector<AttnTile>& list, RowTiles& out) -> int32_t {
+        if (list.empty()) {
+            out.n = 0;
+            return TSB_OK;
+        }
+        const int32_t* dev = nullptr;
+        if (int32_t rc = session_stage_ints(s, reinterpret_cast<const int32_t*>(list.data()), (int)list.size() * 2, &dev)) return rc;
+        out = RowTiles::list(reinterpret_cast<const AttnTile*>(dev), (int)list.size());
+        return TSB_OK;
+    };
+    int32_t rc = stage(runs, plan.runs);
+    if (rc == TSB_OK) rc = stage(by_row, plan.by_row);
+    return rc == TSB_OK ? stage(by_chunk, plan.by_chunk) : rc;
+}
+
+int32_t plan_pass(tsb_session* s, const PlainModel* m, const ModelRt& rt, const Pass& p, PassPlan& plan) {
+    const PlainRt* b = rt.plain;
     plan.max_len = (p.max_len + 511) / 512 * 512;  // the split plan changes only every 512 positions (graph reuse)
     plan.longest = p.rows_per_seq;
     plan.short_rows = p.rows;
-    if (p.rows_per_seq > 0) return TSB_OK;
+    if (p.rows_per_seq > 0) return m->cfg.output_norm ? plan_states(s, m, rt, p, plan) : TSB_OK;
     plan.is_expanded.assign(p.n_groups, false);
     int first_short = p.rows, end_short = 0;
     for (int i = 0; i < p.n_groups; i++) {
@@ -340,6 +498,8 @@ int32_t plan_pass(tsb_session* s, const PlainModel* m, const PlainRt* b, const P
         if (int32_t rc = session_stage_ints(s, reinterpret_cast<const int32_t*>(plan.expanded.data()), (int)plan.expanded.size() * 3, &dev)) return rc;
         plan.expanded_dev = reinterpret_cast<const ExpandStream*>(dev);
     }
+    if (m->cfg.output_norm)
+        if (int32_t rc = plan_states(s, m, rt, p, plan)) return rc;
     if (m->f32) return TSB_OK;  // the f32 kernel takes rows one by one
     auto add = [&](int set, int group, int rpt, int small_queries) -> int32_t {
         if (plan.find(set, group, rpt)) return TSB_OK;
@@ -368,6 +528,7 @@ int32_t plan_pass(tsb_session* s, const PlainModel* m, const PlainRt* b, const P
     };
     for (const PlainLayer& l : m->layers) {
         int32_t rc = TSB_OK;
+        if (l.mixer == MIX_NONE) continue;
         if (l.mixer != MIX_LATENT) {
             const int grp = l.cfg.n_q_heads / l.cfg.n_kv_heads;
             rc = add(TILES_ALL, grp, wattn_rows_per_tile(l.head_pad, grp, l.cfg.log_bias != 0), WATTN_SMALL_Q);
@@ -402,7 +563,7 @@ struct Forward {
         const tsb_plain_layer& c = l.cfg;
         const InRows r = in_rows(l);
         PlainEpi e;
-        e.kind = PLAIN_MIXER, e.keys = rt.kv->key_layers[L], e.rows = p.rows_dev;
+        e.kind = PLAIN_MIXER, e.keys = rt.kv->key_layers[L], e.rows = p.rows_dev, e.bias = l.in_bias;
         auto seg = [&](int64_t end, int kind, void* to, int64_t stride, int64_t per = 0x7fffffff, int64_t step = 0) {
             PlainSeg& g = e.seg[e.n_seg++];
             g.end = (int)end, g.kind = kind, g.p = to, g.stride = stride, g.per = (int)per, g.step = (int)step;
@@ -418,7 +579,7 @@ struct Forward {
                 seg(r.v, PLAIN_SEG_CACHE, nullptr, 0, c.head_dim, e.keys.head_step);
             }
             seg(r.head_gate, PLAIN_SEG_CACHE, nullptr, e.keys.value_off, c.value_dim, e.keys.head_step);
-        } else {
+        } else if (l.mixer == MIX_LATENT) {
             seg(r.k, PLAIN_SEG_TYPED, b->q, b->q_stride, c.head_dim, l.head_pad);
             if (r.v > r.k) seg(r.v, PLAIN_SEG_F32, b->raw, b->raw_stride);
             if (c.rot_dim > 0) {
@@ -429,7 +590,11 @@ struct Forward {
             }
         }
         if (c.head_gate) seg(r.value_gate, PLAIN_SEG_F32, b->gate, c.n_q_heads);
-        if (c.value_gate) seg(r.segments, PLAIN_SEG_TYPED, b->value_gate, b->value_gate_stride, c.value_dim, l.value_pad);
+        if (c.value_gate) seg(r.rec, PLAIN_SEG_TYPED, b->value_gate, b->value_gate_stride, c.value_dim, l.value_pad);
+        if (c.recurrence) {
+            seg(r.rec_gate, PLAIN_SEG_TYPED, b->rec, b->rec_stride);
+            seg(r.segments, PLAIN_SEG_F32, b->raw + b->raw_rec, b->raw_stride);
+        }
         if (r.n_pairs > 0) {
             e.pair_row0 = (int)r.pairs, e.n_pairs = (int)r.n_pairs, e.act = c.act;
             e.a = at(b->cat, l.o_cols), e.a_stride = l.out.cols;  // a rotation does not use them
@@ -457,6 +622,8 @@ struct Forward {
         WindowAttn a;
         a.q = b->q, a.q_stride = b->q_stride, a.out = b->cat, a.out_stride = l.out.cols, a.rows = p.rows_dev;
         a.n_q_heads = c.n_q_heads, a.scale = c.score_scale, a.cap = c.score_cap, a.window = c.window;
+        a.slopes = l.slopes, a.chunk = c.chunk;
+        if (c.recurrence) a.out_scale = c.attn_scale;
         a.gate = c.head_gate ? b->gate : nullptr;
         if (c.value_gate) a.value_gate = b->value_gate, a.value_gate_stride = b->value_gate_stride;
         if (c.log_bias) a.r1 = l.r1, a.r2 = l.r2;
@@ -540,10 +707,146 @@ struct Forward {
         return launch_window_attn_wide(ctx, st, a, *plan.find(TILES_WIDE, 1, WATTN_WIDE_ROWS), b->attn_ws);
     }
 
+    cudaError_t projection_norms(int L) const {
+        const PlainLayer& l = m->layers[L];
+        ProjectionNorms n;
+        n.raw = b->raw, n.raw_stride = b->raw_stride, n.n_q = l.cfg.n_q_heads, n.n_k = l.cfg.n_kv_heads, n.width = l.cfg.head_dim;
+        n.q_weight = l.q_norm, n.k_weight = l.k_norm, n.eps = m->cfg.norm_eps, n.q = b->q, n.q_stride = b->q_stride, n.q_step = l.head_pad;
+        n.keys = rt.kv->key_layers[L], n.rows = p.rows_dev;
+        return launch_projection_norms(ctx, st, m->f32, n, p.rows);
+    }
+
+    // from the projections to the recurrence's part of b->cat
+    cudaError_t recur(int L) const {
+        const PlainLayer& l = m->layers[L];
+        const tsb_plain_layer& c = l.cfg;
+        const int h = c.rec_heads, D = c.rec_dim, E = c.rec_vdim, inner = h * E;
+        Recurrence r;
+        GatedNorm g;
+        r.kind = c.recurrence, r.heads = h, r.dim = D, r.vdim = E, r.gate = b->raw + b->raw_rec, r.gate_stride = b->raw_stride;
+        r.q = b->rec, r.q_stride = r.k_stride = r.v_stride = b->rec_stride, r.out = b->rec_out, r.out_stride = b->rec_out_stride;
+        r.state = b->states.states[L], r.rows = p.rows_dev;
+        g.o = b->rec_out, g.o_stride = b->rec_out_stride, g.width = inner, g.groups = h, g.weight = l.rec_norm, g.weight_n = inner, g.eps = m->cfg.norm_eps;
+        g.gate_stride = b->rec_stride, g.out = at(b->cat, l.o_cols), g.out_stride = l.out.cols;
+        if (l.mixer != MIX_NONE) g.scale = c.rec_scale;
+        if (c.recurrence == TSB_REC_FORGET) {
+            r.v = at(b->rec, h * D), r.lower = l.rec_lower;
+            g.weight_n = E;
+        } else if (c.recurrence == TSB_REC_MLSTM) {
+            r.k = at(b->rec, h * D), r.v = at(b->rec, 2 * h * D), r.cap = c.rec_cap, r.q_scale = (float)(1.0 / sqrt((double)D));
+            g.post_gate = at(b->rec, 2 * h * D + inner);
+        } else {
+            ShortConv v;
+            v.in = at(b->rec, inner), v.in_stride = b->rec_stride, v.out = b->rec_mixed, v.out_stride = b->rec_mixed_stride, v.channels = (int)rec_conv_channels(c);
+            v.taps = c.rec_taps, v.w = l.rec_conv, v.bias = l.rec_conv_bias, v.ring = b->states.rec[L], v.use_before = plan.use_before;
+            v.rows = p.rows_dev, v.n_rows = p.rows, v.tiles = plan.runs;
+            if (cudaError_t e = launch_short_conv(ctx, st, m->f32, v); e != cudaSuccess) return e;
+            r.v = b->rec_mixed, r.k = at(b->rec_mixed, inner), r.q = at(b->rec_mixed, inner + c.rec_groups * D);
+            r.q_stride = r.k_stride = r.v_stride = b->rec_mixed_stride, r.heads_per_key = h / c.rec_groups, r.a_log = l.rec_a_log, r.skip = l.rec_skip;
+            g.pre_gate = b->rec, g.groups = c.rec_norm_groups;
+        }
+        if (plan.by_chunk.n > 0)
+            if (cudaError_t e = launch_recurrence_chunks(ctx, st, r, plan.by_chunk); e != cudaSuccess) return e;
+        if (plan.by_row.n > 0)
+            if (cudaError_t e = launch_recurrence_rows(ctx, st, m->f32, r, plan.by_row); e != cudaSuccess) return e;
+        return launch_gated_norm(ctx, st, m->f32, g, p.rows);
+    }
+
+    // The routed feed-forward of b->mix: expert outputs by slot, to be summed by the end of the sublayer.
+    cudaError_t route(int L) const {
+        const PlainLayer& l = m->layers[L];
+        const tsb_plain_layer& c = l.cfg;
+        const int slots = p.rows * c.expert_top;
+        PlainEpi z;
+        z.kind = PLAIN_STORE, z.y = b->router_logits, z.y_stride = c.experts, z.n_valid = c.experts;
+        cudaError_t e = matmul(l.router, b->mix, nullptr, b->in_stride, z);
+        if (e != cudaSuccess) return e;
+        // with many slots per expert the tensor-memory kernel, over gathered rows; with few the weight-streaming one
+        const bool tensor = !m->f32 && p.rows > 16 && slots >= 12 * c.experts;
+        ExpertRouting r;
+        r.logits = b->router_logits, r.logits_stride = c.experts, r.correction = l.correction, r.experts = c.experts, r.top = c.expert_top;
+        r.groups = c.expert_groups, r.keep = c.expert_keep, r.rows = p.rows, r.lists = b->lists;
+        r.chunk_slots = m->f32 ? EXPERT_CHUNK_F32 : p.rows <= 8 ? 8 : EXPERT_CHUNK_FEW;
+        if ((e = launch_route_experts(ctx, st, r)) != cudaSuccess) return e;
+        if (tensor && (e = launch_gather_rows(ctx, st, b->mix, b->in_stride * m->elem, b->lists.token_of, slots, b->expert_in, b->in_stride * m->elem)) != cudaSuccess)
+            return e;
+        PlainExperts x;
+        x.n = c.experts, x.slots = slots, x.first = b->lists.first, x.token_of = tensor ? nullptr : b->lists.token_of, x.chunks = b->lists.chunks;
+        x.n_chunks = b->lists.n_chunks, x.chunk_slots = r.chunk_slots;
+        PlainEpi g;
+        g.kind = PLAIN_MIXER, g.pair_row0 = 0, g.n_pairs = l.ffn_pad, g.act = c.act, g.a = b->expert_act, g.a_stride = l.ffn_pad;
+        e = launch_plain_gemm_experts(ctx, st, m->f32, tensor, l.ff_in, tensor ? b->expert_in : b->mix, b->in_stride, tensor ? b->expert_rows : b->rows, x, g);
+        if (e != cudaSuccess) return e;
+        PlainEpi d;
+        d.kind = PLAIN_MIXER, d.n_seg = 1, d.seg[0].end = m->cfg.d_model, d.seg[0].p = b->expert_out, d.seg[0].stride = m->cfg.d_model;
+        x.token_of = nullptr;
+        return launch_plain_gemm_experts(ctx, st, m->f32, tensor, l.ff_out, b->expert_act, l.ffn_pad, b->expert_rows, x, d);
+    }
+
+    // The layers of an output-norm model; returns the buffer that holds the stream at the end.
+    cudaError_t output_norm_layers(float** stream) const {
+        float *x = b->x, *x_next = b->x2;
+        SublayerEnd s;
+        s.d = m->cfg.d_model, s.groups = std::max(1, m->cfg.norm_groups), s.eps = m->cfg.norm_eps, s.taps = m->cfg.conv_taps, s.use_before = plan.use_before;
+        s.out = b->mix, s.out_stride = b->in_stride, s.rows = p.rows_dev, s.n_rows = p.rows, s.tiles = plan.runs;
+        // next: the convolution in front of the next sublayer
+        auto end = [&](SublayerEnd& v, const float* taps, const RowRing& ring) {
+            v.x_in = x, v.x_out = x_next, v.taps_w = taps, v.ring = ring;
+            std::swap(x, x_next);
+            return launch_sublayer_end(ctx, st, m->f32, v);
+        };
+        auto first_of = [&](SublayerEnd& v, int L) {  // the end of whatever comes before layer L
+            if (L < m->cfg.n_layers) return end(v, m->layers[L].conv1, b->states.conv1.empty() ? RowRing() : b->states.conv1[L]);
+            v.taps = 0, v.out = nullptr;
+            return end(v, nullptr, RowRing());
+        };
+        cudaError_t e = plan.use_before ? launch_rings_before(ctx, st, b->states.rings_dev, b->states.n_rings, p.rows_dev, p.rows) : cudaSuccess;
+        if (e != cudaSuccess) return e;
+        SublayerEnd t = s;
+        t.table = m->embed, t.positions = m->positions, t.n_positions = m->cfg.positions, t.tokens = p.tokens, t.token_stride = p.token_stride, t.vocab = m->cfg.vocab;
+        t.embed_scale = m->cfg.embed_scale;
+        e = first_of(t, 0);
+        for (int L = 0; L < m->cfg.n_layers && e == cudaSuccess; L++) {
+            const PlainLayer& l = m->layers[L];
+            e = project(L, b->mix, b->mix);
+            if (e == cudaSuccess) e = mix(L);
+            PlainEpi o;
+            o.kind = PLAIN_STORE, o.y = b->y, o.y_stride = m->cfg.d_model, o.n_valid = m->cfg.d_model;
+            if (e == cudaSuccess) e = matmul(l.out, b->cat, nullptr, l.out.cols, o);
+            SublayerEnd v = s;
+            v.y = b->y, v.norm_w = l.gain;
+            if (e == cudaSuccess) e = l.cfg.ffn > 0 ? end(v, l.conv2, b->states.conv2.empty() ? RowRing() : b->states.conv2[L]) : first_of(v, L + 1);
+            if (e != cudaSuccess || l.cfg.ffn == 0) continue;
+            v = s;
+            v.norm_w = l.norm2;
+            if (l.cfg.experts > 0) {
+                e = route(L);
+                v.experts = b->expert_out, v.expert_stride = m->cfg.d_model, v.slot_of = b->lists.slot_of, v.weight = b->lists.weight, v.top = l.cfg.expert_top;
+            } else {
+                PlainEpi g;
+                g.kind = PLAIN_MIXER, g.pair_row0 = 0, g.n_pairs = l.ffn_pad, g.act = l.cfg.act, g.a = b->act, g.a_stride = l.ffn_pad;
+                e = matmul(l.ff_in, b->mix, b->mix, b->in_stride, g);
+                if (e == cudaSuccess) e = matmul(l.ff_out, b->act, nullptr, l.ffn_pad, o);
+                v.y = b->y;
+            }
+            if (e == cudaSuccess) e = first_of(v, L + 1);
+        }
+        *stream = x;
+        return e;
+    }
+
     // from the projections to the heads' outputs, side by side in b->cat
     cudaError_t mix(int L) const {
         const PlainLayer& l = m->layers[L];
         cudaError_t e = cudaSuccess;
+        if (l.cfg.recurrence) {
+            e = recur(L);
+            if (e != cudaSuccess || l.mixer == MIX_NONE) return e;
+        }
+        if (l.cfg.qk_norm == TSB_NORM_PROJECTION) {
+            if ((e = projection_norms(L)) != cudaSuccess) return e;
+            return attend(L);
+        }
         if (l.cfg.qk_norm || (l.mixer == MIX_LATENT && l.source == L)) e = head_norms(L);
         if (e != cudaSuccess) return e;
         if (l.mixer != MIX_LATENT) return attend(L);
@@ -596,7 +899,7 @@ cudaError_t plain_forward(tsb_session* s, ModelRt& rt, const Pass& p) {
     const int d = m->cfg.d_model;
     const bool post = m->cfg.post_norm != 0;
     PassPlan plan;
-    if (plan_pass(s, m, b, p, plan) != TSB_OK) return cudaErrorMemoryAllocation;
+    if (plan_pass(s, m, rt, p, plan) != TSB_OK) return cudaErrorMemoryAllocation;
     const Forward f{s, rt, p, ctx, st, m, b, plan};
     cudaError_t e;
 #define FW(x)                           \
@@ -605,6 +908,10 @@ cudaError_t plain_forward(tsb_session* s, ModelRt& rt, const Pass& p) {
         if (e != cudaSuccess) return e; \
     } while (0)
     const bool use_before = m->any_shift && plan.longest >= b->shift.ring_rows;
+    float* x = b->x;
+    if (m->cfg.output_norm) {
+        FW(f.output_norm_layers(&x));
+    } else {
     FW(launch_plain_embed(ctx, st, m->f32, m->embed, m->cfg.vocab, d, p.tokens, p.token_stride, p.rows, m->cfg.embed_scale, b->x, post ? b->mix : nullptr,
                           b->in_stride));
     if (use_before) FW(launch_shift_before(ctx, st, b->shift, m->cfg.n_layers, p.rows_dev, p.rows));
@@ -613,12 +920,18 @@ cudaError_t plain_forward(tsb_session* s, ModelRt& rt, const Pass& p) {
         FW(launch_rotary_table(ctx, st, r.freq, r.dims / 2, r.magnitude, p.rows_dev, p.rows, b->rotary[i]));
     }
     for (int L = 0; L < m->cfg.n_layers; L++) FW(post ? f.post_norm_layer(L) : f.parallel_layer(L, use_before));
+    }
     if (p.logits) {
         const bool last = p.last_rows_only && p.rows_per_seq > 1;
         const int n = p.rows_per_seq == 0 ? p.n_want : last ? p.rows / p.rows_per_seq : p.rows;
         if (n > 0) {
-            FW(launch_norm_rows(ctx, st, m->f32, b->x, d, m->final_gain, post ? m->final_gain : nullptr, m->cfg.norm_eps,
-                                p.rows_per_seq == 0 ? p.want_dev : nullptr, last ? p.rows_per_seq - 1 : 0, last ? p.rows_per_seq : 1, n, b->fin, b->in_stride));
+            const int32_t* want = p.rows_per_seq == 0 ? p.want_dev : nullptr;
+            const int want_first = last ? p.rows_per_seq - 1 : 0, want_step = last ? p.rows_per_seq : 1;
+            if (m->cfg.output_norm)
+                FW(launch_group_norm_rows(ctx, st, m->f32, x, d, m->final_gain, std::max(1, m->cfg.norm_groups), m->cfg.norm_eps, want, want_first, want_step, n, b->fin,
+                                          b->in_stride));
+            else
+                FW(launch_norm_rows(ctx, st, m->f32, x, d, m->final_gain, post ? m->final_gain : nullptr, m->cfg.norm_eps, want, want_first, want_step, n, b->fin, b->in_stride));
             PlainEpi hd;
             hd.kind = PLAIN_STORE, hd.y = static_cast<float*>(p.logits.p), hd.y_stride = p.logits_stride, hd.n_valid = m->cfg.vocab, hd.cap = m->cfg.logit_cap;
             FW(launch_plain_gemm(ctx, st, m->f32, m->head, b->fin, nullptr, b->in_stride, b->fin_rows, n, hd, b->gemm_ws));
@@ -665,6 +978,37 @@ const ModelFamily PLAIN_FAMILY = {
 
 }  // namespace
 
+// what only layers of the output-norm form have
+static int32_t check_output_norm_layer(tsb_ctx* ctx, const tsb_plain_config* cfg, const tsb_plain_layer& l, int i) {
+    if (!cfg->output_norm) {
+        TSB_REQUIRE(ctx, !l.recurrence && !l.experts && !l.qkv_bias && !l.linear_bias && !l.chunk && (l.qk_norm == 0 || l.qk_norm == TSB_NORM_HEAD),
+                    "layer %d: recurrences, experts, biases, chunks and projection norms go with the output-norm form", i);
+        return TSB_OK;
+    }
+    TSB_REQUIRE(ctx, !l.kv_rank && !l.token_shift && !l.head_gate && !l.log_bias && l.q_temp_every == 0, "layer %d: not a mechanism of the output-norm form", i);
+    TSB_REQUIRE(ctx, l.n_q_heads >= 0 && (l.n_q_heads > 0 || l.recurrence), "layer %d has no mixer", i);
+    TSB_REQUIRE(ctx, l.n_q_heads == 0 || l.value_dim > 0, "layer %d: attention has values of its own", i);
+    TSB_REQUIRE(ctx, l.chunk >= 0 && !(l.chunk && l.window), "layer %d: a chunk or a window", i);
+    TSB_REQUIRE(ctx, l.qk_norm >= 0 && l.qk_norm <= TSB_NORM_PROJECTION && (!l.qkv_bias || l.qk_norm == TSB_NORM_PROJECTION || l.n_q_heads == 0),
+                "layer %d: biases go with projection norms", i);
+    if (l.recurrence) {
+        TSB_REQUIRE(ctx, l.recurrence <= TSB_REC_SSD && l.rec_heads > 0 && l.rec_dim > 0 && l.rec_vdim > 0, "layer %d: bad recurrence", i);
+        if (l.rec_dim > REC_MAX_DIM || l.rec_heads > 65535)
+            return tsb_fail(ctx, TSB_ERR_UNSUPPORTED, "layer %d: recurrent heads of %d rows are outside the kernels", i, l.rec_dim);
+        const int64_t inner = (int64_t)l.rec_heads * l.rec_vdim;
+        if (inner > 24 * 1024) return tsb_fail(ctx, TSB_ERR_UNSUPPORTED, "layer %d: %lld recurrent columns are outside the kernels", i, (long long)inner);
+        if (l.recurrence == TSB_REC_SSD) {
+            TSB_REQUIRE(ctx, l.rec_groups > 0 && l.rec_heads % l.rec_groups == 0 && l.rec_norm_groups > 0 && inner % l.rec_norm_groups == 0,
+                        "layer %d: groups must divide the recurrence's heads and columns", i);
+            TSB_REQUIRE(ctx, l.rec_taps > 0 && l.rec_taps <= CONV_MAX_TAPS, "layer %d: a convolution has 1 to %d taps", i, CONV_MAX_TAPS);
+        }
+        TSB_REQUIRE(ctx, l.recurrence != TSB_REC_MLSTM || l.rec_cap > 0.f, "layer %d: the gates' cap is positive", i);
+    }
+    TSB_REQUIRE(ctx, l.experts >= 0 && (l.experts == 0 || (l.ffn > 0 && routing_supported(l.experts, l.expert_top, l.expert_groups, l.expert_keep))),
+                "layer %d: %d experts in %d groups, %d groups kept and %d experts taken do not fit together", i, l.experts, l.expert_groups, l.expert_keep, l.expert_top);
+    return TSB_OK;
+}
+
 extern "C" {
 
 int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const tsb_plain_layer* layers, tsb_model** out) {
@@ -674,9 +1018,17 @@ int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const 
     TSB_REQUIRE(ctx, cfg->compute == TSB_BF16 || cfg->compute == TSB_F32, "compute must be TSB_BF16 or TSB_F32");
     TSB_REQUIRE(ctx, cfg->norm_eps >= 0.f, "norm_eps must not be negative");
     const bool f32 = cfg->compute == TSB_F32;
+    TSB_REQUIRE(ctx, cfg->norm_groups >= 0 && cfg->conv_taps >= 0 && cfg->positions >= 0, "norm groups, taps and positions must not be negative");
+    TSB_REQUIRE(ctx, cfg->output_norm ? !cfg->post_norm && cfg->logit_cap <= 0.f : !cfg->norm_groups && !cfg->conv_taps && !cfg->positions,
+                "norm groups, convolutions and learned positions go with the output-norm form");
+    if (cfg->output_norm && !sublayer_end_supported(cfg->d_model, std::max(1, cfg->norm_groups), cfg->conv_taps))
+        return tsb_fail(ctx, TSB_ERR_UNSUPPORTED, "width %d in %d norm groups with %d taps is outside the kernels", cfg->d_model, cfg->norm_groups, cfg->conv_taps);
+    TSB_REQUIRE(ctx, cfg->positions == 0 || cfg->max_context <= cfg->positions, "a context of %d positions exceeds the learned %d", cfg->max_context, cfg->positions);
     for (int i = 0; i < cfg->n_layers; i++) {
         const tsb_plain_layer& l = layers[i];
+        if (int32_t rc = check_output_norm_layer(ctx, cfg, l, i)) return rc;
         const bool latent = l.kv_rank > 0;
+        if (l.n_q_heads == 0 && l.recurrence) continue;
         TSB_REQUIRE(ctx, l.n_q_heads > 0 && l.head_dim > 0 && (latent || (l.n_kv_heads > 0 && l.n_q_heads % l.n_kv_heads == 0)),
                     "layer %d: query heads must be a positive multiple of the key heads", i);
         TSB_REQUIRE(ctx, l.window >= 0 && l.ffn >= 0 && l.value_dim >= 0 && l.kv_rank >= 0 && l.rot_dim >= 0, "layer %d: sizes must not be negative", i);
@@ -716,6 +1068,7 @@ int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const 
     // what the session and the samplers read of a model
     tm->cfg.n_layers = cfg->n_layers, tm->cfg.d_model = cfg->d_model, tm->cfg.vocab = cfg->vocab, tm->cfg.max_context = cfg->max_context;
     tm->cfg.n_q_heads = layers[0].n_q_heads, tm->cfg.n_kv_heads = layers[0].n_kv_heads, tm->cfg.head_dim = layers[0].head_dim, tm->cfg.ffn = layers[0].ffn;
+    if (tm->cfg.n_q_heads == 0) tm->cfg.n_q_heads = tm->cfg.n_kv_heads = tm->cfg.head_dim = 1;
     tm->cfg.rms_eps = cfg->norm_eps;
     m->cfg = *cfg, m->f32 = f32, m->elem = f32 ? 4 : 2;
     if (m->cfg.embed_scale == 0.f) m->cfg.embed_scale = 1.f;
@@ -728,8 +1081,8 @@ int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const 
         l.cfg = layers[i];
         const tsb_plain_layer& c = l.cfg;
         const int H = c.n_q_heads;
-        l.post_norm = cfg->post_norm != 0;
-        l.mixer = c.kv_rank > 0 ? MIX_LATENT : c.value_dim > 0 ? MIX_KV : MIX_KEYS;
+        l.post_norm = cfg->post_norm != 0 || cfg->output_norm != 0;
+        l.mixer = H == 0 ? MIX_NONE : c.kv_rank > 0 ? MIX_LATENT : c.value_dim > 0 ? MIX_KV : MIX_KEYS;
         l.source = c.kv_source > 0 ? c.kv_source - 1 : i;
         m->any_shift |= c.token_shift != 0;
         if (l.mixer == MIX_LATENT) {
@@ -742,18 +1095,32 @@ int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const 
             l.lift.group_rows = (int)plain_pad(c.value_dim, PLAIN_ROW_PAD), l.lift.group_cols = l.rank_pad;
             l.lift.rows = (int64_t)H * l.lift.group_rows, l.lift.cols = plain_pad(c.kv_rank, PLAIN_COL_PAD);
             l.expand.rows = plain_pad((int64_t)H * (c.head_dim + c.value_dim), PLAIN_ROW_PAD), l.expand.cols = l.lift.cols;
-        } else {
+        } else if (l.mixer != MIX_NONE) {
             l.head_pad = l.value_pad = wattn_pad_dim(std::max(c.head_dim, c.value_dim), f32);
         }
         l.q_rows = H * l.head_pad, l.k_rows = c.n_kv_heads * l.head_pad;
         l.ffn_pad = (int)plain_pad(c.ffn, 64);
         l.in.rows = in_rows(l).rows, l.in.cols = m->d_pad;
         l.o_cols = (int)plain_pad((int64_t)H * l.value_pad, PLAIN_COL_PAD);
-        l.out.rows = out_rows, l.out.cols = l.o_cols + (l.post_norm ? 0 : l.ffn_pad);
+        l.rec_cols = (int)plain_pad((int64_t)c.rec_heads * c.rec_vdim * (c.recurrence != 0), PLAIN_COL_PAD);
+        l.out.rows = out_rows, l.out.cols = l.o_cols + l.rec_cols + (l.post_norm ? 0 : l.ffn_pad);
         l.ff_in.rows = 2 * (int64_t)l.ffn_pad, l.ff_in.cols = m->d_pad;
         l.ff_out.rows = out_rows, l.ff_out.cols = l.ffn_pad;
+        l.router.rows = plain_pad(c.experts, PLAIN_ROW_PAD), l.router.cols = m->d_pad;
     }
     DeviceGuard g(ctx);
+    for (PlainLayer& l : m->layers) {
+        if (!l.cfg.linear_bias) continue;
+        std::vector<float> slopes(l.cfg.n_q_heads);
+        for (int h = 0; h < l.cfg.n_q_heads; h++) slopes[h] = (float)exp2(-8.0 * (h + 1) / l.cfg.n_q_heads);
+        int32_t rc = tsb_alloc(ctx, slopes.size() * 4, (void**)&l.slopes);
+        if (rc == TSB_OK && cudaMemcpy(l.slopes, slopes.data(), slopes.size() * 4, cudaMemcpyHostToDevice) != cudaSuccess)
+            rc = tsb_fail(ctx, TSB_ERR_CUDA, "uploading slopes failed");
+        if (rc) {
+            tsb_model_destroy(tm);
+            return rc;
+        }
+    }
     for (PlainRotation& r : m->rotations)
         if (int32_t rc = upload_rotation(ctx, r)) {
             tsb_model_destroy(tm);
@@ -772,23 +1139,29 @@ int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t
     const int64_t d = m->cfg.d_model, V = m->cfg.vocab;
     const bool post = m->cfg.post_norm != 0;
     PlainLayer* l = nullptr;
-    if (which >= TSB_P_NORM) {
+    const bool output = m->cfg.output_norm != 0, seq = post || output;  // seq: the sublayers follow each other
+    if (which >= TSB_P_NORM && which != TSB_P_POSITIONS) {
         TSB_REQUIRE(ctx, layer >= 0 && layer < m->cfg.n_layers, "layer %d outside the model", layer);
         l = &m->layers[layer];
     }
     const tsb_plain_layer c = l ? l->cfg : tsb_plain_layer{};
     const bool latent = l && l->mixer == MIX_LATENT, own_latent = latent && c.kv_source == 0;
     const int64_t H = c.n_q_heads, G = c.n_kv_heads, D = c.head_dim, F = c.ffn, E = l && l->mixer != MIX_KEYS ? c.value_dim : D, R = c.kv_rank;
+    const int64_t rh = c.recurrence ? c.rec_heads : 0, RD = c.rec_dim, RE = c.rec_vdim, X = std::max(1, c.experts), taps = m->cfg.conv_taps;
+    const bool attn = l && l->mixer != MIX_NONE, whole = c.qk_norm == TSB_NORM_PROJECTION;
+    const bool forget = c.recurrence == TSB_REC_FORGET, mlstm = c.recurrence == TSB_REC_MLSTM, ssd = c.recurrence == TSB_REC_SSD;
+    const int64_t channels = rec_conv_channels(c);
     int64_t wr = 1, wc = 1;  // expected shape; -1: no such tensor
     switch (which) {
         case TSB_P_EMBED: case TSB_P_HEAD: wr = V, wc = d; break;
-        case TSB_P_FINAL_NORM: case TSB_P_NORM: wc = post ? d : 1; break;
-        case TSB_P_NORM2: wc = post && F > 0 ? d : -1; break;
+        case TSB_P_FINAL_NORM: case TSB_P_NORM: wc = seq ? d : 1; break;
+        case TSB_P_NORM2: wc = seq && F > 0 ? d : -1; break;
         case TSB_P_SHIFT: wc = c.token_shift ? d : -1; break;
-        case TSB_P_Q: wr = H * (D + c.rot_dim), wc = d; break;
-        case TSB_P_K: wr = latent ? -1 : G * D, wc = d; break;
+        case TSB_P_Q: wr = attn ? H * (D + c.rot_dim) : -1, wc = d; break;
+        case TSB_P_K: wr = latent || !attn ? -1 : G * D, wc = d; break;
         case TSB_P_V: wr = l->mixer == MIX_KV ? G * E : -1, wc = d; break;
-        case TSB_P_Q_NORM: case TSB_P_K_NORM: wc = c.qk_norm ? D : -1; break;
+        case TSB_P_Q_NORM: wc = whole ? H * D : c.qk_norm ? D : -1; break;
+        case TSB_P_K_NORM: wc = whole ? G * D : c.qk_norm ? D : -1; break;
         case TSB_P_SINK: wc = c.sink ? H : -1; break;
         case TSB_P_HEAD_GATE: wr = c.head_gate ? H : -1, wc = d; break;
         case TSB_P_VALUE_GATE: wr = c.value_gate ? H * E : -1, wc = d; break;
@@ -797,9 +1170,32 @@ int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t
         case TSB_P_DKV_NORM: wc = own_latent ? R : -1; break;
         case TSB_P_UK: wr = latent ? H * D : -1, wc = R; break;
         case TSB_P_UV: wr = latent ? H * E : -1, wc = R; break;
-        case TSB_P_O: wr = d, wc = H * E; break;
-        case TSB_P_FF_GATE: case TSB_P_FF_UP: wr = F > 0 ? F : -1, wc = d; break;
-        case TSB_P_FF_DOWN: wr = d, wc = F > 0 ? F : -1; break;
+        case TSB_P_O: wr = d, wc = attn ? H * E : -1; break;
+        case TSB_P_FF_GATE: case TSB_P_FF_UP: wr = F > 0 ? X * F : -1, wc = d; break;
+        case TSB_P_FF_DOWN: wr = X * d, wc = F > 0 ? F : -1; break;
+        case TSB_P_POSITIONS: wr = m->cfg.positions > 0 ? m->cfg.positions : -1, wc = d; break;
+        case TSB_P_CONV1: wr = d, wc = taps > 0 ? taps : -1; break;
+        case TSB_P_CONV2: wr = d, wc = taps > 0 && F > 0 ? taps : -1; break;
+        case TSB_P_Q_BIAS: wc = c.qkv_bias ? H * D : -1; break;
+        case TSB_P_K_BIAS: wc = c.qkv_bias ? G * D : -1; break;
+        case TSB_P_V_BIAS: wc = c.qkv_bias ? G * E : -1; break;
+        case TSB_P_ROUTER: wr = c.experts > 0 ? c.experts : -1, wc = d; break;
+        case TSB_P_CORRECTION: wc = c.experts > 0 ? c.experts : -1; break;
+        case TSB_P_REC_Q: wr = forget || mlstm ? rh * RD : -1, wc = d; break;
+        case TSB_P_REC_K: wr = mlstm ? rh * RD : -1, wc = d; break;
+        case TSB_P_REC_V: wr = forget || mlstm ? rh * RE : -1, wc = d; break;
+        case TSB_P_REC_GATE: wr = mlstm ? rh * RE : -1, wc = d; break;
+        case TSB_P_REC_F: wr = forget ? rh * RD : mlstm ? rh : -1, wc = d; break;
+        case TSB_P_REC_F_BIAS: wc = forget ? rh * RD : mlstm ? rh : -1; break;
+        case TSB_P_REC_LOWER: wc = forget ? rh * RD : -1; break;
+        case TSB_P_REC_I: wr = mlstm ? rh : -1, wc = d; break;
+        case TSB_P_REC_I_BIAS: wc = mlstm ? rh : -1; break;
+        case TSB_P_REC_NORM: wc = forget ? RE : rh > 0 ? rh * RE : -1; break;
+        case TSB_P_REC_O: wr = d, wc = rh > 0 ? rh * RE : -1; break;
+        case TSB_P_REC_IN: wr = ssd ? rec_typed_rows(c) + rh : -1, wc = d; break;
+        case TSB_P_REC_CONV: wr = ssd ? channels : -1, wc = c.rec_taps; break;
+        case TSB_P_REC_CONV_BIAS: wc = ssd ? channels : -1; break;
+        case TSB_P_REC_DT_BIAS: case TSB_P_REC_A_LOG: case TSB_P_REC_D: wc = ssd ? rh : -1; break;
         default: return tsb_fail(ctx, TSB_ERR_INVALID, "no such tensor (%d)", which);
     }
     TSB_REQUIRE(ctx, wr > 0 && wc > 0, "layer %d has no tensor %d", layer, which);
@@ -821,29 +1217,63 @@ int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t
         case TSB_P_K_NORM: vec = &l->k_norm; break;
         case TSB_P_DKV_NORM: vec = &l->c_norm; break;
         case TSB_P_SINK: vec = &l->sink; break;
+        case TSB_P_CORRECTION: vec = &l->correction; break;
+        case TSB_P_REC_LOWER: vec = &l->rec_lower; break;
+        case TSB_P_REC_NORM: vec = &l->rec_norm; break;
+        case TSB_P_REC_CONV_BIAS: vec = &l->rec_conv_bias; break;
+        case TSB_P_REC_A_LOG: vec = &l->rec_a_log; break;
+        case TSB_P_REC_D: vec = &l->rec_skip; break;
+        case TSB_P_CONV1: vec = &l->conv1; break;
+        case TSB_P_CONV2: vec = &l->conv2; break;
+        case TSB_P_REC_CONV: vec = &l->rec_conv; break;
     }
-    uint32_t& set = l ? l->set : m->set;
-    if (vec) {
+    uint64_t& set = l ? l->set : m->set;
+    const InRows at = l ? in_rows(*l) : InRows();
+    // biases: entries of the input matrix's bias, which its epilogue adds
+    int64_t bias_at = -1;
+    switch (which) {
+        case TSB_P_Q_BIAS: bias_at = at.q; break;
+        case TSB_P_K_BIAS: bias_at = at.k; break;
+        case TSB_P_V_BIAS: bias_at = at.v; break;
+        case TSB_P_REC_F_BIAS: bias_at = at.rec_gate + (mlstm ? rh : 0); break;
+        case TSB_P_REC_I_BIAS: case TSB_P_REC_DT_BIAS: bias_at = at.rec_gate; break;
+    }
+    if (bias_at >= 0) {
         convert(host, host_type, wc, true, v);
+        if (!l->in_bias && (rc = zeroed(ctx, (size_t)l->in.rows * 4, (void**)&l->in_bias))) return rc;
+        TSB_CUDA(ctx, cudaMemcpy(l->in_bias + bias_at, v.data(), v.size(), cudaMemcpyHostToDevice));
+        set |= 1ull << which;
+        return TSB_OK;
+    }
+    if (vec) {
+        const int64_t n = wr * wc;
+        convert(host, host_type, n, true, v);
+        if (wr > 1) {  // taps: [channels, taps] -> [taps][channels]
+            std::vector<uint8_t> t(v.size());
+            for (int64_t i = 0; i < wr; i++)
+                for (int64_t k = 0; k < wc; k++) reinterpret_cast<float*>(t.data())[k * wr + i] = reinterpret_cast<const float*>(v.data())[i * wc + k];
+            v.swap(t);
+        }
         if (post && (which == TSB_P_FINAL_NORM || which == TSB_P_NORM || which == TSB_P_NORM2))  // stored as the distance from one
             for (int64_t i = 0; i < wc; i++) reinterpret_cast<float*>(v.data())[i] += 1.f;
-        if (!*vec && (rc = tsb_alloc(ctx, (size_t)wc * 4, (void**)vec))) return rc;
+        if (!*vec && (rc = tsb_alloc(ctx, (size_t)n * 4, (void**)vec))) return rc;
         TSB_CUDA(ctx, cudaMemcpy(*vec, v.data(), v.size(), cudaMemcpyHostToDevice));
-        set |= 1u << which;
+        set |= 1ull << which;
         return TSB_OK;
     }
     const size_t es = m->elem;
     convert(host, host_type, wr * wc, m->f32, v);
-    if (which == TSB_P_EMBED) {
-        if (!m->embed && (rc = tsb_alloc(ctx, v.size(), &m->embed))) return rc;
-        TSB_CUDA(ctx, cudaMemcpy(m->embed, v.data(), v.size(), cudaMemcpyHostToDevice));
-        set |= 1u << which;
+    if (which == TSB_P_EMBED || which == TSB_P_POSITIONS) {
+        void*& table = which == TSB_P_EMBED ? m->embed : m->positions;
+        if (!table && (rc = tsb_alloc(ctx, v.size(), &table))) return rc;
+        TSB_CUDA(ctx, cudaMemcpy(table, v.data(), v.size(), cudaMemcpyHostToDevice));
+        set |= 1ull << which;
         return TSB_OK;
     }
     // block of n_rows x n_cols of the host tensor (hw columns wide) at (hr, hc) -> the packed matrix at (dr, dc)
     auto put_from = [&](PlainMat& mat, const uint8_t* data, int64_t hw, int64_t dr, int64_t dc, int64_t hr, int64_t hc, int64_t n_rows, int64_t n_cols) -> int32_t {
         if (!mat.data)
-            if (int32_t r = zeroed(ctx, (size_t)mat.rows * mat.cols * es, &mat.data)) return r;
+            if (int32_t r = zeroed(ctx, (size_t)mat.rows * (l && (&mat == &l->ff_in || &mat == &l->ff_out) ? X : 1) * mat.cols * es, &mat.data)) return r;
         const size_t pitch = (size_t)mat.cols * es;
         TSB_CUDA(ctx, cudaMemcpy2D(static_cast<uint8_t*>(mat.data) + (size_t)dr * pitch + (size_t)dc * es, pitch, data + ((size_t)hr * hw + hc) * es, (size_t)hw * es,
                                    (size_t)n_cols * es, (size_t)n_rows, cudaMemcpyHostToDevice));
@@ -857,7 +1287,6 @@ int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t
         if ((rc = put(__VA_ARGS__))) return rc;   \
     } while (0)
     // rows hr + i and hr + half + i of the host tensor are the coordinates of pair `first` + i
-    const InRows at = l ? in_rows(*l) : InRows();
     auto put_pairs = [&](int64_t first, int64_t hr, int64_t half) -> int32_t {
         for (int64_t i = 0; i < half;) {
             const int64_t p = first + i, n = std::min<int64_t>(8 - p % 8, half - i), dr = at.pairs + p / 8 * 16 + p % 8;
@@ -914,14 +1343,35 @@ int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t
             for (int64_t h = 0; h < H; h++) PUT(l->out, 0, h * l->value_pad, 0, h * E, d, E);
             break;
         case TSB_P_FF_GATE: case TSB_P_FF_UP: {
-            const int64_t row0 = (post ? 0 : at.pairs) + (which == TSB_P_FF_UP ? 8 : 0);
-            for (int64_t i = 0; i < F; i += 8) PUT(post ? l->ff_in : l->in, row0 + 2 * i, 0, i, 0, std::min<int64_t>(8, F - i), d);
+            const int64_t row0 = (seq ? 0 : at.pairs) + (which == TSB_P_FF_UP ? 8 : 0);
+            for (int64_t x = 0; x < X; x++) {
+                PlainMat& mat = seq ? l->ff_in : l->in;
+                int64_t i = 0;
+                if (mat.data && mat.cols == d && F >= 16) {  // whole groups of eight rows at once
+                    i = F / 8 * 8;
+                    TSB_CUDA(ctx, cudaMemcpy2D(static_cast<uint8_t*>(mat.data) + (size_t)(x * mat.rows * seq + row0) * d * es, (size_t)16 * d * es,
+                                               v.data() + (size_t)x * F * d * es, (size_t)8 * d * es, (size_t)8 * d * es, (size_t)F / 8, cudaMemcpyHostToDevice));
+                }
+                for (; i < F; i += 8) PUT(mat, x * mat.rows * seq + row0 + 2 * i, 0, x * F + i, 0, std::min<int64_t>(8, F - i), d);
+            }
             break;
         }
-        case TSB_P_FF_DOWN: PUT(post ? l->ff_out : l->out, 0, post ? 0 : l->o_cols, 0, 0, d, F); break;
+        case TSB_P_FF_DOWN:
+            for (int64_t x = 0; x < X; x++) PUT(seq ? l->ff_out : l->out, x * l->ff_out.rows, seq ? 0 : l->o_cols, x * d, 0, d, F);
+            break;
+        case TSB_P_ROUTER: PUT(l->router, 0, 0, 0, 0, wr, d); break;
+        // the recurrence's vectors: queries, keys and values (MLSTM), values, output gates; SSD: z | x | B | C, its steps with the gates
+        case TSB_P_REC_Q: PUT(l->in, at.rec, 0, 0, 0, wr, d); break;
+        case TSB_P_REC_K: PUT(l->in, at.rec + rh * RD, 0, 0, 0, wr, d); break;
+        case TSB_P_REC_V: PUT(l->in, at.rec + (mlstm ? 2 : 1) * rh * RD, 0, 0, 0, wr, d); break;
+        case TSB_P_REC_GATE: PUT(l->in, at.rec + 2 * rh * RD + rh * RE, 0, 0, 0, wr, d); break;
+        case TSB_P_REC_I: PUT(l->in, at.rec_gate, 0, 0, 0, wr, d); break;
+        case TSB_P_REC_F: PUT(l->in, at.rec_gate + (mlstm ? rh : 0), 0, 0, 0, wr, d); break;
+        case TSB_P_REC_IN: PUT(l->in, at.rec, 0, 0, 0, wr, d); break;
+        case TSB_P_REC_O: PUT(l->out, 0, l->o_cols, 0, 0, d, rh * RE); break;
     }
 #undef PUT
-    set |= 1u << which;
+    set |= 1ull << which;
     return TSB_OK;
 }
 
@@ -942,11 +1392,12 @@ int32_t tsb_model_fill_plain(tsb_model* tm, uint64_t seed) {
     };
     auto matrix = [&](PlainMat& w, int64_t valid, float gain) { fill(&w.data, m->f32, w.rows, w.cols, valid, 0.f, gain * sqrtf(3.f / (float)valid)); };
     auto vector = [&](float*& p, int64_t n, float mid, float amp) { fill((void**)&p, true, 1, n, n, mid, amp); };
-    const int64_t d = m->cfg.d_model, gains = m->cfg.post_norm ? d : 1;
+    const int64_t d = m->cfg.d_model, gains = m->cfg.post_norm || m->cfg.output_norm ? d : 1;
     fill(&m->embed, m->f32, m->cfg.vocab, d, d, 0.f, 1.7f);
     matrix(m->head, d, 1.f);
     vector(m->final_gain, gains, 1.f, 0.f);
-    m->set = ~0u;
+    if (m->cfg.positions > 0) fill(&m->positions, m->f32, m->cfg.positions, d, d, 0.f, 0.3f);
+    m->set = ~0ull;
     for (PlainLayer& l : m->layers) {
         const tsb_plain_layer& c = l.cfg;
         matrix(l.in, d, 1.f);
@@ -955,14 +1406,30 @@ int32_t tsb_model_fill_plain(tsb_model* tm, uint64_t seed) {
         if (c.token_shift) vector(l.mu, d, 0.5f, 0.4f);
         if (c.log_bias) vector(l.r1, c.n_q_heads, 1.f, 0.5f), vector(l.r2, c.n_q_heads, 0.3f, 0.2f);
         if (c.sink) vector(l.sink, c.n_q_heads, 0.f, 1.f);
-        if (c.qk_norm) vector(l.q_norm, c.head_dim, 1.f, 0.2f), vector(l.k_norm, c.head_dim, 1.f, 0.2f);
-        if (l.post_norm && c.ffn > 0) matrix(l.ff_in, d, 1.f), matrix(l.ff_out, c.ffn, 0.5f), vector(l.norm2, d, 1.f, 0.f);
+        const int64_t whole = c.qk_norm == TSB_NORM_PROJECTION ? 1 : 0;
+        if (c.qk_norm) vector(l.q_norm, c.head_dim * (whole ? c.n_q_heads : 1), 1.f, 0.2f), vector(l.k_norm, c.head_dim * (whole ? c.n_kv_heads : 1), 1.f, 0.2f);
+        auto experts = [&](PlainMat& w, int64_t valid, float gain) {
+            fill(&w.data, m->f32, w.rows * std::max(1, c.experts), w.cols, valid, 0.f, gain * sqrtf(3.f / (float)valid));
+        };
+        if (l.post_norm && c.ffn > 0) experts(l.ff_in, d, 1.f), experts(l.ff_out, c.ffn, 0.5f), vector(l.norm2, d, 1.f, 0.f);
+        if (c.experts > 0) matrix(l.router, d, 1.f), vector(l.correction, c.experts, 0.f, 0.1f);
+        if (m->cfg.conv_taps > 0) vector(l.conv1, d * m->cfg.conv_taps, 0.f, 0.3f);
+        if (m->cfg.conv_taps > 0 && c.ffn > 0) vector(l.conv2, d * m->cfg.conv_taps, 0.f, 0.3f);
+        if (c.qkv_bias || c.recurrence) vector(l.in_bias, l.in.rows, 0.f, 0.2f);
+        if (c.recurrence) {
+            const int64_t inner = (int64_t)c.rec_heads * c.rec_vdim;
+            vector(l.rec_norm, c.recurrence == TSB_REC_FORGET ? c.rec_vdim : inner, 1.f, 0.2f);
+            if (c.recurrence == TSB_REC_FORGET) vector(l.rec_lower, (int64_t)c.rec_heads * c.rec_dim, 0.5f, 0.4f);
+            if (c.recurrence == TSB_REC_SSD)
+                vector(l.rec_conv, rec_conv_channels(c) * c.rec_taps, 0.f, 0.5f), vector(l.rec_conv_bias, rec_conv_channels(c), 0.f, 0.2f),
+                    vector(l.rec_a_log, c.rec_heads, 0.f, 1.f), vector(l.rec_skip, c.rec_heads, 1.f, 0.2f);
+        }
         if (l.mixer == MIX_LATENT) {
             vector(l.c_norm, c.kv_rank, 1.f, 0.f);
             matrix(l.absorb, c.head_dim, 1.f), matrix(l.lift, c.kv_rank, 1.f);
             if (l.expands) matrix(l.expand, c.kv_rank, 1.f);
         }
-        l.set = ~0u;
+        l.set = ~0ull;
     }
     if (rc) return rc;
     TSB_CUDA(ctx, cudaDeviceSynchronize());
@@ -1077,7 +1544,8 @@ int32_t tsb_plain_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, int32_t la
     if (!ctx || !keys) return TSB_ERR_INVALID;
     const tsb_attention_extras x = extras ? *extras : tsb_attention_extras{};
     TSB_REQUIRE(ctx, !keys->key_layers.empty() && layer >= 0 && layer < (int)keys->key_layers.size(), "a plain cache and one of its layers expected");
-    TSB_REQUIRE(ctx, q && out && rows_dev && group_rows && n_groups > 0 && scratch && (x.r1 == nullptr) == (x.r2 == nullptr) && x.window >= 0, "bad arguments");
+    TSB_REQUIRE(ctx, q && out && rows_dev && group_rows && n_groups > 0 && scratch && (x.r1 == nullptr) == (x.r2 == nullptr) && x.window >= 0 &&
+                         x.chunk >= 0 && !(x.window && x.chunk) && !(x.r1 && x.slopes), "bad arguments");
     const KeyView& kv = keys->key_layers[layer];
     const bool f32 = kv.elem_bytes == 4;
     const int vd = kv.value_off ? kv.head_step - kv.value_off : kv.head_dim;
@@ -1097,6 +1565,7 @@ int32_t tsb_plain_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, int32_t la
     a.keys = kv, a.q = q, a.q_stride = q_stride, a.out = out, a.out_stride = out_stride, a.gate = x.head_gate, a.rows = rows_dev;
     a.n_q_heads = n_q_heads, a.scale = scale, a.cap = x.cap, a.r1 = x.r1, a.r2 = x.r2, a.window = x.window;
     a.sink = x.sink, a.value_gate = x.value_gate, a.value_gate_stride = x.value_gate_stride, a.value_dim = vd;
+    a.slopes = x.slopes, a.chunk = x.chunk, a.out_scale = x.out_scale == 0.f ? 1.f : x.out_scale;
     AttnBatch b;
     b.max_len = max_len;
     bool uniform = true;

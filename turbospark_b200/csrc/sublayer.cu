@@ -1,0 +1,505 @@
+// Row operators around the sublayers of output-norm layers (sublayer.cuh).
+#include <cuda_bf16.h>
+
+#include "sublayer.cuh"
+
+namespace {
+
+constexpr int THREADS = 256, WARPS = THREADS / 32;
+
+__device__ __forceinline__ void put(float* p, float v) { *p = v; }
+__device__ __forceinline__ void put(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
+
+// W (1 or 4) neighbouring numbers
+template <int W>
+struct Vec {
+    float v[W];
+};
+template <int W>
+__device__ __forceinline__ Vec<W> zeros() {
+    Vec<W> r;
+#pragma unroll
+    for (int i = 0; i < W; i++) r.v[i] = 0.f;
+    return r;
+}
+__device__ __forceinline__ Vec<1> load(const float* p, Vec<1>) { return Vec<1>{{*p}}; }
+__device__ __forceinline__ Vec<4> load(const float* p, Vec<4>) {
+    const float4 f = *reinterpret_cast<const float4*>(p);
+    return Vec<4>{{f.x, f.y, f.z, f.w}};
+}
+__device__ __forceinline__ Vec<1> load(const __nv_bfloat16* p, Vec<1>) { return Vec<1>{{__bfloat162float(*p)}}; }
+__device__ __forceinline__ Vec<4> load(const __nv_bfloat16* p, Vec<4>) {
+    const uint2 w = *reinterpret_cast<const uint2*>(p);
+    return Vec<4>{{__uint_as_float(w.x << 16), __uint_as_float(w.x & 0xFFFF0000u), __uint_as_float(w.y << 16), __uint_as_float(w.y & 0xFFFF0000u)}};
+}
+__device__ __forceinline__ void store(float* p, const Vec<1>& a) { *p = a.v[0]; }
+__device__ __forceinline__ void store(float* p, const Vec<4>& a) { *reinterpret_cast<float4*>(p) = make_float4(a.v[0], a.v[1], a.v[2], a.v[3]); }
+__device__ __forceinline__ void store(__nv_bfloat16* p, const Vec<1>& a) { *p = __float2bfloat16_rn(a.v[0]); }
+__device__ __forceinline__ void store(__nv_bfloat16* p, const Vec<4>& a) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(a.v[0], a.v[1]), hi = __floats2bfloat162_rn(a.v[2], a.v[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+}
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+    return v;
+}
+__device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+
+// 1 / rms of the group that column c belongs to, from the columns' squares.  A thread holds columns (k * THREADS + thread) * W + i, k < V.
+// FAST: groups are multiples of 32 W columns, so a warp's columns of one k share a group and the whole reduction takes one barrier.
+// sq: shared memory, two of them used in turn (call with parity 0, 1, 0, ...).
+template <int V, int W, bool FAST>
+struct GroupNorm {
+    int d, width, groups;
+    float eps;
+    float *sq, *sums;  // FAST: [2][V * WARPS]; else sq [d / W], sums [groups]
+    __device__ __forceinline__ void rms(const Vec<W> (&x)[V], int parity, float (&inv)[V]) const {
+        float s[V];
+#pragma unroll
+        for (int k = 0; k < V; k++) {
+            s[k] = 0.f;
+#pragma unroll
+            for (int i = 0; i < W; i++) s[k] = fmaf(x[k].v[i], x[k].v[i], s[k]);
+        }
+        const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+        if (FAST) {
+            float* red = sq + parity * V * WARPS;
+#pragma unroll
+            for (int k = 0; k < V; k++) {
+                const float t = warp_sum(s[k]);
+                if (lane == 0) red[k * WARPS + warp] = t;
+            }
+            __syncthreads();
+            const int per = width / (32 * W);  // warp runs per group
+#pragma unroll
+            for (int k = 0; k < V; k++) {
+                const int g = (k * WARPS + warp) / per;
+                float t = 0.f;
+                if ((k * THREADS + (int)threadIdx.x) * W < d)
+                    for (int i = 0; i < per; i++) t += red[g * per + i];
+                inv[k] = 1.f / sqrtf(t / (float)width + eps);
+            }
+        } else {
+#pragma unroll
+            for (int k = 0; k < V; k++) {
+                const int u = k * THREADS + threadIdx.x;
+                if (u * W < d) sq[u] = s[k];
+            }
+            __syncthreads();
+            const int per = width / W;
+            for (int g = warp; g < groups; g += WARPS) {
+                float t = 0.f;
+                for (int i = lane; i < per; i += 32) t += sq[g * per + i];
+                t = warp_sum(t);
+                if (lane == 0) sums[g] = 1.f / sqrtf(t / (float)width + eps);
+            }
+            __syncthreads();
+#pragma unroll
+            for (int k = 0; k < V; k++) {
+                const int c = (k * THREADS + threadIdx.x) * W;
+                inv[k] = c < d ? sums[c / width] : 0.f;
+            }
+            // the next call's first barrier separates its writes of sums from these reads; sq is rewritten only behind the second one above
+        }
+    }
+};
+template <int V, int W>
+size_t group_norm_smem(int d, int groups, bool fast) {
+    return (fast ? (size_t)2 * V * WARPS : (size_t)(d / W + groups)) * sizeof(float);
+}
+
+// ------------------------------------------------------------------ end of a sublayer
+enum SublayerSource { FROM_Y, FROM_EXPERTS, FROM_TABLE };
+
+template <typename T, int V, int W, bool FAST, int TM>
+__global__ void __launch_bounds__(THREADS) sublayer_end_kernel(const __grid_constant__ SublayerEnd s, uint32_t* __restrict__ err) {
+    extern __shared__ float smem[];
+    const AttnTile tile = row_tile(s.tiles, blockIdx.x);
+    const tsb_row_desc rd = s.rows[tile.row_first];
+    const int d = s.d, halo = s.taps > 0 ? min(s.taps - 1, rd.slot) : 0;
+    const bool ok = s.taps == 0 || (rd.seq >= 0 && rd.seq < s.ring.n_streams);
+    GroupNorm<V, W, FAST> norm;
+    norm.d = d, norm.groups = s.groups, norm.width = d / s.groups, norm.eps = s.eps, norm.sq = smem, norm.sums = smem + d / W;
+    Vec<W> hist[TM - 1][V];  // hist[j]: the row j + 1 before the current one
+    Vec<W> w[V];
+#pragma unroll
+    for (int k = 0; k < V; k++) {
+        const int c = (k * THREADS + threadIdx.x) * W;
+        w[k] = c < d && s.norm_w ? load(s.norm_w + c, Vec<W>()) : zeros<W>();
+    }
+    pdl_wait();
+    pdl_launch_dependents();
+    if (!ok) {
+        if (threadIdx.x == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+        return;
+    }
+    const int first = tile.row_first - halo, pos_first = rd.base + rd.slot - halo;
+#pragma unroll
+    for (int j = 0; j < TM - 1; j++) {
+        const int pos = pos_first - 1 - j;
+        const bool in = j < s.taps - 1 - halo && pos >= 0;  // fewer halo rows than taps: the portion starts at `first`
+        const float* p = in ? ring_row_before(s.ring, rd.seq, rd.base, pos, s.use_before) : nullptr;
+#pragma unroll
+        for (int k = 0; k < V; k++) {
+            const int c = (k * THREADS + threadIdx.x) * W;
+            hist[j][k] = in && c < d ? load(p + c, Vec<W>()) : zeros<W>();
+        }
+    }
+    for (int r = first, parity = 0; r < tile.row_first + tile.n_rows; r++, parity ^= 1) {
+        Vec<W> x[V];
+        if (s.table) {
+            const int tok = s.tokens[(int64_t)r * s.token_stride], pos = pos_first + (r - first);
+            const bool bad = tok < 0 || tok >= s.vocab || (s.positions && pos >= s.n_positions);
+            if (bad && threadIdx.x == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+#pragma unroll
+            for (int k = 0; k < V; k++) {
+                const int c = (k * THREADS + threadIdx.x) * W;
+                x[k] = zeros<W>();
+                if (bad || c >= d) continue;
+                x[k] = load(static_cast<const T*>(s.table) + (int64_t)tok * d + c, Vec<W>());
+                const Vec<W> p = s.positions ? load(static_cast<const T*>(s.positions) + (int64_t)pos * d + c, Vec<W>()) : zeros<W>();
+#pragma unroll
+                for (int i = 0; i < W; i++) x[k].v[i] = fmaf(s.embed_scale, x[k].v[i], p.v[i]);
+            }
+        } else {
+            Vec<W> y[V];
+            if (s.y) {
+#pragma unroll
+                for (int k = 0; k < V; k++) {
+                    const int c = (k * THREADS + threadIdx.x) * W;
+                    y[k] = c < d ? load(s.y + (int64_t)r * d + c, Vec<W>()) : zeros<W>();
+                }
+            } else {
+#pragma unroll
+                for (int k = 0; k < V; k++) y[k] = zeros<W>();
+                for (int e = 0; e < s.top; e++) {
+                    const float f = s.weight[(int64_t)r * s.top + e];
+                    const T* row = static_cast<const T*>(s.experts) + (int64_t)s.slot_of[(int64_t)r * s.top + e] * s.expert_stride;
+#pragma unroll
+                    for (int k = 0; k < V; k++) {
+                        const int c = (k * THREADS + threadIdx.x) * W;
+                        if (c >= d) continue;
+                        const Vec<W> v = load(row + c, Vec<W>());
+#pragma unroll
+                        for (int i = 0; i < W; i++) y[k].v[i] = fmaf(f, v.v[i], y[k].v[i]);
+                    }
+                }
+            }
+#pragma unroll
+            for (int k = 0; k < V; k++) {
+                const int c = (k * THREADS + threadIdx.x) * W;
+                x[k] = c < d ? load(s.x_in + (int64_t)r * d + c, Vec<W>()) : zeros<W>();
+            }
+            float inv[V];
+            norm.rms(y, parity, inv);
+#pragma unroll
+            for (int k = 0; k < V; k++)
+#pragma unroll
+                for (int i = 0; i < W; i++) x[k].v[i] = fmaf(y[k].v[i] * inv[k], w[k].v[i], x[k].v[i]);
+        }
+        if (r >= tile.row_first) {
+            float* keep = nullptr;
+            if (s.taps > 1 && ring_keeps(s.ring, s.rows, s.n_rows, r, rd.seq)) keep = ring_row(s.ring, rd.seq, pos_first + (r - first));
+#pragma unroll
+            for (int k = 0; k < V; k++) {
+                const int c = (k * THREADS + threadIdx.x) * W;
+                if (c >= d) continue;
+                store(s.x_out + (int64_t)r * d + c, x[k]);
+                if (s.taps == 0) continue;
+                if (keep) store(keep + c, x[k]);
+                Vec<W> o = x[k];
+                const Vec<W> t0 = load(s.taps_w + (int64_t)(s.taps - 1) * d + c, Vec<W>());
+#pragma unroll
+                for (int i = 0; i < W; i++) o.v[i] = fmaf(t0.v[i], x[k].v[i], o.v[i]);
+#pragma unroll
+                for (int j = 0; j < TM - 1; j++) {
+                    if (j >= s.taps - 1) break;
+                    const Vec<W> t = load(s.taps_w + (int64_t)(s.taps - 2 - j) * d + c, Vec<W>());
+#pragma unroll
+                    for (int i = 0; i < W; i++) o.v[i] = fmaf(t.v[i], hist[j][k].v[i], o.v[i]);
+                }
+                store(static_cast<T*>(s.out) + (int64_t)r * s.out_stride + c, o);
+            }
+        }
+#pragma unroll
+        for (int j = TM - 2; j > 0; j--)
+#pragma unroll
+            for (int k = 0; k < V; k++) hist[j][k] = hist[j - 1][k];
+#pragma unroll
+        for (int k = 0; k < V; k++) hist[0][k] = x[k];
+    }
+}
+
+__global__ void __launch_bounds__(THREADS) rings_before_kernel(const RowRing* __restrict__ rings, const tsb_row_desc* __restrict__ rows) {
+    pdl_wait();
+    pdl_launch_dependents();
+    const tsb_row_desc rd = rows[blockIdx.x];
+    const RowRing r = rings[blockIdx.y];
+    if (rd.slot != 0 || rd.seq < 0 || rd.seq >= r.n_streams) return;
+    for (int k = 0; k < r.keep; k++) {
+        const int pos = rd.base - r.keep + k;
+        if (pos < 0) continue;
+        const float* src = ring_row(r, rd.seq, pos);
+        float* dst = r.before + ((int64_t)rd.seq * r.keep + k) * r.width;
+        for (int i = threadIdx.x; i < r.width; i += THREADS) dst[i] = src[i];
+    }
+}
+
+template <typename T, int V, int W, bool FAST>
+__global__ void __launch_bounds__(THREADS)
+    group_norm_rows_kernel(const float* x, int d, const float* __restrict__ weight, int groups, float eps, const int32_t* __restrict__ want, int want_first,
+                           int want_step, T* out, int64_t out_stride) {
+    extern __shared__ float smem[];
+    pdl_wait();
+    pdl_launch_dependents();
+    const int r = want ? want[blockIdx.x] : (int)blockIdx.x * want_step + want_first;
+    GroupNorm<V, W, FAST> norm;
+    norm.d = d, norm.groups = groups, norm.width = d / groups, norm.eps = eps, norm.sq = smem, norm.sums = smem + d / W;
+    Vec<W> v[V];
+    float inv[V];
+#pragma unroll
+    for (int k = 0; k < V; k++) {
+        const int c = (k * THREADS + threadIdx.x) * W;
+        v[k] = c < d ? load(x + (int64_t)r * d + c, Vec<W>()) : zeros<W>();
+    }
+    norm.rms(v, 0, inv);
+#pragma unroll
+    for (int k = 0; k < V; k++) {
+        const int c = (k * THREADS + threadIdx.x) * W;
+        if (c >= d) continue;
+        const Vec<W> w = load(weight + c, Vec<W>());
+#pragma unroll
+        for (int i = 0; i < W; i++) v[k].v[i] *= inv[k] * w.v[i];
+        store(out + (int64_t)blockIdx.x * out_stride + c, v[k]);
+    }
+}
+
+// ------------------------------------------------------------------ norms of whole projections
+// blockIdx.y: queries or keys of the row.
+template <typename T, int W>
+__global__ void __launch_bounds__(THREADS) projection_norms_kernel(const __grid_constant__ ProjectionNorms p, uint32_t* __restrict__ err) {
+    __shared__ float red[WARPS];
+    const bool query = blockIdx.y == 0;
+    const int r = blockIdx.x, heads = query ? p.n_q : p.n_k, n = heads * p.width;
+    const tsb_row_desc rd = p.rows[r];
+    const float *src = p.raw + (int64_t)r * p.raw_stride + (query ? 0 : (int64_t)p.n_q * p.width), *w = query ? p.q_weight : p.k_weight;
+    pdl_wait();
+    pdl_launch_dependents();
+    float ss = 0.f;
+    for (int i = threadIdx.x * W; i < n; i += THREADS * W) {
+        const Vec<W> v = load(src + i, Vec<W>());
+#pragma unroll
+        for (int j = 0; j < W; j++) ss = fmaf(v.v[j], v.v[j], ss);
+    }
+    ss = warp_sum(ss);
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < WARPS; i++) ss += red[i];
+    const float f = 1.f / sqrtf(ss / (float)n + p.eps);
+    T* dst;
+    int step = p.width;
+    if (query) {
+        dst = static_cast<T*>(p.q) + (int64_t)r * p.q_stride, step = p.q_step;
+    } else {
+        dst = key_row<T>(p.keys, rd.seq, rd.base + rd.slot);
+        if (!dst) {
+            if (threadIdx.x == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+            return;
+        }
+        step = p.keys.head_step;
+    }
+    for (int i = threadIdx.x * W; i < n; i += THREADS * W) {
+        Vec<W> v = load(src + i, Vec<W>());
+        const Vec<W> g = load(w + i, Vec<W>());
+#pragma unroll
+        for (int j = 0; j < W; j++) v.v[j] *= f * g.v[j];
+        store(dst + (int64_t)(i / p.width) * step + i % p.width, v);
+    }
+    if (query && step > p.width) {
+        const int tail = step - p.width;
+        for (int i = threadIdx.x; i < heads * tail; i += THREADS) put(dst + (int64_t)(i / tail) * step + p.width + i % tail, 0.f);
+    }
+}
+
+// ------------------------------------------------------------------ short convolution
+// A thread owns W channels and walks the rows of its tile with the rows before in registers.
+template <typename T, int W, int TM>
+__global__ void __launch_bounds__(THREADS) short_conv_kernel(const __grid_constant__ ShortConv s, uint32_t* __restrict__ err) {
+    const AttnTile tile = row_tile(s.tiles, blockIdx.x);
+    const tsb_row_desc rd = s.rows[tile.row_first];
+    const int c = (blockIdx.y * THREADS + threadIdx.x) * W;
+    const bool ok = rd.seq >= 0 && rd.seq < s.ring.n_streams;
+    pdl_wait();
+    pdl_launch_dependents();
+    if (!ok && threadIdx.x == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+    if (!ok || c >= s.channels) return;
+    Vec<W> w[TM], hist[TM - 1];
+    const Vec<W> bias = load(s.bias + c, Vec<W>());
+#pragma unroll
+    for (int j = 0; j < TM; j++) w[j] = j < s.taps ? load(s.w + (int64_t)(s.taps - 1 - j) * s.channels + c, Vec<W>()) : zeros<W>();  // w[j]: j rows back
+    const T* in = static_cast<const T*>(s.in) + c;
+#pragma unroll
+    for (int j = 0; j < TM - 1; j++) {
+        const int back = j + 1, pos = rd.base + rd.slot - back;
+        hist[j] = zeros<W>();
+        if (back >= s.taps || pos < 0) continue;
+        hist[j] = back <= rd.slot ? load(in + (int64_t)(tile.row_first - back) * s.in_stride, Vec<W>())
+                                  : load(ring_row_before(s.ring, rd.seq, rd.base, pos, s.use_before) + c, Vec<W>());
+    }
+    for (int i = 0; i < tile.n_rows; i++) {
+        const int r = tile.row_first + i;
+        const Vec<W> x = load(in + (int64_t)r * s.in_stride, Vec<W>());
+        if (s.taps > 1 && ring_keeps(s.ring, s.rows, s.n_rows, r, rd.seq)) store(ring_row(s.ring, rd.seq, rd.base + rd.slot + i) + c, x);
+        Vec<W> o = bias;
+#pragma unroll
+        for (int k = 0; k < W; k++) {
+#pragma unroll
+            for (int j = TM - 2; j >= 0; j--) o.v[k] = fmaf(w[j + 1].v[k], hist[j].v[k], o.v[k]);
+            o.v[k] = fmaf(w[0].v[k], x.v[k], o.v[k]);
+            o.v[k] *= sigmoid(o.v[k]);
+        }
+        store(static_cast<T*>(s.out) + (int64_t)r * s.out_stride + c, o);
+#pragma unroll
+        for (int j = TM - 2; j > 0; j--) hist[j] = hist[j - 1];
+        hist[0] = x;
+    }
+}
+
+// ------------------------------------------------------------------ gated norm of a recurrence's output
+template <typename T, int W>
+__global__ void __launch_bounds__(THREADS) gated_norm_kernel(const __grid_constant__ GatedNorm g) {
+    extern __shared__ float smem[];
+    float *v = smem, *sq = smem + g.width, *inv = sq + g.width / W;
+    const int r = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gw = g.width / g.groups;
+    pdl_wait();
+    pdl_launch_dependents();
+    for (int c = threadIdx.x * W; c < g.width; c += THREADS * W) {
+        Vec<W> x = load(g.o + (int64_t)r * g.o_stride + c, Vec<W>());
+        if (g.pre_gate) {
+            const Vec<W> z = load(static_cast<const T*>(g.pre_gate) + (int64_t)r * g.gate_stride + c, Vec<W>());
+#pragma unroll
+            for (int i = 0; i < W; i++) x.v[i] *= z.v[i] * sigmoid(z.v[i]);
+        }
+        float s = 0.f;
+#pragma unroll
+        for (int i = 0; i < W; i++) s = fmaf(x.v[i], x.v[i], s);
+        store(v + c, x);
+        sq[c / W] = s;
+    }
+    __syncthreads();
+    const int per = gw / W;
+    for (int k = warp; k < g.groups; k += WARPS) {
+        float s = 0.f;
+        for (int i = lane; i < per; i += 32) s += sq[k * per + i];
+        s = warp_sum(s);
+        if (lane == 0) inv[k] = g.scale / sqrtf(s / (float)gw + g.eps);
+    }
+    __syncthreads();
+    for (int c = threadIdx.x * W; c < g.width; c += THREADS * W) {
+        Vec<W> x = load(v + c, Vec<W>());
+        const Vec<W> w = load(g.weight + c % g.weight_n, Vec<W>());
+        const float f = inv[c / gw];
+#pragma unroll
+        for (int i = 0; i < W; i++) x.v[i] *= f * w.v[i];
+        if (g.post_gate) {
+            const Vec<W> z = load(static_cast<const T*>(g.post_gate) + (int64_t)r * g.gate_stride + c, Vec<W>());
+#pragma unroll
+            for (int i = 0; i < W; i++) x.v[i] *= sigmoid(z.v[i]);
+        }
+        store(static_cast<T*>(g.out) + (int64_t)r * g.out_stride + c, x);
+    }
+}
+
+// columns per thread and how many of them at a time: (4, V) when groups and strides are whole vectors
+constexpr int MAX_VECS4 = 8, MAX_VECS1 = 16;
+bool by_fours(int d, int groups) { return (d / groups) % 4 == 0 && d <= 4 * THREADS * MAX_VECS4; }
+
+template <typename T, int V, int W, bool FAST>
+cudaError_t launch_end(tsb_ctx* ctx, cudaStream_t st, const SublayerEnd& s) {
+    const size_t smem = group_norm_smem<V, W>(s.d, s.groups, FAST);
+    auto run = [&](auto kernel) { return tsb_launch(ctx, kernel, dim3((unsigned)s.tiles.n), dim3(THREADS), smem, st, true, s, ctx->dev_error); };
+    return s.taps <= 4 ? run(sublayer_end_kernel<T, V, W, FAST, 4>) : run(sublayer_end_kernel<T, V, W, FAST, CONV_MAX_TAPS>);
+}
+template <typename T>
+cudaError_t launch_end_of(tsb_ctx* ctx, cudaStream_t st, const SublayerEnd& s) {
+    const int d = s.d, gw = d / s.groups;
+    if (by_fours(d, s.groups) && s.out_stride % 4 == 0 && s.expert_stride % 4 == 0) {
+        const bool fast = gw % 128 == 0;
+        if (d <= 4 * THREADS) return fast ? launch_end<T, 1, 4, true>(ctx, st, s) : launch_end<T, 1, 4, false>(ctx, st, s);
+        if (d <= 4 * THREADS * 2) return fast ? launch_end<T, 2, 4, true>(ctx, st, s) : launch_end<T, 2, 4, false>(ctx, st, s);
+        if (d <= 4 * THREADS * 4) return fast ? launch_end<T, 4, 4, true>(ctx, st, s) : launch_end<T, 4, 4, false>(ctx, st, s);
+        return fast ? launch_end<T, 8, 4, true>(ctx, st, s) : launch_end<T, 8, 4, false>(ctx, st, s);
+    }
+    return d <= THREADS * 4 ? launch_end<T, 4, 1, false>(ctx, st, s) : launch_end<T, MAX_VECS1, 1, false>(ctx, st, s);
+}
+
+template <typename T>
+cudaError_t launch_norm_of(tsb_ctx* ctx, cudaStream_t st, const float* x, int d, const float* weight, int groups, float eps, const int32_t* want, int first, int step, int n,
+                           T* out, int64_t out_stride) {
+    auto run = [&](auto kernel, size_t smem) {
+        return tsb_launch(ctx, kernel, dim3((unsigned)n), dim3(THREADS), smem, st, true, x, d, weight, groups, eps, want, first, step, out, out_stride);
+    };
+    if (by_fours(d, groups) && out_stride % 4 == 0) {
+        if ((d / groups) % 128 == 0) return run(group_norm_rows_kernel<T, MAX_VECS4, 4, true>, group_norm_smem<MAX_VECS4, 4>(d, groups, true));
+        return run(group_norm_rows_kernel<T, MAX_VECS4, 4, false>, group_norm_smem<MAX_VECS4, 4>(d, groups, false));
+    }
+    return run(group_norm_rows_kernel<T, MAX_VECS1, 1, false>, group_norm_smem<MAX_VECS1, 1>(d, groups, false));
+}
+
+}  // namespace
+
+bool sublayer_end_supported(int d, int groups, int taps) {
+    return groups > 0 && d % groups == 0 && taps >= 0 && taps <= CONV_MAX_TAPS && (by_fours(d, groups) || d <= THREADS * MAX_VECS1) && d / 4 + groups <= 10000;
+}
+int sublayer_rows_per_tile(const tsb_ctx* ctx, int rows) { return rows <= 2 * ctx->sm_count ? 1 : rows <= 8 * ctx->sm_count ? 4 : 8; }
+
+cudaError_t launch_sublayer_end(tsb_ctx* ctx, cudaStream_t st, bool f32, const SublayerEnd& s) {
+    return f32 ? launch_end_of<float>(ctx, st, s) : launch_end_of<__nv_bfloat16>(ctx, st, s);
+}
+
+cudaError_t launch_rings_before(tsb_ctx* ctx, cudaStream_t st, const RowRing* rings_dev, int n, const tsb_row_desc* rows_dev, int rows) {
+    return tsb_launch(ctx, rings_before_kernel, dim3((unsigned)rows, (unsigned)n), dim3(THREADS), 0, st, true, rings_dev, rows_dev);
+}
+
+cudaError_t launch_group_norm_rows(tsb_ctx* ctx, cudaStream_t st, bool f32, const float* x, int d, const float* weight, int groups, float eps, const int32_t* want_dev,
+                                   int want_first, int want_step, int n, void* out, int64_t out_stride) {
+    return f32 ? launch_norm_of(ctx, st, x, d, weight, groups, eps, want_dev, want_first, want_step, n, (float*)out, out_stride)
+               : launch_norm_of(ctx, st, x, d, weight, groups, eps, want_dev, want_first, want_step, n, (__nv_bfloat16*)out, out_stride);
+}
+
+cudaError_t launch_projection_norms(tsb_ctx* ctx, cudaStream_t st, bool f32, const ProjectionNorms& p, int rows) {
+    auto run = [&](auto kernel) { return tsb_launch(ctx, kernel, dim3((unsigned)rows, 2), dim3(THREADS), 0, st, true, p, ctx->dev_error); };
+    const bool vec = p.width % 4 == 0 && p.raw_stride % 4 == 0 && p.q_stride % 4 == 0 && p.q_step % 4 == 0 && p.keys.head_step % 4 == 0;
+    if (f32) return vec ? run(projection_norms_kernel<float, 4>) : run(projection_norms_kernel<float, 1>);
+    return vec ? run(projection_norms_kernel<__nv_bfloat16, 4>) : run(projection_norms_kernel<__nv_bfloat16, 1>);
+}
+
+cudaError_t launch_short_conv(tsb_ctx* ctx, cudaStream_t st, bool f32, const ShortConv& c) {
+    const bool vec = c.channels % 4 == 0 && c.in_stride % 4 == 0 && c.out_stride % 4 == 0 && (uintptr_t)c.in % 16 == 0;
+    auto run = [&](auto kernel, int w) {
+        return tsb_launch(ctx, kernel, dim3((unsigned)c.tiles.n, (unsigned)((c.channels + THREADS * w - 1) / (THREADS * w))), dim3(THREADS), 0, st, true, c, ctx->dev_error);
+    };
+    if (c.taps <= 4) {
+        if (f32) return vec ? run(short_conv_kernel<float, 4, 4>, 4) : run(short_conv_kernel<float, 1, 4>, 1);
+        return vec ? run(short_conv_kernel<__nv_bfloat16, 4, 4>, 4) : run(short_conv_kernel<__nv_bfloat16, 1, 4>, 1);
+    }
+    return f32 ? run(short_conv_kernel<float, 1, CONV_MAX_TAPS>, 1) : run(short_conv_kernel<__nv_bfloat16, 1, CONV_MAX_TAPS>, 1);
+}
+
+cudaError_t launch_gated_norm(tsb_ctx* ctx, cudaStream_t st, bool f32, const GatedNorm& g, int rows) {
+    const int gw = g.width / g.groups;
+    const bool vec = gw % 4 == 0 && g.weight_n % 4 == 0 && g.o_stride % 4 == 0 && g.out_stride % 4 == 0 && g.gate_stride % 4 == 0 &&
+                     (uintptr_t)g.pre_gate % 16 == 0 && (uintptr_t)g.post_gate % 16 == 0 && (uintptr_t)g.out % 16 == 0;
+    auto run = [&](auto kernel, int w, SmemOptIn& configured) {
+        const size_t smem = ((size_t)g.width + g.width / w + g.groups) * sizeof(float);
+        if (smem > 48 * 1024)
+            if (cudaError_t e = tsb_opt_in_smem(ctx, kernel, 200 * 1024, configured); e != cudaSuccess) return e;
+        return tsb_launch(ctx, kernel, dim3((unsigned)rows), dim3(THREADS), smem, st, true, g);
+    };
+    static SmemOptIn configured[4];
+    if (f32) return vec ? run(gated_norm_kernel<float, 4>, 4, configured[0]) : run(gated_norm_kernel<float, 1>, 1, configured[1]);
+    return vec ? run(gated_norm_kernel<__nv_bfloat16, 4>, 4, configured[2]) : run(gated_norm_kernel<__nv_bfloat16, 1>, 1, configured[3]);
+}
