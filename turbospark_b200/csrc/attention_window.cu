@@ -116,13 +116,13 @@ __global__ void __launch_bounds__(F32_WARPS * 32) window_attn_f32_kernel(const _
         float s = -INFINITY;
         if (k) {
             k += (int64_t)kvh * a.keys.head_step;
-            float dot = 0.f;
+            float4 dot = make_float4(0.f, 0.f, 0.f, 0.f);
             for (int i = 0; i < D; i += 4) {
                 const float4 v = *reinterpret_cast<const float4*>(k + i);
-                dot = fmaf(v.x, qs[warp][i], dot), dot = fmaf(v.y, qs[warp][i + 1], dot);
-                dot = fmaf(v.z, qs[warp][i + 2], dot), dot = fmaf(v.w, qs[warp][i + 3], dot);
+                dot.x = fmaf(v.x, qs[warp][i], dot.x), dot.y = fmaf(v.y, qs[warp][i + 1], dot.y);
+                dot.z = fmaf(v.z, qs[warp][i + 2], dot.z), dot.w = fmaf(v.w, qs[warp][i + 3], dot.w);
             }
-            s = dot * a.scale;
+            s = ((dot.x + dot.y) + (dot.z + dot.w)) * a.scale;
             if (a.cap > 0.f) s = a.cap * tanhf(s / a.cap);
             if (a.r1) s -= r1 * logf(1.f + r2 * (float)(pos - j));
             if (a.slopes) s -= slope * (float)(pos - j);

@@ -296,6 +296,7 @@ __global__ void __launch_bounds__(256)
         ws[lc][lr] = a.x, ws[lc + 1][lr] = a.y, ws[lc + 2][lr] = a.z, ws[lc + 3][lr] = a.w;
         xs[lc][lr] = b.x, xs[lc + 1][lr] = b.y, xs[lc + 2][lr] = b.z, xs[lc + 3][lr] = b.w;
         __syncthreads();
+        float part[4][4] = {};  // sums of a slice first: rounding grows with the number of slices, not of columns
 #pragma unroll
         for (int k = 0; k < F32_K; k++) {
             float wv[4], xv[4];
@@ -304,8 +305,12 @@ __global__ void __launch_bounds__(256)
 #pragma unroll
             for (int i = 0; i < 4; i++)
 #pragma unroll
-                for (int j = 0; j < 4; j++) acc[i][j] = fmaf(wv[i], xv[j], acc[i][j]);
+                for (int j = 0; j < 4; j++) part[i][j] = fmaf(wv[i], xv[j], part[i][j]);
         }
+#pragma unroll
+        for (int i = 0; i < 4; i++)
+#pragma unroll
+            for (int j = 0; j < 4; j++) acc[i][j] += part[i][j];
         __syncthreads();
     }
     pdl_launch_dependents();

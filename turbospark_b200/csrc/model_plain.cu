@@ -242,7 +242,7 @@ int32_t states_init(tsb_session* s, const PlainModel* m, const SessionShape& sha
         const size_t heads = (size_t)shape.n_streams * st.ring * c.rec_heads;
         if (c.recurrence && rc == TSB_OK) rc = zero(heads * c.rec_dim * recurrence_v_pitch(c.rec_vdim) * 4, (void**)&r.s);
         if (c.recurrence == TSB_REC_MLSTM && rc == TSB_OK) rc = zero(heads * c.rec_dim * 4, (void**)&r.norm);
-        if (c.recurrence == TSB_REC_MLSTM && rc == TSB_OK) rc = zero(heads * 4, (void**)&r.top);
+        if (c.recurrence == TSB_REC_MLSTM && rc == TSB_OK) rc = zero(heads * 8, (void**)&r.top);
         st.states.push_back(r);
     }
     if (rc) return rc;

@@ -3,7 +3,8 @@
 // A CTA owns 32 value columns of one head of one portion; its slice of the state stays in registers over the portion's rows.  Eight
 // lanes hold four columns each, the CTA's 32 such groups of lanes share out the state's rows (CR each).  Rows go through in batches:
 // their q, k, v and gates are brought to shared memory, every thread steps through the batch without a barrier and leaves its part of
-// each output, then the parts are added.  One batch of one row - a decoded token - reads and writes the state once.
+// each output, then the parts are added.  Decays are applied as s + (decay - 1) s, with decay - 1 from expm1 or the gate itself: close to one
+// the rounding of the factor would add up over a long memory.  One batch of one row - a decoded token - reads and writes the state once.
 #include <algorithm>
 
 #include "recurrence_dev.cuh"
@@ -14,15 +15,18 @@ constexpr int THREADS = 256, COLS = 32, GROUPS = THREADS / 8, BATCH = 8;
 
 template <int KIND>
 size_t rows_smem(int dim_pad) {
-    return ((size_t)BATCH * dim_pad * (KIND == REC_FORGET ? 3 : 2) + BATCH * COLS + (size_t)BATCH * GROUPS * COLS + (KIND == REC_MLSTM ? BATCH * GROUPS : 0) + 3 * BATCH) *
+    return ((size_t)BATCH * dim_pad * 2 + BATCH * COLS + (size_t)BATCH * GROUPS * COLS + (KIND == REC_MLSTM ? BATCH * GROUPS : 0) + 3 * BATCH) *
            sizeof(float);
 }
+
+// is the state after row t of the portion one of those that are kept?
+__device__ __forceinline__ bool is_kept(const Recurrence& a, const AttnTile& p, int t) { return t + a.state.ring >= p.n_rows; }
 
 template <typename T, int KIND, int CR>
 __global__ void __launch_bounds__(THREADS) recurrence_rows_kernel(const __grid_constant__ Recurrence a, const __grid_constant__ RowTiles portions, uint32_t* __restrict__ err) {
     constexpr int DIM = GROUPS * CR;
     extern __shared__ __align__(16) float smem[];
-    float *qs = smem, *ks = qs + BATCH * DIM, *fs = ks + BATCH * DIM, *vs = fs + (KIND == REC_FORGET ? BATCH * DIM : 0);
+    float *qs = smem, *ks = qs + BATCH * DIM, *vs = ks + BATCH * DIM;
     float *parts = vs + BATCH * COLS, *nparts = parts + BATCH * GROUPS * COLS, *decay = nparts + (KIND == REC_MLSTM ? BATCH * GROUPS : 0);
     float *write = decay + BATCH, *floor_ = write + BATCH;
     const int head = blockIdx.y, col0 = blockIdx.x * COLS;
@@ -39,7 +43,7 @@ __global__ void __launch_bounds__(THREADS) recurrence_rows_kernel(const __grid_c
     // the state was written by an earlier pass
     float4 s[CR];
     float n[KIND == REC_MLSTM ? CR : 1];
-    float top = 0.f;
+    double top = 0.0;
     const int64_t head_state = (int64_t)a.dim * vp;
     {
         const int64_t at = (rec_slot(a, rd.seq, pos0 - 1) * a.heads + head);
@@ -62,16 +66,20 @@ __global__ void __launch_bounds__(THREADS) recurrence_rows_kernel(const __grid_c
             if (threadIdx.x < nb) {
                 const int t = threadIdx.x;
                 const float2 g = KIND == REC_MLSTM ? mlstm_gates(a, row0 + t, head) : ssd_gates(a, row0 + t, head, rate);
-                if (KIND == REC_SSD) write[t] = g.x, decay[t] = expf(g.y);
+                if (KIND == REC_SSD) write[t] = g.x, decay[t] = expm1f(g.y);
                 else write[t] = g.x, decay[t] = g.y;
             }
             if (KIND == REC_MLSTM) {
                 // the running maximum: every thread walks it, the first ones keep the factors
                 __syncthreads();
-                float m = top, mine_w = 0.f, mine_d = 0.f, mine_m = 0.f;
+                double m = top;
+                float mine_w = 0.f, mine_d = 0.f, mine_m = 0.f;
                 for (int t = 0; t < nb; t++) {
-                    const float keep = decay[t] + m, m_new = fmaxf(keep, write[t]);
-                    if (t == (int)threadIdx.x) mine_d = expf(keep - m_new), mine_w = expf(write[t] - m_new), mine_m = m_new;
+                    const double keep = (double)decay[t] + m, m_new = fmax(keep, (double)write[t]);
+                    if (t == (int)threadIdx.x) {
+                        mine_d = expm1f((float)(keep - m_new)), mine_w = expf((float)((double)write[t] - m_new)), mine_m = expf(-(float)m_new);
+                        if (is_kept(a, p, b0 + t) && blockIdx.x == 0) a.state.top[rec_slot(a, rd.seq, pos0 + b0 + t) * a.heads + head] = m_new;
+                    }
                     m = m_new;
                 }
                 __syncthreads();
@@ -82,20 +90,19 @@ __global__ void __launch_bounds__(THREADS) recurrence_rows_kernel(const __grid_c
         }
         for (int i = threadIdx.x; i < nb * DIM; i += THREADS) {
             const int t = i / DIM, c = i - t * DIM, row = row0 + t;
-            float q = 0.f, k = 0.f, f = 1.f;
+            float q = 0.f, k = 0.f;
             if (c < a.dim) {
                 q = rec_get(static_cast<const T*>(a.q) + (int64_t)row * a.q_stride + key_at + c);
                 if (KIND == REC_FORGET) {
                     const float l = a.lower[(int64_t)head * a.dim + c];
-                    f = l + (1.f - l) * rec_sigmoid(a.gate[(int64_t)row * a.gate_stride + (int64_t)head * a.dim + c]);
-                    q = rec_silu(q), k = 1.f - f;
+                    k = (1.f - l) * rec_sigmoid(-a.gate[(int64_t)row * a.gate_stride + (int64_t)head * a.dim + c]);  // 1 - f
+                    q = rec_silu(q);
                 } else {
                     k = rec_get(static_cast<const T*>(a.k) + (int64_t)row * a.k_stride + key_at + c) * write[t];
                     q *= a.q_scale;
                 }
             }
             qs[i] = q, ks[i] = k;
-            if (KIND == REC_FORGET) fs[i] = f;
         }
         for (int i = threadIdx.x; i < nb * COLS; i += THREADS) {
             const int t = i / COLS, c = col0 + i % COLS;
@@ -109,15 +116,20 @@ __global__ void __launch_bounds__(THREADS) recurrence_rows_kernel(const __grid_c
             float on = 0.f;
 #pragma unroll
             for (int r = 0; r < CR; r++) {
-                const float k = ks[t * DIM + c0 + r], q = qs[t * DIM + c0 + r], d = KIND == REC_FORGET ? fs[t * DIM + c0 + r] : dt;
-                s[r].x = fmaf(d, s[r].x, k * v.x), s[r].y = fmaf(d, s[r].y, k * v.y);
-                s[r].z = fmaf(d, s[r].z, k * v.z), s[r].w = fmaf(d, s[r].w, k * v.w);
+                const float k = ks[t * DIM + c0 + r], q = qs[t * DIM + c0 + r];
+                if (KIND == REC_FORGET) {  // f s + (1 - f) v
+                    s[r].x = fmaf(k, v.x - s[r].x, s[r].x), s[r].y = fmaf(k, v.y - s[r].y, s[r].y);
+                    s[r].z = fmaf(k, v.z - s[r].z, s[r].z), s[r].w = fmaf(k, v.w - s[r].w, s[r].w);
+                } else {
+                    s[r].x = fmaf(k, v.x, fmaf(dt, s[r].x, s[r].x)), s[r].y = fmaf(k, v.y, fmaf(dt, s[r].y, s[r].y));
+                    s[r].z = fmaf(k, v.z, fmaf(dt, s[r].z, s[r].z)), s[r].w = fmaf(k, v.w, fmaf(dt, s[r].w, s[r].w));
+                }
                 o.x = fmaf(q, s[r].x, o.x), o.y = fmaf(q, s[r].y, o.y), o.z = fmaf(q, s[r].z, o.z), o.w = fmaf(q, s[r].w, o.w);
-                if (KIND == REC_MLSTM) n[r] = fmaf(d, n[r], k), on = fmaf(q, n[r], on);
+                if (KIND == REC_MLSTM) n[r] = fmaf(dt, n[r], n[r]) + k, on = fmaf(q, n[r], on);
             }
             *reinterpret_cast<float4*>(parts + (t * GROUPS + grp) * COLS + vl * 4) = o;
             if (KIND == REC_MLSTM && vl == 0) nparts[t * GROUPS + grp] = on;
-            if (b0 + t + a.state.ring >= p.n_rows) {  // one of the states that are kept
+            if (is_kept(a, p, b0 + t)) {
                 const int64_t at = rec_slot(a, rd.seq, pos0 + b0 + t) * a.heads + head;
                 float* dst = a.state.s + at * head_state;
 #pragma unroll
@@ -126,7 +138,6 @@ __global__ void __launch_bounds__(THREADS) recurrence_rows_kernel(const __grid_c
                     if (col < vp) *reinterpret_cast<float4*>(dst + (int64_t)(c0 + r) * vp + col) = s[r];
                     if (KIND == REC_MLSTM && blockIdx.x == 0 && vl == 0) a.state.norm[at * a.dim + c0 + r] = n[r];
                 }
-                if (KIND == REC_MLSTM && blockIdx.x == 0 && threadIdx.x == 0) a.state.top[at] = floor_[t];
             }
         }
         __syncthreads();
@@ -139,7 +150,7 @@ __global__ void __launch_bounds__(THREADS) recurrence_rows_kernel(const __grid_c
                 float nq = 0.f;
 #pragma unroll 8
                 for (int g = 0; g < GROUPS; g++) nq += nparts[t * GROUPS + g];
-                o /= fmaxf(fabsf(nq), expf(-floor_[t])) + 1e-6f;
+                o /= fmaxf(fabsf(nq), floor_[t]) + 1e-6f;
             }
             if (KIND == REC_SSD) o = fmaf(skip, vs[i], o);
             if (col0 + c < a.vdim) a.out[(int64_t)(row0 + t) * a.out_stride + (int64_t)head * a.vdim + col0 + c] = o;

@@ -13,7 +13,7 @@ enum RecurrenceKind {
 struct RecurrentState {
     float* s = nullptr;     // [stream][ring][heads][dim][v_pitch]
     float* norm = nullptr;  // REC_MLSTM: [stream][ring][heads][dim]
-    float* top = nullptr;   // REC_MLSTM: [stream][ring][heads]
+    double* top = nullptr;  // REC_MLSTM: [stream][ring][heads]; in double, since the decay is the exponential of small differences of it
     int ring = 0, n_streams = 0;
 };
 constexpr int recurrence_v_pitch(int vdim) { return (vdim + 3) / 4 * 4; }
