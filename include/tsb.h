@@ -565,6 +565,61 @@ TSB_API int32_t tsb_post_norm_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, flo
 TSB_API int32_t tsb_head_norm_rows(tsb_ctx* ctx, tsb_stream s, tsb_kv* cache, int32_t layer, const float* raw, int64_t raw_stride, int32_t n_q, int32_t n_k,
                                    int32_t width, const float* q_weight, const float* k_weight, float eps, float temp_coef, int32_t temp_every,
                                    const tsb_row_desc* rows_dev, int32_t rows, void* q, int64_t q_stride);
+/* The end of an output-norm sublayer and the convolution in front of the next: x_out = x_in + norm(y) in f32 (norm in `groups` equal parts, weight
+ * [d]); out = x_out + convolution of it in `type` (taps_w [taps][d], taps 0: not written).  Portions of rows_per_seq rows each.  state: f32
+ * [n_streams][ring][d], ring a power of two: x_out of the rows before and of this call's last rows.  Portions of more than ring - taps + 1
+ * rows read the taps - 1 rows before from `before` [n_streams][taps - 1][d]. */
+TSB_API int32_t tsb_output_norm_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, const float* x_in, const float* y, int32_t d, const float* weight, int32_t groups,
+                                     float eps, const float* taps_w, int32_t taps, float* state, float* before, int32_t n_streams, int32_t ring,
+                                     const tsb_row_desc* rows_dev, int32_t rows, int32_t rows_per_seq, float* x_out, void* out, int64_t out_stride);
+/* Norms of all queries, and of all keys, of a row at once: as tsb_head_norm_rows, weights [n_q * width] and [n_k * width]. */
+TSB_API int32_t tsb_projection_norm_rows(tsb_ctx* ctx, tsb_stream s, tsb_kv* cache, int32_t layer, const float* raw, int64_t raw_stride, int32_t n_q, int32_t n_k,
+                                         int32_t width, const float* q_weight, const float* k_weight, float eps, const tsb_row_desc* rows_dev, int32_t rows,
+                                         void* q, int64_t q_stride);
+/* out = silu(bias + causal convolution per channel of `in`), taps_w [taps][channels]; state and before as above, of `in`. */
+TSB_API int32_t tsb_short_conv_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, const void* in, int64_t in_stride, int32_t channels, const float* taps_w, int32_t taps,
+                                    const float* bias, float* state, float* before, int32_t n_streams, int32_t ring, const tsb_row_desc* rows_dev, int32_t rows,
+                                    int32_t rows_per_seq, void* out, int64_t out_stride);
+/* The recurrences of the recurrent mixers (see above), heads of a layer side by side. */
+typedef struct tsb_recurrence {
+    int32_t kind, heads, dim, vdim;
+    int32_t heads_per_key;           /* heads that share a q and a k (0: one) */
+    float cap, q_scale;              /* q_scale 0: one */
+    const void *q, *k, *v;           /* `type`; head h: q and k at (h / heads_per_key) * dim, v at h * vdim; FORGET: no k */
+    int64_t q_stride, k_stride, v_stride;
+    const float* gate;               /* pre-activations: FORGET [heads * dim], MLSTM [heads] input then [heads] forget gates, SSD [heads] steps */
+    int64_t gate_stride;
+    const float *lower, *a_log, *skip;
+    float* out;                      /* [rows, out_stride] f32, head h at h * vdim */
+    int64_t out_stride;
+    float* state;                    /* [n_streams][ring][heads][dim][vdim rounded up to 4]: position p in slot p & (ring - 1) */
+    float* norm;                     /* MLSTM: [n_streams][ring][heads][dim] */
+    double* top;                     /* MLSTM: [n_streams][ring][heads] */
+    int32_t ring, n_streams;
+} tsb_recurrence;
+/* chunked = 0: row by row, the states after a portion's last `ring` rows are kept; 1 (TSB_BF16): 64 rows at a time, the last one is. */
+TSB_API int32_t tsb_recurrence_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, const tsb_recurrence* r, const tsb_row_desc* rows_dev, int32_t rows,
+                                    int32_t rows_per_seq, int32_t chunked);
+/* From a recurrence's output to the output projection: o, times silu(pre_gate) when given, normed in `groups` equal parts, times weight (repeated
+ * every weight_n columns), times sigmoid(post_gate) when given, times scale. */
+TSB_API int32_t tsb_gated_norm_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, const float* o, int64_t o_stride, int32_t width, int32_t groups, const float* weight,
+                                    int32_t weight_n, float eps, float scale, const void* pre_gate, const void* post_gate, int64_t gate_stride, int32_t rows, void* out,
+                                    int64_t out_stride);
+/* Choice of experts from router logits [rows, experts] f32 (see above).  ids, weight, slot_of [rows, top]; first [experts + 1]; token_of [rows * top];
+ * chunks: room for experts + rows * top / 8 entries of three int32; n_chunks [1].  chunk_slots: 8 or 16 (TSB_BF16), 64 (TSB_F32). */
+typedef struct tsb_expert_lists {
+    int32_t* ids;
+    float* weight;
+    int32_t *slot_of, *token_of, *first, *chunks, *n_chunks;
+} tsb_expert_lists;
+TSB_API int32_t tsb_route_experts(tsb_ctx* ctx, tsb_stream s, const float* logits, const float* correction, int32_t experts, int32_t top, int32_t groups, int32_t keep,
+                                  int32_t rows, int32_t chunk_slots, const tsb_expert_lists* lists);
+/* A product per expert: W holds `experts` matrices of w_rows x cols one after another; the slots of an expert multiply its own.  x has a row per token
+ * (by_token = 1) or per slot.  pairs = 1: gate and up rows interleaved in groups of eight, y[slot, p] = silu(gate_p) * up_p for p < n_valid; 0: y[slot, n].
+ * y in `type`.  tensor = 1 (TSB_BF16, by_token = 0): for many slots per expert; x_rows rows of x are allocated. */
+TSB_API int32_t tsb_plain_gemm_experts(tsb_ctx* ctx, tsb_stream s, int32_t type, const void* w, int32_t experts, int64_t w_rows, int64_t cols, const void* x,
+                                       int64_t x_stride, int32_t x_rows, int32_t by_token, const tsb_expert_lists* lists, int32_t slots, int32_t chunk_slots,
+                                       int32_t tensor, int32_t pairs, void* y, int64_t y_stride, int32_t n_valid);
 TSB_API size_t tsb_window_attention_scratch_bytes(const tsb_ctx* ctx); /* zeroed once by the caller */
 
 /* ------------------------------------------------------------------ resident weight file

@@ -30,7 +30,7 @@ FLAGS = [
 FAMILY_UNITS = {
     "blocks": {"attention.cu", "attention_tc.cu", "comm.cu", "gemm_quant.cu", "gemm_wide.cu", "model_blocks.cu", "moe.cu", "resident.cu", "rowops.cu"},
     "plain": {"attention_kv.cu", "attention_kv_tc.cu", "attention_latent.cu", "attention_window.cu", "attention_window_tc.cu", "experts.cu", "gemm_plain.cu",
-              "model_plain.cu", "recurrence.cu", "recurrence_chunks.cu", "rowops_plain.cu", "sublayer.cu"},
+              "model_plain.cu", "ops_plain.cu", "recurrence.cu", "recurrence_chunks.cu", "rowops_plain.cu", "sublayer.cu"},
 }
 
 

@@ -347,6 +347,44 @@ class Ctx:
                                             C.c_int32(width), _vp(q_weight), _vp(k_weight), C.c_float(eps), C.c_float(temp_coef), C.c_int32(temp_every),
                                             _vp(rows_dev), C.c_int32(rows), _vp(q), C.c_int64(q_stride)))
 
+    def output_norm_rows(self, type_, x_in, y, d, weight, groups, eps, taps_w, taps, state, n_streams, ring, rows_dev, rows, rows_per_seq, x_out, out, out_stride,
+                         before=None, stream=None):
+        self.check(lib().tsb_output_norm_rows(self.h, stream, C.c_int32(type_), _vp(x_in), _vp(y), C.c_int32(d), _vp(weight), C.c_int32(groups), C.c_float(eps),
+                                              _vp(taps_w), C.c_int32(taps), _vp(state), _vp(before), C.c_int32(n_streams), C.c_int32(ring), _vp(rows_dev),
+                                              C.c_int32(rows), C.c_int32(rows_per_seq), _vp(x_out), _vp(out), C.c_int64(out_stride)))
+
+    def projection_norm_rows(self, kv, layer, raw, raw_stride, n_q, n_k, width, q_weight, k_weight, eps, rows_dev, rows, q, q_stride, stream=None):
+        self.check(lib().tsb_projection_norm_rows(self.h, stream, kv.h, C.c_int32(layer), _vp(raw), C.c_int64(raw_stride), C.c_int32(n_q), C.c_int32(n_k),
+                                                  C.c_int32(width), _vp(q_weight), _vp(k_weight), C.c_float(eps), _vp(rows_dev), C.c_int32(rows), _vp(q),
+                                                  C.c_int64(q_stride)))
+
+    def short_conv_rows(self, type_, x, x_stride, channels, taps_w, taps, bias, state, n_streams, ring, rows_dev, rows, rows_per_seq, out, out_stride, before=None,
+                        stream=None):
+        self.check(lib().tsb_short_conv_rows(self.h, stream, C.c_int32(type_), _vp(x), C.c_int64(x_stride), C.c_int32(channels), _vp(taps_w), C.c_int32(taps),
+                                             _vp(bias), _vp(state), _vp(before), C.c_int32(n_streams), C.c_int32(ring), _vp(rows_dev), C.c_int32(rows),
+                                             C.c_int32(rows_per_seq), _vp(out), C.c_int64(out_stride)))
+
+    def recurrence_rows(self, type_, rec, rows_dev, rows, rows_per_seq, chunked=False, stream=None):
+        self.check(lib().tsb_recurrence_rows(self.h, stream, C.c_int32(type_), C.byref(rec), _vp(rows_dev), C.c_int32(rows), C.c_int32(rows_per_seq),
+                                             C.c_int32(int(chunked))))
+
+    def gated_norm_rows(self, type_, o, o_stride, width, groups, weight, weight_n, eps, rows, out, out_stride, scale=1.0, pre_gate=None, post_gate=None, gate_stride=0,
+                        stream=None):
+        self.check(lib().tsb_gated_norm_rows(self.h, stream, C.c_int32(type_), _vp(o), C.c_int64(o_stride), C.c_int32(width), C.c_int32(groups), _vp(weight),
+                                             C.c_int32(weight_n), C.c_float(eps), C.c_float(scale), _vp(pre_gate), _vp(post_gate), C.c_int64(gate_stride),
+                                             C.c_int32(rows), _vp(out), C.c_int64(out_stride)))
+
+    def route_experts(self, logits, correction, experts, top, groups, keep, rows, chunk_slots, lists, stream=None):
+        self.check(lib().tsb_route_experts(self.h, stream, _vp(logits), _vp(correction), C.c_int32(experts), C.c_int32(top), C.c_int32(groups), C.c_int32(keep),
+                                           C.c_int32(rows), C.c_int32(chunk_slots), C.byref(lists.c)))
+
+    def plain_gemm_experts(self, type_, w, experts, w_rows, cols, x, x_stride, x_rows, by_token, lists, slots, chunk_slots, tensor, pairs, y, y_stride, n_valid,
+                           stream=None):
+        self.check(lib().tsb_plain_gemm_experts(self.h, stream, C.c_int32(type_), _vp(w), C.c_int32(experts), C.c_int64(w_rows), C.c_int64(cols), _vp(x),
+                                                C.c_int64(x_stride), C.c_int32(x_rows), C.c_int32(int(by_token)), C.byref(lists.c), C.c_int32(slots),
+                                                C.c_int32(chunk_slots), C.c_int32(int(tensor)), C.c_int32(int(pairs)), _vp(y), C.c_int64(y_stride),
+                                                C.c_int32(n_valid)))
+
     def residual_add(self, x, y, n, stream=None):
         self.check(lib().tsb_residual_add(self.h, stream, _vp(x), _vp(y), C.c_int64(n)))
 
@@ -410,6 +448,31 @@ class KvCache:
         if getattr(self, "h", None):
             lib().tsb_kv_destroy(self.h)
             self.h = None
+
+
+class Recurrence(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("kind", "heads", "dim", "vdim", "heads_per_key")] + [("cap", C.c_float), ("q_scale", C.c_float)] + \
+               [(n, C.c_void_p) for n in ("q", "k", "v")] + [(n, C.c_int64) for n in ("q_stride", "k_stride", "v_stride")] + \
+               [("gate", C.c_void_p), ("gate_stride", C.c_int64)] + [(n, C.c_void_p) for n in ("lower", "a_log", "skip", "out")] + \
+               [("out_stride", C.c_int64)] + [(n, C.c_void_p) for n in ("state", "norm", "top")] + [("ring", C.c_int32), ("n_streams", C.c_int32)]
+
+
+class _ExpertLists(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("ids", "weight", "slot_of", "token_of", "first", "chunks", "n_chunks")]
+
+
+class ExpertLists:
+    """Device buffers of a routed pass."""
+
+    def __init__(self, ctx, rows, top, experts):
+        n = rows * top * 4
+        self.buffers = {"ids": ctx.zeroed(n), "weight": ctx.zeroed(n), "slot_of": ctx.zeroed(n), "token_of": ctx.zeroed(n), "first": ctx.zeroed(4 * (experts + 1)),
+                        "chunks": ctx.zeroed(12 * (experts + rows * top // 8 + 1)), "n_chunks": ctx.zeroed(4)}
+        self.c = _ExpertLists(**{k: _vp(b) for k, b in self.buffers.items()})
+
+    def free(self):
+        for b in self.buffers.values():
+            b.free()
 
 
 class AttentionExtras(C.Structure):

@@ -415,8 +415,8 @@ struct PassPlan {
     std::vector<bool> is_expanded;
     const ExpandStream* expanded_dev = nullptr;
     int expanded_pages = 0, expanded_len = 0, short_first = 0, short_rows = 0;
-    // output-norm form: runs of rows for the row operators; portions whose recurrences go row by row, and chunk by chunk
-    RowTiles runs, by_row, by_chunk;
+    // output-norm form: runs of rows for the row operators; portions whose recurrences go row by row, and chunk by chunk where there is a kernel
+    RowTiles runs, by_row, by_chunk, portions;  // portions: all of them
     bool use_before = false;
 
     const AttnBatch* find(int set, int group, int rows_per_tile) const {
@@ -439,20 +439,15 @@ int32_t plan_states(tsb_session* s, const PlainModel* m, const ModelRt& rt, cons
     const int per = sublayer_rows_per_tile(s->ctx, p.rows);
     if (p.rows_per_seq > 0) {
         plan.runs = RowTiles::uniform(p.rows, p.rows_per_seq, per);
-        plan.by_row = RowTiles::uniform(p.rows, p.rows_per_seq, p.rows_per_seq);
+        plan.by_row = plan.portions = RowTiles::uniform(p.rows, p.rows_per_seq, p.rows_per_seq);
         return TSB_OK;
     }
-    bool chunks = !m->f32;
-    for (const PlainLayer& l : m->layers) {
-        Recurrence r;
-        r.kind = l.cfg.recurrence, r.dim = l.cfg.rec_dim, r.vdim = l.cfg.rec_vdim;
-        if (l.cfg.recurrence) chunks &= recurrence_chunks_supported(r);
-    }
-    std::vector<AttnTile> runs, by_row, by_chunk;
+    std::vector<AttnTile> runs, by_row, by_chunk, portions;
     for (int i = 0; i < p.n_groups; i++) {
         const RowGroup& g = p.groups[i];
         for (int r = 0; r < g.n_rows; r += per) runs.push_back({g.first_row + r, std::min(per, g.n_rows - r)});
-        const bool long_portion = chunks && g.n_rows >= CHUNK_MIN_ROWS;
+        const bool long_portion = !m->f32 && g.n_rows >= CHUNK_MIN_ROWS;
+        portions.push_back({g.first_row, g.n_rows});
         (long_portion ? by_chunk : by_row).push_back({g.first_row, g.n_rows});
         if (long_portion) rt.kv->state_lo[g.seq] = g.base + g.n_rows - 1;  // the states in between are not kept
     }
@@ -468,7 +463,8 @@ int32_t plan_states(tsb_session* s, const PlainModel* m, const ModelRt& rt, cons
     };
     int32_t rc = stage(runs, plan.runs);
     if (rc == TSB_OK) rc = stage(by_row, plan.by_row);
-    return rc == TSB_OK ? stage(by_chunk, plan.by_chunk) : rc;
+    if (rc == TSB_OK) rc = stage(by_chunk, plan.by_chunk);
+    return rc == TSB_OK ? stage(portions, plan.portions) : rc;
 }
 
 int32_t plan_pass(tsb_session* s, const PlainModel* m, const ModelRt& rt, const Pass& p, PassPlan& plan) {
@@ -745,10 +741,10 @@ struct Forward {
             r.q_stride = r.k_stride = r.v_stride = b->rec_mixed_stride, r.heads_per_key = h / c.rec_groups, r.a_log = l.rec_a_log, r.skip = l.rec_skip;
             g.pre_gate = b->rec, g.groups = c.rec_norm_groups;
         }
-        if (plan.by_chunk.n > 0)
+        const bool chunks = plan.by_chunk.n > 0 && recurrence_chunks_supported(c.recurrence, D, E);
+        if (chunks)
             if (cudaError_t e = launch_recurrence_chunks(ctx, st, r, plan.by_chunk); e != cudaSuccess) return e;
-        if (plan.by_row.n > 0)
-            if (cudaError_t e = launch_recurrence_rows(ctx, st, m->f32, r, plan.by_row); e != cudaSuccess) return e;
+        if (cudaError_t e = launch_recurrence_rows(ctx, st, m->f32, r, chunks ? plan.by_row : plan.portions); e != cudaSuccess) return e;
         return launch_gated_norm(ctx, st, m->f32, g, p.rows);
     }
 

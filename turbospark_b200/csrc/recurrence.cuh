@@ -42,5 +42,5 @@ constexpr int REC_MAX_DIM = 1024;
 cudaError_t launch_recurrence_rows(tsb_ctx* ctx, cudaStream_t st, bool f32, const Recurrence& r, const RowTiles& portions);
 // Long portions in bfloat16, REC_CHUNK rows at a time on the tensor cores; the state after the last row is kept.
 constexpr int REC_CHUNK = 64;
-bool recurrence_chunks_supported(const Recurrence& r);
+bool recurrence_chunks_supported(int kind, int dim, int vdim);
 cudaError_t launch_recurrence_chunks(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RowTiles& portions);

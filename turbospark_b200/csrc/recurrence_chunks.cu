@@ -495,12 +495,14 @@ cudaError_t launch_chunks(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, co
 template <int KIND>
 cudaError_t launch_chunks_dim(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RowTiles& portions) {
     if (r.dim <= 64) return launch_chunks<KIND, 64, 32>(ctx, st, r, portions);
+    if constexpr (KIND != REC_FORGET)
+        if (r.dim > 128) return launch_chunks<KIND, 256, 32>(ctx, st, r, portions);
     return launch_chunks<KIND, 128, 32>(ctx, st, r, portions);
 }
 
 }  // namespace
 
-bool recurrence_chunks_supported(const Recurrence& r) { return r.dim <= 128 && r.dim % 8 == 0 && r.vdim % 8 == 0; }
+bool recurrence_chunks_supported(int kind, int dim, int vdim) { return dim <= (kind == REC_FORGET ? 128 : 256) && dim % 8 == 0 && vdim % 8 == 0; }
 
 cudaError_t launch_recurrence_chunks(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RowTiles& portions) {
     if (portions.n == 0) return cudaSuccess;
