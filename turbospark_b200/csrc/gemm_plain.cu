@@ -603,7 +603,7 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
         // ---- MMA issue: the warp walks the items together, lane 0 issues.  f32 accumulate, bfloat16 operands, both
         // K-major and 128-byte swizzled (eight-row groups 1024 bytes apart; a K = 16 step moves the start by 32 bytes)
         const uint32_t leader = lane == 0 ? 1u : 0u;
-        const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(nt >> 3) << 17) | ((uint32_t)(TCG_M >> 4) << 24);
+        auto idesc_of = [](int n) { return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(TCG_M >> 4) << 24); };
         constexpr uint64_t DESC = ((uint64_t)1u << 16) | ((uint64_t)(1024u >> 4) << 32) | (1ull << 46) | (2ull << 61);
         bool ok = true;
         uint32_t it = 0, tile = 0;
@@ -614,6 +614,8 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
             if (!ok) break;
             tc_fence_after();
             const uint32_t d = tmem + buf * (uint32_t)nt;
+            // an expert's last tile multiplies only the tokens it has
+            const uint32_t idesc = EXPERTS ? idesc_of((w.n_tok + 15) & ~15) : idesc_of(nt);
             for (int u = 0; u < w.n; u++, it++) {
                 const int s = it % stages;
                 ok = __all_sync(0xffffffffu, mbar_wait(&bars->full[s], (it / stages) & 1, err));

@@ -53,8 +53,10 @@ struct Smem {
     static constexpr int V = 4 * KEY;                 // two stages
     static constexpr int W = V + 2 * VAL;             // weighted values, high and low (not FORGET)
     static constexpr int S = W + (FORGET ? 0 : 2 * VAL);  // two states, high and low each
-    static constexpr int F = S + 4 * STATE;           // f32 vectors
-    static constexpr int N_F = FORGET ? DK + 8 * DK : 4 * C + 8 + 2 * DK;
+    static constexpr int Z = S + 4 * STATE;           // FORGET: pre-activations (f32) and queries as they come
+    static constexpr int RAW_Q = Z + C * DK * 4;
+    static constexpr int F = FORGET ? RAW_Q + KEY : Z;  // f32 vectors
+    static constexpr int N_F = FORGET ? 2 * DK + THREADS : 5 * C + 8 + 2 * DK;
     static constexpr int BYTES = F + N_F * 4;
 };
 
@@ -64,14 +66,14 @@ __global__ void __launch_bounds__(THREADS, 1)
     using M = Smem<KIND, DK, VB>;
     constexpr bool FORGET = KIND == REC_FORGET, MLSTM = KIND == REC_MLSTM, SSD = KIND == REC_SSD;
     constexpr int KS = DK / 16, NV = VB / 8, MS = DK / 64, KB = DK * 2, BV = VB * 2;
-    constexpr int RS = FORGET ? THREADS / DK : 1, TR = C / RS;  // FORGET: a thread owns one channel of TR rows
+    constexpr int RS = FORGET ? THREADS / DK : 1, TR = C / RS;  // FORGET: a thread makes queries and keys of one channel and TR rows
     extern __shared__ __align__(128) uint8_t smem[];
     const uint32_t base = smem_u32(smem);
     float* fv = reinterpret_cast<float*>(smem + M::F);
     // decay per head: row factor and exponents per row, scalars of the chunk
-    float *ea = fv, *eb = fv + C, *gain = fv + 2 * C, *floor_ = fv + 3 * C, *scal = fv + 4 * C, *norm = scal + 8;
-    // decay per channel: E at the end of the cut, products of the row splits
-    float *e_end = fv, *totals = fv + DK;
+    float *ea = fv, *eb = fv + C, *gain = fv + 2 * C, *floor_ = fv + 3 * C, *wv = fv + 4 * C, *scal = fv + 5 * C, *norm = scal + 8;
+    // decay per channel: E at the end of the cut, lower bounds, products of the row splits
+    float *e_end = fv, *lower = fv + DK, *totals = fv + 2 * DK;
     __shared__ int cut_end;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
     const int head = blockIdx.y, col0 = blockIdx.x * VB, vp = recurrence_v_pitch(a.vdim);
@@ -108,20 +110,21 @@ __global__ void __launch_bounds__(THREADS, 1)
         }
         cp_async_commit();
     };
-    // FORGET: the thread's channel and rows; pre-activations and queries of the next chunk wait in registers
-    const int ch = threadIdx.x % DK, split_i = threadIdx.x / DK;
-    float zr[FORGET ? TR : 1], qr[FORGET ? TR : 1];
-    const float low = FORGET && ch < a.dim ? a.lower[(int64_t)head * a.dim + ch] : 0.f;
-    auto fetch = [&](int chunk) {
+    const int ch = threadIdx.x % DK, split_i = threadIdx.x / DK;  // FORGET: the thread's channel and rows
+    auto z_at = [&](int r) -> float& { return reinterpret_cast<float*>(smem + M::Z)[r * DK + ch]; };
+    auto raw = [&](int chunk) {  // FORGET: pre-activations and queries of a chunk
         if (!FORGET || chunk >= n_chunks) return;
-        const int n = min(C, p.n_rows - chunk * C);
-#pragma unroll
-        for (int i = 0; i < (FORGET ? TR : 0); i++) {
-            const int r = split_i * TR + i;
-            const bool ok = r < n && ch < a.dim;
-            const int64_t row = p.row_first + chunk * C + r;
-            zr[i] = ok ? a.gate[row * a.gate_stride + (int64_t)head * a.dim + ch] : 0.f;
-            qr[i] = ok ? __bfloat162float(gq[row * a.q_stride + ch]) : 0.f;
+        const int row0 = p.row_first + chunk * C, n = min(C, p.n_rows - chunk * C);
+        const float* gz = a.gate + (int64_t)head * a.dim;
+        for (int i = threadIdx.x; i < C * (DK / 4); i += THREADS) {
+            const int r = i / (DK / 4), c = i % (DK / 4);
+            const bool ok = r < n && c * 4 < a.dim;
+            cp16(base + M::Z + (r * DK + c * 4) * 4, gz + (ok ? row0 + r : row0) * a.gate_stride + (ok ? c * 4 : 0), ok);
+        }
+        for (int i = threadIdx.x; i < C * (DK / 8); i += THREADS) {
+            const int r = i / (DK / 8), c = i % (DK / 8);
+            const bool ok = r < n && c * 8 < a.dim;
+            cp16(base + M::RAW_Q + (r * DK + c * 8) * 2, gq + (int64_t)(ok ? row0 + r : row0) * a.q_stride + (ok ? c * 8 : 0), ok);
         }
     };
     // decay per head: lane l of warp 0 has the gates of rows 2 l and 2 l + 1 of the next chunk
@@ -174,27 +177,19 @@ __global__ void __launch_bounds__(THREADS, 1)
     }
     if (MLSTM && pos0 > 0) top = a.state.top[slot0];
     const float skip = SSD ? a.skip[head] : 0.f;
+    if (FORGET)
+        for (int i = threadIdx.x; i < DK; i += THREADS) lower[i] = i < a.dim ? a.lower[(int64_t)head * a.dim + i] : 1.f;
     pdl_wait();
+    raw(0);
     issue(0);
-    fetch(0);
     fetch_gates(0);
 
     int state_buf = 0;
     for (int chunk = 0; chunk < n_chunks; chunk++) {
         const int n = min(C, p.n_rows - chunk * C), row0 = p.row_first + chunk * C;
-        issue(chunk + 1);
-        cp_async_wait<1>();
-        float f[FORGET ? TR : 1], k[FORGET ? TR : 1], q[FORGET ? TR : 1];
-        if (FORGET) {
-#pragma unroll
-            for (int i = 0; i < (FORGET ? TR : 0); i++) {
-                const bool ok = split_i * TR + i < n && ch < a.dim;
-                // sigmoid(-z) = e / (1 + e) with e = exp(-z): 1 - f without a difference
-                const float e = expf(-fabsf(zr[i])), d = 1.f / (1.f + e), neg = zr[i] >= 0.f ? e * d : d;
-                k[i] = ok ? (1.f - low) * neg : 0.f, f[i] = 1.f - k[i], q[i] = ok ? rec_silu(qr[i]) : 0.f;
-            }
-            fetch(chunk + 1);
-        } else if (warp == 0) {
+        if (!FORGET) issue(chunk + 1), cp_async_wait<1>();
+        else cp_async_wait<0>();
+        if (!FORGET && warp == 0) {
             const float d0 = gate2[0].y, d1 = gate2[1].y;
             float sum = d0 + d1;
 #pragma unroll
@@ -233,35 +228,48 @@ __global__ void __launch_bounds__(THREADS, 1)
         for (int cut = 0; cut < n;) {  // FORGET: usually once
             int end = n;
             if (FORGET) {
-                // E from row `cut` on: products within the thread's rows, then over the row splits
+                // E from row `cut` on: products within the thread's rows, then over the row splits.  The first time round the pre-activations
+                // become 1 - f = (1 - l) sigmoid(-z).
+                const float low = lower[ch];
                 float mine = 1.f;
-#pragma unroll
-                for (int i = 0; i < (FORGET ? TR : 0); i++)
-                    if (split_i * TR + i >= cut) mine *= f[i];
-                totals[split_i * DK + ch] = mine;
+#pragma unroll 4
+                for (int i = 0; i < TR; i++) {
+                    const int r = split_i * TR + i;
+                    float& x = z_at(r);
+                    if (cut == 0) {
+                        const float e = __expf(-fabsf(x)), d = __fdividef(1.f, 1.f + e);
+                        x = r < n ? (1.f - low) * (x >= 0.f ? e * d : d) : 0.f;
+                    }
+                    if (r >= cut) mine *= 1.f - x;
+                }
+                totals[threadIdx.x] = mine;
                 if (threadIdx.x == 0) cut_end = n;
                 __syncthreads();
                 float e0 = 1.f;
                 for (int i = 0; i < split_i; i++) e0 *= totals[i * DK + ch];
-                float e = e0;
-                int first_low = n;
-#pragma unroll
-                for (int i = 0; i < (FORGET ? TR : 0); i++) {
-                    const int r = split_i * TR + i;
-                    if (r < cut) continue;
-                    e *= f[i];
-                    if (e < E_MIN && r > cut && first_low > r) first_low = r;
+                // E only falls: the chunk is cut if it ends too low
+                if (__syncthreads_or(e0 * mine < E_MIN)) {
+                    float e = e0;
+                    for (int i = 0; i < TR; i++) {
+                        const int r = split_i * TR + i;
+                        if (r < cut || r >= n) continue;
+                        e *= 1.f - z_at(r);
+                        if (e < E_MIN && r > cut) {
+                            atomicMin(&cut_end, r);
+                            break;
+                        }
+                    }
+                    __syncthreads();
+                    end = cut_end;
                 }
-                if (first_low < n) atomicMin(&cut_end, first_low);
-                __syncthreads();
-                end = cut_end;
-                e = e0;
-#pragma unroll
-                for (int i = 0; i < (FORGET ? TR : 0); i++) {
+                float e = e0;
+#pragma unroll 4
+                for (int i = 0; i < TR; i++) {
                     const int r = split_i * TR + i;
                     const bool in = r >= cut && r < end;
-                    if (in) e = fmaxf(e * f[i], E_MIN);  // the first row of a cut may fall further: nothing of the rows before is left then
-                    const float qe = in ? q[i] * e : 0.f, ke = in ? k[i] / e : 0.f;
+                    const float k = z_at(r), x = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(smem + M::RAW_Q)[r * DK + ch]);
+                    if (in) e = fmaxf(e * (1.f - k), E_MIN);  // the first row of a cut may fall further: nothing of the rows before is left then
+                    const float qe = in ? __fdividef(x, 1.f + __expf(-x)) * e : 0.f, ke = in ? k * (1.f / e) : 0.f;
                     const __nv_bfloat16 qh = __float2bfloat16_rn(qe), kh = __float2bfloat16_rn(ke);
                     const uint32_t off = at<KB>(r, ch >> 3) + (ch & 7) * 2;
                     *reinterpret_cast<__nv_bfloat16*>(smem + M::Q + off) = qh;
@@ -277,6 +285,7 @@ __global__ void __launch_bounds__(THREADS, 1)
                     const uint32_t off = at<BV>(r, c >> 2) + (c & 3) * 4;
                     const uint32_t v = *reinterpret_cast<const uint32_t*>(smem + M::V + (chunk & 1) * M::VAL + off);
                     const float w = ex2(scal[0] + eb[r]) * gain[r];
+                    if (MLSTM && c == 0) wv[r] = w;
                     uint32_t hi, lo;
                     split(__uint_as_float(v << 16) * w, __uint_as_float(v & 0xFFFF0000u) * w, hi, lo);
                     *reinterpret_cast<uint32_t*>(smem + M::W + off) = hi;
@@ -284,6 +293,7 @@ __global__ void __launch_bounds__(THREADS, 1)
                 }
             }
             __syncthreads();
+            if (FORGET && end == n) raw(chunk + 1), issue(chunk + 1);  // what they overwrite has been used
             const uint32_t qt = base + (FORGET ? 0 : (chunk & 1) * M::KEY_STAGE) + M::Q, kt = base + (FORGET ? 0 : (chunk & 1) * M::KEY_STAGE) + M::K;
             const uint32_t sh = base + M::S + 2 * state_buf * M::STATE, sl = sh + M::STATE;
             if (warp < 4) {
@@ -451,8 +461,9 @@ __global__ void __launch_bounds__(THREADS, 1)
                 if (MLSTM) {
                     for (int c = threadIdx.x - 128; c < DK; c += 128) {
                         float x = norm[state_buf * DK + c] * scal[1];
-                        for (int r = 0; r < n; r++)
-                            x = fmaf(ex2(scal[0] + eb[r]), __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(
+#pragma unroll 8
+                        for (int r = 0; r < C; r++)
+                            x = fmaf(wv[r], __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(
                                                                smem + (chunk & 1) * M::KEY_STAGE + M::K + at<KB>(r, c >> 3) + (c & 7) * 2)), x);
                         norm[(state_buf ^ 1) * DK + c] = x;
                     }

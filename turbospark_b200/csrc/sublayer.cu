@@ -45,6 +45,11 @@ __device__ __forceinline__ float warp_sum(float v) {
     return v;
 }
 __device__ __forceinline__ float sigmoid(float z) { return 1.f / (1.f + expf(-z)); }
+// bfloat16 results take the fast exponential and division (relative error a few 2^-22)
+template <typename T>
+__device__ __forceinline__ float silu(float z) {
+    return sizeof(T) == 4 ? z * sigmoid(z) : __fdividef(z, 1.f + __expf(-z));
+}
 
 // 1 / rms of the group that column c belongs to, from the columns' squares.  A thread holds columns (k * THREADS + thread) * W + i, k < V.
 // FAST: groups are multiples of 32 W columns, so a warp's columns of one k share a group and the whole reduction takes one barrier.
@@ -146,7 +151,33 @@ __global__ void __launch_bounds__(THREADS) sublayer_end_kernel(const __grid_cons
             hist[j][k] = in && c < d ? load(p + c, Vec<W>()) : zeros<W>();
         }
     }
-    for (int r = first, parity = 0; r < tile.row_first + tile.n_rows; r++, parity ^= 1) {
+    // the sublayer's output and the stream of a row; those of the next row are under way while a row is normed
+    Vec<W> y_next[V], x_next[V];
+    auto fetch = [&](int r) {
+#pragma unroll
+        for (int k = 0; k < V; k++) {
+            const int c = (k * THREADS + threadIdx.x) * W;
+            x_next[k] = c < d ? load(s.x_in + (int64_t)r * d + c, Vec<W>()) : zeros<W>();
+            y_next[k] = s.y && c < d ? load(s.y + (int64_t)r * d + c, Vec<W>()) : zeros<W>();
+        }
+        if (s.y) return;
+        for (int e = 0; e < s.top; e++) {
+            const float f = s.weight[(int64_t)r * s.top + e];
+            const T* row = static_cast<const T*>(s.experts) + (int64_t)s.slot_of[(int64_t)r * s.top + e] * s.expert_stride;
+#pragma unroll
+            for (int k = 0; k < V; k++) {
+                const int c = (k * THREADS + threadIdx.x) * W;
+                if (c >= d) continue;
+                const Vec<W> v = load(row + c, Vec<W>());
+#pragma unroll
+                for (int i = 0; i < W; i++) y_next[k].v[i] = fmaf(f, v.v[i], y_next[k].v[i]);
+            }
+        }
+    };
+    const int last = tile.row_first + tile.n_rows - 1;
+    const bool any_kept = s.taps > 1 && ring_keeps(s.ring, s.rows, s.n_rows, last, rd.seq);
+    if (!s.table) fetch(first);
+    for (int r = first, parity = 0; r <= last; r++, parity ^= 1) {
         Vec<W> x[V];
         if (s.table) {
             const int tok = s.tokens[(int64_t)r * s.token_stride], pos = pos_first + (r - first);
@@ -164,33 +195,9 @@ __global__ void __launch_bounds__(THREADS) sublayer_end_kernel(const __grid_cons
             }
         } else {
             Vec<W> y[V];
-            if (s.y) {
 #pragma unroll
-                for (int k = 0; k < V; k++) {
-                    const int c = (k * THREADS + threadIdx.x) * W;
-                    y[k] = c < d ? load(s.y + (int64_t)r * d + c, Vec<W>()) : zeros<W>();
-                }
-            } else {
-#pragma unroll
-                for (int k = 0; k < V; k++) y[k] = zeros<W>();
-                for (int e = 0; e < s.top; e++) {
-                    const float f = s.weight[(int64_t)r * s.top + e];
-                    const T* row = static_cast<const T*>(s.experts) + (int64_t)s.slot_of[(int64_t)r * s.top + e] * s.expert_stride;
-#pragma unroll
-                    for (int k = 0; k < V; k++) {
-                        const int c = (k * THREADS + threadIdx.x) * W;
-                        if (c >= d) continue;
-                        const Vec<W> v = load(row + c, Vec<W>());
-#pragma unroll
-                        for (int i = 0; i < W; i++) y[k].v[i] = fmaf(f, v.v[i], y[k].v[i]);
-                    }
-                }
-            }
-#pragma unroll
-            for (int k = 0; k < V; k++) {
-                const int c = (k * THREADS + threadIdx.x) * W;
-                x[k] = c < d ? load(s.x_in + (int64_t)r * d + c, Vec<W>()) : zeros<W>();
-            }
+            for (int k = 0; k < V; k++) x[k] = x_next[k], y[k] = y_next[k];
+            if (r < last) fetch(r + 1);
             float inv[V];
             norm.rms(y, parity, inv);
 #pragma unroll
@@ -200,7 +207,7 @@ __global__ void __launch_bounds__(THREADS) sublayer_end_kernel(const __grid_cons
         }
         if (r >= tile.row_first) {
             float* keep = nullptr;
-            if (s.taps > 1 && ring_keeps(s.ring, s.rows, s.n_rows, r, rd.seq)) keep = ring_row(s.ring, rd.seq, pos_first + (r - first));
+            if (any_kept && ring_keeps(s.ring, s.rows, s.n_rows, r, rd.seq)) keep = ring_row(s.ring, rd.seq, pos_first + (r - first));
 #pragma unroll
             for (int k = 0; k < V; k++) {
                 const int c = (k * THREADS + threadIdx.x) * W;
@@ -286,8 +293,19 @@ __global__ void __launch_bounds__(THREADS) projection_norms_kernel(const __grid_
     const float *src = p.raw + (int64_t)r * p.raw_stride + (query ? 0 : (int64_t)p.n_q * p.width), *w = query ? p.q_weight : p.k_weight;
     pdl_wait();
     pdl_launch_dependents();
+    constexpr int HELD = 4;  // vectors that stay in registers
+    Vec<W> held[HELD];
     float ss = 0.f;
-    for (int i = threadIdx.x * W; i < n; i += THREADS * W) {
+#pragma unroll
+    for (int k = 0; k < HELD; k++) {
+        const int i = (k * THREADS + threadIdx.x) * W;
+        held[k] = i < n ? load(src + i, Vec<W>()) : zeros<W>();
+    }
+#pragma unroll
+    for (int k = 0; k < HELD; k++)
+#pragma unroll
+        for (int j = 0; j < W; j++) ss = fmaf(held[k].v[j], held[k].v[j], ss);
+    for (int i = (HELD * THREADS + threadIdx.x) * W; i < n; i += THREADS * W) {
         const Vec<W> v = load(src + i, Vec<W>());
 #pragma unroll
         for (int j = 0; j < W; j++) ss = fmaf(v.v[j], v.v[j], ss);
@@ -311,13 +329,16 @@ __global__ void __launch_bounds__(THREADS) projection_norms_kernel(const __grid_
         }
         step = p.keys.head_step;
     }
-    for (int i = threadIdx.x * W; i < n; i += THREADS * W) {
-        Vec<W> v = load(src + i, Vec<W>());
+    auto finish = [&](int i, Vec<W> v) {
         const Vec<W> g = load(w + i, Vec<W>());
 #pragma unroll
         for (int j = 0; j < W; j++) v.v[j] *= f * g.v[j];
         store(dst + (int64_t)(i / p.width) * step + i % p.width, v);
-    }
+    };
+#pragma unroll
+    for (int k = 0; k < HELD; k++)
+        if ((k * THREADS + (int)threadIdx.x) * W < n) finish((k * THREADS + threadIdx.x) * W, held[k]);
+    for (int i = (HELD * THREADS + threadIdx.x) * W; i < n; i += THREADS * W) finish(i, load(src + i, Vec<W>()));
     if (query && step > p.width) {
         const int tail = step - p.width;
         for (int i = threadIdx.x; i < heads * tail; i += THREADS) put(dst + (int64_t)(i / tail) * step + p.width + i % tail, 0.f);
@@ -349,22 +370,31 @@ __global__ void __launch_bounds__(THREADS) short_conv_kernel(const __grid_consta
         hist[j] = back <= rd.slot ? load(in + (int64_t)(tile.row_first - back) * s.in_stride, Vec<W>())
                                   : load(ring_row_before(s.ring, rd.seq, rd.base, pos, s.use_before) + c, Vec<W>());
     }
-    for (int i = 0; i < tile.n_rows; i++) {
-        const int r = tile.row_first + i;
-        const Vec<W> x = load(in + (int64_t)r * s.in_stride, Vec<W>());
-        if (s.taps > 1 && ring_keeps(s.ring, s.rows, s.n_rows, r, rd.seq)) store(ring_row(s.ring, rd.seq, rd.base + rd.slot + i) + c, x);
-        Vec<W> o = bias;
+    const bool any_kept = s.taps > 1 && ring_keeps(s.ring, s.rows, s.n_rows, tile.row_first + tile.n_rows - 1, rd.seq);
+    constexpr int AHEAD = W == 4 ? 4 : 8;  // rows in flight
+    for (int i0 = 0; i0 < tile.n_rows; i0 += AHEAD) {
+        Vec<W> x[AHEAD];
 #pragma unroll
-        for (int k = 0; k < W; k++) {
+        for (int i = 0; i < AHEAD; i++)
+            if (i0 + i < tile.n_rows) x[i] = load(in + (int64_t)(tile.row_first + i0 + i) * s.in_stride, Vec<W>());
 #pragma unroll
-            for (int j = TM - 2; j >= 0; j--) o.v[k] = fmaf(w[j + 1].v[k], hist[j].v[k], o.v[k]);
-            o.v[k] = fmaf(w[0].v[k], x.v[k], o.v[k]);
-            o.v[k] *= sigmoid(o.v[k]);
+        for (int i = 0; i < AHEAD; i++) {
+            if (i0 + i >= tile.n_rows) break;
+            const int r = tile.row_first + i0 + i;
+            if (any_kept && ring_keeps(s.ring, s.rows, s.n_rows, r, rd.seq)) store(ring_row(s.ring, rd.seq, rd.base + rd.slot + i0 + i) + c, x[i]);
+            Vec<W> o = bias;
+#pragma unroll
+            for (int k = 0; k < W; k++) {
+#pragma unroll
+                for (int j = TM - 2; j >= 0; j--) o.v[k] = fmaf(w[j + 1].v[k], hist[j].v[k], o.v[k]);
+                o.v[k] = fmaf(w[0].v[k], x[i].v[k], o.v[k]);
+                o.v[k] = silu<T>(o.v[k]);
+            }
+            store(static_cast<T*>(s.out) + (int64_t)r * s.out_stride + c, o);
+#pragma unroll
+            for (int j = TM - 2; j > 0; j--) hist[j] = hist[j - 1];
+            hist[0] = x[i];
         }
-        store(static_cast<T*>(s.out) + (int64_t)r * s.out_stride + c, o);
-#pragma unroll
-        for (int j = TM - 2; j > 0; j--) hist[j] = hist[j - 1];
-        hist[0] = x;
     }
 }
 
@@ -381,7 +411,7 @@ __global__ void __launch_bounds__(THREADS) gated_norm_kernel(const __grid_consta
         if (g.pre_gate) {
             const Vec<W> z = load(static_cast<const T*>(g.pre_gate) + (int64_t)r * g.gate_stride + c, Vec<W>());
 #pragma unroll
-            for (int i = 0; i < W; i++) x.v[i] *= z.v[i] * sigmoid(z.v[i]);
+            for (int i = 0; i < W; i++) x.v[i] *= silu<T>(z.v[i]);
         }
         float s = 0.f;
 #pragma unroll
