@@ -593,13 +593,15 @@ typedef struct tsb_recurrence {
     float* out;                      /* [rows, out_stride] f32, head h at h * vdim */
     int64_t out_stride;
     float* state;                    /* [n_streams][ring][heads][dim][vdim rounded up to 4]: position p in slot p & (ring - 1) */
-    float* norm;                     /* MLSTM: [n_streams][ring][heads][dim] */
-    double* top;                     /* MLSTM: [n_streams][ring][heads] */
+    float* norm;                     /* MLSTM: [n_streams][ring][heads][copies][dim], a copy for every 32 columns of vdim */
+    double* top;                     /* MLSTM: [n_streams][ring][heads][copies] */
     int32_t ring, n_streams;
+    void* scratch;                   /* chunked: tsb_recurrence_scratch_bytes */
 } tsb_recurrence;
 /* chunked = 0: row by row, the states after a portion's last `ring` rows are kept; 1 (TSB_BF16): 64 rows at a time, the last one is. */
 TSB_API int32_t tsb_recurrence_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, const tsb_recurrence* r, const tsb_row_desc* rows_dev, int32_t rows,
                                     int32_t rows_per_seq, int32_t chunked);
+TSB_API size_t tsb_recurrence_scratch_bytes(int32_t kind, int32_t heads, int32_t dim, int32_t vdim, int32_t rows, int32_t rows_per_seq);
 /* From a recurrence's output to the output projection: o, times silu(pre_gate) when given, normed in `groups` equal parts, times weight (repeated
  * every weight_n columns), times sigmoid(post_gate) when given, times scale. */
 TSB_API int32_t tsb_gated_norm_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, const float* o, int64_t o_stride, int32_t width, int32_t groups, const float* weight,

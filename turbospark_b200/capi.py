@@ -79,7 +79,7 @@ def lib():
         L.tsb_uniform_u64.restype = C.c_uint64
         L.tsb_uniform_u64.argtypes = [C.c_int32, C.c_uint64, C.c_uint64]
         for name in ("tsb_attn_scratch_bytes", "tsb_accept_scratch_bytes", "tsb_accept_history_scratch_bytes", "tsb_gemm_workspace_bytes", "tsb_plain_gemm_workspace_bytes",
-                     "tsb_window_attention_scratch_bytes"):
+                     "tsb_window_attention_scratch_bytes", "tsb_recurrence_scratch_bytes"):
             if hasattr(L, name):
                 getattr(L, name).restype = C.c_size_t
         if hasattr(L, "tsb_kv_cursor"):
@@ -364,6 +364,10 @@ class Ctx:
                                              _vp(bias), _vp(state), _vp(before), C.c_int32(n_streams), C.c_int32(ring), _vp(rows_dev), C.c_int32(rows),
                                              C.c_int32(rows_per_seq), _vp(out), C.c_int64(out_stride)))
 
+    def recurrence_scratch(self, kind, heads, dim, vdim, rows, rows_per_seq):
+        return self.zeroed(int(lib().tsb_recurrence_scratch_bytes(C.c_int32(kind), C.c_int32(heads), C.c_int32(dim), C.c_int32(vdim), C.c_int32(rows),
+                                                                  C.c_int32(rows_per_seq))))
+
     def recurrence_rows(self, type_, rec, rows_dev, rows, rows_per_seq, chunked=False, stream=None):
         self.check(lib().tsb_recurrence_rows(self.h, stream, C.c_int32(type_), C.byref(rec), _vp(rows_dev), C.c_int32(rows), C.c_int32(rows_per_seq),
                                              C.c_int32(int(chunked))))
@@ -454,7 +458,7 @@ class Recurrence(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("kind", "heads", "dim", "vdim", "heads_per_key")] + [("cap", C.c_float), ("q_scale", C.c_float)] + \
                [(n, C.c_void_p) for n in ("q", "k", "v")] + [(n, C.c_int64) for n in ("q_stride", "k_stride", "v_stride")] + \
                [("gate", C.c_void_p), ("gate_stride", C.c_int64)] + [(n, C.c_void_p) for n in ("lower", "a_log", "skip", "out")] + \
-               [("out_stride", C.c_int64)] + [(n, C.c_void_p) for n in ("state", "norm", "top")] + [("ring", C.c_int32), ("n_streams", C.c_int32)]
+               [("out_stride", C.c_int64)] + [(n, C.c_void_p) for n in ("state", "norm", "top")] + [("ring", C.c_int32), ("n_streams", C.c_int32), ("scratch", C.c_void_p)]
 
 
 class _ExpertLists(C.Structure):

@@ -202,6 +202,7 @@ void plain_runtime_free(ModelRt& rt) {
     rt.plain = nullptr;
 }
 
+constexpr int CHUNK_MIN_ROWS = 32;  // rows of a portion from which on its recurrences go chunk by chunk
 // Rings of the convolutions and states of the recurrences.  A cursor may go back by max_rows rows after a pass of as many, so the states of
 // max_rows + 1 positions are kept, and the convolutions' inputs as far back as the oldest of them looks.
 int32_t states_init(tsb_session* s, const PlainModel* m, const SessionShape& shape, StreamStates& st) {
@@ -220,6 +221,7 @@ int32_t states_init(tsb_session* s, const PlainModel* m, const SessionShape& sha
     for (st.ring = 2; st.ring < shape.max_rows + 1;) st.ring *= 2;
     for (st.row_ring = 2; st.row_ring < st.ring + st.keep;) st.row_ring *= 2;
     std::vector<RowRing> rings;
+    size_t scratch = 0;
     int32_t rc = TSB_OK;
     auto ring = [&](std::vector<RowRing>& list, int64_t width, int taps) {
         RowRing r;
@@ -241,10 +243,14 @@ int32_t states_init(tsb_session* s, const PlainModel* m, const SessionShape& sha
         r.ring = st.ring, r.n_streams = shape.n_streams;
         const size_t heads = (size_t)shape.n_streams * st.ring * c.rec_heads;
         if (c.recurrence && rc == TSB_OK) rc = zero(heads * c.rec_dim * recurrence_v_pitch(c.rec_vdim) * 4, (void**)&r.s);
-        if (c.recurrence == TSB_REC_MLSTM && rc == TSB_OK) rc = zero(heads * c.rec_dim * 4, (void**)&r.norm);
-        if (c.recurrence == TSB_REC_MLSTM && rc == TSB_OK) rc = zero(heads * 8, (void**)&r.top);
+        const size_t copies = heads * recurrence_copies(c.rec_vdim);
+        if (c.recurrence == TSB_REC_MLSTM && rc == TSB_OK) rc = zero(copies * c.rec_dim * 4, (void**)&r.norm);
+        if (c.recurrence == TSB_REC_MLSTM && rc == TSB_OK) rc = zero(copies * 8, (void**)&r.top);
+        if (c.recurrence && !m->f32)
+            scratch = std::max(scratch, recurrence_scratch_bytes(c.recurrence, c.rec_heads, c.rec_dim, c.rec_vdim, shape.pass_rows / REC_CHUNK + shape.n_streams));
         st.states.push_back(r);
     }
+    if (rc == TSB_OK && shape.pass_rows >= CHUNK_MIN_ROWS) rc = zero(scratch, &st.chunk_scratch);
     if (rc) return rc;
     st.n_rings = (int)rings.size();
     if (st.n_rings == 0) return TSB_OK;
@@ -416,7 +422,8 @@ struct PassPlan {
     const ExpandStream* expanded_dev = nullptr;
     int expanded_pages = 0, expanded_len = 0, short_first = 0, short_rows = 0;
     // output-norm form: runs of rows for the row operators; portions whose recurrences go row by row, and chunk by chunk where there is a kernel
-    RowTiles runs, by_row, by_chunk, portions;  // portions: all of them
+    RowTiles runs, by_row, portions;  // portions: all of them
+    RecurrenceChunks by_chunk;
     bool use_before = false;
 
     const AttnBatch* find(int set, int group, int rows_per_tile) const {
@@ -431,8 +438,6 @@ LatentTiling latent_tiling(const tsb_ctx* ctx, const PassPlan& plan, const Pass&
     return latent_attn_tiling(ctx, l.cfg.n_q_heads, all ? plan.longest : plan.longest_short, all ? p.rows : plan.rows_short, plan.max_len);
 }
 
-constexpr int CHUNK_MIN_ROWS = 32;  // rows of a portion from which on its recurrences go chunk by chunk
-
 int32_t plan_states(tsb_session* s, const PlainModel* m, const ModelRt& rt, const Pass& p, PassPlan& plan) {
     const StreamStates& states = rt.plain->states;
     plan.use_before = states.n_rings > 0 && plan.longest + states.keep > states.row_ring;
@@ -442,14 +447,20 @@ int32_t plan_states(tsb_session* s, const PlainModel* m, const ModelRt& rt, cons
         plan.by_row = plan.portions = RowTiles::uniform(p.rows, p.rows_per_seq, p.rows_per_seq);
         return TSB_OK;
     }
-    std::vector<AttnTile> runs, by_row, by_chunk, portions;
+    std::vector<AttnTile> runs, by_row, portions, chunks;
+    std::vector<ChunkPortion> by_chunk;
     for (int i = 0; i < p.n_groups; i++) {
         const RowGroup& g = p.groups[i];
         for (int r = 0; r < g.n_rows; r += per) runs.push_back({g.first_row + r, std::min(per, g.n_rows - r)});
         const bool long_portion = !m->f32 && g.n_rows >= CHUNK_MIN_ROWS;
         portions.push_back({g.first_row, g.n_rows});
-        (long_portion ? by_chunk : by_row).push_back({g.first_row, g.n_rows});
-        if (long_portion) rt.kv->state_lo[g.seq] = g.base + g.n_rows - 1;  // the states in between are not kept
+        if (!long_portion) {
+            by_row.push_back({g.first_row, g.n_rows});
+            continue;
+        }
+        by_chunk.push_back({g.first_row, g.n_rows, (int)chunks.size()});
+        for (int r = 0; r < g.n_rows; r += REC_CHUNK) chunks.push_back({g.first_row + r, std::min(REC_CHUNK, g.n_rows - r)});
+        rt.kv->state_lo[g.seq] = g.base + g.n_rows - 1;  // the states in between are not kept
     }
     auto stage = [&](const std::vector<AttnTile>& list, RowTiles& out) -> int32_t {
         if (list.empty()) {
@@ -463,8 +474,14 @@ int32_t plan_states(tsb_session* s, const PlainModel* m, const ModelRt& rt, cons
     };
     int32_t rc = stage(runs, plan.runs);
     if (rc == TSB_OK) rc = stage(by_row, plan.by_row);
-    if (rc == TSB_OK) rc = stage(by_chunk, plan.by_chunk);
-    return rc == TSB_OK ? stage(portions, plan.portions) : rc;
+    if (rc == TSB_OK) rc = stage(portions, plan.portions);
+    if (rc == TSB_OK) rc = stage(chunks, plan.by_chunk.chunks);
+    if (rc || by_chunk.empty()) return rc;
+    const int32_t* dev = nullptr;
+    if ((rc = session_stage_ints(s, reinterpret_cast<const int32_t*>(by_chunk.data()), (int)by_chunk.size() * 3, &dev))) return rc;
+    plan.by_chunk.portions = reinterpret_cast<const ChunkPortion*>(dev), plan.by_chunk.n_portions = (int)by_chunk.size();
+    plan.by_chunk.scratch = states.chunk_scratch;
+    return TSB_OK;
 }
 
 int32_t plan_pass(tsb_session* s, const PlainModel* m, const ModelRt& rt, const Pass& p, PassPlan& plan) {
@@ -721,7 +738,7 @@ struct Forward {
         GatedNorm g;
         r.kind = c.recurrence, r.heads = h, r.dim = D, r.vdim = E, r.gate = b->raw + b->raw_rec, r.gate_stride = b->raw_stride;
         r.q = b->rec, r.q_stride = r.k_stride = r.v_stride = b->rec_stride, r.out = b->rec_out, r.out_stride = b->rec_out_stride;
-        r.state = b->states.states[L], r.rows = p.rows_dev;
+        r.state = b->states.states[L], r.rows = p.rows_dev, r.n_rows = p.rows;
         g.o = b->rec_out, g.o_stride = b->rec_out_stride, g.width = inner, g.groups = h, g.weight = l.rec_norm, g.weight_n = inner, g.eps = m->cfg.norm_eps;
         g.gate_stride = b->rec_stride, g.out = at(b->cat, l.o_cols), g.out_stride = l.out.cols;
         if (l.mixer != MIX_NONE) g.scale = c.rec_scale;
@@ -741,7 +758,7 @@ struct Forward {
             r.q_stride = r.k_stride = r.v_stride = b->rec_mixed_stride, r.heads_per_key = h / c.rec_groups, r.a_log = l.rec_a_log, r.skip = l.rec_skip;
             g.pre_gate = b->rec, g.groups = c.rec_norm_groups;
         }
-        const bool chunks = plan.by_chunk.n > 0 && recurrence_chunks_supported(c.recurrence, D, E);
+        const bool chunks = plan.by_chunk.n_portions > 0 && recurrence_chunks_supported(c.recurrence, D, E);
         if (chunks)
             if (cudaError_t e = launch_recurrence_chunks(ctx, st, r, plan.by_chunk); e != cudaSuccess) return e;
         if (cudaError_t e = launch_recurrence_rows(ctx, st, m->f32, r, chunks ? plan.by_row : plan.portions); e != cudaSuccess) return e;

@@ -78,6 +78,7 @@ struct StreamStates {
     int row_ring = 0, keep = 0;             // rows kept of a convolution's input; the most that any convolution looks back
     std::vector<RowRing> conv1, conv2, rec; // per layer: inputs of the two sublayers' convolutions and of the recurrence's
     std::vector<RecurrentState> states;     // per layer
+    void* chunk_scratch = nullptr;          // of the chunked recurrences
     RowRing* rings_dev = nullptr;           // all rings that look back
     int n_rings = 0;
 };

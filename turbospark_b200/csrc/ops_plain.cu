@@ -95,16 +95,24 @@ int32_t tsb_recurrence_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, const tsb_
     TSB_REQUIRE(ctx, power_of_two(r->ring) && r->ring > 1 && r->n_streams > 0 && (uintptr_t)r->state % 16 == 0, "ring is a power of two above one");
     TSB_REQUIRE(ctx, !chunked || (type == TSB_BF16 && recurrence_chunks_supported(r->kind, r->dim, r->vdim)), "no chunked kernel for this type and these sizes");
     TSB_REQUIRE(ctx, !chunked || ((uintptr_t)r->q % 16 == 0 && (uintptr_t)r->k % 16 == 0 && (uintptr_t)r->v % 16 == 0 && (uintptr_t)r->out % 8 == 0 && r->q_stride % 8 == 0 &&
-                                  r->k_stride % 8 == 0 && r->v_stride % 8 == 0 && r->out_stride % 2 == 0), "rows start on 16-byte boundaries");
+                                  r->k_stride % 8 == 0 && r->v_stride % 8 == 0 && r->out_stride % 2 == 0 && r->scratch && (uintptr_t)r->scratch % 16 == 0 &&
+                                  (!forget || ((uintptr_t)r->gate % 16 == 0 && r->gate_stride % 4 == 0))), "rows start on 16-byte boundaries, and there is scratch memory");
     DeviceGuard g(ctx);
     Recurrence x;
     x.kind = r->kind, x.heads = r->heads, x.dim = r->dim, x.vdim = r->vdim, x.heads_per_key = per_key, x.q = r->q, x.k = r->k, x.v = r->v;
     x.q_stride = r->q_stride, x.k_stride = r->k_stride, x.v_stride = r->v_stride, x.gate = r->gate, x.gate_stride = r->gate_stride, x.lower = r->lower;
     x.a_log = r->a_log, x.skip = r->skip, x.cap = r->cap, x.q_scale = r->q_scale == 0.f ? 1.f : r->q_scale, x.out = r->out, x.out_stride = r->out_stride;
-    x.state.s = r->state, x.state.norm = r->norm, x.state.top = r->top, x.state.ring = r->ring, x.state.n_streams = r->n_streams, x.rows = rows_dev;
+    x.state.s = r->state, x.state.norm = r->norm, x.state.top = r->top, x.state.ring = r->ring, x.state.n_streams = r->n_streams, x.rows = rows_dev, x.n_rows = rows;
     const RowTiles portions = RowTiles::uniform(rows, rows_per_seq, rows_per_seq);
-    TSB_CUDA(ctx, chunked ? launch_recurrence_chunks(ctx, (cudaStream_t)s, x, portions) : launch_recurrence_rows(ctx, (cudaStream_t)s, type == TSB_F32, x, portions));
+    RecurrenceChunks c;
+    c.chunks = RowTiles::uniform(rows, rows_per_seq, REC_CHUNK), c.n_portions = rows / rows_per_seq, c.rows_per_seq = rows_per_seq, c.scratch = r->scratch;
+    TSB_CUDA(ctx, chunked ? launch_recurrence_chunks(ctx, (cudaStream_t)s, x, c) : launch_recurrence_rows(ctx, (cudaStream_t)s, type == TSB_F32, x, portions));
     return TSB_OK;
+}
+
+size_t tsb_recurrence_scratch_bytes(int32_t kind, int32_t heads, int32_t dim, int32_t vdim, int32_t rows, int32_t rows_per_seq) {
+    if (heads <= 0 || dim <= 0 || vdim <= 0 || rows <= 0 || rows_per_seq <= 0) return 0;
+    return recurrence_scratch_bytes(kind, heads, dim, vdim, rows / rows_per_seq * ((rows_per_seq + REC_CHUNK - 1) / REC_CHUNK));
 }
 
 int32_t tsb_gated_norm_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, const float* o, int64_t o_stride, int32_t width, int32_t groups, const float* weight, int32_t weight_n,

@@ -11,7 +11,7 @@
 
 namespace {
 
-constexpr int THREADS = 256, COLS = 32, GROUPS = THREADS / 8, BATCH = 8;
+constexpr int THREADS = 256, COLS = REC_COLS, GROUPS = THREADS / 8, BATCH = 8;
 
 template <int KIND>
 size_t rows_smem(int dim_pad) {
@@ -52,9 +52,9 @@ __global__ void __launch_bounds__(THREADS) recurrence_rows_kernel(const __grid_c
         for (int r = 0; r < CR; r++) {
             const bool in = pos0 > 0 && c0 + r < a.dim && col < vp;
             s[r] = in ? *reinterpret_cast<const float4*>(p0 + (int64_t)(c0 + r) * vp + col) : make_float4(0.f, 0.f, 0.f, 0.f);
-            if (KIND == REC_MLSTM) n[r] = pos0 > 0 && c0 + r < a.dim ? a.state.norm[at * a.dim + c0 + r] : 0.f;
+            if (KIND == REC_MLSTM) n[r] = pos0 > 0 && c0 + r < a.dim ? a.state.norm[(at * gridDim.x + blockIdx.x) * a.dim + c0 + r] : 0.f;
         }
-        if (KIND == REC_MLSTM && pos0 > 0) top = a.state.top[at];
+        if (KIND == REC_MLSTM && pos0 > 0) top = a.state.top[at * gridDim.x + blockIdx.x];
     }
     const float rate = KIND == REC_SSD ? expf(a.a_log[head]) : 0.f, skip = KIND == REC_SSD ? a.skip[head] : 0.f;
     const int key_at = head / a.heads_per_key * a.dim;
@@ -78,7 +78,7 @@ __global__ void __launch_bounds__(THREADS) recurrence_rows_kernel(const __grid_c
                     const double keep = (double)decay[t] + m, m_new = fmax(keep, (double)write[t]);
                     if (t == (int)threadIdx.x) {
                         mine_d = expm1f((float)(keep - m_new)), mine_w = expf((float)((double)write[t] - m_new)), mine_m = expf(-(float)m_new);
-                        if (is_kept(a, p, b0 + t) && blockIdx.x == 0) a.state.top[rec_slot(a, rd.seq, pos0 + b0 + t) * a.heads + head] = m_new;
+                        if (is_kept(a, p, b0 + t)) a.state.top[(rec_slot(a, rd.seq, pos0 + b0 + t) * a.heads + head) * gridDim.x + blockIdx.x] = m_new;
                     }
                     m = m_new;
                 }
@@ -136,7 +136,7 @@ __global__ void __launch_bounds__(THREADS) recurrence_rows_kernel(const __grid_c
                 for (int r = 0; r < CR; r++) {
                     if (c0 + r >= a.dim) continue;
                     if (col < vp) *reinterpret_cast<float4*>(dst + (int64_t)(c0 + r) * vp + col) = s[r];
-                    if (KIND == REC_MLSTM && blockIdx.x == 0 && vl == 0) a.state.norm[at * a.dim + c0 + r] = n[r];
+                    if (KIND == REC_MLSTM && vl == 0) a.state.norm[(at * gridDim.x + blockIdx.x) * a.dim + c0 + r] = n[r];
                 }
             }
         }
@@ -165,7 +165,7 @@ cudaError_t launch_rows(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, cons
     static SmemOptIn configured;
     if (smem > 48 * 1024)
         if (cudaError_t e = tsb_opt_in_smem(ctx, recurrence_rows_kernel<T, KIND, CR>, smem, configured); e != cudaSuccess) return e;
-    return tsb_launch(ctx, recurrence_rows_kernel<T, KIND, CR>, dim3((unsigned)((r.vdim + COLS - 1) / COLS), (unsigned)r.heads, (unsigned)portions.n), dim3(THREADS),
+    return tsb_launch(ctx, recurrence_rows_kernel<T, KIND, CR>, dim3((unsigned)recurrence_copies(r.vdim), (unsigned)r.heads, (unsigned)portions.n), dim3(THREADS),
                       smem, st, true, r, portions, ctx->dev_error);
 }
 template <typename T, int KIND>

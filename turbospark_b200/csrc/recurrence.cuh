@@ -12,10 +12,14 @@ enum RecurrenceKind {
 // States of one layer for every stream and the last `ring` positions (a power of two): position p in slot p & (ring - 1).
 struct RecurrentState {
     float* s = nullptr;     // [stream][ring][heads][dim][v_pitch]
-    float* norm = nullptr;  // REC_MLSTM: [stream][ring][heads][dim]
-    double* top = nullptr;  // REC_MLSTM: [stream][ring][heads]; in double, since the decay is the exponential of small differences of it
+    // REC_MLSTM, a copy for every REC_COLS value columns (their owners read and write them at times of their own): [stream][ring][heads][copies][dim],
+    // [stream][ring][heads][copies]
+    float* norm = nullptr;
+    double* top = nullptr;  // in double, since the decay is the exponential of small differences of it
     int ring = 0, n_streams = 0;
 };
+constexpr int REC_COLS = 32;
+constexpr int recurrence_copies(int vdim) { return (vdim + REC_COLS - 1) / REC_COLS; }
 constexpr int recurrence_v_pitch(int vdim) { return (vdim + 3) / 4 * 4; }
 
 struct Recurrence {
@@ -35,12 +39,24 @@ struct Recurrence {
     int64_t out_stride = 0;
     RecurrentState state{};
     const tsb_row_desc* rows = nullptr;
+    int n_rows = 0;                                  // of the pass
 };
 constexpr int REC_MAX_DIM = 1024;
 
 // Portions (whole portions of streams) row by row; the state after each of a portion's last `ring` rows is kept.
 cudaError_t launch_recurrence_rows(tsb_ctx* ctx, cudaStream_t st, bool f32, const Recurrence& r, const RowTiles& portions);
-// Long portions in bfloat16, REC_CHUNK rows at a time on the tensor cores; the state after the last row is kept.
+// Long portions in bfloat16, REC_CHUNK rows at a time on the tensor cores; the state after a portion's last row is kept.  A portion's chunks
+// are consecutive, in the list and in the scratch memory.
 constexpr int REC_CHUNK = 64;
+struct ChunkPortion {
+    int32_t first_row, n_rows, first_chunk;
+};
+struct RecurrenceChunks {
+    RowTiles chunks{};                       // all chunks of all portions, REC_CHUNK rows each but a portion's last
+    const ChunkPortion* portions = nullptr;  // device; null: portions of rows_per_seq rows each
+    int n_portions = 0, rows_per_seq = 0;
+    void* scratch = nullptr;                 // recurrence_scratch_bytes for as many chunks
+};
 bool recurrence_chunks_supported(int kind, int dim, int vdim);
-cudaError_t launch_recurrence_chunks(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RowTiles& portions);
+size_t recurrence_scratch_bytes(int kind, int heads, int dim, int vdim, int chunks);
+cudaError_t launch_recurrence_chunks(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RecurrenceChunks& c);

@@ -2,17 +2,17 @@
 //
 // With E_t the product of a chunk's decays up to row t and S the state before the chunk,
 //   o_t = E_t q_t . S + sum_{s <= t} (E_t / E_s) (q_t . k_s) v_s,    S' = E_T S + sum_s (E_T / E_s) k_s v_s^T.
-// A CTA owns VB value columns of one head of one portion and walks its chunks.  Four warps make the outputs - sixteen rows each: queries
-// against the state, then against the chunk's keys, weights, values - while four others hold the state in their accumulators, bring it
-// to the end of the chunk and leave it in shared memory for the next one.
+// Three launches: what every chunk adds to the state (all chunks at once), the states before the chunks (a walk over the chunks, element by
+// element), the outputs (all chunks at once).  A CTA of the first and the last has one chunk, one head and 64 value columns.
 //
 // What is f32 stays f32-like: an operand that is not a projection (state, weighted products, decayed queries, keys or values) goes into a
 // product as the sum of two bfloat16 numbers, which keeps 16 bits of it.
 //
 // Decay per head (REC_MLSTM, REC_SSD): E is a number per row; the ratios are exponentials of differences of its logarithm, applied to the
-// products of plain queries and keys.
-// Decay per row of the state (REC_FORGET): E is a vector; queries times E_t and keys over E_s are made per chunk.  The keys grow as E falls,
-// so a chunk is cut where a component of E falls below 2^-80 and goes on from there (rows outside the cut are zero).
+// products of plain queries and keys, and to the values on their way into the state.
+// Decay per row of the state (REC_FORGET): E is a vector.  Into the state go keys times E_T / E_s, a product over the rows behind s; queries take
+// E_t, keys 1 / E_s.  1 / E grows, so where a component of E falls below 2^-80 the chunk is cut: rows behind a cut meet each other with E
+// counted from the cut, and the rows before it with keys brought to the cut.
 #include <algorithm>
 
 #include "mma_dev.cuh"
@@ -20,7 +20,7 @@
 
 namespace {
 
-constexpr int C = REC_CHUNK, THREADS = 256;
+constexpr int C = REC_CHUNK, THREADS = 256, VB = 64, BV = VB * 2;
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr float E_MIN = 8.2718061e-25f;  // 2^-80
 
@@ -38,174 +38,390 @@ __device__ __forceinline__ void split(float a, float b, uint32_t& hi, uint32_t& 
     hi = pack(a, b);
     lo = pack(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xFFFF0000u));
 }
-// byte offset of 16-byte piece p of row r; rows of BYTES, pieces permuted so that eight rows' worth of one piece spread over all banks
+// byte offset of 16-byte piece p of row r; rows of BYTES (a multiple of 128), pieces permuted so that eight rows' worth of one piece spread
+// over all banks
 template <int BYTES>
 __device__ __forceinline__ uint32_t at(int r, int p) {
-    return (uint32_t)(r * BYTES + ((BYTES == 64 ? (p ^ ((r >> 1) & 3)) : (p ^ (r & 7))) << 4));
+    return (uint32_t)(r * BYTES + ((p ^ (r & 7)) << 4));
 }
 
-template <int KIND, int DK, int VB>
-struct Smem {
-    static constexpr int KEY = C * DK * 2, VAL = C * VB * 2, STATE = DK * VB * 2;
+// ---- what the launches leave for each other, per (chunk, head)
+struct Scratch {
+    float* add;     // [dim][vdim]: what the chunk adds; after the walk the state before it, four numbers as four high and four low halves
+    float* norm;    // REC_MLSTM: the same for the normaliser, [dim]
+    float* decay;   // REC_FORGET: E_T [dim]; REC_SSD: E_T; REC_MLSTM: log E_T, and the maximum the chunk's part is relative to
+    double* top;    // REC_MLSTM: the running maximum before the chunk
+};
+__host__ __device__ inline int decay_width(int kind, int dim) { return kind == REC_FORGET ? dim : 2; }
+size_t align16(size_t n) { return (n + 15) / 16 * 16; }
+Scratch scratch_of(const Recurrence& r, void* p, int chunks) {
+    const size_t n = (size_t)chunks * r.heads;
+    Scratch s;
+    uint8_t* b = static_cast<uint8_t*>(p);
+    s.add = reinterpret_cast<float*>(b), b += align16(n * r.dim * r.vdim * 4);
+    s.norm = reinterpret_cast<float*>(b), b += align16(r.kind == REC_MLSTM ? n * r.dim * 4 : 0);
+    s.decay = reinterpret_cast<float*>(b), b += align16(n * decay_width(r.kind, r.dim) * 4);
+    s.top = reinterpret_cast<double*>(b);
+    return s;
+}
+
+// rows x columns of a projection into shared memory, zeros outside
+template <int ROW_BYTES>
+__device__ __forceinline__ void copy_tile(uint32_t dst, const __nv_bfloat16* src, int64_t stride, int n_rows, int n_cols) {
+    for (int i = threadIdx.x; i < C * (ROW_BYTES / 16); i += THREADS) {
+        const int r = i / (ROW_BYTES / 16), c = i % (ROW_BYTES / 16);
+        const bool ok = r < n_rows && c * 8 < n_cols;
+        cp16(dst + at<ROW_BYTES>(r, c), src + (ok ? r * stride + c * 8 : 0), ok);
+    }
+}
+
+// Gates of a chunk, by warp 0: lane l has rows 2 l and 2 l + 1.
+struct RowGates {
+    float in[2], log_e[2], end;  // SSD: step; MLSTM: log input gate.  log E up to the row, and at the chunk's end
+};
+template <int KIND>
+__device__ __forceinline__ RowGates row_gates(const Recurrence& a, int row0, int n, int head, int lane) {
+    RowGates g;
+    const float rate = KIND == REC_SSD ? expf(a.a_log[head]) : 0.f;
+    float d[2];
+#pragma unroll
+    for (int i = 0; i < 2; i++) {
+        const int r = 2 * lane + i;
+        float2 v = make_float2(KIND == REC_MLSTM ? -1e30f : 0.f, 0.f);
+        if (r < n) v = KIND == REC_MLSTM ? mlstm_gates(a, row0 + r, head) : ssd_gates(a, row0 + r, head, rate);
+        g.in[i] = v.x, d[i] = v.y;
+    }
+    float sum = d[0] + d[1];
+#pragma unroll
+    for (int o = 1; o < 32; o <<= 1) {
+        const float v = __shfl_up_sync(0xffffffffu, sum, o);
+        if (lane >= o) sum += v;
+    }
+    g.log_e[1] = sum, g.log_e[0] = sum - d[1], g.end = __shfl_sync(0xffffffffu, sum, 31);
+    return g;
+}
+
+// REC_FORGET: a thread has one channel of TR rows.  pre: pre-activations of the chunk in shared memory, which become 1 - f =
+// (1 - l) sigmoid(-z); returns the product of the thread's f.
+template <int DK>
+__device__ __forceinline__ float forget_gates(const Recurrence& a, float* pre, int head, int n) {
+    constexpr int RS = THREADS / DK, TR = C / RS;
+    const int ch = threadIdx.x % DK, first = threadIdx.x / DK * TR;
+    const float low = ch < a.dim ? a.lower[(int64_t)head * a.dim + ch] : 1.f;
+    float product = 1.f;
+#pragma unroll 4
+    for (int i = 0; i < TR; i++) {
+        float& x = pre[(first + i) * DK + ch];
+        const float e = __expf(-fabsf(x)), d = __fdividef(1.f, 1.f + e);
+        x = first + i < n ? (1.f - low) * (x >= 0.f ? e * d : d) : 0.f;
+        product *= 1.f - x;
+    }
+    return product;
+}
+template <int DK>
+__device__ __forceinline__ void copy_gates(const Recurrence& a, uint32_t dst, int row0, int n, int head) {
+    const float* gz = a.gate + (int64_t)row0 * a.gate_stride + (int64_t)head * a.dim;
+    for (int i = threadIdx.x; i < C * (DK / 4); i += THREADS) {
+        const int r = i / (DK / 4), c = i % (DK / 4);
+        const bool ok = r < n && c * 4 < a.dim;
+        cp16(dst + (r * DK + c * 4) * 4, gz + (ok ? r * a.gate_stride + c * 4 : 0), ok);
+    }
+}
+__device__ __forceinline__ void put_split(uint8_t* hi, uint8_t* lo, uint32_t off, float v) {
+    const __nv_bfloat16 h = __float2bfloat16_rn(v);
+    *reinterpret_cast<__nv_bfloat16*>(hi + off) = h;
+    *reinterpret_cast<__nv_bfloat16*>(lo + off) = __float2bfloat16_rn(v - __bfloat162float(h));
+}
+
+// ------------------------------------------------------------------ what a chunk adds to the state
+template <int KIND, int DK>
+struct AddSmem {
     static constexpr bool FORGET = KIND == REC_FORGET;
-    // FORGET: queries and keys, each high and low part, made per chunk; else two stages of queries and keys as they come
-    static constexpr int Q = 0, K = FORGET ? 2 * KEY : KEY, KEY_STAGE = 2 * KEY;
-    static constexpr int V = 4 * KEY;                 // two stages
-    static constexpr int W = V + 2 * VAL;             // weighted values, high and low (not FORGET)
-    static constexpr int S = W + (FORGET ? 0 : 2 * VAL);  // two states, high and low each
-    static constexpr int Z = S + 4 * STATE;           // FORGET: pre-activations (f32) and queries as they come
-    static constexpr int RAW_Q = Z + C * DK * 4;
-    static constexpr int F = FORGET ? RAW_Q + KEY : Z;  // f32 vectors
-    static constexpr int N_F = FORGET ? 2 * DK + THREADS : 5 * C + 8 + 2 * DK;
-    static constexpr int BYTES = F + N_F * 4;
+    static constexpr int KEY = C * DK * 2, VAL = C * VB * 2;
+    static constexpr int K = 0, V = FORGET ? 2 * KEY : KEY, W = V + VAL;  // FORGET: keys, values; else keys, values, weighted values (high, low)
+    static constexpr int Z = W, F = FORGET ? Z + C * DK * 4 : W + 2 * VAL;
+    static constexpr int BYTES = F + (FORGET ? THREADS : C + 4) * 4;
 };
 
-template <int KIND, int DK, int VB>
-__global__ void __launch_bounds__(THREADS, 1)
-    recurrence_chunks_kernel(const __grid_constant__ Recurrence a, const __grid_constant__ RowTiles portions, uint32_t* __restrict__ err) {
-    using M = Smem<KIND, DK, VB>;
-    constexpr bool FORGET = KIND == REC_FORGET, MLSTM = KIND == REC_MLSTM, SSD = KIND == REC_SSD;
-    constexpr int KS = DK / 16, NV = VB / 8, MS = DK / 64, KB = DK * 2, BV = VB * 2;
-    constexpr int RS = FORGET ? THREADS / DK : 1, TR = C / RS;  // FORGET: a thread makes queries and keys of one channel and TR rows
+template <int KIND, int DK>
+__global__ void __launch_bounds__(THREADS)
+    chunk_add_kernel(const __grid_constant__ Recurrence a, const __grid_constant__ RowTiles chunks, const __grid_constant__ Scratch out, uint32_t* __restrict__ err) {
+    using M = AddSmem<KIND, DK>;
+    constexpr bool FORGET = KIND == REC_FORGET, MLSTM = KIND == REC_MLSTM;
+    constexpr int KB = DK * 2, MT = DK / 16, SPLIT = MT < 8 ? 8 / MT : 1, MS = MT < 8 ? 1 : MT / 8, NV = VB / 8 / SPLIT;
     extern __shared__ __align__(128) uint8_t smem[];
     const uint32_t base = smem_u32(smem);
     float* fv = reinterpret_cast<float*>(smem + M::F);
-    // decay per head: row factor and exponents per row, scalars of the chunk
-    float *ea = fv, *eb = fv + C, *gain = fv + 2 * C, *floor_ = fv + 3 * C, *wv = fv + 4 * C, *scal = fv + 5 * C, *norm = scal + 8;
-    // decay per channel: E at the end of the cut, lower bounds, products of the row splits
-    float *e_end = fv, *lower = fv + DK, *totals = fv + 2 * DK;
-    __shared__ int cut_end;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
-    const int head = blockIdx.y, col0 = blockIdx.x * VB, vp = recurrence_v_pitch(a.vdim);
-    const AttnTile p = row_tile(portions, blockIdx.z);
-    const tsb_row_desc rd = a.rows[p.row_first];
-    const int pos0 = rd.base + rd.slot, key_at = head / a.heads_per_key * a.dim;
+    const int head = blockIdx.y, col0 = blockIdx.x * VB;
+    const AttnTile tile = row_tile(chunks, blockIdx.z);
+    const int row0 = tile.row_first, n = min(tile.n_rows, C);
+    const int64_t slot = (int64_t)blockIdx.z * a.heads + head;
+    const __nv_bfloat16* gv = static_cast<const __nv_bfloat16*>(a.v) + (int64_t)row0 * a.v_stride + (int64_t)head * a.vdim + col0;
+    pdl_wait();
+    pdl_launch_dependents();
+    copy_tile<BV>(base + M::V, gv, a.v_stride, n, a.vdim - col0);
+    if (FORGET) {
+        copy_gates<DK>(a, base + M::Z, row0, n, head);
+    } else {
+        copy_tile<KB>(base + M::K, static_cast<const __nv_bfloat16*>(a.k) + (int64_t)row0 * a.k_stride + head / a.heads_per_key * a.dim, a.k_stride, n, a.dim);
+    }
+    cp_async_commit();
+    if (!FORGET && warp == 0) {
+        // weights of the rows: E_T / E_s times the input scale (MLSTM: relative to the largest of them)
+        const RowGates g = row_gates<FORGET ? REC_SSD : KIND>(a, row0, n, head, lane);
+        float w[2], rel = 0.f;
+        if (MLSTM) {
+            w[0] = g.end - g.log_e[0] + g.in[0], w[1] = g.end - g.log_e[1] + g.in[1];
+            rel = fmaxf(w[0], w[1]);
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1) rel = fmaxf(rel, __shfl_xor_sync(0xffffffffu, rel, o));
+            w[0] = ex2((w[0] - rel) * LOG2E), w[1] = ex2((w[1] - rel) * LOG2E);
+        } else {
+            w[0] = ex2((g.end - g.log_e[0]) * LOG2E) * g.in[0], w[1] = ex2((g.end - g.log_e[1]) * LOG2E) * g.in[1];
+        }
+        fv[2 * lane] = w[0], fv[2 * lane + 1] = w[1];
+        if (blockIdx.x == 0 && lane == 0) {
+            out.decay[slot * 2] = MLSTM ? g.end : expf(g.end);
+            out.decay[slot * 2 + 1] = rel;
+        }
+    }
+    cp_async_wait<0>();
+    __syncthreads();
+    if (FORGET) {
+        float* pre = reinterpret_cast<float*>(smem + M::Z);
+        constexpr int RS = THREADS / DK, TR = C / RS;
+        const int ch = threadIdx.x % DK, part = threadIdx.x / DK;
+        fv[threadIdx.x] = forget_gates<DK>(a, pre, head, n);
+        __syncthreads();
+        float e = 1.f;  // product of the rows behind
+        for (int i = part + 1; i < RS; i++) e *= fv[i * DK + ch];
+#pragma unroll 4
+        for (int i = TR - 1; i >= 0; i--) {
+            const int r = part * TR + i;
+            const float k = pre[r * DK + ch];
+            put_split(smem + M::K, smem + M::K + M::KEY, at<KB>(r, ch >> 3) + (ch & 7) * 2, k * e);
+            e *= 1.f - k;
+        }
+        if (part == 0 && blockIdx.x == 0 && ch < a.dim) out.decay[slot * a.dim + ch] = e;
+    } else {
+        for (int i = threadIdx.x; i < C * (VB / 2); i += THREADS) {
+            const int r = i / (VB / 2), c = i % (VB / 2);
+            const uint32_t off = at<BV>(r, c >> 2) + (c & 3) * 4, v = *reinterpret_cast<const uint32_t*>(smem + M::V + off);
+            uint32_t hi, lo;
+            split(__uint_as_float(v << 16) * fv[r], __uint_as_float(v & 0xFFFF0000u) * fv[r], hi, lo);
+            *reinterpret_cast<uint32_t*>(smem + M::W + off) = hi;
+            *reinterpret_cast<uint32_t*>(smem + M::W + M::VAL + off) = lo;
+        }
+        if (MLSTM && blockIdx.x == 0)
+            for (int c = threadIdx.x; c < a.dim; c += THREADS) {
+                float x = 0.f;
+#pragma unroll 8
+                for (int r = 0; r < C; r++)
+                    x = fmaf(fv[r], __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(smem + M::K + at<KB>(r, c >> 3) + (c & 7) * 2)), x);
+                out.norm[slot * a.dim + c] = x;
+            }
+    }
+    __syncthreads();
+    // keys (transposed) times values: m-tile per warp, or half of the columns of one
+    const int m0 = MT < 8 ? warp % MT : warp, nv0 = MT < 8 ? warp / MT * NV : 0;
+    float s[MS][NV][4] = {};
+    const uint32_t vh = base + (FORGET ? M::V : M::W);
+#pragma unroll
+    for (int ks = 0; ks < C / 16; ks++) {
+        uint32_t bh[NV / 2][4], bl[NV / 2][4];
+#pragma unroll
+        for (int np = 0; np < NV / 2; np++) {
+            ldsm4_t(bh[np], vh + at<BV>(ks * 16 + (lane & 15), nv0 + np * 2 + (lane >> 4)));
+            if (!FORGET) ldsm4_t(bl[np], vh + M::VAL + at<BV>(ks * 16 + (lane & 15), nv0 + np * 2 + (lane >> 4)));
+        }
+#pragma unroll
+        for (int m = 0; m < MS; m++) {
+            const int c8 = (m0 + 8 * m) * 2 + ((lane >> 3) & 1), r = ks * 16 + (lane & 7) + ((lane >> 4) << 3);
+            uint32_t kh[4], kl[4];
+            ldsm4_t(kh, base + M::K + at<KB>(r, c8));
+            if (FORGET) ldsm4_t(kl, base + M::K + M::KEY + at<KB>(r, c8));
+#pragma unroll
+            for (int np = 0; np < NV / 2; np++) {
+                mma_bf16(s[m][2 * np], kh, bh[np][0], bh[np][1]), mma_bf16(s[m][2 * np + 1], kh, bh[np][2], bh[np][3]);
+                if (FORGET) mma_bf16(s[m][2 * np], kl, bh[np][0], bh[np][1]), mma_bf16(s[m][2 * np + 1], kl, bh[np][2], bh[np][3]);
+                else mma_bf16(s[m][2 * np], kh, bl[np][0], bl[np][1]), mma_bf16(s[m][2 * np + 1], kh, bl[np][2], bl[np][3]);
+            }
+        }
+    }
+    float* dst = out.add + slot * a.dim * a.vdim;
+#pragma unroll
+    for (int m = 0; m < MS; m++)
+#pragma unroll
+        for (int i = 0; i < NV; i++)
+#pragma unroll
+            for (int h = 0; h < 2; h++) {
+                const int r = (m0 + 8 * m) * 16 + gid + 8 * h, c = col0 + (nv0 + i) * 8 + 2 * tig;
+                if (r < a.dim && c < a.vdim) *reinterpret_cast<float2*>(dst + (int64_t)r * a.vdim + c) = make_float2(s[m][i][2 * h], s[m][i][2 * h + 1]);
+            }
+}
+
+// ------------------------------------------------------------------ states before the chunks
+// A thread owns four neighbouring numbers of a head's state and walks the chunks of the portion.  The running maximum after the portion is left to
+// the next launch: every thread reads the one before it.
+template <int KIND>
+__global__ void __launch_bounds__(THREADS)
+    chunk_walk_kernel(const __grid_constant__ Recurrence a, const __grid_constant__ RecurrenceChunks c, const __grid_constant__ Scratch s, uint32_t* __restrict__ err) {
+    constexpr bool FORGET = KIND == REC_FORGET, MLSTM = KIND == REC_MLSTM;
+    const int per_seq = (c.rows_per_seq + C - 1) / C;
+    const ChunkPortion p = c.portions ? c.portions[blockIdx.z] : ChunkPortion{(int)blockIdx.z * c.rows_per_seq, c.rows_per_seq, (int)blockIdx.z * per_seq};
+    const tsb_row_desc rd = a.rows[p.first_row];
+    const int head = blockIdx.y, pos0 = rd.base + rd.slot, n = (p.n_rows + C - 1) / C;
+    const int state4 = a.dim * a.vdim / 4, i4 = blockIdx.x * THREADS + threadIdx.x;
+    const int norm_i = i4 - state4;  // MLSTM: threads behind the state take a number of the normaliser each
     if (rd.seq < 0 || rd.seq >= a.state.n_streams) {
         if (threadIdx.x == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
         pdl_wait();
         return;
     }
-    const int n_chunks = (p.n_rows + C - 1) / C;
-    const __nv_bfloat16 *gq = static_cast<const __nv_bfloat16*>(a.q) + key_at, *gk = static_cast<const __nv_bfloat16*>(a.k) + key_at;
-    const __nv_bfloat16* gv = static_cast<const __nv_bfloat16*>(a.v) + (int64_t)head * a.vdim + col0;
-
-    // ---- copies of a chunk (rows and columns outside are zeros)
-    auto issue = [&](int chunk) {
-        if (chunk < n_chunks) {
-            const int row0 = p.row_first + chunk * C, n = min(C, p.n_rows - chunk * C), st = chunk & 1;
-            if (!FORGET) {
-                for (int i = threadIdx.x; i < C * (DK / 8); i += THREADS) {
-                    const int r = i / (DK / 8), c = i % (DK / 8);
-                    const bool ok = r < n && c * 8 < a.dim;
-                    const int64_t row = ok ? row0 + r : row0, col = ok ? c * 8 : 0;
-                    cp16(base + st * M::KEY_STAGE + M::Q + at<KB>(r, c), gq + row * a.q_stride + col, ok);
-                    cp16(base + st * M::KEY_STAGE + M::K + at<KB>(r, c), gk + row * a.k_stride + col, ok);
-                }
-            }
-            for (int i = threadIdx.x; i < C * (VB / 8); i += THREADS) {
-                const int r = i / (VB / 8), c = i % (VB / 8);
-                const bool ok = r < n && col0 + c * 8 < a.vdim;
-                cp16(base + M::V + st * M::VAL + at<BV>(r, c), gv + (int64_t)(ok ? row0 + r : row0) * a.v_stride + (ok ? c * 8 : 0), ok);
-            }
-        }
-        cp_async_commit();
-    };
-    const int ch = threadIdx.x % DK, split_i = threadIdx.x / DK;  // FORGET: the thread's channel and rows
-    auto z_at = [&](int r) -> float& { return reinterpret_cast<float*>(smem + M::Z)[r * DK + ch]; };
-    auto raw = [&](int chunk) {  // FORGET: pre-activations and queries of a chunk
-        if (!FORGET || chunk >= n_chunks) return;
-        const int row0 = p.row_first + chunk * C, n = min(C, p.n_rows - chunk * C);
-        const float* gz = a.gate + (int64_t)head * a.dim;
-        for (int i = threadIdx.x; i < C * (DK / 4); i += THREADS) {
-            const int r = i / (DK / 4), c = i % (DK / 4);
-            const bool ok = r < n && c * 4 < a.dim;
-            cp16(base + M::Z + (r * DK + c * 4) * 4, gz + (ok ? row0 + r : row0) * a.gate_stride + (ok ? c * 4 : 0), ok);
-        }
-        for (int i = threadIdx.x; i < C * (DK / 8); i += THREADS) {
-            const int r = i / (DK / 8), c = i % (DK / 8);
-            const bool ok = r < n && c * 8 < a.dim;
-            cp16(base + M::RAW_Q + (r * DK + c * 8) * 2, gq + (int64_t)(ok ? row0 + r : row0) * a.q_stride + (ok ? c * 8 : 0), ok);
-        }
-    };
-    // decay per head: lane l of warp 0 has the gates of rows 2 l and 2 l + 1 of the next chunk
-    float2 gate2[2];
-    const float rate = SSD ? expf(a.a_log[head]) : 0.f;
-    auto fetch_gates = [&](int chunk) {
-        if (FORGET || warp != 0 || chunk >= n_chunks) return;
-        const int n = min(C, p.n_rows - chunk * C);
-#pragma unroll
-        for (int i = 0; i < 2; i++) {
-            const int r = 2 * lane + i, row = p.row_first + chunk * C + r;
-            gate2[i] = r < n ? (MLSTM ? mlstm_gates(a, row, head) : ssd_gates(a, row, head, rate)) : make_float2(MLSTM ? -1e30f : 0.f, 0.f);
-        }
-    };
-
-    // ---- the state before the portion, written by an earlier pass: accumulators of warps 4 .. 7, m-tiles warp - 4, warp, ..
-    float s[MS][NV][4];
+    const bool is_norm = MLSTM && norm_i >= 0 && norm_i < a.dim;
+    const int64_t from = rec_slot(a, rd.seq, pos0 - 1) * a.heads + head, to = rec_slot(a, rd.seq, pos0 + p.n_rows - 1) * a.heads + head;
+    const int64_t head_state = (int64_t)a.dim * a.vdim;
+    const int copies = recurrence_copies(a.vdim);
+    const int row = i4 < state4 ? i4 * 4 / a.vdim : 0;
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
     double top = 0.0;
-    const int64_t head_state = (int64_t)a.dim * vp;
-    const int64_t slot0 = rec_slot(a, rd.seq, pos0 - 1) * a.heads + head;
-    auto state_to_smem = [&](int buf) {
-#pragma unroll
-        for (int m = 0; m < MS; m++)
-#pragma unroll
-            for (int n = 0; n < NV; n++)
-#pragma unroll
-                for (int h = 0; h < 2; h++) {
-                    const int r = (warp - 4 + 4 * m) * 16 + gid + 8 * h;
-                    uint32_t hi, lo;
-                    split(s[m][n][2 * h], s[m][n][2 * h + 1], hi, lo);
-                    const uint32_t off = at<BV>(r, n) + tig * 4;
-                    *reinterpret_cast<uint32_t*>(smem + M::S + 2 * buf * M::STATE + off) = hi;
-                    *reinterpret_cast<uint32_t*>(smem + M::S + (2 * buf + 1) * M::STATE + off) = lo;
-                }
-    };
-    if (warp >= 4) {
-        const float* src = a.state.s + slot0 * head_state;
-#pragma unroll
-        for (int m = 0; m < MS; m++)
-#pragma unroll
-            for (int n = 0; n < NV; n++)
-#pragma unroll
-                for (int i = 0; i < 4; i++) {
-                    const int r = (warp - 4 + 4 * m) * 16 + gid + 8 * (i >> 1), c = col0 + n * 8 + 2 * tig + (i & 1);
-                    s[m][n][i] = pos0 > 0 && r < a.dim && c < vp ? src[(int64_t)r * vp + c] : 0.f;
-                }
-        state_to_smem(0);
-        if (MLSTM)
-            for (int i = threadIdx.x - 128; i < DK; i += 128) norm[i] = pos0 > 0 && i < a.dim ? a.state.norm[slot0 * a.dim + i] : 0.f;
+    if (pos0 > 0) {
+        if (i4 < state4) v = *reinterpret_cast<const float4*>(a.state.s + from * head_state + (int64_t)i4 * 4);
+        if (is_norm) v.x = a.state.norm[from * copies * a.dim + norm_i];
+        if (MLSTM) top = a.state.top[from * copies];
     }
-    if (MLSTM && pos0 > 0) top = a.state.top[slot0];
-    const float skip = SSD ? a.skip[head] : 0.f;
-    if (FORGET)
-        for (int i = threadIdx.x; i < DK; i += THREADS) lower[i] = i < a.dim ? a.lower[(int64_t)head * a.dim + i] : 1.f;
     pdl_wait();
-    raw(0);
-    issue(0);
-    fetch_gates(0);
-
-    int state_buf = 0;
-    for (int chunk = 0; chunk < n_chunks; chunk++) {
-        const int n = min(C, p.n_rows - chunk * C), row0 = p.row_first + chunk * C;
-        if (!FORGET) issue(chunk + 1), cp_async_wait<1>();
-        else cp_async_wait<0>();
-        if (!FORGET && warp == 0) {
-            const float d0 = gate2[0].y, d1 = gate2[1].y;
-            float sum = d0 + d1;
+    pdl_launch_dependents();
+    if (i4 >= state4 && !is_norm) return;
+    constexpr int AHEAD = 4;
+    const int width = FORGET ? a.dim : 2;
+    float4 next[AHEAD];
+    float2 gate[AHEAD];
+    auto fetch = [&](int k, float4& x, float2& g) {
+        const int64_t slot = (int64_t)(p.first_chunk + k) * a.heads + head;
+        if (is_norm) x.x = s.norm[slot * a.dim + norm_i];
+        else x = *reinterpret_cast<const float4*>(s.add + slot * head_state + (int64_t)i4 * 4);
+        if (FORGET) g.x = s.decay[slot * width + row];
+        else g = *reinterpret_cast<const float2*>(s.decay + slot * width);
+    };
 #pragma unroll
-            for (int o = 1; o < 32; o <<= 1) {
-                const float v = __shfl_up_sync(0xffffffffu, sum, o);
-                if (lane >= o) sum += v;
+    for (int k = 0; k < AHEAD; k++)
+        if (k < n) fetch(k, next[k], gate[k]);
+    for (int k0 = 0; k0 < n; k0 += AHEAD) {
+#pragma unroll
+        for (int j = 0; j < AHEAD; j++) {
+            const int k = k0 + j;
+            if (k >= n) break;
+            const float4 add = next[j];
+            const float2 g = gate[j];
+            if (k + AHEAD < n) fetch(k + AHEAD, next[j], gate[j]);
+            const int64_t slot = (int64_t)(p.first_chunk + k) * a.heads + head;
+            if (is_norm) {
+                s.norm[slot * a.dim + norm_i] = v.x;
+                if (norm_i == 0) s.top[slot] = top;
+            } else {
+                uint4 w;
+                split(v.x, v.y, w.x, w.z);
+                split(v.z, v.w, w.y, w.w);
+                *reinterpret_cast<uint4*>(s.add + slot * head_state + (int64_t)i4 * 4) = w;
             }
-            const float l1 = sum, l0 = sum - d1;  // log decay up to rows 2 lane + 1 and 2 lane
-            const float l_end = __shfl_sync(0xffffffffu, sum, 31);
+            float keep = g.x, write = 1.f;
+            if (MLSTM) {
+                const double old = top + g.x, m = fmax(old, (double)g.y);
+                keep = expf((float)(old - m)), write = expf((float)(g.y - m));
+                top = m;
+            }
+            v.x = fmaf(keep, v.x, write * add.x), v.y = fmaf(keep, v.y, write * add.y), v.z = fmaf(keep, v.z, write * add.z), v.w = fmaf(keep, v.w, write * add.w);
+        }
+    }
+    if (is_norm) {
+        for (int k = 0; k < copies; k++) a.state.norm[(to * copies + k) * a.dim + norm_i] = v.x;
+    } else {
+        *reinterpret_cast<float4*>(a.state.s + to * head_state + (int64_t)i4 * 4) = v;
+    }
+}
+
+// ------------------------------------------------------------------ outputs of a chunk
+template <int KIND, int DK>
+struct OutSmem {
+    static constexpr bool FORGET = KIND == REC_FORGET;
+    static constexpr int KEY = C * DK * 2, VAL = C * VB * 2, STATE = DK * VB * 2, PROD = C * C * 2;
+    // queries and keys (FORGET: high and low parts of each), values, state (high, low), products (high, low)
+    static constexpr int Q = 0, K = FORGET ? 2 * KEY : KEY, V = 2 * K, S = V + VAL, P = S + 2 * STATE;
+    static constexpr int F = P + 2 * PROD;
+    static constexpr int Z = S;  // FORGET: the gates of the chunk, before the state takes their place
+    static_assert(!FORGET || C * DK * 4 <= 2 * STATE, "");
+    static constexpr int BYTES = F + (FORGET ? THREADS : 4 * C + 8 + DK + 5 * C) * 4;
+};
+
+template <int KIND, int DK>
+__global__ void __launch_bounds__(THREADS, KIND == REC_FORGET || DK > 128 ? 1 : 2)
+    chunk_out_kernel(const __grid_constant__ Recurrence a, const __grid_constant__ RowTiles chunks, const __grid_constant__ Scratch in, uint32_t* __restrict__ err) {
+    using M = OutSmem<KIND, DK>;
+    constexpr bool FORGET = KIND == REC_FORGET, MLSTM = KIND == REC_MLSTM, SSD = KIND == REC_SSD;
+    constexpr int KB = DK * 2, KS = DK / 16, NV = 4;  // a warp has 16 rows and 32 columns of the output
+    constexpr int RS = FORGET ? THREADS / DK : 1, TR = C / RS;
+    extern __shared__ __align__(128) uint8_t smem[];
+    const uint32_t base = smem_u32(smem);
+    float* fv = reinterpret_cast<float*>(smem + M::F);
+    float *ea = fv, *eb = fv + C, *gain = fv + 2 * C, *floor_ = fv + 3 * C, *norm = fv + 4 * C + 8, *nq = norm + DK;  // nq [rows][5]: shares of n . q
+    __shared__ int cut_end;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
+    const int head = blockIdx.y, col0 = blockIdx.x * VB, key_at = head / a.heads_per_key * a.dim;
+    const AttnTile tile = row_tile(chunks, blockIdx.z);
+    const int row0 = tile.row_first, n = min(tile.n_rows, C);
+    const int64_t slot = (int64_t)blockIdx.z * a.heads + head;
+    const __nv_bfloat16* gq = static_cast<const __nv_bfloat16*>(a.q) + (int64_t)row0 * a.q_stride + key_at;
+    pdl_wait();
+    pdl_launch_dependents();
+    copy_tile<BV>(base + M::V, static_cast<const __nv_bfloat16*>(a.v) + (int64_t)row0 * a.v_stride + (int64_t)head * a.vdim + col0, a.v_stride, n, a.vdim - col0);
+    if (FORGET) {
+        copy_gates<DK>(a, base + M::Z, row0, n, head);
+    } else {
+        copy_tile<KB>(base + M::Q, gq, a.q_stride, n, a.dim);
+        copy_tile<KB>(base + M::K, static_cast<const __nv_bfloat16*>(a.k) + (int64_t)row0 * a.k_stride + key_at, a.k_stride, n, a.dim);
+    }
+    cp_async_commit();
+    // the state: four numbers as four high and four low halves, to two tiles
+    constexpr int PIECES = DK * (VB / 4);
+    const float* src = in.add + slot * a.dim * a.vdim + col0;
+    auto state_piece = [&](int i, bool& ok) {
+        const int r = i / (VB / 4), c = i % (VB / 4);
+        ok = r < a.dim && col0 + c * 4 < a.vdim;
+        return ok ? *reinterpret_cast<const uint4*>(src + (int64_t)r * a.vdim + c * 4) : make_uint4(0, 0, 0, 0);
+    };
+    auto state_to_smem = [&](int i, const uint4& w) {
+        const int r = i / (VB / 4), c = i % (VB / 4);
+        const uint32_t off = at<BV>(r, c >> 1) + (c & 1) * 8;
+        *reinterpret_cast<uint2*>(smem + M::S + off) = make_uint2(w.x, w.y);
+        *reinterpret_cast<uint2*>(smem + M::S + M::STATE + off) = make_uint2(w.z, w.w);
+    };
+    auto load_state = [&]() {
+        for (int i0 = threadIdx.x; i0 < PIECES; i0 += 8 * THREADS) {
+            uint4 w[8];
+            bool ok;
+#pragma unroll
+            for (int k = 0; k < 8; k++)
+                if (i0 + k * THREADS < PIECES) w[k] = state_piece(i0 + k * THREADS, ok);
+#pragma unroll
+            for (int k = 0; k < 8; k++)
+                if (i0 + k * THREADS < PIECES) state_to_smem(i0 + k * THREADS, w[k]);
+        }
+    };
+    if (!FORGET) {
+        load_state();
+        if (MLSTM)
+            for (int i = threadIdx.x; i < DK; i += THREADS) norm[i] = i < a.dim ? in.norm[slot * a.dim + i] : 0.f;
+        if (warp == 0) {
+            const RowGates g = row_gates<FORGET ? REC_SSD : KIND>(a, row0, n, head, lane);
             if (SSD) {
-                ea[2 * lane] = l0 * LOG2E, ea[2 * lane + 1] = l1 * LOG2E, eb[2 * lane] = -l0 * LOG2E, eb[2 * lane + 1] = -l1 * LOG2E;
-                gain[2 * lane] = gate2[0].x, gain[2 * lane + 1] = gate2[1].x;
-                if (lane == 0) scal[0] = l_end * LOG2E, scal[1] = expf(l_end);
+#pragma unroll
+                for (int i = 0; i < 2; i++) ea[2 * lane + i] = g.log_e[i] * LOG2E, eb[2 * lane + i] = -g.log_e[i] * LOG2E, gain[2 * lane + i] = g.in[i];
             } else {
                 // relative to the maximum before the chunk: i_s - F_s - m, and its running maximum with 0
-                const float b0 = (float)((double)gate2[0].x - l0 - top), b1 = (float)((double)gate2[1].x - l1 - top);
+                const double top = in.top[slot];
+                const float b0 = (float)((double)g.in[0] - g.log_e[0] - top), b1 = (float)((double)g.in[1] - g.log_e[1] - top);
                 float mx = fmaxf(b0, b1);
 #pragma unroll
                 for (int o = 1; o < 32; o <<= 1) {
@@ -213,314 +429,310 @@ __global__ void __launch_bounds__(THREADS, 1)
                     if (lane >= o) mx = fmaxf(mx, v);
                 }
                 const float before = __shfl_up_sync(0xffffffffu, mx, 1);
-                const float m1 = fmaxf(mx, 0.f), m0 = fmaxf(lane > 0 ? fmaxf(before, b0) : b0, 0.f), m_end = __shfl_sync(0xffffffffu, m1, 31);
+                const float m1 = fmaxf(mx, 0.f), m0 = fmaxf(lane > 0 ? fmaxf(before, b0) : b0, 0.f);
                 ea[2 * lane] = -m0 * LOG2E, ea[2 * lane + 1] = -m1 * LOG2E, eb[2 * lane] = b0 * LOG2E, eb[2 * lane + 1] = b1 * LOG2E;
                 gain[2 * lane] = gain[2 * lane + 1] = 1.f;
-                floor_[2 * lane] = expf(-(float)(top + l0 + m0)), floor_[2 * lane + 1] = expf(-(float)(top + l1 + m1));
-                if (lane == 0) scal[0] = -m_end * LOG2E, scal[1] = expf(-m_end);
-                top += (double)l_end + m_end;
-            }
-            fetch_gates(chunk + 1);
-        }
-        __syncthreads();  // the chunk's copies and gates are there
-        const uint32_t vt = base + M::V + (chunk & 1) * M::VAL;
-
-        for (int cut = 0; cut < n;) {  // FORGET: usually once
-            int end = n;
-            if (FORGET) {
-                // E from row `cut` on: products within the thread's rows, then over the row splits.  The first time round the pre-activations
-                // become 1 - f = (1 - l) sigmoid(-z).
-                const float low = lower[ch];
-                float mine = 1.f;
-#pragma unroll 4
-                for (int i = 0; i < TR; i++) {
-                    const int r = split_i * TR + i;
-                    float& x = z_at(r);
-                    if (cut == 0) {
-                        const float e = __expf(-fabsf(x)), d = __fdividef(1.f, 1.f + e);
-                        x = r < n ? (1.f - low) * (x >= 0.f ? e * d : d) : 0.f;
-                    }
-                    if (r >= cut) mine *= 1.f - x;
-                }
-                totals[threadIdx.x] = mine;
-                if (threadIdx.x == 0) cut_end = n;
-                __syncthreads();
-                float e0 = 1.f;
-                for (int i = 0; i < split_i; i++) e0 *= totals[i * DK + ch];
-                // E only falls: the chunk is cut if it ends too low
-                if (__syncthreads_or(e0 * mine < E_MIN)) {
-                    float e = e0;
-                    for (int i = 0; i < TR; i++) {
-                        const int r = split_i * TR + i;
-                        if (r < cut || r >= n) continue;
-                        e *= 1.f - z_at(r);
-                        if (e < E_MIN && r > cut) {
-                            atomicMin(&cut_end, r);
-                            break;
-                        }
-                    }
-                    __syncthreads();
-                    end = cut_end;
-                }
-                float e = e0;
-#pragma unroll 4
-                for (int i = 0; i < TR; i++) {
-                    const int r = split_i * TR + i;
-                    const bool in = r >= cut && r < end;
-                    const float k = z_at(r), x = __bfloat162float(reinterpret_cast<const __nv_bfloat16*>(smem + M::RAW_Q)[r * DK + ch]);
-                    if (in) e = fmaxf(e * (1.f - k), E_MIN);  // the first row of a cut may fall further: nothing of the rows before is left then
-                    const float qe = in ? __fdividef(x, 1.f + __expf(-x)) * e : 0.f, ke = in ? k * (1.f / e) : 0.f;
-                    const __nv_bfloat16 qh = __float2bfloat16_rn(qe), kh = __float2bfloat16_rn(ke);
-                    const uint32_t off = at<KB>(r, ch >> 3) + (ch & 7) * 2;
-                    *reinterpret_cast<__nv_bfloat16*>(smem + M::Q + off) = qh;
-                    *reinterpret_cast<__nv_bfloat16*>(smem + M::Q + M::KEY + off) = __float2bfloat16_rn(qe - __bfloat162float(qh));
-                    *reinterpret_cast<__nv_bfloat16*>(smem + M::K + off) = kh;
-                    *reinterpret_cast<__nv_bfloat16*>(smem + M::K + M::KEY + off) = __float2bfloat16_rn(ke - __bfloat162float(kh));
-                }
-                if (end > split_i * TR && end <= (split_i + 1) * TR) e_end[ch] = e;
-            } else {
-                // values weighted to the end of the chunk
-                for (int i = threadIdx.x; i < C * (VB / 2); i += THREADS) {
-                    const int r = i / (VB / 2), c = i % (VB / 2);
-                    const uint32_t off = at<BV>(r, c >> 2) + (c & 3) * 4;
-                    const uint32_t v = *reinterpret_cast<const uint32_t*>(smem + M::V + (chunk & 1) * M::VAL + off);
-                    const float w = ex2(scal[0] + eb[r]) * gain[r];
-                    if (MLSTM && c == 0) wv[r] = w;
-                    uint32_t hi, lo;
-                    split(__uint_as_float(v << 16) * w, __uint_as_float(v & 0xFFFF0000u) * w, hi, lo);
-                    *reinterpret_cast<uint32_t*>(smem + M::W + off) = hi;
-                    *reinterpret_cast<uint32_t*>(smem + M::W + M::VAL + off) = lo;
+                floor_[2 * lane] = expf(-(float)(top + g.log_e[0] + m0)), floor_[2 * lane + 1] = expf(-(float)(top + g.log_e[1] + m1));
+                const tsb_row_desc rd = a.rows[row0 + n - 1];
+                if (lane == 31 && blockIdx.x == 0 && (row0 + n >= a.n_rows || a.rows[row0 + n].seq != rd.seq)) {  // the portion's last row
+                    const int copies = recurrence_copies(a.vdim);
+                    double* to = a.state.top + (rec_slot(a, rd.seq, rd.base + rd.slot) * a.heads + head) * copies;
+                    for (int k = 0; k < copies; k++) to[k] = top + g.end + m1;
                 }
             }
-            __syncthreads();
-            if (FORGET && end == n) raw(chunk + 1), issue(chunk + 1);  // what they overwrite has been used
-            const uint32_t qt = base + (FORGET ? 0 : (chunk & 1) * M::KEY_STAGE) + M::Q, kt = base + (FORGET ? 0 : (chunk & 1) * M::KEY_STAGE) + M::K;
-            const uint32_t sh = base + M::S + 2 * state_buf * M::STATE, sl = sh + M::STATE;
-            if (warp < 4) {
-                // ---- outputs of rows 16 warp .. + 15
-                const int t0 = warp * 16;
-                if (t0 < end && t0 + 16 > cut) {
-                    uint32_t qa[KS][4], ql[FORGET ? KS : 1][4];
-#pragma unroll
-                    for (int ks = 0; ks < KS; ks++) {
-                        ldsm4(qa[ks], qt + at<KB>(t0 + (lane & 15), ks * 2 + (lane >> 4)));
-                        if (FORGET) ldsm4(ql[FORGET ? ks : 0], qt + M::KEY + at<KB>(t0 + (lane & 15), ks * 2 + (lane >> 4)));
-                    }
-                    float o[NV][4];
-#pragma unroll
-                    for (int i = 0; i < NV; i++)
-#pragma unroll
-                        for (int j = 0; j < 4; j++) o[i][j] = 0.f;
-#pragma unroll
-                    for (int ks = 0; ks < KS; ks++)
-#pragma unroll
-                        for (int np = 0; np < NV / 2; np++) {
-                            uint32_t bh[4], bl[4];
-                            ldsm4_t(bh, sh + at<BV>(ks * 16 + (lane & 15), np * 2 + (lane >> 4)));
-                            ldsm4_t(bl, sl + at<BV>(ks * 16 + (lane & 15), np * 2 + (lane >> 4)));
-                            mma_bf16(o[2 * np], qa[ks], bh[0], bh[1]), mma_bf16(o[2 * np + 1], qa[ks], bh[2], bh[3]);
-                            mma_bf16(o[2 * np], qa[ks], bl[0], bl[1]), mma_bf16(o[2 * np + 1], qa[ks], bl[2], bl[3]);
-                            if (FORGET) mma_bf16(o[2 * np], ql[FORGET ? ks : 0], bh[0], bh[1]), mma_bf16(o[2 * np + 1], ql[FORGET ? ks : 0], bh[2], bh[3]);
-                        }
-                    const int ta = t0 + gid, tb = ta + 8;
-                    const float ea0 = FORGET ? 0.f : ea[ta], ea1 = FORGET ? 0.f : ea[tb];
-                    float nq[2] = {0.f, 0.f};  // MLSTM: the lane's share of n . q
-                    if (!FORGET) {
-                        const float f0 = ex2(ea0), f1 = ex2(ea1);
-#pragma unroll
-                        for (int i = 0; i < NV; i++) o[i][0] *= f0, o[i][1] *= f0, o[i][2] *= f1, o[i][3] *= f1;
-                        if (MLSTM) {
-                            const float* nb = norm + state_buf * DK;
-#pragma unroll
-                            for (int ks = 0; ks < KS; ks++) {
-                                const float2 n0 = *reinterpret_cast<const float2*>(nb + ks * 16 + 2 * tig), n1 = *reinterpret_cast<const float2*>(nb + ks * 16 + 8 + 2 * tig);
-#pragma unroll
-                                for (int h = 0; h < 2; h++) {
-                                    const uint32_t x = qa[ks][h], y = qa[ks][2 + h];
-                                    nq[h] = fmaf(__uint_as_float(x << 16), n0.x, fmaf(__uint_as_float(x & 0xFFFF0000u), n0.y, nq[h]));
-                                    nq[h] = fmaf(__uint_as_float(y << 16), n1.x, fmaf(__uint_as_float(y & 0xFFFF0000u), n1.y, nq[h]));
-                                }
-                            }
-                            nq[0] *= f0, nq[1] *= f1;
-                        }
-                    }
-                    for (int jt = cut / 16; jt <= warp; jt++) {
-                        float s0[2][4];
-#pragma unroll
-                        for (int i = 0; i < 2; i++)
-#pragma unroll
-                            for (int j = 0; j < 4; j++) s0[i][j] = 0.f;
-#pragma unroll
-                        for (int kp = 0; kp < KS / 2; kp++)
-#pragma unroll
-                            for (int i = 0; i < 2; i++) {
-                                uint32_t b[4];
-                                ldsm4(b, kt + at<KB>(jt * 16 + i * 8 + (lane & 7), kp * 4 + (lane >> 3)));
-                                mma_bf16(s0[i], qa[2 * kp], b[0], b[1]), mma_bf16(s0[i], qa[2 * kp + 1], b[2], b[3]);
-                                if (FORGET) {
-                                    uint32_t bl[4];
-                                    ldsm4(bl, kt + M::KEY + at<KB>(jt * 16 + i * 8 + (lane & 7), kp * 4 + (lane >> 3)));
-                                    mma_bf16(s0[i], qa[2 * kp], bl[0], bl[1]), mma_bf16(s0[i], qa[2 * kp + 1], bl[2], bl[3]);
-                                    mma_bf16(s0[i], ql[FORGET ? 2 * kp : 0], b[0], b[1]), mma_bf16(s0[i], ql[FORGET ? 2 * kp + 1 : 0], b[2], b[3]);
-                                }
-                            }
-                        uint32_t ph[4], pl[4];
-#pragma unroll
-                        for (int i = 0; i < 2; i++) {
-                            const int c0 = jt * 16 + i * 8 + 2 * tig;
-#pragma unroll
-                            for (int j = 0; j < 4; j++) {
-                                const int c = c0 + (j & 1), t = j < 2 ? ta : tb;
-                                float w = 0.f;
-                                if (c <= t) w = FORGET ? s0[i][j] : s0[i][j] * (ex2((j < 2 ? ea0 : ea1) + eb[c]) * gain[c]);
-                                s0[i][j] = w;
-                            }
-                            if (MLSTM) nq[0] += s0[i][0] + s0[i][1], nq[1] += s0[i][2] + s0[i][3];
-                            split(s0[i][0], s0[i][1], ph[2 * i], pl[2 * i]);
-                            split(s0[i][2], s0[i][3], ph[2 * i + 1], pl[2 * i + 1]);
-                        }
-#pragma unroll
-                        for (int np = 0; np < NV / 2; np++) {
-                            uint32_t b[4];
-                            ldsm4_t(b, vt + at<BV>(jt * 16 + (lane & 15), np * 2 + (lane >> 4)));
-                            mma_bf16(o[2 * np], ph, b[0], b[1]), mma_bf16(o[2 * np + 1], ph, b[2], b[3]);
-                            mma_bf16(o[2 * np], pl, b[0], b[1]), mma_bf16(o[2 * np + 1], pl, b[2], b[3]);
-                        }
-                    }
-                    float out_f[2] = {a.q_scale, a.q_scale};
-                    if (MLSTM) {
-#pragma unroll
-                        for (int h = 0; h < 2; h++) {
-                            nq[h] += __shfl_xor_sync(0xffffffffu, nq[h], 1);
-                            nq[h] += __shfl_xor_sync(0xffffffffu, nq[h], 2);
-                            out_f[h] = a.q_scale / (fmaxf(fabsf(nq[h] * a.q_scale), floor_[h ? tb : ta]) + 1e-6f);
-                        }
-                    }
-#pragma unroll
-                    for (int h = 0; h < 2; h++) {
-                        const int t = h ? tb : ta;
-                        if (t < cut || t >= end) continue;
-                        float* dst = a.out + (int64_t)(row0 + t) * a.out_stride + (int64_t)head * a.vdim + col0;
-#pragma unroll
-                        for (int i = 0; i < NV; i++) {
-                            float2 v = make_float2(o[i][2 * h] * out_f[h], o[i][2 * h + 1] * out_f[h]);
-                            if (SSD) {
-                                const uint32_t x = *reinterpret_cast<const uint32_t*>(smem + M::V + (chunk & 1) * M::VAL + at<BV>(t, i) + tig * 4);
-                                v.x = fmaf(skip, __uint_as_float(x << 16), v.x), v.y = fmaf(skip, __uint_as_float(x & 0xFFFF0000u), v.y);
-                            }
-                            if (col0 + i * 8 + 2 * tig < a.vdim) *reinterpret_cast<float2*>(dst + i * 8 + 2 * tig) = v;
-                        }
-                    }
-                }
-            } else {
-                // ---- the state at the end of the chunk (or of the cut)
-                if (!FORGET) {
-                    const float d = scal[1];
-#pragma unroll
-                    for (int m = 0; m < MS; m++)
-#pragma unroll
-                        for (int i = 0; i < NV; i++)
-#pragma unroll
-                            for (int j = 0; j < 4; j++) s[m][i][j] *= d;
-                }
-                const uint32_t bh_at = FORGET ? vt : base + M::W;
-                for (int ks = cut / 16; ks * 16 < end; ks++) {
-                    uint32_t bh[NV / 2][4], bl[FORGET ? 1 : NV / 2][4];
-#pragma unroll
-                    for (int np = 0; np < NV / 2; np++) {
-                        ldsm4_t(bh[np], bh_at + at<BV>(ks * 16 + (lane & 15), np * 2 + (lane >> 4)));
-                        if (!FORGET) ldsm4_t(bl[FORGET ? 0 : np], bh_at + M::VAL + at<BV>(ks * 16 + (lane & 15), np * 2 + (lane >> 4)));
-                    }
-#pragma unroll
-                    for (int m = 0; m < MS; m++) {
-                        const int c8 = (warp - 4 + 4 * m) * 2 + ((lane >> 3) & 1), r = ks * 16 + (lane & 7) + ((lane >> 4) << 3);
-                        uint32_t ka[4], kl[4];
-                        ldsm4_t(ka, kt + at<KB>(r, c8));
-                        if (FORGET) ldsm4_t(kl, kt + M::KEY + at<KB>(r, c8));
-#pragma unroll
-                        for (int np = 0; np < NV / 2; np++) {
-                            mma_bf16(s[m][2 * np], ka, bh[np][0], bh[np][1]), mma_bf16(s[m][2 * np + 1], ka, bh[np][2], bh[np][3]);
-                            if (FORGET) {
-                                mma_bf16(s[m][2 * np], kl, bh[np][0], bh[np][1]), mma_bf16(s[m][2 * np + 1], kl, bh[np][2], bh[np][3]);
-                            } else {
-                                const uint32_t(&x)[4] = bl[FORGET ? 0 : np];
-                                mma_bf16(s[m][2 * np], ka, x[0], x[1]), mma_bf16(s[m][2 * np + 1], ka, x[2], x[3]);
-                            }
-                        }
-                    }
-                }
-                if (FORGET) {
-#pragma unroll
-                    for (int m = 0; m < MS; m++) {
-                        const float d0 = e_end[(warp - 4 + 4 * m) * 16 + gid], d1 = e_end[(warp - 4 + 4 * m) * 16 + gid + 8];
-#pragma unroll
-                        for (int i = 0; i < NV; i++) s[m][i][0] *= d0, s[m][i][1] *= d0, s[m][i][2] *= d1, s[m][i][3] *= d1;
-                    }
-                }
-                state_to_smem(state_buf ^ 1);
-                if (MLSTM) {
-                    for (int c = threadIdx.x - 128; c < DK; c += 128) {
-                        float x = norm[state_buf * DK + c] * scal[1];
-#pragma unroll 8
-                        for (int r = 0; r < C; r++)
-                            x = fmaf(wv[r], __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(
-                                                               smem + (chunk & 1) * M::KEY_STAGE + M::K + at<KB>(r, c >> 3) + (c & 7) * 2)), x);
-                        norm[(state_buf ^ 1) * DK + c] = x;
-                    }
-                }
-            }
-            state_buf ^= 1;
-            cut = end;
-            __syncthreads();  // outputs have read what the next cut or chunk overwrites
         }
     }
     cp_async_wait<0>();
-    pdl_launch_dependents();
-    const int64_t slot = rec_slot(a, rd.seq, pos0 + p.n_rows - 1) * a.heads + head;
-    if (warp >= 4) {
-        float* dst = a.state.s + slot * head_state;
+    __syncthreads();
+
+    // ---- FORGET: queries times E_t, keys over E_s
+    const int ch = FORGET ? threadIdx.x % DK : 0, part = FORGET ? threadIdx.x / DK : 0;
+    float kk[FORGET ? TR : 1];  // 1 - f of the thread's rows
+    auto query = [&](int r) {
+        const float x = r < n && ch < a.dim ? __bfloat162float(gq[r * a.q_stride + ch]) : 0.f;
+        return __fdividef(x, 1.f + __expf(-x));
+    };
+    bool cuts = false;
+    float before = 1.f;  // E at the start of the thread's rows
+    if (FORGET) {
+        float* pre = reinterpret_cast<float*>(smem + M::Z);
+        const float mine = forget_gates<DK>(a, pre, head, n);
+        fv[threadIdx.x] = mine;
 #pragma unroll
-        for (int m = 0; m < MS; m++)
+        for (int i = 0; i < (FORGET ? TR : 0); i++) kk[i] = pre[(part * TR + i) * DK + ch];
+        __syncthreads();
+        for (int i = 0; i < part; i++) before *= fv[i * DK + ch];
+        cuts = __syncthreads_or(before * mine < E_MIN);  // E only falls
+        load_state();                                   // over the gates
+        float e = before;
 #pragma unroll
-            for (int n = 0; n < NV; n++)
+        for (int i = 0; i < (FORGET ? TR : 0); i++) {
+            const int r = part * TR + i;
+            e *= 1.f - kk[i];
+            const uint32_t off = at<KB>(r, ch >> 3) + (ch & 7) * 2;
+            put_split(smem + M::Q, smem + M::Q + M::KEY, off, query(r) * e);
+            put_split(smem + M::K, smem + M::K + M::KEY, off, cuts ? 0.f : __fdividef(kk[i], e));
+        }
+        __syncthreads();
+    }
+
+    const int mt = warp & 3, c8 = (warp >> 2) * NV;  // row tile, first column group
+    const int ta = mt * 16 + gid, tb = ta + 8;
+    float o[NV][4] = {};
+    // ---- queries against the state
+    {
+        float share[2] = {0.f, 0.f};
+#pragma unroll 4
+        for (int ks = 0; ks < KS; ks++) {
+            uint32_t qa[4], ql[4];
+            ldsm4(qa, base + M::Q + at<KB>(mt * 16 + (lane & 15), ks * 2 + (lane >> 4)));
+            if (FORGET) ldsm4(ql, base + M::Q + M::KEY + at<KB>(mt * 16 + (lane & 15), ks * 2 + (lane >> 4)));
+#pragma unroll
+            for (int np = 0; np < NV / 2; np++) {
+                uint32_t bh[4], bl[4];
+                ldsm4_t(bh, base + M::S + at<BV>(ks * 16 + (lane & 15), c8 + np * 2 + (lane >> 4)));
+                ldsm4_t(bl, base + M::S + M::STATE + at<BV>(ks * 16 + (lane & 15), c8 + np * 2 + (lane >> 4)));
+                mma_bf16(o[2 * np], qa, bh[0], bh[1]), mma_bf16(o[2 * np + 1], qa, bh[2], bh[3]);
+                mma_bf16(o[2 * np], qa, bl[0], bl[1]), mma_bf16(o[2 * np + 1], qa, bl[2], bl[3]);
+                if (FORGET) mma_bf16(o[2 * np], ql, bh[0], bh[1]), mma_bf16(o[2 * np + 1], ql, bh[2], bh[3]);
+            }
+            if (MLSTM && warp < 4) {
+                const float2 n0 = *reinterpret_cast<const float2*>(norm + ks * 16 + 2 * tig), n1 = *reinterpret_cast<const float2*>(norm + ks * 16 + 8 + 2 * tig);
 #pragma unroll
                 for (int h = 0; h < 2; h++) {
-                    const int r = (warp - 4 + 4 * m) * 16 + gid + 8 * h, c = col0 + n * 8 + 2 * tig;
-                    if (r < a.dim && c < vp) *reinterpret_cast<float2*>(dst + (int64_t)r * vp + c) = make_float2(s[m][n][2 * h], s[m][n][2 * h + 1]);
+                    const uint32_t x = qa[h], y = qa[2 + h];
+                    share[h] = fmaf(__uint_as_float(x << 16), n0.x, fmaf(__uint_as_float(x & 0xFFFF0000u), n0.y, share[h]));
+                    share[h] = fmaf(__uint_as_float(y << 16), n1.x, fmaf(__uint_as_float(y & 0xFFFF0000u), n1.y, share[h]));
                 }
-        if (MLSTM && blockIdx.x == 0)
-            for (int i = threadIdx.x - 128; i < a.dim; i += 128) a.state.norm[slot * a.dim + i] = norm[state_buf * DK + i];
+            }
+        }
+        if (!FORGET) {
+            const float f0 = ex2(ea[ta]), f1 = ex2(ea[tb]);
+#pragma unroll
+            for (int i = 0; i < NV; i++) o[i][0] *= f0, o[i][1] *= f0, o[i][2] *= f1, o[i][3] *= f1;
+            if (MLSTM && warp < 4) {
+#pragma unroll
+                for (int h = 0; h < 2; h++) {
+                    share[h] += __shfl_xor_sync(0xffffffffu, share[h], 1);
+                    share[h] += __shfl_xor_sync(0xffffffffu, share[h], 2);
+                }
+                if (tig == 0) nq[ta * 5 + 4] = share[0] * f0, nq[tb * 5 + 4] = share[1] * f1;
+            }
+        }
     }
-    if (MLSTM && blockIdx.x == 0 && threadIdx.x == 0) a.state.top[slot] = top;
+    // ---- queries against keys, weighted, to shared memory: ten tiles at and below the diagonal over eight warps.  rect: FORGET, every key before
+    // `from` for the queries at and after it.
+    auto products = [&](bool rect, int from) {
+        for (int t = warp; t < 10; t += 8) {
+            const int ti = t < 1 ? 0 : t < 3 ? 1 : t < 6 ? 2 : 3, j = t - ti * (ti + 1) / 2;
+            const int ra = ti * 16 + gid, rb = ra + 8;
+            float s0[2][4] = {};
+#pragma unroll 4
+            for (int kp = 0; kp < KS / 2; kp++) {
+                uint32_t q0[4], q1[4], l0[4], l1[4];
+                const int qr = ti * 16 + (lane & 15), qc = kp * 4 + (lane >> 4);
+                ldsm4(q0, base + M::Q + at<KB>(qr, qc));
+                ldsm4(q1, base + M::Q + at<KB>(qr, qc + 2));
+                if (FORGET) {
+                    ldsm4(l0, base + M::Q + M::KEY + at<KB>(qr, qc));
+                    ldsm4(l1, base + M::Q + M::KEY + at<KB>(qr, qc + 2));
+                }
+#pragma unroll
+                for (int i = 0; i < 2; i++) {
+                    uint32_t b[4], bl[4];
+                    const uint32_t off = at<KB>(j * 16 + i * 8 + (lane & 7), kp * 4 + (lane >> 3));
+                    ldsm4(b, base + M::K + off);
+                    mma_bf16(s0[i], q0, b[0], b[1]), mma_bf16(s0[i], q1, b[2], b[3]);
+                    if (FORGET) {
+                        ldsm4(bl, base + M::K + M::KEY + off);
+                        mma_bf16(s0[i], q0, bl[0], bl[1]), mma_bf16(s0[i], q1, bl[2], bl[3]);
+                        mma_bf16(s0[i], l0, b[0], b[1]), mma_bf16(s0[i], l1, b[2], b[3]);
+                    }
+                }
+            }
+            float sum[2] = {0.f, 0.f};
+#pragma unroll
+            for (int i = 0; i < 2; i++) {
+                const int c0 = j * 16 + i * 8 + 2 * tig;
+#pragma unroll
+                for (int x = 0; x < 4; x++) {
+                    const int c = c0 + (x & 1), r = x < 2 ? ra : rb;
+                    const bool seen = rect ? c < from && r >= from : c <= r;
+                    s0[i][x] = seen ? FORGET ? s0[i][x] : s0[i][x] * (ex2(ea[r] + eb[c]) * gain[c]) : 0.f;
+                }
+                sum[0] += s0[i][0] + s0[i][1], sum[1] += s0[i][2] + s0[i][3];
+                uint32_t h0, l0, h1, l1;
+                split(s0[i][0], s0[i][1], h0, l0);
+                split(s0[i][2], s0[i][3], h1, l1);
+                const uint32_t oa = at<C * 2>(ra, c0 >> 3) + (c0 & 7) * 2, ob = at<C * 2>(rb, c0 >> 3) + (c0 & 7) * 2;
+                *reinterpret_cast<uint32_t*>(smem + M::P + oa) = h0;
+                *reinterpret_cast<uint32_t*>(smem + M::P + M::PROD + oa) = l0;
+                *reinterpret_cast<uint32_t*>(smem + M::P + ob) = h1;
+                *reinterpret_cast<uint32_t*>(smem + M::P + M::PROD + ob) = l1;
+            }
+            if (MLSTM) {
+#pragma unroll
+                for (int h = 0; h < 2; h++) {
+                    sum[h] += __shfl_xor_sync(0xffffffffu, sum[h], 1);
+                    sum[h] += __shfl_xor_sync(0xffffffffu, sum[h], 2);
+                }
+                if (tig == 0) nq[ra * 5 + j] = sum[0], nq[rb * 5 + j] = sum[1];
+            }
+        }
+    };
+    auto times_values = [&]() {
+        for (int j = 0; j <= mt; j++) {
+            uint32_t ph[4], pl[4];
+            ldsm4(ph, base + M::P + at<C * 2>(mt * 16 + (lane & 15), j * 2 + (lane >> 4)));
+            ldsm4(pl, base + M::P + M::PROD + at<C * 2>(mt * 16 + (lane & 15), j * 2 + (lane >> 4)));
+#pragma unroll
+            for (int np = 0; np < NV / 2; np++) {
+                uint32_t b[4];
+                ldsm4_t(b, base + M::V + at<BV>(j * 16 + (lane & 15), c8 + np * 2 + (lane >> 4)));
+                mma_bf16(o[2 * np], ph, b[0], b[1]), mma_bf16(o[2 * np + 1], ph, b[2], b[3]);
+                mma_bf16(o[2 * np], pl, b[0], b[1]), mma_bf16(o[2 * np + 1], pl, b[2], b[3]);
+            }
+        }
+    };
+    if (!FORGET || !cuts) {
+        products(false, 0);
+        __syncthreads();
+        times_values();
+    } else {
+        for (int cut = 0; cut < n;) {
+            // where a component of E, counted from the cut, falls too low
+            __syncthreads();
+            float mine = 1.f;
+#pragma unroll
+            for (int i = 0; i < (FORGET ? TR : 0); i++)
+                if (part * TR + i >= cut) mine *= 1.f - kk[i];
+            fv[threadIdx.x] = mine;
+            if (threadIdx.x == 0) cut_end = n;
+            __syncthreads();
+            float e0 = 1.f;
+            for (int i = 0; i < part; i++) e0 *= fv[i * DK + ch];
+            float e = e0;
+            int low = n;
+#pragma unroll
+            for (int i = 0; i < (FORGET ? TR : 0); i++) {
+                const int r = part * TR + i;
+                if (r < cut || r >= n) continue;
+                e *= 1.f - kk[i];
+                if (e < E_MIN && r > cut && low == n) low = r;
+            }
+            if (low < n) atomicMin(&cut_end, low);
+            __syncthreads();
+            const int end = cut_end;
+            e = e0;
+#pragma unroll
+            for (int i = 0; i < (FORGET ? TR : 0); i++) {
+                const int r = part * TR + i;
+                const bool now = r >= cut && r < end;
+                if (now) e = fmaxf(e * (1.f - kk[i]), E_MIN);  // a cut's first row may fall further: nothing of the rows before is left then
+                const uint32_t off = at<KB>(r, ch >> 3) + (ch & 7) * 2;
+                put_split(smem + M::Q, smem + M::Q + M::KEY, off, now ? query(r) * e : 0.f);
+                put_split(smem + M::K, smem + M::K + M::KEY, off, now ? __fdividef(kk[i], e) : 0.f);
+            }
+            __syncthreads();
+            products(false, 0);
+            __syncthreads();
+            times_values();
+            if (cut > 0) {
+                // the rows before the cut: keys brought to it.  Products of f over the rows between
+                __syncthreads();
+                mine = 1.f;
+#pragma unroll
+                for (int i = 0; i < (FORGET ? TR : 0); i++)
+                    if (part * TR + i < cut) mine *= 1.f - kk[i];
+                fv[threadIdx.x] = mine;
+                __syncthreads();
+                e = 1.f;
+                for (int i = part + 1; i < RS; i++) e *= fv[i * DK + ch];
+#pragma unroll
+                for (int i = (FORGET ? TR : 0) - 1; i >= 0; i--) {
+                    const int r = part * TR + i;
+                    const bool old = r < cut;
+                    put_split(smem + M::K, smem + M::K + M::KEY, at<KB>(r, ch >> 3) + (ch & 7) * 2, old ? kk[i] * e : 0.f);
+                    if (old) e *= 1.f - kk[i];
+                }
+                __syncthreads();
+                products(true, cut);
+                __syncthreads();
+                times_values();
+            }
+            cut = end;
+        }
+    }
+    float f[2] = {a.q_scale, a.q_scale};
+    if (MLSTM) {
+#pragma unroll
+        for (int h = 0; h < 2; h++) {
+            const int t = h ? tb : ta;
+            float s = nq[t * 5 + 4];
+            for (int j = 0; j <= mt; j++) s += nq[t * 5 + j];
+            f[h] = a.q_scale / (fmaxf(fabsf(s * a.q_scale), floor_[t]) + 1e-6f);
+        }
+    }
+    const float skip = SSD ? a.skip[head] : 0.f;
+#pragma unroll
+    for (int h = 0; h < 2; h++) {
+        const int t = h ? tb : ta;
+        if (t >= n) continue;
+        float* dst = a.out + (int64_t)(row0 + t) * a.out_stride + (int64_t)head * a.vdim;
+#pragma unroll
+        for (int i = 0; i < NV; i++) {
+            const int c = col0 + (c8 + i) * 8 + 2 * tig;
+            float2 v = make_float2(o[i][2 * h] * f[h], o[i][2 * h + 1] * f[h]);
+            if (SSD) {
+                const uint32_t x = *reinterpret_cast<const uint32_t*>(smem + M::V + at<BV>(t, c8 + i) + tig * 4);
+                v.x = fmaf(skip, __uint_as_float(x << 16), v.x), v.y = fmaf(skip, __uint_as_float(x & 0xFFFF0000u), v.y);
+            }
+            if (c < a.vdim) *reinterpret_cast<float2*>(dst + c) = v;
+        }
+    }
 }
 
-template <int KIND, int DK, int VB>
-cudaError_t launch_chunks(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RowTiles& portions) {
-    constexpr size_t smem = Smem<KIND, DK, VB>::BYTES;
-    static_assert(smem <= 226 * 1024, "");
-    static SmemOptIn configured;
-    if (cudaError_t e = tsb_opt_in_smem(ctx, recurrence_chunks_kernel<KIND, DK, VB>, smem, configured); e != cudaSuccess) return e;
-    return tsb_launch(ctx, recurrence_chunks_kernel<KIND, DK, VB>, dim3((unsigned)((r.vdim + VB - 1) / VB), (unsigned)r.heads, (unsigned)portions.n), dim3(THREADS), smem,
-                      st, true, r, portions, ctx->dev_error);
+template <int KIND, int DK>
+cudaError_t launch_chunks(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RecurrenceChunks& c) {
+    constexpr size_t add_smem = AddSmem<KIND, DK>::BYTES, out_smem = OutSmem<KIND, DK>::BYTES;
+    static_assert(add_smem <= 226 * 1024 && out_smem <= 226 * 1024, "");
+    static SmemOptIn configured[2];
+    cudaError_t e = tsb_opt_in_smem(ctx, chunk_add_kernel<KIND, DK>, add_smem, configured[0]);
+    if (e == cudaSuccess) e = tsb_opt_in_smem(ctx, chunk_out_kernel<KIND, DK>, out_smem, configured[1]);
+    const Scratch s = scratch_of(r, c.scratch, c.chunks.n);
+    const dim3 grid((unsigned)((r.vdim + VB - 1) / VB), (unsigned)r.heads, (unsigned)c.chunks.n);
+    if (e == cudaSuccess) e = tsb_launch(ctx, chunk_add_kernel<KIND, DK>, grid, dim3(THREADS), add_smem, st, true, r, c.chunks, s, ctx->dev_error);
+    const int items = r.dim * r.vdim / 4 + (KIND == REC_MLSTM ? r.dim : 0);
+    if (e == cudaSuccess)
+        e = tsb_launch(ctx, chunk_walk_kernel<KIND>, dim3((unsigned)((items + THREADS - 1) / THREADS), (unsigned)r.heads, (unsigned)c.n_portions), dim3(THREADS), 0, st, true,
+                       r, c, s, ctx->dev_error);
+    if (e == cudaSuccess) e = tsb_launch(ctx, chunk_out_kernel<KIND, DK>, grid, dim3(THREADS), out_smem, st, true, r, c.chunks, s, ctx->dev_error);
+    return e;
 }
 template <int KIND>
-cudaError_t launch_chunks_dim(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RowTiles& portions) {
-    if (r.dim <= 64) return launch_chunks<KIND, 64, 32>(ctx, st, r, portions);
+cudaError_t launch_chunks_dim(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RecurrenceChunks& c) {
+    if (r.dim <= 64) return launch_chunks<KIND, 64>(ctx, st, r, c);
     if constexpr (KIND != REC_FORGET)
-        if (r.dim > 128) return launch_chunks<KIND, 256, 32>(ctx, st, r, portions);
-    return launch_chunks<KIND, 128, 32>(ctx, st, r, portions);
+        if (r.dim > 128) return launch_chunks<KIND, 256>(ctx, st, r, c);
+    return launch_chunks<KIND, 128>(ctx, st, r, c);
 }
 
 }  // namespace
 
 bool recurrence_chunks_supported(int kind, int dim, int vdim) { return dim <= (kind == REC_FORGET ? 128 : 256) && dim % 8 == 0 && vdim % 8 == 0; }
 
-cudaError_t launch_recurrence_chunks(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RowTiles& portions) {
-    if (portions.n == 0) return cudaSuccess;
+size_t recurrence_scratch_bytes(int kind, int heads, int dim, int vdim, int chunks) {
+    if (!recurrence_chunks_supported(kind, dim, vdim)) return 0;
+    const size_t n = (size_t)chunks * heads;
+    return align16(n * dim * vdim * 4) + align16(kind == REC_MLSTM ? n * dim * 4 : 0) + align16(n * decay_width(kind, dim) * 4) + n * 8;
+}
+
+cudaError_t launch_recurrence_chunks(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RecurrenceChunks& c) {
+    if (c.chunks.n == 0) return cudaSuccess;
     switch (r.kind) {
-        case REC_FORGET: return launch_chunks_dim<REC_FORGET>(ctx, st, r, portions);
-        case REC_MLSTM: return launch_chunks_dim<REC_MLSTM>(ctx, st, r, portions);
-        case REC_SSD: return launch_chunks_dim<REC_SSD>(ctx, st, r, portions);
+        case REC_FORGET: return launch_chunks_dim<REC_FORGET>(ctx, st, r, c);
+        case REC_MLSTM: return launch_chunks_dim<REC_MLSTM>(ctx, st, r, c);
+        case REC_SSD: return launch_chunks_dim<REC_SSD>(ctx, st, r, c);
         default: return cudaErrorInvalidValue;
     }
 }

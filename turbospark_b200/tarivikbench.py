@@ -56,17 +56,20 @@ def recurrence(ctx, peaks, kind, heads, dim, vdim, rows, streams, iters, groups=
     gate = ctx.to_device(np.random.default_rng(4).standard_normal(n * gates).astype(np.float32) + (3.0 if kind != REC_SSD else 0.0))
     lower, a_log, skip = _f32(ctx, heads * dim, 5, 0.0, 0.9), _f32(ctx, heads, 6), _f32(ctx, heads, 7)
     out, state = ctx.alloc(n * inner * 4), [ctx.zeroed(streams * 2 * state_bytes) for _ in range(copies if rows < 64 else 1)]
-    norm, top, rd = ctx.zeroed(streams * 2 * heads * dim * 4), ctx.zeroed(streams * 2 * heads * 8), _rows(ctx, 0 if rows >= 64 else 4096, rows, streams)
+    copies_ = (vdim + 31) // 32
+    norm, top, rd = ctx.zeroed(streams * 2 * heads * copies_ * dim * 4), ctx.zeroed(streams * 2 * heads * copies_ * 8), _rows(ctx, 0 if rows >= 64 else 4096, rows, streams)
+
+    scratch = ctx.recurrence_scratch(kind, heads, dim, vdim, n, rows) if rows >= 64 else ctx.zeroed(16)
 
     def call(i, s):
         at = i % copies
         r = capi.Recurrence(kind=kind, heads=heads, dim=dim, vdim=vdim, heads_per_key=heads // keys, cap=15.0, q_scale=dim ** -0.5 if kind == REC_MLSTM else 0.0,
                             q=q.ptr + at * n * kd * 2, k=k.ptr + at * n * kd * 2, v=v.ptr + at * n * inner * 2, q_stride=kd, k_stride=kd, v_stride=inner, gate=gate.ptr,
                             gate_stride=gates, lower=lower.ptr, a_log=a_log.ptr, skip=skip.ptr, out=out.ptr, out_stride=inner, state=state[i % len(state)].ptr,
-                            norm=norm.ptr, top=top.ptr, ring=2, n_streams=streams)
+                            norm=norm.ptr, top=top.ptr, ring=2, n_streams=streams, scratch=scratch.ptr)
         ctx.recurrence_rows(BF16, r, rd, n, rows, chunked=rows >= 64, stream=s)
     ms = time_graph(call, iters)
-    for b in [q, k, v, gate, lower, a_log, skip, out, norm, top, rd] + state:
+    for b in [q, k, v, gate, lower, a_log, skip, out, norm, top, rd, scratch] + state:
         b.free()
     vectors = (kd if kind == REC_FORGET else 2 * kd) + inner
     nbytes = streams * state_bytes * (2 if rows < 64 else 1) + n * (2 * vectors + 4 * gates + 4 * inner)
