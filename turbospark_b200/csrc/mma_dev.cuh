@@ -19,4 +19,8 @@ __device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool valid) 
     const int n = valid ? 16 : 0;
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
 }
+__device__ __forceinline__ void cp8(uint32_t dst, const void* src, bool valid) {
+    const int n = valid ? 8 : 0;
+    asm volatile("cp.async.ca.shared.global [%0], [%1], 8, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
+}
 }  // namespace

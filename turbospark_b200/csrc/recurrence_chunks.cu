@@ -3,7 +3,7 @@
 // With E_t the product of a chunk's decays up to row t and S the state before the chunk,
 //   o_t = E_t q_t . S + sum_{s <= t} (E_t / E_s) (q_t . k_s) v_s,    S' = E_T S + sum_s (E_T / E_s) k_s v_s^T.
 // Three launches: what every chunk adds to the state (all chunks at once), the states before the chunks (a walk over the chunks, element by
-// element), the outputs (all chunks at once).  A CTA of the first and the last has one chunk, one head and 64 value columns.
+// element), the outputs (all chunks at once).  A CTA of the first and the last has one chunk, one head and 64 or 128 value columns.
 //
 // What is f32 stays f32-like: an operand that is not a projection (state, weighted products, decayed queries, keys or values) goes into a
 // product as the sum of two bfloat16 numbers, which keeps 16 bits of it.
@@ -20,7 +20,7 @@
 
 namespace {
 
-constexpr int C = REC_CHUNK, THREADS = 256, VB = 64, BV = VB * 2;
+constexpr int C = REC_CHUNK, THREADS = 256;
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr float E_MIN = 8.2718061e-25f;  // 2^-80
 
@@ -134,19 +134,20 @@ __device__ __forceinline__ void put_split(uint8_t* hi, uint8_t* lo, uint32_t off
 }
 
 // ------------------------------------------------------------------ what a chunk adds to the state
-template <int KIND, int DK>
+template <int KIND, int DK, int VB>
 struct AddSmem {
     static constexpr bool FORGET = KIND == REC_FORGET;
-    static constexpr int KEY = C * DK * 2, VAL = C * VB * 2;
+    static constexpr int KEY = C * DK * 2, VAL = C * VB * 2;  // a tile of keys, of values
     static constexpr int K = 0, V = FORGET ? 2 * KEY : KEY, W = V + VAL;  // FORGET: keys, values; else keys, values, weighted values (high, low)
     static constexpr int Z = W, F = FORGET ? Z + C * DK * 4 : W + 2 * VAL;
     static constexpr int BYTES = F + (FORGET ? THREADS : C + 4) * 4;
 };
 
-template <int KIND, int DK>
+template <int KIND, int DK, int VB>
 __global__ void __launch_bounds__(THREADS)
     chunk_add_kernel(const __grid_constant__ Recurrence a, const __grid_constant__ RowTiles chunks, const __grid_constant__ Scratch out, uint32_t* __restrict__ err) {
-    using M = AddSmem<KIND, DK>;
+    using M = AddSmem<KIND, DK, VB>;
+    constexpr int BV = VB * 2;
     constexpr bool FORGET = KIND == REC_FORGET, MLSTM = KIND == REC_MLSTM;
     constexpr int KB = DK * 2, MT = DK / 16, SPLIT = MT < 8 ? 8 / MT : 1, MS = MT < 8 ? 1 : MT / 8, NV = VB / 8 / SPLIT;
     extern __shared__ __align__(128) uint8_t smem[];
@@ -294,7 +295,7 @@ __global__ void __launch_bounds__(THREADS)
     pdl_wait();
     pdl_launch_dependents();
     if (i4 >= state4 && !is_norm) return;
-    constexpr int AHEAD = 4;
+    constexpr int AHEAD = 8;
     const int width = FORGET ? a.dim : 2;
     float4 next[AHEAD];
     float2 gate[AHEAD];
@@ -343,20 +344,21 @@ __global__ void __launch_bounds__(THREADS)
 }
 
 // ------------------------------------------------------------------ outputs of a chunk
+constexpr int VB = 64, BV = VB * 2;  // value columns of a CTA
 template <int KIND, int DK>
 struct OutSmem {
     static constexpr bool FORGET = KIND == REC_FORGET;
     static constexpr int KEY = C * DK * 2, VAL = C * VB * 2, STATE = DK * VB * 2, PROD = C * C * 2;
-    // queries and keys (FORGET: high and low parts of each), values, state (high, low), products (high, low)
-    static constexpr int Q = 0, K = FORGET ? 2 * KEY : KEY, V = 2 * K, S = V + VAL, P = S + 2 * STATE;
-    static constexpr int F = P + 2 * PROD;
+    // queries and keys (FORGET: high and low parts of each), values, state (high, low), products (high, low; FORGET: where the keys were)
+    static constexpr int Q = 0, K = FORGET ? 2 * KEY : KEY, V = 2 * K, S = V + VAL, P = FORGET ? K : S + 2 * STATE;
+    static constexpr int F = FORGET ? S + 2 * STATE : P + 2 * PROD;
     static constexpr int Z = S;  // FORGET: the gates of the chunk, before the state takes their place
-    static_assert(!FORGET || C * DK * 4 <= 2 * STATE, "");
+    static_assert(!FORGET || (C * DK * 4 <= 2 * STATE && PROD <= KEY), "");
     static constexpr int BYTES = F + (FORGET ? THREADS : 4 * C + 8 + DK + 5 * C) * 4;
 };
 
 template <int KIND, int DK>
-__global__ void __launch_bounds__(THREADS, KIND == REC_FORGET || DK > 128 ? 1 : 2)
+__global__ void __launch_bounds__(THREADS, DK > 128 ? 1 : DK > 64 || KIND == REC_FORGET ? 2 : 3)
     chunk_out_kernel(const __grid_constant__ Recurrence a, const __grid_constant__ RowTiles chunks, const __grid_constant__ Scratch in, uint32_t* __restrict__ err) {
     using M = OutSmem<KIND, DK>;
     constexpr bool FORGET = KIND == REC_FORGET, MLSTM = KIND == REC_MLSTM, SSD = KIND == REC_SSD;
@@ -376,41 +378,30 @@ __global__ void __launch_bounds__(THREADS, KIND == REC_FORGET || DK > 128 ? 1 : 
     pdl_wait();
     pdl_launch_dependents();
     copy_tile<BV>(base + M::V, static_cast<const __nv_bfloat16*>(a.v) + (int64_t)row0 * a.v_stride + (int64_t)head * a.vdim + col0, a.v_stride, n, a.vdim - col0);
+    copy_tile<KB>(base + M::Q, gq, a.q_stride, n, a.dim);
     if (FORGET) {
         copy_gates<DK>(a, base + M::Z, row0, n, head);
     } else {
-        copy_tile<KB>(base + M::Q, gq, a.q_stride, n, a.dim);
         copy_tile<KB>(base + M::K, static_cast<const __nv_bfloat16*>(a.k) + (int64_t)row0 * a.k_stride + key_at, a.k_stride, n, a.dim);
     }
-    cp_async_commit();
     // the state: four numbers as four high and four low halves, to two tiles
-    constexpr int PIECES = DK * (VB / 4);
+    constexpr int PIECES = DK * (VB / 4), MINE = PIECES / THREADS;
     const float* src = in.add + slot * a.dim * a.vdim + col0;
-    auto state_piece = [&](int i, bool& ok) {
-        const int r = i / (VB / 4), c = i % (VB / 4);
-        ok = r < a.dim && col0 + c * 4 < a.vdim;
-        return ok ? *reinterpret_cast<const uint4*>(src + (int64_t)r * a.vdim + c * 4) : make_uint4(0, 0, 0, 0);
-    };
-    auto state_to_smem = [&](int i, const uint4& w) {
-        const int r = i / (VB / 4), c = i % (VB / 4);
-        const uint32_t off = at<BV>(r, c >> 1) + (c & 1) * 8;
-        *reinterpret_cast<uint2*>(smem + M::S + off) = make_uint2(w.x, w.y);
-        *reinterpret_cast<uint2*>(smem + M::S + M::STATE + off) = make_uint2(w.z, w.w);
-    };
-    auto load_state = [&]() {
-        for (int i0 = threadIdx.x; i0 < PIECES; i0 += 8 * THREADS) {
-            uint4 w[8];
-            bool ok;
+    uint4 held[FORGET ? MINE : 1];  // FORGET: their place is still taken
 #pragma unroll
-            for (int k = 0; k < 8; k++)
-                if (i0 + k * THREADS < PIECES) w[k] = state_piece(i0 + k * THREADS, ok);
-#pragma unroll
-            for (int k = 0; k < 8; k++)
-                if (i0 + k * THREADS < PIECES) state_to_smem(i0 + k * THREADS, w[k]);
+    for (int k = 0; k < MINE; k++) {
+        const int i = k * THREADS + threadIdx.x, r = i / (VB / 4), c = i % (VB / 4);
+        const bool ok = r < a.dim && col0 + c * 4 < a.vdim;
+        const float* p = ok ? src + (int64_t)r * a.vdim + c * 4 : in.add;
+        if (FORGET) {
+            held[FORGET ? k : 0] = ok ? *reinterpret_cast<const uint4*>(p) : make_uint4(0, 0, 0, 0);
+        } else {
+            const uint32_t off = base + M::S + at<BV>(r, c >> 1) + (c & 1) * 8;
+            cp8(off, p, ok), cp8(off + M::STATE, p + 2, ok);
         }
-    };
+    }
+    cp_async_commit();
     if (!FORGET) {
-        load_state();
         if (MLSTM)
             for (int i = threadIdx.x; i < DK; i += THREADS) norm[i] = i < a.dim ? in.norm[slot * a.dim + i] : 0.f;
         if (warp == 0) {
@@ -447,31 +438,33 @@ __global__ void __launch_bounds__(THREADS, KIND == REC_FORGET || DK > 128 ? 1 : 
 
     // ---- FORGET: queries times E_t, keys over E_s
     const int ch = FORGET ? threadIdx.x % DK : 0, part = FORGET ? threadIdx.x / DK : 0;
-    float kk[FORGET ? TR : 1];  // 1 - f of the thread's rows
-    auto query = [&](int r) {
-        const float x = r < n && ch < a.dim ? __bfloat162float(gq[r * a.q_stride + ch]) : 0.f;
-        return __fdividef(x, 1.f + __expf(-x));
-    };
     bool cuts = false;
-    float before = 1.f;  // E at the start of the thread's rows
     if (FORGET) {
         float* pre = reinterpret_cast<float*>(smem + M::Z);
         const float mine = forget_gates<DK>(a, pre, head, n);
         fv[threadIdx.x] = mine;
-#pragma unroll
-        for (int i = 0; i < (FORGET ? TR : 0); i++) kk[i] = pre[(part * TR + i) * DK + ch];
         __syncthreads();
-        for (int i = 0; i < part; i++) before *= fv[i * DK + ch];
-        cuts = __syncthreads_or(before * mine < E_MIN);  // E only falls
-        load_state();                                   // over the gates
-        float e = before;
-#pragma unroll
-        for (int i = 0; i < (FORGET ? TR : 0); i++) {
+        float e = 1.f;  // E at the start of the thread's rows
+        for (int i = 0; i < part; i++) e *= fv[i * DK + ch];
+        cuts = __syncthreads_or(e * mine < E_MIN);  // E only falls
+#pragma unroll 8
+        for (int i = 0; i < TR; i++) {
             const int r = part * TR + i;
-            e *= 1.f - kk[i];
+            const float k = pre[r * DK + ch];
+            e *= 1.f - k;
             const uint32_t off = at<KB>(r, ch >> 3) + (ch & 7) * 2;
-            put_split(smem + M::Q, smem + M::Q + M::KEY, off, query(r) * e);
-            put_split(smem + M::K, smem + M::K + M::KEY, off, cuts ? 0.f : __fdividef(kk[i], e));
+            const float x = __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(smem + M::Q + off));
+            put_split(smem + M::Q, smem + M::Q + M::KEY, off, __fdividef(x, 1.f + __expf(-x)) * e);
+            put_split(smem + M::K, smem + M::K + M::KEY, off, cuts ? 0.f : __fdividef(k, e));
+        }
+        __syncthreads();  // the gates have been read
+#pragma unroll
+        for (int k = 0; k < MINE; k++) {
+            const int i = k * THREADS + threadIdx.x, r = i / (VB / 4), c = i % (VB / 4);
+            const uint32_t off = at<BV>(r, c >> 1) + (c & 1) * 8;
+            const uint4 w = held[FORGET ? k : 0];
+            *reinterpret_cast<uint2*>(smem + M::S + off) = make_uint2(w.x, w.y);
+            *reinterpret_cast<uint2*>(smem + M::S + M::STATE + off) = make_uint2(w.z, w.w);
         }
         __syncthreads();
     }
@@ -522,8 +515,22 @@ __global__ void __launch_bounds__(THREADS, KIND == REC_FORGET || DK > 128 ? 1 : 
     }
     // ---- queries against keys, weighted, to shared memory: ten tiles at and below the diagonal over eight warps.  rect: FORGET, every key before
     // `from` for the queries at and after it.
+    auto store_products = [&](int ra, int c0, const float (&p)[4]) {
+        uint32_t h0, l0, h1, l1;
+        split(p[0], p[1], h0, l0);
+        split(p[2], p[3], h1, l1);
+        const uint32_t oa = at<C * 2>(ra, c0 >> 3) + (c0 & 7) * 2, ob = at<C * 2>(ra + 8, c0 >> 3) + (c0 & 7) * 2;
+        *reinterpret_cast<uint32_t*>(smem + M::P + oa) = h0;
+        *reinterpret_cast<uint32_t*>(smem + M::P + M::PROD + oa) = l0;
+        *reinterpret_cast<uint32_t*>(smem + M::P + ob) = h1;
+        *reinterpret_cast<uint32_t*>(smem + M::P + M::PROD + ob) = l1;
+    };
     auto products = [&](bool rect, int from) {
-        for (int t = warp; t < 10; t += 8) {
+        float held_p[2][2][4];  // FORGET: a warp's tiles wait until every warp has read the keys
+#pragma unroll
+        for (int u = 0; u < 2; u++) {
+            const int t = warp + 8 * u;
+            if (t >= 10) break;
             const int ti = t < 1 ? 0 : t < 3 ? 1 : t < 6 ? 2 : 3, j = t - ti * (ti + 1) / 2;
             const int ra = ti * 16 + gid, rb = ra + 8;
             float s0[2][4] = {};
@@ -559,16 +566,10 @@ __global__ void __launch_bounds__(THREADS, KIND == REC_FORGET || DK > 128 ? 1 : 
                     const int c = c0 + (x & 1), r = x < 2 ? ra : rb;
                     const bool seen = rect ? c < from && r >= from : c <= r;
                     s0[i][x] = seen ? FORGET ? s0[i][x] : s0[i][x] * (ex2(ea[r] + eb[c]) * gain[c]) : 0.f;
+                    held_p[u][i][x] = s0[i][x];
                 }
                 sum[0] += s0[i][0] + s0[i][1], sum[1] += s0[i][2] + s0[i][3];
-                uint32_t h0, l0, h1, l1;
-                split(s0[i][0], s0[i][1], h0, l0);
-                split(s0[i][2], s0[i][3], h1, l1);
-                const uint32_t oa = at<C * 2>(ra, c0 >> 3) + (c0 & 7) * 2, ob = at<C * 2>(rb, c0 >> 3) + (c0 & 7) * 2;
-                *reinterpret_cast<uint32_t*>(smem + M::P + oa) = h0;
-                *reinterpret_cast<uint32_t*>(smem + M::P + M::PROD + oa) = l0;
-                *reinterpret_cast<uint32_t*>(smem + M::P + ob) = h1;
-                *reinterpret_cast<uint32_t*>(smem + M::P + M::PROD + ob) = l1;
+                if (!FORGET) store_products(ra, c0, s0[i]);
             }
             if (MLSTM) {
 #pragma unroll
@@ -577,6 +578,17 @@ __global__ void __launch_bounds__(THREADS, KIND == REC_FORGET || DK > 128 ? 1 : 
                     sum[h] += __shfl_xor_sync(0xffffffffu, sum[h], 2);
                 }
                 if (tig == 0) nq[ra * 5 + j] = sum[0], nq[rb * 5 + j] = sum[1];
+            }
+        }
+        if (FORGET) {
+            __syncthreads();
+#pragma unroll
+            for (int u = 0; u < 2; u++) {
+                const int t = warp + 8 * u;
+                if (t >= 10) break;
+                const int ti = t < 1 ? 0 : t < 3 ? 1 : t < 6 ? 2 : 3, j = t - ti * (ti + 1) / 2;
+#pragma unroll
+                for (int i = 0; i < 2; i++) store_products(ti * 16 + gid, j * 16 + i * 8 + 2 * tig, held_p[u][i]);
             }
         }
     };
@@ -599,61 +611,64 @@ __global__ void __launch_bounds__(THREADS, KIND == REC_FORGET || DK > 128 ? 1 : 
         __syncthreads();
         times_values();
     } else {
+        // the chunk is cut: gates and queries come from memory again
+        const float low_bound = ch < a.dim ? a.lower[(int64_t)head * a.dim + ch] : 1.f;
+        auto one_minus_f = [&](int r) {
+            if (r >= n || ch >= a.dim) return 0.f;
+            const float x = a.gate[(int64_t)(row0 + r) * a.gate_stride + (int64_t)head * a.dim + ch], e = __expf(-fabsf(x)), d = __fdividef(1.f, 1.f + e);
+            return (1.f - low_bound) * (x >= 0.f ? e * d : d);
+        };
+        auto query = [&](int r) {
+            const float x = r < n && ch < a.dim ? __bfloat162float(gq[r * a.q_stride + ch]) : 0.f;
+            return __fdividef(x, 1.f + __expf(-x));
+        };
         for (int cut = 0; cut < n;) {
             // where a component of E, counted from the cut, falls too low
             __syncthreads();
             float mine = 1.f;
-#pragma unroll
-            for (int i = 0; i < (FORGET ? TR : 0); i++)
-                if (part * TR + i >= cut) mine *= 1.f - kk[i];
+            for (int r = max(cut, part * TR); r < (part + 1) * TR; r++) mine *= 1.f - one_minus_f(r);
             fv[threadIdx.x] = mine;
             if (threadIdx.x == 0) cut_end = n;
             __syncthreads();
             float e0 = 1.f;
             for (int i = 0; i < part; i++) e0 *= fv[i * DK + ch];
             float e = e0;
-            int low = n;
-#pragma unroll
-            for (int i = 0; i < (FORGET ? TR : 0); i++) {
-                const int r = part * TR + i;
-                if (r < cut || r >= n) continue;
-                e *= 1.f - kk[i];
-                if (e < E_MIN && r > cut && low == n) low = r;
+            for (int r = max(cut, part * TR); r < min(n, (part + 1) * TR); r++) {
+                e *= 1.f - one_minus_f(r);
+                if (e < E_MIN && r > cut) {
+                    atomicMin(&cut_end, r);
+                    break;
+                }
             }
-            if (low < n) atomicMin(&cut_end, low);
             __syncthreads();
             const int end = cut_end;
             e = e0;
-#pragma unroll
-            for (int i = 0; i < (FORGET ? TR : 0); i++) {
-                const int r = part * TR + i;
+            for (int r = part * TR; r < (part + 1) * TR; r++) {
                 const bool now = r >= cut && r < end;
-                if (now) e = fmaxf(e * (1.f - kk[i]), E_MIN);  // a cut's first row may fall further: nothing of the rows before is left then
+                const float k = one_minus_f(r);
+                if (now) e = fmaxf(e * (1.f - k), E_MIN);  // a cut's first row may fall further: nothing of the rows before is left then
                 const uint32_t off = at<KB>(r, ch >> 3) + (ch & 7) * 2;
                 put_split(smem + M::Q, smem + M::Q + M::KEY, off, now ? query(r) * e : 0.f);
-                put_split(smem + M::K, smem + M::K + M::KEY, off, now ? __fdividef(kk[i], e) : 0.f);
+                put_split(smem + M::K, smem + M::K + M::KEY, off, now ? __fdividef(k, e) : 0.f);
             }
             __syncthreads();
             products(false, 0);
             __syncthreads();
             times_values();
             if (cut > 0) {
-                // the rows before the cut: keys brought to it.  Products of f over the rows between
+                // the rows before the cut: keys brought to it, times the f of the rows between
                 __syncthreads();
                 mine = 1.f;
-#pragma unroll
-                for (int i = 0; i < (FORGET ? TR : 0); i++)
-                    if (part * TR + i < cut) mine *= 1.f - kk[i];
+                for (int r = part * TR; r < min(cut, (part + 1) * TR); r++) mine *= 1.f - one_minus_f(r);
                 fv[threadIdx.x] = mine;
                 __syncthreads();
                 e = 1.f;
                 for (int i = part + 1; i < RS; i++) e *= fv[i * DK + ch];
-#pragma unroll
-                for (int i = (FORGET ? TR : 0) - 1; i >= 0; i--) {
-                    const int r = part * TR + i;
+                for (int r = (part + 1) * TR - 1; r >= part * TR; r--) {
                     const bool old = r < cut;
-                    put_split(smem + M::K, smem + M::K + M::KEY, at<KB>(r, ch >> 3) + (ch & 7) * 2, old ? kk[i] * e : 0.f);
-                    if (old) e *= 1.f - kk[i];
+                    const float k = one_minus_f(r);
+                    put_split(smem + M::K, smem + M::K + M::KEY, at<KB>(r, ch >> 3) + (ch & 7) * 2, old ? k * e : 0.f);
+                    if (old) e *= 1.f - k;
                 }
                 __syncthreads();
                 products(true, cut);
@@ -692,16 +707,23 @@ __global__ void __launch_bounds__(THREADS, KIND == REC_FORGET || DK > 128 ? 1 : 
     }
 }
 
+template <int KIND, int DK, int COLS>
+cudaError_t launch_add(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RecurrenceChunks& c, const Scratch& s) {
+    constexpr size_t smem = AddSmem<KIND, DK, COLS>::BYTES;
+    static_assert(smem <= 226 * 1024 && OutSmem<KIND, DK>::BYTES <= 226 * 1024, "");
+    static SmemOptIn configured;
+    if (cudaError_t e = tsb_opt_in_smem(ctx, chunk_add_kernel<KIND, DK, COLS>, smem, configured); e != cudaSuccess) return e;
+    return tsb_launch(ctx, chunk_add_kernel<KIND, DK, COLS>, dim3((unsigned)((r.vdim + COLS - 1) / COLS), (unsigned)r.heads, (unsigned)c.chunks.n), dim3(THREADS), smem, st,
+                      true, r, c.chunks, s, ctx->dev_error);
+}
 template <int KIND, int DK>
 cudaError_t launch_chunks(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RecurrenceChunks& c) {
-    constexpr size_t add_smem = AddSmem<KIND, DK>::BYTES, out_smem = OutSmem<KIND, DK>::BYTES;
-    static_assert(add_smem <= 226 * 1024 && out_smem <= 226 * 1024, "");
-    static SmemOptIn configured[2];
-    cudaError_t e = tsb_opt_in_smem(ctx, chunk_add_kernel<KIND, DK>, add_smem, configured[0]);
-    if (e == cudaSuccess) e = tsb_opt_in_smem(ctx, chunk_out_kernel<KIND, DK>, out_smem, configured[1]);
+    constexpr size_t out_smem = OutSmem<KIND, DK>::BYTES;
+    static SmemOptIn configured;
     const Scratch s = scratch_of(r, c.scratch, c.chunks.n);
+    cudaError_t e = r.vdim > 64 ? launch_add<KIND, DK, 128>(ctx, st, r, c, s) : launch_add<KIND, DK, 64>(ctx, st, r, c, s);
+    if (e == cudaSuccess) e = tsb_opt_in_smem(ctx, chunk_out_kernel<KIND, DK>, out_smem, configured);
     const dim3 grid((unsigned)((r.vdim + VB - 1) / VB), (unsigned)r.heads, (unsigned)c.chunks.n);
-    if (e == cudaSuccess) e = tsb_launch(ctx, chunk_add_kernel<KIND, DK>, grid, dim3(THREADS), add_smem, st, true, r, c.chunks, s, ctx->dev_error);
     const int items = r.dim * r.vdim / 4 + (KIND == REC_MLSTM ? r.dim : 0);
     if (e == cudaSuccess)
         e = tsb_launch(ctx, chunk_walk_kernel<KIND>, dim3((unsigned)((items + THREADS - 1) / THREADS), (unsigned)r.heads, (unsigned)c.n_portions), dim3(THREADS), 0, st, true,
