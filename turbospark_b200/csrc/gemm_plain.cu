@@ -549,7 +549,9 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
             }
             const int tiles = tile0[lo + 1] - tile0[lo], j = i - tile0[lo] * n_row_tiles;
             it.tok = j % tiles, it.row = j / tiles, it.run = 0, it.u0 = 0, it.n = units;
-            it.tok0 = slot0[lo] + it.tok * nt, it.n_tok = min(nt, slot0[lo + 1] - it.tok0);
+            // the expert's slots over its tiles, evenly
+            const int n = slot0[lo + 1] - slot0[lo], width = ((n + tiles - 1) / tiles + 15) & ~15;
+            it.tok0 = slot0[lo] + min(n, it.tok * width), it.n_tok = min(width, slot0[lo + 1] - it.tok0);
             it.wrow = (lo * n_row_tiles + it.row) * TCG_M;
             return it;
         }
@@ -614,8 +616,8 @@ __global__ void __launch_bounds__(TCG_THREADS, 1)
             if (!ok) break;
             tc_fence_after();
             const uint32_t d = tmem + buf * (uint32_t)nt;
-            // an expert's last tile multiplies only the tokens it has
-            const uint32_t idesc = EXPERTS ? idesc_of((w.n_tok + 15) & ~15) : idesc_of(nt);
+            // an expert's tile multiplies only the tokens it has
+            const uint32_t idesc = EXPERTS ? idesc_of(max(16, (w.n_tok + 15) & ~15)) : idesc_of(nt);
             for (int u = 0; u < w.n; u++, it++) {
                 const int s = it % stages;
                 ok = __all_sync(0xffffffffu, mbar_wait(&bars->full[s], (it / stages) & 1, err));

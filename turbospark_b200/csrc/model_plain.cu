@@ -813,7 +813,7 @@ struct Forward {
             v.taps = 0, v.out = nullptr;
             return end(v, nullptr, RowRing());
         };
-        cudaError_t e = plan.use_before ? launch_rings_before(ctx, st, b->states.rings_dev, b->states.n_rings, p.rows_dev, p.rows) : cudaSuccess;
+        cudaError_t e = plan.use_before ? launch_rings_before(ctx, st, b->states.rings_dev, b->states.n_rings, p.rows_dev, plan.portions) : cudaSuccess;
         if (e != cudaSuccess) return e;
         SublayerEnd t = s;
         t.table = m->embed, t.positions = m->positions, t.n_positions = m->cfg.positions, t.tokens = p.tokens, t.token_stride = p.token_stride, t.vocab = m->cfg.vocab;

@@ -11,8 +11,8 @@
 // Decay per head (REC_MLSTM, REC_SSD): E is a number per row; the ratios are exponentials of differences of its logarithm, applied to the
 // products of plain queries and keys, and to the values on their way into the state.
 // Decay per row of the state (REC_FORGET): E is a vector.  Into the state go keys times E_T / E_s, a product over the rows behind s; queries take
-// E_t, keys 1 / E_s.  1 / E grows, so where a component of E falls below 2^-80 the chunk is cut: rows behind a cut meet each other with E
-// counted from the cut, and the rows before it with keys brought to the cut.
+// E_t, keys 1 / E_s, both shifted by 2^60 to use the whole range of exponents.  1 / E grows, so where a component of E falls below 2^-140
+// the chunk is cut: rows behind a cut meet each other with E counted from the cut, and the rows before it with keys brought to the cut.
 #include <algorithm>
 
 #include "mma_dev.cuh"
@@ -22,7 +22,7 @@ namespace {
 
 constexpr int C = REC_CHUNK, THREADS = 256;
 constexpr float LOG2E = 1.4426950408889634f;
-constexpr float E_MIN = 8.2718061e-25f;  // 2^-80
+constexpr float E_ONE = 1152921504606846976.f, E_MIN = 8.2718061e-25f;  // 2^60 stands for E = 1, 2^-80 for the least E
 
 __device__ __forceinline__ float ex2(float x) {
     float y;
@@ -444,7 +444,7 @@ __global__ void __launch_bounds__(THREADS, DK > 128 ? 1 : DK > 64 || KIND == REC
         const float mine = forget_gates<DK>(a, pre, head, n);
         fv[threadIdx.x] = mine;
         __syncthreads();
-        float e = 1.f;  // E at the start of the thread's rows
+        float e = E_ONE;  // E at the start of the thread's rows
         for (int i = 0; i < part; i++) e *= fv[i * DK + ch];
         cuts = __syncthreads_or(e * mine < E_MIN);  // E only falls
 #pragma unroll 8
@@ -499,7 +499,12 @@ __global__ void __launch_bounds__(THREADS, DK > 128 ? 1 : DK > 64 || KIND == REC
                 }
             }
         }
-        if (!FORGET) {
+        if (FORGET) {
+#pragma unroll
+            for (int i = 0; i < NV; i++)
+#pragma unroll
+                for (int j = 0; j < 4; j++) o[i][j] *= 1.f / E_ONE;
+        } else {
             const float f0 = ex2(ea[ta]), f1 = ex2(ea[tb]);
 #pragma unroll
             for (int i = 0; i < NV; i++) o[i][0] *= f0, o[i][1] *= f0, o[i][2] *= f1, o[i][3] *= f1;
@@ -630,7 +635,7 @@ __global__ void __launch_bounds__(THREADS, DK > 128 ? 1 : DK > 64 || KIND == REC
             fv[threadIdx.x] = mine;
             if (threadIdx.x == 0) cut_end = n;
             __syncthreads();
-            float e0 = 1.f;
+            float e0 = E_ONE;
             for (int i = 0; i < part; i++) e0 *= fv[i * DK + ch];
             float e = e0;
             for (int r = max(cut, part * TR); r < min(n, (part + 1) * TR); r++) {
@@ -667,7 +672,7 @@ __global__ void __launch_bounds__(THREADS, DK > 128 ? 1 : DK > 64 || KIND == REC
                 for (int r = (part + 1) * TR - 1; r >= part * TR; r--) {
                     const bool old = r < cut;
                     const float k = one_minus_f(r);
-                    put_split(smem + M::K, smem + M::K + M::KEY, at<KB>(r, ch >> 3) + (ch & 7) * 2, old ? k * e : 0.f);
+                    put_split(smem + M::K, smem + M::K + M::KEY, at<KB>(r, ch >> 3) + (ch & 7) * 2, old ? k * e * (1.f / E_ONE) : 0.f);
                     if (old) e *= 1.f - k;
                 }
                 __syncthreads();

@@ -1,6 +1,9 @@
 // Row operators around the sublayers of output-norm layers (sublayer.cuh).
 #include <cuda_bf16.h>
 
+#include <algorithm>
+#include <type_traits>
+
 #include "sublayer.cuh"
 
 namespace {
@@ -51,14 +54,15 @@ __device__ __forceinline__ float silu(float z) {
     return sizeof(T) == 4 ? z * sigmoid(z) : __fdividef(z, 1.f + __expf(-z));
 }
 
-// 1 / rms of the group that column c belongs to, from the columns' squares.  A thread holds columns (k * THREADS + thread) * W + i, k < V.
+// 1 / rms of the group that column c belongs to, from the columns' squares.  One of NT threads holds columns (k * NT + thread) * W + i, k < V.
 // FAST: groups are multiples of 32 W columns, so a warp's columns of one k share a group and the whole reduction takes one barrier.
 // sq: shared memory, two of them used in turn (call with parity 0, 1, 0, ...).
-template <int V, int W, bool FAST>
+template <int NT, int V, int W, bool FAST>
 struct GroupNorm {
+    static constexpr int NW = NT / 32;
     int d, width, groups;
     float eps;
-    float *sq, *sums;  // FAST: [2][V * WARPS]; else sq [d / W], sums [groups]
+    float *sq, *sums;  // FAST: [2][V * NW]; else sq [d / W], sums [groups]
     __device__ __forceinline__ void rms(const Vec<W> (&x)[V], int parity, float (&inv)[V]) const {
         float s[V];
 #pragma unroll
@@ -69,31 +73,31 @@ struct GroupNorm {
         }
         const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
         if (FAST) {
-            float* red = sq + parity * V * WARPS;
+            float* red = sq + parity * V * NW;
 #pragma unroll
             for (int k = 0; k < V; k++) {
                 const float t = warp_sum(s[k]);
-                if (lane == 0) red[k * WARPS + warp] = t;
+                if (lane == 0) red[k * NW + warp] = t;
             }
             __syncthreads();
             const int per = width / (32 * W);  // warp runs per group
 #pragma unroll
             for (int k = 0; k < V; k++) {
-                const int g = (k * WARPS + warp) / per;
+                const int g = (k * NW + warp) / per;
                 float t = 0.f;
-                if ((k * THREADS + (int)threadIdx.x) * W < d)
+                if ((k * NT + (int)threadIdx.x) * W < d)
                     for (int i = 0; i < per; i++) t += red[g * per + i];
                 inv[k] = 1.f / sqrtf(t / (float)width + eps);
             }
         } else {
 #pragma unroll
             for (int k = 0; k < V; k++) {
-                const int u = k * THREADS + threadIdx.x;
+                const int u = k * NT + threadIdx.x;
                 if (u * W < d) sq[u] = s[k];
             }
             __syncthreads();
             const int per = width / W;
-            for (int g = warp; g < groups; g += WARPS) {
+            for (int g = warp; g < groups; g += NW) {
                 float t = 0.f;
                 for (int i = lane; i < per; i += 32) t += sq[g * per + i];
                 t = warp_sum(t);
@@ -102,37 +106,45 @@ struct GroupNorm {
             __syncthreads();
 #pragma unroll
             for (int k = 0; k < V; k++) {
-                const int c = (k * THREADS + threadIdx.x) * W;
+                const int c = (k * NT + threadIdx.x) * W;
                 inv[k] = c < d ? sums[c / width] : 0.f;
             }
             // the next call's first barrier separates its writes of sums from these reads; sq is rewritten only behind the second one above
         }
     }
 };
-template <int V, int W>
+template <int NT, int V, int W>
 size_t group_norm_smem(int d, int groups, bool fast) {
-    return (fast ? (size_t)2 * V * WARPS : (size_t)(d / W + groups)) * sizeof(float);
+    return (fast ? (size_t)2 * V * (NT / 32) : (size_t)(d / W + groups)) * sizeof(float);
 }
 
 // ------------------------------------------------------------------ end of a sublayer
 enum SublayerSource { FROM_Y, FROM_EXPERTS, FROM_TABLE };
 
-template <typename T, int V, int W, bool FAST, int TM>
-__global__ void __launch_bounds__(THREADS) sublayer_end_kernel(const __grid_constant__ SublayerEnd s, uint32_t* __restrict__ err) {
+template <typename T, int NT, int V, int W, bool FAST, int TM>
+__global__ void __launch_bounds__(NT) sublayer_end_kernel(const __grid_constant__ SublayerEnd s, uint32_t* __restrict__ err) {
     extern __shared__ float smem[];
     const AttnTile tile = row_tile(s.tiles, blockIdx.x);
     const tsb_row_desc rd = s.rows[tile.row_first];
     const int d = s.d, halo = s.taps > 0 ? min(s.taps - 1, rd.slot) : 0;
     const bool ok = s.taps == 0 || (rd.seq >= 0 && rd.seq < s.ring.n_streams);
-    GroupNorm<V, W, FAST> norm;
+    GroupNorm<NT, V, W, FAST> norm;
     norm.d = d, norm.groups = s.groups, norm.width = d / s.groups, norm.eps = s.eps, norm.sq = smem, norm.sums = smem + d / W;
-    Vec<W> hist[TM - 1][V];  // hist[j]: the row j + 1 before the current one
+    Vec<W> hist[TM > 1 ? TM - 1 : 1][V];  // hist[j]: the row j + 1 before the current one
     Vec<W> w[V];
 #pragma unroll
     for (int k = 0; k < V; k++) {
-        const int c = (k * THREADS + threadIdx.x) * W;
+        const int c = (k * NT + threadIdx.x) * W;
         w[k] = c < d && s.norm_w ? load(s.norm_w + c, Vec<W>()) : zeros<W>();
     }
+    Vec<W> taps[TM][V];  // taps[j]: of the row j before
+#pragma unroll
+    for (int j = 0; j < TM; j++)
+#pragma unroll
+        for (int k = 0; k < V; k++) {
+            const int c = (k * NT + threadIdx.x) * W;
+            taps[j][k] = j < s.taps && c < d ? load(s.taps_w + (int64_t)(s.taps - 1 - j) * d + c, Vec<W>()) : zeros<W>();
+        }
     pdl_wait();
     pdl_launch_dependents();
     if (!ok) {
@@ -147,7 +159,7 @@ __global__ void __launch_bounds__(THREADS) sublayer_end_kernel(const __grid_cons
         const float* p = in ? ring_row_before(s.ring, rd.seq, rd.base, pos, s.use_before) : nullptr;
 #pragma unroll
         for (int k = 0; k < V; k++) {
-            const int c = (k * THREADS + threadIdx.x) * W;
+            const int c = (k * NT + threadIdx.x) * W;
             hist[j][k] = in && c < d ? load(p + c, Vec<W>()) : zeros<W>();
         }
     }
@@ -156,22 +168,33 @@ __global__ void __launch_bounds__(THREADS) sublayer_end_kernel(const __grid_cons
     auto fetch = [&](int r) {
 #pragma unroll
         for (int k = 0; k < V; k++) {
-            const int c = (k * THREADS + threadIdx.x) * W;
+            const int c = (k * NT + threadIdx.x) * W;
             x_next[k] = c < d ? load(s.x_in + (int64_t)r * d + c, Vec<W>()) : zeros<W>();
             y_next[k] = s.y && c < d ? load(s.y + (int64_t)r * d + c, Vec<W>()) : zeros<W>();
         }
         if (s.y) return;
-        for (int e = 0; e < s.top; e++) {
-            const float f = s.weight[(int64_t)r * s.top + e];
-            const T* row = static_cast<const T*>(s.experts) + (int64_t)s.slot_of[(int64_t)r * s.top + e] * s.expert_stride;
+        constexpr int AT_ONCE = V * W <= 8 ? 4 : 2;  // expert rows in flight
+        for (int e0 = 0; e0 < s.top; e0 += AT_ONCE) {
+            float f[AT_ONCE];
+            Vec<W> v[AT_ONCE][V];
 #pragma unroll
-            for (int k = 0; k < V; k++) {
-                const int c = (k * THREADS + threadIdx.x) * W;
-                if (c >= d) continue;
-                const Vec<W> v = load(row + c, Vec<W>());
+            for (int e = 0; e < AT_ONCE; e++) {
+                const int64_t at = (int64_t)r * s.top + e0 + e;
+                const bool in = e0 + e < s.top;
+                f[e] = in ? s.weight[at] : 0.f;
+                const T* row = static_cast<const T*>(s.experts) + (int64_t)(in ? s.slot_of[at] : 0) * s.expert_stride;
 #pragma unroll
-                for (int i = 0; i < W; i++) y_next[k].v[i] = fmaf(f, v.v[i], y_next[k].v[i]);
+                for (int k = 0; k < V; k++) {
+                    const int c = (k * NT + threadIdx.x) * W;
+                    v[e][k] = in && c < d ? load(row + c, Vec<W>()) : zeros<W>();
+                }
             }
+#pragma unroll
+            for (int e = 0; e < AT_ONCE; e++)
+#pragma unroll
+                for (int k = 0; k < V; k++)
+#pragma unroll
+                    for (int i = 0; i < W; i++) y_next[k].v[i] = fmaf(f[e], v[e][k].v[i], y_next[k].v[i]);
         }
     };
     const int last = tile.row_first + tile.n_rows - 1;
@@ -185,7 +208,7 @@ __global__ void __launch_bounds__(THREADS) sublayer_end_kernel(const __grid_cons
             if (bad && threadIdx.x == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
 #pragma unroll
             for (int k = 0; k < V; k++) {
-                const int c = (k * THREADS + threadIdx.x) * W;
+                const int c = (k * NT + threadIdx.x) * W;
                 x[k] = zeros<W>();
                 if (bad || c >= d) continue;
                 x[k] = load(static_cast<const T*>(s.table) + (int64_t)tok * d + c, Vec<W>());
@@ -210,21 +233,17 @@ __global__ void __launch_bounds__(THREADS) sublayer_end_kernel(const __grid_cons
             if (any_kept && ring_keeps(s.ring, s.rows, s.n_rows, r, rd.seq)) keep = ring_row(s.ring, rd.seq, pos_first + (r - first));
 #pragma unroll
             for (int k = 0; k < V; k++) {
-                const int c = (k * THREADS + threadIdx.x) * W;
+                const int c = (k * NT + threadIdx.x) * W;
                 if (c >= d) continue;
                 store(s.x_out + (int64_t)r * d + c, x[k]);
                 if (s.taps == 0) continue;
                 if (keep) store(keep + c, x[k]);
-                Vec<W> o = x[k];
-                const Vec<W> t0 = load(s.taps_w + (int64_t)(s.taps - 1) * d + c, Vec<W>());
+                Vec<W> o;
 #pragma unroll
-                for (int i = 0; i < W; i++) o.v[i] = fmaf(t0.v[i], x[k].v[i], o.v[i]);
+                for (int i = 0; i < W; i++) {
+                    o.v[i] = fmaf(taps[0][k].v[i], x[k].v[i], x[k].v[i]);
 #pragma unroll
-                for (int j = 0; j < TM - 1; j++) {
-                    if (j >= s.taps - 1) break;
-                    const Vec<W> t = load(s.taps_w + (int64_t)(s.taps - 2 - j) * d + c, Vec<W>());
-#pragma unroll
-                    for (int i = 0; i < W; i++) o.v[i] = fmaf(t.v[i], hist[j][k].v[i], o.v[i]);
+                    for (int j = 0; j < TM - 1; j++) o.v[i] = fmaf(taps[j + 1][k].v[i], hist[j][k].v[i], o.v[i]);
                 }
                 store(static_cast<T*>(s.out) + (int64_t)r * s.out_stride + c, o);
             }
@@ -233,15 +252,18 @@ __global__ void __launch_bounds__(THREADS) sublayer_end_kernel(const __grid_cons
         for (int j = TM - 2; j > 0; j--)
 #pragma unroll
             for (int k = 0; k < V; k++) hist[j][k] = hist[j - 1][k];
+        if (TM > 1) {
 #pragma unroll
-        for (int k = 0; k < V; k++) hist[0][k] = x[k];
+            for (int k = 0; k < V; k++) hist[0][k] = x[k];
+        }
     }
 }
 
-__global__ void __launch_bounds__(THREADS) rings_before_kernel(const RowRing* __restrict__ rings, const tsb_row_desc* __restrict__ rows) {
+__global__ void __launch_bounds__(THREADS)
+    rings_before_kernel(const RowRing* __restrict__ rings, const tsb_row_desc* __restrict__ rows, const __grid_constant__ RowTiles portions) {
     pdl_wait();
     pdl_launch_dependents();
-    const tsb_row_desc rd = rows[blockIdx.x];
+    const tsb_row_desc rd = rows[row_tile(portions, blockIdx.x).row_first];
     const RowRing r = rings[blockIdx.y];
     if (rd.slot != 0 || rd.seq < 0 || rd.seq >= r.n_streams) return;
     for (int k = 0; k < r.keep; k++) {
@@ -261,7 +283,7 @@ __global__ void __launch_bounds__(THREADS)
     pdl_wait();
     pdl_launch_dependents();
     const int r = want ? want[blockIdx.x] : (int)blockIdx.x * want_step + want_first;
-    GroupNorm<V, W, FAST> norm;
+    GroupNorm<THREADS, V, W, FAST> norm;
     norm.d = d, norm.groups = groups, norm.width = d / groups, norm.eps = eps, norm.sq = smem, norm.sums = smem + d / W;
     Vec<W> v[V];
     float inv[V];
@@ -347,7 +369,8 @@ __global__ void __launch_bounds__(THREADS) projection_norms_kernel(const __grid_
 
 // ------------------------------------------------------------------ short convolution
 // A thread owns W channels and walks the rows of its tile with the rows before in registers.
-template <typename T, int W, int TM>
+// RESIDUAL: `in` (f32) itself is added, and there is neither bias nor activation.
+template <typename T, int W, int TM, bool RESIDUAL>
 __global__ void __launch_bounds__(THREADS) short_conv_kernel(const __grid_constant__ ShortConv s, uint32_t* __restrict__ err) {
     const AttnTile tile = row_tile(s.tiles, blockIdx.x);
     const tsb_row_desc rd = s.rows[tile.row_first];
@@ -358,10 +381,11 @@ __global__ void __launch_bounds__(THREADS) short_conv_kernel(const __grid_consta
     if (!ok && threadIdx.x == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
     if (!ok || c >= s.channels) return;
     Vec<W> w[TM], hist[TM - 1];
-    const Vec<W> bias = load(s.bias + c, Vec<W>());
+    const Vec<W> bias = RESIDUAL ? zeros<W>() : load(s.bias + c, Vec<W>());
 #pragma unroll
     for (int j = 0; j < TM; j++) w[j] = j < s.taps ? load(s.w + (int64_t)(s.taps - 1 - j) * s.channels + c, Vec<W>()) : zeros<W>();  // w[j]: j rows back
-    const T* in = static_cast<const T*>(s.in) + c;
+    using In = std::conditional_t<RESIDUAL, float, T>;
+    const In* in = static_cast<const In*>(s.in) + c;
 #pragma unroll
     for (int j = 0; j < TM - 1; j++) {
         const int back = j + 1, pos = rd.base + rd.slot - back;
@@ -370,25 +394,25 @@ __global__ void __launch_bounds__(THREADS) short_conv_kernel(const __grid_consta
         hist[j] = back <= rd.slot ? load(in + (int64_t)(tile.row_first - back) * s.in_stride, Vec<W>())
                                   : load(ring_row_before(s.ring, rd.seq, rd.base, pos, s.use_before) + c, Vec<W>());
     }
-    const bool any_kept = s.taps > 1 && ring_keeps(s.ring, s.rows, s.n_rows, tile.row_first + tile.n_rows - 1, rd.seq);
     constexpr int AHEAD = W == 4 ? 4 : 8;  // rows in flight
     for (int i0 = 0; i0 < tile.n_rows; i0 += AHEAD) {
         Vec<W> x[AHEAD];
 #pragma unroll
         for (int i = 0; i < AHEAD; i++)
             if (i0 + i < tile.n_rows) x[i] = load(in + (int64_t)(tile.row_first + i0 + i) * s.in_stride, Vec<W>());
+        const bool any_kept = s.taps > 1 && ring_keeps(s.ring, s.rows, s.n_rows, tile.row_first + tile.n_rows - 1, rd.seq);
 #pragma unroll
         for (int i = 0; i < AHEAD; i++) {
             if (i0 + i >= tile.n_rows) break;
             const int r = tile.row_first + i0 + i;
             if (any_kept && ring_keeps(s.ring, s.rows, s.n_rows, r, rd.seq)) store(ring_row(s.ring, rd.seq, rd.base + rd.slot + i0 + i) + c, x[i]);
-            Vec<W> o = bias;
+            Vec<W> o = RESIDUAL ? x[i] : bias;
 #pragma unroll
             for (int k = 0; k < W; k++) {
 #pragma unroll
                 for (int j = TM - 2; j >= 0; j--) o.v[k] = fmaf(w[j + 1].v[k], hist[j].v[k], o.v[k]);
                 o.v[k] = fmaf(w[0].v[k], x[i].v[k], o.v[k]);
-                o.v[k] = silu<T>(o.v[k]);
+                if (!RESIDUAL) o.v[k] = silu<T>(o.v[k]);
             }
             store(static_cast<T*>(s.out) + (int64_t)r * s.out_stride + c, o);
 #pragma unroll
@@ -447,23 +471,24 @@ __global__ void __launch_bounds__(THREADS) gated_norm_kernel(const __grid_consta
 constexpr int MAX_VECS4 = 8, MAX_VECS1 = 16;
 bool by_fours(int d, int groups) { return (d / groups) % 4 == 0 && d <= 4 * THREADS * MAX_VECS4; }
 
-template <typename T, int V, int W, bool FAST>
+template <typename T, int NT, int V, int W, bool FAST>
 cudaError_t launch_end(tsb_ctx* ctx, cudaStream_t st, const SublayerEnd& s) {
-    const size_t smem = group_norm_smem<V, W>(s.d, s.groups, FAST);
-    auto run = [&](auto kernel) { return tsb_launch(ctx, kernel, dim3((unsigned)s.tiles.n), dim3(THREADS), smem, st, true, s, ctx->dev_error); };
-    return s.taps <= 4 ? run(sublayer_end_kernel<T, V, W, FAST, 4>) : run(sublayer_end_kernel<T, V, W, FAST, CONV_MAX_TAPS>);
+    const size_t smem = group_norm_smem<NT, V, W>(s.d, s.groups, FAST);
+    auto run = [&](auto kernel) { return tsb_launch(ctx, kernel, dim3((unsigned)s.tiles.n), dim3(NT), smem, st, true, s, ctx->dev_error); };
+    if (s.taps == 0) return run(sublayer_end_kernel<T, NT, V, W, FAST, 1>);
+    return s.taps <= 4 ? run(sublayer_end_kernel<T, NT, V, W, FAST, 4>) : run(sublayer_end_kernel<T, NT, V, W, FAST, CONV_MAX_TAPS>);
 }
 template <typename T>
 cudaError_t launch_end_of(tsb_ctx* ctx, cudaStream_t st, const SublayerEnd& s) {
     const int d = s.d, gw = d / s.groups;
     if (by_fours(d, s.groups) && s.out_stride % 4 == 0 && s.expert_stride % 4 == 0) {
         const bool fast = gw % 128 == 0;
-        if (d <= 4 * THREADS) return fast ? launch_end<T, 1, 4, true>(ctx, st, s) : launch_end<T, 1, 4, false>(ctx, st, s);
-        if (d <= 4 * THREADS * 2) return fast ? launch_end<T, 2, 4, true>(ctx, st, s) : launch_end<T, 2, 4, false>(ctx, st, s);
-        if (d <= 4 * THREADS * 4) return fast ? launch_end<T, 4, 4, true>(ctx, st, s) : launch_end<T, 4, 4, false>(ctx, st, s);
-        return fast ? launch_end<T, 8, 4, true>(ctx, st, s) : launch_end<T, 8, 4, false>(ctx, st, s);
+        if (d <= 1024) return fast ? launch_end<T, 256, 1, 4, true>(ctx, st, s) : launch_end<T, 256, 1, 4, false>(ctx, st, s);
+        if (d <= 2048) return fast ? launch_end<T, 512, 1, 4, true>(ctx, st, s) : launch_end<T, 512, 1, 4, false>(ctx, st, s);
+        if (d <= 4096) return fast ? launch_end<T, 512, 2, 4, true>(ctx, st, s) : launch_end<T, 512, 2, 4, false>(ctx, st, s);
+        return fast ? launch_end<T, 512, 4, 4, true>(ctx, st, s) : launch_end<T, 512, 4, 4, false>(ctx, st, s);
     }
-    return d <= THREADS * 4 ? launch_end<T, 4, 1, false>(ctx, st, s) : launch_end<T, MAX_VECS1, 1, false>(ctx, st, s);
+    return d <= 1024 ? launch_end<T, 256, 4, 1, false>(ctx, st, s) : launch_end<T, 512, 8, 1, false>(ctx, st, s);
 }
 
 template <typename T>
@@ -473,10 +498,23 @@ cudaError_t launch_norm_of(tsb_ctx* ctx, cudaStream_t st, const float* x, int d,
         return tsb_launch(ctx, kernel, dim3((unsigned)n), dim3(THREADS), smem, st, true, x, d, weight, groups, eps, want, first, step, out, out_stride);
     };
     if (by_fours(d, groups) && out_stride % 4 == 0) {
-        if ((d / groups) % 128 == 0) return run(group_norm_rows_kernel<T, MAX_VECS4, 4, true>, group_norm_smem<MAX_VECS4, 4>(d, groups, true));
-        return run(group_norm_rows_kernel<T, MAX_VECS4, 4, false>, group_norm_smem<MAX_VECS4, 4>(d, groups, false));
+        if ((d / groups) % 128 == 0) return run(group_norm_rows_kernel<T, MAX_VECS4, 4, true>, group_norm_smem<THREADS, MAX_VECS4, 4>(d, groups, true));
+        return run(group_norm_rows_kernel<T, MAX_VECS4, 4, false>, group_norm_smem<THREADS, MAX_VECS4, 4>(d, groups, false));
     }
-    return run(group_norm_rows_kernel<T, MAX_VECS1, 1, false>, group_norm_smem<MAX_VECS1, 1>(d, groups, false));
+    return run(group_norm_rows_kernel<T, MAX_VECS1, 1, false>, group_norm_smem<THREADS, MAX_VECS1, 1>(d, groups, false));
+}
+
+template <bool RESIDUAL>
+cudaError_t launch_conv(tsb_ctx* ctx, cudaStream_t st, bool f32, const ShortConv& c) {
+    const bool vec = c.channels % 4 == 0 && c.in_stride % 4 == 0 && c.out_stride % 4 == 0 && (uintptr_t)c.in % 16 == 0;
+    auto run = [&](auto kernel, int w) {
+        return tsb_launch(ctx, kernel, dim3((unsigned)c.tiles.n, (unsigned)((c.channels + THREADS * w - 1) / (THREADS * w))), dim3(THREADS), 0, st, true, c, ctx->dev_error);
+    };
+    if (c.taps <= 4) {
+        if (f32) return vec ? run(short_conv_kernel<float, 4, 4, RESIDUAL>, 4) : run(short_conv_kernel<float, 1, 4, RESIDUAL>, 1);
+        return vec ? run(short_conv_kernel<__nv_bfloat16, 4, 4, RESIDUAL>, 4) : run(short_conv_kernel<__nv_bfloat16, 1, 4, RESIDUAL>, 1);
+    }
+    return f32 ? run(short_conv_kernel<float, 1, CONV_MAX_TAPS, RESIDUAL>, 1) : run(short_conv_kernel<__nv_bfloat16, 1, CONV_MAX_TAPS, RESIDUAL>, 1);
 }
 
 }  // namespace
@@ -484,14 +522,27 @@ cudaError_t launch_norm_of(tsb_ctx* ctx, cudaStream_t st, const float* x, int d,
 bool sublayer_end_supported(int d, int groups, int taps) {
     return groups > 0 && d % groups == 0 && taps >= 0 && taps <= CONV_MAX_TAPS && (by_fours(d, groups) || d <= THREADS * MAX_VECS1) && d / 4 + groups <= 10000;
 }
-int sublayer_rows_per_tile(const tsb_ctx* ctx, int rows) { return rows <= 2 * ctx->sm_count ? 1 : rows <= 8 * ctx->sm_count ? 4 : 8; }
-
-cudaError_t launch_sublayer_end(tsb_ctx* ctx, cudaStream_t st, bool f32, const SublayerEnd& s) {
-    return f32 ? launch_end_of<float>(ctx, st, s) : launch_end_of<__nv_bfloat16>(ctx, st, s);
+int sublayer_rows_per_tile(const tsb_ctx* ctx, int rows) {
+    const int sms = ctx->sm_count > 0 ? ctx->sm_count : 148;
+    if (rows <= 2 * sms) return 1;
+    return rows <= 8 * sms ? 4 : std::max(8, std::min(16, (rows + sms - 1) / sms));  // one CTA per SM where that is enough
 }
 
-cudaError_t launch_rings_before(tsb_ctx* ctx, cudaStream_t st, const RowRing* rings_dev, int n, const tsb_row_desc* rows_dev, int rows) {
-    return tsb_launch(ctx, rings_before_kernel, dim3((unsigned)rows, (unsigned)n), dim3(THREADS), 0, st, true, rings_dev, rows_dev);
+cudaError_t launch_sublayer_end(tsb_ctx* ctx, cudaStream_t st, bool f32, const SublayerEnd& s) {
+    auto run = [&](const SublayerEnd& v) { return f32 ? launch_end_of<float>(ctx, st, v) : launch_end_of<__nv_bfloat16>(ctx, st, v); };
+    if (s.taps == 0 || !s.experts || s.n_rows <= 2 * ctx->sm_count) return run(s);
+    // many sums of experts: a CTA per row, then the convolution, instead of runs of rows that make the rows before them again
+    SublayerEnd sum = s;
+    sum.taps = 0, sum.tiles = RowTiles::uniform(s.n_rows, 1, 1);
+    if (cudaError_t e = run(sum); e != cudaSuccess) return e;
+    ShortConv c;
+    c.in = s.x_out, c.in_stride = s.d, c.out = s.out, c.out_stride = s.out_stride, c.channels = s.d, c.taps = s.taps, c.w = s.taps_w, c.ring = s.ring;
+    c.use_before = s.use_before, c.rows = s.rows, c.n_rows = s.n_rows, c.tiles = s.tiles;
+    return launch_conv<true>(ctx, st, f32, c);
+}
+
+cudaError_t launch_rings_before(tsb_ctx* ctx, cudaStream_t st, const RowRing* rings_dev, int n, const tsb_row_desc* rows_dev, const RowTiles& portions) {
+    return tsb_launch(ctx, rings_before_kernel, dim3((unsigned)portions.n, (unsigned)n), dim3(THREADS), 0, st, true, rings_dev, rows_dev, portions);
 }
 
 cudaError_t launch_group_norm_rows(tsb_ctx* ctx, cudaStream_t st, bool f32, const float* x, int d, const float* weight, int groups, float eps, const int32_t* want_dev,
@@ -507,17 +558,7 @@ cudaError_t launch_projection_norms(tsb_ctx* ctx, cudaStream_t st, bool f32, con
     return vec ? run(projection_norms_kernel<__nv_bfloat16, 4>) : run(projection_norms_kernel<__nv_bfloat16, 1>);
 }
 
-cudaError_t launch_short_conv(tsb_ctx* ctx, cudaStream_t st, bool f32, const ShortConv& c) {
-    const bool vec = c.channels % 4 == 0 && c.in_stride % 4 == 0 && c.out_stride % 4 == 0 && (uintptr_t)c.in % 16 == 0;
-    auto run = [&](auto kernel, int w) {
-        return tsb_launch(ctx, kernel, dim3((unsigned)c.tiles.n, (unsigned)((c.channels + THREADS * w - 1) / (THREADS * w))), dim3(THREADS), 0, st, true, c, ctx->dev_error);
-    };
-    if (c.taps <= 4) {
-        if (f32) return vec ? run(short_conv_kernel<float, 4, 4>, 4) : run(short_conv_kernel<float, 1, 4>, 1);
-        return vec ? run(short_conv_kernel<__nv_bfloat16, 4, 4>, 4) : run(short_conv_kernel<__nv_bfloat16, 1, 4>, 1);
-    }
-    return f32 ? run(short_conv_kernel<float, 1, CONV_MAX_TAPS>, 1) : run(short_conv_kernel<__nv_bfloat16, 1, CONV_MAX_TAPS>, 1);
-}
+cudaError_t launch_short_conv(tsb_ctx* ctx, cudaStream_t st, bool f32, const ShortConv& c) { return launch_conv<false>(ctx, st, f32, c); }
 
 cudaError_t launch_gated_norm(tsb_ctx* ctx, cudaStream_t st, bool f32, const GatedNorm& g, int rows) {
     const int gw = g.width / g.groups;

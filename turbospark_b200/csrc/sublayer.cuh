@@ -39,8 +39,8 @@ bool sublayer_end_supported(int d, int groups, int taps);
 int sublayer_rows_per_tile(const tsb_ctx* ctx, int rows);  // rows of a tile that suit a pass of so many rows
 cudaError_t launch_sublayer_end(tsb_ctx* ctx, cudaStream_t st, bool f32, const SublayerEnd& s);
 
-// Copies of the rows before every portion of the pass (rows with slot 0), of n rings in device memory, to their `before`.
-cudaError_t launch_rings_before(tsb_ctx* ctx, cudaStream_t st, const RowRing* rings_dev, int n, const tsb_row_desc* rows_dev, int rows);
+// Copies of the rows before every portion of the pass, of n rings in device memory, to their `before`.
+cudaError_t launch_rings_before(tsb_ctx* ctx, cudaStream_t st, const RowRing* rings_dev, int n, const tsb_row_desc* rows_dev, const RowTiles& portions);
 
 // out[i] = x[want(i)] normed in groups, want(i) as in launch_norm_rows.
 cudaError_t launch_group_norm_rows(tsb_ctx* ctx, cudaStream_t st, bool f32, const float* x, int d, const float* weight, int groups, float eps, const int32_t* want_dev,
