@@ -127,7 +127,7 @@ __global__ void __launch_bounds__(NT) sublayer_end_kernel(const __grid_constant_
     const AttnTile tile = row_tile(s.tiles, blockIdx.x);
     const tsb_row_desc rd = s.rows[tile.row_first];
     const int d = s.d, halo = s.taps > 0 ? min(s.taps - 1, rd.slot) : 0;
-    const bool ok = s.taps == 0 || (rd.seq >= 0 && rd.seq < s.ring.n_streams);
+    const bool ok = s.taps <= 1 || (rd.seq >= 0 && rd.seq < s.ring.n_streams);
     GroupNorm<NT, V, W, FAST> norm;
     norm.d = d, norm.groups = s.groups, norm.width = d / s.groups, norm.eps = s.eps, norm.sq = smem, norm.sums = smem + d / W;
     Vec<W> hist[TM > 1 ? TM - 1 : 1][V];  // hist[j]: the row j + 1 before the current one
