@@ -29,6 +29,7 @@ __device__ __forceinline__ float ex2(float x) {
     asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
+__device__ __forceinline__ float silu(float z) { return __fdividef(z, 1.f + __expf(-z)); }
 __device__ __forceinline__ uint32_t pack(float lo, float hi) {
     const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<const uint32_t*>(&h);
@@ -66,9 +67,9 @@ Scratch scratch_of(const Recurrence& r, void* p, int chunks) {
 }
 
 // rows x columns of a projection into shared memory, zeros outside
-template <int ROW_BYTES>
+template <int ROW_BYTES, int NT>
 __device__ __forceinline__ void copy_tile(uint32_t dst, const __nv_bfloat16* src, int64_t stride, int n_rows, int n_cols) {
-    for (int i = threadIdx.x; i < C * (ROW_BYTES / 16); i += THREADS) {
+    for (int i = threadIdx.x; i < C * (ROW_BYTES / 16); i += NT) {
         const int r = i / (ROW_BYTES / 16), c = i % (ROW_BYTES / 16);
         const bool ok = r < n_rows && c * 8 < n_cols;
         cp16(dst + at<ROW_BYTES>(r, c), src + (ok ? r * stride + c * 8 : 0), ok);
@@ -101,36 +102,55 @@ __device__ __forceinline__ RowGates row_gates(const Recurrence& a, int row0, int
     return g;
 }
 
-// REC_FORGET: a thread has one channel of TR rows.  pre: pre-activations of the chunk in shared memory, which become 1 - f =
-// (1 - l) sigmoid(-z); returns the product of the thread's f.
+// REC_FORGET: a thread has two neighbouring channels, 2 (thread % (DK / 2)), of TR rows.
+template <int DK, int NT>
+struct Channels {
+    static constexpr int RS = NT / (DK / 2), TR = C / RS;  // row splits, rows of a thread
+    int ch, part, first;
+    __device__ __forceinline__ Channels() : ch(threadIdx.x % (DK / 2) * 2), part(threadIdx.x / (DK / 2)), first(part * TR) {}
+    // of the split i and the thread's channels
+    __device__ __forceinline__ float2& total(float* fv, int i) const { return reinterpret_cast<float2*>(fv)[i * (DK / 2) + ch / 2]; }
+    __device__ __forceinline__ uint32_t key(int r) const { return at<DK * 2>(r, ch >> 3) + (ch & 7) * 2; }
+};
+// 1 - f = (1 - l) sigmoid(-z)
+__device__ __forceinline__ float one_minus_f(float z, float open) {
+    const float e = __expf(-fabsf(z)), d = __fdividef(1.f, 1.f + e);
+    return open * (z >= 0.f ? e * d : d);
+}
 template <int DK>
-__device__ __forceinline__ float forget_gates(const Recurrence& a, float* pre, int head, int n) {
-    constexpr int RS = THREADS / DK, TR = C / RS;
-    const int ch = threadIdx.x % DK, first = threadIdx.x / DK * TR;
-    const float low = ch < a.dim ? a.lower[(int64_t)head * a.dim + ch] : 1.f;
-    float product = 1.f;
+__device__ __forceinline__ float2 open_of(const Recurrence& a, int head, int ch) {  // 1 - l; channels outside stay open
+    const float* l = a.lower + (int64_t)head * a.dim + ch;
+    return ch < a.dim ? make_float2(1.f - l[0], 1.f - l[1]) : make_float2(0.f, 0.f);
+}
+// pre: pre-activations of the chunk in shared memory, which become 1 - f; returns the products of the thread's f.
+template <int DK, int NT>
+__device__ __forceinline__ float2 forget_gates(const Recurrence& a, float* pre, int head, int n) {
+    const Channels<DK, NT> me;
+    const float2 open = open_of<DK>(a, head, me.ch);
+    float2 product = make_float2(1.f, 1.f);
 #pragma unroll 4
-    for (int i = 0; i < TR; i++) {
-        float& x = pre[(first + i) * DK + ch];
-        const float e = __expf(-fabsf(x)), d = __fdividef(1.f, 1.f + e);
-        x = first + i < n ? (1.f - low) * (x >= 0.f ? e * d : d) : 0.f;
-        product *= 1.f - x;
+    for (int i = 0; i < me.TR; i++) {
+        float2& x = *reinterpret_cast<float2*>(pre + (me.first + i) * DK + me.ch);
+        const bool in = me.first + i < n;
+        x = in ? make_float2(one_minus_f(x.x, open.x), one_minus_f(x.y, open.y)) : make_float2(0.f, 0.f);
+        product.x *= 1.f - x.x, product.y *= 1.f - x.y;
     }
     return product;
 }
-template <int DK>
+template <int DK, int NT>
 __device__ __forceinline__ void copy_gates(const Recurrence& a, uint32_t dst, int row0, int n, int head) {
     const float* gz = a.gate + (int64_t)row0 * a.gate_stride + (int64_t)head * a.dim;
-    for (int i = threadIdx.x; i < C * (DK / 4); i += THREADS) {
+    for (int i = threadIdx.x; i < C * (DK / 4); i += NT) {
         const int r = i / (DK / 4), c = i % (DK / 4);
         const bool ok = r < n && c * 4 < a.dim;
         cp16(dst + (r * DK + c * 4) * 4, gz + (ok ? r * a.gate_stride + c * 4 : 0), ok);
     }
 }
-__device__ __forceinline__ void put_split(uint8_t* hi, uint8_t* lo, uint32_t off, float v) {
-    const __nv_bfloat16 h = __float2bfloat16_rn(v);
-    *reinterpret_cast<__nv_bfloat16*>(hi + off) = h;
-    *reinterpret_cast<__nv_bfloat16*>(lo + off) = __float2bfloat16_rn(v - __bfloat162float(h));
+__device__ __forceinline__ void put_split(uint8_t* hi, uint8_t* lo, uint32_t off, float a, float b) {
+    uint32_t h, l;
+    split(a, b, h, l);
+    *reinterpret_cast<uint32_t*>(hi + off) = h;
+    *reinterpret_cast<uint32_t*>(lo + off) = l;
 }
 
 // ------------------------------------------------------------------ what a chunk adds to the state
@@ -140,7 +160,7 @@ struct AddSmem {
     static constexpr int KEY = C * DK * 2, VAL = C * VB * 2;  // a tile of keys, of values
     static constexpr int K = 0, V = FORGET ? 2 * KEY : KEY, W = V + VAL;  // FORGET: keys, values; else keys, values, weighted values (high, low)
     static constexpr int Z = W, F = FORGET ? Z + C * DK * 4 : W + 2 * VAL;
-    static constexpr int BYTES = F + (FORGET ? THREADS : C + 4) * 4;
+    static constexpr int BYTES = F + (FORGET ? 2 * THREADS : C + 4) * 4;
 };
 
 template <int KIND, int DK, int VB>
@@ -161,11 +181,11 @@ __global__ void __launch_bounds__(THREADS)
     const __nv_bfloat16* gv = static_cast<const __nv_bfloat16*>(a.v) + (int64_t)row0 * a.v_stride + (int64_t)head * a.vdim + col0;
     pdl_wait();
     pdl_launch_dependents();
-    copy_tile<BV>(base + M::V, gv, a.v_stride, n, a.vdim - col0);
+    copy_tile<BV, THREADS>(base + M::V, gv, a.v_stride, n, a.vdim - col0);
     if (FORGET) {
-        copy_gates<DK>(a, base + M::Z, row0, n, head);
+        copy_gates<DK, THREADS>(a, base + M::Z, row0, n, head);
     } else {
-        copy_tile<KB>(base + M::K, static_cast<const __nv_bfloat16*>(a.k) + (int64_t)row0 * a.k_stride + head / a.heads_per_key * a.dim, a.k_stride, n, a.dim);
+        copy_tile<KB, THREADS>(base + M::K, static_cast<const __nv_bfloat16*>(a.k) + (int64_t)row0 * a.k_stride + head / a.heads_per_key * a.dim, a.k_stride, n, a.dim);
     }
     cp_async_commit();
     if (!FORGET && warp == 0) {
@@ -191,20 +211,19 @@ __global__ void __launch_bounds__(THREADS)
     __syncthreads();
     if (FORGET) {
         float* pre = reinterpret_cast<float*>(smem + M::Z);
-        constexpr int RS = THREADS / DK, TR = C / RS;
-        const int ch = threadIdx.x % DK, part = threadIdx.x / DK;
-        fv[threadIdx.x] = forget_gates<DK>(a, pre, head, n);
+        const Channels<DK, THREADS> me;
+        me.total(fv, me.part) = forget_gates<DK, THREADS>(a, pre, head, n);
         __syncthreads();
-        float e = 1.f;  // product of the rows behind
-        for (int i = part + 1; i < RS; i++) e *= fv[i * DK + ch];
+        float2 e = make_float2(1.f, 1.f);  // products of the rows behind
+        for (int i = me.part + 1; i < me.RS; i++) e.x *= me.total(fv, i).x, e.y *= me.total(fv, i).y;
 #pragma unroll 4
-        for (int i = TR - 1; i >= 0; i--) {
-            const int r = part * TR + i;
-            const float k = pre[r * DK + ch];
-            put_split(smem + M::K, smem + M::K + M::KEY, at<KB>(r, ch >> 3) + (ch & 7) * 2, k * e);
-            e *= 1.f - k;
+        for (int i = me.TR - 1; i >= 0; i--) {
+            const int r = me.first + i;
+            const float2 k = *reinterpret_cast<const float2*>(pre + r * DK + me.ch);
+            put_split(smem + M::K, smem + M::K + M::KEY, me.key(r), k.x * e.x, k.y * e.y);
+            e.x *= 1.f - k.x, e.y *= 1.f - k.y;
         }
-        if (part == 0 && blockIdx.x == 0 && ch < a.dim) out.decay[slot * a.dim + ch] = e;
+        if (me.part == 0 && blockIdx.x == 0 && me.ch < a.dim) *reinterpret_cast<float2*>(out.decay + slot * a.dim + me.ch) = e;
     } else {
         for (int i = threadIdx.x; i < C * (VB / 2); i += THREADS) {
             const int r = i / (VB / 2), c = i % (VB / 2);
@@ -344,30 +363,30 @@ __global__ void __launch_bounds__(THREADS)
 }
 
 // ------------------------------------------------------------------ outputs of a chunk
-constexpr int VB = 64, BV = VB * 2;  // value columns of a CTA
-template <int KIND, int DK>
+template <int KIND, int DK, int VB, int NT>
 struct OutSmem {
     static constexpr bool FORGET = KIND == REC_FORGET;
     static constexpr int KEY = C * DK * 2, VAL = C * VB * 2, STATE = DK * VB * 2, PROD = C * C * 2;
-    // queries and keys (FORGET: high and low parts of each), values, state (high, low), products (high, low; FORGET: where the keys were)
-    static constexpr int Q = 0, K = FORGET ? 2 * KEY : KEY, V = 2 * K, S = V + VAL, P = FORGET ? K : S + 2 * STATE;
-    static constexpr int F = FORGET ? S + 2 * STATE : P + 2 * PROD;
+    // queries and keys (FORGET: high and low parts of each), values, state (high, low); products (high, low) where the keys were, or from there on
+    static constexpr int Q = 0, K = FORGET ? 2 * KEY : KEY, KEYS = (FORGET ? 2 : 1) * KEY > 2 * PROD ? (FORGET ? 2 : 1) * KEY : 2 * PROD;
+    static constexpr int V = K + KEYS, S = V + VAL, P = K, F = S + 2 * STATE;
     static constexpr int Z = S;  // FORGET: the gates of the chunk, before the state takes their place
-    static_assert(!FORGET || (C * DK * 4 <= 2 * STATE && PROD <= KEY), "");
-    static constexpr int BYTES = F + (FORGET ? THREADS : 4 * C + 8 + DK + 5 * C) * 4;
+    static_assert(!FORGET || C * DK * 4 <= 2 * STATE, "");
+    static constexpr int BYTES = F + (FORGET ? 2 * NT : KIND == REC_MLSTM ? 4 * C + DK + 5 * C : 3 * C) * 4;
 };
 
-template <int KIND, int DK>
-__global__ void __launch_bounds__(THREADS, DK > 128 ? 1 : DK > 64 || KIND == REC_FORGET ? 2 : 3)
+// NT threads: a warp per 16 rows and 32 value columns
+template <int KIND, int DK, int VB, int NT>
+__global__ void __launch_bounds__(NT, NT > 256 ? 1 : DK > 128 || KIND == REC_FORGET ? 2 : 3)
     chunk_out_kernel(const __grid_constant__ Recurrence a, const __grid_constant__ RowTiles chunks, const __grid_constant__ Scratch in, uint32_t* __restrict__ err) {
-    using M = OutSmem<KIND, DK>;
+    using M = OutSmem<KIND, DK, VB, NT>;
+    static_assert(NT / 32 == 4 * (VB / 32), "");
     constexpr bool FORGET = KIND == REC_FORGET, MLSTM = KIND == REC_MLSTM, SSD = KIND == REC_SSD;
-    constexpr int KB = DK * 2, KS = DK / 16, NV = 4;  // a warp has 16 rows and 32 columns of the output
-    constexpr int RS = FORGET ? THREADS / DK : 1, TR = C / RS;
+    constexpr int KB = DK * 2, BV = VB * 2, KS = DK / 16, NV = 4, NW = NT / 32;
     extern __shared__ __align__(128) uint8_t smem[];
     const uint32_t base = smem_u32(smem);
     float* fv = reinterpret_cast<float*>(smem + M::F);
-    float *ea = fv, *eb = fv + C, *gain = fv + 2 * C, *floor_ = fv + 3 * C, *norm = fv + 4 * C + 8, *nq = norm + DK;  // nq [rows][5]: shares of n . q
+    float *ea = fv, *eb = fv + C, *gain = fv + 2 * C, *floor_ = fv + 3 * C, *norm = fv + 4 * C, *nq = norm + DK;  // nq [rows][5]: shares of n . q
     __shared__ int cut_end;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gid = lane >> 2, tig = lane & 3;
     const int head = blockIdx.y, col0 = blockIdx.x * VB, key_at = head / a.heads_per_key * a.dim;
@@ -377,20 +396,20 @@ __global__ void __launch_bounds__(THREADS, DK > 128 ? 1 : DK > 64 || KIND == REC
     const __nv_bfloat16* gq = static_cast<const __nv_bfloat16*>(a.q) + (int64_t)row0 * a.q_stride + key_at;
     pdl_wait();
     pdl_launch_dependents();
-    copy_tile<BV>(base + M::V, static_cast<const __nv_bfloat16*>(a.v) + (int64_t)row0 * a.v_stride + (int64_t)head * a.vdim + col0, a.v_stride, n, a.vdim - col0);
-    copy_tile<KB>(base + M::Q, gq, a.q_stride, n, a.dim);
+    copy_tile<BV, NT>(base + M::V, static_cast<const __nv_bfloat16*>(a.v) + (int64_t)row0 * a.v_stride + (int64_t)head * a.vdim + col0, a.v_stride, n, a.vdim - col0);
+    copy_tile<KB, NT>(base + M::Q, gq, a.q_stride, n, a.dim);
     if (FORGET) {
-        copy_gates<DK>(a, base + M::Z, row0, n, head);
+        copy_gates<DK, NT>(a, base + M::Z, row0, n, head);
     } else {
-        copy_tile<KB>(base + M::K, static_cast<const __nv_bfloat16*>(a.k) + (int64_t)row0 * a.k_stride + key_at, a.k_stride, n, a.dim);
+        copy_tile<KB, NT>(base + M::K, static_cast<const __nv_bfloat16*>(a.k) + (int64_t)row0 * a.k_stride + key_at, a.k_stride, n, a.dim);
     }
     // the state: four numbers as four high and four low halves, to two tiles
-    constexpr int PIECES = DK * (VB / 4), MINE = PIECES / THREADS;
+    constexpr int PIECES = DK * (VB / 4), MINE = PIECES / NT;
     const float* src = in.add + slot * a.dim * a.vdim + col0;
     uint4 held[FORGET ? MINE : 1];  // FORGET: their place is still taken
 #pragma unroll
     for (int k = 0; k < MINE; k++) {
-        const int i = k * THREADS + threadIdx.x, r = i / (VB / 4), c = i % (VB / 4);
+        const int i = k * NT + threadIdx.x, r = i / (VB / 4), c = i % (VB / 4);
         const bool ok = r < a.dim && col0 + c * 4 < a.vdim;
         const float* p = ok ? src + (int64_t)r * a.vdim + c * 4 : in.add;
         if (FORGET) {
@@ -403,7 +422,7 @@ __global__ void __launch_bounds__(THREADS, DK > 128 ? 1 : DK > 64 || KIND == REC
     cp_async_commit();
     if (!FORGET) {
         if (MLSTM)
-            for (int i = threadIdx.x; i < DK; i += THREADS) norm[i] = i < a.dim ? in.norm[slot * a.dim + i] : 0.f;
+            for (int i = threadIdx.x; i < DK; i += NT) norm[i] = i < a.dim ? in.norm[slot * a.dim + i] : 0.f;
         if (warp == 0) {
             const RowGates g = row_gates<FORGET ? REC_SSD : KIND>(a, row0, n, head, lane);
             if (SSD) {
@@ -437,30 +456,29 @@ __global__ void __launch_bounds__(THREADS, DK > 128 ? 1 : DK > 64 || KIND == REC
     __syncthreads();
 
     // ---- FORGET: queries times E_t, keys over E_s
-    const int ch = FORGET ? threadIdx.x % DK : 0, part = FORGET ? threadIdx.x / DK : 0;
+    const Channels<FORGET ? DK : 64, NT> me;
     bool cuts = false;
     if (FORGET) {
         float* pre = reinterpret_cast<float*>(smem + M::Z);
-        const float mine = forget_gates<DK>(a, pre, head, n);
-        fv[threadIdx.x] = mine;
+        const float2 mine = forget_gates<DK, NT>(a, pre, head, n);
+        me.total(fv, me.part) = mine;
         __syncthreads();
-        float e = E_ONE;  // E at the start of the thread's rows
-        for (int i = 0; i < part; i++) e *= fv[i * DK + ch];
-        cuts = __syncthreads_or(e * mine < E_MIN);  // E only falls
-#pragma unroll 8
-        for (int i = 0; i < TR; i++) {
-            const int r = part * TR + i;
-            const float k = pre[r * DK + ch];
-            e *= 1.f - k;
-            const uint32_t off = at<KB>(r, ch >> 3) + (ch & 7) * 2;
-            const float x = __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(smem + M::Q + off));
-            put_split(smem + M::Q, smem + M::Q + M::KEY, off, __fdividef(x, 1.f + __expf(-x)) * e);
-            put_split(smem + M::K, smem + M::K + M::KEY, off, cuts ? 0.f : __fdividef(k, e));
+        float2 e = make_float2(E_ONE, E_ONE);  // E at the start of the thread's rows
+        for (int i = 0; i < me.part; i++) e.x *= me.total(fv, i).x, e.y *= me.total(fv, i).y;
+        cuts = __syncthreads_or(fminf(e.x * mine.x, e.y * mine.y) < E_MIN);  // E only falls
+#pragma unroll 4
+        for (int i = 0; i < me.TR; i++) {
+            const int r = me.first + i;
+            const float2 k = *reinterpret_cast<const float2*>(pre + r * DK + me.ch);
+            e.x *= 1.f - k.x, e.y *= 1.f - k.y;
+            const uint32_t off = me.key(r), x = *reinterpret_cast<const uint32_t*>(smem + M::Q + off);
+            put_split(smem + M::Q, smem + M::Q + M::KEY, off, silu(__uint_as_float(x << 16)) * e.x, silu(__uint_as_float(x & 0xFFFF0000u)) * e.y);
+            put_split(smem + M::K, smem + M::K + M::KEY, off, cuts ? 0.f : __fdividef(k.x, e.x), cuts ? 0.f : __fdividef(k.y, e.y));
         }
         __syncthreads();  // the gates have been read
 #pragma unroll
         for (int k = 0; k < MINE; k++) {
-            const int i = k * THREADS + threadIdx.x, r = i / (VB / 4), c = i % (VB / 4);
+            const int i = k * NT + threadIdx.x, r = i / (VB / 4), c = i % (VB / 4);
             const uint32_t off = at<BV>(r, c >> 1) + (c & 1) * 8;
             const uint4 w = held[FORGET ? k : 0];
             *reinterpret_cast<uint2*>(smem + M::S + off) = make_uint2(w.x, w.y);
@@ -531,10 +549,10 @@ __global__ void __launch_bounds__(THREADS, DK > 128 ? 1 : DK > 64 || KIND == REC
         *reinterpret_cast<uint32_t*>(smem + M::P + M::PROD + ob) = l1;
     };
     auto products = [&](bool rect, int from) {
-        float held_p[2][2][4];  // FORGET: a warp's tiles wait until every warp has read the keys
+        float held_p[(10 + NW - 1) / NW][2][4];  // a warp's tiles wait until every warp has read the keys
 #pragma unroll
-        for (int u = 0; u < 2; u++) {
-            const int t = warp + 8 * u;
+        for (int u = 0; u < (10 + NW - 1) / NW; u++) {
+            const int t = warp + NW * u;
             if (t >= 10) break;
             const int ti = t < 1 ? 0 : t < 3 ? 1 : t < 6 ? 2 : 3, j = t - ti * (ti + 1) / 2;
             const int ra = ti * 16 + gid, rb = ra + 8;
@@ -574,7 +592,6 @@ __global__ void __launch_bounds__(THREADS, DK > 128 ? 1 : DK > 64 || KIND == REC
                     held_p[u][i][x] = s0[i][x];
                 }
                 sum[0] += s0[i][0] + s0[i][1], sum[1] += s0[i][2] + s0[i][3];
-                if (!FORGET) store_products(ra, c0, s0[i]);
             }
             if (MLSTM) {
 #pragma unroll
@@ -585,16 +602,14 @@ __global__ void __launch_bounds__(THREADS, DK > 128 ? 1 : DK > 64 || KIND == REC
                 if (tig == 0) nq[ra * 5 + j] = sum[0], nq[rb * 5 + j] = sum[1];
             }
         }
-        if (FORGET) {
-            __syncthreads();
+        __syncthreads();
 #pragma unroll
-            for (int u = 0; u < 2; u++) {
-                const int t = warp + 8 * u;
-                if (t >= 10) break;
-                const int ti = t < 1 ? 0 : t < 3 ? 1 : t < 6 ? 2 : 3, j = t - ti * (ti + 1) / 2;
+        for (int u = 0; u < (10 + NW - 1) / NW; u++) {
+            const int t = warp + NW * u;
+            if (t >= 10) break;
+            const int ti = t < 1 ? 0 : t < 3 ? 1 : t < 6 ? 2 : 3, j = t - ti * (ti + 1) / 2;
 #pragma unroll
-                for (int i = 0; i < 2; i++) store_products(ti * 16 + gid, j * 16 + i * 8 + 2 * tig, held_p[u][i]);
-            }
+            for (int i = 0; i < 2; i++) store_products(ti * 16 + gid, j * 16 + i * 8 + 2 * tig, held_p[u][i]);
         }
     };
     auto times_values = [&]() {
@@ -617,30 +632,37 @@ __global__ void __launch_bounds__(THREADS, DK > 128 ? 1 : DK > 64 || KIND == REC
         times_values();
     } else {
         // the chunk is cut: gates and queries come from memory again
-        const float low_bound = ch < a.dim ? a.lower[(int64_t)head * a.dim + ch] : 1.f;
-        auto one_minus_f = [&](int r) {
-            if (r >= n || ch >= a.dim) return 0.f;
-            const float x = a.gate[(int64_t)(row0 + r) * a.gate_stride + (int64_t)head * a.dim + ch], e = __expf(-fabsf(x)), d = __fdividef(1.f, 1.f + e);
-            return (1.f - low_bound) * (x >= 0.f ? e * d : d);
+        const float2 open = open_of<DK>(a, head, me.ch);
+        auto key = [&](int r) {
+            if (r >= n || me.ch >= a.dim) return make_float2(0.f, 0.f);
+            const float* z = a.gate + (int64_t)(row0 + r) * a.gate_stride + (int64_t)head * a.dim + me.ch;
+            return make_float2(one_minus_f(z[0], open.x), one_minus_f(z[1], open.y));
         };
         auto query = [&](int r) {
-            const float x = r < n && ch < a.dim ? __bfloat162float(gq[r * a.q_stride + ch]) : 0.f;
-            return __fdividef(x, 1.f + __expf(-x));
+            if (r >= n || me.ch >= a.dim) return make_float2(0.f, 0.f);
+            const __nv_bfloat16* q = gq + r * a.q_stride + me.ch;
+            return make_float2(silu(__bfloat162float(q[0])), silu(__bfloat162float(q[1])));
         };
+        auto fall = [&](float2& e, int r) {
+            const float2 k = key(r);
+            e.x *= 1.f - k.x, e.y *= 1.f - k.y;
+            return k;
+        };
+        const int last = me.first + me.TR;
         for (int cut = 0; cut < n;) {
             // where a component of E, counted from the cut, falls too low
             __syncthreads();
-            float mine = 1.f;
-            for (int r = max(cut, part * TR); r < (part + 1) * TR; r++) mine *= 1.f - one_minus_f(r);
-            fv[threadIdx.x] = mine;
+            float2 mine = make_float2(1.f, 1.f);
+            for (int r = max(cut, me.first); r < last; r++) fall(mine, r);
+            me.total(fv, me.part) = mine;
             if (threadIdx.x == 0) cut_end = n;
             __syncthreads();
-            float e0 = E_ONE;
-            for (int i = 0; i < part; i++) e0 *= fv[i * DK + ch];
-            float e = e0;
-            for (int r = max(cut, part * TR); r < min(n, (part + 1) * TR); r++) {
-                e *= 1.f - one_minus_f(r);
-                if (e < E_MIN && r > cut) {
+            float2 e0 = make_float2(E_ONE, E_ONE);
+            for (int i = 0; i < me.part; i++) e0.x *= me.total(fv, i).x, e0.y *= me.total(fv, i).y;
+            float2 e = e0;
+            for (int r = max(cut, me.first); r < min(n, last); r++) {
+                fall(e, r);
+                if (fminf(e.x, e.y) < E_MIN && r > cut) {
                     atomicMin(&cut_end, r);
                     break;
                 }
@@ -648,13 +670,15 @@ __global__ void __launch_bounds__(THREADS, DK > 128 ? 1 : DK > 64 || KIND == REC
             __syncthreads();
             const int end = cut_end;
             e = e0;
-            for (int r = part * TR; r < (part + 1) * TR; r++) {
+            for (int r = me.first; r < last; r++) {
                 const bool now = r >= cut && r < end;
-                const float k = one_minus_f(r);
-                if (now) e = fmaxf(e * (1.f - k), E_MIN);  // a cut's first row may fall further: nothing of the rows before is left then
-                const uint32_t off = at<KB>(r, ch >> 3) + (ch & 7) * 2;
-                put_split(smem + M::Q, smem + M::Q + M::KEY, off, now ? query(r) * e : 0.f);
-                put_split(smem + M::K, smem + M::K + M::KEY, off, now ? __fdividef(k, e) : 0.f);
+                float2 k = make_float2(0.f, 0.f), q = k;
+                if (now) {
+                    k = fall(e, r), q = query(r);
+                    e.x = fmaxf(e.x, E_MIN), e.y = fmaxf(e.y, E_MIN);  // a cut's first row may fall further: nothing of the rows before is left then
+                }
+                put_split(smem + M::Q, smem + M::Q + M::KEY, me.key(r), q.x * e.x, q.y * e.y);
+                put_split(smem + M::K, smem + M::K + M::KEY, me.key(r), now ? __fdividef(k.x, e.x) : 0.f, now ? __fdividef(k.y, e.y) : 0.f);
             }
             __syncthreads();
             products(false, 0);
@@ -663,17 +687,16 @@ __global__ void __launch_bounds__(THREADS, DK > 128 ? 1 : DK > 64 || KIND == REC
             if (cut > 0) {
                 // the rows before the cut: keys brought to it, times the f of the rows between
                 __syncthreads();
-                mine = 1.f;
-                for (int r = part * TR; r < min(cut, (part + 1) * TR); r++) mine *= 1.f - one_minus_f(r);
-                fv[threadIdx.x] = mine;
+                mine = make_float2(1.f, 1.f);
+                for (int r = me.first; r < min(cut, last); r++) fall(mine, r);
+                me.total(fv, me.part) = mine;
                 __syncthreads();
-                e = 1.f;
-                for (int i = part + 1; i < RS; i++) e *= fv[i * DK + ch];
-                for (int r = (part + 1) * TR - 1; r >= part * TR; r--) {
-                    const bool old = r < cut;
-                    const float k = one_minus_f(r);
-                    put_split(smem + M::K, smem + M::K + M::KEY, at<KB>(r, ch >> 3) + (ch & 7) * 2, old ? k * e * (1.f / E_ONE) : 0.f);
-                    if (old) e *= 1.f - k;
+                e = make_float2(1.f / E_ONE, 1.f / E_ONE);
+                for (int i = me.part + 1; i < me.RS; i++) e.x *= me.total(fv, i).x, e.y *= me.total(fv, i).y;
+                for (int r = last - 1; r >= me.first; r--) {
+                    const float2 at_cut = e;
+                    const float2 k = r < cut ? fall(e, r) : make_float2(0.f, 0.f);
+                    put_split(smem + M::K, smem + M::K + M::KEY, me.key(r), k.x * at_cut.x, k.y * at_cut.y);
                 }
                 __syncthreads();
                 products(true, cut);
@@ -715,26 +738,33 @@ __global__ void __launch_bounds__(THREADS, DK > 128 ? 1 : DK > 64 || KIND == REC
 template <int KIND, int DK, int COLS>
 cudaError_t launch_add(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RecurrenceChunks& c, const Scratch& s) {
     constexpr size_t smem = AddSmem<KIND, DK, COLS>::BYTES;
-    static_assert(smem <= 226 * 1024 && OutSmem<KIND, DK>::BYTES <= 226 * 1024, "");
+    static_assert(smem <= 226 * 1024, "");
     static SmemOptIn configured;
     if (cudaError_t e = tsb_opt_in_smem(ctx, chunk_add_kernel<KIND, DK, COLS>, smem, configured); e != cudaSuccess) return e;
     return tsb_launch(ctx, chunk_add_kernel<KIND, DK, COLS>, dim3((unsigned)((r.vdim + COLS - 1) / COLS), (unsigned)r.heads, (unsigned)c.chunks.n), dim3(THREADS), smem, st,
                       true, r, c.chunks, s, ctx->dev_error);
 }
+template <int KIND, int DK, int COLS, int NT>
+cudaError_t launch_out(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RecurrenceChunks& c, const Scratch& s) {
+    constexpr size_t smem = OutSmem<KIND, DK, COLS, NT>::BYTES;
+    static_assert(smem <= 226 * 1024, "");
+    static SmemOptIn configured;
+    if (cudaError_t e = tsb_opt_in_smem(ctx, chunk_out_kernel<KIND, DK, COLS, NT>, smem, configured); e != cudaSuccess) return e;
+    return tsb_launch(ctx, chunk_out_kernel<KIND, DK, COLS, NT>, dim3((unsigned)((r.vdim + COLS - 1) / COLS), (unsigned)r.heads, (unsigned)c.chunks.n), dim3(NT), smem, st,
+                      true, r, c.chunks, s, ctx->dev_error);
+}
 template <int KIND, int DK>
 cudaError_t launch_chunks(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RecurrenceChunks& c) {
-    constexpr size_t out_smem = OutSmem<KIND, DK>::BYTES;
-    static SmemOptIn configured;
     const Scratch s = scratch_of(r, c.scratch, c.chunks.n);
     cudaError_t e = r.vdim > 64 ? launch_add<KIND, DK, 128>(ctx, st, r, c, s) : launch_add<KIND, DK, 64>(ctx, st, r, c, s);
-    if (e == cudaSuccess) e = tsb_opt_in_smem(ctx, chunk_out_kernel<KIND, DK>, out_smem, configured);
-    const dim3 grid((unsigned)((r.vdim + VB - 1) / VB), (unsigned)r.heads, (unsigned)c.chunks.n);
     const int items = r.dim * r.vdim / 4 + (KIND == REC_MLSTM ? r.dim : 0);
     if (e == cudaSuccess)
         e = tsb_launch(ctx, chunk_walk_kernel<KIND>, dim3((unsigned)((items + THREADS - 1) / THREADS), (unsigned)r.heads, (unsigned)c.n_portions), dim3(THREADS), 0, st, true,
                        r, c, s, ctx->dev_error);
-    if (e == cudaSuccess) e = tsb_launch(ctx, chunk_out_kernel<KIND, DK>, grid, dim3(THREADS), out_smem, st, true, r, c.chunks, s, ctx->dev_error);
-    return e;
+    if (e != cudaSuccess) return e;
+    if constexpr (KIND == REC_FORGET)  // the work on queries and keys is the larger part: all value columns share it
+        if (r.vdim > 64) return launch_out<KIND, DK, 128, 512>(ctx, st, r, c, s);
+    return launch_out<KIND, DK, 64, 256>(ctx, st, r, c, s);
 }
 template <int KIND>
 cudaError_t launch_chunks_dim(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RecurrenceChunks& c) {
