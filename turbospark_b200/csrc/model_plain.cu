@@ -470,6 +470,7 @@ int32_t plan_states(tsb_session* s, const PlainModel* m, const ModelRt& rt, cons
         const int32_t* dev = nullptr;
         if (int32_t rc = session_stage_ints(s, reinterpret_cast<const int32_t*>(list.data()), (int)list.size() * 2, &dev)) return rc;
         out = RowTiles::list(reinterpret_cast<const AttnTile*>(dev), (int)list.size());
+        for (const AttnTile& t : list) out.longest = std::max(out.longest, t.n_rows);
         return TSB_OK;
     };
     int32_t rc = stage(runs, plan.runs);
@@ -925,14 +926,14 @@ cudaError_t plain_forward(tsb_session* s, ModelRt& rt, const Pass& p) {
     if (m->cfg.output_norm) {
         FW(f.output_norm_layers(&x));
     } else {
-    FW(launch_plain_embed(ctx, st, m->f32, m->embed, m->cfg.vocab, d, p.tokens, p.token_stride, p.rows, m->cfg.embed_scale, b->x, post ? b->mix : nullptr,
-                          b->in_stride));
-    if (use_before) FW(launch_shift_before(ctx, st, b->shift, m->cfg.n_layers, p.rows_dev, p.rows));
-    for (size_t i = 0; i < m->rotations.size(); i++) {
-        const PlainRotation& r = m->rotations[i];
-        FW(launch_rotary_table(ctx, st, r.freq, r.dims / 2, r.magnitude, p.rows_dev, p.rows, b->rotary[i]));
-    }
-    for (int L = 0; L < m->cfg.n_layers; L++) FW(post ? f.post_norm_layer(L) : f.parallel_layer(L, use_before));
+        FW(launch_plain_embed(ctx, st, m->f32, m->embed, m->cfg.vocab, d, p.tokens, p.token_stride, p.rows, m->cfg.embed_scale, x, post ? b->mix : nullptr,
+                              b->in_stride));
+        if (use_before) FW(launch_shift_before(ctx, st, b->shift, m->cfg.n_layers, p.rows_dev, p.rows));
+        for (size_t i = 0; i < m->rotations.size(); i++) {
+            const PlainRotation& r = m->rotations[i];
+            FW(launch_rotary_table(ctx, st, r.freq, r.dims / 2, r.magnitude, p.rows_dev, p.rows, b->rotary[i]));
+        }
+        for (int L = 0; L < m->cfg.n_layers; L++) FW(post ? f.post_norm_layer(L) : f.parallel_layer(L, use_before));
     }
     if (p.logits) {
         const bool last = p.last_rows_only && p.rows_per_seq > 1;

@@ -1,19 +1,20 @@
 // Recurrent mixers row by row: decoded tokens, short portions, and every portion in f32.
 //
 // A CTA owns 32 value columns of one head of one portion; its slice of the state stays in registers over the portion's rows.  Eight
-// lanes hold four columns each, the CTA's 32 such groups of lanes share out the state's rows (CR each).  Rows go through in batches:
-// their q, k, v and gates are brought to shared memory, every thread steps through the batch without a barrier and leaves its part of
-// each output, then the parts are added.  Decays are applied as s + (decay - 1) s, with decay - 1 from expm1 or the gate itself: close to one
-// the rounding of the factor would add up over a long memory.  One batch of one row - a decoded token - reads and writes the state once.
+// lanes hold four columns each, the CTA's 32 such groups of lanes share out the state's rows (CR each).  Rows go through in batches of
+// eight (or one by one where every portion is a row): their q, k, v and gates are brought to shared memory, every thread steps through the
+// batch without a barrier and leaves its part of each output, then the parts are added.  Decays are applied as s + (decay - 1) s, with
+// decay - 1 from expm1 or the gate itself: close to one the rounding of the factor would add up over a long memory.  A decoded token reads and
+// writes the state once.
 #include <algorithm>
 
 #include "recurrence_dev.cuh"
 
 namespace {
 
-constexpr int THREADS = 256, COLS = REC_COLS, GROUPS = THREADS / 8, BATCH = 8;
+constexpr int THREADS = 256, COLS = REC_COLS, GROUPS = THREADS / 8;
 
-template <int KIND>
+template <int KIND, int BATCH>
 size_t rows_smem(int dim_pad) {
     return ((size_t)BATCH * dim_pad * 2 + BATCH * COLS + (size_t)BATCH * GROUPS * COLS + (KIND == REC_MLSTM ? BATCH * GROUPS : 0) + 3 * BATCH) *
            sizeof(float);
@@ -22,7 +23,7 @@ size_t rows_smem(int dim_pad) {
 // is the state after row t of the portion one of those that are kept?
 __device__ __forceinline__ bool is_kept(const Recurrence& a, const AttnTile& p, int t) { return t + a.state.ring >= p.n_rows; }
 
-template <typename T, int KIND, int CR>
+template <typename T, int KIND, int CR, int BATCH>
 __global__ void __launch_bounds__(THREADS) recurrence_rows_kernel(const __grid_constant__ Recurrence a, const __grid_constant__ RowTiles portions, uint32_t* __restrict__ err) {
     constexpr int DIM = GROUPS * CR;
     extern __shared__ __align__(16) float smem[];
@@ -159,14 +160,20 @@ __global__ void __launch_bounds__(THREADS) recurrence_rows_kernel(const __grid_c
     }
 }
 
-template <typename T, int KIND, int CR>
-cudaError_t launch_rows(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RowTiles& portions) {
-    const size_t smem = rows_smem<KIND>(GROUPS * CR);
+template <typename T, int KIND, int CR, int BATCH>
+cudaError_t launch_batch(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RowTiles& portions) {
+    const size_t smem = rows_smem<KIND, BATCH>(GROUPS * CR);
     static SmemOptIn configured;
     if (smem > 48 * 1024)
-        if (cudaError_t e = tsb_opt_in_smem(ctx, recurrence_rows_kernel<T, KIND, CR>, smem, configured); e != cudaSuccess) return e;
-    return tsb_launch(ctx, recurrence_rows_kernel<T, KIND, CR>, dim3((unsigned)recurrence_copies(r.vdim), (unsigned)r.heads, (unsigned)portions.n), dim3(THREADS),
+        if (cudaError_t e = tsb_opt_in_smem(ctx, recurrence_rows_kernel<T, KIND, CR, BATCH>, smem, configured); e != cudaSuccess) return e;
+    return tsb_launch(ctx, recurrence_rows_kernel<T, KIND, CR, BATCH>, dim3((unsigned)recurrence_copies(r.vdim), (unsigned)r.heads, (unsigned)portions.n), dim3(THREADS),
                       smem, st, true, r, portions, ctx->dev_error);
+}
+template <typename T, int KIND, int CR>
+cudaError_t launch_rows(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RowTiles& portions) {
+    if constexpr (sizeof(T) == 2 && CR <= 8)  // decoded tokens: little shared memory, more CTAs per SM
+        if (portions.longest == 1) return launch_batch<T, KIND, CR, 1>(ctx, st, r, portions);
+    return launch_batch<T, KIND, CR, 8>(ctx, st, r, portions);
 }
 template <typename T, int KIND>
 cudaError_t launch_dim(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RowTiles& portions) {

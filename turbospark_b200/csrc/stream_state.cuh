@@ -15,10 +15,11 @@ struct RowRing {
 struct RowTiles {
     const AttnTile* tiles = nullptr;
     int n = 0, rows_per_seq = 1, per_tile = 1, tiles_per_seq = 1;
+    int longest = 0;  // rows of the longest tile
     static RowTiles uniform(int rows, int rows_per_seq, int per_tile) {
         RowTiles t;
         t.rows_per_seq = rows_per_seq, t.per_tile = per_tile, t.tiles_per_seq = (rows_per_seq + per_tile - 1) / per_tile;
-        t.n = rows / rows_per_seq * t.tiles_per_seq;
+        t.n = rows / rows_per_seq * t.tiles_per_seq, t.longest = per_tile < rows_per_seq ? per_tile : rows_per_seq;
         return t;
     }
     static RowTiles list(const AttnTile* dev, int n) {
