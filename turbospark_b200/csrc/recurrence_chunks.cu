@@ -52,6 +52,7 @@ struct Scratch {
     float* norm;    // REC_MLSTM: the same for the normaliser, [dim]
     float* decay;   // REC_FORGET: E_T [dim]; REC_SSD: E_T; REC_MLSTM: log E_T, and the maximum the chunk's part is relative to
     double* top;    // REC_MLSTM: the running maximum before the chunk
+    float4* rows;   // decay per head: input scales and log E of rows 2 l and 2 l + 1, [32]
 };
 __host__ __device__ inline int decay_width(int kind, int dim) { return kind == REC_FORGET ? dim : 2; }
 size_t align16(size_t n) { return (n + 15) / 16 * 16; }
@@ -62,7 +63,8 @@ Scratch scratch_of(const Recurrence& r, void* p, int chunks) {
     s.add = reinterpret_cast<float*>(b), b += align16(n * r.dim * r.vdim * 4);
     s.norm = reinterpret_cast<float*>(b), b += align16(r.kind == REC_MLSTM ? n * r.dim * 4 : 0);
     s.decay = reinterpret_cast<float*>(b), b += align16(n * decay_width(r.kind, r.dim) * 4);
-    s.top = reinterpret_cast<double*>(b);
+    s.top = reinterpret_cast<double*>(b), b += align16(n * 8);
+    s.rows = reinterpret_cast<float4*>(b);
     return s;
 }
 
@@ -202,6 +204,7 @@ __global__ void __launch_bounds__(THREADS)
             w[0] = ex2((g.end - g.log_e[0]) * LOG2E) * g.in[0], w[1] = ex2((g.end - g.log_e[1]) * LOG2E) * g.in[1];
         }
         fv[2 * lane] = w[0], fv[2 * lane + 1] = w[1];
+        if (blockIdx.x == 0) out.rows[slot * 32 + lane] = make_float4(g.in[0], g.in[1], g.log_e[0], g.log_e[1]);
         if (blockIdx.x == 0 && lane == 0) {
             out.decay[slot * 2] = MLSTM ? g.end : expf(g.end);
             out.decay[slot * 2 + 1] = rel;
@@ -285,7 +288,7 @@ __global__ void __launch_bounds__(THREADS)
 // A thread owns four neighbouring numbers of a head's state and walks the chunks of the portion.  The running maximum after the portion is left to
 // the next launch: every thread reads the one before it.
 template <int KIND>
-__global__ void __launch_bounds__(THREADS)
+__global__ void __launch_bounds__(THREADS, 4)
     chunk_walk_kernel(const __grid_constant__ Recurrence a, const __grid_constant__ RecurrenceChunks c, const __grid_constant__ Scratch s, uint32_t* __restrict__ err) {
     constexpr bool FORGET = KIND == REC_FORGET, MLSTM = KIND == REC_MLSTM;
     const int per_seq = (c.rows_per_seq + C - 1) / C;
@@ -314,7 +317,7 @@ __global__ void __launch_bounds__(THREADS)
     pdl_wait();
     pdl_launch_dependents();
     if (i4 >= state4 && !is_norm) return;
-    constexpr int AHEAD = 8;
+    constexpr int AHEAD = 4;
     const int width = FORGET ? a.dim : 2;
     float4 next[AHEAD];
     float2 gate[AHEAD];
@@ -424,7 +427,8 @@ __global__ void __launch_bounds__(NT, NT > 256 ? 1 : DK > 128 || KIND == REC_FOR
         if (MLSTM)
             for (int i = threadIdx.x; i < DK; i += NT) norm[i] = i < a.dim ? in.norm[slot * a.dim + i] : 0.f;
         if (warp == 0) {
-            const RowGates g = row_gates<FORGET ? REC_SSD : KIND>(a, row0, n, head, lane);
+            const float4 kept = in.rows[slot * 32 + lane];
+            const RowGates g{{kept.x, kept.y}, {kept.z, kept.w}, __shfl_sync(0xffffffffu, kept.w, 31)};
             if (SSD) {
 #pragma unroll
                 for (int i = 0; i < 2; i++) ea[2 * lane + i] = g.log_e[i] * LOG2E, eb[2 * lane + i] = -g.log_e[i] * LOG2E, gain[2 * lane + i] = g.in[i];
@@ -781,7 +785,7 @@ bool recurrence_chunks_supported(int kind, int dim, int vdim) { return dim <= (k
 size_t recurrence_scratch_bytes(int kind, int heads, int dim, int vdim, int chunks) {
     if (!recurrence_chunks_supported(kind, dim, vdim)) return 0;
     const size_t n = (size_t)chunks * heads;
-    return align16(n * dim * vdim * 4) + align16(kind == REC_MLSTM ? n * dim * 4 : 0) + align16(n * decay_width(kind, dim) * 4) + n * 8;
+    return align16(n * dim * vdim * 4) + align16(kind == REC_MLSTM ? n * dim * 4 : 0) + align16(n * decay_width(kind, dim) * 4) + align16(n * 8) + (kind == REC_FORGET ? 0 : n * 32 * sizeof(float4));
 }
 
 cudaError_t launch_recurrence_chunks(tsb_ctx* ctx, cudaStream_t st, const Recurrence& r, const RecurrenceChunks& c) {
