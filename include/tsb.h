@@ -402,7 +402,7 @@ TSB_API int32_t tsb_router_logits(tsb_ctx* ctx, tsb_stream s, const void* q_u8, 
 /* ------------------------------------------------------------ plain-weight decoders
  * Decoders whose matrices are plain bfloat16 (or f32) and whose layers are put together from the mechanisms below; the
  * reference has no counterpart.  x starts as embed_scale (0: one) times the token's embedding, plus row p of a learned table at
- * position p (positions > 0: that many rows).  A layer has one of three forms:
+ * position p (positions > 0: that many rows).  A layer has one of four forms:
  *   parallel, one norm:   h = x * gain / sqrt(mean(x^2) + eps)                       one gain for all coordinates
  *                         x = x + mixer(shift(h)) + feed_forward(h)
  *   post_norm:            x = norm1(residual_scale * x + mixer(x)),  x = norm2(residual_scale * x + feed_forward(x))
@@ -410,6 +410,7 @@ TSB_API int32_t tsb_router_logits(tsb_ctx* ctx, tsb_stream s, const void* q_u8, 
  *   output_norm:          x = x + norm1(mixer(conv1(x))),  x = x + norm2(feed_forward(conv2(x)))
  *                         norm(y) = y * w / sqrt(mean(y^2) + eps), the mean over each of norm_groups (0: one) equal parts of y
  *                         conv(h)_t = h_t + sum_j w[:, j] * h_(t - conv_taps + 1 + j), zeros before the start (conv_taps 0: h itself)
+ *   pre_norm:             x = x + sublayer_scale * mixer(norm1(x)),  x = x + sublayer_scale * feed_forward(norm2(x)), norm as in post_norm; sublayer_scale 0: one
  *   shift (token_shift): h_t + (h_{t-1} - h_t) * mu, element by element; h_{-1} = 0
  *   mixer: causal attention, n_q_heads query heads over n_kv_heads key heads (see below for latent layers).
  *     value_dim = 0: the values are the keys; else values of value_dim columns with a projection of their own.
@@ -417,13 +418,18 @@ TSB_API int32_t tsb_router_logits(tsb_ctx* ctx, tsb_stream s, const void* q_u8, 
  *     q_temp_every > 0 (with qk_norm): q times 1 + q_temp_coef * ln(floor((p + 1) / q_temp_every) + 1) at position p;
  *     score = (q . k) * score_scale;  score_cap > 0: score = score_cap * tanh(score / score_cap);
  *     log_bias: score -= r1[head] * ln(1 + r2[head] * distance);  window > 0: the last `window` positions only;
- *     sink: exp(sink[head]) joins the softmax's denominator;
+ *     sink = TSB_SINK_TENSOR: exp(sink[head]) joins the softmax's denominator; TSB_SINK_ZERO: one does;
  *     head_gate: each head's output times sigmoid of one number per head, projected from the mixer's input;
  *     value_gate: every output column times sigmoid of a number of its own, projected from the mixer's input;
  *     in the output_norm form also: qkv_bias: q, k and v have biases; qk_norm = TSB_NORM_PROJECTION: queries, and keys, normed over all
  *     heads at once, a weight per row of the projection; linear_bias: score -= 2^(-8 (h + 1) / n_q_heads) * distance for head h; chunk > 0:
  *     a position sees the earlier ones of its own run of `chunk` positions, counted from position 0
- *   recurrent mixer (recurrence > 0, output_norm form): heads with a state S [rec_dim, rec_vdim] in f32,
+ *     in the pre_norm form also: qk_norm = TSB_NORM_PROJECTION; rot_dim > 0: behind the norms, coordinates i and i + rot_dim / 2 of every query and key head
+ *     (i below rot_dim / 2) are rotated by position * f_i, f_i = rot_base^(-2 i / rot_dim), divided by rot_factor when that is given; value_rot: values are
+ *     rotated over all their coordinates by position * rot_base^(-2 i / value_dim), cached so, and a head's output is rotated back by its own position;
+ *     before a window stay visible: keep_first: the first keep_first positions; pool > 0: a key and a value for every block of `pool` positions (b pool ..
+ *     b pool + pool - 1) that lies wholly before the window, the means of the block's cached ones
+ *   recurrent mixer (recurrence > 0; TSB_REC_MINGRU in the pre_norm form, the others in the output_norm form): heads with a state S [rec_dim, rec_vdim] in f32,
  *     S_t = decay_t S_(t-1) + k_t v_t^T, o_t = S_t^T q_t, starting from zero
  *     TSB_REC_FORGET: q = silu(W_q h), v = W_v h; per row of S: decay = f = l + (1 - l) sigmoid(W_f h + b_f), k = 1 - f; o normed per head
  *       (a weight per column, shared by the heads)
@@ -433,33 +439,39 @@ TSB_API int32_t tsb_router_logits(tsb_ctx* ctx, tsb_stream s, const void* q_u8, 
  *     TSB_REC_SSD: W_in h = z | x | B | C | dt; x, B, C (rec_groups of rec_dim columns) through a causal convolution per channel with
  *       bias and silu; dt = softplus(dt + b); decay = exp(-exp(A_log) dt), k = dt B, v = x, q = C; o + D x, times silu(z), normed in
  *       rec_norm_groups parts with a weight per column
- *     with n_q_heads > 0 as well the layer has both, side by side: attn_scale * attention + rec_scale * recurrence
+ *     TSB_REC_MINGRU (rec_heads = rec_dim = 1; rec_vdim channels): z = sigmoid(W_z h + b_z), u = W_x h + b_x, S_t = (1 - z) S_(t-1) + z c with c = u + 1/2 where
+ *       u >= 0 and sigmoid(u) elsewhere, times silu(W_g h), through W_o (TSB_P_REC_F: W_z, TSB_P_REC_I: W_x, TSB_P_REC_GATE: W_g)
+ *     with n_q_heads > 0 as well an output_norm layer has both, side by side: attn_scale * attention + rec_scale * recurrence
  *   latent mixer (kv_rank > 0): the cache holds per position c, kv_rank numbers projected and normed (plain weight), and one
  *     rotated key part of rot_dim columns for all heads.  Head: key = [W_uk c (head_dim), rotated part], value = W_uv c
  *     (value_dim), query = [head_dim plain, rot_dim rotated] columns.  Coordinates i and i + rot_dim / 2 are rotated by position * f_i,
  *     f_i = rot_base^(-2 i / rot_dim); rot_factor > 0 scales the frequencies between f_i and f_i / rot_factor by how often they
  *     turn within rot_original positions (rot_fast .. rot_slow turns), and cos and sin by 0.1 ln(rot_factor) + 1.
  *     kv_source = j + 1: the layer has no latent of its own and reads the one of layer j (0: its own).
- *   feed_forward (ffn > 0): W_down(act(W_gate h) * (W_up h)); a post_norm or output_norm layer without one has no norm2
+ *   feed_forward (ffn > 0): W_down(act(W_gate h) * (W_up h)), or - ff_plain, pre_norm form - W_down act(W_up h); a layer without one has no norm2
  *     experts > 0 (output_norm form): `experts` of them; s = sigmoid(W_router h), choice = s + correction; of expert_groups equal groups the
  *     expert_keep ones with the largest sum of their two largest choices stay, the expert_top largest choices in them are taken, and
  *     the sum of their outputs is weighted with s
+ *   weights_of = j + 1: the layer has no tensors and uses those of layer j, which it equals, with cache and state of its own (0: its own tensors)
  * then logits = W_head norm(x), through logit_cap * tanh(logits / logit_cap) when logit_cap > 0.
  * Residual stream, norms, shift, rotation, scores, softmax and gates are f32 in both modes.  compute = TSB_BF16: matrices,
  * activations and the cache in bfloat16 with f32 accumulation; TSB_F32: everything in f32.
  * Models with a token shift, a convolution or a recurrence keep per stream what the next row needs of the last rows of every layer (a
  * cursor can be moved back by max_rows rows after a pass of at most that many, or to 0).  Verify passes are chains; tree rounds are refused with TSB_ERR_UNSUPPORTED. */
 enum { TSB_BF16 = 0, TSB_F32 = 1 };
-enum { TSB_ACT_GELU_TANH = 0, TSB_ACT_SILU = 1 };
+enum { TSB_ACT_GELU_TANH = 0, TSB_ACT_SILU = 1, TSB_ACT_RELU2 = 2 }; /* RELU2: max(z, 0)^2 */
+enum { TSB_SINK_NONE = 0, TSB_SINK_TENSOR = 1, TSB_SINK_ZERO = 2 };
 typedef struct tsb_plain_config {
     int32_t n_layers, d_model, vocab, max_context, compute;
     float norm_eps, logit_cap;
     int32_t post_norm;
     float residual_scale, embed_scale;
     int32_t output_norm, norm_groups, conv_taps, positions;
+    int32_t pre_norm;
+    float sublayer_scale;
 } tsb_plain_config;
 enum { TSB_NORM_HEAD = 1, TSB_NORM_PROJECTION = 2 };                                   /* qk_norm */
-enum { TSB_REC_NONE = 0, TSB_REC_FORGET = 1, TSB_REC_MLSTM = 2, TSB_REC_SSD = 3 };      /* recurrence */
+enum { TSB_REC_NONE = 0, TSB_REC_FORGET = 1, TSB_REC_MLSTM = 2, TSB_REC_SSD = 3, TSB_REC_MINGRU = 4 }; /* recurrence */
 typedef struct tsb_plain_layer {
     int32_t n_q_heads, n_kv_heads, head_dim, window;
     float score_scale, score_cap;
@@ -467,7 +479,7 @@ typedef struct tsb_plain_layer {
     int32_t ffn, act;
     int32_t value_dim, qk_norm, q_temp_every;
     float q_temp_coef;
-    int32_t sink, value_gate; /* 0 / 1 */
+    int32_t sink, value_gate; /* TSB_SINK_*; 0 / 1 */
     int32_t kv_rank, rot_dim, kv_source;
     double rot_base, rot_factor, rot_original, rot_fast, rot_slow;
     int32_t qkv_bias, linear_bias, chunk;
@@ -475,10 +487,11 @@ typedef struct tsb_plain_layer {
     int32_t recurrence, rec_heads, rec_dim, rec_vdim, rec_groups, rec_taps, rec_norm_groups;
     float rec_cap;
     int32_t experts, expert_top, expert_groups, expert_keep;
+    int32_t keep_first, pool, value_rot, ff_plain, weights_of;
 } tsb_plain_layer;
 enum {
-    TSB_P_EMBED = 0, TSB_P_HEAD, TSB_P_FINAL_NORM,                     /* layer ignored; [vocab, d], [vocab, d], [1] (post_norm: [d]) */
-    TSB_P_NORM, TSB_P_SHIFT,                                           /* [1] (post_norm: norm1, [d]), [d] */
+    TSB_P_EMBED = 0, TSB_P_HEAD, TSB_P_FINAL_NORM,                     /* layer ignored; [vocab, d], [vocab, d], [1] (all forms but the parallel one: [d]) */
+    TSB_P_NORM, TSB_P_SHIFT,                                           /* [1] (all forms but the parallel one: norm1, [d]), [d] */
     TSB_P_Q, TSB_P_K, TSB_P_HEAD_GATE, TSB_P_R1, TSB_P_R2, TSB_P_O,    /* [H D, d], [G D, d], [H, d], [H], [H], [d, H D] */
     TSB_P_FF_GATE, TSB_P_FF_UP, TSB_P_FF_DOWN,                         /* [ffn, d], [ffn, d], [d, ffn] */
     TSB_P_NORM2, TSB_P_V, TSB_P_Q_NORM, TSB_P_K_NORM,                  /* [d], [G E, d], [D], [D] with E = value_dim */
@@ -489,8 +502,8 @@ enum {
     TSB_P_Q_BIAS, TSB_P_K_BIAS, TSB_P_V_BIAS,                          /* [H D], [G D], [G E]; projection norms: TSB_P_Q_NORM [H D], TSB_P_K_NORM [G D] */
     TSB_P_ROUTER, TSB_P_CORRECTION,                                    /* [experts, d], [experts]; TSB_P_FF_*: the experts' matrices one after another */
     TSB_P_REC_Q, TSB_P_REC_K, TSB_P_REC_V, TSB_P_REC_GATE,             /* [h D, d], [h D, d], [h E, d], [h E, d] with h, D, E = rec_heads, rec_dim, rec_vdim */
-    TSB_P_REC_F, TSB_P_REC_F_BIAS, TSB_P_REC_LOWER,                    /* FORGET: [h D, d], [h D], [h D]; MLSTM: [h, d], [h] */
-    TSB_P_REC_I, TSB_P_REC_I_BIAS, TSB_P_REC_NORM, TSB_P_REC_O,        /* [h, d], [h], [E] (FORGET) or [h E], [d, h E] */
+    TSB_P_REC_F, TSB_P_REC_F_BIAS, TSB_P_REC_LOWER,                    /* FORGET: [h D, d], [h D], [h D]; MLSTM: [h, d], [h]; MINGRU: [E, d], [E] */
+    TSB_P_REC_I, TSB_P_REC_I_BIAS, TSB_P_REC_NORM, TSB_P_REC_O,        /* [h, d], [h] (MINGRU: [E, d], [E]), [E] (FORGET) or [h E], [d, h E] */
     TSB_P_REC_IN, TSB_P_REC_CONV, TSB_P_REC_CONV_BIAS,                 /* SSD: [2 h E + 2 rec_groups D + h, d], [h E + 2 rec_groups D, rec_taps], ... */
     TSB_P_REC_DT_BIAS, TSB_P_REC_A_LOG, TSB_P_REC_D                    /* [h] each */
 };                                                                     /* with values: W_o [d, H E]; latent layers: W_q [H (D + rot_dim), d] */
@@ -530,6 +543,12 @@ TSB_API int32_t tsb_window_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, i
 TSB_API int32_t tsb_kv_create_plain(tsb_ctx* ctx, int32_t type, int32_t layers, int32_t kv_heads, int32_t key_dim, int32_t value_dim, int32_t page_tokens,
                                     int32_t num_pages, int32_t max_seqs, int32_t max_pages_per_seq, tsb_kv** out); /* value_dim 0: the values are the keys;
                                     else rows of [key, value] per head */
+/* The same with a row for every block of `pool` positions (0: none), shaped like the rows. */
+TSB_API int32_t tsb_kv_create_blocks(tsb_ctx* ctx, int32_t type, int32_t layers, int32_t kv_heads, int32_t key_dim, int32_t value_dim, int32_t pool, int32_t page_tokens,
+                                     int32_t num_pages, int32_t max_seqs, int32_t max_pages_per_seq, tsb_kv** out);
+/* The rows' blocks: where a row is the last position of a block, the block's row becomes the mean of the cached rows at its positions. */
+TSB_API int32_t tsb_block_mean_rows(tsb_ctx* ctx, tsb_stream s, tsb_kv* cache, int32_t layer, const tsb_row_desc* rows_dev, int32_t rows);
+TSB_API int32_t tsb_kv_read_blocks(tsb_kv* kv, tsb_stream s, int32_t seq, int32_t layer, int64_t block0, int32_t n, void* host);
 typedef struct tsb_attention_extras {
     float cap;                    /* > 0: soft cap */
     int32_t window;               /* > 0: sliding window */
@@ -541,6 +560,10 @@ typedef struct tsb_attention_extras {
     const float* slopes;          /* [n_q_heads] or NULL: score -= slope * distance (not with r1, r2) */
     int32_t chunk;                /* > 0: keys of the query's own run of `chunk` positions (not with a window) */
     float out_scale;              /* of the outputs; 0: one */
+    int32_t keep;                 /* > 0: the first `keep` positions stay visible before the window */
+    int32_t blocks;               /* 1: so do the cache's blocks (tsb_kv_create_blocks) that lie wholly before it */
+    const float* turn;            /* [rows, turn_half] of (cos, sin) or NULL: columns 2 m and 2 m + 1 of every output are turned back by them */
+    int32_t turn_half;
 } tsb_attention_extras;
 /* bfloat16 with keys and values of different widths: one query head per key head, keys of 64, 128 or 192, values of 64 or 128 columns. */
 TSB_API int32_t tsb_plain_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, int32_t layer, const void* q, int64_t q_stride, void* out,
@@ -565,6 +588,30 @@ TSB_API int32_t tsb_post_norm_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, flo
 TSB_API int32_t tsb_head_norm_rows(tsb_ctx* ctx, tsb_stream s, tsb_kv* cache, int32_t layer, const float* raw, int64_t raw_stride, int32_t n_q, int32_t n_k,
                                    int32_t width, const float* q_weight, const float* k_weight, float eps, float temp_coef, int32_t temp_every,
                                    const tsb_row_desc* rows_dev, int32_t rows, void* q, int64_t q_stride);
+/* The same without rewriting x. */
+TSB_API int32_t tsb_pre_norm_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, const float* x, int32_t d, const float* weight, float eps, int32_t rows, void* out,
+                                  int64_t out_stride);
+/* Norms of queries and keys, per head (projection = 0) or of whole projections, followed by rotations: columns 2 i and 2 i + 1 of every head turned by (cos, sin)
+ * of rot [rows, rot_half].  raw [rows, n_q * width | n_k * width | n_v * v_width] f32; values (n_v > 0, per head norms only) are turned by turn [rows, turn_half]
+ * and stored behind the keys.  Tables NULL: not turned. */
+typedef struct tsb_turned_norms {
+    int32_t projection, n_q, n_k, n_v, width, v_width, rot_half, turn_half;
+    const float *raw, *q_weight, *k_weight, *rot, *turn;
+    int64_t raw_stride, q_stride;
+    void* q;
+    float eps;
+} tsb_turned_norms;
+TSB_API int32_t tsb_turned_norm_rows(tsb_ctx* ctx, tsb_stream s, tsb_kv* cache, int32_t layer, const tsb_turned_norms* n, const tsb_row_desc* rows_dev, int32_t rows);
+/* minGRU (see TSB_REC_MINGRU): gate [rows, z pre-activations | u], out = S silu(out_gate), both in `type`; state [n_streams][ring][width rounded up to 4], position p in slot
+ * p & (ring - 1), ring a power of two above one.  Portions of rows_per_seq rows each; the states after a portion's last `ring` rows are kept. */
+TSB_API int32_t tsb_gated_scan_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, const float* gate, int64_t gate_stride, const void* out_gate, int64_t out_gate_stride,
+                                    int32_t width, float* state, int32_t n_streams, int32_t ring, const tsb_row_desc* rows_dev, int32_t rows, int32_t rows_per_seq,
+                                    void* out, int64_t out_stride);
+/* y[t, n] = act(sum_k W[n, k] x[t, k]) in `type`; and y[t, n] = alpha * y[t, n] + beta * sum in f32. */
+TSB_API int32_t tsb_plain_gemm_act(tsb_ctx* ctx, tsb_stream s, int32_t type, const void* w, int64_t rows, int64_t cols, const void* x, int32_t x_rows, int32_t tokens,
+                                   void* y, int64_t y_stride, int32_t n_valid, int32_t act, void* workspace);
+TSB_API int32_t tsb_plain_gemm_add(tsb_ctx* ctx, tsb_stream s, int32_t type, const void* w, int64_t rows, int64_t cols, const void* x, int32_t x_rows, int32_t tokens,
+                                   float* y, int64_t y_stride, int32_t n_valid, float alpha, float beta, void* workspace);
 /* The end of an output-norm sublayer and the convolution in front of the next: x_out = x_in + norm(y) in f32 (norm in `groups` equal parts, weight
  * [d]); out = x_out + convolution of it in `type` (taps_w [taps][d], taps 0: not written).  Portions of rows_per_seq rows each.  state: f32
  * [n_streams][ring][d], ring a power of two: x_out of the rows before and of this call's last rows.  Portions of more than ring - taps + 1

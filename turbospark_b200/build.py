@@ -29,8 +29,8 @@ FLAGS = [
 # Units of one model family only; a library of one family leaves the other's out (build(family=...)).
 FAMILY_UNITS = {
     "blocks": {"attention.cu", "attention_tc.cu", "comm.cu", "gemm_quant.cu", "gemm_wide.cu", "model_blocks.cu", "moe.cu", "resident.cu", "rowops.cu"},
-    "plain": {"attention_kv.cu", "attention_kv_tc.cu", "attention_latent.cu", "attention_window.cu", "attention_window_tc.cu", "experts.cu", "gemm_plain.cu",
-              "model_plain.cu", "ops_plain.cu", "recurrence.cu", "recurrence_chunks.cu", "rowops_plain.cu", "sublayer.cu"},
+    "plain": {"attention_kv.cu", "attention_kv_tc.cu", "attention_latent.cu", "attention_prefix.cu", "attention_prefix_tc.cu", "attention_window.cu", "attention_window_tc.cu", "experts.cu", "gemm_plain.cu",
+              "model_plain.cu", "ops_plain.cu", "recurrence.cu", "recurrence_chunks.cu", "rowops_plain.cu", "scan.cu", "sublayer.cu"},
 }
 
 

@@ -481,19 +481,25 @@ class ExpertLists:
 
 class AttentionExtras(C.Structure):
     _fields_ = [("cap", C.c_float), ("window", C.c_int32)] + [(n, C.c_void_p) for n in ("r1", "r2", "head_gate", "sink", "value_gate")] + \
-               [("value_gate_stride", C.c_int64), ("slopes", C.c_void_p), ("chunk", C.c_int32), ("out_scale", C.c_float)]
+               [("value_gate_stride", C.c_int64), ("slopes", C.c_void_p), ("chunk", C.c_int32), ("out_scale", C.c_float), ("keep", C.c_int32), ("blocks", C.c_int32),
+                ("turn", C.c_void_p), ("turn_half", C.c_int32)]
+
+
+class TurnedNorms(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in ("projection", "n_q", "n_k", "n_v", "width", "v_width", "rot_half", "turn_half")] + \
+               [(n, C.c_void_p) for n in ("raw", "q_weight", "k_weight", "rot", "turn")] + [("raw_stride", C.c_int64), ("q_stride", C.c_int64), ("q", C.c_void_p), ("eps", C.c_float)]
 
 
 class PlainCache(KvCache):
     """A plain cache: rows of kv_heads * [key, value] (value_dim 0: the values are the keys), bfloat16 bit patterns (type 0) or f32
-    values (type 1)."""
+    values (type 1).  pool > 0: beside them a row for every block of so many positions."""
 
-    def __init__(self, ctx, type_, layers, kv_heads, key_dim, value_dim, page_tokens, num_pages, max_seqs, max_pages_per_seq):
+    def __init__(self, ctx, type_, layers, kv_heads, key_dim, value_dim, page_tokens, num_pages, max_seqs, max_pages_per_seq, pool=0):
         self.ctx, self.type = ctx, type_
         self.layers, self.kv_heads, self.head_dim = layers, kv_heads, key_dim + value_dim
         h = C.c_void_p()
-        ctx.check(lib().tsb_kv_create_plain(ctx.h, C.c_int32(type_), C.c_int32(layers), C.c_int32(kv_heads), C.c_int32(key_dim), C.c_int32(value_dim),
-                                            C.c_int32(page_tokens), C.c_int32(num_pages), C.c_int32(max_seqs), C.c_int32(max_pages_per_seq), C.byref(h)))
+        ctx.check(lib().tsb_kv_create_blocks(ctx.h, C.c_int32(type_), C.c_int32(layers), C.c_int32(kv_heads), C.c_int32(key_dim), C.c_int32(value_dim),
+                                            C.c_int32(pool), C.c_int32(page_tokens), C.c_int32(num_pages), C.c_int32(max_seqs), C.c_int32(max_pages_per_seq), C.byref(h)))
         self.h = h
 
     def write_rows(self, seq, layer, pos0, k, stream=None):
@@ -504,6 +510,11 @@ class PlainCache(KvCache):
     def read_rows(self, seq, layer, pos0, n, stream=None):
         k = np.empty((n, self.kv_heads * self.head_dim), dtype=np.float32 if self.type else np.uint16)
         self.ctx.check(lib().tsb_kv_read_rows(self.h, stream, C.c_int32(seq), C.c_int32(layer), C.c_int64(pos0), C.c_int32(n), _vp(k), None))
+        return k
+
+    def read_blocks(self, seq, layer, block0, n, stream=None):
+        k = np.empty((n, self.kv_heads * self.head_dim), dtype=np.float32 if self.type else np.uint16)
+        self.ctx.check(lib().tsb_kv_read_blocks(self.h, stream, C.c_int32(seq), C.c_int32(layer), C.c_int64(block0), C.c_int32(n), _vp(k)))
         return k
 
 

@@ -1,5 +1,5 @@
 // Attention over a plain paged cache (attention_window.cuh): this unit has the kernels for caches whose values are their keys, the
-// f32 kernel and the merge; attention_kv.cu has the kernels for caches with values of their own.
+// f32 kernel and the merge; attention_kv.cu has the kernels for caches with values of their own, attention_prefix.cu those with a prefix.
 //
 // bfloat16: one kernel template <D, MT, SL> on mma.sync m16n8k16.  A CTA owns one (query tile, key head, run of key tiles):
 // MT m-tiles of 16 queries - the tile's rows x the heads that share the key head - and walks 64-token key tiles that
@@ -77,6 +77,7 @@ __global__ void __launch_bounds__(256)
                     acc.x = fmaf(x.x, w, acc.x), acc.y = fmaf(x.y, w, acc.y), acc.z = fmaf(x.z, w, acc.z), acc.w = fmaf(x.w, w, acc.w);
                 }
             }
+            if (c < D && a.turn) turn_back(a, row_first + r, c, acc.x, acc.y), turn_back(a, row_first + r, c + 2, acc.z, acc.w);
             if (c < D && a.value_gate) value_gates(a, row_first + r, head, c, acc);
             if (c < D) *reinterpret_cast<uint2*>(out + c) = make_uint2(pack_bf16(acc.x * f, acc.y * f), pack_bf16(acc.z * f, acc.w * f));
         }
@@ -108,10 +109,14 @@ __global__ void __launch_bounds__(F32_WARPS * 32) window_attn_f32_kernel(const _
     float m = a.sink ? a.sink[head] : -INFINITY, l = a.sink ? 1.f : 0.f, acc[F32_MAX_DIM / 32];
 #pragma unroll
     for (int i = 0; i < F32_MAX_DIM / 32; i++) acc[i] = 0.f;
-    for (int j0 = lo & ~31; j0 <= pos; j0 += 32) {
-        const int j = j0 + lane;
-        const bool seen = j >= lo && j <= pos;
-        const float* k = seen ? key_row<float>(a.keys, rd.seq, j) : nullptr;
+    // first what is seen of the prefix, then the window
+    const int n_pre = a.window > 0 && (a.keep > 0 || a.pool > 0) ? prefix_len(a, pos) : 0, pre_end = (n_pre + 31) & ~31;
+    for (int i0 = 0; i0 < pre_end + pos + 1 - (lo & ~31); i0 += 32) {
+        const bool pre = i0 < pre_end;
+        const int j0 = pre ? i0 : i0 - pre_end + (lo & ~31), j = j0 + lane;
+        const KeyView& rows_of = pre && a.pool > 0 ? a.pooled : a.keys;
+        const bool seen = pre ? j < n_pre : j >= lo && j <= pos;
+        const float* k = seen ? key_row<float>(rows_of, rd.seq, j) : nullptr;
         if (seen && !k) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
         float s = -INFINITY;
         if (k) {
@@ -143,7 +148,7 @@ __global__ void __launch_bounds__(F32_WARPS * 32) window_attn_f32_kernel(const _
         for (int t = 0; t < 32; t++) {
             const float pt = __shfl_sync(0xffffffffu, p, t);
             if (pt == 0.f) continue;  // the same for every lane
-            const float* kt = key_row<float>(a.keys, rd.seq, j0 + t);
+            const float* kt = key_row<float>(rows_of, rd.seq, j0 + t);
             if (!kt) continue;
             kt += (int64_t)kvh * a.keys.head_step + a.keys.value_off;
 #pragma unroll
@@ -156,7 +161,15 @@ __global__ void __launch_bounds__(F32_WARPS * 32) window_attn_f32_kernel(const _
     const float* vg = a.value_gate ? reinterpret_cast<const float*>(a.value_gate) + (int64_t)row * a.value_gate_stride + (int64_t)head * DV : nullptr;
 #pragma unroll
     for (int i = 0; i < F32_MAX_DIM / 32; i++)
-        if (i * 32 + lane < DV) out[i * 32 + lane] = acc[i] * f * (vg ? sigmoid(vg[i * 32 + lane]) : 1.f);
+        if (i * 32 < DV) {
+            float v = acc[i];
+            if (a.turn) {  // the columns of a pair sit in neighbouring lanes
+                float u = __shfl_xor_sync(0xffffffffu, v, 1);
+                if (lane & 1) turn_back(a, row, i * 32 + lane - 1, u, v);
+                else turn_back(a, row, i * 32 + lane, v, u);
+            }
+            if (i * 32 + lane < DV) out[i * 32 + lane] = v * f * (vg ? sigmoid(vg[i * 32 + lane]) : 1.f);
+        }
 }
 
 }  // namespace
@@ -186,16 +199,19 @@ int wattn_pad_dim(int head_dim, bool f32) {
 bool wattn_supported(int head_dim, int group, bool f32) { return wattn_pad_dim(head_dim, f32) > 0 && group >= 1 && (f32 || group <= WATTN_LARGE_Q); }
 
 cudaError_t launch_window_attn(tsb_ctx* ctx, cudaStream_t st, bool f32, const WindowAttn& a, const AttnBatch& b, void* scratch) {
+    if (has_prefix(a) && (a.window <= 0 || a.keys.value_off == 0 || a.r1 || a.slopes || (a.keep > 0 && a.pool > 0))) return cudaErrorInvalidValue;
     if (f32)
         return tsb_launch(ctx, window_attn_f32_kernel, dim3((unsigned)(((int64_t)b.rows * a.n_q_heads + F32_WARPS - 1) / F32_WARPS)), dim3(F32_WARPS * 32),
                           0, st, true, a, b.rows, ctx->dev_error);
     const int grp = a.n_q_heads / a.keys.kv_heads, rpt = wattn_rows_per_tile(a.keys.head_dim, grp, a.r1 != nullptr);
-    const bool kv = a.keys.value_off > 0;
+    const bool kv = a.keys.value_off > 0, pre = has_prefix(a);
     auto large = [&](const WattnLaunch& l) {
-        if (wattn_tc_supported(a.keys.head_dim, grp, a.r1 != nullptr)) return (kv ? launch_kv_attn_tc : launch_window_attn_tc)(ctx, st, a, l, scratch);
+        if (wattn_tc_supported(a.keys.head_dim, grp, a.r1 != nullptr)) return (pre ? launch_prefix_attn_tc : kv ? launch_kv_attn_tc : launch_window_attn_tc)(ctx, st, a, l, scratch);
+        if (pre) return launch_prefix_attn_large(ctx, st, a, l, scratch);
         return kv ? launch_kv_attn_large(ctx, st, a, l, scratch) : launch_large<8, 1, false>(ctx, st, a, l, scratch);
     };
     auto small = [&](const WattnLaunch& l, int queries) {
+        if (pre) return launch_prefix_attn_small(ctx, st, a, l, queries, scratch);
         return kv ? launch_kv_attn_small(ctx, st, a, l, queries, scratch) : launch_small<false>(ctx, st, a, l, queries, scratch);
     };
     if (b.rows_per_seq > 0) {

@@ -1,6 +1,7 @@
 // Attention over a plain paged cache - a layer's values are its keys, or stand behind them - with a sliding window
-// or a chunk mask, a soft cap on the scores, a per-head logarithmic or linear distance bias, a per-head sink, and output gates per head
-// or per value column - each of them optional.
+// or a chunk mask, a prefix that stays visible beside the window (kept first tokens, or means of the blocks before it), a soft cap on the
+// scores, a per-head logarithmic or linear distance bias, a per-head sink, values that turn with their position, and output gates per
+// head or per value column - each of them optional.
 #pragma once
 #include <cuda_bf16.h>
 
@@ -21,10 +22,18 @@ struct WindowAttn {
     const float* slopes = nullptr;             // per head: score <- score - slope * distance; null: no such bias (not with r1)
     int chunk = 0;            // > 0: a query sees the positions of its own chunk (counted from position 0) up to itself; not with a window
     int window = 0;           // a query sees itself and the window - 1 positions before it; 0: every earlier position
+    // What stays visible before the window (window > 0, values of their own, no distance bias): the stream's first `keep` positions, or - pool > 0 -
+    // a row of `pooled` for each block of `pool` positions that lies wholly before the window.
+    int keep = 0, pool = 0;
+    KeyView pooled{};             // shaped like keys but for its pages
     const float* sink = nullptr;  // per head: exp(sink) joins the softmax's denominator
     // [rows, n_q_heads * value columns], the compute type: a head's output is multiplied by the sigmoid, column by column
     const void* value_gate = nullptr;
     int64_t value_gate_stride = 0;
+    // values that turn with their position: (cos, sin) of [rows, turn_half] at the rows' positions; columns 2 m and 2 m + 1 of a head's output
+    // are turned back by them, before any gate
+    const float2* turn = nullptr;
+    int turn_half = 0;
     float out_scale = 1.f;    // of the heads' outputs
     int value_dim = 0;        // value columns (the heads of out and value_gate are as wide); 0: as many as a key has
 };

@@ -37,6 +37,27 @@ __device__ __forceinline__ float head_factor(const WindowAttn& a, int row, int h
 __device__ __forceinline__ int first_visible(const WindowAttn& a, int pos) {
     return a.window > 0 ? max(0, pos - a.window + 1) : a.chunk > 0 ? pos - pos % a.chunk : 0;
 }
+// How much of the prefix - kept positions, or blocks - a query at `pos` sees: all of it that lies before the window.
+__host__ __device__ __forceinline__ int prefix_len(const WindowAttn& a, int pos) {
+    const int before = pos - a.window + 1;  // positions before the window
+    return before <= 0 ? 0 : a.pool > 0 ? before / a.pool : before < a.keep ? before : a.keep;
+}
+// Row i of the prefix, or position i of the stream; nullptr outside the reserved pages.
+__device__ __forceinline__ const __nv_bfloat16* run_row(const WindowAttn& a, bool prefix, int seq, int i) {
+    const bool pooled = prefix && a.pool > 0;
+    const int shift = pooled ? a.pooled.page_shift : a.keys.page_shift, lp = i >> shift;
+    if (i < 0 || lp >= a.keys.max_pages_per_seq) return nullptr;
+    const int page = a.keys.page_table[(size_t)seq * a.keys.max_pages_per_seq + lp];
+    if (page < 0) return nullptr;
+    return reinterpret_cast<const __nv_bfloat16*>(pooled ? a.pooled.base : a.keys.base) + (((int64_t)page << shift) + (i & ((1 << shift) - 1))) * a.keys.row;
+}
+// The output columns c and c + 1 (c even) of a row, turned back to the row's position.
+__device__ __forceinline__ void turn_back(const WindowAttn& a, int row, int c, float& u, float& v) {
+    if (c >= 2 * a.turn_half) return;
+    const float2 t = a.turn[(int64_t)row * a.turn_half + (c >> 1)];
+    const float x = fmaf(u, t.x, v * t.y);
+    v = fmaf(v, t.x, -u * t.y), u = x;
+}
 // how many positions, itself included, a query at `pos` sees at most (a number no distance reaches: all of them)
 __device__ __forceinline__ float visible_span(const WindowAttn& a, int pos) {
     return a.window > 0 ? (float)a.window : a.chunk > 0 ? (float)(pos % a.chunk + 1) : 3e38f;
@@ -97,6 +118,8 @@ struct ScoreConst {
     }
 };
 
+inline bool has_prefix(const WindowAttn& a) { return a.keep > 0 || a.pool > 0; }
+
 constexpr int WATTN_TICKETS = 16384;
 constexpr int WATTN_MAX_SPLITS = 64;
 
@@ -123,10 +146,10 @@ inline WattnScratch wattn_scratch(const tsb_ctx* ctx, void* p) {
 // How many runs the key tiles of a launch are cut into: the number whose waves come out most even.  base: CTAs of an uncut
 // launch; a CTA costs its key tiles plus about three tiles' time of fixed work, a cut tile also the merge of its runs.
 inline int wattn_splits(const tsb_ctx* ctx, int window, const WattnLaunch& l, int tile_tokens, int queries_per_cta, int ctas_per_sm, int base,
-                        size_t part_queries) {
+                        size_t part_queries, int prefix = 0) {
     const int sms = ctx->sm_count > 0 ? ctx->sm_count : 148;
     const int span = window > 0 && window + l.rows_per_tile < l.max_len ? window + l.rows_per_tile : l.max_len;
-    const int key_tiles = (span + tile_tokens - 1) / tile_tokens + (window > 0 ? 1 : 0);
+    const int key_tiles = (span + tile_tokens - 1) / tile_tokens + (window > 0 ? 1 : 0) + (prefix + tile_tokens - 1) / tile_tokens;
     int splits = 1;
     float best = 1e30f;
     for (int s = 1; s <= WATTN_MAX_SPLITS && s <= (key_tiles + 1) / 2; s++) {
@@ -138,7 +161,8 @@ inline int wattn_splits(const tsb_ctx* ctx, int window, const WattnLaunch& l, in
     return splits;
 }
 inline int wattn_splits(const tsb_ctx* ctx, const WindowAttn& a, const WattnLaunch& l, int tile_tokens, int queries_per_cta, int ctas_per_sm) {
-    return wattn_splits(ctx, a.window > 0 ? a.window : a.chunk, l, tile_tokens, queries_per_cta, ctas_per_sm, l.n_tiles * a.keys.kv_heads, wattn_part_queries(ctx));
+    return wattn_splits(ctx, a.window > 0 ? a.window : a.chunk, l, tile_tokens, queries_per_cta, ctas_per_sm, l.n_tiles * a.keys.kv_heads, wattn_part_queries(ctx),
+                        a.window > 0 && has_prefix(a) ? prefix_len(a, l.max_len - 1) : 0);
 }
 
 // Adds the runs of cut tiles, in order, and writes the finished rows.  A tile has `slots` query slots per run: row r of the
@@ -153,3 +177,7 @@ cudaError_t launch_window_attn_tc(tsb_ctx* ctx, cudaStream_t st, const WindowAtt
 cudaError_t launch_kv_attn_small(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, int queries, void* scratch);
 cudaError_t launch_kv_attn_large(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch);
 cudaError_t launch_kv_attn_tc(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch);
+// The same with a prefix before the window (attention_prefix.cu, attention_prefix_tc.cu).
+cudaError_t launch_prefix_attn_small(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, int queries, void* scratch);
+cudaError_t launch_prefix_attn_large(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch);
+cudaError_t launch_prefix_attn_tc(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch);

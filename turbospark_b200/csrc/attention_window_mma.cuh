@@ -1,6 +1,7 @@
 // The mma.sync attention kernels over a plain paged cache (attention_window.cu describes them).  Instantiated once for
 // caches whose values are their keys (KV = false: a key tile serves both products) and once for caches with values of their own
-// (KV = true: a stage of the ring holds a key tile and a value tile).
+// (KV = true: a stage of the ring holds a key tile and a value tile).  PRE: the prefix before the window goes first, in key tiles of its own;
+// its rows are counted from zero, and a query sees those below its own number of them.
 #pragma once
 #include "attention_window_dev.cuh"
 #include "mma_dev.cuh"
@@ -83,6 +84,7 @@ __device__ __forceinline__ void finish_slices(const WindowAttn& a, int row_first
     auto store = [&](int qi, int c, float4 v, float m, float l) {
         const int row = row_first + qi / grp, head = kvh * grp + qi % grp;
         const float f = head_factor(a, row, head, m, l);
+        if (a.turn) turn_back(a, row, c, v.x, v.y), turn_back(a, row, c + 2, v.z, v.w);
         if (a.value_gate) value_gates(a, row, head, c, v);
         *reinterpret_cast<uint2*>(reinterpret_cast<__nv_bfloat16*>(a.out) + (int64_t)row * a.out_stride + head * D + c) =
             make_uint2(pack_bf16(v.x * f, v.y * f), pack_bf16(v.z * f, v.w * f));
@@ -146,7 +148,7 @@ constexpr size_t wattn_smem() {
     return ring > merge ? ring : merge;
 }
 
-template <int D, int MT, int SL, bool KV>
+template <int D, int MT, int SL, bool KV, bool PRE>
 __global__ void __launch_bounds__(32 * MT * SL, MT * SL <= 4 ? 3 : 1)
     window_attn_kernel(const __grid_constant__ WindowAttn a, const AttnTile* __restrict__ tiles, int tiles_per_group, int rows_per_seq, int rows_per_tile,
                        float* __restrict__ part_o, float2* __restrict__ part_ml, uint32_t* __restrict__ tickets, uint32_t* __restrict__ err) {
@@ -180,17 +182,20 @@ __global__ void __launch_bounds__(32 * MT * SL, MT * SL <= 4 ? 3 : 1)
     // visible positions of the tile's queries, in whole key tiles; this CTA's run of them
     const int lo = first_visible(a, pos0) & ~(TOK - 1);
     const int hi = pos0 + n_rows, lo_last = first_visible(a, hi - 1);
-    const int total = (hi - lo + TOK - 1) / TOK;
+    const int n_pre = PRE ? prefix_len(a, hi - 1) : 0, pre_all = PRE ? prefix_len(a, pos0) : 0;  // of the prefix: seen by some row, by every row
+    const int pre_tiles = (n_pre + TOK - 1) / TOK;
+    const int total = pre_tiles + (hi - lo + TOK - 1) / TOK;
     const int per = (total + n_splits - 1) / n_splits;
     const int t_first = min(total, (int)blockIdx.x * per), n_tiles = min(total, t_first + per) - t_first;
-    const int begin = lo + t_first * TOK;
+    const int begin = lo + (t_first - pre_tiles) * TOK;
 
     const uint32_t ring = smem_u32(smem);
     auto issue = [&](int tile, int stage) {
         constexpr int TPR = NTHR / TOK;  // threads per token row
         const int r = threadIdx.x / TPR, part = threadIdx.x % TPR;
-        const int pos = begin + tile * TOK + r;
-        const __nv_bfloat16* src = pos < hi ? key_row<__nv_bfloat16>(a.keys, seq, pos) : nullptr;
+        const bool pre = PRE && t_first + tile < pre_tiles;
+        const int pos = (pre ? (t_first + tile) * TOK : begin + tile * TOK) + r;
+        const __nv_bfloat16* src = pos >= (pre ? n_pre : hi) ? nullptr : PRE ? run_row(a, pre, seq, pos) : key_row<__nv_bfloat16>(a.keys, seq, pos);
         const bool ok = src != nullptr;
         src = ok ? src + (int64_t)kvh * a.keys.head_step : reinterpret_cast<const __nv_bfloat16*>(a.keys.base);
         const uint32_t dst = ring + stage * STAGE;
@@ -210,7 +215,8 @@ __global__ void __launch_bounds__(32 * MT * SL, MT * SL <= 4 ? 3 : 1)
         }
     };
     // key tiles of earlier passes may start moving while the kernel that writes this pass's rows still runs
-    const bool early = begin + NST * TOK <= rd0.base;
+    // (a prefix: rows of positions before this pass)
+    const bool early = begin + NST * TOK <= rd0.base && (!PRE || min(n_pre, (t_first + NST) * TOK) * max(a.pool, 1) <= rd0.base);
     if (early) prologue();
     pdl_wait();
     if (!early) prologue();
@@ -266,7 +272,8 @@ __global__ void __launch_bounds__(32 * MT * SL, MT * SL <= 4 ? 3 : 1)
         __syncthreads();
         const uint32_t kt = ring + stage * STAGE, vt = kt + V_AT;
         const int tok0 = sl * WTOK;
-        const int p0 = begin + tile * TOK + tok0;
+        const bool pre = PRE && t_first + tile < pre_tiles;
+        const int p0 = (pre ? (t_first + tile) * TOK : begin + tile * TOK) + tok0;
         float s[NT8][4];
 #pragma unroll
         for (int n = 0; n < NT8; n++)
@@ -297,10 +304,14 @@ __global__ void __launch_bounds__(32 * MT * SL, MT * SL <= 4 ? 3 : 1)
             }
         }
         // the mask only where the tile meets an edge
-        const bool edge = p0 + WTOK > pos0 || p0 < lo_last;
-        float mx[2] = {-INFINITY, -INFINITY};
-        const float db[2] = {(float)(pq[0] - p0 - 2 * tig), (float)(pq[1] - p0 - 2 * tig)};
-        base2_logits<NT8, false>(s, a, sc, db, r1, r2, span, edge, mx);
+        const bool edge = pre ? p0 + WTOK > pre_all : p0 + WTOK > pos0 || p0 < lo_last;
+        float mx[2] = {-INFINITY, -INFINITY}, db[2], sp[2];
+#pragma unroll
+        for (int h = 0; h < 2; h++) {
+            const int last = pre ? prefix_len(a, pq[h]) - 1 : pq[h];  // the last one that the query sees
+            db[h] = (float)(last - p0 - 2 * tig), sp[h] = pre ? 3e38f : span[h];
+        }
+        base2_logits<NT8, false>(s, a, sc, db, r1, r2, sp, edge, mx);
         float alpha[2], m_use[2];
 #pragma unroll
         for (int h = 0; h < 2; h++) {
@@ -366,6 +377,7 @@ __global__ void __launch_bounds__(32 * MT * SL, MT * SL <= 4 ? 3 : 1)
 #pragma unroll
                 for (int n = 0; n < NO; n++) {
                     float2 v = make_float2(o[n][2 * h] * f, o[n][2 * h + 1] * f);
+                    if (a.turn) turn_back(a, row, n * 8 + 2 * tig, v.x, v.y);
                     if (a.value_gate) v.x *= value_gate(a, row, head, n * 8 + 2 * tig), v.y *= value_gate(a, row, head, n * 8 + 2 * tig + 1);
                     *reinterpret_cast<uint32_t*>(p + n * 8 + 2 * tig) = pack_bf16(v.x, v.y);
                 }
@@ -413,7 +425,7 @@ struct FewQ {
     static constexpr int PER_SM = D > 128 ? 2 : NQ == 1 ? 4 : NQ == 2 ? 3 : 2;
 };
 
-template <int D, int NQ, bool KV>
+template <int D, int NQ, bool KV, bool PRE>
 __global__ void __launch_bounds__(128, FewQ<D, NQ, KV>::PER_SM)
     window_attn_few_kernel(const __grid_constant__ WindowAttn a, const AttnTile* __restrict__ tiles, int rows_per_seq, float* __restrict__ part_o,
                         float2* __restrict__ part_ml, uint32_t* __restrict__ tickets, uint32_t* __restrict__ err) {
@@ -437,17 +449,20 @@ __global__ void __launch_bounds__(128, FewQ<D, NQ, KV>::PER_SM)
     // key tiles start at multiples of 64 positions; this CTA's run of them
     const int lo = first_visible(a, pos0) & ~63;
     const int hi = pos0 + n_rows, lo_last = first_visible(a, hi - 1);
-    const int total = (hi - lo + F::TILE - 1) / F::TILE;
+    const int n_pre = PRE ? prefix_len(a, hi - 1) : 0, pre_all = PRE ? prefix_len(a, pos0) : 0;  // of the prefix: seen by some row, by every row
+    const int pre_tiles = (n_pre + F::TILE - 1) / F::TILE;
+    const int total = pre_tiles + (hi - lo + F::TILE - 1) / F::TILE;
     const int per = (total + n_splits - 1) / n_splits;
     const int t_first = min(total, (int)blockIdx.x * per), n_tiles = min(total, t_first + per) - t_first;
-    const int begin = lo + t_first * F::TILE;
+    const int begin = lo + (t_first - pre_tiles) * F::TILE;
 
     const uint32_t ring = smem_u32(smem);
     auto issue = [&](int tile, int stage) {
         constexpr int TPR = 128 / F::TILE;  // threads per token row
         const int r = threadIdx.x / TPR, part = threadIdx.x % TPR;
-        const int pos = begin + tile * F::TILE + r;
-        const __nv_bfloat16* src = pos < hi ? key_row<__nv_bfloat16>(a.keys, seq, pos) : nullptr;
+        const bool pre = PRE && t_first + tile < pre_tiles;
+        const int pos = (pre ? (t_first + tile) * F::TILE : begin + tile * F::TILE) + r;
+        const __nv_bfloat16* src = pos >= (pre ? n_pre : hi) ? nullptr : PRE ? run_row(a, pre, seq, pos) : key_row<__nv_bfloat16>(a.keys, seq, pos);
         const bool ok = src != nullptr;
         src = ok ? src + (int64_t)kvh * a.keys.head_step : reinterpret_cast<const __nv_bfloat16*>(a.keys.base);
         const uint32_t dst = ring + stage * F::STAGE;
@@ -466,7 +481,8 @@ __global__ void __launch_bounds__(128, FewQ<D, NQ, KV>::PER_SM)
             else cp_async_commit();
         }
     };
-    const bool early = begin + NST * F::TILE <= rd0.base;  // key tiles of earlier passes
+    // key tiles of earlier passes, prefix rows of their positions
+    const bool early = begin + NST * F::TILE <= rd0.base && (!PRE || min(n_pre, (t_first + NST) * F::TILE) * max(a.pool, 1) <= rd0.base);
     if (early) prologue();
     // score columns of this lane: queries 2 tig and 2 tig + 1 of every query tile
     int pq[NQ][2];
@@ -511,7 +527,8 @@ __global__ void __launch_bounds__(128, FewQ<D, NQ, KV>::PER_SM)
         cp_async_wait<NST - 1>();
         __syncthreads();
         const uint32_t kt = ring + stage * F::STAGE, vt = kt + F::V_AT;
-        const int tok0 = warp * F::WTOK, p0 = begin + tile * F::TILE + tok0;
+        const bool pre = PRE && t_first + tile < pre_tiles;
+        const int tok0 = warp * F::WTOK, p0 = (pre ? (t_first + tile) * F::TILE : begin + tile * F::TILE) + tok0;
         float s[NQ][NK][4];  // rows gid, gid + 8 of sixteen keys x the lane's two queries
 #pragma unroll
         for (int n = 0; n < NK; n++) {
@@ -527,13 +544,17 @@ __global__ void __launch_bounds__(128, FewQ<D, NQ, KV>::PER_SM)
                 for (int q = 0; q < NQ; q++) mma_bf16(s[q][n], k, qb[q][ks][0], qb[q][ks][1]);
             }
         }
-        const bool edge = p0 + F::WTOK > pos0 || p0 < lo_last;
+        const bool edge = pre ? p0 + F::WTOK > pre_all : p0 + F::WTOK > pos0 || p0 < lo_last;
         uint32_t pb[NQ][NK][2];
 #pragma unroll
         for (int q = 0; q < NQ; q++) {
-            float mx[2] = {-INFINITY, -INFINITY};
-            const float db[2] = {(float)(pq[q][0] - p0 - gid), (float)(pq[q][1] - p0 - gid)};
-            base2_logits<NK, true>(s[q], a, sc, db, r1[q], r2[q], span[q], edge, mx);
+            float mx[2] = {-INFINITY, -INFINITY}, db[2], sp[2];
+#pragma unroll
+            for (int h = 0; h < 2; h++) {
+                const int last = pre ? prefix_len(a, pq[q][h]) - 1 : pq[q][h];
+                db[h] = (float)(last - p0 - gid), sp[h] = pre ? 3e38f : span[q][h];
+            }
+            base2_logits<NK, true>(s[q], a, sc, db, r1[q], r2[q], sp, edge, mx);
             float alpha[2], m_use[2];
 #pragma unroll
             for (int h = 0; h < 2; h++) {
@@ -596,63 +617,63 @@ __global__ void __launch_bounds__(128, FewQ<D, NQ, KV>::PER_SM)
     finish_slices<D, QT, 4, 128, NQ == 1>(a, row_first, kvh, grp, n_queries, n_splits, wo, wml, part_o, part_ml, tickets);
 }
 
-template <int D, int MT, int SL, bool KV>
+template <int D, int MT, int SL, bool KV, bool PRE = false>
 cudaError_t launch_one(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch) {
     const int splits = wattn_splits(ctx, a, l, TOK, 16 * MT, SL == 1 ? 1 : MT == 1 ? 3 : 2);
     const WattnScratch sc = wattn_scratch(ctx, scratch);
     constexpr size_t smem = wattn_smem<D, MT, SL, KV>();
     static SmemOptIn configured;
-    if (cudaError_t e = tsb_opt_in_smem(ctx, window_attn_kernel<D, MT, SL, KV>, smem, configured); e != cudaSuccess) return e;
-    cudaError_t e = tsb_launch(ctx, window_attn_kernel<D, MT, SL, KV>, dim3((unsigned)splits, (unsigned)a.keys.kv_heads, (unsigned)l.n_tiles), dim3(32 * MT * SL),
+    if (cudaError_t e = tsb_opt_in_smem(ctx, window_attn_kernel<D, MT, SL, KV, PRE>, smem, configured); e != cudaSuccess) return e;
+    cudaError_t e = tsb_launch(ctx, window_attn_kernel<D, MT, SL, KV, PRE>, dim3((unsigned)splits, (unsigned)a.keys.kv_heads, (unsigned)l.n_tiles), dim3(32 * MT * SL),
                                smem, st, true, a, l.tiles, l.tiles_per_group, l.rows_per_seq, l.rows_per_tile, sc.o, sc.ml, sc.tickets, ctx->dev_error);
     return e == cudaSuccess && splits > 1 ? launch_window_attn_merge(ctx, st, a, l, splits, 16 * MT, sc) : e;
 }
 
-template <int D, int NQ, bool KV>
+template <int D, int NQ, bool KV, bool PRE>
 cudaError_t launch_few(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch) {
     using F = FewQ<D, NQ, KV>;
     const int splits = wattn_splits(ctx, a, l, F::TILE, 8 * NQ, F::PER_SM);
     const WattnScratch sc = wattn_scratch(ctx, scratch);
     static SmemOptIn configured;
-    if (cudaError_t e = tsb_opt_in_smem(ctx, window_attn_few_kernel<D, NQ, KV>, F::SMEM, configured); e != cudaSuccess) return e;
-    cudaError_t e = tsb_launch(ctx, window_attn_few_kernel<D, NQ, KV>, dim3((unsigned)splits, (unsigned)a.keys.kv_heads, (unsigned)l.n_tiles), dim3(128), F::SMEM,
+    if (cudaError_t e = tsb_opt_in_smem(ctx, window_attn_few_kernel<D, NQ, KV, PRE>, F::SMEM, configured); e != cudaSuccess) return e;
+    cudaError_t e = tsb_launch(ctx, window_attn_few_kernel<D, NQ, KV, PRE>, dim3((unsigned)splits, (unsigned)a.keys.kv_heads, (unsigned)l.n_tiles), dim3(128), F::SMEM,
                                st, true, a, l.tiles, l.rows_per_seq, sc.o, sc.ml, sc.tickets, ctx->dev_error);
     return e == cudaSuccess && splits > 1 && NQ > 1 ? launch_window_attn_merge(ctx, st, a, l, splits, 8 * NQ, sc) : e;
 }
 // query tiles by the number of queries; head sizes above 128 have registers for one
-template <int D, bool KV>
+template <int D, bool KV, bool PRE>
 cudaError_t launch_few_dim(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, int queries, void* scratch) {
-    if (queries <= 8) return launch_few<D, 1, KV>(ctx, st, a, l, scratch);
-    if (queries <= 16) return launch_one<D, 1, 4, KV>(ctx, st, a, l, scratch);  // sixteen query rows of one mma tile: faster than two tiles of eight
+    if (queries <= 8) return launch_few<D, 1, KV, PRE>(ctx, st, a, l, scratch);
+    if (queries <= 16) return launch_one<D, 1, 4, KV, PRE>(ctx, st, a, l, scratch);  // sixteen query rows of one mma tile: faster than two tiles of eight
     if constexpr (D <= 128) {
-        if (queries <= 24) return launch_few<D, 3, KV>(ctx, st, a, l, scratch);
-        if (queries <= 32) return launch_few<D, 4, KV>(ctx, st, a, l, scratch);
+        if (queries <= 24) return launch_few<D, 3, KV, PRE>(ctx, st, a, l, scratch);
+        if (queries <= 32) return launch_few<D, 4, KV, PRE>(ctx, st, a, l, scratch);
     }
-    return launch_one<D, 4, 2, KV>(ctx, st, a, l, scratch);
+    return launch_one<D, 4, 2, KV, PRE>(ctx, st, a, l, scratch);
 }
 
-template <int MT, int SL, bool KV>
+template <int MT, int SL, bool KV, bool PRE = false>
 cudaError_t launch_large(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch) {
     switch (a.keys.head_dim) {
-        case 32: return launch_one<32, MT, SL, KV>(ctx, st, a, l, scratch);
-        case 64: return launch_one<64, MT, SL, KV>(ctx, st, a, l, scratch);
-        case 96: return launch_one<96, MT, SL, KV>(ctx, st, a, l, scratch);
-        case 128: return launch_one<128, MT, SL, KV>(ctx, st, a, l, scratch);
-        case 192: return launch_one<192, MT, SL, KV>(ctx, st, a, l, scratch);
-        case 256: return launch_one<256, MT, SL, KV>(ctx, st, a, l, scratch);
+        case 32: return launch_one<32, MT, SL, KV, PRE>(ctx, st, a, l, scratch);
+        case 64: return launch_one<64, MT, SL, KV, PRE>(ctx, st, a, l, scratch);
+        case 96: return launch_one<96, MT, SL, KV, PRE>(ctx, st, a, l, scratch);
+        case 128: return launch_one<128, MT, SL, KV, PRE>(ctx, st, a, l, scratch);
+        case 192: return launch_one<192, MT, SL, KV, PRE>(ctx, st, a, l, scratch);
+        case 256: return launch_one<256, MT, SL, KV, PRE>(ctx, st, a, l, scratch);
         default: return cudaErrorInvalidValue;
     }
 }
 
-template <bool KV>
+template <bool KV, bool PRE = false>
 cudaError_t launch_small(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, int queries, void* scratch) {
     switch (a.keys.head_dim) {
-        case 32: return launch_few_dim<32, KV>(ctx, st, a, l, queries, scratch);
-        case 64: return launch_few_dim<64, KV>(ctx, st, a, l, queries, scratch);
-        case 96: return launch_few_dim<96, KV>(ctx, st, a, l, queries, scratch);
-        case 128: return launch_few_dim<128, KV>(ctx, st, a, l, queries, scratch);
-        case 192: return launch_few_dim<192, KV>(ctx, st, a, l, queries, scratch);
-        case 256: return launch_few_dim<256, KV>(ctx, st, a, l, queries, scratch);
+        case 32: return launch_few_dim<32, KV, PRE>(ctx, st, a, l, queries, scratch);
+        case 64: return launch_few_dim<64, KV, PRE>(ctx, st, a, l, queries, scratch);
+        case 96: return launch_few_dim<96, KV, PRE>(ctx, st, a, l, queries, scratch);
+        case 128: return launch_few_dim<128, KV, PRE>(ctx, st, a, l, queries, scratch);
+        case 192: return launch_few_dim<192, KV, PRE>(ctx, st, a, l, queries, scratch);
+        case 256: return launch_few_dim<256, KV, PRE>(ctx, st, a, l, queries, scratch);
         default: return cudaErrorInvalidValue;
     }
 }

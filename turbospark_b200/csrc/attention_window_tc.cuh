@@ -8,7 +8,7 @@
 //                   and writes P = 2^(v - m) as bfloat16 over the scores, the A operand of the second product.  Row maxima
 //                   and sums stay in the thread.  m moves only when a tile's maximum exceeds it by more than 8; only then
 //                   the output accumulator is rescaled in place.
-//   warp 8          one thread fetches key tiles through TMA (a 2-D map over the layer's pages, one box per page and 64
+//   warp 8          fetches key tiles, a lane per box, through TMA (a 2-D map over the layer's pages, one box per page and 64
 //                   columns, 128-byte swizzle).  Keys are the K-major B operand of Q K^T, values the MN-major B operand of P V:
 //                   where the values are the keys the same bytes serve as both, and a tile is fetched once.
 //   warp 9          (of a third warpgroup, whose other two warps only give up their registers) issues tcgen05.mma, alternating between the two query tiles: while one warpgroup works on its scores the
@@ -17,6 +17,7 @@
 // in shared memory before its scores arrive, so the inner loop has no logarithm.
 // CTAs take the tiles from the last one on: with a causal mask it has the most keys.
 // A cut context leaves (m, l, O) per query and run; a merge launch finishes the rows.
+// PRE: the prefix before the window goes first, in key tiles of its own whose rows are counted from zero; its pages have a map of their own.
 // All waits are bounded; a wait that runs out marks the launch failed, the roles keep their arrivals going, tensor memory is
 // freed and the kernel returns.
 #pragma once
@@ -73,9 +74,9 @@ __device__ __forceinline__ void st_32bytes(void* p, const uint32_t (&r)[8]) {  /
                  : "memory");
 }
 
-template <int DK, int DV, int TN, bool KV>
+template <int DK, int DV, int TN, bool KV, bool PRE>
 __global__ void __launch_bounds__(WT_THREADS, 1)
-    window_attn_tc_kernel(const __grid_constant__ CUtensorMap kmap, int box_rows, const __grid_constant__ WindowAttn a, const AttnTile* __restrict__ tiles,
+    window_attn_tc_kernel(const __grid_constant__ CUtensorMap kmap, int box_rows, const __grid_constant__ CUtensorMap pmap, int pre_box_rows, const __grid_constant__ WindowAttn a, const AttnTile* __restrict__ tiles,
                           int tiles_per_group, int rows_per_seq, int rows_per_tile, float* __restrict__ part_o, float2* __restrict__ part_ml,
                           uint32_t* __restrict__ err) {
     using Geo = WtGeo<DK, DV, TN, KV>;
@@ -108,10 +109,11 @@ __global__ void __launch_bounds__(WT_THREADS, 1)
     // visible positions, in key tiles that start at a copy box; this CTA's run of them
     const int lo = first_visible(a, pos0) & ~(box_rows - 1);
     const int hi = pos0 + n_rows;
-    const int total = seq_ok ? (hi - lo + WT_TN - 1) / WT_TN : 0;
+    const int n_pre = PRE && seq_ok ? prefix_len(a, hi - 1) : 0, pre_tiles = (n_pre + WT_TN - 1) / WT_TN;
+    const int total = seq_ok ? pre_tiles + (hi - lo + WT_TN - 1) / WT_TN : 0;
     const int per = (total + n_splits - 1) / n_splits;
     const int t_first = min(total, (int)blockIdx.x * per), n_tiles = min(total, t_first + per) - t_first;
-    const int begin = lo + t_first * WT_TN;
+    const int begin = lo + (t_first - pre_tiles) * WT_TN;  // of the window's tiles
 
     if (threadIdx.x == 0) {
         for (int i = 0; i < WT_STAGES; i++) mbar_init(&bars->kv_full[i], 1), mbar_init(&bars->kv_empty[i], 1);
@@ -142,39 +144,45 @@ __global__ void __launch_bounds__(WT_THREADS, 1)
 
     if (warp >= 8) {
         asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(WT_REGS_SMALL));
-        if (warp == 8 && lane == 0) {
+        if (warp == 8) {
             bool ok = true;
             int issued = 0;
             for (int t = 0; t < n_tiles && ok; t++) {
                 const int st = t % WT_STAGES;
-                if (t >= WT_STAGES) ok = mbar_wait(&bars->kv_empty[st], ((t / WT_STAGES) - 1) & 1, err);
+                if (t >= WT_STAGES && lane == 0) ok = mbar_wait(&bars->kv_empty[st], ((t / WT_STAGES) - 1) & 1, err);
+                ok = __shfl_sync(0xffffffffu, (int)ok, 0) != 0;
                 if (!ok) break;
                 const uint32_t dst = smem_u32(ring + st * STAGE);
-                mbar_expect_tx(&bars->kv_full[st], (uint32_t)STAGE);
-                for (int part = 0; part * box_rows < WT_TN; part++) {
-                    int pos = begin + t * WT_TN + part * box_rows;
-                    if (pos >= hi) pos = (hi - 1) & ~(box_rows - 1);  // past the end: masked later, read from a page that exists
-                    const int lp = pos >> a.keys.page_shift;
+                if (lane == 0) mbar_expect_tx(&bars->kv_full[st], (uint32_t)STAGE);
+                __syncwarp();
+                const bool pre = PRE && t_first + t < pre_tiles, pooled = pre && a.pool > 0;
+                const int box = pre ? pre_box_rows : box_rows, end = pre ? n_pre : hi, shift = pooled ? a.pooled.page_shift : a.keys.page_shift;
+                const CUtensorMap* map = pre ? &pmap : &kmap;
+                for (int part = lane; part * box < WT_TN; part += 32) {
+                    int pos = (pre ? (t_first + t) * WT_TN : begin + t * WT_TN) + part * box;
+                    if (pos >= end) pos = (end - 1) & ~(box - 1);  // past the end: masked later, read from a page that exists
+                    const int lp = pos >> shift;
                     int page = lp < a.keys.max_pages_per_seq ? a.keys.page_table[(int64_t)seq * a.keys.max_pages_per_seq + lp] : -1;
                     if (page < 0) {  // not a reserved position: flagged; the copy reads page 0 so that the byte count stays whole
                         atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
                         page = 0;
                     }
-                    const int row = page * a.keys.page_tokens + (pos & (a.keys.page_tokens - 1));
+                    const int row = (page << shift) + (pos & ((1 << shift) - 1));
 #pragma unroll
                     for (int b = 0; b < DK / 64; b++)
-                        wt_g2s_2d(dst + b * (WT_TN * 128) + part * box_rows * 128, &kmap, kvh * a.keys.head_step + b * 64, row, &bars->kv_full[st]);
+                        wt_g2s_2d(dst + b * (WT_TN * 128) + part * box * 128, map, kvh * a.keys.head_step + b * 64, row, &bars->kv_full[st]);
                     if (KV) {
 #pragma unroll
                         for (int b = 0; b < DV / 64; b++)
-                            wt_g2s_2d(dst + Geo::V_AT + b * (WT_TN * 128) + part * box_rows * 128, &kmap, kvh * a.keys.head_step + a.keys.value_off + b * 64, row,
+                            wt_g2s_2d(dst + Geo::V_AT + b * (WT_TN * 128) + part * box * 128, map, kvh * a.keys.head_step + a.keys.value_off + b * 64, row,
                                       &bars->kv_full[st]);
                     }
                 }
                 issued = t + 1;
+                __syncwarp();
             }
             // no copy is in flight when the CTA leaves, also when another role has given up
-            for (int t = issued > WT_STAGES ? issued - WT_STAGES : 0; t < issued; t++) mbar_wait(&bars->kv_full[t % WT_STAGES], (t / WT_STAGES) & 1, err);
+            for (int t = lane > 0 ? issued : issued > WT_STAGES ? issued - WT_STAGES : 0; t < issued; t++) mbar_wait(&bars->kv_full[t % WT_STAGES], (t / WT_STAGES) & 1, err);
         }
         if (warp == 9) {
             const uint32_t leader = lane == 0 ? 1u : 0u;
@@ -243,6 +251,7 @@ __global__ void __launch_bounds__(WT_THREADS, 1)
             const ScoreConst sc(a);
             const float slope = a.slopes ? a.slopes[kvh * grp + min(head_l, grp - 1)] * 1.4426950408889634f : 0.f;
             const int lo_last = first_visible(a, wg_last), lo_mine = first_visible(a, pq);
+            const int pre_all = PRE ? prefix_len(a, wg_first) : 0, pre_mine = PRE ? prefix_len(a, pq) : 0;  // of the prefix: seen by every row, by this one
             // bias tables: entry k of a head holds the bias at distance wg_first - p0 + rows_wg - 1 - k; row_l's key j is entry
             // rows_wg - 1 - row_l + j.  The pitch keeps the 32 queries of a warp on different banks.
             const int need = rows_wg + WT_TN - 1;
@@ -252,7 +261,8 @@ __global__ void __launch_bounds__(WT_THREADS, 1)
             float m_ref = -INFINITY, l_run = 0.f;
             bool ok = true;
             for (int t = 0; t < n_tiles; t++) {
-                const int p0 = begin + t * WT_TN;
+                const bool pre = PRE && t_first + t < pre_tiles;
+                const int p0 = pre ? (t_first + t) * WT_TN : begin + t * WT_TN;
                 const float* bias = tab[t & 1] + tab_at;
                 if (biased) {
                     for (int h = 0; h < grp; h++) {
@@ -306,8 +316,8 @@ __global__ void __launch_bounds__(WT_THREADS, 1)
 #pragma unroll
                     for (int j = 0; j < WT_TN; j++) s[j] += fmaf(slope, (float)j, at0);
                 }
-                if (p0 + WT_TN - 1 > wg_first || p0 < lo_last) {  // the tile meets an edge of some row
-                    const int j_max = pq - p0, j_min = lo_mine - p0;
+                if (pre ? p0 + WT_TN > pre_all : p0 + WT_TN - 1 > wg_first || p0 < lo_last) {  // the tile meets an edge of some row
+                    const int j_max = (pre ? pre_mine - 1 : pq) - p0, j_min = pre ? 0 : lo_mine - p0;
 #pragma unroll
                     for (int j = 0; j < WT_TN; j++)
                         if (j > j_max || j < j_min) s[j] = -INFINITY;
@@ -374,6 +384,10 @@ __global__ void __launch_bounds__(WT_THREADS, 1)
                 for (int i = 0; i < 16; i++) v[i] = n_tiles > 0 && ok ? __uint_as_float(r[i]) : 0.f;
                 if (!valid) continue;
                 if (n_splits == 1) {
+                    if (a.turn) {
+#pragma unroll
+                        for (int i = 0; i < 16; i += 2) turn_back(a, row, c + i, v[i], v[i + 1]);
+                    }
                     if (a.value_gate) {
                         const uint4* g = reinterpret_cast<const uint4*>(value_gate_at(a, row, head, c));
 #pragma unroll
@@ -455,18 +469,23 @@ cudaError_t wt_map(const KeyView& k, int box_rows, CUtensorMap* out) {
     return cudaSuccess;
 }
 
-template <int DK, int DV, int TN, bool KV>
+template <int DK, int DV, int TN, bool KV, bool PRE = false>
 cudaError_t launch_tc(tsb_ctx* ctx, cudaStream_t st, const WindowAttn& a, const WattnLaunch& l, void* scratch) {
     const int splits = wattn_splits(ctx, a, l, TN, 2 * WT_QM, 1);
     const WattnScratch sc = wattn_scratch(ctx, scratch);
     const int box_rows = std::min(a.keys.page_tokens, TN);
     CUtensorMap map;
     if (cudaError_t e = wt_map(a.keys, box_rows, &map); e != cudaSuccess) return e;
+    const KeyView& prefix = a.pool > 0 ? a.pooled : a.keys;
+    const int pre_box_rows = std::min(prefix.page_tokens, TN);
+    CUtensorMap pmap = map;
+    if (PRE)
+        if (cudaError_t e = wt_map(prefix, pre_box_rows, &pmap); e != cudaSuccess) return e;
     static SmemOptIn configured;
     constexpr size_t smem = WtGeo<DK, DV, TN, KV>::SMEM;
-    if (cudaError_t e = tsb_opt_in_smem(ctx, window_attn_tc_kernel<DK, DV, TN, KV>, smem, configured); e != cudaSuccess) return e;
-    cudaError_t e = tsb_launch(ctx, window_attn_tc_kernel<DK, DV, TN, KV>, dim3((unsigned)splits, (unsigned)a.keys.kv_heads, (unsigned)l.n_tiles),
-                               dim3(WT_THREADS), smem, st, true, map, box_rows, a, l.tiles, l.tiles_per_group, l.rows_per_seq, l.rows_per_tile, sc.o, sc.ml,
+    if (cudaError_t e = tsb_opt_in_smem(ctx, window_attn_tc_kernel<DK, DV, TN, KV, PRE>, smem, configured); e != cudaSuccess) return e;
+    cudaError_t e = tsb_launch(ctx, window_attn_tc_kernel<DK, DV, TN, KV, PRE>, dim3((unsigned)splits, (unsigned)a.keys.kv_heads, (unsigned)l.n_tiles),
+                               dim3(WT_THREADS), smem, st, true, map, box_rows, pmap, pre_box_rows, a, l.tiles, l.tiles_per_group, l.rows_per_seq, l.rows_per_tile, sc.o, sc.ml,
                                ctx->dev_error);
     return e == cudaSuccess && splits > 1 ? launch_window_attn_merge(ctx, st, a, l, splits, 2 * WT_QM, sc) : e;
 }

@@ -33,6 +33,7 @@ __device__ __forceinline__ void put(__nv_bfloat16* p, float v) { *p = __float2bf
 // division (relative error a few 2^-22), the f32 path the library's.
 template <typename T>
 __device__ __forceinline__ float activate(int act, float z) {
+    if (act == PLAIN_RELU2) return fmaxf(z, 0.f) * fmaxf(z, 0.f);
     const float u = act == PLAIN_GELU_TANH ? 1.5957691216057308f * (z + 0.044715f * z * z * z) : z;  // 2 sqrt(2 / pi)
     if (sizeof(T) == 4) {
         if (act == PLAIN_GELU_TANH) return 0.5f * z * (1.f + tanhf(0.5f * u));
@@ -51,6 +52,7 @@ struct SegAt {
     int64_t stride = 0;
     const void* gate = nullptr;
     int64_t gate_stride = 0;
+    int act = -1;
 };
 __device__ __forceinline__ SegAt seg_at(const PlainEpi& e, int n) {
     SegAt at;
@@ -63,7 +65,7 @@ __device__ __forceinline__ SegAt seg_at(const PlainEpi& e, int n) {
             const int g = (n - first) / s.per, i = (n - first) - g * s.per;
             if (i < s.valid) {
                 at.kind = s.kind, at.col = g * s.step + i, at.p = s.p, at.stride = s.stride;
-                at.gate = s.gate, at.gate_stride = s.gate_stride, at.gate_col = g * s.gate_step + i;
+                at.gate = s.gate, at.gate_stride = s.gate_stride, at.gate_col = g * s.gate_step + i, at.act = s.act;
             }
             break;
         }
@@ -74,6 +76,7 @@ __device__ __forceinline__ SegAt seg_at(const PlainEpi& e, int n) {
 template <typename T>
 __device__ __forceinline__ void seg_put(const PlainEpi& e, const SegAt& at, int t, float v, uint32_t* err) {
     if (at.kind == PLAIN_SEG_TYPED) {
+        if (at.act >= 0) v = activate<T>(at.act, v);
         if (at.gate) {
             const float z = get(static_cast<const T*>(at.gate) + (int64_t)t * at.gate_stride + at.gate_col);
             v *= 1.f / (1.f + expf(-z));
@@ -96,7 +99,7 @@ __device__ __forceinline__ void epi_one(const PlainEpi& e, int t, int n, float v
     } else if (e.kind == PLAIN_ADD) {
         if (n < e.n_valid) {
             float* y = e.y + (int64_t)t * e.y_stride + n;
-            *y = fmaf(e.alpha, *y, v);
+            *y = fmaf(e.alpha, *y, e.beta * v);
         }
     } else {
         if (e.bias) v += e.bias[n];
@@ -391,7 +394,7 @@ struct TcgOut {
                 for (int j = 0; j < 16; j++) old[j] = j < left ? y[j * step] : 0.f;
 #pragma unroll
                 for (int j = 0; j < 16; j++)
-                    if (j < left) y[j * step] = fmaf(e.alpha, old[j], v[j]);
+                    if (j < left) y[j * step] = fmaf(e.alpha, old[j], e.beta * v[j]);
             } else {
                 if (e.cap > 0.f) {
 #pragma unroll 1
@@ -417,6 +420,10 @@ struct TcgOut {
                 for (int j = 0; j < 16; j++)
                     if (j < left) y[j * at.stride] = v[j];
             } else if (at.kind == PLAIN_SEG_TYPED) {
+                if (at.act >= 0) {
+#pragma unroll
+                    for (int j = 0; j < 16; j++) v[j] = activate<__nv_bfloat16>(at.act, v[j]);
+                }
                 if (at.gate) {
                     const __nv_bfloat16* g = static_cast<const __nv_bfloat16*>(at.gate) + (int64_t)t0 * at.gate_stride + at.gate_col;
                     float z[16];

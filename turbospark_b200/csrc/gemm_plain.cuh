@@ -17,7 +17,7 @@ inline int64_t plain_pad(int64_t n, int64_t to) { return (n + to - 1) / to * to;
 
 enum PlainEpiKind {
     PLAIN_STORE = 0,  // y[t, n] = acc, through cap * tanh(acc / cap) when cap > 0
-    PLAIN_ADD = 1,    // y[t, n] = alpha * y[t, n] + acc  (the residual stream)
+    PLAIN_ADD = 1,    // y[t, n] = alpha * y[t, n] + beta * acc  (the residual stream)
     PLAIN_MIXER = 2,  // by row of the matrix: segments with destinations of their own, then pairs of rows (gate and up of a
                       // feed-forward as act(gate) * up, or the two coordinates of a rotation)
 };
@@ -37,6 +37,7 @@ struct PlainSeg {
     const void* gate = nullptr;  // PLAIN_SEG_TYPED: times sigmoid of element g * gate_step + i of row t of this buffer (compute type)
     int64_t gate_stride = 0;
     int gate_step = 0;
+    int act = -1;                // PLAIN_SEG_TYPED: a PlainAct of the row's own number (a feed-forward without gates); -1: none
 };
 constexpr int PLAIN_SEGS = 6;
 // Pairs (u, v) as coordinates i and i + half of a rotated part: u c - v s and v c + u s with (c, s) of the token's position.
@@ -49,14 +50,14 @@ struct PlainRotate {
     int q_step[2] = {0, 0}, q_off[2] = {0, 0};
     int key_off = 0;                     // the key's elements start here in the cache row
 };
-enum PlainAct { PLAIN_GELU_TANH = 0, PLAIN_SILU = 1 };
+enum PlainAct { PLAIN_GELU_TANH = 0, PLAIN_SILU = 1, PLAIN_RELU2 = 2 };  // RELU2: max(z, 0)^2
 
 struct PlainEpi {
     int kind = PLAIN_STORE;
     int n_valid = 0;       // PLAIN_STORE / PLAIN_ADD: rows of the matrix that have an output column
     float* y = nullptr;
     int64_t y_stride = 0;
-    float cap = 0.f, alpha = 1.f;
+    float cap = 0.f, alpha = 1.f, beta = 1.f;
     // PLAIN_MIXER
     PlainSeg seg[PLAIN_SEGS];
     int n_seg = 0;

@@ -197,13 +197,19 @@ int32_t kv_create_keys(tsb_ctx* ctx, int n_layers, const KeyLayerShape* shapes, 
     int32_t rc = kv_init_pages(ctx, kv, page_tokens, num_pages, max_seqs, max_pages_per_seq);
     size_t bytes = 0;
     auto row_of = [&](int l) { return shapes[l].kv_heads * (shapes[l].head_dim + shapes[l].value_dim); };
+    auto pooled_rows = [&](int pool) {  // per page
+        int n = pool > 0 ? POOLED_MIN_ROWS : 0;
+        while (pool > 0 && (int64_t)n * pool < page_tokens) n *= 2;
+        return n;
+    };
     for (int l = 0; l < n_layers && rc == TSB_OK; l++) {
         const KeyLayerShape& k = shapes[l];
         if (k.kv_heads < 0 || (k.kv_heads > 0 && k.head_dim <= 0) || k.value_dim < 0 || (k.head_dim * elem_bytes) % 16 || (k.value_dim * elem_bytes) % 16)
             rc = tsb_fail(ctx, TSB_ERR_INVALID, "layer %d: bad head count or head size", l);
         else if (k.source < 0 || k.source > l || shapes[k.source].source != k.source || row_of(k.source) != row_of(l))
             rc = tsb_fail(ctx, TSB_ERR_INVALID, "layer %d cannot read the rows of layer %d", l, k.source);
-        if (k.source == l) bytes += (size_t)num_pages * page_tokens * row_of(l) * elem_bytes;
+        else if (k.pool < 0 || (k.pool > 0 && k.source != l)) rc = tsb_fail(ctx, TSB_ERR_INVALID, "layer %d: blocks are of rows of its own", l);
+        if (k.source == l) bytes += (size_t)num_pages * (page_tokens + pooled_rows(k.pool)) * row_of(l) * elem_bytes;
     }
     if (rc == TSB_OK) rc = pool_alloc(ctx, std::max<size_t>(bytes, 16), (void**)&kv->key_pool);
     if (rc) {
@@ -222,6 +228,15 @@ int32_t kv_create_keys(tsb_ctx* ctx, int n_layers, const KeyLayerShape* shapes, 
         k.max_seqs = max_seqs, k.max_pages_per_seq = max_pages_per_seq;
         kv->key_layers.push_back(k);
         if (own) off += (size_t)num_pages * page_tokens * k.row * elem_bytes;
+        KeyView p = k;
+        p.base = nullptr;
+        if (const int rows = pooled_rows(shapes[l].pool)) {
+            p.base = kv->key_pool + off, p.page_tokens = rows;
+            for (p.page_shift = 0; 1 << p.page_shift < rows;) p.page_shift++;
+            off += (size_t)num_pages * rows * k.row * elem_bytes;
+        }
+        kv->pooled_layers.push_back(p);
+        kv->pool_sizes.push_back(shapes[l].pool);
     }
     *out = kv;
     return TSB_OK;
@@ -231,9 +246,13 @@ int32_t kv_fill_keys(tsb_kv* kv, cudaStream_t st, int32_t seq, int64_t tokens, u
     int32_t rc = tsb_kv_reserve(kv, seq, tokens);
     if (rc) return rc;
     DeviceGuard g(kv->ctx);
-    for (size_t l = 0; l < kv->key_layers.size(); l++)
-        if (kv->key_layers[l].row > 0) TSB_CUDA(kv->ctx, tsb_launch(kv->ctx, keys_fill_random_kernel, dim3((unsigned)(kv->ctx->sm_count * 4)), dim3(256), 0, st, false, kv->key_layers[l],
-                                     (int)seq, (int)tokens, (uint32_t)(seed * 1000003u + l)));
+    auto fill = [&](const KeyView& k, int64_t rows, uint32_t sd) {
+        return tsb_launch(kv->ctx, keys_fill_random_kernel, dim3((unsigned)(kv->ctx->sm_count * 4)), dim3(256), 0, st, false, k, (int)seq, (int)rows, sd);
+    };
+    for (size_t l = 0; l < kv->key_layers.size(); l++) {
+        if (kv->key_layers[l].row > 0) TSB_CUDA(kv->ctx, fill(kv->key_layers[l], tokens, (uint32_t)(seed * 1000003u + l)));
+        if (kv->pooled_layers[l].base) TSB_CUDA(kv->ctx, fill(kv->pooled_layers[l], tokens / kv->pool_sizes[l], (uint32_t)(seed * 1000003u + l + 500009u)));
+    }
     return TSB_OK;
 }
 
@@ -355,25 +374,27 @@ int32_t tsb_kv_rewind_by(tsb_kv* kv, int32_t seq, int64_t count) {
 }
 
 static int32_t kv_copy_rows(tsb_kv* kv, tsb_stream s, int32_t seq, int32_t layer, int64_t pos0, int32_t n, void* hk, void* hv,
-                            bool to_device) {
+                            bool to_device, bool pooled = false) {
     int32_t rc = kv_check(kv, seq);
     if (rc) return rc;
     tsb_ctx* ctx = kv->ctx;
     const KvView& v = kv->view;
     const bool keys = !kv->key_layers.empty();
     TSB_REQUIRE(ctx, layer >= 0 && layer < v.layers && n >= 0 && pos0 >= 0 && hk && (keys || hv), "bad arguments");
-    if (pos0 + n > (int64_t)kv->pages_of_seq[seq] * v.page_tokens)
+    // bytes of a row, and where the layer's K and V halves start (a plain cache has one)
+    const KeyView* kl = keys ? pooled ? &kv->pooled_layers[layer] : &kv->key_layers[layer] : nullptr;
+    TSB_REQUIRE(ctx, !pooled || (kl && kl->base), "layer %d keeps no blocks", layer);
+    const int page_tokens = kl ? kl->page_tokens : v.page_tokens, page_shift = kl ? kl->page_shift : v.page_shift;
+    if (pos0 + n > (int64_t)kv->pages_of_seq[seq] * page_tokens)
         return tsb_fail(ctx, TSB_ERR_STATE, "rows %lld..%lld are not reserved", (long long)pos0, (long long)(pos0 + n));
     DeviceGuard g(ctx);
-    // bytes of a row, and where the layer's K and V halves start (a plain cache has one)
-    const KeyView* kl = keys ? &kv->key_layers[layer] : nullptr;
     const size_t row = keys ? (size_t)kl->row * kl->elem_bytes : (size_t)v.kv_heads * v.head_dim * sizeof(__half);
     const int32_t* pt = &kv->page_table_host[(size_t)seq * v.max_pages_per_seq];
     int64_t p = pos0;
     while (p < pos0 + n) {  // one copy per page run
-        const int64_t in_page = p & (v.page_tokens - 1);
-        const int64_t run = std::min<int64_t>(v.page_tokens - in_page, pos0 + n - p);
-        const int64_t slot = (int64_t)pt[p >> v.page_shift] * v.page_tokens + in_page;
+        const int64_t in_page = p & (page_tokens - 1);
+        const int64_t run = std::min<int64_t>(page_tokens - in_page, pos0 + n - p);
+        const int64_t slot = (int64_t)pt[p >> page_shift] * page_tokens + in_page;
         for (int which = 0; which < (keys ? 1 : 2); which++) {
             char* half = keys ? (char*)kl->base : (char*)(v.pool + (int64_t)layer * v.layer_stride + (int64_t)which * v.kv_stride);
             char* dev = half + slot * (int64_t)row;
@@ -395,6 +416,10 @@ int32_t tsb_kv_write_rows(tsb_kv* kv, tsb_stream s, int32_t seq, int32_t layer, 
 }
 int32_t tsb_kv_read_rows(tsb_kv* kv, tsb_stream s, int32_t seq, int32_t layer, int64_t pos0, int32_t n, void* hk, void* hv) {
     return kv_copy_rows(kv, s, seq, layer, pos0, n, hk, hv, false);
+}
+int32_t tsb_kv_read_blocks(tsb_kv* kv, tsb_stream s, int32_t seq, int32_t layer, int64_t block0, int32_t n, void* host) {
+    if (!kv || kv->key_layers.empty()) return TSB_ERR_INVALID;
+    return kv_copy_rows(kv, s, seq, layer, block0, n, host, nullptr, false, true);
 }
 
 int32_t tsb_kv_fill_random(tsb_kv* kv, tsb_stream s, int32_t seq, int64_t tokens, uint64_t seed) {

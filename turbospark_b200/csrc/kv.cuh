@@ -34,12 +34,18 @@ struct KeyLayerShape {
     int kv_heads, head_dim;  // no heads: the layer has no rows
     int value_dim; // elements of the value behind every key (0: the values are the keys)
     int source;    // the layer whose rows this one reads (itself: rows of its own)
+    int pool = 0;  // > 0: the layer also keeps a row for every block of this many positions
 };
 
 struct tsb_kv {
     tsb_ctx* ctx = nullptr;
     KvView view{};                    // page geometry; pool and strides of a key + value cache
     std::vector<KeyView> key_layers;  // not empty: a plain cache (view.pool is then null)
+    // Rows of blocks (KeyLayerShape::pool), shaped like the layer's rows: row b of a stream belongs to its positions b pool .. b pool + pool - 1.
+    // A page of positions brings room for a page of blocks - page_tokens / pool of them, rounded up to a power of two of at least
+    // POOLED_MIN_ROWS - and both go by the same page table.  Layers without have no base.
+    std::vector<KeyView> pooled_layers;
+    std::vector<int> pool_sizes;  // of the layers; 0: none
     uint8_t* key_pool = nullptr;
     // A model whose rows also need their predecessors' state keeps the last state_ring - 1 rows' worth of it per stream
     // (0: no such state).  state_lo is the oldest position whose state is still there: a cursor may go back to 0 or to
@@ -53,6 +59,7 @@ struct tsb_kv {
     std::vector<int64_t> cursor;
 };
 
+constexpr int POOLED_MIN_ROWS = 8;  // a copy box of eight rows fills the 1024 bytes after which a 128-byte swizzle repeats
 // A plain cache of n_layers layers with their own head counts and (padded) head sizes.
 int32_t kv_create_keys(tsb_ctx* ctx, int n_layers, const KeyLayerShape* shapes, int elem_bytes, int page_tokens, int num_pages, int max_seqs,
                        int max_pages_per_seq, tsb_kv** out);

@@ -19,6 +19,9 @@
 // In output-norm form a sublayer reads the stream through a short convolution, and its output is normed and added by one kernel that also
 // makes the next sublayer's input (launch_sublayer_end); the stream goes back and forth between two buffers.  Mixers: attention over keys
 // and values, a recurrence (recurrence.cuh), or both side by side - one input matmul, one output matmul over [heads | recurrence].
+// In pre-norm form a norm makes each sublayer's input, and its output matmul adds to the stream (f32).  Attention over keys and values there turns
+// queries, keys and - if the layer says so - values with their positions in the kernel that norms them: coordinates of a pair are packed side by side
+// (rows of W_q, W_k, W_v, columns of W_o), whichever layout the model stores.  Blocks before a window get their means behind it.
 // Routed feed-forwards: router matmul, choice and lists, a grouped product each for gate-up pairs and down.
 #include <algorithm>
 #include <cstring>
@@ -99,19 +102,22 @@ int32_t plain_complete(const tsb_model* tm) {
         need(l.mixer == MIX_KV, {TSB_P_V});
         need(l.cfg.qk_norm, {TSB_P_Q_NORM, TSB_P_K_NORM});
         need(l.cfg.qkv_bias, {TSB_P_Q_BIAS, TSB_P_K_BIAS, TSB_P_V_BIAS});
-        need(l.cfg.sink, {TSB_P_SINK});
+        need(l.cfg.sink == TSB_SINK_TENSOR, {TSB_P_SINK});
         need(l.cfg.value_gate, {TSB_P_VALUE_GATE});
         need(l.cfg.token_shift, {TSB_P_SHIFT});
         need(l.cfg.head_gate, {TSB_P_HEAD_GATE});
         need(l.cfg.log_bias, {TSB_P_R1, TSB_P_R2});
-        need(rec, {TSB_P_REC_NORM, TSB_P_REC_O});
+        need(rec, {TSB_P_REC_O});
+        need(rec && rec != TSB_REC_MINGRU, {TSB_P_REC_NORM});
+        need(rec == TSB_REC_MINGRU, {TSB_P_REC_F, TSB_P_REC_F_BIAS, TSB_P_REC_I, TSB_P_REC_I_BIAS, TSB_P_REC_GATE});
         need(rec == TSB_REC_FORGET || rec == TSB_REC_MLSTM, {TSB_P_REC_Q, TSB_P_REC_V, TSB_P_REC_F, TSB_P_REC_F_BIAS});
         need(rec == TSB_REC_FORGET, {TSB_P_REC_LOWER});
         need(rec == TSB_REC_MLSTM, {TSB_P_REC_K, TSB_P_REC_GATE, TSB_P_REC_I, TSB_P_REC_I_BIAS});
         need(rec == TSB_REC_SSD, {TSB_P_REC_IN, TSB_P_REC_CONV, TSB_P_REC_CONV_BIAS, TSB_P_REC_DT_BIAS, TSB_P_REC_A_LOG, TSB_P_REC_D});
         need(m->cfg.conv_taps > 0, {TSB_P_CONV1});
         need(m->cfg.conv_taps > 0 && l.cfg.ffn > 0, {TSB_P_CONV2});
-        need(l.cfg.ffn > 0, {TSB_P_FF_GATE, TSB_P_FF_UP, TSB_P_FF_DOWN});
+        need(l.cfg.ffn > 0, {TSB_P_FF_UP, TSB_P_FF_DOWN});
+        need(l.cfg.ffn > 0 && !l.cfg.ff_plain, {TSB_P_FF_GATE});
         need(l.cfg.ffn > 0 && l.post_norm, {TSB_P_NORM2});
         need(l.cfg.experts > 0, {TSB_P_ROUTER, TSB_P_CORRECTION});
         TSB_REQUIRE(ctx, (l.set & w) == w, "layer %zu is missing a tensor (have %llx, need %llx)", i, (unsigned long long)l.set, (unsigned long long)w);
@@ -123,6 +129,18 @@ void free_layer(tsb_ctx* ctx, PlainLayer& l) {
     if (!l.owned) return;
     for (void** p : l.buffers())
         if (*p) tsb_free(ctx, *p);
+}
+
+// layers that use the tensors of layer `from` get its pointers
+void mirror_layer(PlainModel* m, int from) {
+    for (int i = 0; i < m->cfg.n_layers; i++) {
+        PlainLayer& l = m->layers[i];
+        if (l.tied != from) continue;
+        const tsb_plain_layer cfg = l.cfg;
+        const int source = l.source;
+        l = m->layers[from];
+        l.cfg = cfg, l.source = source, l.tied = from, l.owned = false;
+    }
 }
 
 void plain_free(tsb_model* tm) {
@@ -142,11 +160,11 @@ void plain_free(tsb_model* tm) {
 // rows of a recurrence in the input matrix: vectors in the compute type, gates in f32
 int64_t rec_typed_rows(const tsb_plain_layer& c) {
     const int64_t h = c.rec_heads, D = c.rec_dim, E = c.rec_vdim;
-    return c.recurrence == TSB_REC_FORGET ? h * (D + E) : c.recurrence == TSB_REC_MLSTM ? 2 * h * (D + E) : c.recurrence == TSB_REC_SSD ? 2 * h * E + 2 * c.rec_groups * D : 0;
+    return c.recurrence == TSB_REC_MINGRU ? E : c.recurrence == TSB_REC_FORGET ? h * (D + E) : c.recurrence == TSB_REC_MLSTM ? 2 * h * (D + E) : c.recurrence == TSB_REC_SSD ? 2 * h * E + 2 * c.rec_groups * D : 0;
 }
 int64_t rec_gate_rows(const tsb_plain_layer& c) {
     const int64_t h = c.rec_heads;
-    return c.recurrence == TSB_REC_FORGET ? h * c.rec_dim : c.recurrence == TSB_REC_MLSTM ? 2 * h : c.recurrence == TSB_REC_SSD ? h : 0;
+    return c.recurrence == TSB_REC_MINGRU ? 2 * (int64_t)c.rec_vdim : c.recurrence == TSB_REC_FORGET ? h * c.rec_dim : c.recurrence == TSB_REC_MLSTM ? 2 * h : c.recurrence == TSB_REC_SSD ? h : 0;
 }
 int64_t rec_conv_channels(const tsb_plain_layer& c) { return c.recurrence == TSB_REC_SSD ? (int64_t)c.rec_heads * c.rec_vdim + 2 * (int64_t)c.rec_groups * c.rec_dim : 0; }
 // numbers of a layer's matrices that a pass over one row reads
@@ -154,7 +172,7 @@ int64_t layer_numbers(const PlainLayer& l, int64_t d) {
     const tsb_plain_layer& c = l.cfg;
     const int64_t H = c.n_q_heads, G = c.n_kv_heads, D = c.head_dim, E = l.mixer == MIX_KEYS ? D : c.value_dim;
     int64_t n = d * (H * E + (c.head_gate ? H : 0) + (c.value_gate ? H * E : 0));
-    n += c.experts > 0 ? d * (c.experts + 3 * (int64_t)c.ffn * c.expert_top) : d * 3 * (int64_t)c.ffn;
+    n += c.experts > 0 ? d * (c.experts + 3 * (int64_t)c.ffn * c.expert_top) : d * (c.ff_plain ? 2 : 3) * (int64_t)c.ffn;
     n += d * (rec_typed_rows(c) + rec_gate_rows(c) + (c.recurrence ? (int64_t)c.rec_heads * c.rec_vdim : 0));
     if (l.mixer == MIX_LATENT) {
         n += d * H * (D + c.rot_dim) + (int64_t)c.kv_rank * H * (D + E);
@@ -177,7 +195,7 @@ int32_t plain_share(tsb_model* dt, int32_t dst_layer, const tsb_model* st, int32
     PlainModel* d = dt->plain;
     const PlainModel* s = st->plain;
     TSB_REQUIRE(ctx, d->cfg.d_model == s->cfg.d_model && d->cfg.vocab == s->cfg.vocab && d->f32 == s->f32 && d->cfg.post_norm == s->cfg.post_norm &&
-                         d->cfg.output_norm == s->cfg.output_norm && d->cfg.conv_taps == s->cfg.conv_taps && d->cfg.positions == s->cfg.positions,
+                         d->cfg.output_norm == s->cfg.output_norm && d->cfg.pre_norm == s->cfg.pre_norm && d->cfg.conv_taps == s->cfg.conv_taps && d->cfg.positions == s->cfg.positions,
                 "models differ in width, vocabulary, type or form");
     if (dst_layer < 0) {
         if (d->owned)
@@ -189,11 +207,13 @@ int32_t plain_share(tsb_model* dt, int32_t dst_layer, const tsb_model* st, int32
     TSB_REQUIRE(ctx, dst_layer < d->cfg.n_layers && src_layer >= 0 && src_layer < s->cfg.n_layers, "layer out of range");
     PlainLayer& l = d->layers[dst_layer];
     TSB_REQUIRE(ctx, memcmp(&l.cfg, &s->layers[src_layer].cfg, sizeof l.cfg) == 0, "layer shapes differ");
+    TSB_REQUIRE(ctx, l.tied < 0, "layer %d uses the tensors of layer %d", dst_layer, l.tied);
     free_layer(ctx, l);
-    const int rotation = l.rotation, source = l.source;
+    const int rotation = l.rotation, value_rotation = l.value_rotation, source = l.source;
     l = s->layers[src_layer];
-    l.rotation = rotation, l.source = source;
-    l.owned = false;
+    l.rotation = rotation, l.value_rotation = value_rotation, l.source = source;
+    l.tied = -1, l.owned = false;
+    mirror_layer(d, dst_layer);
     return TSB_OK;
 }
 
@@ -246,7 +266,7 @@ int32_t states_init(tsb_session* s, const PlainModel* m, const SessionShape& sha
         const size_t copies = heads * recurrence_copies(c.rec_vdim);
         if (c.recurrence == TSB_REC_MLSTM && rc == TSB_OK) rc = zero(copies * c.rec_dim * 4, (void**)&r.norm);
         if (c.recurrence == TSB_REC_MLSTM && rc == TSB_OK) rc = zero(copies * 8, (void**)&r.top);
-        if (c.recurrence && !m->f32)
+        if (c.recurrence && c.recurrence != TSB_REC_MINGRU && !m->f32)
             scratch = std::max(scratch, recurrence_scratch_bytes(c.recurrence, c.rec_heads, c.rec_dim, c.rec_vdim, shape.pass_rows / REC_CHUNK + shape.n_streams));
         st.states.push_back(r);
     }
@@ -271,7 +291,7 @@ int32_t plain_runtime_init(tsb_session* s, ModelRt& rt, const tsb_model* tm, con
     for (const PlainLayer& l : m->layers) {
         if (l.mixer == MIX_LATENT) shapes.push_back({1, l.key_dim, 0, l.source});
         else if (l.mixer == MIX_NONE) shapes.push_back({0, 0, 0, (int)shapes.size()});
-        else shapes.push_back({l.cfg.n_kv_heads, l.head_pad, l.mixer == MIX_KV ? l.head_pad : 0, (int)shapes.size()});
+        else shapes.push_back({l.cfg.n_kv_heads, l.head_pad, l.mixer == MIX_KV ? l.head_pad : 0, (int)shapes.size(), l.cfg.pool});
     }
     int32_t rc = kv_create_keys(ctx, m->cfg.n_layers, shapes.data(), m->elem, shape.page_tokens, shape.num_pages, shape.n_streams, shape.pages_per_seq, &rt.kv);
     if (rc) return rc;
@@ -285,15 +305,16 @@ int32_t plain_runtime_init(tsb_session* s, ModelRt& rt, const tsb_model* tm, con
         const int64_t H = l.cfg.n_q_heads, inner = (int64_t)l.cfg.rec_heads * l.cfg.rec_vdim;
         p->rec_stride = std::max<int64_t>(p->rec_stride, plain_pad(rec_typed_rows(l.cfg), 16));
         p->rec_mixed_stride = std::max<int64_t>(p->rec_mixed_stride, plain_pad(rec_conv_channels(l.cfg), 16));
-        if (l.cfg.recurrence) p->rec_out_stride = std::max<int64_t>(p->rec_out_stride, plain_pad(inner, 4));
-        p->raw_rec = std::max<int64_t>(p->raw_rec, l.cfg.qk_norm ? plain_pad((H + l.cfg.n_kv_heads) * l.cfg.head_dim, 4) : 0);
+        if (l.cfg.recurrence && l.cfg.recurrence != TSB_REC_MINGRU) p->rec_out_stride = std::max<int64_t>(p->rec_out_stride, plain_pad(inner, 4));
+        const int64_t heads = l.cfg.qk_norm ? plain_pad((H + l.cfg.n_kv_heads) * l.cfg.head_dim + (l.cfg.value_rot ? l.cfg.n_kv_heads * l.cfg.value_dim : 0), 4) : 0;
+        p->raw_stride = std::max<int64_t>(p->raw_stride, heads);
+        if (l.cfg.recurrence) p->raw_rec = std::max<int64_t>(p->raw_rec, heads);
         if (l.cfg.experts > 0)
             experts = std::max<int64_t>(experts, l.cfg.experts), top = std::max<int64_t>(top, l.cfg.expert_top), expert_ffn = std::max<int64_t>(expert_ffn, l.ffn_pad);
         p->q_stride = std::max<int64_t>(p->q_stride, plain_pad(H * l.head_pad, 16));
         p->cat_stride = std::max<int64_t>(p->cat_stride, l.out.cols);
         p->gate_stride = std::max(p->gate_stride, l.cfg.n_q_heads);
         if (l.post_norm && l.cfg.experts == 0) p->act_stride = std::max<int64_t>(p->act_stride, l.ffn_pad);
-        if (l.cfg.qk_norm) p->raw_stride = std::max<int64_t>(p->raw_stride, plain_pad((H + l.cfg.n_kv_heads) * l.cfg.head_dim, 4));
         if (l.cfg.value_gate) p->value_gate_stride = std::max<int64_t>(p->value_gate_stride, plain_pad(H * l.value_pad, 16));
         if (l.mixer != MIX_LATENT) continue;
         p->raw_stride = std::max<int64_t>(p->raw_stride, plain_pad(l.cfg.kv_rank, 4));
@@ -312,7 +333,7 @@ int32_t plain_runtime_init(tsb_session* s, ModelRt& rt, const tsb_model* tm, con
     };
     const size_t R = p->rows, e = m->elem;
     if ((rc = A(R * m->cfg.d_model * 4, (void**)&p->x)) || (rc = A(R * p->in_stride * e, &p->mix)) ||
-        (rc = A(m->cfg.post_norm || m->cfg.output_norm ? 0 : R * p->in_stride * e, &p->h)) || (rc = A(R * p->q_stride * e, &p->q)) || (rc = A(R * p->cat_stride * e, &p->cat)) ||
+        (rc = A(m->sequential() ? 0 : R * p->in_stride * e, &p->h)) || (rc = A(R * p->q_stride * e, &p->q)) || (rc = A(R * p->cat_stride * e, &p->cat)) ||
         (rc = A(R * p->gate_stride * 4, (void**)&p->gate)) || (rc = A((size_t)p->fin_rows * p->in_stride * e, &p->fin)) ||
         (rc = A(plain_gemm_workspace_bytes(ctx), &p->gemm_ws)) || (rc = A(wattn_scratch_bytes(ctx), &p->attn_ws)) ||
         (rc = A(R * p->act_stride * e, &p->act)) || (rc = A(R * p->raw_stride * 4, (void**)&p->raw)) || (rc = A(R * p->absorbed_stride * e, &p->absorbed)) ||
@@ -321,9 +342,7 @@ int32_t plain_runtime_init(tsb_session* s, ModelRt& rt, const tsb_model* tm, con
     if (m->cfg.output_norm) {
         const size_t slots = plain_pad(R * top, 32) + 256;  // token tiles of a product may reach behind the last slot
         p->expert_rows = top > 0 ? (int)slots : 0;
-        if ((rc = A(R * m->cfg.d_model * 4, (void**)&p->x2)) || (rc = A(R * m->cfg.d_model * 4, (void**)&p->y)) || (rc = A(R * p->rec_stride * e, &p->rec)) ||
-            (rc = A(R * p->rec_mixed_stride * e, &p->rec_mixed)) || (rc = A(R * p->rec_out_stride * 4, (void**)&p->rec_out)))
-            return rc;
+        if ((rc = A(R * m->cfg.d_model * 4, (void**)&p->x2)) || (rc = A(R * m->cfg.d_model * 4, (void**)&p->y))) return rc;
         if (top > 0) {
             ExpertLists& x = p->lists;
             const size_t ints = R * top * sizeof(int32_t);
@@ -334,6 +353,9 @@ int32_t plain_runtime_init(tsb_session* s, ModelRt& rt, const tsb_model* tm, con
                 (rc = A(sizeof(int32_t), (void**)&x.n_chunks)))
                 return rc;
         }
+    }
+    if (m->cfg.output_norm || m->cfg.pre_norm) {
+        if ((rc = A(R * p->rec_stride * e, &p->rec)) || (rc = A(R * p->rec_mixed_stride * e, &p->rec_mixed)) || (rc = A(R * p->rec_out_stride * 4, (void**)&p->rec_out))) return rc;
         if ((rc = states_init(s, m, shape, p->states))) return rc;
         if (p->states.ring > 0) rt.kv->state_ring = p->states.ring + 1;
     }
@@ -421,8 +443,9 @@ struct PassPlan {
     std::vector<bool> is_expanded;
     const ExpandStream* expanded_dev = nullptr;
     int expanded_pages = 0, expanded_len = 0, short_first = 0, short_rows = 0;
-    // output-norm form: runs of rows for the row operators; portions whose recurrences go row by row, and chunk by chunk where there is a kernel
+    // output-norm form and recurrences: runs of rows for the row operators; portions whose recurrences go row by row, and chunk by chunk where there is a kernel
     RowTiles runs, by_row, portions;  // portions: all of them
+    RowTiles by_scan;                 // those that are not in by_row
     RecurrenceChunks by_chunk;
     bool use_before = false;
 
@@ -447,7 +470,7 @@ int32_t plan_states(tsb_session* s, const PlainModel* m, const ModelRt& rt, cons
         plan.by_row = plan.portions = RowTiles::uniform(p.rows, p.rows_per_seq, p.rows_per_seq);
         return TSB_OK;
     }
-    std::vector<AttnTile> runs, by_row, portions, chunks;
+    std::vector<AttnTile> runs, by_row, by_scan, portions, chunks;
     std::vector<ChunkPortion> by_chunk;
     for (int i = 0; i < p.n_groups; i++) {
         const RowGroup& g = p.groups[i];
@@ -458,6 +481,7 @@ int32_t plan_states(tsb_session* s, const PlainModel* m, const ModelRt& rt, cons
             by_row.push_back({g.first_row, g.n_rows});
             continue;
         }
+        by_scan.push_back({g.first_row, g.n_rows});
         by_chunk.push_back({g.first_row, g.n_rows, (int)chunks.size()});
         for (int r = 0; r < g.n_rows; r += REC_CHUNK) chunks.push_back({g.first_row + r, std::min(REC_CHUNK, g.n_rows - r)});
         rt.kv->state_lo[g.seq] = g.base + g.n_rows - 1;  // the states in between are not kept
@@ -476,6 +500,7 @@ int32_t plan_states(tsb_session* s, const PlainModel* m, const ModelRt& rt, cons
     int32_t rc = stage(runs, plan.runs);
     if (rc == TSB_OK) rc = stage(by_row, plan.by_row);
     if (rc == TSB_OK) rc = stage(portions, plan.portions);
+    if (rc == TSB_OK) rc = stage(by_scan, plan.by_scan);
     if (rc == TSB_OK) rc = stage(chunks, plan.by_chunk.chunks);
     if (rc || by_chunk.empty()) return rc;
     const int32_t* dev = nullptr;
@@ -490,7 +515,8 @@ int32_t plan_pass(tsb_session* s, const PlainModel* m, const ModelRt& rt, const 
     plan.max_len = (p.max_len + 511) / 512 * 512;  // the split plan changes only every 512 positions (graph reuse)
     plan.longest = p.rows_per_seq;
     plan.short_rows = p.rows;
-    if (p.rows_per_seq > 0) return m->cfg.output_norm ? plan_states(s, m, rt, p, plan) : TSB_OK;
+    const bool states = m->cfg.output_norm || b->states.ring > 0;
+    if (p.rows_per_seq > 0) return states ? plan_states(s, m, rt, p, plan) : TSB_OK;
     plan.is_expanded.assign(p.n_groups, false);
     int first_short = p.rows, end_short = 0;
     for (int i = 0; i < p.n_groups; i++) {
@@ -512,7 +538,7 @@ int32_t plan_pass(tsb_session* s, const PlainModel* m, const ModelRt& rt, const 
         if (int32_t rc = session_stage_ints(s, reinterpret_cast<const int32_t*>(plan.expanded.data()), (int)plan.expanded.size() * 3, &dev)) return rc;
         plan.expanded_dev = reinterpret_cast<const ExpandStream*>(dev);
     }
-    if (m->cfg.output_norm)
+    if (states)
         if (int32_t rc = plan_states(s, m, rt, p, plan)) return rc;
     if (m->f32) return TSB_OK;  // the f32 kernel takes rows one by one
     auto add = [&](int set, int group, int rpt, int small_queries) -> int32_t {
@@ -587,12 +613,12 @@ struct Forward {
             seg(r.v, PLAIN_SEG_CACHE, nullptr, 0);
         } else if (l.mixer == MIX_KV) {
             if (c.qk_norm) {
-                seg(r.v, PLAIN_SEG_F32, b->raw, b->raw_stride);
+                seg(c.value_rot ? r.head_gate : r.v, PLAIN_SEG_F32, b->raw, b->raw_stride);
             } else {
                 seg(r.k, PLAIN_SEG_TYPED, b->q, b->q_stride, c.head_dim, l.head_pad);
                 seg(r.v, PLAIN_SEG_CACHE, nullptr, 0, c.head_dim, e.keys.head_step);
             }
-            seg(r.head_gate, PLAIN_SEG_CACHE, nullptr, e.keys.value_off, c.value_dim, e.keys.head_step);
+            if (!c.value_rot) seg(r.head_gate, PLAIN_SEG_CACHE, nullptr, e.keys.value_off, c.value_dim, e.keys.head_step);
         } else if (l.mixer == MIX_LATENT) {
             seg(r.k, PLAIN_SEG_TYPED, b->q, b->q_stride, c.head_dim, l.head_pad);
             if (r.v > r.k) seg(r.v, PLAIN_SEG_F32, b->raw, b->raw_stride);
@@ -627,6 +653,8 @@ struct Forward {
             h.n_q = c.n_q_heads, h.n_k = c.n_kv_heads, h.width = c.head_dim, h.q_weight = l.q_norm, h.k_weight = l.k_norm;
             h.temp_coef = c.q_temp_coef, h.temp_every = c.q_temp_every;
             h.q = b->q, h.q_stride = b->q_stride, h.q_step = h.q_width = l.head_pad;
+            if (l.rotation >= 0) h.rot = b->rotary[l.rotation], h.rot_half = c.rot_dim / 2;
+            if (c.value_rot) h.n_v = c.n_kv_heads, h.v_width = c.value_dim, h.turn = b->rotary[l.value_rotation], h.turn_half = c.value_dim / 2;
         }
         return launch_head_norms(ctx, st, m->f32, h, p.rows);
     }
@@ -636,7 +664,8 @@ struct Forward {
         WindowAttn a;
         a.q = b->q, a.q_stride = b->q_stride, a.out = b->cat, a.out_stride = l.out.cols, a.rows = p.rows_dev;
         a.n_q_heads = c.n_q_heads, a.scale = c.score_scale, a.cap = c.score_cap, a.window = c.window;
-        a.slopes = l.slopes, a.chunk = c.chunk;
+        a.slopes = l.slopes, a.chunk = c.chunk, a.keep = c.keep_first, a.pool = c.pool;
+        if (c.value_rot) a.turn = b->rotary[l.value_rotation], a.turn_half = c.value_dim / 2;
         if (c.recurrence) a.out_scale = c.attn_scale;
         a.gate = c.head_gate ? b->gate : nullptr;
         if (c.value_gate) a.value_gate = b->value_gate, a.value_gate_stride = b->value_gate_stride;
@@ -650,6 +679,7 @@ struct Forward {
         const int grp = l.cfg.n_q_heads / l.cfg.n_kv_heads;
         WindowAttn a = attention_of(l);
         a.keys = rt.kv->key_layers[L];
+        if (a.pool > 0) a.pooled = rt.kv->pooled_layers[L];
         AttnBatch batch;
         if (const AttnBatch* t = plan.find(TILES_ALL, grp, wattn_rows_per_tile(l.head_pad, grp, l.cfg.log_bias != 0))) batch = *t;
         batch.rows = p.rows, batch.rows_per_seq = p.rows_per_seq, batch.max_len = plan.max_len;
@@ -727,13 +757,30 @@ struct Forward {
         n.raw = b->raw, n.raw_stride = b->raw_stride, n.n_q = l.cfg.n_q_heads, n.n_k = l.cfg.n_kv_heads, n.width = l.cfg.head_dim;
         n.q_weight = l.q_norm, n.k_weight = l.k_norm, n.eps = m->cfg.norm_eps, n.q = b->q, n.q_stride = b->q_stride, n.q_step = l.head_pad;
         n.keys = rt.kv->key_layers[L], n.rows = p.rows_dev;
+        if (l.rotation >= 0) n.rot = b->rotary[l.rotation], n.rot_half = l.cfg.rot_dim / 2;
         return launch_projection_norms(ctx, st, m->f32, n, p.rows);
+    }
+
+    cudaError_t scan(int L) const {
+        const PlainLayer& l = m->layers[L];
+        GatedScan g;
+        g.gate = b->raw + b->raw_rec, g.gate_stride = b->raw_stride, g.out_gate = b->rec, g.out_gate_stride = b->rec_stride;
+        g.out = at(b->cat, l.o_cols), g.out_stride = l.out.cols, g.width = l.cfg.rec_vdim, g.state = b->states.states[L], g.rows = p.rows_dev;
+        if (cudaError_t e = launch_gated_scan(ctx, st, m->f32, g, plan.by_row); e != cudaSuccess) return e;
+        return launch_gated_scan(ctx, st, m->f32, g, plan.by_scan);
+    }
+
+    cudaError_t block_means(int L) const {
+        BlockMeans v;
+        v.keys = rt.kv->key_layers[L], v.pooled = rt.kv->pooled_layers[L], v.pool = m->layers[L].cfg.pool, v.rows = p.rows_dev;
+        return launch_block_means(ctx, st, m->f32, v, p.rows);
     }
 
     // from the projections to the recurrence's part of b->cat
     cudaError_t recur(int L) const {
         const PlainLayer& l = m->layers[L];
         const tsb_plain_layer& c = l.cfg;
+        if (c.recurrence == TSB_REC_MINGRU) return scan(L);
         const int h = c.rec_heads, D = c.rec_dim, E = c.rec_vdim, inner = h * E;
         Recurrence r;
         GatedNorm g;
@@ -857,11 +904,9 @@ struct Forward {
             e = recur(L);
             if (e != cudaSuccess || l.mixer == MIX_NONE) return e;
         }
-        if (l.cfg.qk_norm == TSB_NORM_PROJECTION) {
-            if ((e = projection_norms(L)) != cudaSuccess) return e;
-            return attend(L);
-        }
-        if (l.cfg.qk_norm || (l.mixer == MIX_LATENT && l.source == L)) e = head_norms(L);
+        if (l.cfg.qk_norm == TSB_NORM_PROJECTION) e = projection_norms(L);
+        else if (l.cfg.qk_norm || (l.mixer == MIX_LATENT && l.source == L)) e = head_norms(L);
+        if (e == cudaSuccess && l.cfg.pool > 0) e = block_means(L);
         if (e != cudaSuccess) return e;
         if (l.mixer != MIX_LATENT) return attend(L);
         const bool expand = l.expands && !plan.expanded.empty();
@@ -874,6 +919,7 @@ struct Forward {
         PlainEpi e;
         e.kind = PLAIN_ADD, e.y = b->x, e.y_stride = m->cfg.d_model, e.n_valid = m->cfg.d_model;
         if (m->cfg.post_norm) e.alpha = m->cfg.residual_scale;
+        if (m->cfg.pre_norm) e.beta = m->cfg.sublayer_scale;
         return matmul(w, x, nullptr, stride, e);
     }
 
@@ -902,6 +948,26 @@ struct Forward {
         e = matmul(l.ff_in, b->mix, b->mix, b->in_stride, g);
         if (e == cudaSuccess) e = add_to_stream(l.ff_out, b->act, l.ffn_pad);
         return e == cudaSuccess ? norm(l.norm2) : e;
+    }
+
+    cudaError_t pre_norm_layer(int L) const {
+        const PlainLayer& l = m->layers[L];
+        auto norm = [&](const float* w) { return launch_pre_norm(ctx, st, m->f32, b->x, m->cfg.d_model, w, m->cfg.norm_eps, p.rows, b->mix, b->in_stride); };
+        cudaError_t e = norm(l.gain);
+        if (e == cudaSuccess) e = project(L, b->mix, b->mix);
+        if (e == cudaSuccess) e = mix(L);
+        if (e == cudaSuccess) e = add_to_stream(l.out, b->cat, l.out.cols);
+        if (e != cudaSuccess || l.cfg.ffn == 0) return e;
+        e = norm(l.norm2);
+        PlainEpi g;
+        g.kind = PLAIN_MIXER;
+        if (l.cfg.ff_plain) {
+            g.n_seg = 1, g.seg[0].end = l.ffn_pad, g.seg[0].act = l.cfg.act, g.seg[0].p = b->act, g.seg[0].stride = l.ffn_pad;
+        } else {
+            g.pair_row0 = 0, g.n_pairs = l.ffn_pad, g.act = l.cfg.act, g.a = b->act, g.a_stride = l.ffn_pad;
+        }
+        if (e == cudaSuccess) e = matmul(l.ff_in, b->mix, b->mix, b->in_stride, g);
+        return e == cudaSuccess ? add_to_stream(l.ff_out, b->act, l.ffn_pad) : e;
     }
 };
 
@@ -933,7 +999,7 @@ cudaError_t plain_forward(tsb_session* s, ModelRt& rt, const Pass& p) {
             const PlainRotation& r = m->rotations[i];
             FW(launch_rotary_table(ctx, st, r.freq, r.dims / 2, r.magnitude, p.rows_dev, p.rows, b->rotary[i]));
         }
-        for (int L = 0; L < m->cfg.n_layers; L++) FW(post ? f.post_norm_layer(L) : f.parallel_layer(L, use_before));
+        for (int L = 0; L < m->cfg.n_layers; L++) FW(post ? f.post_norm_layer(L) : m->cfg.pre_norm ? f.pre_norm_layer(L) : f.parallel_layer(L, use_before));
     }
     if (p.logits) {
         const bool last = p.last_rows_only && p.rows_per_seq > 1;
@@ -945,7 +1011,7 @@ cudaError_t plain_forward(tsb_session* s, ModelRt& rt, const Pass& p) {
                 FW(launch_group_norm_rows(ctx, st, m->f32, x, d, m->final_gain, std::max(1, m->cfg.norm_groups), m->cfg.norm_eps, want, want_first, want_step, n, b->fin,
                                           b->in_stride));
             else
-                FW(launch_norm_rows(ctx, st, m->f32, x, d, m->final_gain, post ? m->final_gain : nullptr, m->cfg.norm_eps, want, want_first, want_step, n, b->fin, b->in_stride));
+                FW(launch_norm_rows(ctx, st, m->f32, x, d, m->final_gain, m->sequential() ? m->final_gain : nullptr, m->cfg.norm_eps, want, want_first, want_step, n, b->fin, b->in_stride));
             PlainEpi hd;
             hd.kind = PLAIN_STORE, hd.y = static_cast<float*>(p.logits.p), hd.y_stride = p.logits_stride, hd.n_valid = m->cfg.vocab, hd.cap = m->cfg.logit_cap;
             FW(launch_plain_gemm(ctx, st, m->f32, m->head, b->fin, nullptr, b->in_stride, b->fin_rows, n, hd, b->gemm_ws));
@@ -956,9 +1022,17 @@ cudaError_t plain_forward(tsb_session* s, ModelRt& rt, const Pass& p) {
 }
 
 // ------------------------------------------------------------------ rotations
-int rotation_of(PlainModel* m, const tsb_plain_layer& c) {
+PlainRotation rotation_of(const tsb_plain_layer& c) {
     PlainRotation r;
     r.dims = c.rot_dim, r.base = c.rot_base, r.factor = c.rot_factor, r.original = c.rot_original, r.fast = c.rot_fast, r.slow = c.rot_slow;
+    return r;
+}
+PlainRotation value_rotation_of(const tsb_plain_layer& c) {
+    PlainRotation r;
+    r.dims = c.value_dim, r.base = c.rot_base;
+    return r;
+}
+int rotation_of(PlainModel* m, const PlainRotation& r) {
     for (size_t i = 0; i < m->rotations.size(); i++) {
         const PlainRotation& o = m->rotations[i];
         if (o.dims == r.dims && o.base == r.base && o.factor == r.factor && o.original == r.original && o.fast == r.fast && o.slow == r.slow) return (int)i;
@@ -969,7 +1043,7 @@ int rotation_of(PlainModel* m, const tsb_plain_layer& c) {
 
 int32_t upload_rotation(tsb_ctx* ctx, PlainRotation& r) {
     std::vector<double> freq(r.dims / 2);
-    const bool scaled = r.factor > 0;
+    const bool scaled = r.factor > 0 && r.original > 0, linear = r.factor > 0 && !scaled;
     // the pair that turns t times within the original context
     auto pair_with_turns = [&](double t) { return r.dims * log(r.original / (2 * M_PI * t)) / (2 * log(r.base)); };
     const double lo = scaled ? std::max(floor(pair_with_turns(r.fast)), 0.0) : 0;
@@ -977,7 +1051,7 @@ int32_t upload_rotation(tsb_ctx* ctx, PlainRotation& r) {
     for (int i = 0; i < r.dims / 2; i++) {
         const double f = pow(r.base, -2.0 * i / r.dims);
         const double ramp = scaled ? std::min(std::max((i - lo) / std::max(hi - lo, 0.001), 0.0), 1.0) : 0;
-        freq[i] = scaled ? f / r.factor * ramp + f * (1 - ramp) : f;
+        freq[i] = linear ? f / r.factor : scaled ? f / r.factor * ramp + f * (1 - ramp) : f;
     }
     r.magnitude = scaled ? (float)(0.1 * log(r.factor) + 1.0) : 1.f;
     if (int32_t rc = tsb_alloc(ctx, freq.size() * sizeof(double), (void**)&r.freq)) return rc;
@@ -993,9 +1067,32 @@ const ModelFamily PLAIN_FAMILY = {
 }  // namespace
 
 // what only layers of the output-norm form have
+static int32_t check_pre_norm_layer(tsb_ctx* ctx, const tsb_plain_config* cfg, const tsb_plain_layer& l, int i) {
+    if (!cfg->pre_norm) {
+        TSB_REQUIRE(ctx, !l.keep_first && !l.pool && !l.value_rot && !l.ff_plain && l.act != TSB_ACT_RELU2 && l.recurrence != TSB_REC_MINGRU,
+                    "layer %d: prefixes of a window, turning values, feed-forwards without gates and element-wise recurrences go with the pre-norm form", i);
+        TSB_REQUIRE(ctx, l.rot_dim == 0 || l.kv_rank > 0, "layer %d: only latent layers and those of the pre-norm form rotate", i);
+        return TSB_OK;
+    }
+    TSB_REQUIRE(ctx, !l.kv_rank && !l.token_shift && !l.head_gate && !l.log_bias && !l.qkv_bias && !l.linear_bias && !l.chunk && !l.experts,
+                "layer %d: not a mechanism of the pre-norm form", i);
+    TSB_REQUIRE(ctx, l.n_q_heads >= 0 && (l.n_q_heads > 0) != (l.recurrence != 0), "layer %d has one mixer", i);
+    if (l.recurrence)
+        TSB_REQUIRE(ctx, l.recurrence == TSB_REC_MINGRU && l.rec_heads == 1 && l.rec_dim == 1 && l.rec_vdim > 0, "layer %d: an element-wise recurrence of rec_vdim channels expected", i);
+    if (l.n_q_heads == 0) return TSB_OK;
+    TSB_REQUIRE(ctx, l.value_dim > 0 && (l.qk_norm == TSB_NORM_HEAD || l.qk_norm == TSB_NORM_PROJECTION), "layer %d: attention has values of its own and normed queries and keys", i);
+    TSB_REQUIRE(ctx, l.q_temp_every == 0 || l.qk_norm == TSB_NORM_HEAD, "layer %d: a query temperature goes with norms per head", i);
+    TSB_REQUIRE(ctx, l.rot_dim >= 0 && l.rot_dim % 2 == 0 && l.rot_dim <= l.head_dim && ((l.rot_dim == 0 && !l.value_rot) || l.rot_base > 0) && l.rot_factor >= 0,
+                "layer %d: an even number of a head's columns is rotated", i);
+    TSB_REQUIRE(ctx, !l.value_rot || (l.value_dim % 2 == 0 && l.qk_norm == TSB_NORM_HEAD), "layer %d: values that turn have an even width and go with norms per head", i);
+    TSB_REQUIRE(ctx, l.keep_first >= 0 && l.pool >= 0 && !(l.keep_first && l.pool) && ((!l.keep_first && !l.pool) || l.window > 0),
+                "layer %d: kept tokens or blocks, before a window", i);
+    return TSB_OK;
+}
+
 static int32_t check_output_norm_layer(tsb_ctx* ctx, const tsb_plain_config* cfg, const tsb_plain_layer& l, int i) {
     if (!cfg->output_norm) {
-        TSB_REQUIRE(ctx, !l.recurrence && !l.experts && !l.qkv_bias && !l.linear_bias && !l.chunk && (l.qk_norm == 0 || l.qk_norm == TSB_NORM_HEAD),
+        TSB_REQUIRE(ctx, cfg->pre_norm || (!l.recurrence && !l.experts && !l.qkv_bias && !l.linear_bias && !l.chunk && (l.qk_norm == 0 || l.qk_norm == TSB_NORM_HEAD)),
                     "layer %d: recurrences, experts, biases, chunks and projection norms go with the output-norm form", i);
         return TSB_OK;
     }
@@ -1033,6 +1130,7 @@ int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const 
     TSB_REQUIRE(ctx, cfg->norm_eps >= 0.f, "norm_eps must not be negative");
     const bool f32 = cfg->compute == TSB_F32;
     TSB_REQUIRE(ctx, cfg->norm_groups >= 0 && cfg->conv_taps >= 0 && cfg->positions >= 0, "norm groups, taps and positions must not be negative");
+    TSB_REQUIRE(ctx, !cfg->pre_norm || (!cfg->post_norm && !cfg->output_norm), "a model has one form");
     TSB_REQUIRE(ctx, cfg->output_norm ? !cfg->post_norm && cfg->logit_cap <= 0.f : !cfg->norm_groups && !cfg->conv_taps && !cfg->positions,
                 "norm groups, convolutions and learned positions go with the output-norm form");
     if (cfg->output_norm && !sublayer_end_supported(cfg->d_model, std::max(1, cfg->norm_groups), cfg->conv_taps))
@@ -1041,12 +1139,20 @@ int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const 
     for (int i = 0; i < cfg->n_layers; i++) {
         const tsb_plain_layer& l = layers[i];
         if (int32_t rc = check_output_norm_layer(ctx, cfg, l, i)) return rc;
+        if (int32_t rc = check_pre_norm_layer(ctx, cfg, l, i)) return rc;
+        TSB_REQUIRE(ctx, l.sink >= 0 && l.sink <= TSB_SINK_ZERO, "layer %d: unknown sink", i);
+        if (l.weights_of) {
+            TSB_REQUIRE(ctx, l.weights_of > 0 && l.weights_of <= cfg->n_layers && layers[l.weights_of - 1].weights_of == 0, "layer %d: weights_of names a layer with tensors", i);
+            tsb_plain_layer same = l;
+            same.weights_of = 0;
+            TSB_REQUIRE(ctx, memcmp(&same, &layers[l.weights_of - 1], sizeof same) == 0, "layer %d differs from layer %d, whose tensors it uses", i, l.weights_of - 1);
+        }
         const bool latent = l.kv_rank > 0;
         if (l.n_q_heads == 0 && l.recurrence) continue;
         TSB_REQUIRE(ctx, l.n_q_heads > 0 && l.head_dim > 0 && (latent || (l.n_kv_heads > 0 && l.n_q_heads % l.n_kv_heads == 0)),
                     "layer %d: query heads must be a positive multiple of the key heads", i);
         TSB_REQUIRE(ctx, l.window >= 0 && l.ffn >= 0 && l.value_dim >= 0 && l.kv_rank >= 0 && l.rot_dim >= 0, "layer %d: sizes must not be negative", i);
-        TSB_REQUIRE(ctx, l.act == TSB_ACT_GELU_TANH || l.act == TSB_ACT_SILU, "layer %d: unknown activation", i);
+        TSB_REQUIRE(ctx, l.act >= TSB_ACT_GELU_TANH && l.act <= TSB_ACT_RELU2, "layer %d: unknown activation", i);
         TSB_REQUIRE(ctx, l.q_temp_every >= 0 && (l.q_temp_every == 0 || l.qk_norm), "layer %d: a query temperature goes with normed queries", i);
         TSB_REQUIRE(ctx, !l.qk_norm || (l.value_dim > 0 && !latent), "layer %d: normed queries and keys go with values of their own", i);
         TSB_REQUIRE(ctx, !cfg->post_norm || !l.token_shift, "layer %d: a token shift goes with the parallel form", i);
@@ -1064,7 +1170,7 @@ int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const 
             if (!latent_attn_dims(l.kv_rank, l.rot_dim, &dk, &dv) || dk > 1024)
                 return tsb_fail(ctx, TSB_ERR_UNSUPPORTED, "layer %d: latents of %d + %d numbers are outside the attention kernels", i, l.kv_rank, l.rot_dim);
         } else {
-            TSB_REQUIRE(ctx, l.kv_source == 0 && l.rot_dim == 0, "layer %d: only latent layers rotate or read another layer's rows", i);
+            TSB_REQUIRE(ctx, l.kv_source == 0, "layer %d: only latent layers read another layer's rows", i);
             const int head = std::max(l.head_dim, l.value_dim);
             if (!wattn_supported(head, l.n_q_heads / l.n_kv_heads, f32))
                 return tsb_fail(ctx, TSB_ERR_UNSUPPORTED, "layer %d: head size %d with %d query heads per key head is outside the attention kernels", i, head,
@@ -1086,6 +1192,7 @@ int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const 
     tm->cfg.rms_eps = cfg->norm_eps;
     m->cfg = *cfg, m->f32 = f32, m->elem = f32 ? 4 : 2;
     if (m->cfg.embed_scale == 0.f) m->cfg.embed_scale = 1.f;
+    if (m->cfg.sublayer_scale == 0.f) m->cfg.sublayer_scale = 1.f;
     m->d_pad = plain_pad(cfg->d_model, PLAIN_COL_PAD);
     m->head.rows = plain_pad(cfg->vocab, PLAIN_ROW_PAD), m->head.cols = m->d_pad;
     m->layers.resize(cfg->n_layers);
@@ -1095,7 +1202,8 @@ int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const 
         l.cfg = layers[i];
         const tsb_plain_layer& c = l.cfg;
         const int H = c.n_q_heads;
-        l.post_norm = cfg->post_norm != 0 || cfg->output_norm != 0;
+        l.post_norm = m->sequential();
+        l.tied = c.weights_of - 1;
         l.mixer = H == 0 ? MIX_NONE : c.kv_rank > 0 ? MIX_LATENT : c.value_dim > 0 ? MIX_KV : MIX_KEYS;
         l.source = c.kv_source > 0 ? c.kv_source - 1 : i;
         m->any_shift |= c.token_shift != 0;
@@ -1103,7 +1211,7 @@ int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const 
             l.head_pad = (int)plain_pad(c.head_dim + c.rot_dim, PLAIN_COL_PAD), l.value_pad = (int)plain_pad(c.value_dim, PLAIN_COL_PAD);
             latent_attn_dims(c.kv_rank, c.rot_dim, &l.key_dim, &l.rank_pad);
             l.expands = !f32 && wattn_wide_supported(l.head_pad, l.value_pad);
-            l.rotation = c.rot_dim > 0 ? rotation_of(m, c) : -1;
+            l.rotation = c.rot_dim > 0 ? rotation_of(m, rotation_of(c)) : -1;
             l.absorb.group_rows = (int)plain_pad(c.kv_rank, PLAIN_ROW_PAD), l.absorb.group_cols = l.head_pad;
             l.absorb.rows = (int64_t)H * l.absorb.group_rows, l.absorb.cols = plain_pad(c.head_dim, PLAIN_COL_PAD);
             l.lift.group_rows = (int)plain_pad(c.value_dim, PLAIN_ROW_PAD), l.lift.group_cols = l.rank_pad;
@@ -1111,6 +1219,8 @@ int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const 
             l.expand.rows = plain_pad((int64_t)H * (c.head_dim + c.value_dim), PLAIN_ROW_PAD), l.expand.cols = l.lift.cols;
         } else if (l.mixer != MIX_NONE) {
             l.head_pad = l.value_pad = wattn_pad_dim(std::max(c.head_dim, c.value_dim), f32);
+            if (c.rot_dim > 0) l.rotation = rotation_of(m, rotation_of(c));
+            if (c.value_rot) l.value_rotation = rotation_of(m, value_rotation_of(c));
         }
         l.q_rows = H * l.head_pad, l.k_rows = c.n_kv_heads * l.head_pad;
         l.ffn_pad = (int)plain_pad(c.ffn, 64);
@@ -1118,12 +1228,18 @@ int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const 
         l.o_cols = (int)plain_pad((int64_t)H * l.value_pad, PLAIN_COL_PAD);
         l.rec_cols = (int)plain_pad((int64_t)c.rec_heads * c.rec_vdim * (c.recurrence != 0), PLAIN_COL_PAD);
         l.out.rows = out_rows, l.out.cols = l.o_cols + l.rec_cols + (l.post_norm ? 0 : l.ffn_pad);
-        l.ff_in.rows = 2 * (int64_t)l.ffn_pad, l.ff_in.cols = m->d_pad;
+        l.ff_in.rows = c.ff_plain ? plain_pad(l.ffn_pad, PLAIN_ROW_PAD) : 2 * (int64_t)l.ffn_pad, l.ff_in.cols = m->d_pad;
         l.ff_out.rows = out_rows, l.ff_out.cols = l.ffn_pad;
         l.router.rows = plain_pad(c.experts, PLAIN_ROW_PAD), l.router.cols = m->d_pad;
     }
     DeviceGuard g(ctx);
     for (PlainLayer& l : m->layers) {
+        if (l.tied >= 0) continue;
+        if (l.cfg.sink == TSB_SINK_ZERO)
+            if (int32_t rc = zeroed(ctx, (size_t)l.cfg.n_q_heads * 4, (void**)&l.sink)) {
+                tsb_model_destroy(tm);
+                return rc;
+            }
         if (!l.cfg.linear_bias) continue;
         std::vector<float> slopes(l.cfg.n_q_heads);
         for (int h = 0; h < l.cfg.n_q_heads; h++) slopes[h] = (float)exp2(-8.0 * (h + 1) / l.cfg.n_q_heads);
@@ -1140,30 +1256,31 @@ int32_t tsb_model_create_plain(tsb_ctx* ctx, const tsb_plain_config* cfg, const 
             tsb_model_destroy(tm);
             return rc;
         }
+    for (int i = 0; i < cfg->n_layers; i++) mirror_layer(m, i);
     *out = tm;
     return TSB_OK;
 }
 
-int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t host_type, const void* host, int64_t rows, int64_t cols) {
+static int32_t set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t host_type, const void* host, int64_t rows, int64_t cols) {
     if (!tm) return TSB_ERR_INVALID;
     tsb_ctx* ctx = tm->ctx;
     TSB_REQUIRE(ctx, tm->family == &PLAIN_FAMILY, "the model does not hold plain tensors");
     TSB_REQUIRE(ctx, host && (host_type == TSB_BF16 || host_type == TSB_F32), "null data or unknown host type");
     PlainModel* m = tm->plain;
     const int64_t d = m->cfg.d_model, V = m->cfg.vocab;
-    const bool post = m->cfg.post_norm != 0;
     PlainLayer* l = nullptr;
-    const bool output = m->cfg.output_norm != 0, seq = post || output;  // seq: the sublayers follow each other
+    const bool seq = m->sequential();
     if (which >= TSB_P_NORM && which != TSB_P_POSITIONS) {
         TSB_REQUIRE(ctx, layer >= 0 && layer < m->cfg.n_layers, "layer %d outside the model", layer);
         l = &m->layers[layer];
+        TSB_REQUIRE(ctx, l->tied < 0, "layer %d uses the tensors of layer %d", layer, l->tied);
     }
     const tsb_plain_layer c = l ? l->cfg : tsb_plain_layer{};
     const bool latent = l && l->mixer == MIX_LATENT, own_latent = latent && c.kv_source == 0;
     const int64_t H = c.n_q_heads, G = c.n_kv_heads, D = c.head_dim, F = c.ffn, E = l && l->mixer != MIX_KEYS ? c.value_dim : D, R = c.kv_rank;
     const int64_t rh = c.recurrence ? c.rec_heads : 0, RD = c.rec_dim, RE = c.rec_vdim, X = std::max(1, c.experts), taps = m->cfg.conv_taps;
     const bool attn = l && l->mixer != MIX_NONE, whole = c.qk_norm == TSB_NORM_PROJECTION;
-    const bool forget = c.recurrence == TSB_REC_FORGET, mlstm = c.recurrence == TSB_REC_MLSTM, ssd = c.recurrence == TSB_REC_SSD;
+    const bool forget = c.recurrence == TSB_REC_FORGET, mlstm = c.recurrence == TSB_REC_MLSTM, ssd = c.recurrence == TSB_REC_SSD, gru = c.recurrence == TSB_REC_MINGRU;
     const int64_t channels = rec_conv_channels(c);
     int64_t wr = 1, wc = 1;  // expected shape; -1: no such tensor
     switch (which) {
@@ -1171,12 +1288,12 @@ int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t
         case TSB_P_FINAL_NORM: case TSB_P_NORM: wc = seq ? d : 1; break;
         case TSB_P_NORM2: wc = seq && F > 0 ? d : -1; break;
         case TSB_P_SHIFT: wc = c.token_shift ? d : -1; break;
-        case TSB_P_Q: wr = attn ? H * (D + c.rot_dim) : -1, wc = d; break;
+        case TSB_P_Q: wr = attn ? H * (D + (latent ? c.rot_dim : 0)) : -1, wc = d; break;
         case TSB_P_K: wr = latent || !attn ? -1 : G * D, wc = d; break;
         case TSB_P_V: wr = l->mixer == MIX_KV ? G * E : -1, wc = d; break;
         case TSB_P_Q_NORM: wc = whole ? H * D : c.qk_norm ? D : -1; break;
         case TSB_P_K_NORM: wc = whole ? G * D : c.qk_norm ? D : -1; break;
-        case TSB_P_SINK: wc = c.sink ? H : -1; break;
+        case TSB_P_SINK: wc = c.sink == TSB_SINK_TENSOR ? H : -1; break;
         case TSB_P_HEAD_GATE: wr = c.head_gate ? H : -1, wc = d; break;
         case TSB_P_VALUE_GATE: wr = c.value_gate ? H * E : -1, wc = d; break;
         case TSB_P_R1: case TSB_P_R2: wc = c.log_bias ? H : -1; break;
@@ -1185,7 +1302,8 @@ int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t
         case TSB_P_UK: wr = latent ? H * D : -1, wc = R; break;
         case TSB_P_UV: wr = latent ? H * E : -1, wc = R; break;
         case TSB_P_O: wr = d, wc = attn ? H * E : -1; break;
-        case TSB_P_FF_GATE: case TSB_P_FF_UP: wr = F > 0 ? X * F : -1, wc = d; break;
+        case TSB_P_FF_GATE: wr = F > 0 && !c.ff_plain ? X * F : -1, wc = d; break;
+        case TSB_P_FF_UP: wr = F > 0 ? X * F : -1, wc = d; break;
         case TSB_P_FF_DOWN: wr = X * d, wc = F > 0 ? F : -1; break;
         case TSB_P_POSITIONS: wr = m->cfg.positions > 0 ? m->cfg.positions : -1, wc = d; break;
         case TSB_P_CONV1: wr = d, wc = taps > 0 ? taps : -1; break;
@@ -1198,13 +1316,13 @@ int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t
         case TSB_P_REC_Q: wr = forget || mlstm ? rh * RD : -1, wc = d; break;
         case TSB_P_REC_K: wr = mlstm ? rh * RD : -1, wc = d; break;
         case TSB_P_REC_V: wr = forget || mlstm ? rh * RE : -1, wc = d; break;
-        case TSB_P_REC_GATE: wr = mlstm ? rh * RE : -1, wc = d; break;
-        case TSB_P_REC_F: wr = forget ? rh * RD : mlstm ? rh : -1, wc = d; break;
-        case TSB_P_REC_F_BIAS: wc = forget ? rh * RD : mlstm ? rh : -1; break;
+        case TSB_P_REC_GATE: wr = mlstm || gru ? rh * RE : -1, wc = d; break;
+        case TSB_P_REC_F: wr = forget ? rh * RD : mlstm ? rh : gru ? RE : -1, wc = d; break;
+        case TSB_P_REC_F_BIAS: wc = forget ? rh * RD : mlstm ? rh : gru ? RE : -1; break;
         case TSB_P_REC_LOWER: wc = forget ? rh * RD : -1; break;
-        case TSB_P_REC_I: wr = mlstm ? rh : -1, wc = d; break;
-        case TSB_P_REC_I_BIAS: wc = mlstm ? rh : -1; break;
-        case TSB_P_REC_NORM: wc = forget ? RE : rh > 0 ? rh * RE : -1; break;
+        case TSB_P_REC_I: wr = mlstm ? rh : gru ? RE : -1, wc = d; break;
+        case TSB_P_REC_I_BIAS: wc = mlstm ? rh : gru ? RE : -1; break;
+        case TSB_P_REC_NORM: wc = gru ? -1 : forget ? RE : rh > 0 ? rh * RE : -1; break;
         case TSB_P_REC_O: wr = d, wc = rh > 0 ? rh * RE : -1; break;
         case TSB_P_REC_IN: wr = ssd ? rec_typed_rows(c) + rh : -1, wc = d; break;
         case TSB_P_REC_CONV: wr = ssd ? channels : -1, wc = c.rec_taps; break;
@@ -1250,7 +1368,7 @@ int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t
         case TSB_P_K_BIAS: bias_at = at.k; break;
         case TSB_P_V_BIAS: bias_at = at.v; break;
         case TSB_P_REC_F_BIAS: bias_at = at.rec_gate + (mlstm ? rh : 0); break;
-        case TSB_P_REC_I_BIAS: case TSB_P_REC_DT_BIAS: bias_at = at.rec_gate; break;
+        case TSB_P_REC_I_BIAS: case TSB_P_REC_DT_BIAS: bias_at = at.rec_gate + (gru ? RE : 0); break;
     }
     if (bias_at >= 0) {
         convert(host, host_type, wc, true, v);
@@ -1259,16 +1377,28 @@ int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t
         set |= 1ull << which;
         return TSB_OK;
     }
+    // halves of rotated coordinates -> pairs side by side, in each of `blocks` blocks of `width` items
+    auto pair_up = [&](int64_t blocks, int64_t width, int64_t dims, size_t item) {
+        std::vector<uint8_t> t(v.size());
+        for (int64_t b = 0; b < blocks; b++)
+            for (int64_t i = 0; i < width; i++) {
+                const int64_t to = i >= dims ? i : i < dims / 2 ? 2 * i : 2 * (i - dims / 2) + 1;
+                memcpy(t.data() + (size_t)(b * width + to) * item, v.data() + (size_t)(b * width + i) * item, item);
+            }
+        v.swap(t);
+    };
+    const int64_t rotated = l && l->mixer == MIX_KV ? c.rot_dim : 0;
     if (vec) {
         const int64_t n = wr * wc;
         convert(host, host_type, n, true, v);
+        if (rotated > 0 && (which == TSB_P_Q_NORM || which == TSB_P_K_NORM)) pair_up(n / D, D, rotated, 4);
         if (wr > 1) {  // taps: [channels, taps] -> [taps][channels]
             std::vector<uint8_t> t(v.size());
             for (int64_t i = 0; i < wr; i++)
                 for (int64_t k = 0; k < wc; k++) reinterpret_cast<float*>(t.data())[k * wr + i] = reinterpret_cast<const float*>(v.data())[i * wc + k];
             v.swap(t);
         }
-        if (post && (which == TSB_P_FINAL_NORM || which == TSB_P_NORM || which == TSB_P_NORM2))  // stored as the distance from one
+        if (m->shifted_gains() && (which == TSB_P_FINAL_NORM || which == TSB_P_NORM || which == TSB_P_NORM2))  // stored as the distance from one
             for (int64_t i = 0; i < wc; i++) reinterpret_cast<float*>(v.data())[i] += 1.f;
         if (!*vec && (rc = tsb_alloc(ctx, (size_t)n * 4, (void**)vec))) return rc;
         TSB_CUDA(ctx, cudaMemcpy(*vec, v.data(), v.size(), cudaMemcpyHostToDevice));
@@ -1277,6 +1407,9 @@ int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t
     }
     const size_t es = m->elem;
     convert(host, host_type, wr * wc, m->f32, v);
+    if (rotated > 0 && (which == TSB_P_Q || which == TSB_P_K)) pair_up(wr / D, D, rotated, (size_t)d * es);
+    if (c.value_rot && which == TSB_P_V) pair_up(G, E, E, (size_t)d * es);
+    if (c.value_rot && which == TSB_P_O) pair_up(d * H, E, E, es);
     if (which == TSB_P_EMBED || which == TSB_P_POSITIONS) {
         void*& table = which == TSB_P_EMBED ? m->embed : m->positions;
         if (!table && (rc = tsb_alloc(ctx, v.size(), &table))) return rc;
@@ -1357,6 +1490,10 @@ int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t
             for (int64_t h = 0; h < H; h++) PUT(l->out, 0, h * l->value_pad, 0, h * E, d, E);
             break;
         case TSB_P_FF_GATE: case TSB_P_FF_UP: {
+            if (c.ff_plain) {
+                PUT(l->ff_in, 0, 0, 0, 0, F, d);
+                break;
+            }
             const int64_t row0 = (seq ? 0 : at.pairs) + (which == TSB_P_FF_UP ? 8 : 0);
             for (int64_t x = 0; x < X; x++) {
                 PlainMat& mat = seq ? l->ff_in : l->in;
@@ -1378,8 +1515,8 @@ int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t
         case TSB_P_REC_Q: PUT(l->in, at.rec, 0, 0, 0, wr, d); break;
         case TSB_P_REC_K: PUT(l->in, at.rec + rh * RD, 0, 0, 0, wr, d); break;
         case TSB_P_REC_V: PUT(l->in, at.rec + (mlstm ? 2 : 1) * rh * RD, 0, 0, 0, wr, d); break;
-        case TSB_P_REC_GATE: PUT(l->in, at.rec + 2 * rh * RD + rh * RE, 0, 0, 0, wr, d); break;
-        case TSB_P_REC_I: PUT(l->in, at.rec_gate, 0, 0, 0, wr, d); break;
+        case TSB_P_REC_GATE: PUT(l->in, at.rec + (gru ? 0 : 2 * rh * RD + rh * RE), 0, 0, 0, wr, d); break;
+        case TSB_P_REC_I: PUT(l->in, at.rec_gate + (gru ? RE : 0), 0, 0, 0, wr, d); break;  // MINGRU: z, then the candidate
         case TSB_P_REC_F: PUT(l->in, at.rec_gate + (mlstm ? rh : 0), 0, 0, 0, wr, d); break;
         case TSB_P_REC_IN: PUT(l->in, at.rec, 0, 0, 0, wr, d); break;
         case TSB_P_REC_O: PUT(l->out, 0, l->o_cols, 0, 0, d, rh * RE); break;
@@ -1387,6 +1524,12 @@ int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t
 #undef PUT
     set |= 1ull << which;
     return TSB_OK;
+}
+
+int32_t tsb_model_set_plain(tsb_model* tm, int32_t layer, int32_t which, int32_t host_type, const void* host, int64_t rows, int64_t cols) {
+    const int32_t rc = set_plain(tm, layer, which, host_type, host, rows, cols);
+    if (rc == TSB_OK && which >= TSB_P_NORM && which != TSB_P_POSITIONS) mirror_layer(tm->plain, layer);
+    return rc;
 }
 
 int32_t tsb_model_fill_plain(tsb_model* tm, uint64_t seed) {
@@ -1406,7 +1549,7 @@ int32_t tsb_model_fill_plain(tsb_model* tm, uint64_t seed) {
     };
     auto matrix = [&](PlainMat& w, int64_t valid, float gain) { fill(&w.data, m->f32, w.rows, w.cols, valid, 0.f, gain * sqrtf(3.f / (float)valid)); };
     auto vector = [&](float*& p, int64_t n, float mid, float amp) { fill((void**)&p, true, 1, n, n, mid, amp); };
-    const int64_t d = m->cfg.d_model, gains = m->cfg.post_norm || m->cfg.output_norm ? d : 1;
+    const int64_t d = m->cfg.d_model, gains = m->sequential() ? d : 1;
     fill(&m->embed, m->f32, m->cfg.vocab, d, d, 0.f, 1.7f);
     matrix(m->head, d, 1.f);
     vector(m->final_gain, gains, 1.f, 0.f);
@@ -1414,12 +1557,13 @@ int32_t tsb_model_fill_plain(tsb_model* tm, uint64_t seed) {
     m->set = ~0ull;
     for (PlainLayer& l : m->layers) {
         const tsb_plain_layer& c = l.cfg;
+        if (l.tied >= 0) continue;
         matrix(l.in, d, 1.f);
         matrix(l.out, l.out.cols, 0.5f);
         vector(l.gain, gains, 1.f, 0.f);
         if (c.token_shift) vector(l.mu, d, 0.5f, 0.4f);
         if (c.log_bias) vector(l.r1, c.n_q_heads, 1.f, 0.5f), vector(l.r2, c.n_q_heads, 0.3f, 0.2f);
-        if (c.sink) vector(l.sink, c.n_q_heads, 0.f, 1.f);
+        if (c.sink == TSB_SINK_TENSOR) vector(l.sink, c.n_q_heads, 0.f, 1.f);
         const int64_t whole = c.qk_norm == TSB_NORM_PROJECTION ? 1 : 0;
         if (c.qk_norm) vector(l.q_norm, c.head_dim * (whole ? c.n_q_heads : 1), 1.f, 0.2f), vector(l.k_norm, c.head_dim * (whole ? c.n_kv_heads : 1), 1.f, 0.2f);
         auto experts = [&](PlainMat& w, int64_t valid, float gain) {
@@ -1430,7 +1574,7 @@ int32_t tsb_model_fill_plain(tsb_model* tm, uint64_t seed) {
         if (m->cfg.conv_taps > 0) vector(l.conv1, d * m->cfg.conv_taps, 0.f, 0.3f);
         if (m->cfg.conv_taps > 0 && c.ffn > 0) vector(l.conv2, d * m->cfg.conv_taps, 0.f, 0.3f);
         if (c.qkv_bias || c.recurrence) vector(l.in_bias, l.in.rows, 0.f, 0.2f);
-        if (c.recurrence) {
+        if (c.recurrence && c.recurrence != TSB_REC_MINGRU) {
             const int64_t inner = (int64_t)c.rec_heads * c.rec_vdim;
             vector(l.rec_norm, c.recurrence == TSB_REC_FORGET ? c.rec_vdim : inner, 1.f, 0.2f);
             if (c.recurrence == TSB_REC_FORGET) vector(l.rec_lower, (int64_t)c.rec_heads * c.rec_dim, 0.5f, 0.4f);
@@ -1445,6 +1589,7 @@ int32_t tsb_model_fill_plain(tsb_model* tm, uint64_t seed) {
         }
         l.set = ~0ull;
     }
+    for (int i = 0; i < m->cfg.n_layers; i++) mirror_layer(m, i);
     if (rc) return rc;
     TSB_CUDA(ctx, cudaDeviceSynchronize());
     return TSB_OK;
@@ -1484,12 +1629,39 @@ int32_t tsb_plain_gemm_pairs(tsb_ctx* ctx, tsb_stream s, int32_t type, const voi
     int32_t rc = check_gemm(ctx, type, w, rows, cols, x, x_rows, tokens, workspace);
     if (rc) return rc;
     TSB_REQUIRE(ctx, a && n_pairs > 0 && 2 * (int64_t)n_pairs <= rows && a_stride >= n_pairs, "bad output");
-    TSB_REQUIRE(ctx, act == TSB_ACT_GELU_TANH || act == TSB_ACT_SILU, "unknown activation");
+    TSB_REQUIRE(ctx, act >= TSB_ACT_GELU_TANH && act <= TSB_ACT_RELU2, "unknown activation");
     DeviceGuard g(ctx);
     PlainEpi e;
     e.kind = PLAIN_MIXER, e.pair_row0 = 0, e.n_pairs = n_pairs, e.act = act, e.a = a, e.a_stride = a_stride;
     TSB_CUDA(ctx, launch_plain_gemm(ctx, (cudaStream_t)s, type == TSB_F32, PlainMat{const_cast<void*>(w), rows, cols}, x, x, cols, x_rows, tokens, e,
                                     workspace));
+    return TSB_OK;
+}
+
+int32_t tsb_plain_gemm_act(tsb_ctx* ctx, tsb_stream s, int32_t type, const void* w, int64_t rows, int64_t cols, const void* x, int32_t x_rows, int32_t tokens,
+                           void* y, int64_t y_stride, int32_t n_valid, int32_t act, void* workspace) {
+    if (!ctx) return TSB_ERR_INVALID;
+    int32_t rc = check_gemm(ctx, type, w, rows, cols, x, x_rows, tokens, workspace);
+    if (rc) return rc;
+    TSB_REQUIRE(ctx, y && n_valid > 0 && n_valid <= rows && y_stride >= n_valid, "bad output");
+    TSB_REQUIRE(ctx, act >= TSB_ACT_GELU_TANH && act <= TSB_ACT_RELU2, "unknown activation");
+    DeviceGuard g(ctx);
+    PlainEpi e;
+    e.kind = PLAIN_MIXER, e.n_seg = 1, e.seg[0].end = n_valid, e.seg[0].act = act, e.seg[0].p = y, e.seg[0].stride = y_stride;
+    TSB_CUDA(ctx, launch_plain_gemm(ctx, (cudaStream_t)s, type == TSB_F32, PlainMat{const_cast<void*>(w), rows, cols}, x, nullptr, cols, x_rows, tokens, e, workspace));
+    return TSB_OK;
+}
+
+int32_t tsb_plain_gemm_add(tsb_ctx* ctx, tsb_stream s, int32_t type, const void* w, int64_t rows, int64_t cols, const void* x, int32_t x_rows, int32_t tokens,
+                           float* y, int64_t y_stride, int32_t n_valid, float alpha, float beta, void* workspace) {
+    if (!ctx) return TSB_ERR_INVALID;
+    int32_t rc = check_gemm(ctx, type, w, rows, cols, x, x_rows, tokens, workspace);
+    if (rc) return rc;
+    TSB_REQUIRE(ctx, y && n_valid > 0 && n_valid <= rows && y_stride >= n_valid, "bad output");
+    DeviceGuard g(ctx);
+    PlainEpi e;
+    e.kind = PLAIN_ADD, e.y = y, e.y_stride = y_stride, e.n_valid = n_valid, e.alpha = alpha, e.beta = beta;
+    TSB_CUDA(ctx, launch_plain_gemm(ctx, (cudaStream_t)s, type == TSB_F32, PlainMat{const_cast<void*>(w), rows, cols}, x, nullptr, cols, x_rows, tokens, e, workspace));
     return TSB_OK;
 }
 
@@ -1517,10 +1689,15 @@ int32_t tsb_kv_create_keys(tsb_ctx* ctx, int32_t type, int32_t layers, int32_t k
 
 int32_t tsb_kv_create_plain(tsb_ctx* ctx, int32_t type, int32_t layers, int32_t kv_heads, int32_t key_dim, int32_t value_dim, int32_t page_tokens,
                             int32_t num_pages, int32_t max_seqs, int32_t max_pages_per_seq, tsb_kv** out) {
+    return tsb_kv_create_blocks(ctx, type, layers, kv_heads, key_dim, value_dim, 0, page_tokens, num_pages, max_seqs, max_pages_per_seq, out);
+}
+
+int32_t tsb_kv_create_blocks(tsb_ctx* ctx, int32_t type, int32_t layers, int32_t kv_heads, int32_t key_dim, int32_t value_dim, int32_t pool, int32_t page_tokens,
+                             int32_t num_pages, int32_t max_seqs, int32_t max_pages_per_seq, tsb_kv** out) {
     if (!ctx || !out) return TSB_ERR_INVALID;
-    TSB_REQUIRE(ctx, (type == TSB_BF16 || type == TSB_F32) && layers > 0 && kv_heads > 0, "unknown type or bad sizes");
+    TSB_REQUIRE(ctx, (type == TSB_BF16 || type == TSB_F32) && layers > 0 && kv_heads > 0 && pool >= 0, "unknown type or bad sizes");
     std::vector<KeyLayerShape> shapes;
-    for (int l = 0; l < layers; l++) shapes.push_back({kv_heads, key_dim, value_dim, l});
+    for (int l = 0; l < layers; l++) shapes.push_back({kv_heads, key_dim, value_dim, l, pool});
     return kv_create_keys(ctx, layers, shapes.data(), type == TSB_F32 ? 4 : 2, page_tokens, num_pages, max_seqs, max_pages_per_seq, out);
 }
 
@@ -1561,6 +1738,8 @@ int32_t tsb_plain_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, int32_t la
     TSB_REQUIRE(ctx, q && out && rows_dev && group_rows && n_groups > 0 && scratch && (x.r1 == nullptr) == (x.r2 == nullptr) && x.window >= 0 &&
                          x.chunk >= 0 && !(x.window && x.chunk) && !(x.r1 && x.slopes), "bad arguments");
     const KeyView& kv = keys->key_layers[layer];
+    TSB_REQUIRE(ctx, x.keep >= 0 && ((x.keep == 0 && !x.blocks) || (x.window > 0 && kv.value_off > 0 && !x.r1 && !x.slopes && !(x.keep && x.blocks))) &&
+                         (!x.blocks || keys->pool_sizes[layer] > 0), "a prefix goes with a window over values of their own and no distance bias");
     const bool f32 = kv.elem_bytes == 4;
     const int vd = kv.value_off ? kv.head_step - kv.value_off : kv.head_dim;
     const bool wide = vd != kv.head_dim;  // keys and values of different widths: the many-query kernel alone takes them
@@ -1571,6 +1750,7 @@ int32_t tsb_plain_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, int32_t la
     TSB_REQUIRE(ctx, (uintptr_t)q % 32 == 0 && (uintptr_t)out % 32 == 0 && q_stride % 16 == 0 && out_stride % 16 == 0 &&
                          q_stride >= (int64_t)n_q_heads * kv.head_dim && out_stride >= (int64_t)n_q_heads * vd,
                 "q and out rows hold every head and start on 32-byte boundaries (strides a multiple of 16)");
+    TSB_REQUIRE(ctx, !x.turn || (x.turn_half > 0 && 2 * x.turn_half <= vd && (uintptr_t)x.turn % 8 == 0 && !wide), "turned columns are a head's first ones");
     TSB_REQUIRE(ctx, !x.value_gate || ((uintptr_t)x.value_gate % 32 == 0 && x.value_gate_stride % 16 == 0 && x.value_gate_stride >= (int64_t)n_q_heads * vd),
                 "rows of value gates hold every head and start on 32-byte boundaries");
     cudaStream_t st = (cudaStream_t)s;
@@ -1580,6 +1760,8 @@ int32_t tsb_plain_attention(tsb_ctx* ctx, tsb_stream s, tsb_kv* keys, int32_t la
     a.n_q_heads = n_q_heads, a.scale = scale, a.cap = x.cap, a.r1 = x.r1, a.r2 = x.r2, a.window = x.window;
     a.sink = x.sink, a.value_gate = x.value_gate, a.value_gate_stride = x.value_gate_stride, a.value_dim = vd;
     a.slopes = x.slopes, a.chunk = x.chunk, a.out_scale = x.out_scale == 0.f ? 1.f : x.out_scale;
+    a.keep = x.keep, a.turn = reinterpret_cast<const float2*>(x.turn), a.turn_half = x.turn ? x.turn_half : 0;
+    if (x.blocks) a.pool = keys->pool_sizes[layer], a.pooled = keys->pooled_layers[layer];
     AttnBatch b;
     b.max_len = max_len;
     bool uniform = true;

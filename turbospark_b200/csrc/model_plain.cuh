@@ -6,6 +6,7 @@
 #include "model.cuh"
 #include "recurrence.cuh"
 #include "rowops_plain.cuh"
+#include "scan.cuh"
 #include "sublayer.cuh"
 
 // attention: values that are the keys; values of their own; latent rows; none (the layer's mixer is a recurrence alone)
@@ -14,7 +15,8 @@ enum PlainMixer { MIX_KEYS = 0, MIX_KV = 1, MIX_LATENT = 2, MIX_NONE = 3 };
 struct PlainLayer {
     tsb_plain_layer cfg{};
     PlainMixer mixer = MIX_KEYS;
-    bool post_norm = false;    // one of the forms whose sublayers follow each other (post-norm, output norm)
+    bool post_norm = false;    // one of the forms whose sublayers follow each other (post-norm, output norm, pre-norm)
+    int tied = -1;             // the layer whose tensors this one uses
     int source = 0;            // the layer whose cache rows this one reads
     int head_pad = 0;          // head size the attention kernels work on; latent layers: columns of a head in q (and of an expanded key)
     int value_pad = 0;         // columns of a head in the attention's output
@@ -22,14 +24,14 @@ struct PlainLayer {
     int q_rows = 0, k_rows = 0;
     int ffn_pad = 0;           // feed-forward width, padded
     int o_cols = 0;            // columns of the output projection before the feed-forward's (padded)
-    int rotation = -1;         // which of the model's rotations
+    int rotation = -1, value_rotation = -1;  // which of the model's rotations
     bool expands = false;      // long portions expand the latents to keys and values
     int rec_cols = 0;          // columns of the output projection that belong to the recurrence (padded), behind the heads'
     // parallel form: in = [queries | keys | head gates | (gate, up) pairs] x d, out = d x [heads | feed-forward]
     // post-norm form: in = [queries | keys | values] x d or [queries | latent | value gates | rotated pairs] x d, out = d x heads
     // output-norm form: in = [queries | keys | values | value gates | recurrence's vectors | recurrence's gates] x d, out = d x [heads | recurrence]
     PlainMat in, out;
-    PlainMat ff_in, ff_out;    // post-norm and output-norm form; with experts: one expert's shape, the matrices one after another
+    PlainMat ff_in, ff_out;    // forms whose sublayers follow each other; with experts: one expert's shape, the matrices one after another
     PlainMat router;
     float *in_bias = nullptr, *slopes = nullptr, *conv1 = nullptr, *conv2 = nullptr, *correction = nullptr;
     float *rec_lower = nullptr, *rec_norm = nullptr, *rec_conv = nullptr, *rec_conv_bias = nullptr, *rec_a_log = nullptr, *rec_skip = nullptr;
@@ -66,13 +68,15 @@ struct PlainModel {
     PlainMat head;
     void* embed = nullptr;     // [vocab, d], natural rows
     void* positions = nullptr;  // [positions, d]
-    float* final_gain = nullptr;  // [1], or [d] in a post-norm or output-norm model
+    float* final_gain = nullptr;  // [1], or [d] where the sublayers follow each other
     uint64_t set = 0;
     bool owned = true;
     bool any_shift = false;
+    bool sequential() const { return cfg.post_norm || cfg.output_norm || cfg.pre_norm; }
+    bool shifted_gains() const { return cfg.post_norm || cfg.pre_norm; }  // norm weights are given as their distance from one
 };
 
-// What the streams of an output-norm model keep from row to row.
+// What the streams of an output-norm or pre-norm model keep from row to row.
 struct StreamStates {
     int ring = 0;                           // states of a recurrence kept per stream
     int row_ring = 0, keep = 0;             // rows kept of a convolution's input; the most that any convolution looks back
@@ -102,7 +106,7 @@ struct PlainRt {
     std::vector<float2*> rotary;  // per rotation: [rows, dims / 2]
     ExpandRt expand;
     int fin_rows = 0;
-    // output-norm form
+    // output-norm form; recurrences
     float *x2 = nullptr, *y = nullptr, *rec_out = nullptr, *router_logits = nullptr;
     void *rec = nullptr, *rec_mixed = nullptr, *expert_in = nullptr, *expert_act = nullptr, *expert_out = nullptr;
     int64_t rec_stride = 0, rec_mixed_stride = 0, rec_out_stride = 0, raw_rec = 0;  // raw_rec: where the recurrence's numbers start in a raw row

@@ -1,6 +1,8 @@
-// The mechanisms of output-norm layers as operators (include/tsb.h).
+// The mechanisms of output-norm and pre-norm layers as operators (include/tsb.h).
 #include "gemm_plain.cuh"
 #include "recurrence.cuh"
+#include "rowops_plain.cuh"
+#include "scan.cuh"
 #include "sublayer.cuh"
 
 namespace {
@@ -163,6 +165,67 @@ int32_t tsb_plain_gemm_experts(tsb_ctx* ctx, tsb_stream s, int32_t type, const v
     if (pairs) p.pair_row0 = 0, p.n_pairs = n_valid, p.act = PLAIN_SILU, p.a = y, p.a_stride = y_stride;
     else p.n_seg = 1, p.seg[0].end = n_valid, p.seg[0].p = y, p.seg[0].stride = y_stride;
     TSB_CUDA(ctx, launch_plain_gemm_experts(ctx, (cudaStream_t)s, type == TSB_F32, tensor != 0, PlainMat{const_cast<void*>(w), w_rows, cols}, x, x_stride, x_rows, e, p));
+    return TSB_OK;
+}
+
+int32_t tsb_pre_norm_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, const float* x, int32_t d, const float* weight, float eps, int32_t rows, void* out,
+                          int64_t out_stride) {
+    if (!ctx) return TSB_ERR_INVALID;
+    TSB_REQUIRE(ctx, known(type) && x && weight && out && d > 0 && rows > 0 && out_stride >= d, "bad arguments");
+    TSB_REQUIRE(ctx, (uintptr_t)x % 16 == 0 && (uintptr_t)weight % 16 == 0 && (uintptr_t)out % 16 == 0, "buffers must be 16-byte aligned");
+    DeviceGuard g(ctx);
+    TSB_CUDA(ctx, launch_pre_norm(ctx, (cudaStream_t)s, type == TSB_F32, x, d, weight, eps, rows, out, out_stride));
+    return TSB_OK;
+}
+
+int32_t tsb_turned_norm_rows(tsb_ctx* ctx, tsb_stream s, tsb_kv* cache, int32_t layer, const tsb_turned_norms* n, const tsb_row_desc* rows_dev, int32_t rows) {
+    if (!ctx || !cache || !n) return TSB_ERR_INVALID;
+    TSB_REQUIRE(ctx, !cache->key_layers.empty() && layer >= 0 && layer < (int)cache->key_layers.size(), "a plain cache and one of its layers expected");
+    const KeyView& kv = cache->key_layers[layer];
+    TSB_REQUIRE(ctx, n->raw && rows_dev && rows > 0 && n->n_q > 0 && n->n_k > 0 && n->n_k <= kv.kv_heads && n->width > 0 && n->width <= kv.head_dim && n->q && n->q_weight &&
+                         n->k_weight && n->n_v >= 0 && n->n_v <= kv.kv_heads && n->raw_stride >= (int64_t)(n->n_q + n->n_k) * n->width + (int64_t)n->n_v * n->v_width &&
+                         n->q_stride >= (int64_t)n->n_q * kv.head_dim, "bad arguments");
+    TSB_REQUIRE(ctx, n->n_v == 0 || (!n->projection && n->v_width > 0 && kv.value_off > 0 && n->v_width <= kv.head_step - kv.value_off), "the cache has no room for the values");
+    TSB_REQUIRE(ctx, (!n->rot || (n->rot_half > 0 && 2 * n->rot_half <= n->width)) && (!n->turn || (n->turn_half > 0 && 2 * n->turn_half <= n->v_width)), "more columns are turned than there are");
+    const float2 *rot = reinterpret_cast<const float2*>(n->rot), *turn = reinterpret_cast<const float2*>(n->turn);
+    DeviceGuard g(ctx);
+    if (n->projection) {
+        ProjectionNorms p;
+        p.raw = n->raw, p.raw_stride = n->raw_stride, p.n_q = n->n_q, p.n_k = n->n_k, p.width = n->width, p.q_weight = n->q_weight, p.k_weight = n->k_weight, p.eps = n->eps;
+        p.q = n->q, p.q_stride = n->q_stride, p.q_step = kv.head_dim, p.keys = kv, p.rows = rows_dev, p.rot = rot, p.rot_half = rot ? n->rot_half : 0;
+        TSB_CUDA(ctx, launch_projection_norms(ctx, (cudaStream_t)s, kv.elem_bytes == 4, p, rows));
+        return TSB_OK;
+    }
+    HeadNorms h;
+    h.raw = n->raw, h.raw_stride = n->raw_stride, h.n_q = n->n_q, h.n_k = n->n_k, h.n_v = n->n_v, h.width = n->width, h.v_width = n->v_width, h.q_weight = n->q_weight;
+    h.k_weight = n->k_weight, h.eps = n->eps, h.q = n->q, h.q_stride = n->q_stride, h.q_step = h.q_width = kv.head_dim, h.keys = kv, h.rows = rows_dev;
+    h.rot = rot, h.rot_half = rot ? n->rot_half : 0, h.turn = turn, h.turn_half = turn ? n->turn_half : 0;
+    TSB_CUDA(ctx, launch_head_norms(ctx, (cudaStream_t)s, kv.elem_bytes == 4, h, rows));
+    return TSB_OK;
+}
+
+int32_t tsb_block_mean_rows(tsb_ctx* ctx, tsb_stream s, tsb_kv* cache, int32_t layer, const tsb_row_desc* rows_dev, int32_t rows) {
+    if (!ctx || !cache) return TSB_ERR_INVALID;
+    TSB_REQUIRE(ctx, layer >= 0 && layer < (int)cache->pool_sizes.size() && cache->pool_sizes[layer] > 0 && rows_dev && rows > 0, "a layer that keeps blocks expected");
+    DeviceGuard g(ctx);
+    BlockMeans b;
+    b.keys = cache->key_layers[layer], b.pooled = cache->pooled_layers[layer], b.pool = cache->pool_sizes[layer], b.rows = rows_dev;
+    TSB_CUDA(ctx, launch_block_means(ctx, (cudaStream_t)s, b.keys.elem_bytes == 4, b, rows));
+    return TSB_OK;
+}
+
+int32_t tsb_gated_scan_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, const float* gate, int64_t gate_stride, const void* out_gate, int64_t out_gate_stride, int32_t width,
+                            float* state, int32_t n_streams, int32_t ring, const tsb_row_desc* rows_dev, int32_t rows, int32_t rows_per_seq, void* out, int64_t out_stride) {
+    if (!ctx) return TSB_ERR_INVALID;
+    int32_t rc = check_portions(ctx, rows_dev, rows, rows_per_seq);
+    if (rc) return rc;
+    TSB_REQUIRE(ctx, known(type) && gate && out_gate && state && out && width > 0 && gate_stride >= 2 * (int64_t)width && out_gate_stride >= width && out_stride >= width, "bad arguments");
+    TSB_REQUIRE(ctx, power_of_two(ring) && ring > 1 && n_streams > 0, "ring is a power of two above one");
+    DeviceGuard g(ctx);
+    GatedScan x;
+    x.gate = gate, x.gate_stride = gate_stride, x.out_gate = out_gate, x.out_gate_stride = out_gate_stride, x.out = out, x.out_stride = out_stride, x.width = width;
+    x.state.s = state, x.state.ring = ring, x.state.n_streams = n_streams, x.rows = rows_dev;
+    TSB_CUDA(ctx, launch_gated_scan(ctx, (cudaStream_t)s, type == TSB_F32, x, RowTiles::uniform(rows, rows_per_seq, rows_per_seq)));
     return TSB_OK;
 }
 

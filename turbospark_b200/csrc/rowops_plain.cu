@@ -1,6 +1,8 @@
 // Row operators of the plain-weight decoders (rowops_plain.cuh).
 #include <cuda_bf16.h>
 
+#include <algorithm>
+
 #include "rowops_plain.cuh"
 
 namespace {
@@ -175,8 +177,9 @@ __global__ void __launch_bounds__(ROW_THREADS)
 // VEC as in the norm + shift kernel: a thread holds its columns of the row in registers.
 template <typename T, bool VEC>
 __global__ void __launch_bounds__(ROW_THREADS)
-    post_norm_kernel(float* x, int d, const float* __restrict__ weight, float eps, T* out, int64_t out_stride) {
-    float* xr = x + (int64_t)blockIdx.x * d;
+    post_norm_kernel(const float* x, float* x_out, int d, const float* __restrict__ weight, float eps, T* out, int64_t out_stride) {
+    const float* xr = x + (int64_t)blockIdx.x * d;
+    float* xo = x_out ? x_out + (int64_t)blockIdx.x * d : nullptr;  // may be the row itself
     T* o = out + (int64_t)blockIdx.x * out_stride;
     float4 w[VEC ? ROW_VECS : 1];
     if (VEC) {
@@ -204,7 +207,7 @@ __global__ void __launch_bounds__(ROW_THREADS)
             const int i = (k * ROW_THREADS + threadIdx.x) * 4;
             if (i >= d) break;
             const float4 h = make_float4(v[k].x * s * w[k].x, v[k].y * s * w[k].y, v[k].z * s * w[k].z, v[k].w * s * w[k].w);
-            put4(xr + i, h);
+            if (xo) put4(xo + i, h);
             put4(o + i, h);
         }
         return;
@@ -213,9 +216,17 @@ __global__ void __launch_bounds__(ROW_THREADS)
     const float s = 1.f / sqrtf(block_sum2(ss).x / (float)d + eps);
     for (int i = threadIdx.x; i < d; i += ROW_THREADS) {
         const float h = xr[i] * s * weight[i];
-        xr[i] = h;
+        if (xo) xo[i] = h;
         put(o + i, h);
     }
+}
+
+// the pair of columns i and i + 1 (i even), turned; columns behind the turned ones pass
+__device__ __forceinline__ void turn_pair(const float2* table, int half, int r, int i, float& u, float& v) {
+    if (i >= 2 * half) return;
+    const float2 t = table[(int64_t)r * half + (i >> 1)];
+    const float x = fmaf(u, t.x, -v * t.y);
+    v = fmaf(v, t.x, u * t.y), u = x;
 }
 
 // LANES lanes per (row, head).  VEC > 0: the width is a multiple of four and at most 4 LANES VEC, and a lane holds its columns in
@@ -224,15 +235,42 @@ template <typename T, int LANES, int VEC>
 __global__ void __launch_bounds__(ROW_THREADS) head_norms_kernel(const __grid_constant__ HeadNorms h, int rows, uint32_t* __restrict__ err) {
     const int lane = threadIdx.x & (LANES - 1);
     const int64_t item = (int64_t)blockIdx.x * (ROW_THREADS / LANES) + threadIdx.x / LANES;
-    const int per = h.n_q + h.n_k;
+    const int per = h.n_q + h.n_k + h.n_v;
     const bool in = item < (int64_t)rows * per;
     const int r = in ? (int)(item / per) : 0, head = in ? (int)(item % per) : 0;
     const tsb_row_desc rd = h.rows[r];
     pdl_wait();
     pdl_launch_dependents();
     if (!in) return;
-    const bool query = head < h.n_q;
+    const bool query = head < h.n_q, value = head >= h.n_q + h.n_k;
     const float* src = h.raw + (int64_t)r * h.raw_stride + (int64_t)head * h.width;
+    if (value) {
+        src += (int64_t)(head - h.n_q - h.n_k) * (h.v_width - h.width);
+        T* dst = key_row<T>(h.keys, rd.seq, rd.base + rd.slot);
+        if (!dst) {
+            if (lane == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+            return;
+        }
+        dst += (int64_t)(head - h.n_q - h.n_k) * h.keys.head_step + h.keys.value_off;
+        if (VEC > 0) {
+#pragma unroll
+            for (int k = 0; k < VEC; k++) {
+                const int i = (k * LANES + lane) * 4;
+                if (i >= h.v_width) break;
+                float4 v = *reinterpret_cast<const float4*>(src + i);
+                turn_pair(h.turn, h.turn_half, r, i, v.x, v.y), turn_pair(h.turn, h.turn_half, r, i + 2, v.z, v.w);
+                put4(dst + i, v);
+            }
+            return;
+        }
+        for (int i = 2 * lane; i < h.v_width; i += 2 * LANES) {
+            float u = src[i], v = i + 1 < h.v_width ? src[i + 1] : 0.f;
+            turn_pair(h.turn, h.turn_half, r, i, u, v);
+            put(dst + i, u);
+            if (i + 1 < h.v_width) put(dst + i + 1, v);
+        }
+        return;
+    }
     const float* w = query ? h.q_weight : h.k_weight;
     float ss = 0.f;
     float4 v[VEC > 0 ? VEC : 1], g[VEC > 0 ? VEC : 1];
@@ -271,12 +309,20 @@ __global__ void __launch_bounds__(ROW_THREADS) head_norms_kernel(const __grid_co
 #pragma unroll
         for (int k = 0; k < VEC; k++) {
             const int i = (k * LANES + lane) * 4;
-            if (i < h.width) put4(dst + i, make_float4(v[k].x * s * g[k].x, v[k].y * s * g[k].y, v[k].z * s * g[k].z, v[k].w * s * g[k].w));
+            if (i >= h.width) break;
+            float4 o = make_float4(v[k].x * s * g[k].x, v[k].y * s * g[k].y, v[k].z * s * g[k].z, v[k].w * s * g[k].w);
+            if (h.rot) turn_pair(h.rot, h.rot_half, r, i, o.x, o.y), turn_pair(h.rot, h.rot_half, r, i + 2, o.z, o.w);
+            put4(dst + i, o);
         }
         for (int i = h.width + lane; i < width; i += LANES) put(dst + i, 0.f);
         return;
     }
-    for (int i = lane; i < width; i += LANES) put(dst + i, i < h.width ? src[i] * s * w[i] : 0.f);
+    for (int i = 2 * lane; i < width; i += 2 * LANES) {
+        float u = i < h.width ? src[i] * s * w[i] : 0.f, v = i + 1 < h.width ? src[i + 1] * s * w[i + 1] : 0.f;
+        if (h.rot) turn_pair(h.rot, h.rot_half, r, i, u, v);
+        put(dst + i, u);
+        if (i + 1 < width) put(dst + i + 1, v);
+    }
 }
 
 __global__ void __launch_bounds__(ROW_THREADS)
@@ -292,6 +338,38 @@ __global__ void __launch_bounds__(ROW_THREADS)
     float s, c;
     sincosf((float)a, &s, &c);
     table[k] = make_float2(magnitude * c, magnitude * s);
+}
+
+// Rows that end no block leave at once; a thread sums eight (f32: four) columns.
+template <typename T>
+__global__ void __launch_bounds__(ROW_THREADS) block_means_kernel(const __grid_constant__ BlockMeans b, uint32_t* __restrict__ err) {
+    constexpr int N = 16 / sizeof(T);
+    const tsb_row_desc rd = b.rows[blockIdx.x];
+    const int pos = rd.base + rd.slot, block = pos / b.pool;
+    pdl_wait();
+    pdl_launch_dependents();
+    if (pos - block * b.pool != b.pool - 1) return;
+    T* dst = key_row<T>(b.pooled, rd.seq, block);
+    if (!dst) {
+        if (threadIdx.x == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+        return;
+    }
+    for (int c = threadIdx.x * N; c < b.keys.row; c += ROW_THREADS * N) {
+        float sum[N];
+#pragma unroll
+        for (int i = 0; i < N; i++) sum[i] = 0.f;
+#pragma unroll 8
+        for (int j = 0; j < b.pool; j++) {
+            const T* src = key_row<T>(b.keys, rd.seq, block * b.pool + j);
+            if (!src) continue;  // positions before a reserved one are reserved
+            const uint4 v = *reinterpret_cast<const uint4*>(src + c);
+            const T* e = reinterpret_cast<const T*>(&v);
+#pragma unroll
+            for (int i = 0; i < N; i++) sum[i] += get(e + i);
+        }
+#pragma unroll
+        for (int i = 0; i < N; i++) put(dst + c + i, sum[i] / (float)b.pool);
+    }
 }
 
 // a CTA per position and stream
@@ -361,29 +439,45 @@ cudaError_t launch_norm_rows(tsb_ctx* ctx, cudaStream_t st, bool f32, const floa
                       want_first, want_step, (__nv_bfloat16*)out, out_stride);
 }
 
-cudaError_t launch_post_norm(tsb_ctx* ctx, cudaStream_t st, bool f32, float* x, int d, const float* weight, float eps, int rows, void* out,
-                             int64_t out_stride) {
-    auto run = [&](auto kernel, auto* o) { return tsb_launch(ctx, kernel, dim3((unsigned)rows), dim3(ROW_THREADS), 0, st, true, x, d, weight, eps, o, out_stride); };
+static cudaError_t launch_norm_of(tsb_ctx* ctx, cudaStream_t st, bool f32, const float* x, float* x_out, int d, const float* weight, float eps, int rows, void* out,
+                                  int64_t out_stride) {
+    auto run = [&](auto kernel, auto* o) {
+        return tsb_launch(ctx, kernel, dim3((unsigned)rows), dim3(ROW_THREADS), 0, st, true, x, x_out, d, weight, eps, o, out_stride);
+    };
     const bool vec = d % 4 == 0 && out_stride % 4 == 0 && d <= 4 * ROW_THREADS * ROW_VECS;
     if (f32) return run(vec ? post_norm_kernel<float, true> : post_norm_kernel<float, false>, (float*)out);
     return run(vec ? post_norm_kernel<__nv_bfloat16, true> : post_norm_kernel<__nv_bfloat16, false>, (__nv_bfloat16*)out);
+}
+cudaError_t launch_post_norm(tsb_ctx* ctx, cudaStream_t st, bool f32, float* x, int d, const float* weight, float eps, int rows, void* out,
+                             int64_t out_stride) {
+    return launch_norm_of(ctx, st, f32, x, x, d, weight, eps, rows, out, out_stride);
+}
+cudaError_t launch_pre_norm(tsb_ctx* ctx, cudaStream_t st, bool f32, const float* x, int d, const float* weight, float eps, int rows, void* out,
+                            int64_t out_stride) {
+    return launch_norm_of(ctx, st, f32, x, nullptr, d, weight, eps, rows, out, out_stride);
 }
 
 cudaError_t launch_head_norms(tsb_ctx* ctx, cudaStream_t st, bool f32, const HeadNorms& h, int rows) {
     auto run = [&](auto kernel, int lanes) {
         const int per_cta = ROW_THREADS / lanes;
-        const dim3 grid((unsigned)(((int64_t)rows * (h.n_q + h.n_k) + per_cta - 1) / per_cta));
+        const dim3 grid((unsigned)(((int64_t)rows * (h.n_q + h.n_k + h.n_v) + per_cta - 1) / per_cta));
         return tsb_launch(ctx, kernel, grid, dim3(ROW_THREADS), 0, st, true, h, rows, ctx->dev_error);
     };
-    const bool vec = h.width % 4 == 0 && h.width <= 512 && h.raw_stride % 4 == 0 && (uintptr_t)h.raw % 16 == 0 && h.q_step % 4 == 0 && h.q_stride % 4 == 0;
+    const int wide = h.n_v > 0 ? std::max(h.width, h.v_width) : h.width;
+    const bool vec = h.width % 4 == 0 && (h.n_v == 0 || h.v_width % 4 == 0) && wide <= 512 && h.raw_stride % 4 == 0 && (uintptr_t)h.raw % 16 == 0 && h.q_step % 4 == 0 && h.q_stride % 4 == 0;
     if (f32) {
-        if (vec && h.width <= 64) return run(head_norms_kernel<float, 8, 2>, 8);
-        if (vec && h.width <= 128) return run(head_norms_kernel<float, 16, 2>, 16);
+        if (vec && wide <= 64) return run(head_norms_kernel<float, 8, 2>, 8);
+        if (vec && wide <= 128) return run(head_norms_kernel<float, 16, 2>, 16);
         return vec ? run(head_norms_kernel<float, 32, 4>, 32) : run(head_norms_kernel<float, 32, 0>, 32);
     }
-    if (vec && h.width <= 64) return run(head_norms_kernel<__nv_bfloat16, 8, 2>, 8);
-    if (vec && h.width <= 128) return run(head_norms_kernel<__nv_bfloat16, 16, 2>, 16);
+    if (vec && wide <= 64) return run(head_norms_kernel<__nv_bfloat16, 8, 2>, 8);
+    if (vec && wide <= 128) return run(head_norms_kernel<__nv_bfloat16, 16, 2>, 16);
     return vec ? run(head_norms_kernel<__nv_bfloat16, 32, 4>, 32) : run(head_norms_kernel<__nv_bfloat16, 32, 0>, 32);
+}
+
+cudaError_t launch_block_means(tsb_ctx* ctx, cudaStream_t st, bool f32, const BlockMeans& b, int rows) {
+    auto run = [&](auto kernel) { return tsb_launch(ctx, kernel, dim3((unsigned)rows), dim3(ROW_THREADS), 0, st, true, b, ctx->dev_error); };
+    return f32 ? run(block_means_kernel<float>) : run(block_means_kernel<__nv_bfloat16>);
 }
 
 cudaError_t launch_rotary_table(tsb_ctx* ctx, cudaStream_t st, const double* freq, int half, float magnitude, const tsb_row_desc* rows_dev, int rows,

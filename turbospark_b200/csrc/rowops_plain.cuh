@@ -30,11 +30,16 @@ cudaError_t launch_norm_rows(tsb_ctx* ctx, cudaStream_t st, bool f32, const floa
 // Norm after the sum, in place: x[r, :] = x * weight / sqrt(mean(x^2) + eps) in f32, and in the compute type to out.
 cudaError_t launch_post_norm(tsb_ctx* ctx, cudaStream_t st, bool f32, float* x, int d, const float* weight, float eps, int rows, void* out,
                              int64_t out_stride);
+// The same without rewriting x: the input of a pre-norm sublayer.
+cudaError_t launch_pre_norm(tsb_ctx* ctx, cudaStream_t st, bool f32, const float* x, int d, const float* weight, float eps, int rows, void* out,
+                            int64_t out_stride);
 
 // Norms over the heads of a projection: raw [rows, raw_stride] f32 holds n_q heads of `width` numbers, then n_k such heads.
 // Each is normed over its width with the weight of its kind; queries are scaled by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1)
 // at position p (temp_every 0: not) and stored to q at (head * q_step) with zeros up to q_width; keys go to the token's cache row
-// at (head * keys.head_step).  n_q = 0, n_k = 1 is the norm of a latent.
+// at (head * keys.head_step).  n_q = 0, n_k = 1 is the norm of a latent.  With `rot`, columns 2 i and 2 i + 1 of a normed head are turned by
+// (cos, sin) of [rows, rot_half].  n_v heads of v_width numbers behind the keys are values: not normed, turned by `turn`, stored keys.value_off
+// elements into the cache's heads.
 struct HeadNorms {
     const float* raw = nullptr;
     int64_t raw_stride = 0;
@@ -46,10 +51,21 @@ struct HeadNorms {
     void* q = nullptr;
     int64_t q_stride = 0;
     int q_step = 0, q_width = 0;
+    const float2 *rot = nullptr, *turn = nullptr;
+    int rot_half = 0, turn_half = 0, n_v = 0, v_width = 0;
     KeyView keys{};
     const tsb_row_desc* rows = nullptr;
 };
 cudaError_t launch_head_norms(tsb_ctx* ctx, cudaStream_t st, bool f32, const HeadNorms& h, int rows);
+
+// Rows of blocks (KeyLayerShape::pool): where a row of the pass is the last position of a block of `pool`, the block's row becomes the mean of the cache's
+// rows at its positions - all of them written before - summed in f32 in their order.
+struct BlockMeans {
+    KeyView keys{}, pooled{};
+    int pool = 0;
+    const tsb_row_desc* rows = nullptr;
+};
+cudaError_t launch_block_means(tsb_ctx* ctx, cudaStream_t st, bool f32, const BlockMeans& b, int rows);
 
 // table[r, i] = magnitude * (cos, sin)(position of row r * freq[i]), i below half; the product is reduced to one turn in double
 cudaError_t launch_rotary_table(tsb_ctx* ctx, cudaStream_t st, const double* freq, int half, float magnitude, const tsb_row_desc* rows_dev, int rows,

@@ -355,7 +355,24 @@ __global__ void __launch_bounds__(THREADS) projection_norms_kernel(const __grid_
         const Vec<W> g = load(w + i, Vec<W>());
 #pragma unroll
         for (int j = 0; j < W; j++) v.v[j] *= f * g.v[j];
-        store(dst + (int64_t)(i / p.width) * step + i % p.width, v);
+        const int at = i % p.width;
+        if (p.rot) {
+#pragma unroll
+            for (int j = 0; j < W; j++) {
+                const int c = at + j;
+                if (c >= 2 * p.rot_half || (W > 1 && (j & 1))) continue;
+                const float2 t = p.rot[(int64_t)r * p.rot_half + (c >> 1)];
+                if (W == 1) {  // the other column of the pair is another thread's
+                    const int other = i - at + (at ^ 1);
+                    const float o = src[other] * f * w[other];
+                    v.v[0] = c & 1 ? fmaf(v.v[0], t.x, o * t.y) : fmaf(v.v[0], t.x, -o * t.y);
+                } else {
+                    const float a = v.v[j], b = v.v[(j + 1) % W];
+                    v.v[j] = fmaf(a, t.x, -b * t.y), v.v[(j + 1) % W] = fmaf(b, t.x, a * t.y);
+                }
+            }
+        }
+        store(dst + (int64_t)(i / p.width) * step + at, v);
     };
 #pragma unroll
     for (int k = 0; k < HELD; k++)

@@ -48,7 +48,7 @@ cudaError_t launch_group_norm_rows(tsb_ctx* ctx, cudaStream_t st, bool f32, cons
 
 // Norms of whole projections: raw [rows, raw_stride] f32 holds n_q heads of `width` numbers, then n_k heads.  All queries of a row are
 // normed at once, and all keys; weights [n_q * width] and [n_k * width].  Queries go to q (head * q_step, zeros up to q_step), keys to the
-// token's cache row (head * keys.head_step).
+// token's cache row (head * keys.head_step).  With `rot`, columns 2 i and 2 i + 1 of a normed head are turned by (cos, sin) of [rows, rot_half].
 struct ProjectionNorms {
     const float* raw = nullptr;
     int64_t raw_stride = 0;
@@ -58,6 +58,8 @@ struct ProjectionNorms {
     void* q = nullptr;
     int64_t q_stride = 0;
     int q_step = 0;
+    const float2* rot = nullptr;
+    int rot_half = 0;
     KeyView keys{};
     const tsb_row_desc* rows = nullptr;
 };

@@ -7,19 +7,21 @@ from .capi import lib
 from .model import Model
 
 BF16, F32 = 0, 1
-GELU_TANH, SILU = 0, 1
+GELU_TANH, SILU, RELU2 = 0, 1, 2
+SINK_TENSOR, SINK_ZERO = 1, 2
 (P_EMBED, P_HEAD, P_FINAL_NORM, P_NORM, P_SHIFT, P_Q, P_K, P_HEAD_GATE, P_R1, P_R2, P_O, P_FF_GATE, P_FF_UP,
  P_FF_DOWN, P_NORM2, P_V, P_Q_NORM, P_K_NORM, P_SINK, P_VALUE_GATE, P_DKV, P_DKV_NORM, P_UK, P_UV, P_POSITIONS, P_CONV1, P_CONV2, P_Q_BIAS,
  P_K_BIAS, P_V_BIAS, P_ROUTER, P_CORRECTION, P_REC_Q, P_REC_K, P_REC_V, P_REC_GATE, P_REC_F, P_REC_F_BIAS, P_REC_LOWER, P_REC_I, P_REC_I_BIAS, P_REC_NORM,
  P_REC_O, P_REC_IN, P_REC_CONV, P_REC_CONV_BIAS, P_REC_DT_BIAS, P_REC_A_LOG, P_REC_D) = range(49)
 NORM_HEAD, NORM_PROJECTION = 1, 2
-REC_FORGET, REC_MLSTM, REC_SSD = 1, 2, 3
+REC_FORGET, REC_MLSTM, REC_SSD, REC_MINGRU = 1, 2, 3, 4
 
 
 class PlainConfig(C.Structure):
     _fields_ = [(n, C.c_int32) for n in ("n_layers", "d_model", "vocab", "max_context", "compute")] + \
                [("norm_eps", C.c_float), ("logit_cap", C.c_float), ("post_norm", C.c_int32), ("residual_scale", C.c_float),
-                ("embed_scale", C.c_float)] + [(n, C.c_int32) for n in ("output_norm", "norm_groups", "conv_taps", "positions")]
+                ("embed_scale", C.c_float)] + [(n, C.c_int32) for n in ("output_norm", "norm_groups", "conv_taps", "positions", "pre_norm")] + \
+               [("sublayer_scale", C.c_float)]
 
 
 class PlainLayer(C.Structure):
@@ -31,7 +33,8 @@ class PlainLayer(C.Structure):
                [(n, C.c_double) for n in ("rot_base", "rot_factor", "rot_original", "rot_fast", "rot_slow")] + \
                [(n, C.c_int32) for n in ("qkv_bias", "linear_bias", "chunk")] + [(n, C.c_float) for n in ("attn_scale", "rec_scale")] + \
                [(n, C.c_int32) for n in ("recurrence", "rec_heads", "rec_dim", "rec_vdim", "rec_groups", "rec_taps", "rec_norm_groups")] + \
-               [("rec_cap", C.c_float)] + [(n, C.c_int32) for n in ("experts", "expert_top", "expert_groups", "expert_keep")]
+               [("rec_cap", C.c_float)] + [(n, C.c_int32) for n in ("experts", "expert_top", "expert_groups", "expert_keep",
+                                                                        "keep_first", "pool", "value_rot", "ff_plain", "weights_of")]
 
 
 def need(d, key, where):

@@ -2,12 +2,12 @@
 import json
 import os
 
-from . import gimozen, nigenex, plain, tarivik
+from . import gimozen, nigenex, plain, ronelorn, tarivik
 from .safetensors import SafeTensors
 
 COMPUTE = {"bfloat16": plain.BF16, "float32": plain.F32}
 # config.json "architecture" -> build(ctx, config, get_tensor, max_context, compute)
-ARCHITECTURES = {m.ARCHITECTURE: m.build for m in (gimozen, nigenex, tarivik)}
+ARCHITECTURES = {m.ARCHITECTURE: m.build for m in (gimozen, nigenex, ronelorn, tarivik)}
 
 
 def read_config(folder):
