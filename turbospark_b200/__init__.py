@@ -12,4 +12,4 @@ __all__ = ["row_descs", "shaping", "Ctx", "DeviceBuffer", "TsbError", "lib", "li
 from .model import (Model, Session, ModelConfig, RunConfig, RunResult, TreeNode, run_config, config_tiny, config_8b_target,
                     config_8b_draft)
 from .plain import PlainConfig, PlainLayer, PlainModel
-from . import gimozen, nigenex, registry, tarivik
+from . import gimozen, nigenex, registry, ronelorn, tarivik

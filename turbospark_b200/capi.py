@@ -315,10 +315,11 @@ class Ctx:
                                               _vp(r1), _vp(r2), _vp(gate), C.c_int32(window), C.c_int32(max_len), _vp(scratch)))
 
     def plain_attention(self, kv, layer, q, q_stride, out, out_stride, rows_dev, group_rows, n_q_heads, scale, max_len, scratch, stream=None, cap=0.0,
-                        window=0, r1=None, r2=None, head_gate=None, sink=None, value_gate=None, value_gate_stride=0, slopes=None, chunk=0, out_scale=0.0):
+                        window=0, r1=None, r2=None, head_gate=None, sink=None, value_gate=None, value_gate_stride=0, slopes=None, chunk=0, out_scale=0.0,
+                        keep=0, blocks=False, turn=None, turn_half=0):
         gr = (C.c_int32 * len(group_rows))(*group_rows)
         x = AttentionExtras(cap, window, _vp(r1), _vp(r2), _vp(head_gate), _vp(sink), _vp(value_gate), value_gate_stride,
-                            _vp(slopes), chunk, out_scale)
+                            _vp(slopes), chunk, out_scale, keep, int(blocks), _vp(turn), turn_half)
         self.check(lib().tsb_plain_attention(self.h, stream, kv.h, C.c_int32(layer), _vp(q), C.c_int64(q_stride), _vp(out), C.c_int64(out_stride),
                                              _vp(rows_dev), gr, C.c_int32(len(group_rows)), C.c_int32(n_q_heads), C.c_float(scale), C.byref(x),
                                              C.c_int32(max_len), _vp(scratch)))
@@ -340,6 +341,32 @@ class Ctx:
     def post_norm_rows(self, type_, x, d, weight, eps, rows, out, out_stride, stream=None):
         self.check(lib().tsb_post_norm_rows(self.h, stream, C.c_int32(type_), _vp(x), C.c_int32(d), _vp(weight), C.c_float(eps), C.c_int32(rows), _vp(out),
                                             C.c_int64(out_stride)))
+
+    def pre_norm_rows(self, type_, x, d, weight, eps, rows, out, out_stride, stream=None):
+        self.check(lib().tsb_pre_norm_rows(self.h, stream, C.c_int32(type_), _vp(x), C.c_int32(d), _vp(weight), C.c_float(eps), C.c_int32(rows), _vp(out),
+                                           C.c_int64(out_stride)))
+
+    def turned_norm_rows(self, kv, layer, raw, raw_stride, n_q, n_k, width, q_weight, k_weight, eps, rows_dev, rows, q, q_stride, rot=None, rot_half=0, n_v=0, v_width=0,
+                         turn=None, turn_half=0, projection=False, stream=None):
+        n = TurnedNorms(int(projection), n_q, n_k, n_v, width, v_width, rot_half, turn_half, _vp(raw), _vp(q_weight), _vp(k_weight), _vp(rot), _vp(turn), raw_stride, q_stride,
+                        _vp(q), eps)
+        self.check(lib().tsb_turned_norm_rows(self.h, stream, kv.h, C.c_int32(layer), C.byref(n), _vp(rows_dev), C.c_int32(rows)))
+
+    def block_mean_rows(self, kv, layer, rows_dev, rows, stream=None):
+        self.check(lib().tsb_block_mean_rows(self.h, stream, kv.h, C.c_int32(layer), _vp(rows_dev), C.c_int32(rows)))
+
+    def gated_scan_rows(self, type_, gate, gate_stride, out_gate, out_gate_stride, width, state, n_streams, ring, rows_dev, rows, rows_per_seq, out, out_stride, stream=None):
+        self.check(lib().tsb_gated_scan_rows(self.h, stream, C.c_int32(type_), _vp(gate), C.c_int64(gate_stride), _vp(out_gate), C.c_int64(out_gate_stride), C.c_int32(width),
+                                             _vp(state), C.c_int32(n_streams), C.c_int32(ring), _vp(rows_dev), C.c_int32(rows), C.c_int32(rows_per_seq), _vp(out),
+                                             C.c_int64(out_stride)))
+
+    def plain_gemm_act(self, type_, w, rows, cols, x, x_rows, tokens, y, y_stride, n_valid, act, workspace, stream=None):
+        self.check(lib().tsb_plain_gemm_act(self.h, stream, C.c_int32(type_), _vp(w), C.c_int64(rows), C.c_int64(cols), _vp(x), C.c_int32(x_rows), C.c_int32(tokens), _vp(y),
+                                            C.c_int64(y_stride), C.c_int32(n_valid), C.c_int32(act), _vp(workspace)))
+
+    def plain_gemm_add(self, type_, w, rows, cols, x, x_rows, tokens, y, y_stride, n_valid, alpha, beta, workspace, stream=None):
+        self.check(lib().tsb_plain_gemm_add(self.h, stream, C.c_int32(type_), _vp(w), C.c_int64(rows), C.c_int64(cols), _vp(x), C.c_int32(x_rows), C.c_int32(tokens), _vp(y),
+                                            C.c_int64(y_stride), C.c_int32(n_valid), C.c_float(alpha), C.c_float(beta), _vp(workspace)))
 
     def head_norm_rows(self, kv, layer, raw, raw_stride, n_q, n_k, width, q_weight, k_weight, eps, rows_dev, rows, q, q_stride, temp_coef=0.0, temp_every=0,
                        stream=None):
