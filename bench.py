@@ -363,8 +363,8 @@ def run_ours(args, rank, world, local_rank):
 
 
 def run_design(args):
-    from turbospark_b200 import latentbench, plainbench, tarivikbench
-    bench = {"gimozen": latentbench, "nigenex": plainbench, "tarivik": tarivikbench}[args.design]
+    from turbospark_b200 import latentbench, plainbench, ronelornbench, tarivikbench
+    bench = {"gimozen": latentbench, "nigenex": plainbench, "ronelorn": ronelornbench, "tarivik": tarivikbench}[args.design]
     hbm, src = peaks()
     p = os.path.join(ROOT, "MEASURED_PEAKS.json")
     tf = float(json.load(open(p))["bf16_tflops"]) if os.path.exists(p) else 1590.0
@@ -387,9 +387,9 @@ def main():
     ap.add_argument("--streams", type=int, default=1, help="independent request streams per GPU")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--no-streams64", action="store_true", help="skip the 64-streams-in-total leg")
-    ap.add_argument("--design", default="", choices=["", "gimozen", "nigenex", "tarivik"],
+    ap.add_argument("--design", default="", choices=["", "gimozen", "nigenex", "ronelorn", "tarivik"],
                     help="instead of the default workload: prefill, decode and kernel times of this design beside a model of equal size - Nigenex beside "
-                         "the block-quantised dense model, Gimozen beside Nigenex, Tarivik beside Gimozen (one GPU)")
+                         "the block-quantised dense model, Gimozen beside Nigenex, Tarivik and Ronelorn beside Gimozen (one GPU)")
     ap.add_argument("--shapes", default="8b,2b", help="layer shapes of --design, with commas between them")
     ap.add_argument("--parts", default="kernels,models", help="what --design measures")
     args = ap.parse_args()

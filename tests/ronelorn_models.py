@@ -51,7 +51,7 @@ CONFIGS = {
     # windows and kept tokens that no prompt of the tests leaves; many heads per key head
     "near": config(128, 75, [pooled(12, 1, 20, 28, 1000, 3, 40, rot=4, cap=3.0), kept(16, 2, 32, 32, 600, 800, 24, rot=2), kept(5, 5, 48, 16, 33, 0, None, rot=16)], embed=1.0),
     # constants and sizes that are one
-    "ones": config(64, 40, [pooled(1, 1, 8, 2, 1, 1, 8, rot=2, factor=1.0, cap=1.0), kept(1, 1, 2, 1, 1, 1, 1, rot=2), mingru(1, mlp=3), mingru(8)], mult=1.0),
+    "ones": config(64, 40, [pooled(1, 1, 8, 2, 1, 1, 8, rot=2, factor=1.0, cap=1.0), kept(1, 1, 8, 1, 1, 1, 1, rot=2), mingru(1, mlp=3), mingru(8)], mult=1.0, embed=4.0),
 }
 
 

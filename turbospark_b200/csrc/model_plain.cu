@@ -206,12 +206,15 @@ int32_t plain_share(tsb_model* dt, int32_t dst_layer, const tsb_model* st, int32
     }
     TSB_REQUIRE(ctx, dst_layer < d->cfg.n_layers && src_layer >= 0 && src_layer < s->cfg.n_layers, "layer out of range");
     PlainLayer& l = d->layers[dst_layer];
-    TSB_REQUIRE(ctx, memcmp(&l.cfg, &s->layers[src_layer].cfg, sizeof l.cfg) == 0, "layer shapes differ");
     TSB_REQUIRE(ctx, l.tied < 0, "layer %d uses the tensors of layer %d", dst_layer, l.tied);
+    const tsb_plain_layer own = l.cfg;
+    tsb_plain_layer theirs = s->layers[src_layer].cfg;
+    theirs.weights_of = 0;
+    TSB_REQUIRE(ctx, memcmp(&own, &theirs, sizeof own) == 0, "layer shapes differ");
     free_layer(ctx, l);
     const int rotation = l.rotation, value_rotation = l.value_rotation, source = l.source;
     l = s->layers[src_layer];
-    l.rotation = rotation, l.value_rotation = value_rotation, l.source = source;
+    l.cfg = own, l.rotation = rotation, l.value_rotation = value_rotation, l.source = source;
     l.tied = -1, l.owned = false;
     mirror_layer(d, dst_layer);
     return TSB_OK;
