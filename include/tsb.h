@@ -603,10 +603,11 @@ typedef struct tsb_turned_norms {
 } tsb_turned_norms;
 TSB_API int32_t tsb_turned_norm_rows(tsb_ctx* ctx, tsb_stream s, tsb_kv* cache, int32_t layer, const tsb_turned_norms* n, const tsb_row_desc* rows_dev, int32_t rows);
 /* minGRU (see TSB_REC_MINGRU): gate [rows, z pre-activations | u], out = S silu(out_gate), both in `type`; state [n_streams][ring][width rounded up to 4], position p in slot
- * p & (ring - 1), ring a power of two above one.  Portions of rows_per_seq rows each; the states after a portion's last `ring` rows are kept. */
+ * p & (ring - 1), ring a power of two above one.  Portions of rows_per_seq rows each; the states after a portion's last `ring` rows are kept.
+ * chunked = 1: 128 rows of a portion side by side, for long ones; sums: room for two f32 per channel and chunk where portions have several. */
 TSB_API int32_t tsb_gated_scan_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, const float* gate, int64_t gate_stride, const void* out_gate, int64_t out_gate_stride,
                                     int32_t width, float* state, int32_t n_streams, int32_t ring, const tsb_row_desc* rows_dev, int32_t rows, int32_t rows_per_seq,
-                                    void* out, int64_t out_stride);
+                                    int32_t chunked, void* sums, void* out, int64_t out_stride);
 /* y[t, n] = act(sum_k W[n, k] x[t, k]) in `type`; and y[t, n] = alpha * y[t, n] + beta * sum in f32. */
 TSB_API int32_t tsb_plain_gemm_act(tsb_ctx* ctx, tsb_stream s, int32_t type, const void* w, int64_t rows, int64_t cols, const void* x, int32_t x_rows, int32_t tokens,
                                    void* y, int64_t y_stride, int32_t n_valid, int32_t act, void* workspace);

@@ -238,8 +238,9 @@ def test_products_with_an_activation_and_scaled_sums(rig, type_, tokens, cols):
 
 # ------------------------------------------------------------------ element-wise recurrence
 @pytest.mark.parametrize("type_", [F32, BF16])
-@pytest.mark.parametrize("width,sizes", [(136, [1] * 9 + [2, 7, 40, 31, 33]), (57, [500]), (2048, [128, 1, 129, 31]), (5000, [64, 3]), (8, [300, 200, 1, 1]), (4100, [1, 32])])
-def test_gated_scan(rig, type_, width, sizes):
+@pytest.mark.parametrize("chunked", [False, True])
+@pytest.mark.parametrize("width,sizes", [(136, [1] * 9 + [2, 7, 40, 31, 33]), (57, [500]), (2048, [128, 1, 129, 31]), (5000, [64, 3]), (8, [300, 5000, 1, 1]), (4100, [1, 32])])
+def test_gated_scan(rig, type_, chunked, width, sizes):
     """Three streams in the portions given, the state carried over in a ring that wraps; channels that keep next to everything and channels that keep nothing."""
     ctx, rng, n, streams = rig["ctx"], np.random.default_rng(width), sum(sizes), 3
     z = (rng.standard_normal((streams, n, width)) * 2 + np.linspace(-9, 6, width)).astype(np.float32)
@@ -256,7 +257,7 @@ def test_gated_scan(rig, type_, width, sizes):
         gp[:, :width] = gu[order, at:at + m].reshape(-1, width)
         out = ctx.zeroed(streams * m * stride * 4)
         ctx.gated_scan_rows(type_, f32(ctx, gate), 2 * width, ctx.to_device(gp), stride, width, state, streams, ring, ctx.to_device(descs(rig["tsb"], [(i, at, m) for i in order])),
-                            streams * m, m, out, stride)
+                            streams * m, m, out, stride, chunked=chunked, sums=ctx.zeroed(streams * (m // 128 + 1) * width * 8))
         got, w = fetch(out, type_, (streams * m, stride))[:, :width], want[order, at:at + m].reshape(-1, width)
         assert (np.abs(got - w) <= (3e-5 if type_ == F32 else 5e-3) * np.abs(w) + 3e-5).all()
         kept = fetch(state, F32, (streams, ring, pitch))

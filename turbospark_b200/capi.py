@@ -355,10 +355,11 @@ class Ctx:
     def block_mean_rows(self, kv, layer, rows_dev, rows, stream=None):
         self.check(lib().tsb_block_mean_rows(self.h, stream, kv.h, C.c_int32(layer), _vp(rows_dev), C.c_int32(rows)))
 
-    def gated_scan_rows(self, type_, gate, gate_stride, out_gate, out_gate_stride, width, state, n_streams, ring, rows_dev, rows, rows_per_seq, out, out_stride, stream=None):
+    def gated_scan_rows(self, type_, gate, gate_stride, out_gate, out_gate_stride, width, state, n_streams, ring, rows_dev, rows, rows_per_seq, out, out_stride, chunked=False, sums=None,
+                        stream=None):
         self.check(lib().tsb_gated_scan_rows(self.h, stream, C.c_int32(type_), _vp(gate), C.c_int64(gate_stride), _vp(out_gate), C.c_int64(out_gate_stride), C.c_int32(width),
-                                             _vp(state), C.c_int32(n_streams), C.c_int32(ring), _vp(rows_dev), C.c_int32(rows), C.c_int32(rows_per_seq), _vp(out),
-                                             C.c_int64(out_stride)))
+                                             _vp(state), C.c_int32(n_streams), C.c_int32(ring), _vp(rows_dev), C.c_int32(rows), C.c_int32(rows_per_seq), C.c_int32(int(chunked)),
+                                             _vp(sums), _vp(out), C.c_int64(out_stride)))
 
     def plain_gemm_act(self, type_, w, rows, cols, x, x_rows, tokens, y, y_stride, n_valid, act, workspace, stream=None):
         self.check(lib().tsb_plain_gemm_act(self.h, stream, C.c_int32(type_), _vp(w), C.c_int64(rows), C.c_int64(cols), _vp(x), C.c_int32(x_rows), C.c_int32(tokens), _vp(y),

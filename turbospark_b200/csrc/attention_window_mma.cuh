@@ -47,8 +47,7 @@ __device__ __forceinline__ void base2_logits(float (&s)[N][4], const WindowAttn&
             for (int n = 0; n < N; n++)
 #pragma unroll
                 for (int i = 0; i < 4; i += 2) {
-                    const float2 x = make_float2(s[n][i], s[n][i + 1]), z = mul2(x, x);
-                    const float2 v = mul2(x, fma2(z, fma2(z, fma2(z, fma2(z, both(sc.k4), both(sc.k3)), both(sc.k2)), both(sc.k1)), both(sc.k0)));
+                    const float2 x = make_float2(s[n][i], s[n][i + 1]), v = mul2(x, sc.factor(x));
                     s[n][i] = v.x, s[n][i + 1] = v.y;
                 }
         }

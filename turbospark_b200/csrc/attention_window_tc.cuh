@@ -293,9 +293,7 @@ __global__ void __launch_bounds__(WT_THREADS, 1)
                 if (capped && series) {
 #pragma unroll
                     for (int j = 0; j < WT_TN; j += 2) {
-                        const float2 x = make_float2(s[j], s[j + 1]), z = mul2(x, x);
-                        const float2 w = fma2(z, fma2(z, fma2(z, fma2(z, both(sc.k4), both(sc.k3)), both(sc.k2)), both(sc.k1)), both(sc.k0));
-                        const float2 v = fma2(x, w, biased ? make_float2(bias[j], bias[j + 1]) : both(0.f));
+                        const float2 x = make_float2(s[j], s[j + 1]), v = fma2(x, sc.factor(x), biased ? make_float2(bias[j], bias[j + 1]) : both(0.f));
                         s[j] = v.x, s[j + 1] = v.y;
                     }
                 } else {
@@ -324,9 +322,9 @@ __global__ void __launch_bounds__(WT_THREADS, 1)
                 }
                 float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
-                for (int j = 0; j < WT_TN; j += 4) {
-                    mx4[0] = fmaxf(mx4[0], s[j]), mx4[1] = fmaxf(mx4[1], s[j + 1]);
-                    mx4[2] = fmaxf(mx4[2], s[j + 2]), mx4[3] = fmaxf(mx4[3], s[j + 3]);
+                for (int j = 0; j < WT_TN; j += 8) {
+                    mx4[0] = max3(mx4[0], s[j], s[j + 1]), mx4[1] = max3(mx4[1], s[j + 2], s[j + 3]);
+                    mx4[2] = max3(mx4[2], s[j + 4], s[j + 5]), mx4[3] = max3(mx4[3], s[j + 6], s[j + 7]);
                 }
                 const float mx = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3]));
                 const bool grow = mx > m_ref + 8.f;

@@ -244,7 +244,7 @@ int32_t states_init(tsb_session* s, const PlainModel* m, const SessionShape& sha
     for (st.ring = 2; st.ring < shape.max_rows + 1;) st.ring *= 2;
     for (st.row_ring = 2; st.row_ring < st.ring + st.keep;) st.row_ring *= 2;
     std::vector<RowRing> rings;
-    size_t scratch = 0;
+    size_t scratch = 0, sums = 0;
     int32_t rc = TSB_OK;
     auto ring = [&](std::vector<RowRing>& list, int64_t width, int taps) {
         RowRing r;
@@ -269,11 +269,13 @@ int32_t states_init(tsb_session* s, const PlainModel* m, const SessionShape& sha
         const size_t copies = heads * recurrence_copies(c.rec_vdim);
         if (c.recurrence == TSB_REC_MLSTM && rc == TSB_OK) rc = zero(copies * c.rec_dim * 4, (void**)&r.norm);
         if (c.recurrence == TSB_REC_MLSTM && rc == TSB_OK) rc = zero(copies * 8, (void**)&r.top);
-        if (c.recurrence && c.recurrence != TSB_REC_MINGRU && !m->f32)
+        if (c.recurrence == TSB_REC_MINGRU) sums = std::max(sums, (size_t)(shape.pass_rows / SCAN_CHUNK + shape.n_streams) * c.rec_vdim * sizeof(float2));
+        else if (c.recurrence && !m->f32)
             scratch = std::max(scratch, recurrence_scratch_bytes(c.recurrence, c.rec_heads, c.rec_dim, c.rec_vdim, shape.pass_rows / REC_CHUNK + shape.n_streams));
         st.states.push_back(r);
     }
     if (rc == TSB_OK && shape.pass_rows >= CHUNK_MIN_ROWS) rc = zero(scratch, &st.chunk_scratch);
+    if (rc == TSB_OK && shape.pass_rows > SCAN_CHUNK) rc = zero(sums, (void**)&st.scan_sums);
     if (rc) return rc;
     st.n_rings = (int)rings.size();
     if (st.n_rings == 0) return TSB_OK;
@@ -448,7 +450,8 @@ struct PassPlan {
     int expanded_pages = 0, expanded_len = 0, short_first = 0, short_rows = 0;
     // output-norm form and recurrences: runs of rows for the row operators; portions whose recurrences go row by row, and chunk by chunk where there is a kernel
     RowTiles runs, by_row, portions;  // portions: all of them
-    RowTiles by_scan;                 // those that are not in by_row
+    RowTiles scan_chunks;             // those that are not in by_row, in chunks for element-wise recurrences
+    bool several_chunks = false;      // of one portion
     RecurrenceChunks by_chunk;
     bool use_before = false;
 
@@ -473,7 +476,7 @@ int32_t plan_states(tsb_session* s, const PlainModel* m, const ModelRt& rt, cons
         plan.by_row = plan.portions = RowTiles::uniform(p.rows, p.rows_per_seq, p.rows_per_seq);
         return TSB_OK;
     }
-    std::vector<AttnTile> runs, by_row, by_scan, portions, chunks;
+    std::vector<AttnTile> runs, by_row, scan_chunks, portions, chunks;
     std::vector<ChunkPortion> by_chunk;
     for (int i = 0; i < p.n_groups; i++) {
         const RowGroup& g = p.groups[i];
@@ -484,7 +487,8 @@ int32_t plan_states(tsb_session* s, const PlainModel* m, const ModelRt& rt, cons
             by_row.push_back({g.first_row, g.n_rows});
             continue;
         }
-        by_scan.push_back({g.first_row, g.n_rows});
+        for (int r = 0; r < g.n_rows; r += SCAN_CHUNK) scan_chunks.push_back({g.first_row + r, std::min(SCAN_CHUNK, g.n_rows - r)});
+        plan.several_chunks |= g.n_rows > SCAN_CHUNK;
         by_chunk.push_back({g.first_row, g.n_rows, (int)chunks.size()});
         for (int r = 0; r < g.n_rows; r += REC_CHUNK) chunks.push_back({g.first_row + r, std::min(REC_CHUNK, g.n_rows - r)});
         rt.kv->state_lo[g.seq] = g.base + g.n_rows - 1;  // the states in between are not kept
@@ -503,7 +507,7 @@ int32_t plan_states(tsb_session* s, const PlainModel* m, const ModelRt& rt, cons
     int32_t rc = stage(runs, plan.runs);
     if (rc == TSB_OK) rc = stage(by_row, plan.by_row);
     if (rc == TSB_OK) rc = stage(portions, plan.portions);
-    if (rc == TSB_OK) rc = stage(by_scan, plan.by_scan);
+    if (rc == TSB_OK) rc = stage(scan_chunks, plan.scan_chunks);
     if (rc == TSB_OK) rc = stage(chunks, plan.by_chunk.chunks);
     if (rc || by_chunk.empty()) return rc;
     const int32_t* dev = nullptr;
@@ -657,6 +661,7 @@ struct Forward {
             h.temp_coef = c.q_temp_coef, h.temp_every = c.q_temp_every;
             h.q = b->q, h.q_stride = b->q_stride, h.q_step = h.q_width = l.head_pad;
             if (l.rotation >= 0) h.rot = b->rotary[l.rotation], h.rot_half = c.rot_dim / 2;
+            if (c.pool > 0) h.pool = c.pool, h.pooled = rt.kv->pooled_layers[L];
             if (c.value_rot) h.n_v = c.n_kv_heads, h.v_width = c.value_dim, h.turn = b->rotary[l.value_rotation], h.turn_half = c.value_dim / 2;
         }
         return launch_head_norms(ctx, st, m->f32, h, p.rows);
@@ -769,8 +774,9 @@ struct Forward {
         GatedScan g;
         g.gate = b->raw + b->raw_rec, g.gate_stride = b->raw_stride, g.out_gate = b->rec, g.out_gate_stride = b->rec_stride;
         g.out = at(b->cat, l.o_cols), g.out_stride = l.out.cols, g.width = l.cfg.rec_vdim, g.state = b->states.states[L], g.rows = p.rows_dev;
-        if (cudaError_t e = launch_gated_scan(ctx, st, m->f32, g, plan.by_row); e != cudaSuccess) return e;
-        return launch_gated_scan(ctx, st, m->f32, g, plan.by_scan);
+        g.n_rows = p.rows;
+        if (cudaError_t e = launch_gated_scan_rows(ctx, st, m->f32, g, plan.by_row); e != cudaSuccess) return e;
+        return launch_gated_scan_chunks(ctx, st, m->f32, g, plan.scan_chunks, plan.several_chunks, b->states.scan_sums);
     }
 
     cudaError_t block_means(int L) const {
@@ -909,7 +915,8 @@ struct Forward {
         }
         if (l.cfg.qk_norm == TSB_NORM_PROJECTION) e = projection_norms(L);
         else if (l.cfg.qk_norm || (l.mixer == MIX_LATENT && l.source == L)) e = head_norms(L);
-        if (e == cudaSuccess && l.cfg.pool > 0) e = block_means(L);
+        // (norms per head see to the blocks before their portions: enough where those are single rows)
+        if (e == cudaSuccess && l.cfg.pool > 0 && (plan.longest > 1 || l.cfg.qk_norm != TSB_NORM_HEAD)) e = block_means(L);
         if (e != cudaSuccess) return e;
         if (l.mixer != MIX_LATENT) return attend(L);
         const bool expand = l.expands && !plan.expanded.empty();

@@ -83,6 +83,7 @@ struct StreamStates {
     std::vector<RowRing> conv1, conv2, rec; // per layer: inputs of the two sublayers' convolutions and of the recurrence's
     std::vector<RecurrentState> states;     // per layer
     void* chunk_scratch = nullptr;          // of the chunked recurrences
+    float2* scan_sums = nullptr;            // of the element-wise ones
     RowRing* rings_dev = nullptr;           // all rings that look back
     int n_rings = 0;
 };

@@ -215,17 +215,21 @@ int32_t tsb_block_mean_rows(tsb_ctx* ctx, tsb_stream s, tsb_kv* cache, int32_t l
 }
 
 int32_t tsb_gated_scan_rows(tsb_ctx* ctx, tsb_stream s, int32_t type, const float* gate, int64_t gate_stride, const void* out_gate, int64_t out_gate_stride, int32_t width,
-                            float* state, int32_t n_streams, int32_t ring, const tsb_row_desc* rows_dev, int32_t rows, int32_t rows_per_seq, void* out, int64_t out_stride) {
+                            float* state, int32_t n_streams, int32_t ring, const tsb_row_desc* rows_dev, int32_t rows, int32_t rows_per_seq, int32_t chunked, void* sums, void* out, int64_t out_stride) {
     if (!ctx) return TSB_ERR_INVALID;
     int32_t rc = check_portions(ctx, rows_dev, rows, rows_per_seq);
     if (rc) return rc;
+    TSB_REQUIRE(ctx, !chunked || rows_per_seq <= SCAN_CHUNK || (sums && (uintptr_t)sums % 8 == 0), "portions of several chunks need room for their sums");
     TSB_REQUIRE(ctx, known(type) && gate && out_gate && state && out && width > 0 && gate_stride >= 2 * (int64_t)width && out_gate_stride >= width && out_stride >= width, "bad arguments");
     TSB_REQUIRE(ctx, power_of_two(ring) && ring > 1 && n_streams > 0, "ring is a power of two above one");
     DeviceGuard g(ctx);
     GatedScan x;
     x.gate = gate, x.gate_stride = gate_stride, x.out_gate = out_gate, x.out_gate_stride = out_gate_stride, x.out = out, x.out_stride = out_stride, x.width = width;
     x.state.s = state, x.state.ring = ring, x.state.n_streams = n_streams, x.rows = rows_dev;
-    TSB_CUDA(ctx, launch_gated_scan(ctx, (cudaStream_t)s, type == TSB_F32, x, RowTiles::uniform(rows, rows_per_seq, rows_per_seq)));
+    x.n_rows = rows;
+    const bool f32 = type == TSB_F32;
+    TSB_CUDA(ctx, chunked ? launch_gated_scan_chunks(ctx, (cudaStream_t)s, f32, x, RowTiles::uniform(rows, rows_per_seq, SCAN_CHUNK), rows_per_seq > SCAN_CHUNK, static_cast<float2*>(sums))
+                          : launch_gated_scan_rows(ctx, (cudaStream_t)s, f32, x, RowTiles::uniform(rows, rows_per_seq, rows_per_seq)));
     return TSB_OK;
 }
 

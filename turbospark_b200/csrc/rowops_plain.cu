@@ -2,6 +2,7 @@
 #include <cuda_bf16.h>
 
 #include <algorithm>
+#include <type_traits>
 
 #include "rowops_plain.cuh"
 
@@ -221,6 +222,31 @@ __global__ void __launch_bounds__(ROW_THREADS)
     }
 }
 
+// Columns c .. of a block's mean: the cache's rows at its positions, summed in their order, eight loads in flight.
+template <typename T>
+__device__ __forceinline__ void block_mean(const KeyView& keys, int pool, int seq, int block, int c, T* dst) {
+    constexpr int N = 16 / sizeof(T), AHEAD = 8;
+    float sum[N];
+#pragma unroll
+    for (int i = 0; i < N; i++) sum[i] = 0.f;
+    for (int j0 = 0; j0 < pool; j0 += AHEAD) {
+        const T* src[AHEAD];
+        uint4 v[AHEAD];
+#pragma unroll
+        for (int j = 0; j < AHEAD; j++) src[j] = j0 + j < pool ? key_row<T>(keys, seq, block * pool + j0 + j) : nullptr;  // reserved, as later ones are
+#pragma unroll
+        for (int j = 0; j < AHEAD; j++) v[j] = src[j] ? *reinterpret_cast<const uint4*>(src[j] + c) : make_uint4(0, 0, 0, 0);
+#pragma unroll
+        for (int j = 0; j < AHEAD; j++) {
+            const T* e = reinterpret_cast<const T*>(&v[j]);
+#pragma unroll
+            for (int i = 0; i < N; i++) sum[i] += get(e + i);
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < N; i++) put(dst + c + i, sum[i] / (float)pool);
+}
+
 // the pair of columns i and i + 1 (i even), turned; columns behind the turned ones pass
 __device__ __forceinline__ void turn_pair(const float2* table, int half, int r, int i, float& u, float& v) {
     if (i >= 2 * half) return;
@@ -231,18 +257,26 @@ __device__ __forceinline__ void turn_pair(const float2* table, int half, int r, 
 
 // LANES lanes per (row, head).  VEC > 0: the width is a multiple of four and at most 4 LANES VEC, and a lane holds its columns in
 // registers.
-template <typename T, int LANES, int VEC>
+template <typename T, int LANES, int VEC, bool MORE>
 __global__ void __launch_bounds__(ROW_THREADS) head_norms_kernel(const __grid_constant__ HeadNorms h, int rows, uint32_t* __restrict__ err) {
     const int lane = threadIdx.x & (LANES - 1);
     const int64_t item = (int64_t)blockIdx.x * (ROW_THREADS / LANES) + threadIdx.x / LANES;
-    const int per = h.n_q + h.n_k + h.n_v;
+    const int per = h.n_q + h.n_k + (MORE ? h.n_v + (h.pool > 0 ? h.keys.kv_heads : 0) : 0);
     const bool in = item < (int64_t)rows * per;
     const int r = in ? (int)(item / per) : 0, head = in ? (int)(item % per) : 0;
     const tsb_row_desc rd = h.rows[r];
     pdl_wait();
     pdl_launch_dependents();
     if (!in) return;
-    const bool query = head < h.n_q, value = head >= h.n_q + h.n_k;
+    const bool query = head < h.n_q, value = MORE && head >= h.n_q + h.n_k;
+    if (MORE && head >= h.n_q + h.n_k + h.n_v) {
+        const int pos = rd.base + rd.slot, block = pos / h.pool - 1, at = (head - h.n_q - h.n_k - h.n_v) * h.keys.head_step;
+        if (rd.slot != 0 || block < 0 || (block + 1) * h.pool != pos) return;
+        T* dst = key_row<T>(h.pooled, rd.seq, block);
+        if (!dst && lane == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+        for (int c = lane * (16 / (int)sizeof(T)); dst && c < h.keys.head_step; c += LANES * (16 / (int)sizeof(T))) block_mean<T>(h.keys, h.pool, rd.seq, block, at + c, dst);
+        return;
+    }
     const float* src = h.raw + (int64_t)r * h.raw_stride + (int64_t)head * h.width;
     if (value) {
         src += (int64_t)(head - h.n_q - h.n_k) * (h.v_width - h.width);
@@ -311,7 +345,7 @@ __global__ void __launch_bounds__(ROW_THREADS) head_norms_kernel(const __grid_co
             const int i = (k * LANES + lane) * 4;
             if (i >= h.width) break;
             float4 o = make_float4(v[k].x * s * g[k].x, v[k].y * s * g[k].y, v[k].z * s * g[k].z, v[k].w * s * g[k].w);
-            if (h.rot) turn_pair(h.rot, h.rot_half, r, i, o.x, o.y), turn_pair(h.rot, h.rot_half, r, i + 2, o.z, o.w);
+            if (MORE && h.rot) turn_pair(h.rot, h.rot_half, r, i, o.x, o.y), turn_pair(h.rot, h.rot_half, r, i + 2, o.z, o.w);
             put4(dst + i, o);
         }
         for (int i = h.width + lane; i < width; i += LANES) put(dst + i, 0.f);
@@ -319,7 +353,7 @@ __global__ void __launch_bounds__(ROW_THREADS) head_norms_kernel(const __grid_co
     }
     for (int i = 2 * lane; i < width; i += 2 * LANES) {
         float u = i < h.width ? src[i] * s * w[i] : 0.f, v = i + 1 < h.width ? src[i + 1] * s * w[i + 1] : 0.f;
-        if (h.rot) turn_pair(h.rot, h.rot_half, r, i, u, v);
+        if (MORE && h.rot) turn_pair(h.rot, h.rot_half, r, i, u, v);
         put(dst + i, u);
         if (i + 1 < width) put(dst + i + 1, v);
     }
@@ -354,22 +388,7 @@ __global__ void __launch_bounds__(ROW_THREADS) block_means_kernel(const __grid_c
         if (threadIdx.x == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
         return;
     }
-    for (int c = threadIdx.x * N; c < b.keys.row; c += ROW_THREADS * N) {
-        float sum[N];
-#pragma unroll
-        for (int i = 0; i < N; i++) sum[i] = 0.f;
-#pragma unroll 8
-        for (int j = 0; j < b.pool; j++) {
-            const T* src = key_row<T>(b.keys, rd.seq, block * b.pool + j);
-            if (!src) continue;  // positions before a reserved one are reserved
-            const uint4 v = *reinterpret_cast<const uint4*>(src + c);
-            const T* e = reinterpret_cast<const T*>(&v);
-#pragma unroll
-            for (int i = 0; i < N; i++) sum[i] += get(e + i);
-        }
-#pragma unroll
-        for (int i = 0; i < N; i++) put(dst + c + i, sum[i] / (float)b.pool);
-    }
+    for (int c = threadIdx.x * N; c < b.keys.row; c += ROW_THREADS * N) block_mean<T>(b.keys, b.pool, rd.seq, block, c, dst);
 }
 
 // a CTA per position and stream
@@ -460,19 +479,22 @@ cudaError_t launch_pre_norm(tsb_ctx* ctx, cudaStream_t st, bool f32, const float
 cudaError_t launch_head_norms(tsb_ctx* ctx, cudaStream_t st, bool f32, const HeadNorms& h, int rows) {
     auto run = [&](auto kernel, int lanes) {
         const int per_cta = ROW_THREADS / lanes;
-        const dim3 grid((unsigned)(((int64_t)rows * (h.n_q + h.n_k + h.n_v) + per_cta - 1) / per_cta));
+        const dim3 grid((unsigned)(((int64_t)rows * (h.n_q + h.n_k + h.n_v + (h.pool > 0 ? h.keys.kv_heads : 0)) + per_cta - 1) / per_cta));
         return tsb_launch(ctx, kernel, grid, dim3(ROW_THREADS), 0, st, true, h, rows, ctx->dev_error);
     };
     const int wide = h.n_v > 0 ? std::max(h.width, h.v_width) : h.width;
     const bool vec = h.width % 4 == 0 && (h.n_v == 0 || h.v_width % 4 == 0) && wide <= 512 && h.raw_stride % 4 == 0 && (uintptr_t)h.raw % 16 == 0 && h.q_step % 4 == 0 && h.q_stride % 4 == 0;
-    if (f32) {
-        if (vec && wide <= 64) return run(head_norms_kernel<float, 8, 2>, 8);
-        if (vec && wide <= 128) return run(head_norms_kernel<float, 16, 2>, 16);
-        return vec ? run(head_norms_kernel<float, 32, 4>, 32) : run(head_norms_kernel<float, 32, 0>, 32);
-    }
-    if (vec && wide <= 64) return run(head_norms_kernel<__nv_bfloat16, 8, 2>, 8);
-    if (vec && wide <= 128) return run(head_norms_kernel<__nv_bfloat16, 16, 2>, 16);
-    return vec ? run(head_norms_kernel<__nv_bfloat16, 32, 4>, 32) : run(head_norms_kernel<__nv_bfloat16, 32, 0>, 32);
+    // MORE: rotations, values, blocks
+    const bool more = h.rot || h.n_v > 0 || h.pool > 0;
+    auto pick = [&](auto type, auto with) {
+        using T = decltype(type);
+        constexpr bool MORE = decltype(with)::value;
+        if (vec && wide <= 64) return run(head_norms_kernel<T, 8, 2, MORE>, 8);
+        if (vec && wide <= 128) return run(head_norms_kernel<T, 16, 2, MORE>, 16);
+        return vec ? run(head_norms_kernel<T, 32, 4, MORE>, 32) : run(head_norms_kernel<T, 32, 0, MORE>, 32);
+    };
+    if (f32) return more ? pick(0.f, std::true_type{}) : pick(0.f, std::false_type{});
+    return more ? pick(__nv_bfloat16{}, std::true_type{}) : pick(__nv_bfloat16{}, std::false_type{});
 }
 
 cudaError_t launch_block_means(tsb_ctx* ctx, cudaStream_t st, bool f32, const BlockMeans& b, int rows) {

@@ -39,7 +39,7 @@ cudaError_t launch_pre_norm(tsb_ctx* ctx, cudaStream_t st, bool f32, const float
 // at position p (temp_every 0: not) and stored to q at (head * q_step) with zeros up to q_width; keys go to the token's cache row
 // at (head * keys.head_step).  n_q = 0, n_k = 1 is the norm of a latent.  With `rot`, columns 2 i and 2 i + 1 of a normed head are turned by
 // (cos, sin) of [rows, rot_half].  n_v heads of v_width numbers behind the keys are values: not normed, turned by `turn`, stored keys.value_off
-// elements into the cache's heads.
+// elements into the cache's heads.  pool > 0: the block that ends right before a portion gets its mean (see BlockMeans; its rows are all of earlier passes).
 struct HeadNorms {
     const float* raw = nullptr;
     int64_t raw_stride = 0;
@@ -53,7 +53,8 @@ struct HeadNorms {
     int q_step = 0, q_width = 0;
     const float2 *rot = nullptr, *turn = nullptr;
     int rot_half = 0, turn_half = 0, n_v = 0, v_width = 0;
-    KeyView keys{};
+    KeyView keys{}, pooled{};
+    int pool = 0;
     const tsb_row_desc* rows = nullptr;
 };
 cudaError_t launch_head_norms(tsb_ctx* ctx, cudaStream_t st, bool f32, const HeadNorms& h, int rows);

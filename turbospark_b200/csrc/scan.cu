@@ -1,11 +1,11 @@
 // Gated recurrences element by element (scan.cuh).
 //
-//   scan_rows_kernel  short portions: a thread per channel walks the portion's rows, eight of them in flight.
-//   scan_kernel       long portions: a CTA owns CH channels of a portion and goes through it in batches of 32 runs of RUN rows.  A thread composes
-//                     its run's rows into one step S -> A S + B; the 32 steps of a channel meet in shared memory, where a warp per channel scans
-//                     them; then every thread walks its run from the state before it.  Gates are read once and stay in registers.
-// f32 throughout.  1 - z is sigmoid(-x), not a difference, and a step is S + z (c - S): close to zero or one the rounding of z would
-// otherwise add up over a long memory.
+//   row by row   short portions: a thread per channel walks the portion's rows, eight of them in flight.
+//   by chunks    long portions: a CTA owns CH channels of a chunk, 32 runs of a few rows.  A thread composes its run's rows into one step S -> A S + B; the
+//                32 steps of a channel meet in shared memory, where a warp per channel scans them; then every thread walks its run from the state
+//                before it.  Chunks with others behind them leave their step as a whole in a first launch, the second scans the steps before its own.
+// f32 throughout.  A step is S + z (c - S), and a product of factors 1 - z is A - z A: where z is next to nothing the rounding of 1 - z would add up over a
+// long memory.
 #include <algorithm>
 
 #include "recurrence_dev.cuh"
@@ -14,11 +14,20 @@
 namespace {
 
 constexpr int ROWS_THREADS = 128, AHEAD = 8;
-constexpr int RUNS = 32;  // of a batch: the lanes of the warp that scans a channel
+constexpr int RUNS = 32;  // of a chunk: the lanes of the warp that scans a channel
 
 __device__ __forceinline__ void scan_put(float* p, float v) { *p = v; }
 __device__ __forceinline__ void scan_put(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
-__device__ __forceinline__ float candidate(float u) { return u >= 0.f ? u + 0.5f : rec_sigmoid(u); }
+// 1 / (1 + e^-x): with bfloat16 outputs by the fast exponential and division (relative error a few 2^-22), in the f32 mode by the library's.
+template <typename T>
+__device__ __forceinline__ float sigmoid_of(float x) {
+    return sizeof(T) == 4 ? rec_sigmoid(x) : __fdividef(1.f, 1.f + __expf(-x));
+}
+template <typename T>
+__device__ __forceinline__ float candidate(float u) {
+    const float low = sigmoid_of<T>(fminf(u, 0.f));
+    return u >= 0.f ? u + 0.5f : low;
+}
 
 __device__ __forceinline__ float* state_at(const GatedScan& g, int seq, int pos) {
     return g.state.s + ((int64_t)seq * g.state.ring + (pos & (g.state.ring - 1))) * recurrence_v_pitch(g.width);
@@ -49,92 +58,146 @@ __global__ void __launch_bounds__(ROWS_THREADS) scan_rows_kernel(const __grid_co
         for (int i = 0; i < AHEAD; i++) {
             const int t = t0 + i;
             if (t >= p.n_rows) break;
-            s = fmaf(rec_sigmoid(x[i]), candidate(u[i]) - s, s);
-            scan_put(static_cast<T*>(g.out) + (int64_t)(p.row_first + t) * g.out_stride + c, s * rec_silu(o[i]));
+            s = fmaf(sigmoid_of<T>(x[i]), candidate<T>(u[i]) - s, s);
+            scan_put(static_cast<T*>(g.out) + (int64_t)(p.row_first + t) * g.out_stride + c, s * o[i] * sigmoid_of<T>(o[i]));
             if (t + g.state.ring >= p.n_rows) state_at(g, rd.seq, pos0 + t)[c] = s;
         }
     }
 }
 
-template <typename T, int CH, int RUN>
-__global__ void __launch_bounds__(CH * RUNS) scan_kernel(const __grid_constant__ GatedScan g, const __grid_constant__ RowTiles portions, uint32_t* __restrict__ err) {
-    __shared__ float2 step[RUNS][CH + 1];
-    __shared__ float before[RUNS][CH + 1], carry[CH];
-    const int ch = threadIdx.x % CH, run = threadIdx.x / CH, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int c = blockIdx.x * CH + ch;
-    const AttnTile p = row_tile(portions, blockIdx.y);
-    const tsb_row_desc rd = g.rows[p.row_first];
-    const int pos0 = rd.base + rd.slot;
-    const bool ok = rd.seq >= 0 && rd.seq < g.state.n_streams, in = ok && c < g.width;
-    if (!ok && threadIdx.x == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
-    if (run == 0) carry[ch] = in && pos0 > 0 ? state_at(g, rd.seq, pos0 - 1)[c] : 0.f;
-    pdl_wait();
-    pdl_launch_dependents();
-    if (!ok) return;
-    for (int b0 = 0; b0 < p.n_rows; b0 += RUNS * RUN) {
-        const int t0 = b0 + run * RUN, n = in ? min(RUN, p.n_rows - t0) : 0;  // may be negative
-        const int64_t row0 = p.row_first + t0;
-        float z[RUN], x[RUN], o[RUN];
+// The gates of a thread's run, and the run as one step.
+template <int RUN>
+struct Run {
+    float z[RUN], x[RUN];  // pre-activations, then z and c
+    int n;                 // rows of the run that are there (may be negative)
+    __device__ __forceinline__ void load(const GatedScan& g, int64_t row0, int c, int rows) {
+        n = rows;
 #pragma unroll
         for (int i = 0; i < RUN; i++) {
-            z[i] = x[i] = o[i] = 0.f;
+            z[i] = x[i] = 0.f;
             if (i < n) {
                 const float* gate = g.gate + (row0 + i) * g.gate_stride + c;
                 z[i] = gate[0], x[i] = gate[g.width];
-                o[i] = rec_get(static_cast<const T*>(g.out_gate) + (row0 + i) * g.out_gate_stride + c);
             }
         }
+    }
+    template <typename T>
+    __device__ __forceinline__ float2 step() {
         float a = 1.f, b = 0.f;
 #pragma unroll
         for (int i = 0; i < RUN; i++) {
             if (i >= n) continue;
-            const float left = rec_sigmoid(-z[i]);
-            z[i] = rec_sigmoid(z[i]), x[i] = candidate(x[i]);
-            a *= left, b = fmaf(z[i], x[i] - b, b);
+            z[i] = sigmoid_of<T>(z[i]), x[i] = candidate<T>(x[i]);
+            a = fmaf(-z[i], a, a), b = fmaf(z[i], x[i] - b, b);
         }
-        step[run][ch] = make_float2(a, b);
-        __syncthreads();
-        {
-            // warp = channel, lane = run: steps composed with all that come before
-            float2 s = step[lane][warp];
+        return make_float2(a, b);
+    }
+};
+// steps of the lanes composed with all that come before them
+__device__ __forceinline__ float2 compose_before(float2 s, int lane) {
 #pragma unroll
-            for (int d = 1; d < 32; d <<= 1) {
-                const float pa = __shfl_up_sync(0xffffffffu, s.x, d), pb = __shfl_up_sync(0xffffffffu, s.y, d);
-                if (lane >= d) s.y = fmaf(s.x, pb, s.y), s.x *= pa;
-            }
-            const float start = carry[warp], end = fmaf(s.x, start, s.y), prev = __shfl_up_sync(0xffffffffu, end, 1);
-            before[lane][warp] = lane == 0 ? start : prev;
-            __syncwarp();
-            if (lane == 31) carry[warp] = end;
-        }
-        __syncthreads();
-        float s = before[run][ch];
+    for (int d = 1; d < 32; d <<= 1) {
+        const float pa = __shfl_up_sync(0xffffffffu, s.x, d), pb = __shfl_up_sync(0xffffffffu, s.y, d);
+        if (lane >= d) s.y = fmaf(s.x, pb, s.y), s.x *= pa;
+    }
+    return s;
+}
+constexpr int RUN = SCAN_CHUNK / RUNS;
+
+// What comes before a chunk, as steps: sums[chunk][channel] is the chunk before it as one step, and for a portion's first chunk the state before the portion (which
+// the second launch, whose CTAs write states, could not read).
+template <typename T, int CH>
+__global__ void __launch_bounds__(CH * RUNS) scan_sums_kernel(const __grid_constant__ GatedScan g, const __grid_constant__ RowTiles chunks, float2* __restrict__ sums) {
+    __shared__ float2 step[RUNS][CH + 1];
+    const int ch = threadIdx.x % CH, run = threadIdx.x / CH, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int c = blockIdx.x * CH + ch;
+    const AttnTile p = row_tile(chunks, blockIdx.y);
+    const int next = p.row_first + p.n_rows;
+    const bool last = next >= g.n_rows || g.rows[next].slot == 0;
+    const tsb_row_desc rd = g.rows[p.row_first];
+    const bool ok = rd.seq >= 0 && rd.seq < g.state.n_streams;
+    float2* out = sums + (int64_t)blockIdx.y * g.width;
+    pdl_wait();
+    pdl_launch_dependents();
+    if (!ok) return;  // the second launch tells
+    if (rd.slot == 0 && run == 0 && c < g.width) out[c] = make_float2(0.f, rd.base > 0 ? state_at(g, rd.seq, rd.base - 1)[c] : 0.f);
+    if (last) return;
+    Run<RUN> r;
+    r.load(g, p.row_first + run * RUN, c, c < g.width ? RUN : 0);
+    step[run][ch] = r.step<T>();
+    __syncthreads();
+    const float2 s = compose_before(step[lane][warp], lane);
+    if (lane == 31 && blockIdx.x * CH + warp < g.width) out[g.width + blockIdx.x * CH + warp] = s;
+}
+
+template <typename T, int CH>
+__global__ void __launch_bounds__(CH * RUNS) scan_chunks_kernel(const __grid_constant__ GatedScan g, const __grid_constant__ RowTiles chunks, const float2* __restrict__ sums,
+                                                               uint32_t* __restrict__ err) {
+    __shared__ float2 step[RUNS][CH + 1];
+    __shared__ float before[RUNS][CH + 1];
+    const int ch = threadIdx.x % CH, run = threadIdx.x / CH, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int c = blockIdx.x * CH + ch, wc = blockIdx.x * CH + warp;  // the thread's channel, and the one its warp scans
+    const AttnTile p = row_tile(chunks, blockIdx.y);
+    const tsb_row_desc rd = g.rows[p.row_first];
+    const int pos0 = rd.base + rd.slot, n_before = rd.slot / SCAN_CHUNK;  // chunks of the portion before this one
+    const bool ok = rd.seq >= 0 && rd.seq < g.state.n_streams && n_before <= (int)blockIdx.y;
+    if (!ok && threadIdx.x == 0) atomicCAS(err, 0u, (uint32_t)TSB_DEV_BAD_INDEX);
+    const float carry = ok && !sums && wc < g.width && rd.base > 0 ? state_at(g, rd.seq, rd.base - 1)[wc] : 0.f;  // the portion is one chunk
+    pdl_wait();
+    pdl_launch_dependents();
+    if (!ok) return;
+    const int64_t row0 = p.row_first + run * RUN;
+    Run<RUN> r;
+    r.load(g, row0, c, c < g.width ? p.n_rows - run * RUN : 0);
+    float o[RUN];
 #pragma unroll
-        for (int i = 0; i < RUN; i++) {
-            if (i >= n) continue;
-            s = fmaf(z[i], x[i] - s, s);
-            scan_put(static_cast<T*>(g.out) + (row0 + i) * g.out_stride + c, s * rec_silu(o[i]));
-            if (t0 + i + g.state.ring >= p.n_rows) state_at(g, rd.seq, pos0 + t0 + i)[c] = s;
-        }
+    for (int i = 0; i < RUN; i++) o[i] = i < r.n ? rec_get(static_cast<const T*>(g.out_gate) + (row0 + i) * g.out_gate_stride + c) : 0.f;
+    // what comes before, 32 steps at a time
+    float start = carry;
+    for (int k0 = 0; sums && k0 <= n_before; k0 += 32) {
+        float2 s = make_float2(1.f, 0.f);
+        if (k0 + lane <= n_before && wc < g.width) s = __ldcg(sums + (int64_t)(blockIdx.y - n_before + k0 + lane) * g.width + wc);
+        s = compose_before(s, lane);
+        start = __shfl_sync(0xffffffffu, fmaf(s.x, start, s.y), 31);
+    }
+    step[run][ch] = r.step<T>();
+    __syncthreads();
+    {
+        const float2 s = compose_before(step[lane][warp], lane);
+        const float end = fmaf(s.x, start, s.y), prev = __shfl_up_sync(0xffffffffu, end, 1);
+        before[lane][warp] = lane == 0 ? start : prev;
+    }
+    __syncthreads();
+    float s = before[run][ch];
+#pragma unroll
+    for (int i = 0; i < RUN; i++) {
+        if (i >= r.n) continue;
+        const int row = (int)row0 + i, after = row + g.state.ring;
+        s = fmaf(r.z[i], r.x[i] - s, s);
+        scan_put(static_cast<T*>(g.out) + (row0 + i) * g.out_stride + c, s * o[i] * sigmoid_of<T>(o[i]));
+        if (after >= g.n_rows || g.rows[after].seq != rd.seq) state_at(g, rd.seq, pos0 + run * RUN + i)[c] = s;  // one of the portion's last rows
     }
 }
 
-template <typename T>
-cudaError_t launch_of(tsb_ctx* ctx, cudaStream_t st, const GatedScan& g, const RowTiles& portions) {
-    if (portions.longest < SCAN_MIN_ROWS)
-        return tsb_launch(ctx, scan_rows_kernel<T>, dim3((unsigned)((g.width + ROWS_THREADS - 1) / ROWS_THREADS), (unsigned)portions.n), dim3(ROWS_THREADS), 0, st, true, g, portions,
-                          ctx->dev_error);
-    auto run = [&](auto kernel, int ch) {
-        return tsb_launch(ctx, kernel, dim3((unsigned)((g.width + ch - 1) / ch), (unsigned)portions.n), dim3(ch * RUNS), 0, st, true, g, portions, ctx->dev_error);
-    };
-    // fewer channels per CTA where whole sectors of them would leave SMs idle
-    const int64_t ctas = (int64_t)portions.n * ((g.width + 15) / 16);
-    return ctas < ctx->sm_count ? run(scan_kernel<T, 8, 4>, 8) : run(scan_kernel<T, 16, 4>, 16);
+template <typename T, int CH>
+cudaError_t launch_chunks(tsb_ctx* ctx, cudaStream_t st, const GatedScan& g, const RowTiles& chunks, bool several, float2* sums) {
+    const dim3 grid((unsigned)((g.width + CH - 1) / CH), (unsigned)chunks.n);
+    if (several)
+        if (cudaError_t e = tsb_launch(ctx, scan_sums_kernel<T, CH>, grid, dim3(CH * RUNS), 0, st, true, g, chunks, sums); e != cudaSuccess) return e;
+    return tsb_launch(ctx, scan_chunks_kernel<T, CH>, grid, dim3(CH * RUNS), 0, st, true, g, chunks, (const float2*)(several ? sums : nullptr), ctx->dev_error);
 }
 
 }  // namespace
 
-cudaError_t launch_gated_scan(tsb_ctx* ctx, cudaStream_t st, bool f32, const GatedScan& g, const RowTiles& portions) {
+cudaError_t launch_gated_scan_rows(tsb_ctx* ctx, cudaStream_t st, bool f32, const GatedScan& g, const RowTiles& portions) {
     if (portions.n == 0) return cudaSuccess;
-    return f32 ? launch_of<float>(ctx, st, g, portions) : launch_of<__nv_bfloat16>(ctx, st, g, portions);
+    auto run = [&](auto kernel) {
+        return tsb_launch(ctx, kernel, dim3((unsigned)((g.width + ROWS_THREADS - 1) / ROWS_THREADS), (unsigned)portions.n), dim3(ROWS_THREADS), 0, st, true, g, portions, ctx->dev_error);
+    };
+    return f32 ? run(scan_rows_kernel<float>) : run(scan_rows_kernel<__nv_bfloat16>);
+}
+
+cudaError_t launch_gated_scan_chunks(tsb_ctx* ctx, cudaStream_t st, bool f32, const GatedScan& g, const RowTiles& chunks, bool several, float2* sums) {
+    if (chunks.n == 0) return cudaSuccess;
+    return f32 ? launch_chunks<float, 16>(ctx, st, g, chunks, several, sums) : launch_chunks<__nv_bfloat16, 16>(ctx, st, g, chunks, several, sums);
 }

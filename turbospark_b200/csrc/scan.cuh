@@ -14,8 +14,11 @@ struct GatedScan {
     int width = 0;
     RecurrentState state{};
     const tsb_row_desc* rows = nullptr;
+    int n_rows = 0;                   // of the pass
 };
-// Whole portions of streams; the state after each of a portion's last `ring` rows is kept.  `longest` of the tiles chooses the kernel: channels that walk
-// their rows, or (from SCAN_MIN_ROWS rows on) runs of rows side by side.
-constexpr int SCAN_MIN_ROWS = 32;
-cudaError_t launch_gated_scan(tsb_ctx* ctx, cudaStream_t st, bool f32, const GatedScan& g, const RowTiles& portions);
+// Whole portions of streams, row by row; the state after each of a portion's last `ring` rows is kept.
+cudaError_t launch_gated_scan_rows(tsb_ctx* ctx, cudaStream_t st, bool f32, const GatedScan& g, const RowTiles& portions);
+// Long portions by chunks of SCAN_CHUNK rows (a portion's last one may be shorter), a portion's chunks one after another in the list.  several: some portion
+// has more than one; sums: [chunks][width] then.
+constexpr int SCAN_CHUNK = 128;
+cudaError_t launch_gated_scan_chunks(tsb_ctx* ctx, cudaStream_t st, bool f32, const GatedScan& g, const RowTiles& chunks, bool several, float2* sums);

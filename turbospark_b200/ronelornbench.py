@@ -53,12 +53,13 @@ def scan(ctx, peaks, name, width, rows, streams, iters):
     gate = [ctx.to_device(np.random.default_rng(i).standard_normal(n * 2 * width).astype(np.float32)) for i in range(copies)]
     g, out = random_bf16(ctx, copies * n * width, 1, amp=2.0), ctx.alloc(copies * n * width * 2)
     state, rd = ctx.zeroed(streams * 2 * width * 4), latentbench._rows(ctx, 0 if rows >= 64 else 4096, rows, streams)
+    sums = ctx.zeroed(streams * (rows // 128 + 1) * width * 8)
 
     def call(i, s):
         at = (i % copies) * n * width * 2
-        ctx.gated_scan_rows(BF16, gate[i % copies], 2 * width, C.c_void_p(g.ptr + at), width, width, state, streams, 2, rd, n, rows, C.c_void_p(out.ptr + at), width, stream=s)
+        ctx.gated_scan_rows(BF16, gate[i % copies], 2 * width, C.c_void_p(g.ptr + at), width, width, state, streams, 2, rd, n, rows, C.c_void_p(out.ptr + at), width, chunked=rows >= 64, sums=sums, stream=s)
     ms = time_graph(call, iters)
-    for b in gate + [g, out, state, rd]:
+    for b in gate + [g, out, state, rd, sums]:
         b.free()
     return dict(peaks.entry(name, ms, n * width * 12.0 + streams * width * 8.0), rows=rows, streams=streams, width=width)
 
