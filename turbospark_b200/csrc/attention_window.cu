@@ -15,7 +15,7 @@
 // Only the key tiles inside the window of some query of the tile are visited; key tiles start at multiples of 64 positions
 // whatever the cut of the prompt, so a row meets its keys in the same grouping in every schedule.
 //
-// Score arithmetic in f32, base 2: v = cap log2(e) tanh(s scale / cap) - r1 log2(1 + r2 d); tanh by its series where every
+// Score arithmetic in f32, base 2: v = cap log2(e) tanh(s scale / cap) - r1 log2(1 + r2 d); tanh by a polynomial where every
 // score of the warp's tile is well inside the cap.
 //
 // f32: one warp per (row, query head), lanes over keys for the scores and over columns for the sum; the reference-precision

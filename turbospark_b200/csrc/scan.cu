@@ -18,14 +18,18 @@ constexpr int RUNS = 32;  // of a chunk: the lanes of the warp that scans a chan
 
 __device__ __forceinline__ void scan_put(float* p, float v) { *p = v; }
 __device__ __forceinline__ void scan_put(__nv_bfloat16* p, float v) { *p = __float2bfloat16_rn(v); }
-// 1 / (1 + e^-x): with bfloat16 outputs by the fast exponential and division (relative error a few 2^-22), in the f32 mode by the library's.
+// 1 / (1 + e^-x): with bfloat16 outputs by the hardware's exponential and reciprocal (relative error a few 2^-22), in the f32 mode by the library's.
 template <typename T>
 __device__ __forceinline__ float sigmoid_of(float x) {
-    return sizeof(T) == 4 ? rec_sigmoid(x) : __fdividef(1.f, 1.f + __expf(-x));
+    if (sizeof(T) == 4) return rec_sigmoid(x);
+    float e, y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(x * -1.4426950408889634f));
+    asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(1.f + e));
+    return y;
 }
 template <typename T>
 __device__ __forceinline__ float candidate(float u) {
-    const float low = sigmoid_of<T>(fminf(u, 0.f));
+    const float low = sigmoid_of<T>(u);
     return u >= 0.f ? u + 0.5f : low;
 }
 
@@ -72,13 +76,11 @@ struct Run {
     int n;                 // rows of the run that are there (may be negative)
     __device__ __forceinline__ void load(const GatedScan& g, int64_t row0, int c, int rows) {
         n = rows;
+        const float* gate = g.gate + row0 * g.gate_stride + c;
 #pragma unroll
-        for (int i = 0; i < RUN; i++) {
+        for (int i = 0; i < RUN; i++, gate += g.gate_stride) {
             z[i] = x[i] = 0.f;
-            if (i < n) {
-                const float* gate = g.gate + (row0 + i) * g.gate_stride + c;
-                z[i] = gate[0], x[i] = gate[g.width];
-            }
+            if (i < n) z[i] = gate[0], x[i] = gate[g.width];
         }
     }
     template <typename T>
@@ -150,8 +152,9 @@ __global__ void __launch_bounds__(CH * RUNS) scan_chunks_kernel(const __grid_con
     Run<RUN> r;
     r.load(g, row0, c, c < g.width ? p.n_rows - run * RUN : 0);
     float o[RUN];
+    const T* gate = static_cast<const T*>(g.out_gate) + row0 * g.out_gate_stride + c;
 #pragma unroll
-    for (int i = 0; i < RUN; i++) o[i] = i < r.n ? rec_get(static_cast<const T*>(g.out_gate) + (row0 + i) * g.out_gate_stride + c) : 0.f;
+    for (int i = 0; i < RUN; i++, gate += g.out_gate_stride) o[i] = i < r.n ? rec_get(gate) : 0.f;
     // what comes before, 32 steps at a time
     float start = carry;
     for (int k0 = 0; sums && k0 <= n_before; k0 += 32) {
@@ -169,14 +172,19 @@ __global__ void __launch_bounds__(CH * RUNS) scan_chunks_kernel(const __grid_con
     }
     __syncthreads();
     float s = before[run][ch];
+    T* out = static_cast<T*>(g.out) + row0 * g.out_stride + c;
 #pragma unroll
-    for (int i = 0; i < RUN; i++) {
+    for (int i = 0; i < RUN; i++, out += g.out_stride) {
         if (i >= r.n) continue;
-        const int row = (int)row0 + i, after = row + g.state.ring;
         s = fmaf(r.z[i], r.x[i] - s, s);
-        scan_put(static_cast<T*>(g.out) + (row0 + i) * g.out_stride + c, s * o[i] * sigmoid_of<T>(o[i]));
-        if (after >= g.n_rows || g.rows[after].seq != rd.seq) state_at(g, rd.seq, pos0 + run * RUN + i)[c] = s;  // one of the portion's last rows
+        r.x[i] = s;
+        scan_put(out, s * o[i] * sigmoid_of<T>(o[i]));
     }
+    auto kept = [&](int row) { return row + g.state.ring >= g.n_rows || g.rows[row + g.state.ring].seq != rd.seq; };  // one of the portion's last rows
+    if (!kept(p.row_first + p.n_rows - 1)) return;
+#pragma unroll
+    for (int i = 0; i < RUN; i++)
+        if (i < r.n && kept((int)row0 + i)) state_at(g, rd.seq, pos0 + run * RUN + i)[c] = r.x[i];
 }
 
 template <typename T, int CH>
